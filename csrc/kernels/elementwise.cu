@@ -503,6 +503,20 @@ RB_API int rb_dropout(const void* a, void* out, unsigned char* mask_out, long lo
   RB_BY_DTYPE((rb::dropout_kernel<float><<<grid, 256, 0, RB_STREAM>>>((const float*)a, (float*)out, mask_out, n, p, seed, offset, rng)),
               (rb::dropout_kernel<__nv_bfloat16><<<grid, 256, 0, RB_STREAM>>>((const __nv_bfloat16*)a, (__nv_bfloat16*)out, mask_out, n, p, seed, offset, rng)))
 }
+namespace rb {
+__global__ void __launch_bounds__(256) scale_softcap_kernel(float* __restrict__ x, long long n, float scale, float cap) {
+  const long long stride = static_cast<long long>(gridDim.x) * blockDim.x;
+  for (long long i = static_cast<long long>(blockIdx.x) * blockDim.x + threadIdx.x; i < n; i += stride) {
+    const float v = x[i] * scale;
+    x[i] = cap > 0.f ? cap * tanhf(v / cap) : v;
+  }
+}
+}  // namespace rb
+RB_API int rb_scale_softcap(float* x, long long n, float scale, float cap, void* stream_v) {
+  if (n <= 0) return 0;
+  rb::scale_softcap_kernel<<<rb::ew_grid(n), 256, 0, RB_STREAM>>>(x, n, scale, cap);
+  return static_cast<int>(cudaGetLastError());
+}
 RB_API int rb_argmax_rows(const void* a, long long lda, long long* out, long long rows, int cols, int dtype, void* stream_v) {
   if (rows <= 0 || cols <= 0) return 0;
   RB_BY_DTYPE((rb::argmax_rows_kernel<float><<<static_cast<int>(rows), 128, 0, RB_STREAM>>>((const float*)a, lda, out, cols)),

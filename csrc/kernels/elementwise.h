@@ -41,6 +41,8 @@ int rb_apply_mask(const void* a, const void* mask, float mask_value, void* out, 
 // (the generator of the reference's WGSL dropout, shaders.wgsl:1238-1281).  mask_out (uint8, optional) gets the keep mask.
 int rb_dropout(const void* a, void* out, unsigned char* mask_out, long long n, float p, unsigned long long seed,
                unsigned long long offset, int rng, int dtype, void* stream);
+// fp32 in place: x <- cap * tanh(scale * x / cap), or x <- scale * x when cap <= 0 (output logits)
+int rb_scale_softcap(float* x, long long n, float scale, float cap, void* stream);
 // out[r] = argmax_c a[r, c]
 int rb_argmax_rows(const void* a, long long lda, long long* out, long long rows, int cols, int dtype, void* stream);
 #ifdef __cplusplus

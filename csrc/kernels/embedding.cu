@@ -149,6 +149,43 @@ pos_grad_kernel(const __nv_bfloat16* __restrict__ dy, float* __restrict__ dwpe, 
 
 }  // namespace rb
 
+namespace rb {
+template <typename T>
+__global__ void __launch_bounds__(128)
+embedding_residual_kernel(const long long* __restrict__ ids, const T* __restrict__ table, float* __restrict__ x,
+                          T* __restrict__ h, long long tokens, int dim, long long vocab RB_BOUNDS_PARAM) {
+  const long long total = tokens * dim;
+  const long long stride = static_cast<long long>(gridDim.x) * blockDim.x;
+  for (long long i = static_cast<long long>(blockIdx.x) * blockDim.x + threadIdx.x; i < total; i += stride) {
+    const long long t = i / dim;
+    const int c = static_cast<int>(i - t * dim);
+    long long id = ids[t];
+    if (id < 0 || id >= vocab) {         // out-of-range ids read row 0 instead of faulting
+      if (c == 0) RB_BOUNDS_HIT(101);
+      id = 0;
+    }
+    const T v = table[id * dim + c];
+    x[i] = static_cast<float>(v);
+    if (h) h[i] = v;
+  }
+}
+}  // namespace rb
+
+RB_API int rb_embedding_residual(const long long* ids, const void* table, int table_f32, float* x, void* h, long long tokens,
+                                 int dim, long long vocab, void* stream_v) {
+  if (tokens <= 0 || dim <= 0 || vocab <= 0) return -1;
+  cudaStream_t stream = reinterpret_cast<cudaStream_t>(stream_v);
+  long long blocks = (tokens * dim + 127) / 128;
+  if (blocks > 148LL * 32) blocks = 148LL * 32;
+  if (table_f32)
+    rb::embedding_residual_kernel<float><<<static_cast<int>(blocks), 128, 0, stream>>>(
+        ids, reinterpret_cast<const float*>(table), x, reinterpret_cast<float*>(h), tokens, dim, vocab RB_BOUNDS_ARG);
+  else
+    rb::embedding_residual_kernel<__nv_bfloat16><<<static_cast<int>(blocks), 128, 0, stream>>>(
+        ids, reinterpret_cast<const __nv_bfloat16*>(table), x, reinterpret_cast<__nv_bfloat16*>(h), tokens, dim, vocab RB_BOUNDS_ARG);
+  return static_cast<int>(cudaGetLastError());
+}
+
 RB_API int rb_embedding_fwd(const long long* ids, const void* wte, const void* wpe, void* out, long long tokens,
                             int dim, int seq_len, long long vocab, void* stream_v) {
   if (tokens <= 0 || dim <= 0 || (dim & 7) || vocab <= 0 || (wpe && seq_len <= 0)) return -1;

@@ -1,0 +1,187 @@
+// Per-head work between the packed attention projection and the attention kernels, in one pass: RMS norm of every query
+// and key head, mixing of the values with an earlier layer's values of the same token, and the append of keys and values
+// to their cache slots.  Norms and mixing are fp32.  A group of 16 lanes owns one head of one token with 16-byte accesses;
+// head sizes that are not whole vectors take the scalar form (one warp per head).
+#include "head_prep.h"
+
+#include "rb_common.cuh"
+
+namespace rb {
+
+constexpr int kHpMaxVec = 4;                       // vectors per lane: head sizes up to 512 (bf16) / 256 (fp32)
+
+template <typename T> struct HpVec;
+template <> struct HpVec<__nv_bfloat16> {
+  static constexpr int N = 8;
+  static __device__ __forceinline__ void load(const __nv_bfloat16* p, float (&v)[8]) {
+    const uint4 u = *reinterpret_cast<const uint4*>(p);
+    const uint32_t w[4] = {u.x, u.y, u.z, u.w};
+#pragma unroll
+    for (int i = 0; i < 4; ++i) { const float2 f = unpack_bf16x2(w[i]); v[2 * i] = f.x; v[2 * i + 1] = f.y; }
+  }
+  static __device__ __forceinline__ void store(__nv_bfloat16* p, const float (&v)[8]) {
+    *reinterpret_cast<uint4*>(p) = make_uint4(pack_bf16x2(v[0], v[1]), pack_bf16x2(v[2], v[3]), pack_bf16x2(v[4], v[5]),
+                                              pack_bf16x2(v[6], v[7]));
+  }
+};
+template <> struct HpVec<float> {
+  static constexpr int N = 4;
+  static __device__ __forceinline__ void load(const float* p, float (&v)[4]) {
+    const float4 u = *reinterpret_cast<const float4*>(p);
+    v[0] = u.x; v[1] = u.y; v[2] = u.z; v[3] = u.w;
+  }
+  static __device__ __forceinline__ void store(float* p, const float (&v)[4]) {
+    *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]);
+  }
+};
+__device__ __forceinline__ float hp_get(const __nv_bfloat16* p) { return __bfloat162float(*p); }
+__device__ __forceinline__ float hp_get(const float* p) { return *p; }
+__device__ __forceinline__ void hp_put(__nv_bfloat16* p, float v) { *p = __float2bfloat16(v); }
+__device__ __forceinline__ void hp_put(float* p, float v) { *p = v; }
+
+struct HpItem {
+  int kind, head;                                  // 0 query, 1 key, 2 value
+};
+__device__ __forceinline__ HpItem hp_item(int i, const RbHeadPrepArgs& a) {
+  if (i < a.heads) return {0, i};
+  i -= a.heads;
+  if (i < a.kv_heads) return {1, i};
+  return {2, i - a.kv_heads};
+}
+
+template <typename T>
+__global__ void __launch_bounds__(128)
+head_prep_kernel(const RbHeadPrepArgs a RB_BOUNDS_PARAM) {
+  using V = HpVec<T>;
+  constexpr int LANES = 16;
+  const int sub = threadIdx.x & (LANES - 1);
+  const int items = a.heads + 2 * a.kv_heads;
+  const long long total = a.tokens * items;
+  const long long per_grid = static_cast<long long>(gridDim.x) * (blockDim.x / LANES);
+  const long long rounds = (total + per_grid - 1) / per_grid;
+  long long g = static_cast<long long>(blockIdx.x) * (blockDim.x / LANES) + threadIdx.x / LANES;
+  for (long long r = 0; r < rounds; ++r, g += per_grid) {
+    const bool live = g < total;                   // idle groups stay in the loop: the shuffles below are warp-wide
+    const long long t = live ? g / items : 0;
+    const HpItem it = hp_item(static_cast<int>(live ? g - t * items : 0), a);
+    const int dim = it.kind == 2 ? a.dv : a.dk;
+    const long long off = it.kind == 0 ? a.off_q : it.kind == 1 ? a.off_k : a.off_v;
+    T* row = reinterpret_cast<T*>(a.p) + t * a.ld + off + static_cast<long long>(it.head) * dim;
+    float v[kHpMaxVec][V::N];
+    float sq = 0.f;
+#pragma unroll
+    for (int c = 0; c < kHpMaxVec; ++c) {
+      const int col = (c * LANES + sub) * V::N;
+      if (live && col < dim) {
+        V::load(row + col, v[c]);
+#pragma unroll
+        for (int i = 0; i < V::N; ++i) sq += v[c][i] * v[c][i];
+      }
+    }
+#pragma unroll
+    for (int o = LANES / 2; o > 0; o >>= 1) sq += __shfl_xor_sync(0xffffffffu, sq, o);
+    if (!live) continue;
+    const T* gamma = reinterpret_cast<const T*>(it.kind == 0 ? a.q_gamma : it.kind == 1 ? a.k_gamma : nullptr);
+    const bool mixed = it.kind == 2 && a.v_first != nullptr;
+    const float rstd = gamma ? rsqrtf(sq / static_cast<float>(dim) + a.eps) : 1.f;
+    const float lam = mixed ? a.mix[0] : 0.f;
+    const T* first = mixed ? reinterpret_cast<const T*>(a.v_first) + t * a.ld_vf + static_cast<long long>(it.head) * dim : nullptr;
+    T* cache = nullptr;
+    if (it.kind != 0 && a.k_cache) {
+      const long long slot = a.slots[t];
+      if (slot >= a.num_slots && sub == 0) RB_BOUNDS_HIT(103);       // a negative slot means "skip this token"
+      if (slot >= 0 && slot < a.num_slots)
+        cache = reinterpret_cast<T*>(it.kind == 1 ? a.k_cache : a.v_cache) + (slot * a.kv_heads + it.head) * dim;
+    }
+#pragma unroll
+    for (int c = 0; c < kHpMaxVec; ++c) {
+      const int col = (c * LANES + sub) * V::N;
+      if (col >= dim) continue;
+      if (gamma) {
+        float w[V::N];
+        V::load(gamma + col, w);
+#pragma unroll
+        for (int i = 0; i < V::N; ++i) v[c][i] = v[c][i] * rstd * w[i];
+      }
+      if (mixed) {
+        float w[V::N];
+        V::load(first + col, w);
+#pragma unroll
+        for (int i = 0; i < V::N; ++i) v[c][i] = (1.f - lam) * v[c][i] + lam * w[i];
+      }
+      if (gamma || mixed) V::store(row + col, v[c]);
+      if (cache) V::store(cache + col, v[c]);
+    }
+  }
+}
+
+// any head size and alignment: one warp per head, element by element
+template <typename T>
+__global__ void __launch_bounds__(128)
+head_prep_scalar_kernel(const RbHeadPrepArgs a RB_BOUNDS_PARAM) {
+  const int lane = threadIdx.x & 31;
+  const int items = a.heads + 2 * a.kv_heads;
+  const long long total = a.tokens * items;
+  const long long stride = static_cast<long long>(gridDim.x) * (blockDim.x >> 5);
+  for (long long g = static_cast<long long>(blockIdx.x) * (blockDim.x >> 5) + (threadIdx.x >> 5); g < total; g += stride) {
+    const long long t = g / items;
+    const HpItem it = hp_item(static_cast<int>(g - t * items), a);
+    const int dim = it.kind == 2 ? a.dv : a.dk;
+    const long long off = it.kind == 0 ? a.off_q : it.kind == 1 ? a.off_k : a.off_v;
+    T* row = reinterpret_cast<T*>(a.p) + t * a.ld + off + static_cast<long long>(it.head) * dim;
+    const T* gamma = reinterpret_cast<const T*>(it.kind == 0 ? a.q_gamma : it.kind == 1 ? a.k_gamma : nullptr);
+    float rstd = 1.f;
+    if (gamma) {
+      float sq = 0.f;
+      for (int c = lane; c < dim; c += 32) { const float x = hp_get(row + c); sq += x * x; }
+      rstd = rsqrtf(warp_sum(sq) / static_cast<float>(dim) + a.eps);
+    }
+    const bool mixed = it.kind == 2 && a.v_first != nullptr;
+    const float lam = mixed ? a.mix[0] : 0.f;
+    T* cache = nullptr;
+    if (it.kind != 0 && a.k_cache) {
+      const long long slot = a.slots[t];
+      if (slot >= a.num_slots && lane == 0) RB_BOUNDS_HIT(103);
+      if (slot >= 0 && slot < a.num_slots)
+        cache = reinterpret_cast<T*>(it.kind == 1 ? a.k_cache : a.v_cache) + (slot * a.kv_heads + it.head) * dim;
+    }
+    for (int c = lane; c < dim; c += 32) {
+      float x = hp_get(row + c);
+      if (gamma) x = x * rstd * hp_get(gamma + c);
+      if (mixed) x = (1.f - lam) * x + lam * hp_get(reinterpret_cast<const T*>(a.v_first) + t * a.ld_vf +
+                                                    static_cast<long long>(it.head) * dim + c);
+      hp_put(row + c, x);
+      if (cache) hp_put(cache + c, x);
+    }
+  }
+}
+
+template <typename T>
+int hp_launch(const RbHeadPrepArgs& a, cudaStream_t s) {
+  constexpr int N = HpVec<T>::N;
+  const uintptr_t bits = reinterpret_cast<uintptr_t>(a.p) | reinterpret_cast<uintptr_t>(a.q_gamma) |
+                         reinterpret_cast<uintptr_t>(a.k_gamma) | reinterpret_cast<uintptr_t>(a.v_first) |
+                         reinterpret_cast<uintptr_t>(a.k_cache) | reinterpret_cast<uintptr_t>(a.v_cache);
+  const bool vec = !(bits & 15) && !((a.ld | a.off_q | a.off_k | a.off_v | a.dk | a.dv | (a.v_first ? a.ld_vf : 0)) % N) &&
+                   a.dk <= 16 * N * kHpMaxVec && a.dv <= 16 * N * kHpMaxVec;
+  const long long total = a.tokens * (a.heads + 2 * a.kv_heads);
+  const int per_block = vec ? 8 : 4;
+  long long blocks = (total + per_block - 1) / per_block;
+  if (blocks > 148LL * 16) blocks = 148LL * 16;
+  if (vec)
+    head_prep_kernel<T><<<static_cast<int>(blocks), 128, 0, s>>>(a RB_BOUNDS_ARG);
+  else
+    head_prep_scalar_kernel<T><<<static_cast<int>(blocks), 128, 0, s>>>(a RB_BOUNDS_ARG);
+  return static_cast<int>(cudaGetLastError());
+}
+
+}  // namespace rb
+
+RB_API int rb_head_prep(const RbHeadPrepArgs* args, void* stream_v) {
+  const RbHeadPrepArgs& a = *args;
+  if (a.tokens <= 0) return 0;
+  if (!a.p || a.heads <= 0 || a.kv_heads <= 0 || a.dk <= 0 || a.dv <= 0) return -1;
+  if ((a.k_cache == nullptr) != (a.v_cache == nullptr) || (a.k_cache && !a.slots) || (a.v_first && !a.mix)) return -1;
+  cudaStream_t s = reinterpret_cast<cudaStream_t>(stream_v);
+  return a.f32 ? rb::hp_launch<float>(a, s) : rb::hp_launch<__nv_bfloat16>(a, s);
+}

@@ -1,0 +1,23 @@
+// C interface of the per-head preparation of a packed attention projection (head_prep.cu).
+#pragma once
+#ifdef __cplusplus
+extern "C" {
+#endif
+typedef struct RbHeadPrepArgs {
+  void* p;                    // packed projection [tokens, ld]: query heads at off_q, key heads at off_k, value heads at off_v
+  const void* q_gamma;        // [dk] RMS-norm weight of every query head, or NULL (no norm); type of p
+  const void* k_gamma;        // same for the key heads
+  const void* v_first;        // [tokens, kv_heads * dv] values to mix in (pitch ld_vf), type of p, or NULL
+  const float* mix;           // [1] share of v_first
+  void* k_cache;              // [num_slots, kv_heads, dk] / [num_slots, kv_heads, dv], type of p, or both NULL
+  void* v_cache;
+  const long long* slots;     // cache slot of every token (negative: not stored)
+  long long ld, off_q, off_k, off_v, ld_vf, tokens, num_slots;
+  int f32, heads, kv_heads, dk, dv;
+  float eps;
+} RbHeadPrepArgs;
+// In place: q <- rms(q) * q_gamma, k <- rms(k) * k_gamma, v <- (1 - mix) v + mix v_first; k and v also go to their slots.
+int rb_head_prep(const RbHeadPrepArgs* args, void* stream);
+#ifdef __cplusplus
+}
+#endif

@@ -101,6 +101,105 @@ moe_route_bwd_kernel(const float* __restrict__ probs, const int* __restrict__ id
   if (lane + 32 < E) dlogits[static_cast<long long>(t) * E + lane + 32] = pv1 * (dp[1] - s);
 }
 
+// Router with group-limited choice: one warp per token, scores and group maxima in shared memory.
+__global__ void __launch_bounds__(128)
+moe_route_groups_kernel(const float* __restrict__ logits, int T, int E, int k, int groups, int keep, int renorm, float eps,
+                        int* __restrict__ idx, float* __restrict__ w) {
+  extern __shared__ float route_sm[];
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+  const int t = blockIdx.x * (blockDim.x >> 5) + warp;
+  if (t >= T) return;
+  float* s = route_sm + warp * (E + groups);
+  float* gmax = s + E;
+  const float* x = logits + static_cast<long long>(t) * E;
+  float mx = -INFINITY;
+  for (int e = lane; e < E; e += 32) mx = fmaxf(mx, x[e]);
+  mx = warp_max(mx);
+  float sum = 0.f;
+  for (int e = lane; e < E; e += 32) { const float p = expf(x[e] - mx); s[e] = p; sum += p; }
+  const float inv = 1.f / warp_sum(sum);
+  for (int e = lane; e < E; e += 32) s[e] *= inv;
+  __syncwarp();
+  // arg-max over an array of non-negative values with ties to the lower index (used-up entries are -1)
+  auto pick = [&](const float* v, int n, float& best) {
+    float bv = -2.f;
+    int bi = 0;
+    for (int e = lane; e < n; e += 32)
+      if (v[e] > bv) { bv = v[e]; bi = e; }
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) {
+      const float ov = __shfl_xor_sync(0xffffffffu, bv, o);
+      const int oi = __shfl_xor_sync(0xffffffffu, bi, o);
+      if (ov > bv || (ov == bv && oi < bi)) { bv = ov; bi = oi; }
+    }
+    best = bv;
+    return bi;
+  };
+  float best;
+  if (groups > 1 && keep < groups) {
+    const int per = E / groups;
+    for (int g = lane; g < groups; g += 32) {
+      float m = -1.f;
+      for (int e = g * per; e < (g + 1) * per; ++e) m = fmaxf(m, s[e]);
+      gmax[g] = m;
+    }
+    __syncwarp();
+    for (int j = 0; j < keep; ++j) {                   // kept groups are marked with -2 (below every arg-max candidate)
+      const int g = pick(gmax, groups, best);
+      __syncwarp();
+      if (lane == 0) gmax[g] = -2.f;
+      __syncwarp();
+    }
+    for (int e = lane; e < E; e += 32)
+      if (gmax[e / per] > -1.5f) s[e] = -1.f;
+    __syncwarp();
+  }
+  float tot = 0.f;
+  for (int j = 0; j < k; ++j) {
+    const int e = pick(s, E, best);
+    __syncwarp();
+    if (lane == 0) { s[e] = -1.f; idx[static_cast<long long>(t) * k + j] = e; w[static_cast<long long>(t) * k + j] = best; }
+    tot += best;
+    __syncwarp();
+  }
+  if (renorm) {
+    for (int j = lane; j < k; j += 32) w[static_cast<long long>(t) * k + j] /= tot + eps;
+  }
+}
+
+// silu(gate) * up over the live rows of a permuted expert buffer (the buffer is sized for the worst case; `live` says how
+// many rows the routing used)
+template <typename T, int N>
+__global__ void __launch_bounds__(256)
+swiglu_live_kernel(const T* __restrict__ gu, long long ld_gu, T* __restrict__ h, long long ld_h, int rows, int F,
+                   const int* __restrict__ live) {
+  const int n = live ? min(rows, live[0]) : rows;
+  const int chunks = F / N;
+  const long long total = static_cast<long long>(n) * chunks;
+  const long long stride = static_cast<long long>(gridDim.x) * blockDim.x;
+  for (long long i = static_cast<long long>(blockIdx.x) * blockDim.x + threadIdx.x; i < total; i += stride) {
+    const long long r = i / chunks;
+    const int c = static_cast<int>(i - r * chunks) * N;
+    if (N == 8) {
+      const uint4 g = *reinterpret_cast<const uint4*>(gu + r * ld_gu + c), u = *reinterpret_cast<const uint4*>(gu + r * ld_gu + F + c);
+      const uint32_t gw[4] = {g.x, g.y, g.z, g.w}, uw[4] = {u.x, u.y, u.z, u.w};
+      uint32_t o[4];
+#pragma unroll
+      for (int j = 0; j < 4; ++j) {
+        const float2 a = unpack_bf16x2(gw[j]), b = unpack_bf16x2(uw[j]);
+        o[j] = pack_bf16x2(silu(a.x) * b.x, silu(a.y) * b.y);
+      }
+      *reinterpret_cast<uint4*>(h + r * ld_h + c) = make_uint4(o[0], o[1], o[2], o[3]);
+    } else {
+#pragma unroll
+      for (int j = 0; j < N; ++j) {
+        const float g = static_cast<float>(gu[r * ld_gu + c + j]), u = static_cast<float>(gu[r * ld_gu + F + c + j]);
+        h[r * ld_h + c + j] = static_cast<T>(g / (1.f + expf(-g)) * u);
+      }
+    }
+  }
+}
+
 // ---- permutation plan ---------------------------------------------------------------------------------------
 __device__ __forceinline__ int block_scan_excl(int v, int* sh, int& total) {
   // exclusive scan over 1024 threads; sh has 1024 ints
@@ -262,6 +361,32 @@ inline int grid1d(long long n, int per_block) {
 RB_API int rb_moe_route(const float* logits, int T, int E, int k, int renorm, int* idx, float* w, float* probs_out, void* stream_v) {
   if (T <= 0 || E <= 0 || E > 64 || k <= 0 || k > rb::kMaxK || k > E) return -1;
   rb::moe_route_kernel<<<(T + 3) / 4, 128, 0, RB_ST>>>(logits, T, E, k, renorm, idx, w, probs_out);
+  return static_cast<int>(cudaGetLastError());
+}
+RB_API int rb_moe_route_groups(const float* logits, int T, int E, int k, int groups, int keep, int renorm, float eps,
+                               int* idx, float* w, void* stream_v) {
+  if (groups < 1) groups = 1;
+  if (keep < 1 || keep > groups) keep = groups;
+  if (T <= 0 || E <= 0 || k <= 0 || k > E || E % groups || k > keep * (E / groups)) return -1;
+  const size_t smem = sizeof(float) * 4 * static_cast<size_t>(E + groups);
+  if (smem > 48 * 1024) return -1;
+  rb::moe_route_groups_kernel<<<(T + 3) / 4, 128, smem, RB_ST>>>(logits, T, E, k, groups, keep, renorm, eps, idx, w);
+  return static_cast<int>(cudaGetLastError());
+}
+RB_API int rb_swiglu_live(const void* gu, long long ld_gu, void* h, long long ld_h, int rows, int F, int f32,
+                          const int* live_rows, void* stream_v) {
+  if (rows <= 0 || F <= 0) return -1;
+  const bool vec = !f32 && !((F | ld_gu | ld_h) & 7) && !((reinterpret_cast<uintptr_t>(gu) | reinterpret_cast<uintptr_t>(h)) & 15);
+  const int grid = rb::grid1d(static_cast<long long>(rows) * (vec ? F / 8 : F), 256);
+  if (f32)
+    rb::swiglu_live_kernel<float, 1><<<grid, 256, 0, RB_ST>>>(reinterpret_cast<const float*>(gu), ld_gu, reinterpret_cast<float*>(h),
+                                                             ld_h, rows, F, live_rows);
+  else if (vec)
+    rb::swiglu_live_kernel<__nv_bfloat16, 8><<<grid, 256, 0, RB_ST>>>(reinterpret_cast<const __nv_bfloat16*>(gu), ld_gu,
+                                                                     reinterpret_cast<__nv_bfloat16*>(h), ld_h, rows, F, live_rows);
+  else
+    rb::swiglu_live_kernel<__nv_bfloat16, 1><<<grid, 256, 0, RB_ST>>>(reinterpret_cast<const __nv_bfloat16*>(gu), ld_gu,
+                                                                     reinterpret_cast<__nv_bfloat16*>(h), ld_h, rows, F, live_rows);
   return static_cast<int>(cudaGetLastError());
 }
 RB_API int rb_moe_route_bwd(const float* probs, const int* idx, const float* w, const float* dw, const int* counts, int T,

@@ -14,6 +14,14 @@ int rb_moe_route(const float* logits, int T, int E, int k, int renorm, int* idx,
 // aux_grad_scale multiplies d aux (pass coefficient * upstream gradient).  counts: int32 [E] tokens per expert.
 int rb_moe_route_bwd(const float* probs, const int* idx, const float* w, const float* dw, const int* counts, int T, int E,
                      int k, int renorm, float aux_grad_scale, float* dlogits, void* stream);
+// Grouped-limited router (inference): scores = softmax(logits[T, E]) in fp32; the experts form `groups` equal groups of
+// neighbours, a group counts as its largest score, and only experts of the best `keep` groups can be chosen; the k largest
+// scores are taken (ties to the lower index) and divided by (their sum + eps) when renorm != 0.  groups <= 1: no limit.
+int rb_moe_route_groups(const float* logits, int T, int E, int k, int groups, int keep, int renorm, float eps, int* idx,
+                        float* w, void* stream);
+// h[r, :] = silu(gu[r, 0:F]) * gu[r, F:2F] for the rows r < live_rows[0] (device int32; NULL: all `rows`).  bf16 or fp32.
+int rb_swiglu_live(const void* gu, long long ld_gu, void* h, long long ld_h, int rows, int F, int f32, const int* live_rows,
+                   void* stream);
 // Plan of the permutation: slots s = t * k + j are grouped by expert, in ascending slot order inside an expert
 // (deterministic).  Outputs (all device memory):
 //   counts [E]            tokens per expert

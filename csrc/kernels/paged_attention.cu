@@ -305,7 +305,103 @@ paged_decode_merge_kernel(const float* __restrict__ partial, const int* __restri
   out[static_cast<long long>(b) * ld_o + static_cast<long long>(h) * D + d] = __float2bfloat16(den > 0.f ? num / den : 0.f);
 }
 
+// ---- any rows, any head sizes, bf16 or fp32 ------------------------------------------------------------------------
+__device__ __forceinline__ float pr_get(const __nv_bfloat16* p) { return __bfloat162float(*p); }
+__device__ __forceinline__ float pr_get(const float* p) { return *p; }
+__device__ __forceinline__ void pr_put(__nv_bfloat16* p, float v) { *p = __float2bfloat16(v); }
+__device__ __forceinline__ void pr_put(float* p, float v) { *p = v; }
+
+constexpr int kPrMaxV = 16;                // value columns per lane: dv <= 512
+
+// One warp per (row, query head): lanes are keys for the scores, value columns for the weighted sum.
+template <typename T>
+__global__ void __launch_bounds__(128)
+paged_rows_kernel(const RbPagedRowsArgs a RB_BOUNDS_PARAM) {
+  extern __shared__ float pr_q[];
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+  const long long item = static_cast<long long>(blockIdx.x) * (blockDim.x >> 5) + warp;
+  if (item >= static_cast<long long>(a.rows) * a.heads) return;
+  const int r = static_cast<int>(item / a.heads), h = static_cast<int>(item - static_cast<long long>(r) * a.heads);
+  const int hk = h / (a.heads / a.kv_heads);
+  float* q = pr_q + warp * a.dk;
+  const T* qg = reinterpret_cast<const T*>(a.q) + r * a.ld_q + static_cast<long long>(h) * a.dk;
+  for (int c = lane; c < a.dk; c += 32) q[c] = pr_get(qg + c);
+  __syncwarp();
+  const long long pos = a.row_pos[r];
+  const int* table = a.block_tables + static_cast<long long>(a.row_seq[r]) * a.max_blocks;
+  const long long lo = a.chunk > 0 ? pos / a.chunk * a.chunk : 0;
+  const float slope = a.slopes ? a.slopes[h] : 0.f;
+  const T* K = reinterpret_cast<const T*>(a.k_cache);
+  const T* V = reinterpret_cast<const T*>(a.v_cache);
+  float acc[kPrMaxV];
+#pragma unroll
+  for (int i = 0; i < kPrMaxV; ++i) acc[i] = 0.f;
+  float m = -INFINITY, l = 0.f;
+  for (long long j0 = lo; j0 <= pos; j0 += 32) {
+    const long long j = j0 + lane;
+    long long slot = 0;
+    float s = -INFINITY;
+    if (j <= pos) {
+      const long long bi = j / a.block_size;
+      int blk = bi < a.max_blocks ? table[bi] : -1;
+      if (blk < 0 || blk >= a.num_blocks) {                          // corrupt tables read block 0 instead of faulting
+        RB_BOUNDS_HIT(104);
+        blk = 0;
+      }
+      slot = static_cast<long long>(blk) * a.block_size + (j - bi * a.block_size);
+      const T* k = K + (slot * a.kv_heads + hk) * a.dk;
+      float d = 0.f;
+      for (int c = 0; c < a.dk; ++c) d = fmaf(q[c], pr_get(k + c), d);
+      s = d * a.scale;
+      if (a.softcap > 0.f) s = a.softcap * tanhf(s / a.softcap);
+      s -= slope * static_cast<float>(pos - j);
+    }
+    const float mn = fmaxf(m, warp_max(s));                          // finite: key j0 is always visible
+    const float al = m == -INFINITY ? 0.f : expf(m - mn);
+    const float p = j <= pos ? expf(s - mn) : 0.f;
+    l = l * al + warp_sum(p);
+    m = mn;
+#pragma unroll
+    for (int i = 0; i < kPrMaxV; ++i) acc[i] *= al;
+    const int n = static_cast<int>(pos - j0 + 1 < 32 ? pos - j0 + 1 : 32);
+    for (int jj = 0; jj < n; ++jj) {
+      const float pj = __shfl_sync(0xffffffffu, p, jj);
+      const long long sj = __shfl_sync(0xffffffffu, slot, jj);
+      const T* v = V + (sj * a.kv_heads + hk) * a.dv;
+#pragma unroll
+      for (int i = 0; i < kPrMaxV; ++i) {
+        const int c = i * 32 + lane;
+        if (c < a.dv) acc[i] = fmaf(pj, pr_get(v + c), acc[i]);
+      }
+    }
+  }
+  T* o = reinterpret_cast<T*>(a.out) + r * a.ld_o + static_cast<long long>(h) * a.dv;
+  const T* g = a.gate ? reinterpret_cast<const T*>(a.gate) + r * a.ld_g + static_cast<long long>(h) * a.dv : nullptr;
+  const float inv = 1.f / l;
+#pragma unroll
+  for (int i = 0; i < kPrMaxV; ++i) {
+    const int c = i * 32 + lane;
+    if (c < a.dv) pr_put(o + c, acc[i] * inv * (g ? 1.f / (1.f + expf(-pr_get(g + c))) : 1.f));
+  }
+}
+
 }  // namespace rb
+
+RB_API int rb_paged_attention_rows(const RbPagedRowsArgs* args, void* stream_v) {
+  const RbPagedRowsArgs& a = *args;
+  if (a.rows <= 0) return 0;
+  if (!a.q || !a.out || !a.k_cache || !a.v_cache || !a.block_tables || !a.row_seq || !a.row_pos || a.heads <= 0 ||
+      a.kv_heads <= 0 || a.heads % a.kv_heads || a.dk <= 0 || a.dv <= 0 || a.dv > 32 * rb::kPrMaxV || a.dk > 2048 ||
+      a.block_size <= 0 || a.max_blocks <= 0)
+    return -1;
+  cudaStream_t stream = reinterpret_cast<cudaStream_t>(stream_v);
+  const long long items = static_cast<long long>(a.rows) * a.heads;
+  const int grid = static_cast<int>((items + 3) / 4);
+  const size_t smem = sizeof(float) * 4 * a.dk;
+  if (a.f32) rb::paged_rows_kernel<float><<<grid, 128, smem, stream>>>(a RB_BOUNDS_ARG);
+  else rb::paged_rows_kernel<__nv_bfloat16><<<grid, 128, smem, stream>>>(a RB_BOUNDS_ARG);
+  return static_cast<int>(cudaGetLastError());
+}
 
 RB_API int rb_kv_append(const void* k_new, long long ld_k, const void* v_new, long long ld_v, void* k_cache, void* v_cache,
                         const long long* slot_mapping, long long tokens, int kv_heads, int head_dim, long long num_slots,

@@ -19,6 +19,28 @@ int rb_paged_attention_decode(const void* q, long long ld_q, void* out, long lon
                               const void* v_cache, const int* block_tables, int max_blocks, const int* context_lens,
                               int batch, int heads, int kv_heads, int head_dim, int block_size, long long num_blocks,
                               float scale, float* scratch, void* stream);
+// Attention over the pages for any rows of a batch (prompt portions and decoded tokens alike), any head sizes, bf16 or
+// fp32 operands, fp32 arithmetic: the 32-bit mode and the fallback for head sizes the tensor-core kernels do not take.
+//   row r is the token at position row_pos[r] of the sequence whose pages are block_tables[row_seq[r]]; it sees the keys
+//   j <= pos, and with chunk > 0 only those with j / chunk == pos / chunk
+//   score = q . k * scale; softcap > 0: score <- softcap * tanh(score / softcap); slopes (fp32 [heads], or NULL):
+//   score <- score - slopes[h] * (pos - j)
+//   gate (type of q, pitch ld_g, [rows, heads * dv], or NULL): the output is multiplied by sigmoid(gate)
+typedef struct RbPagedRowsArgs {
+  const void* q;
+  void* out;
+  const void* k_cache;       // [num_blocks, block_size, kv_heads, dk]
+  const void* v_cache;       // [num_blocks, block_size, kv_heads, dv]
+  const int* block_tables;   // [sequences, max_blocks]
+  const int* row_seq;
+  const long long* row_pos;
+  const float* slopes;
+  const void* gate;
+  long long ld_q, ld_o, ld_g, num_blocks;
+  int f32, rows, max_blocks, heads, kv_heads, dk, dv, block_size, chunk;
+  float scale, softcap;
+} RbPagedRowsArgs;
+int rb_paged_attention_rows(const RbPagedRowsArgs* args, void* stream);
 #ifdef __cplusplus
 }
 #endif

@@ -1,0 +1,144 @@
+// Norm on a sublayer's output, added to a 32-bit residual stream, in one pass: x += norm(source), h = copy of x for the
+// next matrix product.  The source is a plain row (attention output projection) or the weighted sum of a token's expert
+// rows plus the shared expert's row, so a routed feed-forward's combine, norm and residual add are one launch.
+// Statistics, sums and the residual are fp32; one CTA owns a row and keeps it in registers.
+#include "residual_norm.h"
+
+#include "rb_common.cuh"
+
+namespace rb {
+
+template <int VEC>
+__device__ __forceinline__ void rn_load(const void* base, long long off, int f32, float (&v)[VEC]) {
+  if (VEC == 4) {
+    if (f32) {
+      const float4 u = *reinterpret_cast<const float4*>(reinterpret_cast<const float*>(base) + off);
+      v[0] = u.x; v[1 % VEC] = u.y; v[2 % VEC] = u.z; v[3 % VEC] = u.w;
+    } else {
+      const uint2 u = *reinterpret_cast<const uint2*>(reinterpret_cast<const __nv_bfloat16*>(base) + off);
+      const float2 a = unpack_bf16x2(u.x), b = unpack_bf16x2(u.y);
+      v[0] = a.x; v[1 % VEC] = a.y; v[2 % VEC] = b.x; v[3 % VEC] = b.y;
+    }
+  } else {
+    v[0] = f32 ? reinterpret_cast<const float*>(base)[off]
+               : __bfloat162float(reinterpret_cast<const __nv_bfloat16*>(base)[off]);
+  }
+}
+template <int VEC>
+__device__ __forceinline__ void rn_store(void* base, long long off, int f32, const float (&v)[VEC]) {
+  if (VEC == 4) {
+    if (f32)
+      *reinterpret_cast<float4*>(reinterpret_cast<float*>(base) + off) = make_float4(v[0], v[1 % VEC], v[2 % VEC], v[3 % VEC]);
+    else
+      *reinterpret_cast<uint2*>(reinterpret_cast<__nv_bfloat16*>(base) + off) =
+          make_uint2(pack_bf16x2(v[0], v[1 % VEC]), pack_bf16x2(v[2 % VEC], v[3 % VEC]));
+  } else if (f32) {
+    reinterpret_cast<float*>(base)[off] = v[0];
+  } else {
+    reinterpret_cast<__nv_bfloat16*>(base)[off] = __float2bfloat16(v[0]);
+  }
+}
+
+// sum over the CTA; `red` holds one float per warp
+__device__ __forceinline__ float rn_block_sum(float v, float* red) {
+  v = warp_sum(v);
+  const int warps = blockDim.x >> 5;
+  if (warps == 1) return v;
+  __syncthreads();
+  if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = v;
+  __syncthreads();
+  float s = 0.f;
+  for (int i = 0; i < warps; ++i) s += red[i];
+  return s;
+}
+
+template <int VEC, int CH>
+__global__ void __launch_bounds__(256)
+residual_norm_kernel(const RbResidualNormArgs a) {
+  __shared__ float red[8];
+  const int t = blockIdx.x, n = a.n;
+  float v[CH][VEC], xr[CH][VEC];
+#pragma unroll
+  for (int c = 0; c < CH; ++c) {
+    const int col = (c * blockDim.x + threadIdx.x) * VEC;
+#pragma unroll
+    for (int i = 0; i < VEC; ++i) { v[c][i] = 0.f; xr[c][i] = 0.f; }
+    if (col >= n) continue;
+    if (a.x) rn_load<VEC>(a.x, t * a.ldx + col, 1, xr[c]);
+    if (a.add) rn_load<VEC>(a.add, t * a.ld_add + col, a.y_f32, v[c]);
+    if (a.slot_pos) {
+      for (int j = 0; j < a.k; ++j) {                     // fixed order: reproducible
+        const float w = a.slot_w[static_cast<long long>(t) * a.k + j];
+        float u[VEC];
+        rn_load<VEC>(a.y, a.slot_pos[static_cast<long long>(t) * a.k + j] * a.ldy + col, a.y_f32, u);
+#pragma unroll
+        for (int i = 0; i < VEC; ++i) v[c][i] = fmaf(w, u[i], v[c][i]);
+      }
+    } else {
+      float u[VEC];
+      rn_load<VEC>(a.y, t * a.ldy + col, a.y_f32, u);
+#pragma unroll
+      for (int i = 0; i < VEC; ++i) v[c][i] += u[i];
+    }
+  }
+  const float inv_n = 1.f / static_cast<float>(n);
+  float mean = 0.f;
+  if (!a.rms) {
+    float s = 0.f;
+#pragma unroll
+    for (int c = 0; c < CH; ++c)
+#pragma unroll
+      for (int i = 0; i < VEC; ++i) s += v[c][i];
+    mean = rn_block_sum(s, red) * inv_n;
+  }
+  float sq = 0.f;
+#pragma unroll
+  for (int c = 0; c < CH; ++c)
+    if ((c * blockDim.x + threadIdx.x) * VEC < n) {
+#pragma unroll
+      for (int i = 0; i < VEC; ++i) { const float d = v[c][i] - mean; sq += d * d; }
+    }
+  const float rstd = rsqrtf(rn_block_sum(sq, red) * inv_n + a.eps);
+#pragma unroll
+  for (int c = 0; c < CH; ++c) {
+    const int col = (c * blockDim.x + threadIdx.x) * VEC;
+    if (col >= n) continue;
+    float g[VEC], b[VEC], o[VEC];
+    rn_load<VEC>(a.gamma, col, a.param_f32, g);
+#pragma unroll
+    for (int i = 0; i < VEC; ++i) b[i] = 0.f;
+    if (a.beta) rn_load<VEC>(a.beta, col, a.param_f32, b);
+#pragma unroll
+    for (int i = 0; i < VEC; ++i) o[i] = xr[c][i] + ((v[c][i] - mean) * rstd * g[i] + b[i]);
+    if (a.x) rn_store<VEC>(a.x, t * a.ldx + col, 1, o);
+    if (a.h) rn_store<VEC>(a.h, t * a.ldh + col, a.h_f32, o);
+  }
+}
+
+template <int VEC>
+int rn_launch(const RbResidualNormArgs& a, cudaStream_t s) {
+  const int units = (a.n + VEC - 1) / VEC;
+  const int threads = units <= 64 ? 64 : units <= 128 ? 128 : 256;
+  const int ch = (units + threads - 1) / threads;
+  if (ch <= 1) residual_norm_kernel<VEC, 1><<<a.rows, threads, 0, s>>>(a);
+  else if (ch <= 2) residual_norm_kernel<VEC, 2><<<a.rows, threads, 0, s>>>(a);
+  else if (ch <= 4) residual_norm_kernel<VEC, 4><<<a.rows, threads, 0, s>>>(a);
+  else if (ch <= 8) residual_norm_kernel<VEC, 8><<<a.rows, threads, 0, s>>>(a);
+  else if (ch <= 16) residual_norm_kernel<VEC, 16><<<a.rows, threads, 0, s>>>(a);
+  else return -6;
+  return static_cast<int>(cudaGetLastError());
+}
+
+}  // namespace rb
+
+RB_API int rb_residual_norm(const RbResidualNormArgs* args, void* stream_v) {
+  const RbResidualNormArgs& a = *args;
+  if (a.rows <= 0 || a.n <= 0 || !a.y || !a.gamma || (!a.x && !a.h)) return -1;
+  if (a.slot_pos && (!a.slot_w || a.k <= 0)) return -1;
+  const uintptr_t bits = reinterpret_cast<uintptr_t>(a.y) | reinterpret_cast<uintptr_t>(a.add) |
+                         reinterpret_cast<uintptr_t>(a.gamma) | reinterpret_cast<uintptr_t>(a.beta) |
+                         reinterpret_cast<uintptr_t>(a.x) | reinterpret_cast<uintptr_t>(a.h);
+  const bool vec = !(bits & 15) && !((a.n | a.ldy | a.ld_add | a.ldx | a.ldh) & 3);
+  cudaStream_t s = reinterpret_cast<cudaStream_t>(stream_v);
+  return vec ? rb::rn_launch<4>(a, s) : rb::rn_launch<1>(a, s);
+}

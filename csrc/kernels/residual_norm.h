@@ -1,0 +1,24 @@
+// C interface of the sublayer-output norm with a 32-bit residual stream (residual_norm.cu).
+#pragma once
+#ifdef __cplusplus
+extern "C" {
+#endif
+typedef struct RbResidualNormArgs {
+  // source row t: y[t] (slot_pos NULL), or the routed sum  sum_j slot_w[t k + j] * y[slot_pos[t k + j]]; plus add[t] if given
+  const void* y;
+  const int* slot_pos;
+  const float* slot_w;
+  const void* add;
+  const void* gamma;        // bf16 or fp32 [n] (param_f32)
+  const void* beta;         // same type, or NULL
+  float* x;                 // fp32 residual [rows, n], updated in place: x += norm(source); NULL: no residual
+  void* h;                  // copy of the new residual (without x: the normalised row), bf16 or fp32, or NULL
+  long long ldy, ld_add, ldx, ldh;
+  int y_f32, param_f32, h_f32;   // y and add share y_f32
+  int k, rows, n, rms;
+  float eps;
+} RbResidualNormArgs;
+int rb_residual_norm(const RbResidualNormArgs* args, void* stream);
+#ifdef __cplusplus
+}
+#endif

@@ -14,6 +14,7 @@ under a minute on a CPU-only machine (nvcc cross-compiles without a GPU).
 from __future__ import annotations
 
 import os
+import re
 import shutil
 import subprocess
 import sys
@@ -49,6 +50,22 @@ def _newer(target: Path, deps) -> bool:
     return all(Path(d).stat().st_mtime <= t for d in deps)
 
 
+_INCLUDE = re.compile(r'^\s*#\s*include\s+"([^"]+)"', re.M)
+
+
+def _included(src: Path, headers) -> list:
+    """The files of `headers` that `src` includes, directly or through another of them."""
+    by_name = {h.name: h for h in headers}
+    seen, todo = {}, [src]
+    while todo:
+        for name in _INCLUDE.findall(todo.pop().read_text()):
+            h = by_name.get(Path(name).name)
+            if h is not None and h.name not in seen:
+                seen[h.name] = h
+                todo.append(h)
+    return list(seen.values())
+
+
 def _run(cmd, verbose):
     if verbose:
         print(" ".join(str(c) for c in cmd), file=sys.stderr)
@@ -65,7 +82,7 @@ def _compile_group(sources, headers, out_lib: Path, compiler_cmd, link_cmd, verb
     for src in sources:
         obj = OBJ_DIR / (out_lib.stem + "__" + src.stem + ".o")
         objs.append(obj)
-        if force or not _newer(obj, [src, *headers]):
+        if force or not _newer(obj, [src, *_included(src, headers)]):
             jobs.append(compiler_cmd(src, obj))
     if jobs:
         with ThreadPoolExecutor(max_workers=min(8, os.cpu_count() or 4)) as ex:
@@ -90,6 +107,24 @@ def build_kernels(force: bool = False, verbose: bool = False, bounds: bool = Fal
         lambda s, o: [nvcc, *NVCC_FLAGS, *extra, *inc, "-c", s, "-o", o],
         lambda objs, out: [nvcc, "-shared", "-gencode", "arch=compute_100a,code=sm_100a", *objs, "-o", out],
         verbose, force)
+
+
+def kernels_current() -> bool:
+    """True when the full kernel library exists and is newer than every source it is made of."""
+    files = [f for d in ("kernels", "comm") for pat in ("*.cu", "*.h", "*.cuh") for f in (CSRC / d).glob(pat)]
+    return _newer(LIB_DIR / "librb200_kernels.so", files)
+
+
+def build_kernels_subset(name: str, stems, verbose: bool = False) -> Path:
+    """``librb200_<name>.so`` from the named files of csrc/kernels and the host side every library needs (rb_host.cu)."""
+    srcs = [CSRC / "kernels" / (s + ".cu") for s in dict.fromkeys((*stems, "rb_host"))]
+    hdrs = sorted((CSRC / "kernels").glob("*.h")) + sorted((CSRC / "kernels").glob("*.cuh"))
+    nvcc = _nvcc()
+    return _compile_group(
+        srcs, hdrs, LIB_DIR / f"librb200_{name}.so",
+        lambda s, o: [nvcc, *NVCC_FLAGS, "-I", str(CSRC / "kernels"), "-c", s, "-o", o],
+        lambda objs, out: [nvcc, "-shared", "-gencode", "arch=compute_100a,code=sm_100a", *objs, "-o", out],
+        verbose, False)
 
 
 def _build_cxx(subdir: str, libname: str, force: bool, verbose: bool) -> Path:

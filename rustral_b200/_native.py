@@ -53,6 +53,35 @@ class RbAttnArgs(C.Structure):
     ]
 
 
+class RbResidualNormArgs(C.Structure):
+    _fields_ = [
+        ("y", c_void_p), ("slot_pos", c_void_p), ("slot_w", c_void_p), ("add", c_void_p), ("gamma", c_void_p), ("beta", c_void_p),
+        ("x", c_void_p), ("h", c_void_p),
+        ("ldy", c_ll), ("ld_add", c_ll), ("ldx", c_ll), ("ldh", c_ll),
+        ("y_f32", c_int), ("param_f32", c_int), ("h_f32", c_int),
+        ("k", c_int), ("rows", c_int), ("n", c_int), ("rms", c_int), ("eps", c_float),
+    ]
+
+
+class RbHeadPrepArgs(C.Structure):
+    _fields_ = [
+        ("p", c_void_p), ("q_gamma", c_void_p), ("k_gamma", c_void_p), ("v_first", c_void_p), ("mix", c_void_p),
+        ("k_cache", c_void_p), ("v_cache", c_void_p), ("slots", c_void_p),
+        ("ld", c_ll), ("off_q", c_ll), ("off_k", c_ll), ("off_v", c_ll), ("ld_vf", c_ll), ("tokens", c_ll), ("num_slots", c_ll),
+        ("f32", c_int), ("heads", c_int), ("kv_heads", c_int), ("dk", c_int), ("dv", c_int), ("eps", c_float),
+    ]
+
+
+class RbPagedRowsArgs(C.Structure):
+    _fields_ = [
+        ("q", c_void_p), ("out", c_void_p), ("k_cache", c_void_p), ("v_cache", c_void_p), ("block_tables", c_void_p),
+        ("row_seq", c_void_p), ("row_pos", c_void_p), ("slopes", c_void_p), ("gate", c_void_p),
+        ("ld_q", c_ll), ("ld_o", c_ll), ("ld_g", c_ll), ("num_blocks", c_ll),
+        ("f32", c_int), ("rows", c_int), ("max_blocks", c_int), ("heads", c_int), ("kv_heads", c_int), ("dk", c_int),
+        ("dv", c_int), ("block_size", c_int), ("chunk", c_int), ("scale", c_float), ("softcap", c_float),
+    ]
+
+
 class RbAdamArgs(C.Structure):
     _fields_ = [
         ("lr", c_float), ("beta1", c_float), ("beta2", c_float), ("eps", c_float), ("weight_decay", c_float),
@@ -101,6 +130,17 @@ def kernels() -> C.CDLL:
     return lib
 
 
+def ensure_kernels(name: str, sources: tuple) -> None:
+    """Makes sure that `kernels()` can load: a full library that is up to date is kept, otherwise one with only `sources`
+    (stems of csrc/kernels files) is compiled into ``librb200_<name>.so`` and selected.  The first serving call in a
+    checkout without built files uses it; it needs nvcc but no GPU."""
+    global KERNEL_LIB
+    from . import _build
+    if "kernels" in _libs or os.environ.get("RUSTRAL_KERNEL_LIB") or _build.kernels_current():
+        return
+    KERNEL_LIB = _build.build_kernels_subset(name, sources).name
+
+
 def have_kernels() -> bool:
     try:
         kernels()
@@ -141,7 +181,9 @@ def _declare_kernels(lib: C.CDLL) -> None:
     P = c_void_p
 
     def sig(name, args, res=c_int):
-        fn = getattr(lib, name)
+        fn = getattr(lib, name, None)
+        if fn is None:                       # a library built from some of the sources only (see ensure_kernels)
+            return
         fn.argtypes = args
         fn.restype = res
 

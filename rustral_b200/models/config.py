@@ -1,7 +1,9 @@
-"""Model configurations for the decoder-only families (GPT-2 style and Llama style) and named presets."""
+"""Model configurations for the decoder-only families (GPT-2 style, Llama style, layered) and named presets."""
 from __future__ import annotations
 
 from dataclasses import dataclass, asdict
+
+from .layered import LayeredConfig, uniform_layers
 
 
 @dataclass
@@ -83,10 +85,23 @@ PRESETS = {
     "gpt2-test": dict(vocab_size=1000, seq_len=128, n_layer=2, n_head=4, d_model=256, ffn_dim=1024, arch="gpt2"),
     "llama-test": dict(vocab_size=1000, seq_len=128, n_layer=2, n_head=4, n_kv_head=2, d_model=256, ffn_dim=512,
                        arch="llama", rope_theta=10000.0),
+    # layered decoders: `n_layer` equal layers of the given mixer and feed-forward
+    "dolurax-test": dict(arch="Dolurax", vocab_size=1000, d_model=128, n_layer=3, seq_len=512, logit_scale=1.5, logit_softcap=20.0,
+                         mixer=dict(heads=6, kv_heads=2, dim=48, vdim=32, scale=0.15, softcap=12.0, chunk=40, v_mix=True),
+                         mlp=dict(ff=64, experts=12, top=3, groups=3, keep=2, shared_ff=40)),
+    # one decoder layer about the size of a Llama-8B layer: same width, heads and head size, same feed-forward work per token
+    # (7 routed experts + the shared one of 1792 = 14336)
+    "dolurax-moe": dict(arch="Dolurax", vocab_size=128256, d_model=4096, n_layer=32, logit_scale=1.0, logit_softcap=30.0,
+                        mixer=dict(heads=32, kv_heads=8, dim=128, vdim=128, scale=0.08838834764831845, softcap=30.0, chunk=8192,
+                                   v_mix=True),
+                        mlp=dict(ff=1792, experts=32, top=7, groups=4, keep=2, shared_ff=1792)),
 }
 
 
-def preset(name: str, **overrides) -> GPTConfig:
+def preset(name: str, **overrides):
     cfg = dict(PRESETS[name])
     cfg.update(overrides)
+    if "mixer" in cfg:
+        cfg["layers"] = uniform_layers(cfg.pop("n_layer"), cfg.pop("mixer"), cfg.pop("mlp"))
+        return LayeredConfig(**cfg)
     return GPTConfig(**cfg)

@@ -5,13 +5,14 @@ PyTorch route (the native library must be loaded), a CPU tensor takes the fp32 r
 also serves as the numerical oracle in the tests.
 """
 from .matmul import gemm, linear, act_reference, act_grad_reference
-from .norm import layer_norm, rms_norm, norm_forward, norm_backward
+from .norm import layer_norm, rms_norm, norm_forward, norm_backward, residual_norm
 from .loss import cross_entropy, cross_entropy_fwd_bwd, softmax, log_softmax
-from .attention import flash_attention, attention_reference
-from .embed import embedding, embedding_forward, embedding_backward
+from .attention import flash_attention, attention_reference, ScoreRule, distance_slopes
+from .heads import head_prep_
+from .embed import embedding, embedding_forward, embedding_backward, embedding_residual
 from .elementwise import (binary, unary, scalar_op, unary_bwd, add_row_vector, sum_dim0, sum_all, transpose2d,
                           gather_rows, scatter_rows, broadcast_to, strided_copy, apply_mask, dropout, argmax_rows,
-                          gelu, relu, silu)
+                          gelu, relu, silu, scale_softcap_)
 from .rotary import rope, rope_, swiglu, swiglu_forward, swiglu_backward
 from .optim import adam_step, sgd_step, sumsq, cast_f32_to_bf16
 

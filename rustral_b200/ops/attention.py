@@ -2,15 +2,42 @@
 from __future__ import annotations
 
 import math
+from dataclasses import dataclass
 
 import torch
 
 from .. import _native as N
 
 
-def attention_reference(q, k, v, causal: bool, scale: float | None = None, kv_lens=None):
-    """fp32 softmax(QK^T * scale + mask) V on [B, S, H, D] tensors (GQA: fewer K/V heads).  `kv_lens` ([B] integers):
-    keys at positions >= kv_lens[b] are padding (a batch entry without any real key gives zero rows)."""
+@dataclass(frozen=True, eq=False)
+class ScoreRule:
+    """What happens to scaled attention scores before the softmax, and which keys a query sees besides causality.
+
+    softcap > 0: score <- softcap * tanh(score / softcap).  slopes (fp32 [heads]): score <- score - slopes[h] * (i - j), after
+    the cap.  chunk > 0: position i sees j only when i // chunk == j // chunk (positions of the sequence; a kernel that is
+    handed keys from a chunk's first one on may count from there)."""
+    softcap: float = 0.0
+    slopes: torch.Tensor | None = None
+    chunk: int = 0
+
+    def first_key(self, pos: int) -> int:
+        """The first position that the token at `pos` can see."""
+        return pos // self.chunk * self.chunk if self.chunk else 0
+
+    @property
+    def plain(self) -> bool:
+        return not self.softcap and self.slopes is None and not self.chunk
+
+
+def distance_slopes(heads: int, device=None) -> torch.Tensor:
+    """Per-head slopes of a linear distance bias: the geometric sequence 2^(-8 (h + 1) / heads)."""
+    return torch.tensor([2.0 ** (-8.0 * (h + 1) / heads) for h in range(heads)], dtype=torch.float32, device=device)
+
+
+def attention_reference(q, k, v, causal: bool, scale: float | None = None, kv_lens=None, rule: ScoreRule | None = None):
+    """fp32 softmax(QK^T * scale + mask) V on [B, S, H, D] tensors (GQA: fewer K/V heads; V may have its own head size).
+    `kv_lens` ([B] integers): keys at positions >= kv_lens[b] are padding (a batch entry without any real key gives zero
+    rows).  `rule`: see ScoreRule; key 0 is taken as the start of a chunk."""
     B, Sq, H, D = q.shape
     Sk, Hk = k.shape[1], k.shape[2]
     scale = 1.0 / math.sqrt(D) if scale is None else scale
@@ -19,9 +46,16 @@ def attention_reference(q, k, v, causal: bool, scale: float | None = None, kv_le
     if H != Hk:                                             # grouped-query attention: every K/V head serves H / Hk query heads
         kf, vf = kf.repeat_interleave(H // Hk, dim=1), vf.repeat_interleave(H // Hk, dim=1)
     s = qf @ kf.transpose(-1, -2) * scale
+    i = torch.arange(Sq, device=q.device)[:, None] + (Sk - Sq)
+    j = torch.arange(Sk, device=q.device)[None, :]
+    if rule is not None:
+        if rule.softcap:
+            s = rule.softcap * torch.tanh(s / rule.softcap)
+        if rule.slopes is not None:
+            s = s - rule.slopes.to(q.device).float()[None, :, None, None] * (i - j).float()
+        if rule.chunk:
+            s = s.masked_fill(i // rule.chunk != j // rule.chunk, float("-inf"))
     if causal:
-        i = torch.arange(Sq, device=q.device)[:, None] + (Sk - Sq)
-        j = torch.arange(Sk, device=q.device)[None, :]
         s = s.masked_fill(j > i, float("-inf"))
     if kv_lens is not None:
         pad = torch.arange(Sk, device=q.device)[None, :] >= kv_lens.to(q.device).long()[:, None]      # [B, Sk]
@@ -105,6 +139,26 @@ def attention_forward(q, k, v, causal: bool, scale: float, out=None, want_lse: b
             return o, lse
     N.check(lib.rb_attention_fwd(a, N.stream_ptr()), "rb_attention_fwd")
     return o, lse
+
+
+def prompt_supported(q, k, v, dk: int, dv: int, rule: ScoreRule | None = None, gate=None) -> bool:
+    """Whether `prompt_attention` takes these operands (2-D [rows, heads * size] views)."""
+    if not q.is_cuda:
+        return True
+    return q.dtype == torch.bfloat16 and dk == dv and dk in (64, 128) and rule is None and gate is None
+
+
+def prompt_attention(q, k, v, scale: float, out, rule: ScoreRule | None = None, gate=None):
+    """Causal attention of a prompt portion in inference: q [1, L, H, dk], k [1, S, G, dk], v [1, S, G, dv] with the last L
+    keys being the portion itself, out [1, L, H, dv].  `rule`: see ScoreRule (key 0 starts a chunk); `gate`
+    [L, H * dv]: out <- out * sigmoid(gate)."""
+    if not q.is_cuda:
+        o = attention_reference(q, k, v, True, scale, rule=rule)
+        if gate is not None:
+            o = o.float() * torch.sigmoid(gate.float().reshape(o.shape))
+        out.copy_(o)
+        return out
+    return attention_forward(q, k, v, True, scale, out=out, want_lse=False)[0]
 
 
 def attention_backward(do, q, k, v, o, lse, causal: bool, scale: float, dq=None, dk=None, dv=None, impl: str | None = None,

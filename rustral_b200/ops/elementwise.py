@@ -317,3 +317,18 @@ def argmax_rows(a):
     N.check(N.kernels().rb_argmax_rows(a2.data_ptr(), a2.stride(0), out.data_ptr(), a2.shape[0], a2.shape[1], _dt(a2),
                                        N.stream_ptr()), "rb_argmax_rows")
     return out
+
+
+N.optional_sig("rb_scale_softcap", [N.c_void_p, N.c_ll, N.c_float, N.c_float, N.c_void_p])
+
+
+def scale_softcap_(x, scale: float = 1.0, cap: float = 0.0):
+    """In place on a contiguous fp32 tensor: x <- cap * tanh(scale * x / cap) (cap 0: only the scale)."""
+    if not x.is_cuda:
+        v = x * scale
+        x.copy_(cap * torch.tanh(v / cap) if cap else v)
+        return x
+    if x.dtype != torch.float32 or not x.is_contiguous():
+        raise TypeError("scale_softcap_: a contiguous fp32 tensor is required")
+    N.check(N.kernels().rb_scale_softcap(x.data_ptr(), x.numel(), scale, cap, N.stream_ptr()), "rb_scale_softcap")
+    return x

@@ -42,6 +42,25 @@ def embedding_forward(ids: torch.Tensor, wte: torch.Tensor, wpe=None, seq_len: i
     return y
 
 
+N.optional_sig("rb_embedding_residual", [N.c_void_p, N.c_void_p, N.c_int, N.c_void_p, N.c_void_p, N.c_ll, N.c_int, N.c_ll, N.c_void_p])
+
+
+def embedding_residual(ids: torch.Tensor, table: torch.Tensor):
+    """Start of a 32-bit residual stream: (x fp32 [tokens, dim], h = the same rows in the table's dtype; x itself for an
+    fp32 table)."""
+    f32 = table.dtype == torch.float32
+    if not table.is_cuda:
+        h = table[ids]
+        return (h, h) if f32 else (h.float(), h)
+    tokens, dim = ids.numel(), table.shape[1]
+    x = torch.empty((tokens, dim), dtype=torch.float32, device=table.device)
+    h = x if f32 else torch.empty((tokens, dim), dtype=table.dtype, device=table.device)
+    N.check(N.kernels().rb_embedding_residual(ids.data_ptr(), table.data_ptr(), int(f32), x.data_ptr(),
+                                              None if f32 else h.data_ptr(), tokens, dim, table.shape[0], N.stream_ptr()),
+            "rb_embedding_residual")
+    return x, h
+
+
 def embedding_backward(ids, dy2, dwte, dwpe=None, seq_len: int = 0):
     """Accumulates into fp32 ``dwte`` [vocab, dim] (and ``dwpe`` [>=seq_len, dim]); rows are summed in token order."""
     flat = ids.reshape(-1)

@@ -182,6 +182,24 @@ def set_plan_hook(fn) -> None:
     _PLAN_HOOK = fn
 
 
+N.optional_sig("rb_gemm_f32", [N.c_void_p, N.c_ll, N.c_void_p, N.c_ll, N.c_void_p, N.c_ll, N.c_int, N.c_int, N.c_int, N.c_float,
+                               N.c_void_p, N.c_void_p, N.c_ll, N.c_void_p])
+
+
+def _gemm_f32(a, b, out, alpha, tile_expert=None, num_tiles=None, expert_stride=0) -> torch.Tensor:
+    """True fp32 product (the 32-bit serving mode); `tile_expert` / `num_tiles`: the grouped form over stacked experts."""
+    M, K = a.shape
+    Nn = b.shape[0]
+    if a.stride(1) != 1 or b.stride(1) != 1:
+        raise ValueError("gemm: operands must have a contiguous last dimension")
+    out = out if out is not None else torch.empty((M, Nn), dtype=torch.float32, device=a.device)
+    if M == 0 or Nn == 0:
+        return out
+    N.check(N.kernels().rb_gemm_f32(a.data_ptr(), a.stride(0), b.data_ptr(), b.stride(0), out.data_ptr(), out.stride(0), M, Nn, K,
+                                    alpha, N.ptr(tile_expert), N.ptr(num_tiles), expert_stride, N.stream_ptr()), "rb_gemm_f32")
+    return out
+
+
 def gemm(a: torch.Tensor, b: torch.Tensor, *, a_mn: bool = False, b_mn: bool = False, bias=None, act: str = "none",
          residual=None, aux_in=None, aux_out=None, out=None, out_dtype=None, accumulate: bool = False,
          alpha: float = 1.0, block_n: int = 0, group_m: int = 0, max_ctas: int = 0, splits: int = 0,
@@ -213,8 +231,13 @@ def gemm(a: torch.Tensor, b: torch.Tensor, *, a_mn: bool = False, b_mn: bool = F
                 b_mn = False
         return _gemm_cpu(a, b, a_mn, b_mn, bias, act, residual, aux_in, aux_out, out, out_dtype, accumulate, alpha)
 
+    if a.dtype == torch.float32 and b.dtype == torch.float32:
+        if (a_mn or b_mn or act != "none" or accumulate or peer is not None or out_dtype != torch.float32
+                or any(t is not None for t in (bias, residual, aux_in, aux_out, row_scale, col_scale))):
+            raise TypeError("gemm: fp32 CUDA operands take the plain product only (no epilogue, no transposed operand)")
+        return _gemm_f32(a, b, out, alpha)
     if a.dtype != torch.bfloat16 or b.dtype != torch.bfloat16:
-        raise TypeError("gemm: CUDA operands must be bf16 (accumulation is fp32)")
+        raise TypeError("gemm: CUDA operands must be both bf16 (accumulation is fp32) or both fp32")
     if M == 0 or Nn == 0:
         # an empty batch (or an empty layer): nothing to launch; a given output is left as it is
         if aux_out is not None and aux_out.numel():

@@ -13,11 +13,13 @@ import torch
 
 from .. import _native as N
 from . import rotary
-from .matmul import gemm, act_reference, act_grad_reference
+from .matmul import gemm, _gemm_f32, act_reference, act_grad_reference
 
 P, I, F, LL = N.c_void_p, N.c_int, N.c_float, N.c_ll
 N.optional_sig("rb_moe_route", [P, I, I, I, I, P, P, P, P])
 N.optional_sig("rb_moe_route_bwd", [P, P, P, P, P, I, I, I, I, F, P, P])
+N.optional_sig("rb_moe_route_groups", [P, I, I, I, I, I, I, F, P, P, P])
+N.optional_sig("rb_swiglu_live", [P, LL, P, LL, I, I, I, P, P])
 N.optional_sig("rb_moe_plan", [P, I, I, I, P, P, P, P, P, P, I, P])
 N.optional_sig("rb_moe_gather", [P, P, P, P, I, I, I, P, P])
 N.optional_sig("rb_moe_combine", [P, P, P, P, P, I, I, I, P])
@@ -44,6 +46,44 @@ def route(logits: torch.Tensor, k: int, renorm: bool = True):
     N.check(N.kernels().rb_moe_route(logits.data_ptr(), T, E, k, int(renorm), idx.data_ptr(), w.data_ptr(), probs.data_ptr(),
                                      N.stream_ptr()), "rb_moe_route")
     return idx, w, probs
+
+
+def route_groups(logits: torch.Tensor, k: int, groups: int = 1, keep: int = 1, renorm: bool = True, eps: float = 1e-20):
+    """Group-limited top-k routing for inference: softmax scores over all experts; the experts form `groups` equal groups
+    of neighbours, a group counts as its largest score and only experts of the best `keep` groups can be chosen; the
+    weights are the chosen scores, divided by (their sum + eps) with `renorm`.  logits fp32 [T, E] ->
+    (idx int32 [T, k], w fp32 [T, k])."""
+    T, E = logits.shape
+    if not logits.is_cuda:
+        s = torch.softmax(logits.float(), -1)
+        c = s
+        if groups > 1 and keep < groups:
+            best = s.view(T, groups, E // groups).amax(-1)
+            kept = torch.sort(-best, dim=-1, stable=True).indices[:, :keep]
+            ok = torch.zeros((T, groups), dtype=torch.bool).scatter_(1, kept, True)
+            c = s.masked_fill(~ok.repeat_interleave(E // groups, 1), -1.0)
+        order = torch.sort(-c, dim=-1, stable=True).indices[:, :k]
+        w = s.gather(1, order)
+        if renorm:
+            w = w / (w.sum(-1, keepdim=True) + eps)
+        return order.to(torch.int32), w
+    idx = torch.empty((T, k), dtype=torch.int32, device=logits.device)
+    w = torch.empty((T, k), dtype=torch.float32, device=logits.device)
+    N.check(N.kernels().rb_moe_route_groups(logits.data_ptr(), T, E, k, groups, keep, int(renorm), float(eps), idx.data_ptr(),
+                                            w.data_ptr(), N.stream_ptr()), "rb_moe_route_groups")
+    return idx, w
+
+
+def swiglu_live(gu: torch.Tensor, live_rows=None) -> torch.Tensor:
+    """silu(gate) * up for gu = [gate | up] rows; `live_rows` (int32 [1] on the device): later rows are left unwritten."""
+    rows, F2 = gu.shape
+    if not gu.is_cuda:
+        g, u = gu.float()[:, :F2 // 2], gu.float()[:, F2 // 2:]
+        return (g * torch.sigmoid(g) * u).to(gu.dtype)
+    h = torch.empty((rows, F2 // 2), dtype=gu.dtype, device=gu.device)
+    N.check(N.kernels().rb_swiglu_live(gu.data_ptr(), gu.stride(0), h.data_ptr(), h.stride(0), rows, F2 // 2,
+                                       int(gu.dtype == torch.float32), N.ptr(live_rows), N.stream_ptr()), "rb_swiglu_live")
+    return h
 
 
 def route_backward(probs, idx, w, dw, counts, renorm: bool, aux_grad_scale: float):
@@ -110,8 +150,9 @@ def plan(idx: torch.Tensor, num_experts: int) -> MoEPlan:
     return pl
 
 
-def gather(x: torch.Tensor, pl: MoEPlan, slot_scale=None) -> torch.Tensor:
-    """x [T, d] -> permuted [max_rows, d] (rows past the last expert segment are left untouched / zero)."""
+def gather(x: torch.Tensor, pl: MoEPlan, slot_scale=None, zero_tail: bool = True) -> torch.Tensor:
+    """x [T, d] -> permuted [max_rows, d].  Padding rows inside the expert segments are zero; rows past the last segment
+    are zero as well, or (`zero_tail` False: inference, nothing reads them) left unwritten."""
     T, d = x.shape
     if not x.is_cuda:
         xp = torch.zeros((pl.max_rows, d), dtype=x.dtype)
@@ -121,9 +162,13 @@ def gather(x: torch.Tensor, pl: MoEPlan, slot_scale=None) -> torch.Tensor:
             src = src * slot_scale.reshape(-1)[pl.row_slot[ok].long()][:, None]
         xp[ok] = src.to(x.dtype)
         return xp
-    xp = torch.zeros((pl.max_rows, d), dtype=x.dtype, device=x.device)   # rows past the last segment stay zero
+    make = torch.zeros if zero_tail else torch.empty
+    xp = make((pl.max_rows, d), dtype=x.dtype, device=x.device)
+    if x.dtype == torch.float32 and slot_scale is not None:
+        raise TypeError("gather: fp32 rows are copied without a scale")
+    halves = d * (2 if x.dtype == torch.float32 else 1)                  # the kernel copies rows of 16-bit elements
     N.check(N.kernels().rb_moe_gather(x.contiguous().data_ptr(), pl.row_slot.data_ptr(), N.ptr(slot_scale), xp.data_ptr(),
-                                      pl.max_rows, pl.k, d, pl.offsets[pl.num_experts:].data_ptr(), N.stream_ptr()),
+                                      pl.max_rows, pl.k, halves, pl.offsets[pl.num_experts:].data_ptr(), N.stream_ptr()),
             "rb_moe_gather")
     return xp
 
@@ -181,6 +226,10 @@ def grouped_gemm(xp: torch.Tensor, W: torch.Tensor, pl: MoEPlan, *, b_mn: bool =
                        aux_out=None if aux_out is None else aux_out[o:o + c])
             y[o:o + c] = seg
         return y
+    if xp.dtype == torch.float32:
+        if b_mn or act != "none" or aux_out is not None or aux_in is not None or arrived is not None:
+            raise TypeError("grouped_gemm: fp32 operands take the plain product only")
+        return _gemm_f32(xp, W[0], out, 1.0, pl.tile_expert, pl.num_tiles, W.stride(0))
     y = out if out is not None else torch.empty((rows, Nn), dtype=xp.dtype, device=xp.device)
     W2 = W.reshape(-1, W.shape[2])
     g = N.RbGemmArgs()

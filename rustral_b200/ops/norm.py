@@ -143,3 +143,49 @@ def rms_norm(x, gamma, eps: float = 1e-5):
     if not N.wants_grad(x, gamma):
         return _norm_inference(x, gamma, None, eps, True)
     return _NormFn.apply(x, gamma, None, eps, True)
+
+
+N.optional_sig("rb_residual_norm", [N.C.POINTER(N.RbResidualNormArgs), N.c_void_p])
+
+
+def residual_norm(y, gamma, beta, eps: float, rms: bool = False, *, x=None, h=None, routed=None, add=None):
+    """Norm of a sublayer's output added to a 32-bit residual stream.
+
+    source row t = y[t], or with `routed` = (slot_pos int32 [T * k], weights fp32 [T, k]) the weighted sum of token t's
+    expert rows of `y`; `add` (same dtype as y) is added to it.  With `x` (fp32 [T, n]): x += norm(source) in place and
+    `h` receives a copy in its own dtype.  Without `x`: `h` receives norm(source).  Returns h (x when h is None)."""
+    rows = x.shape[0] if x is not None else h.shape[0]
+    n = y.shape[1]
+    if not y.is_cuda:
+        src = y.float()
+        if routed is not None:
+            slot_pos, w = routed
+            src = (src[slot_pos.long()].view(rows, -1, n) * w.float()[:, :, None]).sum(1)
+        if add is not None:
+            src = src + add.float()
+        o = norm_forward(src, gamma, beta, eps, rms)[0].float()
+        if x is not None:
+            x += o
+            o = x
+        if h is not None:
+            h.copy_(o)
+        return h if h is not None else x
+    a = N.RbResidualNormArgs()
+    a.y, a.ldy, a.y_f32 = y.data_ptr(), y.stride(0), int(y.dtype == torch.float32)
+    if add is not None:
+        if add.dtype != y.dtype:
+            raise TypeError("residual_norm: `add` and `y` must have the same dtype")
+        a.add, a.ld_add = add.data_ptr(), add.stride(0)
+    if routed is not None:
+        slot_pos, w = routed
+        a.slot_pos, a.slot_w, a.k = slot_pos.data_ptr(), w.data_ptr(), w.shape[1]
+    a.gamma, a.beta, a.param_f32 = gamma.data_ptr(), N.ptr(beta), int(gamma.dtype == torch.float32)
+    if x is not None:
+        if x.dtype != torch.float32:
+            raise TypeError("residual_norm: the residual stream is fp32")
+        a.x, a.ldx = x.data_ptr(), x.stride(0)
+    if h is not None:
+        a.h, a.ldh, a.h_f32 = h.data_ptr(), h.stride(0), int(h.dtype == torch.float32)
+    a.rows, a.n, a.rms, a.eps = rows, n, int(rms), eps
+    N.check(N.kernels().rb_residual_norm(a, N.stream_ptr()), "rb_residual_norm")
+    return h if h is not None else x

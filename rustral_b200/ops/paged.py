@@ -6,6 +6,7 @@ import math
 import torch
 
 from .. import _native as N
+from .attention import ScoreRule, attention_reference
 
 N.optional_sig("rb_kv_append", [N.c_void_p, N.c_ll, N.c_void_p, N.c_ll, N.c_void_p, N.c_void_p, N.c_void_p, N.c_ll, N.c_int,
                                 N.c_int, N.c_ll, N.c_void_p])
@@ -32,14 +33,25 @@ def kv_append(k_new, v_new, k_cache, v_cache, slot_mapping):
             "rb_kv_append")
 
 
-def paged_attention_decode(q, k_cache, v_cache, block_tables, context_lens, scale=None, out=None):
-    """q: [batch, heads * head_dim] (or [batch, heads, head_dim]); block_tables int32 [batch, max_blocks];
-    context_lens int32 [batch].  Returns [batch, heads * head_dim]."""
+def decode_supported(q, dk: int, dv: int, rule: ScoreRule | None = None, gate=None) -> bool:
+    """Whether `paged_attention_decode` takes these operands."""
+    if not q.is_cuda:
+        return True
+    return q.dtype == torch.bfloat16 and dk == dv and dk in (64, 128) and rule is None and gate is None
+
+
+def paged_attention_decode(q, k_cache, v_cache, block_tables, context_lens, scale=None, out=None, rule: ScoreRule | None = None,
+                           gate=None):
+    """q: [batch, heads * dk] (or [batch, heads, dk]); block_tables int32 [batch, max_blocks]; context_lens int32 [batch].
+    Returns [batch, heads * dv].  `rule`: see ops.ScoreRule; `gate` [batch, heads * dv]: the output times sigmoid(gate)."""
     nb, bs, hk, d = k_cache.shape
+    dv = v_cache.shape[3]
     B = q.shape[0]
     q2 = q.reshape(B, -1)
     heads = q2.shape[1] // d
     scale = 1.0 / math.sqrt(d) if scale is None else scale
+    if not q.is_cuda and (rule is not None or gate is not None or dv != d):
+        return paged_attention_rows(q2, k_cache, v_cache, block_tables, torch.arange(B), context_lens.long() - 1, scale, rule, gate, out)
     if not q.is_cuda:
         o = torch.zeros(B, heads, d)
         kc, vc = k_cache.view(nb * bs, hk, d).float(), v_cache.view(nb * bs, hk, d).float()
@@ -64,4 +76,41 @@ def paged_attention_decode(q, k_cache, v_cache, block_tables, context_lens, scal
                                           k_cache.data_ptr(), v_cache.data_ptr(), block_tables.data_ptr(),
                                           block_tables.shape[1], context_lens.data_ptr(), B, heads, hk, d, bs, nb,
                                           scale, scratch.data_ptr(), N.stream_ptr()), "rb_paged_attention_decode")
+    return out
+
+
+N.optional_sig("rb_paged_attention_rows", [N.C.POINTER(N.RbPagedRowsArgs), N.c_void_p])
+
+
+def paged_attention_rows(q, k_cache, v_cache, block_tables, row_seq, row_pos, scale: float, rule: ScoreRule | None = None,
+                         gate=None, out=None):
+    """Attention over the pages for any rows of a batch.  q: [rows, heads * dk] (row-strided views allowed); row r is the
+    token at position row_pos[r] (int64) of the sequence with pages block_tables[row_seq[r]] (int32); its own key is
+    already in the cache.  Takes bf16 and fp32 and any head sizes.  `gate` [rows, heads * dv]: output times sigmoid(gate)."""
+    nb, bs, hk, dk = k_cache.shape
+    dv = v_cache.shape[3]
+    rows, heads = q.shape[0], q.shape[1] // dk
+    rule = rule or ScoreRule()
+    out = out if out is not None else torch.empty((rows, heads * dv), dtype=q.dtype, device=q.device)
+    if not q.is_cuda:
+        kc, vc = k_cache.view(nb * bs, hk, dk), v_cache.view(nb * bs, hk, dv)
+        for r in range(rows):
+            n, table = int(row_pos[r]) + 1, block_tables[int(row_seq[r])].long()
+            lo = rule.first_key(n - 1)
+            toks = torch.arange(lo, n)
+            slots = table[toks // bs] * bs + toks % bs
+            o = attention_reference(q[r].view(1, 1, heads, dk), kc[slots][None], vc[slots][None], True, scale, rule=rule)
+            o = o.reshape(-1).float()
+            out[r] = o * torch.sigmoid(gate[r].float()) if gate is not None else o
+        return out
+    a = N.RbPagedRowsArgs()
+    a.q, a.ld_q, a.out, a.ld_o = q.data_ptr(), q.stride(0), out.data_ptr(), out.stride(0)
+    a.k_cache, a.v_cache, a.num_blocks, a.block_size = k_cache.data_ptr(), v_cache.data_ptr(), nb, bs
+    a.block_tables, a.max_blocks = block_tables.data_ptr(), block_tables.shape[1]
+    a.row_seq, a.row_pos = row_seq.data_ptr(), row_pos.data_ptr()
+    if gate is not None:
+        a.gate, a.ld_g = gate.data_ptr(), gate.stride(0)
+    a.f32, a.rows, a.heads, a.kv_heads, a.dk, a.dv = int(q.dtype == torch.float32), rows, heads, hk, dk, dv
+    a.scale, a.softcap, a.slopes, a.chunk = scale, rule.softcap, N.ptr(rule.slopes), rule.chunk
+    N.check(N.kernels().rb_paged_attention_rows(a, N.stream_ptr()), "rb_paged_attention_rows")
     return out

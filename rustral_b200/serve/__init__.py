@@ -1,5 +1,5 @@
 """Serving: KV caches, continuous-batching scheduler, sampler, model runner, engine, HTTP front end."""
-from .kv_cache import CacheQuantization, CacheConfig, CacheMemoryStats, KVCache, SlidingWindowCache, PagedCache, BatchedCache
+from .kv_cache import CacheQuantization, CacheConfig, CacheMemoryStats, KVCache, SlidingWindowCache, CacheLayer, PagedCache, BatchedCache
 from .scheduler import RequestPriority, RequestState, Request, SchedulingPolicy, Batch, Scheduler, PyScheduler, SchedulerStats
 from .sampler import Sampler
 from .model_runner import ModelRunner

@@ -1,0 +1,166 @@
+"""The layer bodies that the serving runner executes, one class per family of decoders.
+
+A body knows a model's mathematics only: embedding, one layer, output head, and what each layer stores in the cache.  Which
+rows a step holds, where their keys and values go, which kernels attend for which rows, and graph capture belong to the
+runner (serve.model_runner), so every body gets prefill, chunked prefill, mixed batches and graphed decoding from it.
+
+`embed` returns the stream that `layer` takes and returns; `head` turns selected rows of it into logits.
+"""
+from __future__ import annotations
+
+import math
+
+import torch
+
+from .. import ops
+from ..ops import moe as moe_ops
+from ..ops import norm as norm_ops
+from ..ops import paged as paged_ops
+from ..ops import rotary as rope_ops
+from ..ops.attention import ScoreRule, distance_slopes
+from ..ops.heads import head_prep_
+from ..ops.matmul import gemm
+from .kv_cache import CacheLayer
+
+
+class GPTBody:
+    """GPT-2 style and Llama style decoders (pre-norm, residual stream in the activation dtype)."""
+
+    def __init__(self, runner):
+        self.r, self.cfg = runner, runner.cfg
+        self.rms = self.cfg.arch == "llama"
+        self.scale = 1.0 / math.sqrt(self.cfg.head_dim)
+
+    def cache_layers(self) -> list:
+        return None                                   # uniform: the cache's num_layers / num_kv_heads / head_dim form
+
+    def _norm(self, x, name):
+        P, rms = self.r.params, self.rms
+        y, _, _ = norm_ops.norm_forward(x, P.w(name + ".weight"), None if rms else P.w(name + ".bias"), self.cfg.norm_eps, rms)
+        return y
+
+    def _row_parallel(self, a, w, bias, residual):
+        """a @ w^T (+ bias) + residual; with tensor parallelism the partial products are summed over the ranks."""
+        tp = self.r.tp
+        if tp is None:
+            return gemm(a, w, bias=bias, residual=residual)
+        rows = a.shape[0]
+        gemm(a, w, out=tp.staging(rows, w.shape[0]))
+        return tp.all_reduce(rows, w.shape[0], residual=residual)
+
+    def embed(self, sb):
+        P, cfg = self.r.params, self.cfg
+        x = ops.embedding_forward(sb.ids, P.w("tok_embed.embed"))
+        if cfg.arch == "gpt2":
+            x = ops.binary("add", x, ops.gather_rows(P.w("pos_embed.embed"), sb.pos))
+        return x
+
+    def layer(self, l, x, sb):
+        P, r, rms = self.r.params, self.r, self.rms
+        H, Hk, D = r.n_head, r.n_kv_head, self.cfg.head_dim
+        p = f"layers.{l}."
+        h = self._norm(x, p + "ln1")
+        qkv = gemm(h, P.w(p + "attn.wqkv.weight"), bias=None if rms else P.w(p + "attn.wqkv.bias"))
+        if rms:
+            rope_ops.rope_(qkv, H + Hk, D, positions=sb.pos, theta=self.cfg.rope_theta)
+        k2, v2 = qkv[:, H * D:(H + Hk) * D], qkv[:, (H + Hk) * D:]
+        paged_ops.kv_append(k2, v2, r.cache.k[l], r.cache.v[l], sb.slots)
+        a = r.attend(l, qkv[:, :H * D], k2, v2, sb, self.scale)
+        x = self._row_parallel(a, P.w(p + "attn.wo.weight"), None if rms else P.w(p + "attn.wo.bias"), x)
+        h = self._norm(x, p + "ln2")
+        if rms:
+            gu = gemm(h, P.w(p + "ffn.gate_up.weight"))
+            return self._row_parallel(rope_ops.swiglu_forward(gu), P.w(p + "ffn.down.weight"), None, x)
+        h = gemm(h, P.w(p + "ffn.fc1.weight"), bias=P.w(p + "ffn.fc1.bias"), act="gelu")
+        return gemm(h, P.w(p + "ffn.fc2.weight"), bias=P.w(p + "ffn.fc2.bias"), residual=x)
+
+    def head(self, x, rows):
+        P, cfg, tp = self.r.params, self.cfg, self.r.tp
+        if rows is not None:
+            x = x.index_select(0, rows)
+        xf = self._norm(x.contiguous(), "final_norm")
+        if tp is not None:
+            w = P.w("head.weight")
+            gemm(xf, w, out=tp.staging(xf.shape[0], w.shape[0]))
+            return tp.all_gather_cols(xf.shape[0], w.shape[0])
+        return gemm(xf, P.w("tok_embed.embed" if cfg.tie_embeddings else "head.weight"))
+
+
+class Stream:
+    """Residual stream of a layered decoder: `x` fp32, `h` its copy in the activation dtype (the operand of the next
+    products; `x` itself in 32-bit), `v_first` the value columns of the first layer that mixes values."""
+    __slots__ = ("x", "h", "v_first")
+
+    def __init__(self, x, h):
+        self.x, self.h, self.v_first = x, h, None
+
+
+class LayeredBody:
+    """Layered decoders (models.layered): sublayers read the stream itself, the norm sits on their output.
+
+    Per layer: one packed projection; head norms + value mixing + cache append (one kernel); attention with its score rule
+    and output gate; output projection; norm + residual add; router; experts as grouped products; shared expert; then
+    combine + norm + residual add (one kernel)."""
+
+    def __init__(self, runner):
+        self.r, self.cfg = runner, runner.cfg
+        if runner.tp is not None:
+            raise ValueError("tensor-parallel serving covers the llama family")
+        slopes = {}
+        self.rules = []
+        for s in self.cfg.layers:
+            a = s.mixer
+            if a.heads not in slopes:
+                slopes[a.heads] = distance_slopes(a.heads, runner.device)
+            self.rules.append(ScoreRule(softcap=a.softcap, slopes=slopes[a.heads], chunk=a.chunk))
+
+    def cache_layers(self) -> list:
+        return [CacheLayer(s.mixer.kv_heads, s.mixer.dim, s.mixer.vdim) for s in self.cfg.layers]
+
+    def embed(self, sb):
+        return Stream(*ops.embedding_residual(sb.ids, self.r.params.w("embed")))
+
+    def _add_norm(self, st, y, name, **kw):
+        """x += norm(y), h = x in the activation dtype."""
+        P = self.r.params
+        norm_ops.residual_norm(y, P.w(name), P.w(name + ".b"), self.cfg.norm_eps, x=st.x,
+                               h=None if st.h is st.x else st.h, **kw)
+
+    def layer(self, l, st, sb):
+        r, P, s = self.r, self.r.params, self.cfg.layers[l]
+        a, p = s.mixer, f"l{l}."
+        H, G, dk, dv = a.heads, a.kv_heads, a.dim, a.vdim
+        z = gemm(st.h, P.w(p + "attn.in"))
+        ov = (H + G) * dk
+        k2, v2, gate = z[:, H * dk:ov], z[:, ov:ov + G * dv], z[:, ov + G * dv:]
+        mixed = a.v_mix and l != self.cfg.first_mix
+        head_prep_(z, H, G, dk, dv, q_gamma=P.w(p + "attn.q_norm"), k_gamma=P.w(p + "attn.k_norm"), eps=self.cfg.norm_eps,
+                   v_first=st.v_first if mixed else None, mix=P.w(p + "attn.mix") if mixed else None,
+                   k_cache=r.cache.k[l], v_cache=r.cache.v[l], slots=sb.slots)
+        if l == self.cfg.first_mix:
+            st.v_first = v2                            # a view: this layer's projection buffer stays alive
+        o = r.attend(l, z[:, :H * dk], k2, v2, sb, a.scale, self.rules[l], gate)
+        self._add_norm(st, gemm(o, P.w(p + "attn.out"), out_dtype=torch.float32), p + "norm1")
+        if s.mlp is not None:
+            self._experts(st, s.mlp, p)
+        return st
+
+    def _experts(self, st, m, p):
+        P, h = self.r.params, st.h
+        logits = gemm(h, P.w(p + "moe.router"), out_dtype=torch.float32)
+        idx, w = moe_ops.route_groups(logits, m.top, m.groups, m.keep)
+        pl = moe_ops.plan(idx, m.experts)
+        live = pl.offsets[m.experts:]
+        gu = moe_ops.grouped_gemm(moe_ops.gather(h, pl, zero_tail=False), P.w(p + "moe.w1"), pl)
+        y = moe_ops.grouped_gemm(moe_ops.swiglu_live(gu, live), P.w(p + "moe.w2"), pl)
+        shared = None
+        if m.shared_ff:
+            shared = gemm(moe_ops.swiglu_live(gemm(h, P.w(p + "shared.in"))), P.w(p + "shared.out"))
+        self._add_norm(st, y, p + "norm2", routed=(pl.slot_pos, w), add=shared)
+
+    def head(self, st, rows):
+        P, cfg = self.r.params, self.cfg
+        x = st.x if rows is None else ops.gather_rows(st.x, rows)
+        h = norm_ops.residual_norm(x, P.w("final.norm"), P.w("final.norm.b"), cfg.norm_eps, h=torch.empty_like(x, dtype=self.r.dtype))
+        logits = gemm(h, P.w("head"), out_dtype=torch.float32)
+        return ops.scale_softcap_(logits, cfg.logit_scale, cfg.logit_softcap)

@@ -105,8 +105,8 @@ class ServingEngine:
                 take = min(len(inp) - pos, budget)
                 budget -= take
                 chunks.append((rid, inp[pos:pos + take], pos, pos + take == len(inp)))
-        if chunks:
-            chunk_logits, dec_logits = self.runner.step_mixed(chunks, dec_ids, dec_tok, dec_len)
+        if chunks or dec_ids:
+            chunk_logits, dec_logits = self.runner.step(chunks, dec_ids, dec_tok, dec_len)
             for (rid, toks, pos, last), lg in zip(chunks, chunk_logits):
                 if last:
                     self._prefill_pos.pop(rid, None)
@@ -115,10 +115,6 @@ class ServingEngine:
                     self._prefill_pos[rid] = pos + len(toks)
             if dec_ids:
                 outputs.update(dict(zip(dec_ids, self.sampler.sample(dec_logits[:, :vocab]).tolist())))
-        elif dec_ids:
-            logits = self.runner.decode(dec_ids, dec_tok, dec_len)
-            toks = self.sampler.sample(logits[:, :vocab]).tolist()
-            outputs.update(dict(zip(dec_ids, toks)))
         if self.runner.device.type == "cuda":
             torch.cuda.current_stream().synchronize()
         sch.update(outputs, time.perf_counter())

@@ -166,11 +166,22 @@ class SlidingWindowCache(KVCache):
         return self._decode(self.k[:, :, idx], "k"), self._decode(self.v[:, :, idx], "v")
 
 
+@dataclass(frozen=True)
+class CacheLayer:
+    """What one layer stores per token: `kv_heads` keys of size `k_dim` and values of size `v_dim`."""
+    kv_heads: int
+    k_dim: int
+    v_dim: int
+
+
 class PagedCache:
-    """Paged KV storage for all layers plus per-sequence block tables."""
+    """Paged KV storage for all layers plus per-sequence block tables.  All layers share the tables; with `layers` every
+    layer has its own head count and key / value sizes, otherwise all are [num_kv_heads, head_dim]."""
 
     def __init__(self, num_blocks: int, block_size: int = 16, num_layers: int = 1, num_kv_heads: int = 1, head_dim: int = 64,
-                 dtype=torch.bfloat16, device="cpu", allocate_storage: bool = True):
+                 dtype=torch.bfloat16, device="cpu", allocate_storage: bool = True, layers: list | None = None):
+        if layers is not None:
+            num_layers = len(layers)
         self.block_size, self.num_blocks = block_size, num_blocks
         self.num_layers, self.num_kv_heads, self.head_dim = num_layers, num_kv_heads, head_dim
         self._lib = N.runtime()
@@ -178,7 +189,10 @@ class PagedCache:
         if not self._h:
             raise InvalidArgument("PagedCache: num_blocks and block_size must be positive")
         self.k = self.v = None
-        if allocate_storage:
+        if allocate_storage and layers is not None:
+            self.k = [torch.zeros((num_blocks, block_size, c.kv_heads, c.k_dim), dtype=dtype, device=device) for c in layers]
+            self.v = [torch.zeros((num_blocks, block_size, c.kv_heads, c.v_dim), dtype=dtype, device=device) for c in layers]
+        elif allocate_storage:
             shape = (num_layers, num_blocks, block_size, num_kv_heads, head_dim)
             self.k = torch.zeros(shape, dtype=dtype, device=device)
             self.v = torch.zeros(shape, dtype=dtype, device=device)
@@ -220,7 +234,7 @@ class PagedCache:
         return self._lib.rb_ba_num_sequences(self._h)
 
     def memory_bytes(self) -> int:
-        return 0 if self.k is None else 2 * self.k.numel() * self.k.element_size()
+        return 0 if self.k is None else sum(t.numel() * t.element_size() for c in (self.k, self.v) for t in c)
 
 
 class BatchedCache:

@@ -1,4 +1,4 @@
-"""Inference weights: bf16 only, optionally sharded for tensor parallelism, under the parameter names the model
+"""Inference weights (bf16; layered decoders also fp32), optionally sharded for tensor parallelism, under the parameter names the model
 runner uses.  Column-parallel matrices (QKV, gate/up, LM head) keep `1 / world` of their rows, row-parallel ones
 (attention output, down projection) `1 / world` of their columns; norms and the embedding are replicated."""
 from __future__ import annotations
@@ -103,3 +103,80 @@ class InferenceWeights:
             t[p + "ffn.gate_up.weight"] = torch.cat([gu[:F][rank * f:(rank + 1) * f], gu[F:][rank * f:(rank + 1) * f]], 0).contiguous()
             t[p + "ffn.down.weight"] = full.w(p + "ffn.down.weight")[:, rank * f:(rank + 1) * f].contiguous()
         return cls(t, full.lowp.dtype)
+
+    @classmethod
+    def layered(cls, cfg, device, dtype=None, tensors: dict | None = None, seed: int = 0) -> "InferenceWeights":
+        """Weights of a layered decoder (models.layered.LayeredConfig) in the layout of the serving kernels: one packed
+        attention projection [q | k | v | gate], experts stacked as [E, 2 ff, d] (gate over up) and [E, d, ff], the head
+        padded to whole GEMM tiles.  `tensors`: an unsharded checkpoint under `cfg.tensor_shapes()` names, loaded
+        strictly; None: random initialisation on the device.  `dtype`: bf16 or fp32 (default: bf16 on a GPU)."""
+        from ..core.errors import SerializationError, ShapeMismatch
+        dev = torch.device(device)
+        dt = dtype or (torch.bfloat16 if dev.type == "cuda" else torch.float32)
+        shapes = cfg.tensor_shapes()
+        if tensors is not None:
+            missing = [k for k in shapes if k not in tensors]
+            extra = [k for k in tensors if k not in shapes and k not in cfg.unused_tensors()]
+            if missing:
+                raise SerializationError(f"missing keys: {missing}")
+            if extra:
+                raise SerializationError(f"unexpected keys: {extra}")
+            for k, want in shapes.items():
+                if tuple(tensors[k].shape) != tuple(want) and tensors[k].numel() != math.prod(want):
+                    raise ShapeMismatch(want, tensors[k].shape, k)
+
+        def get(name):
+            shape = shapes[name]
+            if tensors is not None:
+                return tensors[name].reshape(shape).to(dev, dt)
+            if name.endswith("norm") or name.endswith("norm1") or name.endswith("norm2"):
+                return torch.ones(shape, dtype=dt, device=dev)
+            if name.endswith(".b"):
+                return torch.zeros(shape, dtype=dt, device=dev)
+            if name.endswith("vmix"):
+                return torch.full(shape, 0.5, dtype=dt, device=dev)
+            g = torch.Generator(device=dev).manual_seed(zlib.crc32(f"{seed}/{name}".encode()))
+            return torch.empty(shape, dtype=torch.float32, device=dev).normal_(0.0, cfg.init_std, generator=g).to(dt)
+
+        def gate_up(p, ff, out):
+            """gate rows over up rows; a hidden size that is not a multiple of 8 gets zero rows (silu(0) * 0 = 0)."""
+            f8 = out.shape[0] // 2
+            out[:ff] = get(p + "gate")
+            out[f8:f8 + ff] = get(p + "up")
+
+        def up8(n):
+            return (n + 7) // 8 * 8
+
+        d = cfg.d_model
+        t = {"embed": get("embed"), "head": torch.zeros((cfg.vocab_padded, d), dtype=dt, device=dev)}
+        t["head"][:cfg.vocab_size] = get("head")
+        t["final.norm"], t["final.norm.b"] = get("final.norm"), get("final.norm.b")
+        for i, s in enumerate(cfg.layers):
+            p, m = f"l{i}.", s.mlp
+            for nm in ("norm1", "norm1.b"):
+                t[p + nm] = get(p + nm)
+            t[p + "attn.in"] = torch.cat([get(p + "mix." + c) for c in "qkvg"], 0)
+            t[p + "attn.out"] = get(p + "mix.o")
+            t[p + "attn.q_norm"], t[p + "attn.k_norm"] = get(p + "mix.q.norm"), get(p + "mix.k.norm")
+            if s.mixer.v_mix:
+                t[p + "attn.mix"] = get(p + "mix.vmix").float().reshape(1).contiguous()
+            if m is None:
+                continue
+            for nm in ("norm2", "norm2.b"):
+                t[p + nm] = get(p + nm)
+            t[p + "moe.router"] = get(p + "mlp.router")
+            f8 = up8(m.ff)
+            w1 = torch.zeros((m.experts, 2 * f8, d), dtype=dt, device=dev)
+            w2 = torch.zeros((m.experts, d, f8), dtype=dt, device=dev)
+            for e in range(m.experts):
+                gate_up(f"{p}mlp.e{e}.", m.ff, w1[e])
+                w2[e, :, :m.ff] = get(f"{p}mlp.e{e}.down")
+            t[p + "moe.w1"], t[p + "moe.w2"] = w1, w2
+            if m.shared_ff:
+                f8 = up8(m.shared_ff)
+                w1 = torch.zeros((2 * f8, d), dtype=dt, device=dev)
+                gate_up(p + "mlp.shared.", m.shared_ff, w1)
+                w2 = torch.zeros((d, f8), dtype=dt, device=dev)
+                w2[:, :m.shared_ff] = get(p + "mlp.shared.down")
+                t[p + "shared.in"], t[p + "shared.out"] = w1, w2
+        return cls(t, dt)
