@@ -19,6 +19,19 @@ typedef struct RbAttnArgs {
   const int* kv_lens;      // optional [batch]: keys at positions >= kv_lens[b] are padding and invisible (NULL: all seq_k
                            // keys are real).  Taken by the "tc2" kernels; the others return -9 when it is set.
 } RbAttnArgs;
+// Score rule of an inference forward pass (causal, queries aligned to the end of the keys, key 0 is the start of a chunk):
+//   s = q . k * scale; softcap > 0: s <- softcap * tanh(s / softcap); slopes (fp32 [heads]): s <- s - slopes[h] * (i - j);
+//   chunk > 0: i sees j only when i / chunk == j / chunk; gate (bf16 [seq_q, heads * v_dim], pitch ld_gate, batch 1):
+//   the output is multiplied by sigmoid(gate)
+typedef struct RbAttnRule {
+  int v_dim;               // value head size (RbAttnArgs.head_dim is the query / key size)
+  float softcap;
+  const float* slopes;
+  int chunk;
+  const void* gate;
+  long long ld_gate;
+} RbAttnRule;
+int rb_attention_fwd_rule(const RbAttnArgs* args, const RbAttnRule* rule, void* stream);
 int rb_attention_fwd(const RbAttnArgs* args, void* stream);
 int rb_attention_bwd(const RbAttnArgs* args, void* stream);
 // tcgen05 paths (attention_tc.cu, attention_fwd2.cu, attention_bwd_tc.cu, attention_bwd2.cu); -9: shape not taken

@@ -13,6 +13,10 @@
 // bounded by 256, exact after the final division by the row sum).  A share of the exponentials can be computed with a
 // polynomial on the FMA pipe (template parameter; off by default, see rb_attention_fwd_tc2).  Warp 8 is the TMA producer (Q once, K / V through a ring of stages), warp 9 issues MMAs.
 //
+// The RULE form serves inference of decoders with their own score rule: separate key / value head sizes (columns beyond the
+// real sizes are zero-filled by TMA), capped scores, a linear distance bias, chunked visibility (key blocks before a
+// tile's first visible chunk are skipped, so the two tiles may start at different blocks) and a sigmoid output gate.
+//
 // Same semantics as the other forward kernels (causal alignment to the end of the keys, GQA, log-sum-exp output).
 // Replaces the reference's materialised-score attention (crates/nn/src/attention.rs:640-836).
 #include "attention.h"
@@ -33,11 +37,23 @@ struct F2Params {
   int seq_q, seq_k, heads, kv_heads, causal;
   float scale;
   const int* kv_lens;       // optional [batch]: number of real keys
+  // RULE kernels only
+  int dk, dv;               // real head sizes
+  float softcap;            // 0: none
+  const float* slopes;      // [heads] or NULL
+  int chunk;                // 0: none; key 0 starts a chunk
+  const __nv_bfloat16* gate;   // [seq_q, heads * dv] or NULL
+  long long ld_gate;
 };
 
 __device__ __forceinline__ float f2_ex2(float x) {
   float y;
   asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+__device__ __forceinline__ float f2_rcp(float x) {
+  float y;
+  asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
   return y;
 }
 // 2^x on the FMA / integer pipes: round-to-nearest split x = n + f, |f| <= 0.5, degree-4 polynomial for 2^f
@@ -84,24 +100,25 @@ __device__ __forceinline__ void tmem_ld_32x32_ptr(uint32_t taddr, uint32_t* r) {
       : "memory");
 }
 
-template <int D>
+template <int D, int DV>
 struct F2Smem {
-  static constexpr int kStages = D == 64 ? 4 : 2;
+  static constexpr int kStages = D == 64 && DV == 64 ? 4 : D == 128 && DV == 128 ? 2 : 3;
   static constexpr int kHalf = kF2Tile * 128;                 // one 64-column swizzle atom: 128 rows x 128 B
-  static constexpr int kTileBytes = (D / 64) * kHalf;         // a 128-row tile of Q, K or V
+  static constexpr int kTileBytes = (D / 64) * kHalf;         // a 128-row tile of Q or K
+  static constexpr int kVTileBytes = (DV / 64) * kHalf;       // a 128-row tile of V
   static constexpr int kQ = 0;                                // two tiles
   static constexpr int kK = kQ + 2 * kTileBytes;
   static constexpr int kV = kK + kStages * kTileBytes;
-  static constexpr int kBar = kV + kStages * kTileBytes;
+  static constexpr int kBar = kV + kStages * kVTileBytes;
   static constexpr int kNumBars = 2 + 3 * kStages + 6;        // q[2], k_full/v_full/kv_empty[stages], s_full[2], p_full[2], o_ready[2]
   static constexpr int kTotal = kBar + kNumBars * 8 + 16;
 };
 
-template <int D, int kPolyEvery>
+template <int D, int DV, int kPolyEvery, bool RULE>
 __global__ void __launch_bounds__(kF2Threads, 1)
 attn_fwd2_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK,
                  const __grid_constant__ CUtensorMap tmV, F2Params p, unsigned int* status) {
-  using L = F2Smem<D>;
+  using L = F2Smem<D, DV>;
   constexpr int kStages = L::kStages;
   extern __shared__ __align__(1024) uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
@@ -140,6 +157,14 @@ attn_fwd2_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
   const int n_a = blocks_of(q0), n_b = blocks_of(q0 + kF2Tile);
   auto n_of = [&](int t) { return t == 0 ? n_a : n_b; };
   const int n_max = n_a > n_b ? n_a : n_b;
+  // first key block of each tile: the one that holds the start of its first row's chunk.  Tile A starts first, and tile B
+  // starts no later than one block after tile A's last.
+  auto first_of = [&](int t) {
+    return RULE && p.chunk > 0 ? (q0 + t * kF2Tile + shift) / p.chunk * p.chunk / kF2Tile : 0;
+  };
+  const int f_a = first_of(0), f_b = first_of(1);
+  auto f_of = [&](int t) { return t == 0 ? f_a : f_b; };
+  const int f_min = n_a > 0 ? f_a : f_b;
   constexpr uint32_t kTmemCols = 512;
 
   if (threadIdx.x == 0) {
@@ -182,30 +207,31 @@ attn_fwd2_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
         for (int hf = 0; hf < D / 64; ++hf)
           tma_load_4d(sQ + t * L::kTileBytes + hf * L::kHalf, &tmQ, hf * 64, h, q0 + t * kF2Tile, b, bar_q + 8 * t);
       }
-      for (int j = 0; j < n_max; ++j) {
-        const int s = j % kStages, use = j / kStages;
+      for (int j = f_min; j < n_max; ++j) {
+        const int s = (j - f_min) % kStages, use = (j - f_min) / kStages;
         if (!mbar_wait(bar_kvempty + 8 * s, (use & 1) ^ 1, abort_flag, status, 41)) break;
         mbar_arrive_expect_tx(bar_kfull + 8 * s, L::kTileBytes);
 #pragma unroll
         for (int hf = 0; hf < D / 64; ++hf)
           tma_load_4d(sK + s * L::kTileBytes + hf * L::kHalf, &tmK, hf * 64, hk, j * kF2Tile, b, bar_kfull + 8 * s);
-        mbar_arrive_expect_tx(bar_vfull + 8 * s, L::kTileBytes);
+        mbar_arrive_expect_tx(bar_vfull + 8 * s, L::kVTileBytes);
 #pragma unroll
-        for (int hf = 0; hf < D / 64; ++hf)
-          tma_load_4d(sV + s * L::kTileBytes + hf * L::kHalf, &tmV, hf * 64, hk, j * kF2Tile, b, bar_vfull + 8 * s);
+        for (int hf = 0; hf < DV / 64; ++hf)
+          tma_load_4d(sV + s * L::kVTileBytes + hf * L::kHalf, &tmV, hf * 64, hk, j * kF2Tile, b, bar_vfull + 8 * s);
       }
     }
   } else if (warp == 9) {
     if (lane == 0) {
       // ---------------------------------------------------------------- MMA issuer
       constexpr uint32_t idesc_qk = umma_idesc_bf16(128, 128, 0, 0);
-      constexpr uint32_t idesc_pv = umma_idesc_bf16(128, D, 0, 1);        // A = P (TMEM, K-major), B = V MN-major
+      constexpr uint32_t idesc_pv = umma_idesc_bf16(128, DV, 0, 1);        // A = P (TMEM, K-major), B = V MN-major
       auto issue_qk = [&](int j, int t) -> bool {
-        const int s = j % kStages;
-        if (!mbar_wait(bar_kfull + 8 * s, (j / kStages) & 1, abort_flag, status, 42)) return false;
+        const int s = (j - f_min) % kStages;
+        if (!mbar_wait(bar_kfull + 8 * s, ((j - f_min) / kStages) & 1, abort_flag, status, 42)) return false;
         tc_fence_after();
 #pragma unroll
         for (int ks = 0; ks < D / 16; ++ks) {
+          if (RULE && ks * 16 >= p.dk) break;               // the rest of the columns is zero
           const uint32_t off = (ks >> 2) * L::kHalf + (ks & 3) * 32;
           umma_bf16_ss(tmem_base + t * 128, umma_smem_desc_sw128(sQ + t * L::kTileBytes + off, 16, 1024),
                        umma_smem_desc_sw128(sK + s * L::kTileBytes + off, 16, 1024), idesc_qk, ks != 0 ? 1u : 0u);
@@ -218,23 +244,27 @@ attn_fwd2_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
       for (int t = 0; t < 2; ++t) {
         if (n_of(t) == 0 || !ok) continue;
         ok = mbar_wait(bar_q + 8 * t, 0, abort_flag, status, 43);
-        if (ok) ok = issue_qk(0, t);
+        if (ok && f_of(t) == f_min) ok = issue_qk(f_min, t);  // a tile that starts later gets its first product below
       }
-      for (int j = 0; j < n_max && ok; ++j) {
-        const int s = j % kStages;
-        if (!mbar_wait(bar_vfull + 8 * s, (j / kStages) & 1, abort_flag, status, 44)) break;
+      for (int j = f_min; j < n_max && ok; ++j) {
+        const int s = (j - f_min) % kStages;
+        if (!mbar_wait(bar_vfull + 8 * s, ((j - f_min) / kStages) & 1, abort_flag, status, 44)) break;
 #pragma unroll
         for (int t = 0; t < 2; ++t) {
           if (j >= n_of(t) || !ok) continue;
-          if (!mbar_wait(bar_pfull + 8 * t, j & 1, abort_flag, status, 45)) { ok = false; break; }
+          if (j < f_of(t)) {
+            if (j + 1 == f_of(t)) ok = issue_qk(j + 1, t);
+            continue;
+          }
+          if (!mbar_wait(bar_pfull + 8 * t, (j - f_of(t)) & 1, abort_flag, status, 45)) { ok = false; break; }
           tc_fence_after();
           const uint32_t tmem_p = tmem_base + t * 128;              // packed bf16 pairs: 8 columns per 16 keys
           const uint32_t tmem_o = tmem_base + 256 + t * 128;
 #pragma unroll
           for (int ks = 0; ks < kF2Tile / 16; ++ks) {
             // V: 16 key rows of 128 B per step; 64-wide head-dim atoms L::kHalf apart
-            const uint64_t db = umma_smem_desc_sw128(sV + s * L::kTileBytes + ks * 2048, L::kHalf, 1024);
-            umma_bf16_ts(tmem_o, tmem_p + ks * 8, db, idesc_pv, (j > 0 || ks != 0) ? 1u : 0u);
+            const uint64_t db = umma_smem_desc_sw128(sV + s * L::kVTileBytes + ks * 2048, L::kHalf, 1024);
+            umma_bf16_ts(tmem_o, tmem_p + ks * 8, db, idesc_pv, (j > f_of(t) || ks != 0) ? 1u : 0u);
           }
           umma_commit(bar_oready + 8 * t);
           if (j + 1 < n_of(t)) ok = issue_qk(j + 1, t);          // overwrites S_t / P_t: ordered behind PV(j, t)
@@ -253,12 +283,17 @@ attn_fwd2_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
     const uint32_t lane_off = static_cast<uint32_t>(wq * 32) << 16;
     const uint32_t tmem_s = tmem_base + t * 128 + lane_off;
     const uint32_t tmem_o = tmem_base + 256 + t * 128 + lane_off;
-    const float sl2 = p.scale * kF2Log2e;
+    // RULE: scores are turned into log2 units when they are read (cap, bias), so the softmax runs with scale 1
+    const float sl2 = RULE ? 1.f : p.scale * kF2Log2e;
+    const float rule_c1 = RULE && p.softcap > 0.f ? 2.f * p.scale / p.softcap * kF2Log2e : 0.f;
+    const float rule_c2 = RULE ? (p.softcap > 0.f ? p.softcap : p.scale) * kF2Log2e : 0.f;
+    const float slope2 = RULE && p.slopes ? p.slopes[h] * kF2Log2e : 0.f;
+    const int key_lo = RULE && p.chunk > 0 ? (q_idx + shift) / p.chunk * p.chunk : 0;      // first visible key of this row
     float m_run = -INFINITY, l_run = 0.f;
-    const int nt = n_of(t);
+    const int nt = n_of(t), ft = f_of(t);
     bool ok = true;
-    for (int j = 0; j < nt && ok; ++j) {
-      if (!mbar_wait(bar_sfull + 8 * t, j & 1, abort_flag, status, 46)) { ok = false; break; }
+    for (int j = ft; j < nt && ok; ++j) {
+      if (!mbar_wait(bar_sfull + 8 * t, (j - ft) & 1, abort_flag, status, 46)) { ok = false; break; }
       tc_fence_after();
       const int k0 = j * kF2Tile;
       const int key_lim = p.causal ? min(kv_len - 1, q_idx + shift) : kv_len - 1;     // last visible key
@@ -280,6 +315,26 @@ attn_fwd2_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
 #pragma unroll
       for (int c = 0; c < 4; ++c) tmem_ld_32x32_ptr(tmem_s + c * 32, r + c * 32);
       tmem_ld_wait();
+      if (RULE) {
+        // cap * tanh(s / cap) = cap - 2 cap / (1 + e^(2 s / cap)); then - slope * (query - key)
+        const float bias0 = -slope2 * static_cast<float>(q_idx + shift - k0);
+        if (p.softcap > 0.f) {
+#pragma unroll
+          for (int i = 0; i < 128; ++i) {
+            const float e = f2_ex2(__uint_as_float(r[i]) * rule_c1);
+            r[i] = __float_as_uint(fmaf(-2.f * rule_c2, f2_rcp(1.f + e), rule_c2 + fmaf(slope2, static_cast<float>(i), bias0)));
+          }
+        } else {
+#pragma unroll
+          for (int i = 0; i < 128; ++i)
+            r[i] = __float_as_uint(fmaf(__uint_as_float(r[i]), rule_c2, fmaf(slope2, static_cast<float>(i), bias0)));
+        }
+        if (k0 < key_lo) {
+#pragma unroll
+          for (int i = 0; i < 128; ++i)
+            if (k0 + i < key_lo) r[i] = 0xff800000u;
+        }
+      }
       if (need_mask) {                               // only blocks that cross the causal diagonal or the end of the keys
 #pragma unroll
         for (int i = 0; i < 128; ++i)
@@ -296,12 +351,12 @@ attn_fwd2_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
         m_run = mx;
         l_run *= alpha;
       }
-      if (j > 0 && __any_sync(0xffffffffu, grow)) {
+      if (j > ft && __any_sync(0xffffffffu, grow)) {
         // O_t holds the sum over blocks 0..j-1 once PV(j-1, t) has completed; PV(j, t) cannot start before P below.
-        if (!mbar_wait(bar_oready + 8 * t, (j - 1) & 1, abort_flag, status, 47)) { ok = false; break; }
+        if (!mbar_wait(bar_oready + 8 * t, (j - 1 - ft) & 1, abort_flag, status, 47)) { ok = false; break; }
         tc_fence_after();
 #pragma unroll
-        for (int c = 0; c < D / 32; ++c) {
+        for (int c = 0; c < DV / 32; ++c) {
           uint32_t o[32];
           tmem_ld_32x32_ptr(tmem_o + c * 32, o);
           tmem_ld_wait();
@@ -351,12 +406,13 @@ attn_fwd2_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
       __syncwarp();
       if (lane == 0) mbar_arrive(bar_pfull + 8 * t);
     }
-    if (ok && nt > 0) ok = mbar_wait(bar_oready + 8 * t, (nt - 1) & 1, abort_flag, status, 48);
+    if (ok && nt > 0) ok = mbar_wait(bar_oready + 8 * t, (nt - 1 - ft) & 1, abort_flag, status, 48);
     if (nt == 0 && q_idx < p.seq_q && q0 + t * kF2Tile < p.seq_q) {
       // no visible key at all (every key of this batch entry is padding): the output row is zero
       __nv_bfloat16* op = p.out + b * p.o_bs + h * p.o_hs + static_cast<long long>(q_idx) * p.o_rs;
 #pragma unroll
-      for (int c = 0; c < D / 8; ++c) reinterpret_cast<uint4*>(op)[c] = make_uint4(0u, 0u, 0u, 0u);
+      for (int c = 0; c < DV / 8; ++c)
+        if (!RULE || c * 8 < p.dv) reinterpret_cast<uint4*>(op)[c] = make_uint4(0u, 0u, 0u, 0u);
       if (p.lse != nullptr) p.lse[(static_cast<long long>(b) * p.heads + h) * p.seq_q + q_idx] = 0.f;
     }
     if (ok && nt > 0) {
@@ -364,13 +420,24 @@ attn_fwd2_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
       const float inv = l_run > 0.f ? 1.f / l_run : 0.f;
       __nv_bfloat16* op = p.out + b * p.o_bs + h * p.o_hs + static_cast<long long>(q_idx) * p.o_rs;
 #pragma unroll
-      for (int c = 0; c < D / 32; ++c) {
+      for (int c = 0; c < DV / 32; ++c) {
         uint32_t o[32];
         tmem_ld_32x32_ptr(tmem_o + c * 32, o);
         tmem_ld_wait();
         if (q_idx < p.seq_q) {
 #pragma unroll
           for (int g = 0; g < 4; ++g) {
+            if (RULE && c * 32 + g * 8 >= p.dv) break;
+            if (RULE && p.gate != nullptr) {
+              const uint4 gv = *reinterpret_cast<const uint4*>(p.gate + q_idx * p.ld_gate + h * p.dv + c * 32 + g * 8);
+              const uint32_t gw[4] = {gv.x, gv.y, gv.z, gv.w};
+#pragma unroll
+              for (int i = 0; i < 4; ++i) {
+                const float2 f = unpack_bf16x2(gw[i]);
+                o[g * 8 + 2 * i] = __float_as_uint(__uint_as_float(o[g * 8 + 2 * i]) * f2_rcp(1.f + f2_ex2(-f.x * kF2Log2e)));
+                o[g * 8 + 2 * i + 1] = __float_as_uint(__uint_as_float(o[g * 8 + 2 * i + 1]) * f2_rcp(1.f + f2_ex2(-f.y * kF2Log2e)));
+              }
+            }
             uint4 v;
             v.x = pack_bf16x2(__uint_as_float(o[g * 8 + 0]) * inv, __uint_as_float(o[g * 8 + 1]) * inv);
             v.y = pack_bf16x2(__uint_as_float(o[g * 8 + 2]) * inv, __uint_as_float(o[g * 8 + 3]) * inv);
@@ -410,11 +477,11 @@ const CUtensorMap* f2_make_map(const void* base, const long long* strides, int s
   return rbhost::get_tmap_4d(base, 2, dims, str, box, 1, err);
 }
 
-template <int D, int P>
+template <int D, int DV, int P, bool RULE>
 int f2_launch(const CUtensorMap* tq, const CUtensorMap* tk, const CUtensorMap* tv, const rb::F2Params& p, dim3 grid,
               cudaStream_t stream) {
-  auto kern = rb::attn_fwd2_kernel<D, P>;
-  const int smem = rb::F2Smem<D>::kTotal + 1024;
+  auto kern = rb::attn_fwd2_kernel<D, DV, P, RULE>;
+  const int smem = rb::F2Smem<D, DV>::kTotal + 1024;
   static bool cfg_dev[64] = {false};
   bool& cfg = cfg_dev[rbhost::device_slot()];
   if (!cfg) {
@@ -452,7 +519,7 @@ RB_API int rb_attention_fwd_tc2(const RbAttnArgs* a, int poly_every, void* strea
   const CUtensorMap* tk = f2_make_map(a->k, ks, a->seq_k, a->kv_heads, a->batch, a->head_dim, &err);
   const CUtensorMap* tv = f2_make_map(a->v, vs, a->seq_k, a->kv_heads, a->batch, a->head_dim, &err);
   if (!tq || !tk || !tv) return err ? err : -5;
-  rb::F2Params p;
+  rb::F2Params p = {};
   p.out = reinterpret_cast<__nv_bfloat16*>(a->o);
   p.lse = a->lse;
   p.o_bs = a->o_strides[0]; p.o_rs = a->o_strides[1]; p.o_hs = a->o_strides[2];
@@ -463,14 +530,47 @@ RB_API int rb_attention_fwd_tc2(const RbAttnArgs* a, int poly_every, void* strea
   dim3 grid((a->seq_q + 2 * rb::kF2Tile - 1) / (2 * rb::kF2Tile), a->heads, a->batch);
   if (a->head_dim == 64) {
     switch (poly_every) {
-      case 0: return f2_launch<64, 0>(tq, tk, tv, p, grid, stream);
-      case 4: return f2_launch<64, 4>(tq, tk, tv, p, grid, stream);
+      case 0: return f2_launch<64, 64, 0, false>(tq, tk, tv, p, grid, stream);
+      case 4: return f2_launch<64, 64, 4, false>(tq, tk, tv, p, grid, stream);
       default: return -1;
     }
   }
   switch (poly_every) {
-    case 0: return f2_launch<128, 0>(tq, tk, tv, p, grid, stream);
-    case 4: return f2_launch<128, 4>(tq, tk, tv, p, grid, stream);
+    case 0: return f2_launch<128, 128, 0, false>(tq, tk, tv, p, grid, stream);
+    case 4: return f2_launch<128, 128, 4, false>(tq, tk, tv, p, grid, stream);
     default: return -1;
   }
+}
+
+// Causal forward with a score rule (see attention.h).  Returns -9 for operands this kernel does not take.
+RB_API int rb_attention_fwd_rule(const RbAttnArgs* a, const RbAttnRule* r, void* stream_v) {
+  const int dk = a->head_dim, dv = r->v_dim;
+  if (a->batch <= 0 || a->heads <= 0 || a->kv_heads <= 0 || a->heads % a->kv_heads) return -1;
+  if (dk <= 0 || dv <= 0 || dk > 128 || dv > 128 || ((dk | dv) & 7)) return -9;
+  if (!a->causal || a->seq_q <= 0 || a->seq_k < a->seq_q || r->chunk < 0 || (r->gate && a->batch != 1)) return -1;
+  const void* ptrs[5] = {a->q, a->k, a->v, a->o, r->gate};
+  for (int i = 0; i < 5; ++i)
+    if ((!ptrs[i] && i < 4) || (reinterpret_cast<uintptr_t>(ptrs[i]) & 15)) return -9;
+  const long long* strs[4] = {a->q_strides, a->k_strides, a->v_strides, a->o_strides};
+  for (int i = 0; i < 4; ++i)
+    for (int j = 0; j < 3; ++j)
+      if (strs[i][j] % 8 || strs[i][j] <= 0) return -9;            // TMA strides are multiples of 16 bytes
+  if (r->ld_gate % 8) return -9;
+  int err = 0;
+  const CUtensorMap* tq = f2_make_map(a->q, a->q_strides, a->seq_q, a->heads, a->batch, dk, &err);
+  const CUtensorMap* tk = f2_make_map(a->k, a->k_strides, a->seq_k, a->kv_heads, a->batch, dk, &err);
+  const CUtensorMap* tv = f2_make_map(a->v, a->v_strides, a->seq_k, a->kv_heads, a->batch, dv, &err);
+  if (!tq || !tk || !tv) return err ? err : -5;
+  rb::F2Params p = {};
+  p.out = reinterpret_cast<__nv_bfloat16*>(a->o);
+  p.o_bs = a->o_strides[0]; p.o_rs = a->o_strides[1]; p.o_hs = a->o_strides[2];
+  p.seq_q = a->seq_q; p.seq_k = a->seq_k; p.heads = a->heads; p.kv_heads = a->kv_heads; p.causal = 1;
+  p.scale = a->scale;
+  p.dk = dk; p.dv = dv; p.softcap = r->softcap; p.slopes = r->slopes; p.chunk = r->chunk;
+  p.gate = reinterpret_cast<const __nv_bfloat16*>(r->gate); p.ld_gate = r->ld_gate;
+  cudaStream_t stream = reinterpret_cast<cudaStream_t>(stream_v);
+  const dim3 grid((a->seq_q + 2 * rb::kF2Tile - 1) / (2 * rb::kF2Tile), a->heads, a->batch);
+  if (dk <= 64)
+    return dv <= 64 ? f2_launch<64, 64, 0, true>(tq, tk, tv, p, grid, stream) : f2_launch<64, 128, 0, true>(tq, tk, tv, p, grid, stream);
+  return dv <= 64 ? f2_launch<128, 64, 0, true>(tq, tk, tv, p, grid, stream) : f2_launch<128, 128, 0, true>(tq, tk, tv, p, grid, stream);
 }

@@ -63,6 +63,10 @@ __device__ __forceinline__ uint32_t pa_pack_bf16(float lo, float hi) {
   return *reinterpret_cast<uint32_t*>(&v);
 }
 
+template <int N>
+struct PaInt { static constexpr int value = N; };
+__device__ __forceinline__ float pa_sigmoid(float x) { return __fdividef(1.f, 1.f + __expf(-x)); }
+
 // Split-KV decode attention.  One CTA = (sequence, KV head, 256-token slice of the context); the slices of a sequence
 // run on different SMs and a second kernel merges their (max, sum, accumulator) triples.  Inside a CTA a warp takes
 // 32 tokens at a time.  Their K rows and V rows are fetched with fully coalesced 16-byte asynchronous copies (cp.async,
@@ -73,41 +77,66 @@ __device__ __forceinline__ uint32_t pa_pack_bf16(float lo, float hi) {
 // k-steps of mma.sync, the softmax runs on the accumulator fragments, and O += P V reuses those fragments as the A
 // operand against ldmatrix.trans-fed V.  One query token per sequence gives M <= 16, far below the 64-row minimum
 // of a tcgen05 tile, which is why this kernel is on the warp-level tensor path; it is bound by the K / V reads.
-template <int D>
+//
+// DK / DV are the key / value head sizes rounded up to a compiled size; columns beyond the real sizes are zero-filled in
+// shared memory and never leave it.  RULE adds a score cap, a distance bias and chunked visibility (see RbPagedRowsArgs).
+struct PaRule {
+  float softcap;
+  const float* slopes;
+  int chunk;
+  const __nv_bfloat16* gate;
+  long long ld_g;
+};
+// cap * tanh(s / cap) as cap * (1 - 2 / (1 + e^(2 s / cap))): two special-function instructions, absolute error about
+// 1e-7 * cap (tanh.approx would be off by 5e-4 of the score)
+__device__ __forceinline__ float pa_softcap(float s, float cap, float two_over_cap) {
+  return fmaf(-2.f * cap, __fdividef(1.f, 1.f + __expf(s * two_over_cap)), cap);
+}
+__device__ __forceinline__ int pa_first_key(int ctx, int chunk) { return chunk > 0 ? (ctx - 1) / chunk * chunk : 0; }
+
+template <int DK, int DV, bool RULE>
 __global__ void __launch_bounds__(kPaWarps * 32, 3)
 paged_decode_split_kernel(const __nv_bfloat16* __restrict__ q, long long ld_q, const __nv_bfloat16* __restrict__ k_cache,
                           const __nv_bfloat16* __restrict__ v_cache, const int* __restrict__ block_tables, int max_blocks,
-                          const int* __restrict__ context_lens, int heads, int kv_heads, int block_size,
-                          long long num_blocks, float scale, int g0, int gcount, float* __restrict__ partial, int nsplit
+                          const int* __restrict__ context_lens, int heads, int kv_heads, int dk_real, int dv_real,
+                          int block_size, long long num_blocks, float scale, int g0, int gcount, float* __restrict__ partial,
+                          int nsplit, __nv_bfloat16* __restrict__ direct_out, long long ld_o, const PaRule rule
                           RB_BOUNDS_PARAM) {
-  constexpr int LPR = D / 8;                 // lanes per K / V row (16-byte pieces)
-  constexpr int RPI = 32 / LPR;              // rows fetched per warp instruction
-  constexpr int NLD = 32 / RPI;              // load instructions per 32-row tile
-  constexpr int KROW = D + 8;                // padded row (elements): ldmatrix rows 272 (144) bytes apart hit distinct banks
-  constexpr int NT = D / 8;                  // n-tiles of the output accumulator
-  constexpr int kTileElems = 32 * KROW;      // one K or V tile of one warp
+  constexpr int LPK = DK / 8, LPV = DV / 8;  // 16-byte pieces per K / V row = copies per lane for a 32-row tile
+  constexpr int KROW = DK + 8, VROW = DV + 8;  // padded rows (elements): ldmatrix rows 272 (144) bytes apart hit distinct banks
+  constexpr int NT = DV / 8;                 // n-tiles of the output accumulator
+  constexpr int kKTile = 32 * KROW, kVTile = 32 * VROW;   // one tile of one warp
+  const int dk = RULE ? dk_real : DK, dv = RULE ? dv_real : DV;
   extern __shared__ __align__(16) uint8_t big[];   // [warp][K tile, V tile] bf16, then q_sh; later the warp merge area
-  __nv_bfloat16* q_sh = reinterpret_cast<__nv_bfloat16*>(big) + kPaWarps * 2 * kTileElems;
+  __nv_bfloat16* q_sh = reinterpret_cast<__nv_bfloat16*>(big) + kPaWarps * (kKTile + kVTile);
   __shared__ float m_sh[kPaWarps][kMaxGroup], l_sh[kPaWarps][kMaxGroup];
   const int b = blockIdx.x, hk = blockIdx.y, sp = blockIdx.z;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int gq = lane >> 2, tq = lane & 3;   // fragment coordinates: row (and row + 8), column pair
   const int group = heads / kv_heads;
   const int ctx = context_lens[b];
-  const int t_begin = sp * kSplitTokens;
+  const int t_begin = (RULE ? pa_first_key(ctx, rule.chunk) : 0) + sp * kSplitTokens;
   if (t_begin >= ctx) return;
   const int t_end = min(ctx, t_begin + kSplitTokens);
   const int h_base = hk * group + g0;        // first query head of this pass
-  const uint32_t kt_u32 = smem_u32(reinterpret_cast<__nv_bfloat16*>(big) + warp * 2 * kTileElems);
-  const uint32_t vt_u32 = kt_u32 + kTileElems * 2;
+  const uint32_t kt_u32 = smem_u32(reinterpret_cast<__nv_bfloat16*>(big) + warp * (kKTile + kVTile));
+  const uint32_t vt_u32 = kt_u32 + kKTile * 2;
   const uint32_t q_u32 = smem_u32(q_sh);
+  float slope0 = 0.f, slope1 = 0.f, two_over_cap = 0.f;
+  if (RULE) {
+    if (rule.slopes) {
+      if (gq < gcount) slope0 = rule.slopes[h_base + gq];
+      if (gq + 8 < gcount) slope1 = rule.slopes[h_base + gq + 8];
+    }
+    if (rule.softcap > 0.f) two_over_cap = 2.f / rule.softcap;
+  }
 
   // the group's query rows as bf16 [16][D] (rows >= gcount are zero)
-  for (int i = threadIdx.x; i < kMaxGroup * LPR; i += blockDim.x) {
-    const int g = i / LPR, c = (i - g * LPR) * 8;
+  for (int i = threadIdx.x; i < kMaxGroup * LPK; i += blockDim.x) {
+    const int g = i / LPK, c = (i - g * LPK) * 8;
     uint4 u = make_uint4(0u, 0u, 0u, 0u);
-    if (g < gcount) {
-      const __nv_bfloat16* src = q + static_cast<long long>(b) * ld_q + static_cast<long long>(h_base + g) * D + c;
+    if (g < gcount && c < dk) {
+      const __nv_bfloat16* src = q + static_cast<long long>(b) * ld_q + static_cast<long long>(h_base + g) * dk + c;
       uint32_t w[4];
 #pragma unroll
       for (int j = 0; j < 4; ++j) w[j] = *reinterpret_cast<const uint32_t*>(src + 2 * j);   // rows are 4-byte aligned at least
@@ -122,16 +151,12 @@ paged_decode_split_kernel(const __nv_bfloat16* __restrict__ q, long long ld_q, c
 #pragma unroll
   for (int n = 0; n < NT; ++n) acc[n][0] = acc[n][1] = acc[n][2] = acc[n][3] = 0.f;
 
-  const long long row = static_cast<long long>(kv_heads) * D;          // elements per cached token
-  const int piece = (lane % LPR) * 8;
-  const long long col = static_cast<long long>(hk) * D + piece;
-  const uint32_t dst_off = ((lane / LPR) * KROW + piece) * 2;          // byte offset of this lane's piece in a tile
-  int srow[NLD];                                                       // cache slot of the row behind each copy (-1: none)
+  int slot = -1;                             // cache slot of token `first + lane` of the located tile (-1: past the end)
   int n_next = 0;
   // cache slots of the 32 tokens that start at `first` (the host bounds num_blocks * block_size below 2^31)
   auto locate = [&](int first) {
     const int tok = first + lane;
-    int slot = 0;
+    slot = -1;
     if (tok < t_end) {
       const int blk_idx = tok / block_size;
       int blk = blk_idx < max_blocks ? block_tables[static_cast<long long>(b) * max_blocks + blk_idx] : -1;
@@ -142,27 +167,29 @@ paged_decode_split_kernel(const __nv_bfloat16* __restrict__ q, long long ld_q, c
       slot = blk * block_size + (tok - blk_idx * block_size);
     }
     n_next = min(32, t_end - first);
-#pragma unroll
-    for (int i = 0; i < NLD; ++i) {
-      const int r = i * RPI + lane / LPR;
-      const int slot_r = __shfl_sync(0xffffffffu, slot, r);
-      srow[i] = r < n_next ? slot_r : -1;
-    }
   };
-  // one tile = NLD asynchronous 16-byte copies per lane, one commit group; rows past the context are zero-filled
-  auto request = [&](const __nv_bfloat16* cache, uint32_t tile_u32) {
+  // one tile = one asynchronous 16-byte copy per lane and piece, one commit group; rows past the context and columns past
+  // the real head size are zero-filled
+  auto request = [&](const __nv_bfloat16* cache, uint32_t tile_u32, auto pieces, int dim) {
+    constexpr int LP = decltype(pieces)::value;
 #pragma unroll
-    for (int i = 0; i < NLD; ++i) {
-      const bool ok = srow[i] >= 0;
-      pa_cp_async16(tile_u32 + dst_off + i * RPI * KROW * 2, ok ? cache + srow[i] * row + col : cache, ok ? 16 : 0);
+    for (int i = 0; i < LP; ++i) {
+      const int idx = i * 32 + lane;
+      const int r = idx / LP, c = (idx - r * LP) * 8;
+      const int s_r = __shfl_sync(0xffffffffu, slot, r);
+      const bool ok = s_r >= 0 && c < dim;
+      pa_cp_async16(tile_u32 + (r * (LP * 8 + 8) + c) * 2,
+                    ok ? cache + (static_cast<long long>(s_r) * kv_heads + hk) * dim + c : cache, ok ? 16 : 0);
     }
     pa_cp_commit();
   };
+  const PaInt<LPK> pk{};
+  const PaInt<LPV> pv{};
   int base = t_begin + warp * 32;
   if (base < t_end) {
     locate(base);
-    request(k_cache, kt_u32);
-    request(v_cache, vt_u32);
+    request(k_cache, kt_u32, pk, dk);
+    request(v_cache, vt_u32, pv, dv);
   }
   for (; base < t_end; base += kPaWarps * 32) {
     const int n_tok = n_next;
@@ -174,7 +201,7 @@ paged_decode_split_kernel(const __nv_bfloat16* __restrict__ q, long long ld_q, c
 #pragma unroll
     for (int n = 0; n < 4; ++n) s[n][0] = s[n][1] = s[n][2] = s[n][3] = 0.f;
 #pragma unroll
-    for (int k0 = 0; k0 < D; k0 += 16) {
+    for (int k0 = 0; k0 < DK; k0 += 16) {
       uint32_t a[4];
       // A fragment: matrices (rows 0-7, k0), (rows 8-15, k0), (rows 0-7, k0 + 8), (rows 8-15, k0 + 8)
       pa_ldsm_x4(q_u32 + ((lane & 15) * KROW + k0 + (lane >> 4) * 8) * 2, a);
@@ -190,7 +217,7 @@ paged_decode_split_kernel(const __nv_bfloat16* __restrict__ q, long long ld_q, c
     __syncwarp();                                                    // every lane has read its K fragments
     if (more) {                                                      // the next pass's K tile flies under softmax and P V
       locate(base + kPaWarps * 32);
-      request(k_cache, kt_u32);
+      request(k_cache, kt_u32, pk, dk);
     }
     // ---- online softmax over the 32 tokens; this thread holds 8 of them for rows gq and gq + 8
     float mx0 = -INFINITY, mx1 = -INFINITY;
@@ -199,8 +226,18 @@ paged_decode_split_kernel(const __nv_bfloat16* __restrict__ q, long long ld_q, c
 #pragma unroll
       for (int j = 0; j < 2; ++j) {
         const bool ok = n * 8 + 2 * tq + j < n_tok;
-        s[n][j] = ok ? s[n][j] * scale : -INFINITY;
-        s[n][2 + j] = ok ? s[n][2 + j] * scale : -INFINITY;
+        float v0 = s[n][j] * scale, v1 = s[n][2 + j] * scale;
+        if (RULE) {
+          if (rule.softcap > 0.f) {
+            v0 = pa_softcap(v0, rule.softcap, two_over_cap);
+            v1 = pa_softcap(v1, rule.softcap, two_over_cap);
+          }
+          const float dist = static_cast<float>(ctx - 1 - (base + n * 8 + 2 * tq + j));
+          v0 = fmaf(-slope0, dist, v0);
+          v1 = fmaf(-slope1, dist, v1);
+        }
+        s[n][j] = ok ? v0 : -INFINITY;
+        s[n][2 + j] = ok ? v1 : -INFINITY;
         mx0 = fmaxf(mx0, s[n][j]);
         mx1 = fmaxf(mx1, s[n][2 + j]);
       }
@@ -235,7 +272,7 @@ paged_decode_split_kernel(const __nv_bfloat16* __restrict__ q, long long ld_q, c
     for (int n = 0; n < NT; ++n) {
       acc[n][0] *= al0; acc[n][1] *= al0; acc[n][2] *= al1; acc[n][3] *= al1;
     }
-    // ---- O[16, D] += P[16, 32] V[32, D]
+    // ---- O[16, DV] += P[16, 32] V[32, DV]
     if (more) pa_cp_wait<1>(); else pa_cp_wait<0>();                 // this pass's V tile has landed
     __syncwarp();
 #pragma unroll
@@ -244,18 +281,18 @@ paged_decode_split_kernel(const __nv_bfloat16* __restrict__ q, long long ld_q, c
       for (int n2 = 0; n2 < NT / 2; ++n2) {
         uint32_t bfr[4];
         // transposed 8x8 blocks: (tokens 16ks..+7, dims 16n2), (tokens +8, same dims), (tokens.., dims + 8), (+8, + 8)
-        pa_ldsm_x4_t(vt_u32 + ((ks * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * KROW + n2 * 16 + (lane >> 4) * 8) * 2, bfr);
+        pa_ldsm_x4_t(vt_u32 + ((ks * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * VROW + n2 * 16 + (lane >> 4) * 8) * 2, bfr);
         pa_mma(acc[2 * n2], pfr[ks], bfr[0], bfr[1]);
         pa_mma(acc[2 * n2 + 1], pfr[ks], bfr[2], bfr[3]);
       }
     }
     __syncwarp();                                                    // every lane has read its V fragments
-    if (more) request(v_cache, vt_u32);
+    if (more) request(v_cache, vt_u32, pv, dv);
   }
 
   // ---- merge the warps, write this slice's (max, sum, accumulator) per head
   __syncthreads();                            // every warp is done with its tile: the buffer becomes the merge area
-  float (*acc_sh)[kMaxGroup][D] = reinterpret_cast<float (*)[kMaxGroup][D]>(big);
+  float (*acc_sh)[kMaxGroup][DV] = reinterpret_cast<float (*)[kMaxGroup][DV]>(big);
   if (tq == 0) {
     m_sh[warp][gq] = m0; l_sh[warp][gq] = l0;
     m_sh[warp][gq + 8] = m1; l_sh[warp][gq + 8] = l1;
@@ -266,8 +303,8 @@ paged_decode_split_kernel(const __nv_bfloat16* __restrict__ q, long long ld_q, c
     *reinterpret_cast<float2*>(&acc_sh[warp][gq + 8][n * 8 + 2 * tq]) = make_float2(acc[n][2], acc[n][3]);
   }
   __syncthreads();
-  for (int i = threadIdx.x; i < gcount * D; i += blockDim.x) {
-    const int g = i / D, d = i - g * D;
+  for (int i = threadIdx.x; i < gcount * dv; i += blockDim.x) {
+    const int g = i / dv, d = i - g * dv;
     float mx = -INFINITY;
 #pragma unroll
     for (int w = 0; w < kPaWarps; ++w) mx = fmaxf(mx, m_sh[w][g]);
@@ -278,31 +315,41 @@ paged_decode_split_kernel(const __nv_bfloat16* __restrict__ q, long long ld_q, c
       num += acc_sh[w][g][d] * sc;
       den += l_sh[w][g] * sc;
     }
-    float* pp = partial + ((static_cast<long long>(b) * heads + h_base + g) * nsplit + sp) * (D + 2);
+    if (direct_out) {                        // a single slice: this is the result
+      const long long col = static_cast<long long>(h_base + g) * dv + d;
+      float o = num / den;
+      if (RULE && rule.gate) o *= pa_sigmoid(__bfloat162float(rule.gate[b * rule.ld_g + col]));
+      direct_out[b * ld_o + col] = __float2bfloat16(o);
+      continue;
+    }
+    float* pp = partial + ((static_cast<long long>(b) * heads + h_base + g) * nsplit + sp) * (dv + 2);
     pp[2 + d] = num;
     if (d == 0) { pp[0] = mx; pp[1] = den; }
   }
 }
 
-// out[b, h, :] = merge over the slices that hold tokens of sequence b
-template <int D>
-__global__ void __launch_bounds__(D)
-paged_decode_merge_kernel(const float* __restrict__ partial, const int* __restrict__ context_lens, int heads, int nsplit,
-                          __nv_bfloat16* __restrict__ out, long long ld_o) {
+// out[b, h, :] = merge over the slices that hold tokens of sequence b (times sigmoid(gate)); one thread per value column
+__global__ void __launch_bounds__(128)
+paged_decode_merge_kernel(const float* __restrict__ partial, const int* __restrict__ context_lens, int heads, int dv,
+                          int nsplit, __nv_bfloat16* __restrict__ out, long long ld_o, const PaRule rule) {
   const int b = blockIdx.x, h = blockIdx.y, d = threadIdx.x;
+  if (d >= dv) return;
   const int ctx = context_lens[b];
-  const int n = min(nsplit, (ctx + kSplitTokens - 1) / kSplitTokens);
-  const float* base = partial + (static_cast<long long>(b) * heads + h) * nsplit * (D + 2);
+  const int n = min(nsplit, (ctx - pa_first_key(ctx, rule.chunk) + kSplitTokens - 1) / kSplitTokens);
+  const float* base = partial + (static_cast<long long>(b) * heads + h) * nsplit * (dv + 2);
   float mx = -INFINITY;
-  for (int s = 0; s < n; ++s) mx = fmaxf(mx, base[s * (D + 2)]);
+  for (int s = 0; s < n; ++s) mx = fmaxf(mx, base[s * (dv + 2)]);
   float num = 0.f, den = 0.f;
   for (int s = 0; s < n; ++s) {
-    const float ms = base[s * (D + 2)];
+    const float ms = base[s * (dv + 2)];
     const float sc = (ms == -INFINITY) ? 0.f : __expf(ms - mx);
-    num += base[s * (D + 2) + 2 + d] * sc;
-    den += base[s * (D + 2) + 1] * sc;
+    num += base[s * (dv + 2) + 2 + d] * sc;
+    den += base[s * (dv + 2) + 1] * sc;
   }
-  out[static_cast<long long>(b) * ld_o + static_cast<long long>(h) * D + d] = __float2bfloat16(den > 0.f ? num / den : 0.f);
+  const long long col = static_cast<long long>(h) * dv + d;
+  float o = den > 0.f ? num / den : 0.f;
+  if (rule.gate) o *= pa_sigmoid(__bfloat162float(rule.gate[b * rule.ld_g + col]));
+  out[static_cast<long long>(b) * ld_o + col] = __float2bfloat16(o);
 }
 
 // ---- any rows, any head sizes, bf16 or fp32 ------------------------------------------------------------------------
@@ -427,6 +474,62 @@ RB_API long long rb_paged_attention_scratch_floats(int batch, int heads, int hea
   return static_cast<long long>(batch) * heads * nsplit * (head_dim + 2);
 }
 
+namespace {
+template <int DK, int DV, bool RULE>
+int pd_launch(const RbPagedDecodeArgs& a, cudaStream_t stream) {
+  const int group = a.heads / a.kv_heads;
+  long long span = static_cast<long long>(a.max_blocks) * a.block_size;      // most keys a row can see
+  if (a.chunk > 0 && a.chunk < span) span = a.chunk;
+  const int nsplit = static_cast<int>((span + rb::kSplitTokens - 1) / rb::kSplitTokens);
+  // dynamic shared memory: per warp a K and a V tile of 32 padded rows, plus the 16 padded query rows
+  const int smem = (rb::kPaWarps * 32 * (DK + 8 + DV + 8) + rb::kMaxGroup * (DK + 8)) * 2;
+  auto kern = rb::paged_decode_split_kernel<DK, DV, RULE>;
+  static bool attr_set[64] = {};
+  int dev = 0;
+  if (cudaGetDevice(&dev) != cudaSuccess || dev < 0 || dev >= 64) return -3;
+  if (!attr_set[dev]) {
+    const cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+    if (e != cudaSuccess) return static_cast<int>(e);
+    attr_set[dev] = true;
+  }
+  auto O = reinterpret_cast<__nv_bfloat16*>(a.out);
+  const rb::PaRule rule = {a.softcap, a.slopes, a.chunk, reinterpret_cast<const __nv_bfloat16*>(a.gate), a.ld_g};
+  const dim3 grid(a.batch, a.kv_heads, nsplit);
+  for (int g0 = 0; g0 < group; g0 += rb::kMaxGroup)       // groups wider than 16 heads take several passes
+    kern<<<grid, rb::kPaWarps * 32, smem, stream>>>(
+        reinterpret_cast<const __nv_bfloat16*>(a.q), a.ld_q, reinterpret_cast<const __nv_bfloat16*>(a.k_cache),
+        reinterpret_cast<const __nv_bfloat16*>(a.v_cache), a.block_tables, a.max_blocks, a.context_lens, a.heads, a.kv_heads,
+        a.dk, a.dv, a.block_size, a.num_blocks, a.scale, g0, group - g0 < rb::kMaxGroup ? group - g0 : rb::kMaxGroup,
+        a.scratch, nsplit, nsplit == 1 ? O : nullptr, a.ld_o, rule RB_BOUNDS_ARG);
+  if (nsplit > 1)
+    rb::paged_decode_merge_kernel<<<dim3(a.batch, a.heads), 128, 0, stream>>>(a.scratch, a.context_lens, a.heads, a.dv, nsplit,
+                                                                              O, a.ld_o, rule);
+  return static_cast<int>(cudaGetLastError());
+}
+
+template <int DK>
+int pd_by_dv(const RbPagedDecodeArgs& a, cudaStream_t s) {
+  if (a.dv <= 64) return pd_launch<DK, 64, true>(a, s);
+  if (a.dv <= 96) return pd_launch<DK, 96, true>(a, s);
+  return pd_launch<DK, 128, true>(a, s);
+}
+}  // namespace
+
+RB_API int rb_paged_attention_decode_rule(const RbPagedDecodeArgs* args, void* stream_v) {
+  const RbPagedDecodeArgs& a = *args;
+  if (a.batch <= 0) return 0;
+  if (a.heads <= 0 || a.kv_heads <= 0 || a.heads % a.kv_heads || a.dk <= 0 || a.dv <= 0 || a.dk > 128 || a.dv > 128 ||
+      ((a.dk | a.dv) & 7) || a.block_size <= 0 || a.max_blocks <= 0 || !a.scratch || (a.ld_q & 1) ||
+      a.num_blocks * a.block_size >= (1ll << 31))
+    return -1;
+  if ((reinterpret_cast<uintptr_t>(a.k_cache) | reinterpret_cast<uintptr_t>(a.v_cache)) & 15) return -2;
+  if (reinterpret_cast<uintptr_t>(a.q) & 3) return -2;
+  cudaStream_t s = reinterpret_cast<cudaStream_t>(stream_v);
+  if (a.dk <= 64) return pd_by_dv<64>(a, s);
+  if (a.dk <= 96) return pd_by_dv<96>(a, s);
+  return pd_by_dv<128>(a, s);
+}
+
 RB_API int rb_paged_attention_decode(const void* q, long long ld_q, void* out, long long ld_o, const void* k_cache,
                                      const void* v_cache, const int* block_tables, int max_blocks, const int* context_lens,
                                      int batch, int heads, int kv_heads, int head_dim, int block_size, long long num_blocks,
@@ -436,42 +539,11 @@ RB_API int rb_paged_attention_decode(const void* q, long long ld_q, void* out, l
       max_blocks <= 0 || !scratch || num_blocks * block_size >= (1ll << 31))
     return -1;
   if ((reinterpret_cast<uintptr_t>(k_cache) | reinterpret_cast<uintptr_t>(v_cache)) & 15) return -2;
+  RbPagedDecodeArgs a = {};
+  a.q = q; a.ld_q = ld_q; a.out = out; a.ld_o = ld_o; a.k_cache = k_cache; a.v_cache = v_cache;
+  a.block_tables = block_tables; a.max_blocks = max_blocks; a.context_lens = context_lens; a.batch = batch;
+  a.heads = heads; a.kv_heads = kv_heads; a.dk = a.dv = head_dim; a.block_size = block_size; a.num_blocks = num_blocks;
+  a.scale = scale; a.scratch = scratch;
   cudaStream_t stream = reinterpret_cast<cudaStream_t>(stream_v);
-  const int group = heads / kv_heads;
-  const int nsplit = static_cast<int>((static_cast<long long>(max_blocks) * block_size + rb::kSplitTokens - 1) / rb::kSplitTokens);
-  dim3 grid(batch, kv_heads, nsplit);
-  auto Q = reinterpret_cast<const __nv_bfloat16*>(q);
-  auto O = reinterpret_cast<__nv_bfloat16*>(out);
-  auto K = reinterpret_cast<const __nv_bfloat16*>(k_cache);
-  auto V = reinterpret_cast<const __nv_bfloat16*>(v_cache);
-  // dynamic shared memory: per warp a K and a V tile of 32 padded rows, plus the 16 padded query rows
-  const int krow = head_dim + 8;
-  const int smem = (rb::kPaWarps * 2 * 32 + rb::kMaxGroup) * krow * 2;
-  static bool attr_set[64][2] = {};
-  int dev = 0;
-  if (cudaGetDevice(&dev) != cudaSuccess || dev < 0 || dev >= 64) return -3;
-  if (!attr_set[dev][head_dim == 128]) {
-    const cudaError_t e = head_dim == 128
-        ? cudaFuncSetAttribute(rb::paged_decode_split_kernel<128>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem)
-        : cudaFuncSetAttribute(rb::paged_decode_split_kernel<64>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
-    if (e != cudaSuccess) return static_cast<int>(e);
-    attr_set[dev][head_dim == 128] = true;
-  }
-  for (int g0 = 0; g0 < group; g0 += rb::kMaxGroup) {     // groups wider than 16 heads take several passes
-    const int gc = group - g0 < rb::kMaxGroup ? group - g0 : rb::kMaxGroup;
-    if (head_dim == 128)
-      rb::paged_decode_split_kernel<128><<<grid, rb::kPaWarps * 32, smem, stream>>>(Q, ld_q, K, V, block_tables, max_blocks,
-                                                                                context_lens, heads, kv_heads, block_size,
-                                                                                num_blocks, scale, g0, gc, scratch, nsplit RB_BOUNDS_ARG);
-    else
-      rb::paged_decode_split_kernel<64><<<grid, rb::kPaWarps * 32, smem, stream>>>(Q, ld_q, K, V, block_tables, max_blocks,
-                                                                               context_lens, heads, kv_heads, block_size,
-                                                                               num_blocks, scale, g0, gc, scratch, nsplit RB_BOUNDS_ARG);
-  }
-  dim3 mgrid(batch, heads);
-  if (head_dim == 128)
-    rb::paged_decode_merge_kernel<128><<<mgrid, 128, 0, stream>>>(scratch, context_lens, heads, nsplit, O, ld_o);
-  else
-    rb::paged_decode_merge_kernel<64><<<mgrid, 64, 0, stream>>>(scratch, context_lens, heads, nsplit, O, ld_o);
-  return static_cast<int>(cudaGetLastError());
+  return head_dim == 128 ? pd_launch<128, 128, false>(a, stream) : pd_launch<64, 64, false>(a, stream);
 }

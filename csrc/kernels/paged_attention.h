@@ -19,6 +19,24 @@ int rb_paged_attention_decode(const void* q, long long ld_q, void* out, long lon
                               const void* v_cache, const int* block_tables, int max_blocks, const int* context_lens,
                               int batch, int heads, int kv_heads, int head_dim, int block_size, long long num_blocks,
                               float scale, float* scratch, void* stream);
+// The same decode attention with separate key / value head sizes (multiples of 8, at most 128), a score rule and an output
+// gate; softcap, slopes, chunk and gate as in RbPagedRowsArgs below.  bf16 operands.  scratch: fp32
+// [rb_paged_attention_scratch_floats(batch, heads, dv, max_blocks, block_size)].
+typedef struct RbPagedDecodeArgs {
+  const void* q;             // [batch, heads * dk], pitch ld_q
+  void* out;                 // [batch, heads * dv], pitch ld_o
+  const void* k_cache;
+  const void* v_cache;
+  const int* block_tables;
+  const int* context_lens;
+  const float* slopes;
+  const void* gate;          // [batch, heads * dv], pitch ld_g
+  float* scratch;
+  long long ld_q, ld_o, ld_g, num_blocks;
+  int batch, max_blocks, heads, kv_heads, dk, dv, block_size, chunk;
+  float scale, softcap;
+} RbPagedDecodeArgs;
+int rb_paged_attention_decode_rule(const RbPagedDecodeArgs* args, void* stream);
 // Attention over the pages for any rows of a batch (prompt portions and decoded tokens alike), any head sizes, bf16 or
 // fp32 operands, fp32 arithmetic: the 32-bit mode and the fallback for head sizes the tensor-core kernels do not take.
 //   row r is the token at position row_pos[r] of the sequence whose pages are block_tables[row_seq[r]]; it sees the keys

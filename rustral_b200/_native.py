@@ -53,6 +53,10 @@ class RbAttnArgs(C.Structure):
     ]
 
 
+class RbAttnRule(C.Structure):
+    _fields_ = [("v_dim", c_int), ("softcap", c_float), ("slopes", c_void_p), ("chunk", c_int), ("gate", c_void_p), ("ld_gate", c_ll)]
+
+
 class RbResidualNormArgs(C.Structure):
     _fields_ = [
         ("y", c_void_p), ("slot_pos", c_void_p), ("slot_w", c_void_p), ("add", c_void_p), ("gamma", c_void_p), ("beta", c_void_p),
@@ -79,6 +83,16 @@ class RbPagedRowsArgs(C.Structure):
         ("ld_q", c_ll), ("ld_o", c_ll), ("ld_g", c_ll), ("num_blocks", c_ll),
         ("f32", c_int), ("rows", c_int), ("max_blocks", c_int), ("heads", c_int), ("kv_heads", c_int), ("dk", c_int),
         ("dv", c_int), ("block_size", c_int), ("chunk", c_int), ("scale", c_float), ("softcap", c_float),
+    ]
+
+
+class RbPagedDecodeArgs(C.Structure):
+    _fields_ = [
+        ("q", c_void_p), ("out", c_void_p), ("k_cache", c_void_p), ("v_cache", c_void_p), ("block_tables", c_void_p),
+        ("context_lens", c_void_p), ("slopes", c_void_p), ("gate", c_void_p), ("scratch", c_void_p),
+        ("ld_q", c_ll), ("ld_o", c_ll), ("ld_g", c_ll), ("num_blocks", c_ll),
+        ("batch", c_int), ("max_blocks", c_int), ("heads", c_int), ("kv_heads", c_int), ("dk", c_int), ("dv", c_int),
+        ("block_size", c_int), ("chunk", c_int), ("scale", c_float), ("softcap", c_float),
     ]
 
 

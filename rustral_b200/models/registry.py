@@ -34,6 +34,8 @@ def _gpt_config(d: dict) -> GPTConfig:
 def _gpt_weights(cfg, device, dtype, tensors, seed):
     from ..runtime.fused_gpt import FlatParams
     from ..serve.weights import InferenceWeights
+    if str(device) != "cpu" and dtype is not None and str(dtype) != "torch.bfloat16":
+        raise ValueError(f"{cfg.arch} is served in bf16 on a GPU")
     if str(device) != "cpu" and cfg.arch == "llama":                 # bf16 inference weights (no optimizer buffers)
         p = InferenceWeights.random_llama(cfg, device, 0, 1, seed)
         if tensors is not None:

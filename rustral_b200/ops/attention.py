@@ -145,7 +145,16 @@ def prompt_supported(q, k, v, dk: int, dv: int, rule: ScoreRule | None = None, g
     """Whether `prompt_attention` takes these operands (2-D [rows, heads * size] views)."""
     if not q.is_cuda:
         return True
-    return q.dtype == torch.bfloat16 and dk == dv and dk in (64, 128) and rule is None and gate is None
+    if q.dtype != torch.bfloat16:
+        return False
+    if rule is None and gate is None and dk == dv:
+        return dk in (64, 128)
+    views = [t for t in (q, k, v, gate) if t is not None]
+    return dk % 8 == 0 and dv % 8 == 0 and max(dk, dv) <= 128 and \
+        all(t.stride(0) % 8 == 0 and t.data_ptr() % 16 == 0 for t in views)
+
+
+N.optional_sig("rb_attention_fwd_rule", [N.C.POINTER(N.RbAttnArgs), N.C.POINTER(N.RbAttnRule), N.c_void_p])
 
 
 def prompt_attention(q, k, v, scale: float, out, rule: ScoreRule | None = None, gate=None):
@@ -158,7 +167,17 @@ def prompt_attention(q, k, v, scale: float, out, rule: ScoreRule | None = None, 
             o = o.float() * torch.sigmoid(gate.float().reshape(o.shape))
         out.copy_(o)
         return out
-    return attention_forward(q, k, v, True, scale, out=out, want_lse=False)[0]
+    dv = v.shape[3]
+    if rule is None and gate is None and dv == q.shape[3]:
+        return attention_forward(q, k, v, True, scale, out=out, want_lse=False)[0]
+    rule = rule or ScoreRule()
+    a, r = N.RbAttnArgs(), N.RbAttnRule()
+    _fill(a, q, k, v, out, True, scale)
+    r.v_dim, r.softcap, r.slopes, r.chunk = dv, rule.softcap, N.ptr(rule.slopes), rule.chunk
+    if gate is not None:
+        r.gate, r.ld_gate = gate.data_ptr(), gate.stride(0)
+    N.check(N.kernels().rb_attention_fwd_rule(a, r, N.stream_ptr()), "rb_attention_fwd_rule")
+    return out
 
 
 def attention_backward(do, q, k, v, o, lse, causal: bool, scale: float, dq=None, dk=None, dv=None, impl: str | None = None,

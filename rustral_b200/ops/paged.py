@@ -13,6 +13,8 @@ N.optional_sig("rb_kv_append", [N.c_void_p, N.c_ll, N.c_void_p, N.c_ll, N.c_void
 N.optional_sig("rb_paged_attention_decode", [N.c_void_p, N.c_ll, N.c_void_p, N.c_ll, N.c_void_p, N.c_void_p, N.c_void_p,
                                              N.c_int, N.c_void_p, N.c_int, N.c_int, N.c_int, N.c_int, N.c_int, N.c_ll,
                                              N.c_float, N.c_void_p, N.c_void_p])
+N.optional_sig("rb_paged_attention_decode_rule", [N.C.POINTER(N.RbPagedDecodeArgs), N.c_void_p])
+N._LAUNCHES["rb_paged_attention_decode_rule"] = 2
 N.optional_sig("rb_paged_attention_scratch_floats", [N.c_int, N.c_int, N.c_int, N.c_int, N.c_int], N.c_ll)
 N._LAUNCHES["rb_paged_attention_decode"] = 2
 
@@ -37,7 +39,11 @@ def decode_supported(q, dk: int, dv: int, rule: ScoreRule | None = None, gate=No
     """Whether `paged_attention_decode` takes these operands."""
     if not q.is_cuda:
         return True
-    return q.dtype == torch.bfloat16 and dk == dv and dk in (64, 128) and rule is None and gate is None
+    if q.dtype != torch.bfloat16:
+        return False
+    if rule is None and gate is None and dk == dv:
+        return dk in (64, 128)
+    return dk % 8 == 0 and dv % 8 == 0 and max(dk, dv) <= 128 and q.stride(0) % 2 == 0 and q.data_ptr() % 4 == 0
 
 
 def paged_attention_decode(q, k_cache, v_cache, block_tables, context_lens, scale=None, out=None, rule: ScoreRule | None = None,
@@ -68,10 +74,22 @@ def paged_attention_decode(q, k_cache, v_cache, block_tables, context_lens, scal
             out.copy_(r)
             return out
         return r
-    out = out if out is not None else torch.empty((B, heads * d), dtype=q.dtype, device=q.device)
+    out = out if out is not None else torch.empty((B, heads * dv), dtype=q.dtype, device=q.device)
     lib = N.kernels()
-    scratch = torch.empty(lib.rb_paged_attention_scratch_floats(B, heads, d, block_tables.shape[1], bs), dtype=torch.float32,
+    scratch = torch.empty(lib.rb_paged_attention_scratch_floats(B, heads, dv, block_tables.shape[1], bs), dtype=torch.float32,
                           device=q.device)
+    if rule is not None or gate is not None or dv != d:
+        rule = rule or ScoreRule()
+        a = N.RbPagedDecodeArgs()
+        a.q, a.ld_q, a.out, a.ld_o = q2.data_ptr(), q2.stride(0), out.data_ptr(), out.stride(0)
+        a.k_cache, a.v_cache, a.num_blocks, a.block_size = k_cache.data_ptr(), v_cache.data_ptr(), nb, bs
+        a.block_tables, a.max_blocks, a.context_lens = block_tables.data_ptr(), block_tables.shape[1], context_lens.data_ptr()
+        if gate is not None:
+            a.gate, a.ld_g = gate.data_ptr(), gate.stride(0)
+        a.scratch, a.batch, a.heads, a.kv_heads, a.dk, a.dv = scratch.data_ptr(), B, heads, hk, d, dv
+        a.scale, a.softcap, a.slopes, a.chunk = scale, rule.softcap, N.ptr(rule.slopes), rule.chunk
+        N.check(lib.rb_paged_attention_decode_rule(a, N.stream_ptr()), "rb_paged_attention_decode_rule")
+        return out
     N.check(lib.rb_paged_attention_decode(q2.data_ptr(), q2.stride(0), out.data_ptr(), out.stride(0),
                                           k_cache.data_ptr(), v_cache.data_ptr(), block_tables.data_ptr(),
                                           block_tables.shape[1], context_lens.data_ptr(), B, heads, hk, d, bs, nb,

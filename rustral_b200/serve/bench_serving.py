@@ -23,14 +23,14 @@ import os
 import torch
 import torch.distributed as dist
 
-from ..models.config import preset
+from ..models.registry import build_weights, load_tensors, resolve_config
 from .engine import ServingEngine, run_poisson_workload
 from .model_runner import ModelRunner
 
 
 def main(argv=None):
     ap = argparse.ArgumentParser()
-    ap.add_argument("--model", default="llama-8b")
+    ap.add_argument("--model", default="llama-8b", help="preset, or a folder with config.json and model.safetensors")
     ap.add_argument("--layers", type=int, default=0, help="override depth (a full 8B model needs ~16 GB of weights)")
     ap.add_argument("--requests", type=int, default=64)
     ap.add_argument("--rate", type=float, default=8.0)
@@ -49,7 +49,7 @@ def main(argv=None):
     ap.add_argument("--prefill-chunk", type=int, default=2048, help="prompt tokens per step (0: whole prompts, one pass each)")
     a = ap.parse_args(argv)
     over = {"n_layer": a.layers} if a.layers else {}
-    cfg = preset(a.model, **over)
+    cfg = resolve_config(a.model, **over)
     rank = 0
     tp = clock = None
     if a.tp > 1:
@@ -65,11 +65,8 @@ def main(argv=None):
         clock = tp.broadcast_scalar
     else:
         dev = "cuda" if torch.cuda.is_available() else "cpu"
-    if tp is None and cfg.arch == "llama" and str(dev) != "cpu":
-        from .weights import InferenceWeights           # bf16 weights only: the trainer's flat buffers would not fit
-        params = InferenceWeights.random_llama(cfg, dev, 0, 1, a.seed)
-    else:
-        params = None
+    # bf16 inference weights where the architecture has them: the trainer's flat buffers would not fit
+    params = build_weights(cfg, dev, None, load_tensors(a.model), a.seed) if tp is None else None
     runner = ModelRunner(cfg, params=params, device=dev, num_blocks=a.blocks, block_size=a.page, seed=a.seed, tp=tp)
     eng = ServingEngine(runner, max_batch_size=a.max_batch, prefill_chunk=a.prefill_chunk)
     # warm-up: one short request end to end

@@ -11,6 +11,7 @@ from __future__ import annotations
 
 import argparse
 import json
+import os
 import signal
 import threading
 import time
@@ -269,27 +270,17 @@ def build_state(a) -> ServerState:
     (continuous batching over the paged KV cache) behind /v1/generate."""
     from ..core import B200Backend, CpuBackend
     if a.model:
-        from ..models.config import preset
         from .engine import ServingEngine
-        from .model_runner import ModelRunner
-        cfg = preset(a.model, **({"n_layer": a.layers} if a.layers else {}))
-        params = None
-        if a.device != "cpu" and cfg.arch == "llama":
-            from .weights import InferenceWeights           # bf16 inference weights (no optimizer buffers)
-            params = InferenceWeights.random_llama(cfg, a.device, 0, 1, a.seed)
-        runner = ModelRunner(cfg, params=params, device=a.device, num_blocks=a.blocks, block_size=a.page, seed=a.seed)
-        if a.weights:
-            from ..io import safetensors_io as st
-            tensors, _ = st.load_file(a.weights)            # strict: names and shapes must match the preset
-            if hasattr(runner.params, "tensors"):
-                runner.params.load_state_dict(tensors, cfg)
-            else:
-                runner.params.load_state_dict(tensors)
+        from .model_runner import load_runner
+        dtype = getattr(torch, a.dtype) if a.dtype else None
+        runner = load_runner(a.model, device=a.device, dtype=dtype, num_blocks=a.blocks, block_size=a.page, weights=a.weights,
+                             seed=a.seed, **({"n_layer": a.layers} if a.layers else {}))   # weights are loaded strictly
+        cfg = runner.cfg
         engine = ServingEngine(runner, max_batch_size=a.max_batch, eos_id=a.eos_id)
         engine.generate([1, 2, 3], 2)                       # warm-up: compiles nothing, but touches every kernel once
         meta = {"model": a.model, "layers": cfg.n_layer, "d_model": cfg.d_model, "vocab_size": cfg.vocab_size,
                 "context": cfg.seq_len, "page_size": a.page, "kv_blocks": a.blocks, "device": a.device,
-                "weights": a.weights or "random-init"}
+                "weights": a.weights or (a.model if os.path.isdir(a.model) else "random-init")}
         loop = EngineLoop(engine)
         return ServerState(generate_fn=engine_generate_fn(engine, loop), metadata=meta, generate_workers=a.max_batch,
                            engine_loop=loop)
@@ -315,7 +306,9 @@ def parse_args(argv=None):
     g.add_argument("--out-features", type=int, default=0)
     g.add_argument("--bias", action="store_true")
     e = ap.add_argument_group("decoder engine (/v1/generate)")
-    e.add_argument("--model", help="model preset, e.g. llama-8b, gpt2-small")
+    e.add_argument("--model", help="model preset (llama-8b, gpt2-small, dolurax-test, ...) or a folder with config.json and "
+                                   "model.safetensors")
+    e.add_argument("--dtype", default=None, choices=["bfloat16", "float32"], help="for architectures that run in both")
     e.add_argument("--layers", type=int, default=0, help="override the preset's depth")
     e.add_argument("--weights", help="safetensors state dict of the model; random-init when absent")
     e.add_argument("--blocks", type=int, default=4096, help="KV-cache pages")
