@@ -41,7 +41,25 @@ def parse_args():
     ap.add_argument("--comm", default="auto", choices=["auto", "nccl", "fused"])
     ap.add_argument("--seq-len", type=int, default=0, help="override the preset's sequence length (tests only)")
     ap.add_argument("--layers", type=int, default=0, help="override the preset's depth (tests only)")
+    ap.add_argument("--decoders", action="store_true", help="serving throughput of the layered decoder beside the Llama-style one "
+                    "at equal size, and their kernels against the roofline (one GPU), instead of the training benchmark")
+    ap.add_argument("--decoder-size", default=None, help="with --decoders: only this size")
     return ap.parse_args()
+
+
+def decoder_arm(args):
+    import torch
+    sys.path.insert(0, os.path.dirname(os.path.abspath(__file__)))
+    from rustral_b200 import _native
+    from rustral_b200.bench import decoders
+    torch.cuda.set_device(0)
+    sampler = ClockSampler(0)
+    sampler.start()
+    out = decoders.run([args.decoder_size] if args.decoder_size else None)
+    out["clocks"] = sampler.stop()
+    out["device_status"] = _native.read_status()[0]
+    print(json.dumps(out))
+    return 0
 
 
 class ClockSampler:
@@ -112,6 +130,8 @@ def main():
     args = parse_args()
     if args.impl == "reference":
         return reference_arm(args)
+    if args.decoders:
+        return decoder_arm(args)
 
     if args.gpus > 1 and "RANK" not in os.environ:
         # launched directly: re-launch one rank per GPU

@@ -504,17 +504,27 @@ RB_API int rb_dropout(const void* a, void* out, unsigned char* mask_out, long lo
               (rb::dropout_kernel<__nv_bfloat16><<<grid, 256, 0, RB_STREAM>>>((const __nv_bfloat16*)a, (__nv_bfloat16*)out, mask_out, n, p, seed, offset, rng)))
 }
 namespace rb {
+__device__ __forceinline__ float scale_softcap(float x, float scale, float cap) {
+  const float v = x * scale;
+  return cap > 0.f ? cap * tanhf(v / cap) : v;
+}
 __global__ void __launch_bounds__(256) scale_softcap_kernel(float* __restrict__ x, long long n, float scale, float cap) {
   const long long stride = static_cast<long long>(gridDim.x) * blockDim.x;
-  for (long long i = static_cast<long long>(blockIdx.x) * blockDim.x + threadIdx.x; i < n; i += stride) {
-    const float v = x[i] * scale;
-    x[i] = cap > 0.f ? cap * tanhf(v / cap) : v;
+  const long long first = static_cast<long long>(blockIdx.x) * blockDim.x + threadIdx.x;
+  float4* x4 = reinterpret_cast<float4*>(x);
+  for (long long i = first; i < n / 4; i += stride) {
+    float4 v = x4[i];
+    v.x = scale_softcap(v.x, scale, cap); v.y = scale_softcap(v.y, scale, cap);
+    v.z = scale_softcap(v.z, scale, cap); v.w = scale_softcap(v.w, scale, cap);
+    x4[i] = v;
   }
+  for (long long i = n / 4 * 4 + first; i < n; i += stride) x[i] = scale_softcap(x[i], scale, cap);
 }
 }  // namespace rb
 RB_API int rb_scale_softcap(float* x, long long n, float scale, float cap, void* stream_v) {
   if (n <= 0) return 0;
-  rb::scale_softcap_kernel<<<rb::ew_grid(n), 256, 0, RB_STREAM>>>(x, n, scale, cap);
+  if (reinterpret_cast<uintptr_t>(x) & 15) return -2;
+  rb::scale_softcap_kernel<<<rb::ew_grid((n + 3) / 4), 256, 0, RB_STREAM>>>(x, n, scale, cap);
   return static_cast<int>(cudaGetLastError());
 }
 RB_API int rb_argmax_rows(const void* a, long long lda, long long* out, long long rows, int cols, int dtype, void* stream_v) {

@@ -1,6 +1,6 @@
 // Per-head work between the packed attention projection and the attention kernels, in one pass: RMS norm of every query
 // and key head, mixing of the values with an earlier layer's values of the same token, and the append of keys and values
-// to their cache slots.  Norms and mixing are fp32.  A group of 16 lanes owns one head of one token with 16-byte accesses;
+// to their cache slots.  Norms and mixing are fp32.  A group of 8 or 16 lanes owns one head of one token with 16-byte accesses;
 // head sizes that are not whole vectors take the scalar form (one warp per head).
 #include "head_prep.h"
 
@@ -49,11 +49,10 @@ __device__ __forceinline__ HpItem hp_item(int i, const RbHeadPrepArgs& a) {
   return {2, i - a.kv_heads};
 }
 
-template <typename T>
+template <typename T, int LANES>
 __global__ void __launch_bounds__(128)
 head_prep_kernel(const RbHeadPrepArgs a RB_BOUNDS_PARAM) {
   using V = HpVec<T>;
-  constexpr int LANES = 16;
   const int sub = threadIdx.x & (LANES - 1);
   const int items = a.heads + 2 * a.kv_heads;
   const long long total = a.tokens * items;
@@ -165,11 +164,14 @@ int hp_launch(const RbHeadPrepArgs& a, cudaStream_t s) {
   const bool vec = !(bits & 15) && !((a.ld | a.off_q | a.off_k | a.off_v | a.dk | a.dv | (a.v_first ? a.ld_vf : 0)) % N) &&
                    a.dk <= 16 * N * kHpMaxVec && a.dv <= 16 * N * kHpMaxVec;
   const long long total = a.tokens * (a.heads + 2 * a.kv_heads);
-  const int per_block = vec ? 8 : 4;
+  const bool narrow = a.dk <= 8 * N && a.dv <= 8 * N;        // one vector per lane of a group of 8
+  const int per_block = vec ? (narrow ? 16 : 8) : 4;
   long long blocks = (total + per_block - 1) / per_block;
   if (blocks > 148LL * 16) blocks = 148LL * 16;
-  if (vec)
-    head_prep_kernel<T><<<static_cast<int>(blocks), 128, 0, s>>>(a RB_BOUNDS_ARG);
+  if (vec && narrow)
+    head_prep_kernel<T, 8><<<static_cast<int>(blocks), 128, 0, s>>>(a RB_BOUNDS_ARG);
+  else if (vec)
+    head_prep_kernel<T, 16><<<static_cast<int>(blocks), 128, 0, s>>>(a RB_BOUNDS_ARG);
   else
     head_prep_scalar_kernel<T><<<static_cast<int>(blocks), 128, 0, s>>>(a RB_BOUNDS_ARG);
   return static_cast<int>(cudaGetLastError());

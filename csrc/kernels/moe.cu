@@ -101,85 +101,89 @@ moe_route_bwd_kernel(const float* __restrict__ probs, const int* __restrict__ id
   if (lane + 32 < E) dlogits[static_cast<long long>(t) * E + lane + 32] = pv1 * (dp[1] - s);
 }
 
-// Router with group-limited choice: one warp per token, scores and group maxima in shared memory.
+// Router with group-limited choice: one warp per token.  Scores are kept in shared memory as order-preserving integer keys
+// (bits of a non-negative float + 1; 0 = not available), so an arg-max is two warp reductions.
 __global__ void __launch_bounds__(128)
 moe_route_groups_kernel(const float* __restrict__ logits, int T, int E, int k, int groups, int keep, int renorm, float eps,
                         int* __restrict__ idx, float* __restrict__ w) {
-  extern __shared__ float route_sm[];
+  extern __shared__ unsigned int route_sm[];
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
   const int t = blockIdx.x * (blockDim.x >> 5) + warp;
   if (t >= T) return;
-  float* s = route_sm + warp * (E + groups);
-  float* gmax = s + E;
+  unsigned int* key = route_sm + warp * (E + groups);
+  unsigned int* gkey = key + E;
   const float* x = logits + static_cast<long long>(t) * E;
   float mx = -INFINITY;
   for (int e = lane; e < E; e += 32) mx = fmaxf(mx, x[e]);
   mx = warp_max(mx);
   float sum = 0.f;
-  for (int e = lane; e < E; e += 32) { const float p = expf(x[e] - mx); s[e] = p; sum += p; }
+  for (int e = lane; e < E; e += 32) {
+    const float p = __expf(x[e] - mx);
+    key[e] = __float_as_uint(p) + 1u;
+    sum += p;
+  }
   const float inv = 1.f / warp_sum(sum);
-  for (int e = lane; e < E; e += 32) s[e] *= inv;
   __syncwarp();
-  // arg-max over an array of non-negative values with ties to the lower index (used-up entries are -1)
-  auto pick = [&](const float* v, int n, float& best) {
-    float bv = -2.f;
-    int bi = 0;
+  // largest key of v[0 .. n), ties to the lower index; the chosen entry is set to 0
+  auto take = [&](unsigned int* v, int n, unsigned int& best) {
+    unsigned int bv = 0u;
+    int bi = n;
     for (int e = lane; e < n; e += 32)
       if (v[e] > bv) { bv = v[e]; bi = e; }
-#pragma unroll
-    for (int o = 16; o > 0; o >>= 1) {
-      const float ov = __shfl_xor_sync(0xffffffffu, bv, o);
-      const int oi = __shfl_xor_sync(0xffffffffu, bi, o);
-      if (ov > bv || (ov == bv && oi < bi)) { bv = ov; bi = oi; }
-    }
-    best = bv;
-    return bi;
+    best = __reduce_max_sync(0xffffffffu, bv);
+    int at = __reduce_min_sync(0xffffffffu, bv == best ? bi : n);
+    if (at >= n) at = 0;                               // nothing available (scores that are not numbers)
+    if ((at & 31) == lane) v[at] = 0u;
+    __syncwarp();
+    return at;
   };
-  float best;
+  unsigned int best;
   if (groups > 1 && keep < groups) {
     const int per = E / groups;
     for (int g = lane; g < groups; g += 32) {
-      float m = -1.f;
-      for (int e = g * per; e < (g + 1) * per; ++e) m = fmaxf(m, s[e]);
-      gmax[g] = m;
+      unsigned int m = 0u;
+      for (int e = g * per; e < (g + 1) * per; ++e) m = max(m, key[e]);
+      gkey[g] = m;
     }
     __syncwarp();
-    for (int j = 0; j < keep; ++j) {                   // kept groups are marked with -2 (below every arg-max candidate)
-      const int g = pick(gmax, groups, best);
-      __syncwarp();
-      if (lane == 0) gmax[g] = -2.f;
-      __syncwarp();
-    }
+    for (int j = 0; j < keep; ++j) take(gkey, groups, best);           // kept groups end up as 0
     for (int e = lane; e < E; e += 32)
-      if (gmax[e / per] > -1.5f) s[e] = -1.f;
+      if (gkey[e / per] != 0u) key[e] = 0u;
     __syncwarp();
   }
-  float tot = 0.f;
+  float tot = 0.f, mine = 0.f;                         // lane j keeps the j-th weight (written in rounds of 32)
+  int mine_e = 0;
   for (int j = 0; j < k; ++j) {
-    const int e = pick(s, E, best);
-    __syncwarp();
-    if (lane == 0) { s[e] = -1.f; idx[static_cast<long long>(t) * k + j] = e; w[static_cast<long long>(t) * k + j] = best; }
-    tot += best;
-    __syncwarp();
+    const int e = take(key, E, best);
+    const float p = best ? __uint_as_float(best - 1u) * inv : 0.f;
+    tot += p;
+    if ((j & 31) == lane) { mine = p; mine_e = e; }
+    if ((j & 31) == 31 || j == k - 1) {
+      const int slot = (j & ~31) + lane;
+      if (slot < k) {
+        idx[static_cast<long long>(t) * k + slot] = mine_e;
+        w[static_cast<long long>(t) * k + slot] = mine;
+      }
+    }
   }
   if (renorm) {
+    __syncwarp();
     for (int j = lane; j < k; j += 32) w[static_cast<long long>(t) * k + j] /= tot + eps;
   }
 }
 
-// silu(gate) * up over the live rows of a permuted expert buffer (the buffer is sized for the worst case; `live` says how
-// many rows the routing used)
+// silu(gate) * up over the rows that hold a token
 template <typename T, int N>
 __global__ void __launch_bounds__(256)
-swiglu_live_kernel(const T* __restrict__ gu, long long ld_gu, T* __restrict__ h, long long ld_h, int rows, int F,
-                   const int* __restrict__ live) {
-  const int n = live ? min(rows, live[0]) : rows;
+swiglu_slots_kernel(const T* __restrict__ gu, long long ld_gu, T* __restrict__ h, long long ld_h, int n, int F,
+                    const int* __restrict__ slot_pos) {
   const int chunks = F / N;
   const long long total = static_cast<long long>(n) * chunks;
   const long long stride = static_cast<long long>(gridDim.x) * blockDim.x;
   for (long long i = static_cast<long long>(blockIdx.x) * blockDim.x + threadIdx.x; i < total; i += stride) {
-    const long long r = i / chunks;
-    const int c = static_cast<int>(i - r * chunks) * N;
+    const long long s = i / chunks;
+    const int c = static_cast<int>(i - s * chunks) * N;
+    const long long r = slot_pos ? slot_pos[s] : s;
     if (N == 8) {
       const uint4 g = *reinterpret_cast<const uint4*>(gu + r * ld_gu + c), u = *reinterpret_cast<const uint4*>(gu + r * ld_gu + F + c);
       const uint32_t gw[4] = {g.x, g.y, g.z, g.w}, uw[4] = {u.x, u.y, u.z, u.w};
@@ -200,23 +204,19 @@ swiglu_live_kernel(const T* __restrict__ gu, long long ld_gu, T* __restrict__ h,
   }
 }
 
-// ---- permutation plan ---------------------------------------------------------------------------------------
-__device__ __forceinline__ int block_scan_excl(int v, int* sh, int& total) {
-  // exclusive scan over 1024 threads; sh has 1024 ints
-  sh[threadIdx.x] = v;
-  __syncthreads();
-  for (int o = 1; o < 1024; o <<= 1) {
-    const int t = threadIdx.x >= o ? sh[threadIdx.x - o] : 0;
-    __syncthreads();
-    sh[threadIdx.x] += t;
-    __syncthreads();
+__global__ void __launch_bounds__(256)
+moe_scatter_kernel(const uint4* __restrict__ x, const int* __restrict__ slot_pos, uint4* __restrict__ xp, int slots, int k,
+                   int chunks) {
+  const long long total = static_cast<long long>(slots) * chunks;
+  const long long stride = static_cast<long long>(gridDim.x) * blockDim.x;
+  for (long long i = static_cast<long long>(blockIdx.x) * blockDim.x + threadIdx.x; i < total; i += stride) {
+    const long long s = i / chunks;
+    const int c = static_cast<int>(i - s * chunks);
+    xp[static_cast<long long>(slot_pos[s]) * chunks + c] = x[s / k * chunks + c];
   }
-  const int incl = sh[threadIdx.x];
-  total = sh[1023];
-  __syncthreads();
-  return incl - v;
 }
 
+// ---- permutation plan ---------------------------------------------------------------------------------------
 __global__ void __launch_bounds__(1024) moe_count_kernel(const int* __restrict__ idx, int slots, int* __restrict__ counts) {
   __shared__ int sh[32];
   const int e = blockIdx.x;
@@ -232,37 +232,63 @@ __global__ void __launch_bounds__(1024) moe_count_kernel(const int* __restrict__
   }
 }
 
-__global__ void moe_offsets_kernel(const int* __restrict__ counts, int E, int* __restrict__ offsets,
-                                   int* __restrict__ tile_expert, int* __restrict__ num_tiles, int max_tiles) {
-  if (threadIdx.x != 0 || blockIdx.x != 0) return;
-  int off = 0, tile = 0;
-  for (int e = 0; e < E; ++e) {
-    offsets[e] = off;
-    const int padded = (counts[e] + RB_MOE_ROW_ALIGN - 1) / RB_MOE_ROW_ALIGN * RB_MOE_ROW_ALIGN;
-    for (int i = 0; i < padded / 128 && tile < max_tiles; ++i) tile_expert[tile++] = e;
-    off += padded;
-  }
-  offsets[E] = off;
-  num_tiles[0] = tile;
-  for (int i = tile; i < max_tiles; ++i) tile_expert[i] = -1;
-}
-
+// One CTA per expert: the expert's segment start from the counts of all experts, then the ranks of its slots in ascending
+// order (each warp owns a contiguous range of slots and counts it with ballots, twice: once for the warp's start).  The
+// CTAs also share the bookkeeping: -1 in padding rows and in the tail, the tile table, the offsets.
 __global__ void __launch_bounds__(1024)
-moe_assign_kernel(const int* __restrict__ idx, int slots, const int* __restrict__ offsets, int* __restrict__ slot_pos,
-                  int* __restrict__ row_slot) {
-  __shared__ int sh[1024];
-  const int e = blockIdx.x;
-  int base = offsets[e];
-  for (int s0 = 0; s0 < slots; s0 += 1024) {
-    const int s = s0 + threadIdx.x;
-    const int match = (s < slots && idx[s] == e) ? 1 : 0;
-    int total;
-    const int rank = block_scan_excl(match, sh, total);
+moe_assign_kernel(const int* __restrict__ idx, int slots, int E, const int* __restrict__ counts, int* __restrict__ offsets,
+                  int* __restrict__ tile_expert, int* __restrict__ num_tiles, int* __restrict__ slot_pos,
+                  int* __restrict__ row_slot, int max_rows) {
+  __shared__ int sh_before[32], sh_all[32], warp_cnt[32];
+  const int e = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+  auto padded = [](int c) { return (c + RB_MOE_ROW_ALIGN - 1) / RB_MOE_ROW_ALIGN * RB_MOE_ROW_ALIGN; };
+  int before = 0, all = 0;                             // rows of the experts before this one, rows of all
+  for (int i = threadIdx.x; i < E; i += 1024) {
+    const int p = padded(counts[i]);
+    all += p;
+    if (i < e) before += p;
+  }
+  for (int o = 16; o > 0; o >>= 1) {
+    before += __shfl_xor_sync(0xffffffffu, before, o);
+    all += __shfl_xor_sync(0xffffffffu, all, o);
+  }
+  if (lane == 0) { sh_before[warp] = before; sh_all[warp] = all; }
+  // this warp's slots, 32 at a time
+  const int per = (slots + 1023) / 1024 * 32;
+  const int lo = min(slots, warp * per), hi = min(slots, lo + per);
+  int cnt = 0;
+#pragma unroll 4
+  for (int s = lo; s < hi; s += 32) cnt += __popc(__ballot_sync(0xffffffffu, s + lane < hi && idx[s + lane] == e));
+  if (lane == 0) warp_cnt[warp] = cnt;
+  __syncthreads();
+  before = all = 0;
+  int rank = 0, count = 0;
+  for (int i = 0; i < 32; ++i) {
+    before += sh_before[i];
+    all += sh_all[i];
+    if (i < warp) rank += warp_cnt[i];
+    count += warp_cnt[i];
+  }
+  rank += before;
+#pragma unroll 4
+  for (int s = lo; s < hi; s += 32) {
+    const bool match = s + lane < hi && idx[s + lane] == e;
+    const unsigned int m = __ballot_sync(0xffffffffu, match);
     if (match) {
-      slot_pos[s] = base + rank;
-      row_slot[base + rank] = s;
+      const int r = rank + __popc(m & ((1u << lane) - 1u));
+      slot_pos[s + lane] = r;
+      row_slot[r] = s + lane;
     }
-    base += total;
+    rank += __popc(m);
+  }
+  const int rows = padded(count);
+  for (int r = before + count + threadIdx.x; r < before + rows; r += 1024) row_slot[r] = -1;
+  for (int i = threadIdx.x; i < rows / 128; i += 1024) tile_expert[before / 128 + i] = e;
+  for (int r = all + e * 1024 + threadIdx.x; r < max_rows; r += E * 1024) row_slot[r] = -1;
+  for (int i = all / 128 + e * 1024 + threadIdx.x; i < max_rows / 128; i += E * 1024) tile_expert[i] = -1;
+  if (threadIdx.x == 0) {
+    offsets[e] = before;
+    if (e == E - 1) { offsets[E] = all; num_tiles[0] = all / 128; }
   }
 }
 
@@ -373,20 +399,27 @@ RB_API int rb_moe_route_groups(const float* logits, int T, int E, int k, int gro
   rb::moe_route_groups_kernel<<<(T + 3) / 4, 128, smem, RB_ST>>>(logits, T, E, k, groups, keep, renorm, eps, idx, w);
   return static_cast<int>(cudaGetLastError());
 }
-RB_API int rb_swiglu_live(const void* gu, long long ld_gu, void* h, long long ld_h, int rows, int F, int f32,
-                          const int* live_rows, void* stream_v) {
-  if (rows <= 0 || F <= 0) return -1;
+RB_API int rb_swiglu_slots(const void* gu, long long ld_gu, void* h, long long ld_h, int n, int F, int f32,
+                           const int* slot_pos, void* stream_v) {
+  if (n <= 0 || F <= 0) return -1;
   const bool vec = !f32 && !((F | ld_gu | ld_h) & 7) && !((reinterpret_cast<uintptr_t>(gu) | reinterpret_cast<uintptr_t>(h)) & 15);
-  const int grid = rb::grid1d(static_cast<long long>(rows) * (vec ? F / 8 : F), 256);
+  const int grid = rb::grid1d(static_cast<long long>(n) * (vec ? F / 8 : F), 256);
   if (f32)
-    rb::swiglu_live_kernel<float, 1><<<grid, 256, 0, RB_ST>>>(reinterpret_cast<const float*>(gu), ld_gu, reinterpret_cast<float*>(h),
-                                                             ld_h, rows, F, live_rows);
+    rb::swiglu_slots_kernel<float, 1><<<grid, 256, 0, RB_ST>>>(reinterpret_cast<const float*>(gu), ld_gu,
+                                                              reinterpret_cast<float*>(h), ld_h, n, F, slot_pos);
   else if (vec)
-    rb::swiglu_live_kernel<__nv_bfloat16, 8><<<grid, 256, 0, RB_ST>>>(reinterpret_cast<const __nv_bfloat16*>(gu), ld_gu,
-                                                                     reinterpret_cast<__nv_bfloat16*>(h), ld_h, rows, F, live_rows);
+    rb::swiglu_slots_kernel<__nv_bfloat16, 8><<<grid, 256, 0, RB_ST>>>(reinterpret_cast<const __nv_bfloat16*>(gu), ld_gu,
+                                                                      reinterpret_cast<__nv_bfloat16*>(h), ld_h, n, F, slot_pos);
   else
-    rb::swiglu_live_kernel<__nv_bfloat16, 1><<<grid, 256, 0, RB_ST>>>(reinterpret_cast<const __nv_bfloat16*>(gu), ld_gu,
-                                                                     reinterpret_cast<__nv_bfloat16*>(h), ld_h, rows, F, live_rows);
+    rb::swiglu_slots_kernel<__nv_bfloat16, 1><<<grid, 256, 0, RB_ST>>>(reinterpret_cast<const __nv_bfloat16*>(gu), ld_gu,
+                                                                      reinterpret_cast<__nv_bfloat16*>(h), ld_h, n, F, slot_pos);
+  return static_cast<int>(cudaGetLastError());
+}
+RB_API int rb_moe_scatter(const void* x, const int* slot_pos, void* xp, int slots, int k, int dim, void* stream_v) {
+  if (slots <= 0 || k <= 0 || dim <= 0 || (dim % 8)) return -1;
+  if ((reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(xp)) & 15) return -2;
+  rb::moe_scatter_kernel<<<rb::grid1d(static_cast<long long>(slots) * (dim / 8), 256), 256, 0, RB_ST>>>(
+      reinterpret_cast<const uint4*>(x), slot_pos, reinterpret_cast<uint4*>(xp), slots, k, dim / 8);
   return static_cast<int>(cudaGetLastError());
 }
 RB_API int rb_moe_route_bwd(const float* probs, const int* idx, const float* w, const float* dw, const int* counts, int T,
@@ -398,11 +431,8 @@ RB_API int rb_moe_route_bwd(const float* probs, const int* idx, const float* w, 
 RB_API int rb_moe_plan(const int* idx, int T, int E, int k, int* counts, int* offsets, int* slot_pos, int* row_slot,
                        int* tile_expert, int* num_tiles, int max_rows, void* stream_v) {
   if (T <= 0 || E <= 0 || k <= 0 || max_rows < T * k + E * RB_MOE_ROW_ALIGN || (max_rows % 128)) return -1;
-  cudaError_t e = cudaMemsetAsync(row_slot, 0xFF, sizeof(int) * static_cast<size_t>(max_rows), RB_ST);
-  if (e != cudaSuccess) return static_cast<int>(e);
   rb::moe_count_kernel<<<E, 1024, 0, RB_ST>>>(idx, T * k, counts);
-  rb::moe_offsets_kernel<<<1, 32, 0, RB_ST>>>(counts, E, offsets, tile_expert, num_tiles, max_rows / 128);
-  rb::moe_assign_kernel<<<E, 1024, 0, RB_ST>>>(idx, T * k, offsets, slot_pos, row_slot);
+  rb::moe_assign_kernel<<<E, 1024, 0, RB_ST>>>(idx, T * k, E, counts, offsets, tile_expert, num_tiles, slot_pos, row_slot, max_rows);
   return static_cast<int>(cudaGetLastError());
 }
 RB_API int rb_moe_gather(const void* x, const int* row_slot, const float* slot_scale, void* xp, int max_rows, int k, int dim,

@@ -19,7 +19,9 @@ P, I, F, LL = N.c_void_p, N.c_int, N.c_float, N.c_ll
 N.optional_sig("rb_moe_route", [P, I, I, I, I, P, P, P, P])
 N.optional_sig("rb_moe_route_bwd", [P, P, P, P, P, I, I, I, I, F, P, P])
 N.optional_sig("rb_moe_route_groups", [P, I, I, I, I, I, I, F, P, P, P])
-N.optional_sig("rb_swiglu_live", [P, LL, P, LL, I, I, I, P, P])
+N.optional_sig("rb_swiglu_slots", [P, LL, P, LL, I, I, I, P, P])
+N.optional_sig("rb_moe_scatter", [P, P, P, I, I, I, P])
+N._LAUNCHES["rb_moe_plan"] = 2
 N.optional_sig("rb_moe_plan", [P, I, I, I, P, P, P, P, P, P, I, P])
 N.optional_sig("rb_moe_gather", [P, P, P, P, I, I, I, P, P])
 N.optional_sig("rb_moe_combine", [P, P, P, P, P, I, I, I, P])
@@ -74,16 +76,32 @@ def route_groups(logits: torch.Tensor, k: int, groups: int = 1, keep: int = 1, r
     return idx, w
 
 
-def swiglu_live(gu: torch.Tensor, live_rows=None) -> torch.Tensor:
-    """silu(gate) * up for gu = [gate | up] rows; `live_rows` (int32 [1] on the device): later rows are left unwritten."""
+def swiglu_rows(gu: torch.Tensor, pl: MoEPlan | None = None) -> torch.Tensor:
+    """silu(gate) * up for gu = [gate | up] rows, bf16 or fp32.  With a plan only the rows that hold a token are computed;
+    padding rows of the expert buffer are left unwritten."""
     rows, F2 = gu.shape
     if not gu.is_cuda:
         g, u = gu.float()[:, :F2 // 2], gu.float()[:, F2 // 2:]
         return (g * torch.sigmoid(g) * u).to(gu.dtype)
     h = torch.empty((rows, F2 // 2), dtype=gu.dtype, device=gu.device)
-    N.check(N.kernels().rb_swiglu_live(gu.data_ptr(), gu.stride(0), h.data_ptr(), h.stride(0), rows, F2 // 2,
-                                       int(gu.dtype == torch.float32), N.ptr(live_rows), N.stream_ptr()), "rb_swiglu_live")
+    n = rows if pl is None else pl.slot_pos.numel()
+    N.check(N.kernels().rb_swiglu_slots(gu.data_ptr(), gu.stride(0), h.data_ptr(), h.stride(0), n, F2 // 2,
+                                        int(gu.dtype == torch.float32), None if pl is None else pl.slot_pos.data_ptr(),
+                                        N.stream_ptr()), "rb_swiglu_slots")
     return h
+
+
+def scatter_tokens(x: torch.Tensor, pl: MoEPlan) -> torch.Tensor:
+    """x [T, d] -> permuted [max_rows, d] for inference: like `gather`, but padding rows are left unwritten (no row of a
+    grouped product depends on another)."""
+    if not x.is_cuda:
+        return gather(x, pl)
+    T, d = x.shape
+    xp = torch.empty((pl.max_rows, d), dtype=x.dtype, device=x.device)
+    halves = d * (2 if x.dtype == torch.float32 else 1)                  # the kernel copies rows of 16-bit elements
+    N.check(N.kernels().rb_moe_scatter(x.contiguous().data_ptr(), pl.slot_pos.data_ptr(), xp.data_ptr(), T * pl.k, pl.k, halves,
+                                       N.stream_ptr()), "rb_moe_scatter")
+    return xp
 
 
 def route_backward(probs, idx, w, dw, counts, renorm: bool, aux_grad_scale: float):
@@ -150,9 +168,8 @@ def plan(idx: torch.Tensor, num_experts: int) -> MoEPlan:
     return pl
 
 
-def gather(x: torch.Tensor, pl: MoEPlan, slot_scale=None, zero_tail: bool = True) -> torch.Tensor:
-    """x [T, d] -> permuted [max_rows, d].  Padding rows inside the expert segments are zero; rows past the last segment
-    are zero as well, or (`zero_tail` False: inference, nothing reads them) left unwritten."""
+def gather(x: torch.Tensor, pl: MoEPlan, slot_scale=None) -> torch.Tensor:
+    """x [T, d] -> permuted [max_rows, d] (rows past the last expert segment are left untouched / zero)."""
     T, d = x.shape
     if not x.is_cuda:
         xp = torch.zeros((pl.max_rows, d), dtype=x.dtype)
@@ -162,13 +179,9 @@ def gather(x: torch.Tensor, pl: MoEPlan, slot_scale=None, zero_tail: bool = True
             src = src * slot_scale.reshape(-1)[pl.row_slot[ok].long()][:, None]
         xp[ok] = src.to(x.dtype)
         return xp
-    make = torch.zeros if zero_tail else torch.empty
-    xp = make((pl.max_rows, d), dtype=x.dtype, device=x.device)
-    if x.dtype == torch.float32 and slot_scale is not None:
-        raise TypeError("gather: fp32 rows are copied without a scale")
-    halves = d * (2 if x.dtype == torch.float32 else 1)                  # the kernel copies rows of 16-bit elements
+    xp = torch.zeros((pl.max_rows, d), dtype=x.dtype, device=x.device)   # rows past the last segment stay zero
     N.check(N.kernels().rb_moe_gather(x.contiguous().data_ptr(), pl.row_slot.data_ptr(), N.ptr(slot_scale), xp.data_ptr(),
-                                      pl.max_rows, pl.k, halves, pl.offsets[pl.num_experts:].data_ptr(), N.stream_ptr()),
+                                      pl.max_rows, pl.k, d, pl.offsets[pl.num_experts:].data_ptr(), N.stream_ptr()),
             "rb_moe_gather")
     return xp
 

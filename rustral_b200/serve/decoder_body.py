@@ -150,12 +150,11 @@ class LayeredBody:
         logits = gemm(h, P.w(p + "moe.router"), out_dtype=torch.float32)
         idx, w = moe_ops.route_groups(logits, m.top, m.groups, m.keep)
         pl = moe_ops.plan(idx, m.experts)
-        live = pl.offsets[m.experts:]
-        gu = moe_ops.grouped_gemm(moe_ops.gather(h, pl, zero_tail=False), P.w(p + "moe.w1"), pl)
-        y = moe_ops.grouped_gemm(moe_ops.swiglu_live(gu, live), P.w(p + "moe.w2"), pl)
+        gu = moe_ops.grouped_gemm(moe_ops.scatter_tokens(h, pl), P.w(p + "moe.w1"), pl)
+        y = moe_ops.grouped_gemm(moe_ops.swiglu_rows(gu, pl), P.w(p + "moe.w2"), pl)
         shared = None
         if m.shared_ff:
-            shared = gemm(moe_ops.swiglu_live(gemm(h, P.w(p + "shared.in"))), P.w(p + "shared.out"))
+            shared = gemm(moe_ops.swiglu_rows(gemm(h, P.w(p + "shared.in"))), P.w(p + "shared.out"))
         self._add_norm(st, y, p + "norm2", routed=(pl.slot_pos, w), add=shared)
 
     def head(self, st, rows):

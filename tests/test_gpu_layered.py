@@ -69,6 +69,17 @@ def test_flash_kernel_with_a_score_rule(case):
         close(out.view(L, -1), oracle_attention(q, k, v, scale, rule, None if g is None else gate), 1.5e-2, (case, g is not None))
 
 
+@pytest.mark.parametrize("sharp", [0.1, 1.0, 4.0, 16.0])
+def test_flash_kernel_cap_at_small_and_large_scores(sharp):
+    """Scores from far below the cap to far above it (the kernel evaluates the cap in two ways)."""
+    L, H, dk, dv, cap = 200, 2, 64, 64, 5.0
+    q, k, v, _ = qkv(L, L, H, 1, dk, dv, seed=7, sharp=sharp)
+    rule = ScoreRule(cap, distance_slopes(H, "cuda"), 90)
+    out = torch.empty(1, L, H, dv, dtype=BF16, device="cuda")
+    attn_ops.prompt_attention(dev(q, BF16)[None], dev(k, BF16)[None], dev(v, BF16)[None], 0.2, out, rule)
+    close(out.view(L, -1), oracle_attention(q, k, v, 0.2, rule), 1.5e-2, sharp)
+
+
 def paged(k, v, bs, dtype, seed=0):
     """One sequence's keys and values on scattered pages among pages full of other values."""
     S, G, dk = k.shape
@@ -197,8 +208,8 @@ def test_expert_products_over_live_rows(dtype):
             e = int(idx[t, j])
             want[t] += w[t, j] * ((O.silu(x[t] @ w1[e, :ff].T) * (x[t] @ w1[e, ff:].T)) @ w2[e].T)
     pl = moe_ops.plan(dev(idx), E)
-    xp = moe_ops.gather(dev(x, dtype), pl, zero_tail=False)
-    h = moe_ops.swiglu_live(moe_ops.grouped_gemm(xp, dev(w1, dtype), pl), pl.offsets[E:])
+    xp = moe_ops.scatter_tokens(dev(x, dtype), pl)
+    h = moe_ops.swiglu_rows(moe_ops.grouped_gemm(xp, dev(w1, dtype), pl), pl)
     y = moe_ops.grouped_gemm(h, dev(w2, dtype), pl)
     got = (y[pl.slot_pos.long()].float().view(T, k, d) * dev(w)[:, :, None]).sum(1)
     close(got, want, 2e-2 if dtype == BF16 else 1e-5)
