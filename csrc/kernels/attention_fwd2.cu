@@ -70,6 +70,11 @@ __device__ __forceinline__ uint64_t f2_fma2(uint64_t a, uint64_t b, uint64_t c) 
   asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(d) : "l"(a), "l"(b), "l"(c));
   return d;
 }
+__device__ __forceinline__ uint64_t f2_add2(uint64_t a, uint64_t b) {
+  uint64_t d;
+  asm("add.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b));
+  return d;
+}
 __device__ __forceinline__ uint64_t f2_mul2(uint64_t a, uint64_t b) {
   uint64_t d;
   asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b));
@@ -77,50 +82,50 @@ __device__ __forceinline__ uint64_t f2_mul2(uint64_t a, uint64_t b) {
 }
 
 // Capped scores of one thread's row, in place and in log2 units: r <- cap2 * tanh(c * r) + slope2 * i + bias0 (i: column).
-// For |c r| < sqrt(2) tanh(x) = x P(x^2), P the degree-7 Chebyshev interpolant of tanh(sqrt(y)) / sqrt(y) on [0, 2]
-// (largest error 4.3e-7): FMA-pipe work on packed pairs, since the special-function unit is what bounds this kernel.
-// Where a warp meets a larger argument it takes 1 - 2 / (1 + e^(2x)) for those 16 columns.
-__device__ __forceinline__ void f2_cap_scores(uint32_t (&r)[128], float c, float cap2, float slope2, float bias0) {
-  const uint64_t cc = f2_pack(c, c), cap = f2_pack(cap2, cap2), two_slope = f2_pack(2.f * slope2, 2.f * slope2);
-  const uint64_t k7 = f2_pack(-0.00011365948f, -0.00011365948f), k6 = f2_pack(0.00118971989f, 0.00118971989f);
-  const uint64_t k5 = f2_pack(-0.00589067675f, -0.00589067675f), k4 = f2_pack(0.0195360109f, 0.0195360109f);
-  const uint64_t k3 = f2_pack(-0.0528990813f, -0.0528990813f), k2 = f2_pack(0.133082107f, 0.133082107f);
-  const uint64_t k1 = f2_pack(-0.333310157f, -0.333310157f), k0 = f2_pack(0.999999642f, 0.999999642f);
+// For |c r| < sqrt(2) tanh(x) = x P(x^2), P the degree-6 Chebyshev interpolant of tanh(sqrt(y)) / sqrt(y) on [0, 2]
+// (largest error 2.0e-6), on packed pairs: no special-function instruction.  Where a warp meets a larger argument it
+// starts over from the raw scores with f2_cap_scores_wide.
+struct F2Cap {
+  uint64_t c, k[7];                                  // c and cap2 * coefficients, each in both halves
+  __device__ __forceinline__ void init(float c1, float cap2) {
+    const float k1[7] = {0.999997556f, -0.333212644f, 0.132326901f, -0.0506877862f, 0.0164362881f, -0.00365187856f, 0.00038573076f};
+    c = f2_pack(c1, c1);
 #pragma unroll
-  for (int g = 0; g < 8; ++g) {
-    uint64_t x[8], y[8];
-    uint32_t any = 0u;
+    for (int i = 0; i < 7; ++i) k[i] = f2_pack(cap2 * k1[i], cap2 * k1[i]);
+  }
+};
+// Returns the bits of all x^2 combined: the top exponent bit (30) says that one of them is >= 2.
+__device__ __forceinline__ uint32_t f2_cap_scores(uint32_t (&r)[128], const F2Cap& f, float slope2, float bias0) {
+  const uint64_t two_slope = f2_pack(2.f * slope2, 2.f * slope2);
+  uint32_t any = 0u;
 #pragma unroll
-    for (int i = 0; i < 8; ++i) {
-      x[i] = f2_mul2(f2_pack(__uint_as_float(r[g * 16 + 2 * i]), __uint_as_float(r[g * 16 + 2 * i + 1])), cc);
-      y[i] = f2_mul2(x[i], x[i]);
+  for (int g = 0; g < 4; ++g) {
+    uint64_t b = f2_pack(fmaf(slope2, static_cast<float>(g * 32), bias0), fmaf(slope2, static_cast<float>(g * 32 + 1), bias0));
+#pragma unroll
+    for (int i = 0; i < 16; ++i) {
+      uint32_t& r0 = r[g * 32 + 2 * i];
+      uint32_t& r1 = r[g * 32 + 2 * i + 1];
+      const uint64_t x = f2_mul2(f2_pack(__uint_as_float(r0), __uint_as_float(r1)), f.c);
+      const uint64_t y = f2_mul2(x, x);
       uint32_t lo, hi;
-      f2_unpack(y[i], lo, hi);
+      f2_unpack(y, lo, hi);
       any |= lo | hi;
-    }
-    uint64_t b = f2_pack(fmaf(slope2, static_cast<float>(g * 16), bias0), fmaf(slope2, static_cast<float>(g * 16 + 1), bias0));
-    if (!__any_sync(0xffffffffu, (any & 0x40000000u) != 0u)) {       // top exponent bit: some x^2 >= 2
+      uint64_t p = f2_fma2(y, f.k[6], f.k[5]);
 #pragma unroll
-      for (int i = 0; i < 8; ++i) {
-        uint64_t p = f2_fma2(y[i], k7, k6);
-        p = f2_fma2(p, y[i], k5);
-        p = f2_fma2(p, y[i], k4);
-        p = f2_fma2(p, y[i], k3);
-        p = f2_fma2(p, y[i], k2);
-        p = f2_fma2(p, y[i], k1);
-        p = f2_fma2(p, y[i], k0);
-        p = f2_fma2(f2_mul2(x[i], cap), p, b);
-        b = f2_fma2(two_slope, f2_pack(1.f, 1.f), b);
-        f2_unpack(p, r[g * 16 + 2 * i], r[g * 16 + 2 * i + 1]);
-      }
-    } else {
-#pragma unroll
-      for (int i = 0; i < 16; ++i) {
-        const float e = f2_ex2(__uint_as_float(r[g * 16 + i]) * (2.f * kF2Log2e) * c);
-        const float bias = fmaf(slope2, static_cast<float>(g * 16 + i), bias0);
-        r[g * 16 + i] = __float_as_uint(fmaf(-2.f * cap2, f2_rcp(1.f + e), cap2 + bias));
-      }
+      for (int q = 4; q >= 0; --q) p = f2_fma2(p, y, f.k[q]);
+      p = f2_fma2(x, p, b);
+      b = f2_add2(b, two_slope);
+      f2_unpack(p, r0, r1);
     }
+  }
+  return any;
+}
+// The same for arguments of any size: tanh(x) = 1 - 2 / (1 + e^(2x)).
+__device__ __forceinline__ void f2_cap_scores_wide(uint32_t (&r)[128], float c, float cap2, float slope2, float bias0) {
+#pragma unroll
+  for (int i = 0; i < 128; ++i) {
+    const float e = f2_ex2(__uint_as_float(r[i]) * (2.f * kF2Log2e) * c);
+    r[i] = __float_as_uint(fmaf(-2.f * cap2, f2_rcp(1.f + e), cap2 + fmaf(slope2, static_cast<float>(i), bias0)));
   }
 }
 // 2^x on the FMA / integer pipes: round-to-nearest split x = n + f, |f| <= 0.5, degree-4 polynomial for 2^f
@@ -356,6 +361,8 @@ attn_fwd2_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
     const float rule_c2 = RULE ? (p.softcap > 0.f ? p.softcap : p.scale) * kF2Log2e : 0.f;
     const float slope2 = RULE && p.slopes ? p.slopes[h] * kF2Log2e : 0.f;
     const int key_lo = RULE && p.chunk > 0 ? (q_idx + shift) / p.chunk * p.chunk : 0;      // first visible key of this row
+    F2Cap cap = {};
+    if (RULE) cap.init(rule_c1, rule_c2);
     float m_run = -INFINITY, l_run = 0.f;
     const int nt = n_of(t), ft = f_of(t);
     bool ok = true;
@@ -386,7 +393,13 @@ attn_fwd2_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
         // cap * tanh(s / cap), then - slope * (query - key)
         const float bias0 = -slope2 * static_cast<float>(q_idx + shift - k0);
         if (p.softcap > 0.f) {
-          f2_cap_scores(r, rule_c1, rule_c2, slope2, bias0);
+          const uint32_t any = f2_cap_scores(r, cap, slope2, bias0);
+          if (__any_sync(0xffffffffu, (any & 0x40000000u) != 0u)) {     // the raw scores are still in TMEM
+#pragma unroll
+            for (int c = 0; c < 4; ++c) tmem_ld_32x32_ptr(tmem_s + c * 32, r + c * 32);
+            tmem_ld_wait();
+            f2_cap_scores_wide(r, rule_c1, rule_c2, slope2, bias0);
+          }
         } else {
 #pragma unroll
           for (int i = 0; i < 128; ++i)
@@ -469,6 +482,13 @@ attn_fwd2_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
       __syncwarp();
       if (lane == 0) mbar_arrive(bar_pfull + 8 * t);
     }
+    uint4 gate_row[RULE ? DV / 8 : 1];                         // the gate of this row, requested while the last product runs
+    const bool gated = RULE && p.gate != nullptr && q_idx < p.seq_q;
+    if (gated) {
+#pragma unroll
+      for (int c = 0; c < DV / 8; ++c)
+        if (c * 8 < p.dv) gate_row[c % (RULE ? DV / 8 : 1)] = *reinterpret_cast<const uint4*>(p.gate + q_idx * p.ld_gate + h * p.dv + c * 8);
+    }
     if (ok && nt > 0) ok = mbar_wait(bar_oready + 8 * t, (nt - 1 - ft) & 1, abort_flag, status, 48);
     if (nt == 0 && q_idx < p.seq_q && q0 + t * kF2Tile < p.seq_q) {
       // no visible key at all (every key of this batch entry is padding): the output row is zero
@@ -491,8 +511,8 @@ attn_fwd2_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
 #pragma unroll
           for (int g = 0; g < 4; ++g) {
             if (RULE && c * 32 + g * 8 >= p.dv) break;
-            if (RULE && p.gate != nullptr) {
-              const uint4 gv = *reinterpret_cast<const uint4*>(p.gate + q_idx * p.ld_gate + h * p.dv + c * 32 + g * 8);
+            if (gated) {
+              const uint4 gv = gate_row[(c * 4 + g) % (RULE ? DV / 8 : 1)];
               const uint32_t gw[4] = {gv.x, gv.y, gv.z, gv.w};
 #pragma unroll
               for (int i = 0; i < 4; ++i) {
