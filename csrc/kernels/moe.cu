@@ -101,8 +101,10 @@ moe_route_bwd_kernel(const float* __restrict__ probs, const int* __restrict__ id
   if (lane + 32 < E) dlogits[static_cast<long long>(t) * E + lane + 32] = pv1 * (dp[1] - s);
 }
 
-// Router with group-limited choice: one warp per token.  Scores are kept in shared memory as order-preserving integer keys
-// (bits of a non-negative float + 1; 0 = not available), so an arg-max is two warp reductions.
+// Router with group-limited choice: one warp per token, R experts per lane (expert e = lane + 32 r).  Scores are held as
+// order-preserving integer keys (bits of a non-negative float + 1; 0 = not available), so an arg-max is two warp
+// reductions.  Shared memory is used for the group maxima only.
+template <int R>
 __global__ void __launch_bounds__(128)
 moe_route_groups_kernel(const float* __restrict__ logits, int T, int E, int k, int groups, int keep, int renorm, float eps,
                         int* __restrict__ idx, float* __restrict__ w) {
@@ -110,63 +112,74 @@ moe_route_groups_kernel(const float* __restrict__ logits, int T, int E, int k, i
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
   const int t = blockIdx.x * (blockDim.x >> 5) + warp;
   if (t >= T) return;
-  unsigned int* key = route_sm + warp * (E + groups);
-  unsigned int* gkey = key + E;
   const float* x = logits + static_cast<long long>(t) * E;
-  float mx = -INFINITY;
-  for (int e = lane; e < E; e += 32) mx = fmaxf(mx, x[e]);
+  float v[R];
+  unsigned int key[R];
+  float mx = -INFINITY, sum = 0.f;
+#pragma unroll
+  for (int r = 0; r < R; ++r) {
+    v[r] = lane + 32 * r < E ? x[lane + 32 * r] : -INFINITY;
+    mx = fmaxf(mx, v[r]);
+  }
   mx = warp_max(mx);
-  float sum = 0.f;
-  for (int e = lane; e < E; e += 32) {
-    const float p = __expf(x[e] - mx);
-    key[e] = __float_as_uint(p) + 1u;
+#pragma unroll
+  for (int r = 0; r < R; ++r) {
+    const float p = lane + 32 * r < E ? __expf(v[r] - mx) : 0.f;
+    key[r] = lane + 32 * r < E ? __float_as_uint(p) + 1u : 0u;
     sum += p;
   }
   const float inv = 1.f / warp_sum(sum);
-  __syncwarp();
-  // largest key of v[0 .. n), ties to the lower index; the chosen entry is set to 0
-  auto take = [&](unsigned int* v, int n, unsigned int& best) {
-    unsigned int bv = 0u;
-    int bi = n;
-    for (int e = lane; e < n; e += 32)
-      if (v[e] > bv) { bv = v[e]; bi = e; }
-    best = __reduce_max_sync(0xffffffffu, bv);
-    int at = __reduce_min_sync(0xffffffffu, bv == best ? bi : n);
-    if (at >= n) at = 0;                               // nothing available (scores that are not numbers)
-    if ((at & 31) == lane) v[at] = 0u;
-    __syncwarp();
-    return at;
-  };
-  unsigned int best;
   if (groups > 1 && keep < groups) {
+    unsigned int* all = route_sm + warp * (E + groups);
+    unsigned int* gkey = all + E;
     const int per = E / groups;
+#pragma unroll
+    for (int r = 0; r < R; ++r)
+      if (lane + 32 * r < E) all[lane + 32 * r] = key[r];
+    __syncwarp();
     for (int g = lane; g < groups; g += 32) {
       unsigned int m = 0u;
-      for (int e = g * per; e < (g + 1) * per; ++e) m = max(m, key[e]);
+      for (int e = g * per; e < (g + 1) * per; ++e) m = max(m, all[e]);
       gkey[g] = m;
     }
     __syncwarp();
-    for (int j = 0; j < keep; ++j) take(gkey, groups, best);           // kept groups end up as 0
-    for (int e = lane; e < E; e += 32)
-      if (gkey[e / per] != 0u) key[e] = 0u;
-    __syncwarp();
+    for (int j = 0; j < keep; ++j) {                   // the best groups, ties to the lower one, end up as 0
+      unsigned int bv = 0u;
+      int bi = groups;
+      for (int g = lane; g < groups; g += 32)
+        if (gkey[g] > bv) { bv = gkey[g]; bi = g; }
+      const unsigned int best = __reduce_max_sync(0xffffffffu, bv);
+      const int at = __reduce_min_sync(0xffffffffu, bv == best ? bi : groups);
+      if (at < groups && (at & 31) == lane) gkey[at] = 0u;
+      __syncwarp();
+    }
+#pragma unroll
+    for (int r = 0; r < R; ++r)
+      if (lane + 32 * r < E && gkey[(lane + 32 * r) / per] != 0u) key[r] = 0u;
   }
   float tot = 0.f, mine = 0.f;                         // lane j keeps the j-th weight (written in rounds of 32)
   int mine_e = 0;
   for (int j = 0; j < k; ++j) {
-    const int e = take(key, E, best);
+    unsigned int bv = 0u;
+    int bi = E;
+#pragma unroll
+    for (int r = 0; r < R; ++r)
+      if (key[r] > bv) { bv = key[r]; bi = lane + 32 * r; }
+    const unsigned int best = __reduce_max_sync(0xffffffffu, bv);
+    int at = __reduce_min_sync(0xffffffffu, bv == best ? bi : E);
+    if (at >= E) at = 0;                               // nothing available (scores that are not numbers)
+#pragma unroll
+    for (int r = 0; r < R; ++r)
+      if (at == lane + 32 * r) key[r] = 0u;
     const float p = best ? __uint_as_float(best - 1u) * inv : 0.f;
     tot += p;
-    if ((j & 31) == lane) { mine = p; mine_e = e; }
-    if ((j & 31) == 31 || j == k - 1) {
-      const int slot = (j & ~31) + lane;
-      if (slot < k) {
-        idx[static_cast<long long>(t) * k + slot] = mine_e;
-        w[static_cast<long long>(t) * k + slot] = mine;
-      }
+    if ((j & 31) == lane) { mine = p; mine_e = at; }
+    if (((j & 31) == 31 || j == k - 1) && (j & ~31) + lane < k) {
+      idx[static_cast<long long>(t) * k + (j & ~31) + lane] = mine_e;
+      w[static_cast<long long>(t) * k + (j & ~31) + lane] = renorm && k <= 32 ? mine / (tot + eps) : mine;
     }
   }
-  if (renorm) {
+  if (renorm && k > 32) {
     __syncwarp();
     for (int j = lane; j < k; j += 32) w[static_cast<long long>(t) * k + j] /= tot + eps;
   }
@@ -394,9 +407,14 @@ RB_API int rb_moe_route_groups(const float* logits, int T, int E, int k, int gro
   if (groups < 1) groups = 1;
   if (keep < 1 || keep > groups) keep = groups;
   if (T <= 0 || E <= 0 || k <= 0 || k > E || E % groups || k > keep * (E / groups)) return -1;
-  const size_t smem = sizeof(float) * 4 * static_cast<size_t>(E + groups);
-  if (smem > 48 * 1024) return -1;
-  rb::moe_route_groups_kernel<<<(T + 3) / 4, 128, smem, RB_ST>>>(logits, T, E, k, groups, keep, renorm, eps, idx, w);
+  const size_t smem = groups > 1 && keep < groups ? sizeof(float) * 4 * static_cast<size_t>(E + groups) : 0;
+  const int grid = (T + 3) / 4;
+  if (E <= 32) rb::moe_route_groups_kernel<1><<<grid, 128, smem, RB_ST>>>(logits, T, E, k, groups, keep, renorm, eps, idx, w);
+  else if (E <= 64) rb::moe_route_groups_kernel<2><<<grid, 128, smem, RB_ST>>>(logits, T, E, k, groups, keep, renorm, eps, idx, w);
+  else if (E <= 128) rb::moe_route_groups_kernel<4><<<grid, 128, smem, RB_ST>>>(logits, T, E, k, groups, keep, renorm, eps, idx, w);
+  else if (E <= 256) rb::moe_route_groups_kernel<8><<<grid, 128, smem, RB_ST>>>(logits, T, E, k, groups, keep, renorm, eps, idx, w);
+  else if (E <= 1024) rb::moe_route_groups_kernel<32><<<grid, 128, smem, RB_ST>>>(logits, T, E, k, groups, keep, renorm, eps, idx, w);
+  else return -1;
   return static_cast<int>(cudaGetLastError());
 }
 RB_API int rb_swiglu_slots(const void* gu, long long ld_gu, void* h, long long ld_h, int n, int F, int f32,

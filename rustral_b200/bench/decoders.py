@@ -125,7 +125,7 @@ def kernels(s, T: int = 8192, B: int = 64, ctx: int = 4000, iters: int = 10) -> 
             lname, lfn, lroof = like
             lms = _time(lfn, iters, flush=flush)
             e["like"] = {"kernel": lname, "ms": round(lms, 4), "of_roofline": round(lroof * 1e3 / lms, 3)}
-            e["times_further"] = round(e["like"]["of_roofline"] / max(e["of_roofline"], 1e-9), 2)
+            e["times_further"] = round((lroof / lms) / (roof_s / ms), 2)
         out[name] = e
 
     # ---- attention: 4096 tokens of one prompt (one chunk), B decoded rows

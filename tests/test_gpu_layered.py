@@ -186,7 +186,7 @@ def test_residual_norm(n, dtype):
             close(xd, xw, 1e-5)                              # the residual is 32-bit in both
 
 
-@pytest.mark.parametrize("E,k,groups,keep", [(16, 2, 2, 1), (12, 3, 3, 2), (128, 8, 8, 4), (256, 8, 8, 2), (1, 1, 1, 1), (6, 6, 1, 1), (40, 5, 40, 6)])
+@pytest.mark.parametrize("E,k,groups,keep", [(16, 2, 2, 1), (12, 3, 3, 2), (128, 8, 8, 4), (256, 8, 8, 2), (1, 1, 1, 1), (6, 6, 1, 1), (40, 5, 40, 6), (80, 40, 1, 1), (600, 4, 6, 3)])
 def test_router(E, k, groups, keep):
     logits = 2 * torch.randn(133, E, generator=torch.Generator().manual_seed(E))
     iw, ww = moe_ops.route_groups(logits, k, groups, keep)
