@@ -46,7 +46,7 @@ def qkv(L, S, H, G, dk, dv, seed=0, sharp=1.0):
 
 
 PROMPTS = [  # L, S, heads, kv heads, dk, dv, cap, chunk
-    (1, 1, 2, 1, 64, 64, 8.0, 0), (2, 2, 2, 2, 8, 8, 8.0, 16), (130, 130, 4, 2, 96, 64, 0.0, 0), (300, 300, 4, 1, 96, 64, 20.0, 64),
+    (1, 1, 2, 1, 64, 64, 8.0, 0), (2, 2, 2, 2, 8, 8, 8.0, 16), (130, 130, 4, 2, 96, 64, 0.0, 0), (300, 300, 4, 1, 88, 56, 17.0, 48),
     (257, 700, 2, 1, 128, 128, 15.0, 300), (256, 256, 2, 2, 64, 128, 9.0, 128), (513, 513, 2, 1, 128, 64, 9.0, 256),
     (2, 200, 4, 2, 48, 40, 30.0, 127), (140, 141, 2, 1, 32, 72, 30.0, 1), (600, 1000, 2, 1, 72, 24, 12.0, 129),
     (384, 1024, 1, 1, 112, 104, 12.0, 513), (129, 400, 6, 3, 64, 32, 6.0, 4096), (700, 700, 2, 1, 80, 96, 10.0, 200),
@@ -93,7 +93,7 @@ def paged(k, v, bs, dtype, seed=0):
 
 
 DECODES = [  # context, heads, kv heads, dk, dv, cap, chunk, page
-    (1, 2, 1, 64, 64, 8.0, 0, 16), (17, 4, 2, 96, 64, 20.0, 16, 16), (16, 4, 2, 96, 64, 20.0, 16, 16), (700, 8, 2, 128, 128, 15.0, 0, 16),
+    (1, 2, 1, 64, 64, 8.0, 0, 16), (17, 4, 2, 96, 56, 18.0, 16, 16), (16, 4, 2, 96, 56, 18.0, 16, 16), (700, 8, 2, 128, 128, 15.0, 0, 16),
     (900, 8, 1, 128, 64, 0.0, 513, 16), (257, 40, 2, 64, 96, 9.0, 256, 4), (333, 4, 4, 48, 40, 9.0, 300, 64), (300, 6, 3, 8, 128, 9.0, 1, 16),
 ]
 

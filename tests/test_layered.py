@@ -290,6 +290,22 @@ def test_trace_replay_refuses_what_does_not_fit():
         rep.step([{"id": "x", "tokens": [1], "want": []}], [])
 
 
+def test_trace_replay_refuses_32_bit_for_families_that_lack_it(tmp_path):
+    from rustral_b200.serve.trace_run import main
+    (tmp_path / "config.json").write_text(json.dumps({"architecture": "llama", "vocab_size": 64, "n_head": 4, "d_model": 64, "n_layer": 1}))
+    assert main(["--model", str(tmp_path), "--dtype", "float32", "--out", str(tmp_path), "--max-tokens", "64"]) == 3
+
+
+def test_kernel_files_of_every_architecture_exist_and_cover_what_they_include():
+    from rustral_b200 import _build
+    for a in ARCHITECTURES.values():
+        for stem in a.kernels:
+            assert (_build.CSRC / "kernels" / f"{stem}.cu").exists(), (a.name, stem)
+    heads = list((_build.CSRC / "kernels").glob("*.h")) + list((_build.CSRC / "kernels").glob("*.cuh"))
+    names = {h.name for h in _build._included(_build.CSRC / "kernels" / "moe.cu", heads)}
+    assert names == {"moe.h", "rb_common.cuh"}
+
+
 def test_server_command_line_serves_a_model_folder(tmp_path):
     import urllib.request
 
