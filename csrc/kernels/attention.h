@@ -21,15 +21,19 @@ typedef struct RbAttnArgs {
 } RbAttnArgs;
 // Score rule of an inference forward pass (causal, queries aligned to the end of the keys, key 0 is the start of a chunk):
 //   s = q . k * scale; softcap > 0: s <- softcap * tanh(s / softcap); slopes (fp32 [heads]): s <- s - slopes[h] * (i - j);
-//   chunk > 0: i sees j only when i / chunk == j / chunk; gate (bf16 [seq_q, heads * v_dim], pitch ld_gate, batch 1):
-//   the output is multiplied by sigmoid(gate)
+//   chunk > 0: i sees j only when i / chunk == j / chunk; window > 0 (without chunk): i sees j only when i - j < window or
+//   j < keep_first; sink: a further score 0 without a value takes part in the softmax; gate (bf16 [seq_q, heads * v_dim], pitch
+//   ld_gate, batch 1) or head_gate (fp32 [seq_q, heads], pitch ld_gate, batch 1): the output is multiplied by sigmoid(gate)
+//   With window and keep_first the keys may leave out positions between the kept ones and the first query's window.
 typedef struct RbAttnRule {
   int v_dim;               // value head size (RbAttnArgs.head_dim is the query / key size)
   float softcap;
   const float* slopes;
   int chunk;
   const void* gate;
+  const float* head_gate;
   long long ld_gate;
+  int window, keep_first, sink;
 } RbAttnRule;
 int rb_attention_fwd_rule(const RbAttnArgs* args, const RbAttnRule* rule, void* stream);
 int rb_attention_fwd(const RbAttnArgs* args, void* stream);

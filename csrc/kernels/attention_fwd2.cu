@@ -14,8 +14,9 @@
 // polynomial on the FMA pipe (template parameter; off by default, see rb_attention_fwd_tc2).  Warp 8 is the TMA producer (Q once, K / V through a ring of stages), warp 9 issues MMAs.
 //
 // The RULE form serves inference of decoders with their own score rule: separate key / value head sizes (columns beyond the
-// real sizes are zero-filled by TMA), capped scores, a linear distance bias, chunked visibility (key blocks before a
-// tile's first visible chunk are skipped, so the two tiles may start at different blocks) and a sigmoid output gate.
+// real sizes are zero-filled by TMA), capped scores, a linear distance bias, chunked or windowed visibility (key blocks before a
+// tile's first visible key are skipped, so the two tiles may start at different blocks), first keys that a window keeps (their
+// blocks are walked before the window's), a sink in the softmax and a sigmoid output gate per value column or per head.
 //
 // Same semantics as the other forward kernels (causal alignment to the end of the keys, GQA, log-sum-exp output).
 // Replaces the reference's materialised-score attention (crates/nn/src/attention.rs:640-836).
@@ -43,7 +44,9 @@ struct F2Params {
   const float* slopes;      // [heads] or NULL
   int chunk;                // 0: none; key 0 starts a chunk
   const __nv_bfloat16* gate;   // [seq_q, heads * dv] or NULL
+  const float* head_gate;      // [seq_q, heads] or NULL
   long long ld_gate;
+  int window, keep, sink;
 };
 
 __device__ __forceinline__ float f2_ex2(float x) {
@@ -226,15 +229,29 @@ attn_fwd2_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
     }
     return n;
   };
-  const int n_a = blocks_of(q0), n_b = blocks_of(q0 + kF2Tile);
-  auto n_of = [&](int t) { return t == 0 ? n_a : n_b; };
-  const int n_max = n_a > n_b ? n_a : n_b;
-  // first key block of each tile: the one that holds the start of its first row's chunk.  Tile A starts first, and tile B
+  int n_a = blocks_of(q0), n_b = blocks_of(q0 + kF2Tile);
+  // first key block of each tile: the one that holds the first key its first row sees.  Tile A starts first, and tile B
   // starts no later than one block after tile A's last.
   auto first_of = [&](int t) {
-    return RULE && p.chunk > 0 ? (q0 + t * kF2Tile + shift) / p.chunk * p.chunk / kF2Tile : 0;
+    const int pos = q0 + t * kF2Tile + shift;
+    if (RULE && p.chunk > 0) return pos / p.chunk * p.chunk / kF2Tile;
+    if (RULE && p.window > 0) return max(0, pos - p.window + 1) / kF2Tile;
+    return 0;
   };
-  const int f_a = first_of(0), f_b = first_of(1);
+  int f_a = first_of(0), f_b = first_of(1);
+  // Kept first keys: both tiles walk their blocks (kept_blocks of them) before those of tile A's window, and the counters below
+  // number the blocks in that order; block_at gives the key block.
+  int kept_blocks = 0, skipped = 0;
+  if (RULE && p.window > 0 && p.keep > 0 && n_a > 0) {
+    kept_blocks = (p.keep + kF2Tile - 1) / kF2Tile;
+    skipped = max(0, f_a - kept_blocks);
+    n_a -= skipped;
+    n_b = max(0, n_b - skipped);
+    f_a = f_b = 0;
+  }
+  auto block_at = [&](int j) { return RULE && j >= kept_blocks ? j + skipped : j; };
+  auto n_of = [&](int t) { return t == 0 ? n_a : n_b; };
+  const int n_max = n_a > n_b ? n_a : n_b;
   auto f_of = [&](int t) { return t == 0 ? f_a : f_b; };
   const int f_min = n_a > 0 ? f_a : f_b;
   constexpr uint32_t kTmemCols = 512;
@@ -285,11 +302,11 @@ attn_fwd2_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
         mbar_arrive_expect_tx(bar_kfull + 8 * s, L::kTileBytes);
 #pragma unroll
         for (int hf = 0; hf < D / 64; ++hf)
-          tma_load_4d(sK + s * L::kTileBytes + hf * L::kHalf, &tmK, hf * 64, hk, j * kF2Tile, b, bar_kfull + 8 * s);
+          tma_load_4d(sK + s * L::kTileBytes + hf * L::kHalf, &tmK, hf * 64, hk, block_at(j) * kF2Tile, b, bar_kfull + 8 * s);
         mbar_arrive_expect_tx(bar_vfull + 8 * s, L::kVTileBytes);
 #pragma unroll
         for (int hf = 0; hf < DV / 64; ++hf)
-          tma_load_4d(sV + s * L::kVTileBytes + hf * L::kHalf, &tmV, hf * 64, hk, j * kF2Tile, b, bar_vfull + 8 * s);
+          tma_load_4d(sV + s * L::kVTileBytes + hf * L::kHalf, &tmV, hf * 64, hk, block_at(j) * kF2Tile, b, bar_vfull + 8 * s);
       }
     }
   } else if (warp == 9) {
@@ -360,16 +377,19 @@ attn_fwd2_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
     const float rule_c1 = RULE && p.softcap > 0.f ? p.scale / p.softcap : 0.f;
     const float rule_c2 = RULE ? (p.softcap > 0.f ? p.softcap : p.scale) * kF2Log2e : 0.f;
     const float slope2 = RULE && p.slopes ? p.slopes[h] * kF2Log2e : 0.f;
-    const int key_lo = RULE && p.chunk > 0 ? (q_idx + shift) / p.chunk * p.chunk : 0;      // first visible key of this row
+    // first visible key of this row, apart from the kept ones below key_keep
+    const int key_lo = !RULE ? 0 : p.chunk > 0 ? (q_idx + shift) / p.chunk * p.chunk : p.window > 0 ? q_idx + shift - p.window + 1 : 0;
+    const int key_keep = RULE && p.window > 0 ? p.keep : 0;
     F2Cap cap = {};
     if (RULE) cap.init(rule_c1, rule_c2);
-    float m_run = -INFINITY, l_run = 0.f;
+    // a sink is a score 0 met before all keys
+    float m_run = RULE && p.sink ? 0.f : -INFINITY, l_run = RULE && p.sink ? 1.f : 0.f;
     const int nt = n_of(t), ft = f_of(t);
     bool ok = true;
     for (int j = ft; j < nt && ok; ++j) {
       if (!mbar_wait(bar_sfull + 8 * t, (j - ft) & 1, abort_flag, status, 46)) { ok = false; break; }
       tc_fence_after();
-      const int k0 = j * kF2Tile;
+      const int k0 = block_at(j) * kF2Tile;
       const int key_lim = p.causal ? min(kv_len - 1, q_idx + shift) : kv_len - 1;     // last visible key
       const bool need_mask = (k0 + kF2Tile - 1 > key_lim);
       float mx0 = -INFINITY, mx1 = -INFINITY, mx2 = -INFINITY, mx3 = -INFINITY;
@@ -408,7 +428,7 @@ attn_fwd2_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
         if (k0 < key_lo) {
 #pragma unroll
           for (int i = 0; i < 128; ++i)
-            if (k0 + i < key_lo) r[i] = 0xff800000u;
+            if (k0 + i < key_lo && k0 + i >= key_keep) r[i] = 0xff800000u;
         }
       }
       if (need_mask) {                               // only blocks that cross the causal diagonal or the end of the keys
@@ -500,7 +520,9 @@ attn_fwd2_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
     }
     if (ok && nt > 0) {
       tc_fence_after();
-      const float inv = l_run > 0.f ? 1.f / l_run : 0.f;
+      float inv = l_run > 0.f ? 1.f / l_run : 0.f;
+      if (RULE && p.head_gate != nullptr && q_idx < p.seq_q)
+        inv *= f2_rcp(1.f + f2_ex2(-p.head_gate[q_idx * p.ld_gate + h] * kF2Log2e));
       __nv_bfloat16* op = p.out + b * p.o_bs + h * p.o_hs + static_cast<long long>(q_idx) * p.o_rs;
 #pragma unroll
       for (int c = 0; c < DV / 32; ++c) {
@@ -630,7 +652,9 @@ RB_API int rb_attention_fwd_rule(const RbAttnArgs* a, const RbAttnRule* r, void*
   const int dk = a->head_dim, dv = r->v_dim;
   if (a->batch <= 0 || a->heads <= 0 || a->kv_heads <= 0 || a->heads % a->kv_heads) return -1;
   if (dk <= 0 || dv <= 0 || dk > 128 || dv > 128 || ((dk | dv) & 7)) return -9;
-  if (!a->causal || a->seq_q <= 0 || a->seq_k < a->seq_q || r->chunk < 0 || (r->gate && a->batch != 1)) return -1;
+  if (!a->causal || a->seq_q <= 0 || a->seq_k < a->seq_q || r->chunk < 0 || r->window < 0 || r->keep_first < 0 || (r->window && r->chunk) ||
+      ((r->gate || r->head_gate) && a->batch != 1) || (r->gate && r->head_gate))
+    return -1;
   const void* ptrs[5] = {a->q, a->k, a->v, a->o, r->gate};
   for (int i = 0; i < 5; ++i)
     if ((!ptrs[i] && i < 4) || (reinterpret_cast<uintptr_t>(ptrs[i]) & 15)) return -9;
@@ -638,7 +662,7 @@ RB_API int rb_attention_fwd_rule(const RbAttnArgs* a, const RbAttnRule* r, void*
   for (int i = 0; i < 4; ++i)
     for (int j = 0; j < 3; ++j)
       if (strs[i][j] % 8 || strs[i][j] <= 0) return -9;            // TMA strides are multiples of 16 bytes
-  if (r->ld_gate % 8) return -9;
+  if (r->gate && r->ld_gate % 8) return -9;
   int err = 0;
   const CUtensorMap* tq = f2_make_map(a->q, a->q_strides, a->seq_q, a->heads, a->batch, dk, &err);
   const CUtensorMap* tk = f2_make_map(a->k, a->k_strides, a->seq_k, a->kv_heads, a->batch, dk, &err);
@@ -651,6 +675,7 @@ RB_API int rb_attention_fwd_rule(const RbAttnArgs* a, const RbAttnRule* r, void*
   p.scale = a->scale;
   p.dk = dk; p.dv = dv; p.softcap = r->softcap; p.slopes = r->slopes; p.chunk = r->chunk;
   p.gate = reinterpret_cast<const __nv_bfloat16*>(r->gate); p.ld_gate = r->ld_gate;
+  p.head_gate = r->head_gate; p.window = r->window; p.keep = r->window > 0 ? r->keep_first : 0; p.sink = r->sink;
   cudaStream_t stream = reinterpret_cast<cudaStream_t>(stream_v);
   const dim3 grid((a->seq_q + 2 * rb::kF2Tile - 1) / (2 * rb::kF2Tile), a->heads, a->batch);
   if (dk <= 64)

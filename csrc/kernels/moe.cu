@@ -185,8 +185,8 @@ moe_route_groups_kernel(const float* __restrict__ logits, int T, int E, int k, i
   }
 }
 
-// silu(gate) * up over the rows that hold a token
-template <typename T, int N>
+// act(gate) * up over the rows that hold a token; act: silu, or relu
+template <typename T, int N, bool RELU>
 __global__ void __launch_bounds__(256)
 swiglu_slots_kernel(const T* __restrict__ gu, long long ld_gu, T* __restrict__ h, long long ld_h, int n, int F,
                     const int* __restrict__ slot_pos) {
@@ -204,14 +204,14 @@ swiglu_slots_kernel(const T* __restrict__ gu, long long ld_gu, T* __restrict__ h
 #pragma unroll
       for (int j = 0; j < 4; ++j) {
         const float2 a = unpack_bf16x2(gw[j]), b = unpack_bf16x2(uw[j]);
-        o[j] = pack_bf16x2(silu(a.x) * b.x, silu(a.y) * b.y);
+        o[j] = RELU ? pack_bf16x2(fmaxf(a.x, 0.f) * b.x, fmaxf(a.y, 0.f) * b.y) : pack_bf16x2(silu(a.x) * b.x, silu(a.y) * b.y);
       }
       *reinterpret_cast<uint4*>(h + r * ld_h + c) = make_uint4(o[0], o[1], o[2], o[3]);
     } else {
 #pragma unroll
       for (int j = 0; j < N; ++j) {
         const float g = static_cast<float>(gu[r * ld_gu + c + j]), u = static_cast<float>(gu[r * ld_gu + F + c + j]);
-        h[r * ld_h + c + j] = static_cast<T>(g / (1.f + expf(-g)) * u);
+        h[r * ld_h + c + j] = static_cast<T>((RELU ? fmaxf(g, 0.f) : g / (1.f + expf(-g))) * u);
       }
     }
   }
@@ -417,21 +417,29 @@ RB_API int rb_moe_route_groups(const float* logits, int T, int E, int k, int gro
   else return -1;
   return static_cast<int>(cudaGetLastError());
 }
-RB_API int rb_swiglu_slots(const void* gu, long long ld_gu, void* h, long long ld_h, int n, int F, int f32,
-                           const int* slot_pos, void* stream_v) {
-  if (n <= 0 || F <= 0) return -1;
+namespace {
+template <bool RELU>
+int glu_launch(const void* gu, long long ld_gu, void* h, long long ld_h, int n, int F, int f32, const int* slot_pos, cudaStream_t s) {
   const bool vec = !f32 && !((F | ld_gu | ld_h) & 7) && !((reinterpret_cast<uintptr_t>(gu) | reinterpret_cast<uintptr_t>(h)) & 15);
   const int grid = rb::grid1d(static_cast<long long>(n) * (vec ? F / 8 : F), 256);
   if (f32)
-    rb::swiglu_slots_kernel<float, 1><<<grid, 256, 0, RB_ST>>>(reinterpret_cast<const float*>(gu), ld_gu,
-                                                              reinterpret_cast<float*>(h), ld_h, n, F, slot_pos);
+    rb::swiglu_slots_kernel<float, 1, RELU><<<grid, 256, 0, s>>>(reinterpret_cast<const float*>(gu), ld_gu,
+                                                                reinterpret_cast<float*>(h), ld_h, n, F, slot_pos);
   else if (vec)
-    rb::swiglu_slots_kernel<__nv_bfloat16, 8><<<grid, 256, 0, RB_ST>>>(reinterpret_cast<const __nv_bfloat16*>(gu), ld_gu,
-                                                                      reinterpret_cast<__nv_bfloat16*>(h), ld_h, n, F, slot_pos);
+    rb::swiglu_slots_kernel<__nv_bfloat16, 8, RELU><<<grid, 256, 0, s>>>(reinterpret_cast<const __nv_bfloat16*>(gu), ld_gu,
+                                                                        reinterpret_cast<__nv_bfloat16*>(h), ld_h, n, F, slot_pos);
   else
-    rb::swiglu_slots_kernel<__nv_bfloat16, 1><<<grid, 256, 0, RB_ST>>>(reinterpret_cast<const __nv_bfloat16*>(gu), ld_gu,
-                                                                      reinterpret_cast<__nv_bfloat16*>(h), ld_h, n, F, slot_pos);
+    rb::swiglu_slots_kernel<__nv_bfloat16, 1, RELU><<<grid, 256, 0, s>>>(reinterpret_cast<const __nv_bfloat16*>(gu), ld_gu,
+                                                                        reinterpret_cast<__nv_bfloat16*>(h), ld_h, n, F, slot_pos);
   return static_cast<int>(cudaGetLastError());
+}
+}  // namespace
+
+RB_API int rb_swiglu_slots(const void* gu, long long ld_gu, void* h, long long ld_h, int n, int F, int f32,
+                           const int* slot_pos, int relu, void* stream_v) {
+  if (n <= 0 || F <= 0) return -1;
+  return relu ? glu_launch<true>(gu, ld_gu, h, ld_h, n, F, f32, slot_pos, RB_ST)
+              : glu_launch<false>(gu, ld_gu, h, ld_h, n, F, f32, slot_pos, RB_ST);
 }
 RB_API int rb_moe_scatter(const void* x, const int* slot_pos, void* xp, int slots, int k, int dim, void* stream_v) {
   if (slots <= 0 || k <= 0 || dim <= 0 || (dim % 8)) return -1;

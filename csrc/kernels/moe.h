@@ -19,10 +19,11 @@ int rb_moe_route_bwd(const float* probs, const int* idx, const float* w, const f
 // scores are taken (ties to the lower index) and divided by (their sum + eps) when renorm != 0.  groups <= 1: no limit.
 int rb_moe_route_groups(const float* logits, int T, int E, int k, int groups, int keep, int renorm, float eps, int* idx,
                         float* w, void* stream);
-// h[r, :] = silu(gu[r, 0:F]) * gu[r, F:2F] for the rows r = slot_pos[0 .. n) (NULL: r = 0 .. n).  bf16 or fp32.  The permuted
+// h[r, :] = act(gu[r, 0:F]) * gu[r, F:2F] for the rows r = slot_pos[0 .. n) (NULL: r = 0 .. n); act: silu, or relu when relu is
+// set.  bf16 or fp32.  The permuted
 // expert buffers are sized for whole tiles per expert; going by slots touches only the rows that hold a token.
 int rb_swiglu_slots(const void* gu, long long ld_gu, void* h, long long ld_h, int n, int F, int f32, const int* slot_pos,
-                    void* stream);
+                    int relu, void* stream);
 // xp[slot_pos[s], :] = x[s / k, :] for the slots s < slots; padding rows of xp are not written (inference).  16-bit elements.
 int rb_moe_scatter(const void* x, const int* slot_pos, void* xp, int slots, int k, int dim, void* stream);
 // Plan of the permutation: slots s = t * k + j are grouped by expert, in ascending slot order inside an expert

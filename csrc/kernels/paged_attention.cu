@@ -79,20 +79,38 @@ __device__ __forceinline__ float pa_sigmoid(float x) { return __fdividef(1.f, 1.
 // of a tcgen05 tile, which is why this kernel is on the warp-level tensor path; it is bound by the K / V reads.
 //
 // DK / DV are the key / value head sizes rounded up to a compiled size; columns beyond the real sizes are zero-filled in
-// shared memory and never leave it.  RULE adds a score cap, a distance bias and chunked visibility (see RbPagedRowsArgs).
+// shared memory and never leave it.  RULE adds a score cap, a distance bias, chunked or windowed visibility, a
+// sink and output gates (see RbPagedRowsArgs).  A window's slices cover the kept first tokens and then the window.
 struct PaRule {
   float softcap;
   const float* slopes;
   int chunk;
   const __nv_bfloat16* gate;
+  const float* head_gate;
   long long ld_g;
+  int window, keep, sink;
 };
 // cap * tanh(s / cap) as cap * (1 - 2 / (1 + e^(2 s / cap))): two special-function instructions, absolute error about
 // 1e-7 * cap (tanh.approx would be off by 5e-4 of the score)
 __device__ __forceinline__ float pa_softcap(float s, float cap, float two_over_cap) {
   return fmaf(-2.f * cap, __fdividef(1.f, 1.f + __expf(s * two_over_cap)), cap);
 }
-__device__ __forceinline__ int pa_first_key(int ctx, int chunk) { return chunk > 0 ? (ctx - 1) / chunk * chunk : 0; }
+// The visible tokens of a sequence, numbered without gaps: number v is token v below `kept`, else token v + gap.
+struct PaVisible {
+  int kept, gap, count;
+};
+__device__ __forceinline__ PaVisible pa_visible(int ctx, const PaRule& r) {
+  if (r.window > 0) {
+    const int kept = min(r.keep, ctx), lo = max(kept, ctx - r.window);
+    return {kept, lo - kept, ctx - (lo - kept)};
+  }
+  const int lo = r.chunk > 0 ? (ctx - 1) / r.chunk * r.chunk : 0;
+  return {0, lo, ctx - lo};
+}
+__device__ __forceinline__ float pa_gate(const PaRule& r, long long row, int head, long long col) {
+  if (r.gate) return pa_sigmoid(__bfloat162float(r.gate[row * r.ld_g + col]));
+  return r.head_gate ? pa_sigmoid(r.head_gate[row * r.ld_g + head]) : 1.f;
+}
 
 template <int DK, int DV, bool RULE>
 __global__ void __launch_bounds__(kPaWarps * 32, 3)
@@ -115,9 +133,10 @@ paged_decode_split_kernel(const __nv_bfloat16* __restrict__ q, long long ld_q, c
   const int gq = lane >> 2, tq = lane & 3;   // fragment coordinates: row (and row + 8), column pair
   const int group = heads / kv_heads;
   const int ctx = context_lens[b];
-  const int t_begin = (RULE ? pa_first_key(ctx, rule.chunk) : 0) + sp * kSplitTokens;
-  if (t_begin >= ctx) return;
-  const int t_end = min(ctx, t_begin + kSplitTokens);
+  const PaVisible vis = RULE ? pa_visible(ctx, rule) : PaVisible{0, 0, ctx};
+  const int t_begin = sp * kSplitTokens;
+  if (t_begin >= vis.count) return;
+  const int t_end = min(vis.count, t_begin + kSplitTokens);
   const int h_base = hk * group + g0;        // first query head of this pass
   const uint32_t kt_u32 = smem_u32(reinterpret_cast<__nv_bfloat16*>(big) + warp * (kKTile + kVTile));
   const uint32_t vt_u32 = kt_u32 + kKTile * 2;
@@ -155,9 +174,10 @@ paged_decode_split_kernel(const __nv_bfloat16* __restrict__ q, long long ld_q, c
   int n_next = 0;
   // cache slots of the 32 tokens that start at `first` (the host bounds num_blocks * block_size below 2^31)
   auto locate = [&](int first) {
-    const int tok = first + lane;
+    const int num = first + lane;
     slot = -1;
-    if (tok < t_end) {
+    if (num < t_end) {
+      const int tok = RULE && num >= vis.kept ? num + vis.gap : num;
       const int blk_idx = tok / block_size;
       int blk = blk_idx < max_blocks ? block_tables[static_cast<long long>(b) * max_blocks + blk_idx] : -1;
       if (blk < 0 || blk >= num_blocks) {                            // corrupt tables read block 0 instead of faulting
@@ -232,7 +252,8 @@ paged_decode_split_kernel(const __nv_bfloat16* __restrict__ q, long long ld_q, c
             v0 = pa_softcap(v0, rule.softcap, two_over_cap);
             v1 = pa_softcap(v1, rule.softcap, two_over_cap);
           }
-          const float dist = static_cast<float>(ctx - 1 - (base + n * 8 + 2 * tq + j));
+          const int num = base + n * 8 + 2 * tq + j;
+          const float dist = static_cast<float>(ctx - 1 - (num < vis.kept ? num : num + vis.gap));
           v0 = fmaf(-slope0, dist, v0);
           v1 = fmaf(-slope1, dist, v1);
         }
@@ -317,8 +338,13 @@ paged_decode_split_kernel(const __nv_bfloat16* __restrict__ q, long long ld_q, c
     }
     if (direct_out) {                        // a single slice: this is the result
       const long long col = static_cast<long long>(h_base + g) * dv + d;
+      if (RULE && rule.sink) {               // a score 0 without a value
+        const float top = fmaxf(mx, 0.f), sc = __expf(mx - top);
+        num *= sc;
+        den = fmaf(den, sc, __expf(-top));
+      }
       float o = num / den;
-      if (RULE && rule.gate) o *= pa_sigmoid(__bfloat162float(rule.gate[b * rule.ld_g + col]));
+      if (RULE) o *= pa_gate(rule, b, h_base + g, col);
       direct_out[b * ld_o + col] = __float2bfloat16(o);
       continue;
     }
@@ -335,11 +361,12 @@ paged_decode_merge_kernel(const float* __restrict__ partial, const int* __restri
   const int b = blockIdx.x, h = blockIdx.y, d = threadIdx.x;
   if (d >= dv) return;
   const int ctx = context_lens[b];
-  const int n = min(nsplit, (ctx - pa_first_key(ctx, rule.chunk) + kSplitTokens - 1) / kSplitTokens);
+  const int n = min(nsplit, (pa_visible(ctx, rule).count + kSplitTokens - 1) / kSplitTokens);
   const float* base = partial + (static_cast<long long>(b) * heads + h) * nsplit * (dv + 2);
   float mx = -INFINITY;
   for (int s = 0; s < n; ++s) mx = fmaxf(mx, base[s * (dv + 2)]);
-  float num = 0.f, den = 0.f;
+  if (rule.sink) mx = fmaxf(mx, 0.f);
+  float num = 0.f, den = rule.sink ? __expf(-mx) : 0.f;      // a sink is a score 0 without a value
   for (int s = 0; s < n; ++s) {
     const float ms = base[s * (dv + 2)];
     const float sc = (ms == -INFINITY) ? 0.f : __expf(ms - mx);
@@ -348,7 +375,7 @@ paged_decode_merge_kernel(const float* __restrict__ partial, const int* __restri
   }
   const long long col = static_cast<long long>(h) * dv + d;
   float o = den > 0.f ? num / den : 0.f;
-  if (rule.gate) o *= pa_sigmoid(__bfloat162float(rule.gate[b * rule.ld_g + col]));
+  o *= pa_gate(rule, b, h, col);
   out[static_cast<long long>(b) * ld_o + col] = __float2bfloat16(o);
 }
 
@@ -376,19 +403,24 @@ paged_rows_kernel(const RbPagedRowsArgs a RB_BOUNDS_PARAM) {
   __syncwarp();
   const long long pos = a.row_pos[r];
   const int* table = a.block_tables + static_cast<long long>(a.row_seq[r]) * a.max_blocks;
-  const long long lo = a.chunk > 0 ? pos / a.chunk * a.chunk : 0;
+  // visible keys are numbered without gaps: number v is key v below `kept`, else key v + gap
+  const long long kept = a.window > 0 ? (a.keep_first < pos + 1 ? a.keep_first : pos + 1) : 0;
+  long long gap = a.chunk > 0 ? pos / a.chunk * a.chunk : a.window > 0 ? pos + 1 - a.window - kept : 0;
+  if (gap < 0) gap = 0;
+  const long long count = pos + 1 - gap;
   const float slope = a.slopes ? a.slopes[h] : 0.f;
   const T* K = reinterpret_cast<const T*>(a.k_cache);
   const T* V = reinterpret_cast<const T*>(a.v_cache);
   float acc[kPrMaxV];
 #pragma unroll
   for (int i = 0; i < kPrMaxV; ++i) acc[i] = 0.f;
-  float m = -INFINITY, l = 0.f;
-  for (long long j0 = lo; j0 <= pos; j0 += 32) {
-    const long long j = j0 + lane;
+  float m = a.sink ? 0.f : -INFINITY, l = a.sink ? 1.f : 0.f;        // a sink is a score 0 met before all keys
+  for (long long j0 = 0; j0 < count; j0 += 32) {
+    const long long num = j0 + lane;
+    const long long j = num < kept ? num : num + gap;
     long long slot = 0;
     float s = -INFINITY;
-    if (j <= pos) {
+    if (num < count) {
       const long long bi = j / a.block_size;
       int blk = bi < a.max_blocks ? table[bi] : -1;
       if (blk < 0 || blk >= a.num_blocks) {                          // corrupt tables read block 0 instead of faulting
@@ -405,26 +437,26 @@ paged_rows_kernel(const RbPagedRowsArgs a RB_BOUNDS_PARAM) {
     }
     const float mn = fmaxf(m, warp_max(s));                          // finite: key j0 is always visible
     const float al = m == -INFINITY ? 0.f : expf(m - mn);
-    const float p = j <= pos ? expf(s - mn) : 0.f;
+    const float p = num < count ? expf(s - mn) : 0.f;
     l = l * al + warp_sum(p);
     m = mn;
 #pragma unroll
     for (int i = 0; i < kPrMaxV; ++i) acc[i] *= al;
-    const int n = static_cast<int>(pos - j0 + 1 < 32 ? pos - j0 + 1 : 32);
+    const int n = static_cast<int>(count - j0 < 32 ? count - j0 : 32);
     for (int jj = 0; jj < n; ++jj) {
       const float pj = __shfl_sync(0xffffffffu, p, jj);
       const long long sj = __shfl_sync(0xffffffffu, slot, jj);
-      const T* v = V + (sj * a.kv_heads + hk) * a.dv;
+      const T* vals = V + (sj * a.kv_heads + hk) * a.dv;
 #pragma unroll
       for (int i = 0; i < kPrMaxV; ++i) {
         const int c = i * 32 + lane;
-        if (c < a.dv) acc[i] = fmaf(pj, pr_get(v + c), acc[i]);
+        if (c < a.dv) acc[i] = fmaf(pj, pr_get(vals + c), acc[i]);
       }
     }
   }
   T* o = reinterpret_cast<T*>(a.out) + r * a.ld_o + static_cast<long long>(h) * a.dv;
   const T* g = a.gate ? reinterpret_cast<const T*>(a.gate) + r * a.ld_g + static_cast<long long>(h) * a.dv : nullptr;
-  const float inv = 1.f / l;
+  const float inv = a.head_gate ? 1.f / (l * (1.f + expf(-a.head_gate[r * a.ld_g + h]))) : 1.f / l;
 #pragma unroll
   for (int i = 0; i < kPrMaxV; ++i) {
     const int c = i * 32 + lane;
@@ -480,6 +512,7 @@ int pd_launch(const RbPagedDecodeArgs& a, cudaStream_t stream) {
   const int group = a.heads / a.kv_heads;
   long long span = static_cast<long long>(a.max_blocks) * a.block_size;      // most keys a row can see
   if (a.chunk > 0 && a.chunk < span) span = a.chunk;
+  if (a.window > 0 && static_cast<long long>(a.window) + a.keep_first < span) span = a.window + a.keep_first;
   const int nsplit = static_cast<int>((span + rb::kSplitTokens - 1) / rb::kSplitTokens);
   // dynamic shared memory: per warp a K and a V tile of 32 padded rows, plus the 16 padded query rows
   const int smem = (rb::kPaWarps * 32 * (DK + 8 + DV + 8) + rb::kMaxGroup * (DK + 8)) * 2;
@@ -493,7 +526,8 @@ int pd_launch(const RbPagedDecodeArgs& a, cudaStream_t stream) {
     attr_set[dev] = true;
   }
   auto O = reinterpret_cast<__nv_bfloat16*>(a.out);
-  const rb::PaRule rule = {a.softcap, a.slopes, a.chunk, reinterpret_cast<const __nv_bfloat16*>(a.gate), a.ld_g};
+  const rb::PaRule rule = {a.softcap, a.slopes, a.chunk, reinterpret_cast<const __nv_bfloat16*>(a.gate), a.head_gate, a.ld_g,
+                           a.window, a.keep_first, a.sink};
   const dim3 grid(a.batch, a.kv_heads, nsplit);
   for (int g0 = 0; g0 < group; g0 += rb::kMaxGroup)       // groups wider than 16 heads take several passes
     kern<<<grid, rb::kPaWarps * 32, smem, stream>>>(

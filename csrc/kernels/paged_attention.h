@@ -20,7 +20,7 @@ int rb_paged_attention_decode(const void* q, long long ld_q, void* out, long lon
                               int batch, int heads, int kv_heads, int head_dim, int block_size, long long num_blocks,
                               float scale, float* scratch, void* stream);
 // The same decode attention with separate key / value head sizes (multiples of 8, at most 128), a score rule and an output
-// gate; softcap, slopes, chunk and gate as in RbPagedRowsArgs below.  bf16 operands.  scratch: fp32
+// gate; softcap, slopes, chunk, window, sink and gates as in RbPagedRowsArgs below.  bf16 operands.  scratch: fp32
 // [rb_paged_attention_scratch_floats(batch, heads, dv, max_blocks, block_size)].
 typedef struct RbPagedDecodeArgs {
   const void* q;             // [batch, heads * dk], pitch ld_q
@@ -31,19 +31,23 @@ typedef struct RbPagedDecodeArgs {
   const int* context_lens;
   const float* slopes;
   const void* gate;          // [batch, heads * dv], pitch ld_g
+  const float* head_gate;    // [batch, heads], pitch ld_g
   float* scratch;
   long long ld_q, ld_o, ld_g, num_blocks;
-  int batch, max_blocks, heads, kv_heads, dk, dv, block_size, chunk;
+  int batch, max_blocks, heads, kv_heads, dk, dv, block_size, chunk, window, keep_first, sink;
   float scale, softcap;
 } RbPagedDecodeArgs;
 int rb_paged_attention_decode_rule(const RbPagedDecodeArgs* args, void* stream);
 // Attention over the pages for any rows of a batch (prompt portions and decoded tokens alike), any head sizes, bf16 or
 // fp32 operands, fp32 arithmetic: the 32-bit mode and the fallback for head sizes the tensor-core kernels do not take.
 //   row r is the token at position row_pos[r] of the sequence whose pages are block_tables[row_seq[r]]; it sees the keys
-//   j <= pos, and with chunk > 0 only those with j / chunk == pos / chunk
+//   j <= pos, and with chunk > 0 only those with j / chunk == pos / chunk, with window > 0 only those with pos - j < window or
+//   j < keep_first
+//   sink: a further score 0 without a value takes part in the softmax
 //   score = q . k * scale; softcap > 0: score <- softcap * tanh(score / softcap); slopes (fp32 [heads], or NULL):
 //   score <- score - slopes[h] * (pos - j)
-//   gate (type of q, pitch ld_g, [rows, heads * dv], or NULL): the output is multiplied by sigmoid(gate)
+//   gate (type of q, pitch ld_g, [rows, heads * dv], or NULL) or head_gate (fp32 [rows, heads], pitch ld_g, or NULL): the output
+//   is multiplied by sigmoid(gate)
 typedef struct RbPagedRowsArgs {
   const void* q;
   void* out;
@@ -54,8 +58,9 @@ typedef struct RbPagedRowsArgs {
   const long long* row_pos;
   const float* slopes;
   const void* gate;
+  const float* head_gate;
   long long ld_q, ld_o, ld_g, num_blocks;
-  int f32, rows, max_blocks, heads, kv_heads, dk, dv, block_size, chunk;
+  int f32, rows, max_blocks, heads, kv_heads, dk, dv, block_size, chunk, window, keep_first, sink;
   float scale, softcap;
 } RbPagedRowsArgs;
 int rb_paged_attention_rows(const RbPagedRowsArgs* args, void* stream);

@@ -2,6 +2,9 @@
 // next matrix product.  The source is a plain row (attention output projection) or the weighted sum of a token's expert
 // rows plus the shared expert's row, so a routed feed-forward's combine, norm and residual add are one launch.
 // Statistics, sums and the residual are fp32; one CTA owns a row and keeps it in registers.
+//
+// The second kernel serves blocks whose sublayers are computed side by side: up to two RMS-normed outputs and a plain one are
+// added to the residual, and the dynamic tanh in front of the next block is taken on the way.
 #include "residual_norm.h"
 
 #include "rb_common.cuh"
@@ -129,7 +132,89 @@ int rn_launch(const RbResidualNormArgs& a, cudaStream_t s) {
   return static_cast<int>(cudaGetLastError());
 }
 
+template <int VEC, int CH>
+__global__ void __launch_bounds__(256)
+stream_update_kernel(const RbStreamUpdateArgs a) {
+  __shared__ float red[8];
+  const int t = blockIdx.x, n = a.n;
+  float x[CH][VEC], va[CH][VEC], vb[CH][VEC], v[CH][VEC];
+  float sa = 0.f, sb = 0.f;
+#pragma unroll
+  for (int c = 0; c < CH; ++c) {
+    const int col = (c * blockDim.x + threadIdx.x) * VEC;
+#pragma unroll
+    for (int i = 0; i < VEC; ++i) { x[c][i] = 0.f; va[c][i] = 0.f; vb[c][i] = 0.f; v[c][i] = 0.f; }
+    if (col >= n) continue;
+    rn_load<VEC>(a.x, t * a.ldx + col, 1, x[c]);
+    if (a.a) rn_load<VEC>(a.a, t * a.lda + col, a.y_f32, va[c]);
+    if (a.b) rn_load<VEC>(a.b, t * a.ldb + col, a.y_f32, vb[c]);
+    if (a.c) rn_load<VEC>(a.c, t * a.ldc + col, a.y_f32, v[c]);
+#pragma unroll
+    for (int i = 0; i < VEC; ++i) { sa = fmaf(va[c][i], va[c][i], sa); sb = fmaf(vb[c][i], vb[c][i], sb); }
+  }
+  const float inv_n = 1.f / static_cast<float>(n);
+  const float ra = a.a ? a.normed / sqrtf(rn_block_sum(sa, red) * inv_n + a.eps) : 0.f;
+  const float rb_ = a.b ? a.normed / sqrtf(rn_block_sum(sb, red) * inv_n + a.eps) : 0.f;
+  const bool add = a.a || a.b || a.c;
+  const float alpha = a.h ? a.alpha[0] : 0.f;
+#pragma unroll
+  for (int c = 0; c < CH; ++c) {
+    const int col = (c * blockDim.x + threadIdx.x) * VEC;
+    if (col >= n) continue;
+    float w[VEC];
+    if (a.a) {
+      rn_load<VEC>(a.wa, col, 1, w);
+#pragma unroll
+      for (int i = 0; i < VEC; ++i) v[c][i] = fmaf(va[c][i] * ra, w[i], v[c][i]);
+    }
+    if (a.b) {
+      rn_load<VEC>(a.wb, col, 1, w);
+#pragma unroll
+      for (int i = 0; i < VEC; ++i) v[c][i] = fmaf(vb[c][i] * rb_, w[i], v[c][i]);
+    }
+    if (add) {
+#pragma unroll
+      for (int i = 0; i < VEC; ++i) x[c][i] = fmaf(a.mult, v[c][i], x[c][i]);
+      rn_store<VEC>(a.x, t * a.ldx + col, 1, x[c]);
+    }
+    if (a.h) {
+      float b[VEC], o[VEC];
+      rn_load<VEC>(a.gamma, col, 1, w);
+      rn_load<VEC>(a.beta, col, 1, b);
+#pragma unroll
+      for (int i = 0; i < VEC; ++i) o[i] = fmaf(tanhf(alpha * x[c][i]), w[i], b[i]);
+      rn_store<VEC>(a.h, t * a.ldh + col, a.h_f32, o);
+    }
+  }
+}
+
+template <int VEC>
+int su_launch(const RbStreamUpdateArgs& a, cudaStream_t s) {
+  const int units = (a.n + VEC - 1) / VEC;
+  const int threads = units <= 64 ? 64 : units <= 128 ? 128 : 256;
+  const int ch = (units + threads - 1) / threads;
+  if (ch <= 1) stream_update_kernel<VEC, 1><<<a.rows, threads, 0, s>>>(a);
+  else if (ch <= 2) stream_update_kernel<VEC, 2><<<a.rows, threads, 0, s>>>(a);
+  else if (ch <= 4) stream_update_kernel<VEC, 4><<<a.rows, threads, 0, s>>>(a);
+  else if (ch <= 8) stream_update_kernel<VEC, 8><<<a.rows, threads, 0, s>>>(a);
+  else if (ch <= 16) stream_update_kernel<VEC, 16><<<a.rows, threads, 0, s>>>(a);
+  else return -6;
+  return static_cast<int>(cudaGetLastError());
+}
+
 }  // namespace rb
+
+RB_API int rb_stream_update(const RbStreamUpdateArgs* args, void* stream_v) {
+  const RbStreamUpdateArgs& a = *args;
+  if (a.rows <= 0) return 0;
+  if (a.n <= 0 || !a.x || (a.a && !a.wa) || (a.b && !a.wb) || (a.h && (!a.alpha || !a.gamma || !a.beta))) return -1;
+  const void* ptrs[9] = {a.a, a.b, a.c, a.wa, a.wb, a.x, a.gamma, a.beta, a.h};
+  uintptr_t bits = 0;
+  for (int i = 0; i < 9; ++i) bits |= reinterpret_cast<uintptr_t>(ptrs[i]);
+  const bool vec = !(bits & 15) && !((a.n | a.lda | a.ldb | a.ldc | a.ldx | a.ldh) & 3);
+  cudaStream_t s = reinterpret_cast<cudaStream_t>(stream_v);
+  return vec ? rb::su_launch<4>(a, s) : rb::su_launch<1>(a, s);
+}
 
 RB_API int rb_residual_norm(const RbResidualNormArgs* args, void* stream_v) {
   const RbResidualNormArgs& a = *args;

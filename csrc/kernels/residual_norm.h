@@ -19,6 +19,25 @@ typedef struct RbResidualNormArgs {
   float eps;
 } RbResidualNormArgs;
 int rb_residual_norm(const RbResidualNormArgs* args, void* stream);
+// Update of a residual stream behind a block whose sublayers were computed side by side, and the dynamic tanh in front of the
+// next block:  x += mult * (normed * rms(a) * wa + normed * rms(b) * wb + c),   h = tanh(alpha x) * gamma + beta
+// a, b, c share their type (y_f32); any may be NULL; rms over the row with eps inside the root; a and b come with a weight.
+typedef struct RbStreamUpdateArgs {
+  const void* a;
+  const void* b;
+  const void* c;
+  const float* wa;          // [n]
+  const float* wb;          // [n]
+  float* x;                 // fp32 [rows, n], in place (only read when a, b and c are NULL)
+  const float* alpha;       // [1]
+  const float* gamma;       // [n]
+  const float* beta;        // [n]
+  void* h;                  // bf16 or fp32 [rows, n], or NULL (then alpha, gamma and beta are not read)
+  long long lda, ldb, ldc, ldx, ldh;
+  int y_f32, h_f32, rows, n;
+  float mult, normed, eps;
+} RbStreamUpdateArgs;
+int rb_stream_update(const RbStreamUpdateArgs* args, void* stream);
 #ifdef __cplusplus
 }
 #endif

@@ -1,4 +1,5 @@
-// Paged-KV block allocator: a free list of fixed-size blocks and one block table per sequence.
+// Paged-KV block allocator: a free list of fixed-size blocks and one block table per sequence, and for models with
+// recurrent layers a free list of state slots of which every sequence holds one from its first reservation to its end.
 // Semantics follow the reference's PagedCache (crates/nn/src/kv_cache.rs:382-432) with its defect removed: a
 // second reservation for a sequence extends the table instead of overwriting it (kv_cache.rs:420-423).
 #include <mutex>
@@ -11,6 +12,9 @@ struct RbBlockAllocator {
   int num_blocks, block_size;
   std::vector<int32_t> free_list;                                // stack; lowest ids are handed out first
   std::unordered_map<int64_t, std::vector<int32_t>> tables;
+  bool slotted = false;                                          // sequences also hold a state slot
+  std::vector<int32_t> free_slots;
+  std::unordered_map<int64_t, int32_t> slots;
   mutable std::mutex mu;
 };
 
@@ -25,6 +29,24 @@ RbBlockAllocator* rb_ba_create(int num_blocks, int block_size) {
   for (int i = num_blocks - 1; i >= 0; --i) a->free_list.push_back(i);
   return a;
 }
+// Every sequence from now on also takes one of `num_slots` state slots; call it before the first reservation.
+int rb_ba_set_state_slots(RbBlockAllocator* a, int num_slots) {
+  std::lock_guard<std::mutex> l(a->mu);
+  if (num_slots <= 0 || !a->tables.empty()) return -1;
+  a->slotted = true;
+  a->free_slots.clear();
+  for (int i = num_slots - 1; i >= 0; --i) a->free_slots.push_back(i);
+  return 0;
+}
+int rb_ba_state_slot(const RbBlockAllocator* a, int64_t seq_id) {
+  std::lock_guard<std::mutex> l(a->mu);
+  auto it = a->slots.find(seq_id);
+  return it == a->slots.end() ? -1 : it->second;
+}
+int rb_ba_num_free_slots(const RbBlockAllocator* a) {
+  std::lock_guard<std::mutex> l(a->mu);
+  return (int)a->free_slots.size();
+}
 void rb_ba_destroy(RbBlockAllocator* a) { delete a; }
 int rb_ba_num_free(const RbBlockAllocator* a) { std::lock_guard<std::mutex> l(a->mu); return (int)a->free_list.size(); }
 int rb_ba_num_blocks(const RbBlockAllocator* a) { return a->num_blocks; }
@@ -37,6 +59,7 @@ int rb_ba_can_reserve(const RbBlockAllocator* a, int64_t seq_id, int num_tokens)
   auto it = a->tables.find(seq_id);
   const int have = it == a->tables.end() ? 0 : (int)it->second.size();
   const int need = blocks_for(a, num_tokens) - have;
+  if (a->slotted && it == a->tables.end() && a->free_slots.empty()) return 0;
   return need <= (int)a->free_list.size() ? 1 : 0;
 }
 
@@ -46,11 +69,17 @@ int rb_ba_reserve(RbBlockAllocator* a, int64_t seq_id, int num_tokens) {
   auto it = a->tables.find(seq_id);
   const int have = it == a->tables.end() ? 0 : (int)it->second.size();
   const int need = blocks_for(a, num_tokens) - have;
+  const bool fresh = it == a->tables.end();
+  if (need > (int)a->free_list.size()) return -1;
+  if (fresh && a->slotted) {
+    if (a->free_slots.empty()) return -1;
+    a->slots[seq_id] = a->free_slots.back();
+    a->free_slots.pop_back();
+  }
   if (need <= 0) {
-    if (it == a->tables.end()) a->tables[seq_id];
+    if (fresh) a->tables[seq_id];
     return 0;
   }
-  if (need > (int)a->free_list.size()) return -1;
   auto& tab = a->tables[seq_id];
   for (int i = 0; i < need; ++i) {
     tab.push_back(a->free_list.back());
@@ -66,6 +95,11 @@ int rb_ba_free(RbBlockAllocator* a, int64_t seq_id) {
   const int n = (int)it->second.size();
   for (auto rit = it->second.rbegin(); rit != it->second.rend(); ++rit) a->free_list.push_back(*rit);
   a->tables.erase(it);
+  auto st = a->slots.find(seq_id);
+  if (st != a->slots.end()) {
+    a->free_slots.push_back(st->second);
+    a->slots.erase(st);
+  }
   return n;
 }
 

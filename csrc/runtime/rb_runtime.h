@@ -23,6 +23,11 @@ int rb_ba_table_len(const RbBlockAllocator* a, int64_t seq_id);
 int rb_ba_table(const RbBlockAllocator* a, int64_t seq_id, int32_t* out, int max_out);   // copies the table; returns its length
 int64_t rb_ba_slot(const RbBlockAllocator* a, int64_t seq_id, int token_index);          // block * block_size + offset, -1 if unmapped
 int rb_ba_num_sequences(const RbBlockAllocator* a);
+// State slots of models with recurrent layers: once set, a sequence's first reservation takes a free slot (and fails without
+// one) and rb_ba_free gives it back.
+int rb_ba_set_state_slots(RbBlockAllocator* a, int num_slots);
+int rb_ba_state_slot(const RbBlockAllocator* a, int64_t seq_id);                         // -1: none
+int rb_ba_num_free_slots(const RbBlockAllocator* a);
 
 // ---- tile-configuration search (autotuner core) --------------------------------------------------------------
 // A search space is a list of dimensions, each with a list of integer choices.  Strategies: 0 grid, 1 random,

@@ -54,7 +54,8 @@ class RbAttnArgs(C.Structure):
 
 
 class RbAttnRule(C.Structure):
-    _fields_ = [("v_dim", c_int), ("softcap", c_float), ("slopes", c_void_p), ("chunk", c_int), ("gate", c_void_p), ("ld_gate", c_ll)]
+    _fields_ = [("v_dim", c_int), ("softcap", c_float), ("slopes", c_void_p), ("chunk", c_int), ("gate", c_void_p),
+                ("head_gate", c_void_p), ("ld_gate", c_ll), ("window", c_int), ("keep_first", c_int), ("sink", c_int)]
 
 
 class RbResidualNormArgs(C.Structure):
@@ -79,20 +80,68 @@ class RbHeadPrepArgs(C.Structure):
 class RbPagedRowsArgs(C.Structure):
     _fields_ = [
         ("q", c_void_p), ("out", c_void_p), ("k_cache", c_void_p), ("v_cache", c_void_p), ("block_tables", c_void_p),
-        ("row_seq", c_void_p), ("row_pos", c_void_p), ("slopes", c_void_p), ("gate", c_void_p),
+        ("row_seq", c_void_p), ("row_pos", c_void_p), ("slopes", c_void_p), ("gate", c_void_p), ("head_gate", c_void_p),
         ("ld_q", c_ll), ("ld_o", c_ll), ("ld_g", c_ll), ("num_blocks", c_ll),
         ("f32", c_int), ("rows", c_int), ("max_blocks", c_int), ("heads", c_int), ("kv_heads", c_int), ("dk", c_int),
-        ("dv", c_int), ("block_size", c_int), ("chunk", c_int), ("scale", c_float), ("softcap", c_float),
+        ("dv", c_int), ("block_size", c_int), ("chunk", c_int), ("window", c_int), ("keep_first", c_int), ("sink", c_int),
+        ("scale", c_float), ("softcap", c_float),
     ]
 
 
 class RbPagedDecodeArgs(C.Structure):
     _fields_ = [
         ("q", c_void_p), ("out", c_void_p), ("k_cache", c_void_p), ("v_cache", c_void_p), ("block_tables", c_void_p),
-        ("context_lens", c_void_p), ("slopes", c_void_p), ("gate", c_void_p), ("scratch", c_void_p),
+        ("context_lens", c_void_p), ("slopes", c_void_p), ("gate", c_void_p), ("head_gate", c_void_p),
+        ("scratch", c_void_p),
         ("ld_q", c_ll), ("ld_o", c_ll), ("ld_g", c_ll), ("num_blocks", c_ll),
         ("batch", c_int), ("max_blocks", c_int), ("heads", c_int), ("kv_heads", c_int), ("dk", c_int), ("dv", c_int),
-        ("block_size", c_int), ("chunk", c_int), ("scale", c_float), ("softcap", c_float),
+        ("block_size", c_int), ("chunk", c_int), ("window", c_int), ("keep_first", c_int), ("sink", c_int),
+        ("scale", c_float), ("softcap", c_float),
+    ]
+
+
+class RbStreamUpdateArgs(C.Structure):
+    _fields_ = [
+        ("a", c_void_p), ("b", c_void_p), ("c", c_void_p), ("wa", c_void_p), ("wb", c_void_p), ("x", c_void_p),
+        ("alpha", c_void_p), ("gamma", c_void_p), ("beta", c_void_p), ("h", c_void_p),
+        ("lda", c_ll), ("ldb", c_ll), ("ldc", c_ll), ("ldx", c_ll), ("ldh", c_ll),
+        ("y_f32", c_int), ("h_f32", c_int), ("rows", c_int), ("n", c_int),
+        ("mult", c_float), ("normed", c_float), ("eps", c_float),
+    ]
+
+
+class RbShortConvArgs(C.Structure):
+    _fields_ = [
+        ("x", c_void_p), ("out", c_void_p), ("state", c_void_p), ("w", c_void_p), ("bias", c_void_p), ("segments", c_void_p),
+        ("tiles", c_void_p), ("ld_x", c_ll), ("ld_o", c_ll),
+        ("num_tiles", c_int), ("channels", c_int), ("taps", c_int), ("f32", c_int), ("silu", c_int), ("num_slots", c_int),
+    ]
+
+
+class RbStateSpaceArgs(C.Structure):
+    _fields_ = [
+        ("xbc", c_void_p), ("dt_raw", c_void_p), ("dt_bias", c_void_p), ("a_log", c_void_p), ("D", c_void_p), ("state", c_void_p),
+        ("y", c_void_p), ("segments", c_void_p), ("tiles", c_void_p), ("ld_xbc", c_ll), ("ld_dt", c_ll), ("ld_y", c_ll),
+        ("num_segments", c_int), ("num_tiles", c_int), ("heads", c_int), ("groups", c_int), ("p", c_int), ("n", c_int),
+        ("f32", c_int), ("num_slots", c_int),
+    ]
+
+
+class RbDeltaRuleArgs(C.Structure):
+    _fields_ = [
+        ("qkv", c_void_p), ("a_raw", c_void_p), ("b_raw", c_void_p), ("dt_bias", c_void_p), ("a_log", c_void_p),
+        ("state", c_void_p), ("o", c_void_p), ("segments", c_void_p), ("tiles", c_void_p), ("scratch", c_void_p),
+        ("ld_qkv", c_ll), ("ld_ab", c_ll), ("ld_o", c_ll),
+        ("num_segments", c_int), ("num_tiles", c_int), ("heads", c_int), ("kv_heads", c_int), ("dk", c_int), ("dv", c_int),
+        ("f32", c_int), ("num_slots", c_int),
+    ]
+
+
+class RbGatedNormArgs(C.Structure):
+    _fields_ = [
+        ("y", c_void_p), ("z", c_void_p), ("out", c_void_p), ("weight", c_void_p), ("ld_y", c_ll), ("ld_z", c_ll), ("ld_o", c_ll),
+        ("rows", c_int), ("parts", c_int), ("part_n", c_int), ("weight_n", c_int), ("f32", c_int), ("gate_first", c_int),
+        ("eps", c_float),
     ]
 
 

@@ -31,7 +31,7 @@ def declare_cpu(lib) -> None:
 def declare_runtime(lib) -> None:
     _sig(lib, "rb_ba_create", [I, I], P)
     _sig(lib, "rb_ba_destroy", [P])
-    for n in ("rb_ba_num_free", "rb_ba_num_blocks", "rb_ba_block_size", "rb_ba_num_sequences"):
+    for n in ("rb_ba_num_free", "rb_ba_num_blocks", "rb_ba_block_size", "rb_ba_num_sequences", "rb_ba_num_free_slots"):
         _sig(lib, n, [P], I)
     _sig(lib, "rb_ba_reserve", [P, LL, I], I)
     _sig(lib, "rb_ba_can_reserve", [P, LL, I], I)
@@ -39,6 +39,8 @@ def declare_runtime(lib) -> None:
     _sig(lib, "rb_ba_table_len", [P, LL], I)
     _sig(lib, "rb_ba_table", [P, LL, P, I], I)
     _sig(lib, "rb_ba_slot", [P, LL, I], LL)
+    _sig(lib, "rb_ba_set_state_slots", [P, I], I)
+    _sig(lib, "rb_ba_state_slot", [P, LL], I)
     _sig(lib, "rb_search_create", [I, I, P, P, C.c_uint64, I], P)
     _sig(lib, "rb_search_destroy", [P])
     _sig(lib, "rb_search_next", [P, P], I)

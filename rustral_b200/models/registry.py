@@ -56,11 +56,14 @@ _GPT_KERNELS = ("gemm_tcgen05", "embedding", "elementwise", "norm", "rope", "att
                 "paged_attention", "optim")
 _LAYERED_KERNELS = ("gemm_tcgen05", "gemm_f32", "embedding", "elementwise", "residual_norm", "head_prep", "moe",
                     "attention_fwd2", "paged_attention")
+_HYBRID_KERNELS = ("gemm_tcgen05", "gemm_f32", "embedding", "elementwise", "residual_norm", "head_prep", "moe", "attention_fwd2",
+                   "paged_attention", "short_conv", "state_space", "delta_rule", "gated_norm")
 
 ARCHITECTURES = {a.name: a for a in (
     Architecture("gpt2", _gpt_config, "GPTBody", False, _gpt_weights, _GPT_KERNELS),
     Architecture("llama", _gpt_config, "GPTBody", False, _gpt_weights, _GPT_KERNELS),
     Architecture("Dolurax", LayeredConfig.from_json, "LayeredBody", True, _layered_weights, _LAYERED_KERNELS),
+    Architecture("Vafodra", LayeredConfig.from_json, "ParallelBody", True, _layered_weights, _HYBRID_KERNELS),
 )}
 
 

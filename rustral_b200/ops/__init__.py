@@ -5,10 +5,11 @@ PyTorch route (the native library must be loaded), a CPU tensor takes the fp32 r
 also serves as the numerical oracle in the tests.
 """
 from .matmul import gemm, linear, act_reference, act_grad_reference
-from .norm import layer_norm, rms_norm, norm_forward, norm_backward, residual_norm
+from .norm import layer_norm, rms_norm, norm_forward, norm_backward, residual_norm, stream_update
 from .loss import cross_entropy, cross_entropy_fwd_bwd, softmax, log_softmax
 from .attention import flash_attention, attention_reference, ScoreRule, distance_slopes
 from .heads import head_prep_
+from .recurrent import Segments, delta_rule, gated_norm, short_conv, state_space
 from .embed import embedding, embedding_forward, embedding_backward, embedding_residual
 from .elementwise import (binary, unary, scalar_op, unary_bwd, add_row_vector, sum_dim0, sum_all, transpose2d,
                           gather_rows, scatter_rows, broadcast_to, strided_copy, apply_mask, dropout, argmax_rows,

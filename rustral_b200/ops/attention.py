@@ -15,18 +15,38 @@ class ScoreRule:
 
     softcap > 0: score <- softcap * tanh(score / softcap).  slopes (fp32 [heads]): score <- score - slopes[h] * (i - j), after
     the cap.  chunk > 0: position i sees j only when i // chunk == j // chunk (positions of the sequence; a kernel that is
-    handed keys from a chunk's first one on may count from there)."""
+    handed keys from a chunk's first one on may count from there).  window > 0: position i sees j only when i - j < window or
+    j < keep_first (a kernel may be handed the kept keys and then those from the first query's window on).  sink: a further
+    score 0 without a value takes part in the softmax."""
     softcap: float = 0.0
     slopes: torch.Tensor | None = None
     chunk: int = 0
+    window: int = 0
+    keep_first: int = 0
+    sink: bool = False
 
     def first_key(self, pos: int) -> int:
-        """The first position that the token at `pos` can see."""
+        """The first position that the token at `pos` can see, apart from the kept ones."""
+        if self.window:
+            return max(0, pos - self.window + 1)
         return pos // self.chunk * self.chunk if self.chunk else 0
+
+    def key_ranges(self, pos: int) -> tuple:
+        """(kept, first): the token at `pos` and those behind it need the keys [0, kept) and [first, ...)."""
+        first = self.first_key(pos)
+        kept = self.keep_first if self.window else 0
+        if kept and self.slopes is not None:
+            first = 0                                         # a distance bias wants the keys without a gap
+        return (0, 0) if first <= kept else (kept, first)
 
     @property
     def plain(self) -> bool:
-        return not self.softcap and self.slopes is None and not self.chunk
+        return not self.softcap and self.slopes is None and not self.chunk and not self.window and not self.sink
+
+
+def softmax_with_sink(s: torch.Tensor) -> torch.Tensor:
+    """Softmax over the last dimension with a further score 0 whose weight is dropped."""
+    return torch.softmax(torch.cat([s, torch.zeros_like(s[..., :1])], -1), -1)[..., :-1]
 
 
 def distance_slopes(heads: int, device=None) -> torch.Tensor:
@@ -55,12 +75,14 @@ def attention_reference(q, k, v, causal: bool, scale: float | None = None, kv_le
             s = s - rule.slopes.to(q.device).float()[None, :, None, None] * (i - j).float()
         if rule.chunk:
             s = s.masked_fill(i // rule.chunk != j // rule.chunk, float("-inf"))
+        if rule.window:
+            s = s.masked_fill((i - j >= rule.window) & (j >= rule.keep_first), float("-inf"))
     if causal:
         s = s.masked_fill(j > i, float("-inf"))
     if kv_lens is not None:
         pad = torch.arange(Sk, device=q.device)[None, :] >= kv_lens.to(q.device).long()[:, None]      # [B, Sk]
         s = s.masked_fill(pad[:, None, None, :], float("-inf"))
-    p = torch.softmax(s, -1)
+    p = softmax_with_sink(s) if rule is not None and rule.sink else torch.softmax(s, -1)
     if kv_lens is not None:
         p = torch.nan_to_num(p, nan=0.0)                      # rows without a visible key
     return (p @ vf).permute(0, 2, 1, 3).to(q.dtype)
@@ -157,25 +179,30 @@ def prompt_supported(q, k, v, dk: int, dv: int, rule: ScoreRule | None = None, g
 N.optional_sig("rb_attention_fwd_rule", [N.C.POINTER(N.RbAttnArgs), N.C.POINTER(N.RbAttnRule), N.c_void_p])
 
 
-def prompt_attention(q, k, v, scale: float, out, rule: ScoreRule | None = None, gate=None):
+def prompt_attention(q, k, v, scale: float, out, rule: ScoreRule | None = None, gate=None, head_gate=None):
     """Causal attention of a prompt portion in inference: q [1, L, H, dk], k [1, S, G, dk], v [1, S, G, dv] with the last L
-    keys being the portion itself, out [1, L, H, dv].  `rule`: see ScoreRule (key 0 starts a chunk); `gate`
-    [L, H * dv]: out <- out * sigmoid(gate)."""
+    keys being the portion itself, out [1, L, H, dv].  `rule`: see ScoreRule (key 0 starts a chunk; with a window the keys may
+    be those of `key_ranges`); `gate` [L, H * dv] or `head_gate` fp32 [L, H]: out <- out * sigmoid(gate)."""
     if not q.is_cuda:
         o = attention_reference(q, k, v, True, scale, rule=rule)
         if gate is not None:
             o = o.float() * torch.sigmoid(gate.float().reshape(o.shape))
+        if head_gate is not None:
+            o = o.float() * torch.sigmoid(head_gate.float())[None, :, :, None]
         out.copy_(o)
         return out
     dv = v.shape[3]
-    if rule is None and gate is None and dv == q.shape[3]:
+    if rule is None and gate is None and head_gate is None and dv == q.shape[3]:
         return attention_forward(q, k, v, True, scale, out=out, want_lse=False)[0]
     rule = rule or ScoreRule()
     a, r = N.RbAttnArgs(), N.RbAttnRule()
     _fill(a, q, k, v, out, True, scale)
     r.v_dim, r.softcap, r.slopes, r.chunk = dv, rule.softcap, N.ptr(rule.slopes), rule.chunk
+    r.window, r.keep_first, r.sink = rule.window, rule.keep_first, int(rule.sink)
     if gate is not None:
         r.gate, r.ld_gate = gate.data_ptr(), gate.stride(0)
+    if head_gate is not None:
+        r.head_gate, r.ld_gate = head_gate.data_ptr(), head_gate.stride(0)
     N.check(N.kernels().rb_attention_fwd_rule(a, r, N.stream_ptr()), "rb_attention_fwd_rule")
     return out
 

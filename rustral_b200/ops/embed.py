@@ -42,21 +42,24 @@ def embedding_forward(ids: torch.Tensor, wte: torch.Tensor, wpe=None, seq_len: i
     return y
 
 
-N.optional_sig("rb_embedding_residual", [N.c_void_p, N.c_void_p, N.c_int, N.c_void_p, N.c_void_p, N.c_ll, N.c_int, N.c_ll, N.c_void_p])
+N.optional_sig("rb_embedding_residual", [N.c_void_p, N.c_void_p, N.c_int, N.c_void_p, N.c_void_p, N.c_ll, N.c_int, N.c_ll,
+                                        N.c_float, N.c_void_p])
 
 
-def embedding_residual(ids: torch.Tensor, table: torch.Tensor):
-    """Start of a 32-bit residual stream: (x fp32 [tokens, dim], h = the same rows in the table's dtype; x itself for an
-    fp32 table)."""
+def embedding_residual(ids: torch.Tensor, table: torch.Tensor, scale: float = 1.0, want_h: bool = True):
+    """Start of a 32-bit residual stream: (x fp32 [tokens, dim] = scale * rows of the table, h = the same rows in the table's
+    dtype; x itself for an fp32 table; None without `want_h`)."""
     f32 = table.dtype == torch.float32
     if not table.is_cuda:
-        h = table[ids]
-        return (h, h) if f32 else (h.float(), h)
+        x = table[ids].float() * scale
+        return x, (None if not want_h else x if f32 else x.to(table.dtype))
     tokens, dim = ids.numel(), table.shape[1]
     x = torch.empty((tokens, dim), dtype=torch.float32, device=table.device)
-    h = x if f32 else torch.empty((tokens, dim), dtype=table.dtype, device=table.device)
+    h = None
+    if want_h:
+        h = x if f32 else torch.empty((tokens, dim), dtype=table.dtype, device=table.device)
     N.check(N.kernels().rb_embedding_residual(ids.data_ptr(), table.data_ptr(), int(f32), x.data_ptr(),
-                                              None if f32 else h.data_ptr(), tokens, dim, table.shape[0], N.stream_ptr()),
+                                              None if f32 else N.ptr(h), tokens, dim, table.shape[0], scale, N.stream_ptr()),
             "rb_embedding_residual")
     return x, h
 

@@ -19,7 +19,7 @@ P, I, F, LL = N.c_void_p, N.c_int, N.c_float, N.c_ll
 N.optional_sig("rb_moe_route", [P, I, I, I, I, P, P, P, P])
 N.optional_sig("rb_moe_route_bwd", [P, P, P, P, P, I, I, I, I, F, P, P])
 N.optional_sig("rb_moe_route_groups", [P, I, I, I, I, I, I, F, P, P, P])
-N.optional_sig("rb_swiglu_slots", [P, LL, P, LL, I, I, I, P, P])
+N.optional_sig("rb_swiglu_slots", [P, LL, P, LL, I, I, I, P, I, P])
 N.optional_sig("rb_moe_scatter", [P, P, P, I, I, I, P])
 N._LAUNCHES["rb_moe_plan"] = 2
 N.optional_sig("rb_moe_plan", [P, I, I, I, P, P, P, P, P, P, I, P])
@@ -76,18 +76,21 @@ def route_groups(logits: torch.Tensor, k: int, groups: int = 1, keep: int = 1, r
     return idx, w
 
 
-def swiglu_rows(gu: torch.Tensor, pl: MoEPlan | None = None) -> torch.Tensor:
-    """silu(gate) * up for gu = [gate | up] rows, bf16 or fp32.  With a plan only the rows that hold a token are computed;
-    padding rows of the expert buffer are left unwritten."""
+def swiglu_rows(gu: torch.Tensor, pl: MoEPlan | None = None, act: str = "silu", out=None) -> torch.Tensor:
+    """act(gate) * up for gu = [gate | up] rows (row-strided views allowed, `out` too), bf16 or fp32; act "silu" or "relu".  With
+    a plan only the rows that hold a token are computed; padding rows of the expert buffer are left unwritten."""
     rows, F2 = gu.shape
+    if act not in ("silu", "relu"):
+        raise ValueError(f"swiglu_rows: unknown activation {act!r}")
     if not gu.is_cuda:
         g, u = gu.float()[:, :F2 // 2], gu.float()[:, F2 // 2:]
-        return (g * torch.sigmoid(g) * u).to(gu.dtype)
-    h = torch.empty((rows, F2 // 2), dtype=gu.dtype, device=gu.device)
+        h = ((torch.relu(g) if act == "relu" else g * torch.sigmoid(g)) * u).to(gu.dtype)
+        return h if out is None else out.copy_(h)
+    h = out if out is not None else torch.empty((rows, F2 // 2), dtype=gu.dtype, device=gu.device)
     n = rows if pl is None else pl.slot_pos.numel()
     N.check(N.kernels().rb_swiglu_slots(gu.data_ptr(), gu.stride(0), h.data_ptr(), h.stride(0), n, F2 // 2,
                                         int(gu.dtype == torch.float32), None if pl is None else pl.slot_pos.data_ptr(),
-                                        N.stream_ptr()), "rb_swiglu_slots")
+                                        int(act == "relu"), N.stream_ptr()), "rb_swiglu_slots")
     return h
 
 

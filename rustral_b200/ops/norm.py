@@ -189,3 +189,48 @@ def residual_norm(y, gamma, beta, eps: float, rms: bool = False, *, x=None, h=No
     a.rows, a.n, a.rms, a.eps = rows, n, int(rms), eps
     N.check(N.kernels().rb_residual_norm(a, N.stream_ptr()), "rb_residual_norm")
     return h if h is not None else x
+
+
+N.optional_sig("rb_stream_update", [N.C.POINTER(N.RbStreamUpdateArgs), N.c_void_p])
+
+
+def stream_update(x, *, a=None, wa=None, b=None, wb=None, c=None, normed: float = 1.0, mult: float = 1.0, eps: float = 1e-5,
+                  dyt=None, h=None):
+    """x += mult * (normed * rms(a) * wa + normed * rms(b) * wb + c) on a 32-bit residual stream (in place; x is left as it is
+    without a, b and c), then h = tanh(alpha x) * gamma + beta with dyt = (gamma fp32 [n], beta fp32 [n], alpha fp32 [1]).  a, b
+    and c share their dtype.  Returns h, or x without `dyt`."""
+    rows, n = x.shape
+    src = [t for t in (a, b, c) if t is not None]
+    if not x.is_cuda:
+        v = torch.zeros_like(x)
+        for t, w in ((a, wa), (b, wb)):
+            if t is not None:
+                tf = t.float()
+                v += normed * tf * torch.rsqrt((tf * tf).mean(-1, keepdim=True) + eps) * w
+        if c is not None:
+            v += c.float()
+        if src:
+            x += mult * v
+        if dyt is None:
+            return x
+        g, beta, alpha = dyt
+        o = torch.tanh(alpha * x) * g + beta
+        return o if h is None else h.copy_(o)
+    if x.dtype != torch.float32 or len({t.dtype for t in src}) > 1:
+        raise TypeError("stream_update: the residual stream is fp32 and its sources share a dtype")
+    s = N.RbStreamUpdateArgs()
+    s.x, s.ldx, s.rows, s.n, s.mult, s.normed, s.eps = x.data_ptr(), x.stride(0), rows, n, mult, normed, eps
+    if a is not None:
+        s.a, s.lda, s.wa = a.data_ptr(), a.stride(0), wa.data_ptr()
+    if b is not None:
+        s.b, s.ldb, s.wb = b.data_ptr(), b.stride(0), wb.data_ptr()
+    if c is not None:
+        s.c, s.ldc = c.data_ptr(), c.stride(0)
+    s.y_f32 = int(bool(src) and src[0].dtype == torch.float32)
+    if dyt is not None:
+        g, beta, alpha = dyt
+        h = h if h is not None else torch.empty_like(x)
+        s.gamma, s.beta, s.alpha = g.data_ptr(), beta.data_ptr(), alpha.data_ptr()
+        s.h, s.ldh, s.h_f32 = h.data_ptr(), h.stride(0), int(h.dtype == torch.float32)
+    N.check(N.kernels().rb_stream_update(s, N.stream_ptr()), "rb_stream_update")
+    return x if dyt is None else h

@@ -47,17 +47,20 @@ def decode_supported(q, dk: int, dv: int, rule: ScoreRule | None = None, gate=No
 
 
 def paged_attention_decode(q, k_cache, v_cache, block_tables, context_lens, scale=None, out=None, rule: ScoreRule | None = None,
-                           gate=None):
+                           gate=None, head_gate=None):
     """q: [batch, heads * dk] (or [batch, heads, dk]); block_tables int32 [batch, max_blocks]; context_lens int32 [batch].
-    Returns [batch, heads * dv].  `rule`: see ops.ScoreRule; `gate` [batch, heads * dv]: the output times sigmoid(gate)."""
+    Returns [batch, heads * dv].  `rule`: see ops.ScoreRule; `gate` [batch, heads * dv] or `head_gate` fp32 [batch, heads]: the
+    output times sigmoid(gate)."""
     nb, bs, hk, d = k_cache.shape
     dv = v_cache.shape[3]
     B = q.shape[0]
     q2 = q.reshape(B, -1)
     heads = q2.shape[1] // d
     scale = 1.0 / math.sqrt(d) if scale is None else scale
-    if not q.is_cuda and (rule is not None or gate is not None or dv != d):
-        return paged_attention_rows(q2, k_cache, v_cache, block_tables, torch.arange(B), context_lens.long() - 1, scale, rule, gate, out)
+    plain = rule is None and gate is None and head_gate is None and dv == d
+    if not q.is_cuda and not plain:
+        return paged_attention_rows(q2, k_cache, v_cache, block_tables, torch.arange(B), context_lens.long() - 1, scale, rule, gate, out,
+                                    head_gate)
     if not q.is_cuda:
         o = torch.zeros(B, heads, d)
         kc, vc = k_cache.view(nb * bs, hk, d).float(), v_cache.view(nb * bs, hk, d).float()
@@ -78,7 +81,7 @@ def paged_attention_decode(q, k_cache, v_cache, block_tables, context_lens, scal
     lib = N.kernels()
     scratch = torch.empty(lib.rb_paged_attention_scratch_floats(B, heads, dv, block_tables.shape[1], bs), dtype=torch.float32,
                           device=q.device)
-    if rule is not None or gate is not None or dv != d:
+    if not plain:
         rule = rule or ScoreRule()
         a = N.RbPagedDecodeArgs()
         a.q, a.ld_q, a.out, a.ld_o = q2.data_ptr(), q2.stride(0), out.data_ptr(), out.stride(0)
@@ -86,6 +89,9 @@ def paged_attention_decode(q, k_cache, v_cache, block_tables, context_lens, scal
         a.block_tables, a.max_blocks, a.context_lens = block_tables.data_ptr(), block_tables.shape[1], context_lens.data_ptr()
         if gate is not None:
             a.gate, a.ld_g = gate.data_ptr(), gate.stride(0)
+        if head_gate is not None:
+            a.head_gate, a.ld_g = head_gate.data_ptr(), head_gate.stride(0)
+        a.window, a.keep_first, a.sink = rule.window, rule.keep_first, int(rule.sink)
         a.scratch, a.batch, a.heads, a.kv_heads, a.dk, a.dv = scratch.data_ptr(), B, heads, hk, d, dv
         a.scale, a.softcap, a.slopes, a.chunk = scale, rule.softcap, N.ptr(rule.slopes), rule.chunk
         N.check(lib.rb_paged_attention_decode_rule(a, N.stream_ptr()), "rb_paged_attention_decode_rule")
@@ -101,10 +107,11 @@ N.optional_sig("rb_paged_attention_rows", [N.C.POINTER(N.RbPagedRowsArgs), N.c_v
 
 
 def paged_attention_rows(q, k_cache, v_cache, block_tables, row_seq, row_pos, scale: float, rule: ScoreRule | None = None,
-                         gate=None, out=None):
+                         gate=None, out=None, head_gate=None):
     """Attention over the pages for any rows of a batch.  q: [rows, heads * dk] (row-strided views allowed); row r is the
     token at position row_pos[r] (int64) of the sequence with pages block_tables[row_seq[r]] (int32); its own key is
-    already in the cache.  Takes bf16 and fp32 and any head sizes.  `gate` [rows, heads * dv]: output times sigmoid(gate)."""
+    already in the cache.  Takes bf16 and fp32 and any head sizes.  `gate` [rows, heads * dv] or `head_gate` fp32 [rows, heads]:
+    output times sigmoid(gate)."""
     nb, bs, hk, dk = k_cache.shape
     dv = v_cache.shape[3]
     rows, heads = q.shape[0], q.shape[1] // dk
@@ -114,11 +121,13 @@ def paged_attention_rows(q, k_cache, v_cache, block_tables, row_seq, row_pos, sc
         kc, vc = k_cache.view(nb * bs, hk, dk), v_cache.view(nb * bs, hk, dv)
         for r in range(rows):
             n, table = int(row_pos[r]) + 1, block_tables[int(row_seq[r])].long()
-            lo = rule.first_key(n - 1)
-            toks = torch.arange(lo, n)
+            kept, lo = rule.key_ranges(n - 1)
+            toks = torch.cat([torch.arange(kept), torch.arange(lo, n)])
             slots = table[toks // bs] * bs + toks % bs
             o = attention_reference(q[r].view(1, 1, heads, dk), kc[slots][None], vc[slots][None], True, scale, rule=rule)
             o = o.reshape(-1).float()
+            if head_gate is not None:
+                o = (o.view(heads, dv) * torch.sigmoid(head_gate[r].float())[:, None]).reshape(-1)
             out[r] = o * torch.sigmoid(gate[r].float()) if gate is not None else o
         return out
     a = N.RbPagedRowsArgs()
@@ -128,6 +137,9 @@ def paged_attention_rows(q, k_cache, v_cache, block_tables, row_seq, row_pos, sc
     a.row_seq, a.row_pos = row_seq.data_ptr(), row_pos.data_ptr()
     if gate is not None:
         a.gate, a.ld_g = gate.data_ptr(), gate.stride(0)
+    if head_gate is not None:
+        a.head_gate, a.ld_g = head_gate.data_ptr(), head_gate.stride(0)
+    a.window, a.keep_first, a.sink = rule.window, rule.keep_first, int(rule.sink)
     a.f32, a.rows, a.heads, a.kv_heads, a.dk, a.dv = int(q.dtype == torch.float32), rows, heads, hk, dk, dv
     a.scale, a.softcap, a.slopes, a.chunk = scale, rule.softcap, N.ptr(rule.slopes), rule.chunk
     N.check(N.kernels().rb_paged_attention_rows(a, N.stream_ptr()), "rb_paged_attention_rows")

@@ -1,0 +1,195 @@
+"""Mixers that carry state from token to token, over batches of unequal segments: short causal convolution, Mamba-2 state-space
+recurrence, gated delta rule, and the gated norm behind them.
+
+Every op takes a `Segments` table (which rows belong to which sequence, where its state lives, whether it has just begun),
+reads and updates the state tensors in place, and treats a sequence's state as zero at position 0.
+"""
+from __future__ import annotations
+
+import torch
+
+from .. import _native as N
+
+CONV_TILE = 16
+MAX_STATE_ROWS = 256
+UNIT_EPS = 1e-6
+
+N.optional_sig("rb_short_conv", [N.C.POINTER(N.RbShortConvArgs), N.c_void_p])
+N.optional_sig("rb_state_space_scan", [N.C.POINTER(N.RbStateSpaceArgs), N.c_void_p])
+N.optional_sig("rb_delta_rule_scan", [N.C.POINTER(N.RbDeltaRuleArgs), N.c_void_p])
+N.optional_sig("rb_gated_norm", [N.C.POINTER(N.RbGatedNormArgs), N.c_void_p])
+
+
+class Segments:
+    """Rows of a batch as segments, each the next tokens of one sequence.
+
+    `table`: int32 [n, 4] on the device: first row, number of rows, state slot, position of the first row.  `rows`: the same as
+    a list of tuples on the host, or None where only the device knows them (a captured decode step): then every segment is one
+    row."""
+
+    def __init__(self, table: torch.Tensor, rows: list | None):
+        self.table, self.rows = table, rows
+        self.n = table.shape[0]
+        self._tiles: dict = {}
+
+    @classmethod
+    def of(cls, rows: list, device) -> "Segments":
+        return cls(torch.tensor(rows, dtype=torch.int32).view(-1, 4).to(device), rows)
+
+    @property
+    def single(self) -> bool:
+        """Every segment is one row (a decode step)."""
+        return self.rows is None or all(r[1] == 1 for r in self.rows)
+
+    def tiles(self, size: int) -> torch.Tensor:
+        """int32 [tiles, 2]: (segment, first row inside it) of pieces of at most `size` rows."""
+        if size not in self._tiles:
+            if self.single:
+                if 1 not in self._tiles:
+                    t = torch.zeros((self.n, 2), dtype=torch.int32, device=self.table.device)
+                    t[:, 0] = torch.arange(self.n, dtype=torch.int32, device=self.table.device)
+                    self._tiles[1] = t
+                self._tiles[size] = self._tiles[1]
+            else:
+                pairs = [(i, o) for i, r in enumerate(self.rows) for o in range(0, r[1], size)]
+                self._tiles[size] = torch.tensor(pairs, dtype=torch.int32).to(self.table.device)
+        return self._tiles[size]
+
+    def host(self) -> list:
+        return self.rows if self.rows is not None else [tuple(r) for r in self.table.tolist()]
+
+
+def up4(n: int) -> int:
+    return (n + 3) // 4 * 4
+
+
+def _check(t, dtype, what):
+    if t.dtype != dtype or t.stride(-1) != 1:
+        raise TypeError(f"{what}: {dtype} with a contiguous last dimension is required")
+
+
+def short_conv(x, w, bias, state, seg: Segments, silu: bool = True, out=None):
+    """out[t] = act(bias + sum_i w[:, i] * x[t - (taps - 1) + i]) per sequence.  x [rows, channels] (row-strided views allowed),
+    w fp32 [channels, taps], bias fp32 [channels] or None, state [slots, taps - 1, channels] in the dtype of x."""
+    rows, C = x.shape
+    taps = w.shape[1]
+    out = out if out is not None else torch.empty((rows, C), dtype=x.dtype, device=x.device)
+    if not x.is_cuda:
+        for first, n, slot, start in seg.host():
+            past = state[slot].float() if start > 0 else torch.zeros(taps - 1, C)
+            full = torch.cat([past, x[first:first + n].float()])
+            y = sum(w[:, i].float() * full[i:i + n] for i in range(taps))
+            if bias is not None:
+                y = y + bias.float()
+            out[first:first + n] = (y * torch.sigmoid(y) if silu else y).to(out.dtype)
+            if taps > 1:
+                state[slot] = full[n:].to(state.dtype)
+        return out
+    _check(w, torch.float32, "short_conv")
+    a = N.RbShortConvArgs()
+    tiles = seg.tiles(CONV_TILE)
+    a.x, a.ld_x, a.out, a.ld_o = x.data_ptr(), x.stride(0), out.data_ptr(), out.stride(0)
+    a.state, a.num_slots = state.data_ptr(), state.shape[0]
+    a.w, a.bias, a.segments, a.tiles, a.num_tiles = w.data_ptr(), N.ptr(bias), seg.table.data_ptr(), tiles.data_ptr(), tiles.shape[0]
+    a.channels, a.taps, a.f32, a.silu = C, taps, int(x.dtype == torch.float32), int(silu)
+    N.check(N.kernels().rb_short_conv(a, N.stream_ptr()), "rb_short_conv")
+    return out
+
+
+def _softplus(z):
+    return torch.clamp(z, min=0) + torch.log1p(torch.exp(-z.abs()))
+
+
+def state_space(xbc, dt_raw, *, dt_bias, a_log, D, state, heads: int, groups: int, vdim: int, n: int, seg: Segments, out=None):
+    """Mamba-2 recurrence.  xbc [rows, heads * vdim + 2 * groups * n] = x | B | C behind the convolution; dt_raw fp32
+    [rows, heads]; dt_bias, a_log, D fp32 [heads]; state fp32 [slots, heads, n, up4(vdim)].  Returns y [rows, heads * vdim]."""
+    rows = xbc.shape[0]
+    inner = heads * vdim
+    out = out if out is not None else torch.empty((rows, inner), dtype=xbc.dtype, device=xbc.device)
+    if not xbc.is_cuda:
+        per = heads // groups
+        x = xbc[:, :inner].float().view(rows, heads, vdim)
+        B = xbc[:, inner:inner + groups * n].float().view(rows, groups, n).repeat_interleave(per, 1)
+        C = xbc[:, inner + groups * n:inner + 2 * groups * n].float().view(rows, groups, n).repeat_interleave(per, 1)
+        dt = _softplus(dt_raw.float() + dt_bias)
+        decay = torch.exp(-torch.exp(a_log) * dt)
+        for first, m, slot, start in seg.host():
+            S = state[slot, :, :, :vdim].clone() if start > 0 else torch.zeros(heads, n, vdim)
+            for t in range(first, first + m):
+                S = decay[t, :, None, None] * S + (dt[t, :, None] * B[t])[:, :, None] * x[t, :, None, :]
+                out[t] = (torch.einsum("hnp,hn->hp", S, C[t]) + D[:, None] * x[t]).reshape(-1).to(out.dtype)
+            state[slot, :, :, :vdim] = S
+        return out
+    if n > MAX_STATE_ROWS:
+        raise ValueError(f"state_space: at most {MAX_STATE_ROWS} state rows per head")
+    _check(dt_raw, torch.float32, "state_space")
+    a = N.RbStateSpaceArgs()
+    a.xbc, a.ld_xbc, a.dt_raw, a.ld_dt, a.y, a.ld_y = xbc.data_ptr(), xbc.stride(0), dt_raw.data_ptr(), dt_raw.stride(0), out.data_ptr(), out.stride(0)
+    a.dt_bias, a.a_log, a.D, a.state, a.num_slots = dt_bias.data_ptr(), a_log.data_ptr(), D.data_ptr(), state.data_ptr(), state.shape[0]
+    a.segments, a.num_segments = seg.table.data_ptr(), seg.n
+    a.heads, a.groups, a.p, a.n, a.f32 = heads, groups, vdim, n, int(xbc.dtype == torch.float32)
+    N.check(N.kernels().rb_state_space_scan(a, N.stream_ptr()), "rb_state_space_scan")
+    return out
+
+
+def delta_rule(qkv, a_raw, b_raw, *, dt_bias, a_log, state, heads: int, kv_heads: int, dk: int, dv: int, seg: Segments, out=None):
+    """Gated delta rule.  qkv [rows, 2 * kv_heads * dk + heads * dv] = q | k | v behind the convolution; a_raw, b_raw fp32
+    [rows, heads] (same pitch); dt_bias, a_log fp32 [heads]; state fp32 [slots, heads, dk, up4(dv)].  Returns o
+    [rows, heads * dv] (row-strided `out` allowed)."""
+    rows = qkv.shape[0]
+    out = out if out is not None else torch.empty((rows, heads * dv), dtype=qkv.dtype, device=qkv.device)
+    if not qkv.is_cuda:
+        per, nk = heads // kv_heads, kv_heads * dk
+        unit = lambda t: t / torch.sqrt((t * t).sum(-1, keepdim=True) + UNIT_EPS)
+        q = unit(qkv[:, :nk].float().view(rows, kv_heads, dk)).repeat_interleave(per, 1) * dk ** -0.5
+        k = unit(qkv[:, nk:2 * nk].float().view(rows, kv_heads, dk)).repeat_interleave(per, 1)
+        v = qkv[:, 2 * nk:2 * nk + heads * dv].float().view(rows, heads, dv)
+        beta = torch.sigmoid(b_raw.float())
+        decay = torch.exp(-torch.exp(a_log) * _softplus(a_raw.float() + dt_bias))
+        for first, m, slot, start in seg.host():
+            S = state[slot, :, :, :dv].clone() if start > 0 else torch.zeros(heads, dk, dv)
+            for t in range(first, first + m):
+                S = decay[t, :, None, None] * S
+                u = beta[t, :, None] * (v[t] - torch.einsum("hkv,hk->hv", S, k[t]))
+                S = S + k[t, :, :, None] * u[:, None, :]
+                out[t] = torch.einsum("hkv,hk->hv", S, q[t]).reshape(-1).to(out.dtype)
+            state[slot, :, :, :dv] = S
+        return out
+    if dk > MAX_STATE_ROWS:
+        raise ValueError(f"delta_rule: key size at most {MAX_STATE_ROWS}")
+    _check(a_raw, torch.float32, "delta_rule")
+    _check(b_raw, torch.float32, "delta_rule")
+    if a_raw.stride(0) != b_raw.stride(0):
+        raise ValueError("delta_rule: a_raw and b_raw must have the same pitch")
+    a = N.RbDeltaRuleArgs()
+    a.qkv, a.ld_qkv, a.o, a.ld_o = qkv.data_ptr(), qkv.stride(0), out.data_ptr(), out.stride(0)
+    a.a_raw, a.b_raw, a.ld_ab = a_raw.data_ptr(), b_raw.data_ptr(), a_raw.stride(0)
+    a.dt_bias, a.a_log, a.state, a.num_slots = dt_bias.data_ptr(), a_log.data_ptr(), state.data_ptr(), state.shape[0]
+    a.segments, a.num_segments = seg.table.data_ptr(), seg.n
+    a.heads, a.kv_heads, a.dk, a.dv, a.f32 = heads, kv_heads, dk, dv, int(qkv.dtype == torch.float32)
+    N.check(N.kernels().rb_delta_rule_scan(a, N.stream_ptr()), "rb_delta_rule_scan")
+    return out
+
+
+def gated_norm(y, z, weight, parts: int, eps: float, gate_first: bool, out=None):
+    """RMS norm of every one of `parts` equal parts of y's rows, gated with silu(z) before (gate_first) or behind the norm.
+    weight fp32: one per column, or one part's, shared by all parts."""
+    rows, n = y.shape
+    m = n // parts
+    out = out if out is not None else torch.empty((rows, n), dtype=y.dtype, device=y.device)
+    if not y.is_cuda:
+        zf = z.float().view(rows, parts, m)
+        g = zf * torch.sigmoid(zf)
+        u = y.float().view(rows, parts, m)
+        if gate_first:
+            u = u * g
+        u = u * torch.rsqrt((u * u).mean(-1, keepdim=True) + eps) * weight.view(-1, m)
+        if not gate_first:
+            u = u * g
+        return out.copy_(u.reshape(rows, n))
+    a = N.RbGatedNormArgs()
+    a.y, a.ld_y, a.z, a.ld_z, a.out, a.ld_o = y.data_ptr(), y.stride(0), z.data_ptr(), z.stride(0), out.data_ptr(), out.stride(0)
+    a.weight, a.weight_n = weight.data_ptr(), weight.numel()
+    a.rows, a.parts, a.part_n, a.f32, a.gate_first, a.eps = rows, parts, m, int(y.dtype == torch.float32), int(gate_first), eps
+    N.check(N.kernels().rb_gated_norm(a, N.stream_ptr()), "rb_gated_norm")
+    return out

@@ -13,14 +13,17 @@ import math
 import torch
 
 from .. import ops
+from ..models.layered import ParallelSpec, up8
 from ..ops import moe as moe_ops
 from ..ops import norm as norm_ops
 from ..ops import paged as paged_ops
+from ..ops import recurrent as rc_ops
 from ..ops import rotary as rope_ops
 from ..ops.attention import ScoreRule, distance_slopes
 from ..ops.heads import head_prep_
 from ..ops.matmul import gemm
 from .kv_cache import CacheLayer
+from .weights import packed_columns
 
 
 class GPTBody:
@@ -163,3 +166,111 @@ class LayeredBody:
         h = norm_ops.residual_norm(x, P.w("final.norm"), P.w("final.norm.b"), cfg.norm_eps, h=torch.empty_like(x, dtype=self.r.dtype))
         logits = gemm(h, P.w("head"), out_dtype=torch.float32)
         return ops.scale_softcap_(logits, cfg.logit_scale, cfg.logit_softcap)
+
+
+class ParallelBody:
+    """Layered decoders with one norm in front of a layer and mixer and feed-forward side by side behind it (Vafodra).
+
+    Per layer: one packed projection of everything that reads the norm's output, and a narrow one whose results stay fp32 (step
+    sizes, decays, per-head gates); the mixers; act(gate) * up; output projections (mixer and feed-forward as one product where
+    their sum needs no norm); then norms of the mixer's outputs, residual add and the next layer's norm in one kernel."""
+
+    def __init__(self, runner):
+        self.r, self.cfg = runner, runner.cfg
+        if runner.tp is not None:
+            raise ValueError("tensor-parallel serving covers the llama family")
+        self.columns = [packed_columns(s) for s in self.cfg.layers]
+        self.prefix = [f"l{self.cfg.owner(i)}." for i in range(self.cfg.n_layer)]
+        slopes = {}
+        self.rules = []
+        for s in self.cfg.layers:
+            a = s.mixer.left if isinstance(s.mixer, ParallelSpec) else None
+            if a is not None and a.distance_bias and a.heads not in slopes:
+                slopes[a.heads] = distance_slopes(a.heads, runner.device)
+            self.rules.append(None if a is None else ScoreRule(a.softcap, slopes.get(a.heads), a.chunk, a.window, a.keep_first, a.sink))
+
+    def cache_layers(self) -> list:
+        out = []
+        for s in self.cfg.layers:
+            m = s.mixer
+            if isinstance(m, ParallelSpec):
+                a, r = m.left, m.right
+                out.append(CacheLayer(a.kv_heads, a.dim, a.vdim, (("conv", (r.conv - 1, r.channels), None),
+                                                                  ("state", (r.heads, r.state, rc_ops.up4(r.vdim)), torch.float32))))
+            else:
+                out.append(CacheLayer(state=(("conv", (m.conv - 1, m.channels), None),
+                                             ("state", (m.heads, m.dim, rc_ops.up4(m.vdim)), torch.float32))))
+        return out
+
+    def _norm(self, name):
+        P = self.r.params
+        return P.w(name), P.w(name + ".b"), P.w(name + ".alpha")
+
+    def _update(self, st, l, **sources):
+        """x += residual_mult * (...), then the norm in front of layer l + 1 (the head takes its norm over the wanted rows)."""
+        dyt = h = None
+        if l + 1 < self.cfg.n_layer:
+            dyt = self._norm(self.prefix[l + 1] + "norm1")
+            h = torch.empty(st.x.shape, dtype=self.r.dtype, device=st.x.device)
+        if sources or dyt is not None:
+            norm_ops.stream_update(st.x, mult=self.cfg.residual_mult, eps=self.cfg.norm_eps, dyt=dyt, h=h, **sources)
+        st.h = h
+        return st
+
+    def embed(self, sb):
+        x, _ = ops.embedding_residual(sb.ids, self.r.params.w("embed"), self.cfg.embed_scale, want_h=False)
+        return self._update(Stream(x, None), -1)
+
+    def layer(self, l, st, sb):
+        P, p, s = self.r.params, self.prefix[l], self.cfg.layers[l]
+        cols, gates = self.columns[l]
+        z = gemm(st.h, P.w(p + "in"))
+        small = gemm(st.h, P.w(p + "gates"), out_dtype=torch.float32)
+        run = self._parallel if isinstance(s.mixer, ParallelSpec) else self._delta
+        return run(l, st, sb, s, p, lambda c: z[:, cols[c][0]:cols[c][0] + cols[c][1]], lambda c: small[:, gates[c][0]:gates[c][0] + gates[c][1]],
+                   z)
+
+    def _feed_forward(self, l, s, z, out=None):
+        lo = self.columns[l][0]["gate"][0]
+        return moe_ops.swiglu_rows(z[:, lo:lo + 2 * up8(s.mlp.ff)], act=s.mlp.act, out=out)
+
+    def _parallel(self, l, st, sb, s, p, col, gate, z):
+        r, P, cfg = self.r, self.r.params, self.cfg
+        a, m = s.mixer.left, s.mixer.right
+        k2, v2 = col("k"), col("v")
+        head_prep_(z, a.heads, a.kv_heads, a.dim, a.vdim, k_cache=r.cache.k[l], v_cache=r.cache.v[l], slots=sb.slots)
+        o = r.attend(l, col("q"), k2, v2, sb, a.scale, self.rules[l], head_gate=gate("g"))
+        state = r.cache.state[l]
+        xbc = rc_ops.short_conv(col("conv"), P.w(p + "conv"), P.w(p + "conv.b"), state["conv"], sb.segments)
+        y = rc_ops.state_space(xbc, gate("dt"), dt_bias=P.w(p + "dt_bias"), a_log=P.w(p + "A_log"), D=P.w(p + "D"), state=state["state"],
+                               heads=m.heads, groups=m.groups, vdim=m.vdim, n=m.state, seg=sb.segments)
+        y = rc_ops.gated_norm(y, col("z"), P.w(p + "norm"), m.norm_groups, cfg.norm_eps, gate_first=True, out=y)
+        out = dict(a=gemm(o, P.w(p + "left.o"), out_dtype=torch.float32), wa=P.w(p + "left.out"),
+                   b=gemm(y, P.w(p + "right.o"), out_dtype=torch.float32), wb=P.w(p + "right.out"), normed=0.5)
+        if s.mlp is not None:
+            out["c"] = gemm(self._feed_forward(l, s, z), P.w(p + "down"), out_dtype=torch.float32)
+        return self._update(st, l, **out)
+
+    def _delta(self, l, st, sb, s, p, col, gate, z):
+        P, m = self.r.params, s.mixer
+        state = self.r.cache.state[l]
+        n, w_out = m.heads * m.vdim, P.w(p + "out")
+        qkv = rc_ops.short_conv(z[:, :m.channels], P.w(p + "conv"), None, state["conv"], sb.segments)
+        joined = torch.empty((sb.rows, w_out.shape[1]), dtype=z.dtype, device=z.device)      # mixer output | feed-forward
+        if up8(n) != n:
+            joined[:, n:up8(n)] = 0
+        o = rc_ops.delta_rule(qkv, gate("a"), gate("b"), dt_bias=P.w(p + "dt_bias"), a_log=P.w(p + "A_log"), state=state["state"],
+                              heads=m.heads, kv_heads=m.kv_heads, dk=m.dim, dv=m.vdim, seg=sb.segments, out=joined[:, :n])
+        rc_ops.gated_norm(o, col("z"), P.w(p + "norm"), m.heads, self.cfg.norm_eps, gate_first=False, out=o)
+        if s.mlp is not None:
+            self._feed_forward(l, s, z, out=joined[:, up8(n):])
+        return self._update(st, l, c=gemm(joined, w_out, out_dtype=torch.float32))
+
+    def head(self, st, rows):
+        P = self.r.params
+        x = st.x if rows is None else ops.gather_rows(st.x, rows)
+        h = norm_ops.stream_update(x, dyt=self._norm("final.norm"), h=torch.empty(x.shape, dtype=self.r.dtype, device=x.device))
+        logits = gemm(h, P.w("head"), out_dtype=torch.float32)
+        if self.cfg.logit_scale != 1.0 or self.cfg.logit_softcap:
+            ops.scale_softcap_(logits, self.cfg.logit_scale, self.cfg.logit_softcap)
+        return logits

@@ -274,7 +274,7 @@ def build_state(a) -> ServerState:
         from .model_runner import load_runner
         dtype = getattr(torch, a.dtype) if a.dtype else None
         runner = load_runner(a.model, device=a.device, dtype=dtype, num_blocks=a.blocks, block_size=a.page, weights=a.weights,
-                             seed=a.seed, **({"n_layer": a.layers} if a.layers else {}))   # weights are loaded strictly
+                             seed=a.seed, num_slots=a.max_batch, **({"n_layer": a.layers} if a.layers else {}))   # weights are loaded strictly
         cfg = runner.cfg
         engine = ServingEngine(runner, max_batch_size=a.max_batch, eos_id=a.eos_id)
         engine.generate([1, 2, 3], 2)                       # warm-up: compiles nothing, but touches every kernel once

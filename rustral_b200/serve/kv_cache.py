@@ -168,18 +168,25 @@ class SlidingWindowCache(KVCache):
 
 @dataclass(frozen=True)
 class CacheLayer:
-    """What one layer stores per token: `kv_heads` keys of size `k_dim` and values of size `v_dim`."""
-    kv_heads: int
-    k_dim: int
-    v_dim: int
+    """What one layer stores: per token `kv_heads` keys of size `k_dim` and values of size `v_dim` (kv_heads 0: none), and
+    per sequence the tensors of `state`, each (name, shape, dtype or None for the cache's)."""
+    kv_heads: int = 0
+    k_dim: int = 0
+    v_dim: int = 0
+    state: tuple = ()
 
 
 class PagedCache:
     """Paged KV storage for all layers plus per-sequence block tables.  All layers share the tables; with `layers` every
-    layer has its own head count and key / value sizes, otherwise all are [num_kv_heads, head_dim]."""
+    layer has its own head count and key / value sizes, otherwise all are [num_kv_heads, head_dim].
+
+    Layers with recurrent state add one tensor [num_slots, ...] per state name (`state[layer][name]`); a sequence holds the
+    same slot in all of them from its first `allocate` to `free`.  A slot is not cleared when it changes hands: the layers
+    take a sequence's state as zero at position 0, whatever the slot holds."""
 
     def __init__(self, num_blocks: int, block_size: int = 16, num_layers: int = 1, num_kv_heads: int = 1, head_dim: int = 64,
-                 dtype=torch.bfloat16, device="cpu", allocate_storage: bool = True, layers: list | None = None):
+                 dtype=torch.bfloat16, device="cpu", allocate_storage: bool = True, layers: list | None = None,
+                 num_slots: int = 64):
         if layers is not None:
             num_layers = len(layers)
         self.block_size, self.num_blocks = block_size, num_blocks
@@ -189,9 +196,17 @@ class PagedCache:
         if not self._h:
             raise InvalidArgument("PagedCache: num_blocks and block_size must be positive")
         self.k = self.v = None
+        self.state = [{} for _ in range(num_layers)]
+        self.num_slots = num_slots if layers is not None and any(c.state for c in layers) else 0
+        if self.num_slots and self._lib.rb_ba_set_state_slots(self._h, num_slots) != 0:
+            raise InvalidArgument("PagedCache: num_slots must be positive")
         if allocate_storage and layers is not None:
-            self.k = [torch.zeros((num_blocks, block_size, c.kv_heads, c.k_dim), dtype=dtype, device=device) for c in layers]
-            self.v = [torch.zeros((num_blocks, block_size, c.kv_heads, c.v_dim), dtype=dtype, device=device) for c in layers]
+            def pages(c, d):
+                return torch.zeros((num_blocks, block_size, c.kv_heads, d), dtype=dtype, device=device) if c.kv_heads else None
+            self.k = [pages(c, c.k_dim) for c in layers]
+            self.v = [pages(c, c.v_dim) for c in layers]
+            self.state = [{n: torch.zeros((num_slots, *shape), dtype=dt or dtype, device=device) for n, shape, dt in c.state}
+                          for c in layers]
         elif allocate_storage:
             shape = (num_layers, num_blocks, block_size, num_kv_heads, head_dim)
             self.k = torch.zeros(shape, dtype=dtype, device=device)
@@ -230,11 +245,22 @@ class PagedCache:
     def slot(self, seq_id: int, token_index: int) -> int:
         return int(self._lib.rb_ba_slot(self._h, seq_id, token_index))
 
+    def state_slot(self, seq_id: int) -> int:
+        """The sequence's state slot (-1: the model has no recurrent state, or the sequence holds nothing)."""
+        return int(self._lib.rb_ba_state_slot(self._h, seq_id))
+
+    @property
+    def free_slots(self) -> int:
+        return self._lib.rb_ba_num_free_slots(self._h)
+
     def num_sequences(self) -> int:
         return self._lib.rb_ba_num_sequences(self._h)
 
     def memory_bytes(self) -> int:
-        return 0 if self.k is None else sum(t.numel() * t.element_size() for c in (self.k, self.v) for t in c)
+        if self.k is None:
+            return 0
+        held = [t for c in (self.k, self.v) for t in c if t is not None] + [t for d in self.state for t in d.values()]
+        return sum(t.numel() * t.element_size() for t in held)
 
 
 class BatchedCache:

@@ -3,7 +3,7 @@ decoded tokens, and batched single-token decode, all against a paged KV cache.  
 (positions, cache slots, block tables), runs the model's layer body (serve.decoder_body, chosen by the configuration's
 architecture) over them and replays decode steps from CUDA graphs.  Every matmul is the tcgen05 GEMM, prompt attention is
 the flash kernel, decode attention the paged kernel; K and V of new tokens go straight from the packed projection into
-their cache slots.
+their cache slots.  Layers with recurrent state find each sequence's rows and state slot in the step's segment table.
 
 This is the model forward the reference's ServingEngine lacks (it fabricates token 1, crates/nn/src/continuous_batching.rs:516-526)
 and the cached decode its TransformerDecoder::generate_token does not have (full re-forward per token, crates/nn/src/transformer.rs:837-862).
@@ -16,30 +16,33 @@ from .. import ops
 from ..models.registry import architecture, build_weights
 from ..ops import attention as attn_ops
 from ..ops import paged as paged_ops
+from ..ops.recurrent import Segments
 from ..runtime.fused_gpt import FlatParams
 from . import decoder_body
 from .kv_cache import PagedCache
 
 
 class StepBatch:
-    """The rows of one model pass: prompt portions first (`spans`), then one row per decoded sequence (from row `rd`)."""
+    """The rows of one model pass: prompt portions first (`spans`), then one row per decoded sequence (from row `rd`).
+    `segments`: the same sequences for layers with recurrent state (None: the model has none)."""
 
-    def __init__(self, ids, pos, slots, spans, rd, tables, bt, ctx, block_size):
+    def __init__(self, ids, pos, slots, spans, rd, tables, bt, ctx, block_size, segments=None):
         self.ids, self.pos, self.slots = ids, pos, slots          # int64 device tensors, one entry per row
         self.spans = spans                                        # (first row, end row, first position) per portion
         self.rd, self.rows = rd, ids.shape[0]
         self.tables = tables                                      # block table (list) of every portion's sequence
         self.bt, self.ctx = bt, ctx                               # decode rows: block tables, context lengths (int32)
         self.block_size = block_size
+        self.segments = segments
         self._keys, self._row_tables = {}, None
 
-    def key_slots(self, i: int, first: int) -> torch.Tensor:
-        """Cache slots of positions `first` .. end of portion i (earlier portions and this one)."""
-        key = (i, first)
+    def key_slots(self, i: int, first: int, kept: int = 0) -> torch.Tensor:
+        """Cache slots of positions 0 .. `kept` and `first` .. end of portion i (earlier portions and this one)."""
+        key = (i, first, kept)
         if key not in self._keys:
             r0, r1, start = self.spans[i]
             t, bs = self.tables[i], self.block_size
-            self._keys[key] = torch.tensor([t[p // bs] * bs + p % bs for p in range(first, start + r1 - r0)],
+            self._keys[key] = torch.tensor([t[p // bs] * bs + p % bs for r in (range(kept), range(first, start + r1 - r0)) for p in r],
                                            dtype=torch.int64, device=self.ids.device)
         return self._keys[key]
 
@@ -66,10 +69,11 @@ class ModelRunner:
     attention-output, down-projection and LM-head results are exchanged with one-shot peer-memory collectives.  All
     ranks run the same calls in the same order and obtain bit-identical logits.
 
-    `dtype` (bf16 or fp32, where the architecture runs in both) applies when `params` is not given."""
+    `dtype` (bf16 or fp32, where the architecture runs in both) applies when `params` is not given.  `num_slots`: sequences
+    that can hold recurrent state at a time (models without such layers have no limit of that kind)."""
 
     def __init__(self, cfg, params=None, device=None, num_blocks: int = 1024, block_size: int = 16, seed: int = 0, tp=None,
-                 dtype=None):
+                 dtype=None, num_slots: int = 64):
         if device is None:
             device = "cuda" if torch.cuda.is_available() else "cpu"
         self.cfg = cfg
@@ -95,17 +99,19 @@ class ModelRunner:
         if layers is None:
             self.cache = PagedCache(num_blocks, block_size, cfg.n_layer, self.n_kv_head, cfg.head_dim, self.dtype, self.device)
         else:
-            self.cache = PagedCache(num_blocks, block_size, dtype=self.dtype, device=self.device, layers=layers)
+            self.cache = PagedCache(num_blocks, block_size, dtype=self.dtype, device=self.device, layers=layers, num_slots=num_slots)
+        self.recurrent = self.cache.num_slots > 0
         self.block_size = block_size
         self.use_graphs = True          # CUDA-graph replay of decode steps
         self._graphs: dict = {}
 
     # ---- attention over the rows of a step -------------------------------------------------------------------------
-    def attend(self, l: int, q, k2, v2, sb: StepBatch, scale: float, rule=None, gate=None) -> torch.Tensor:
+    def attend(self, l: int, q, k2, v2, sb: StepBatch, scale: float, rule=None, gate=None, head_gate=None) -> torch.Tensor:
         """Attention of layer `l` for every row of `sb`; the rows' keys and values (`k2`, `v2`) are already in the cache.
         Prompt portions go through the flash kernel (keys: the cached positions the portion can still see, gathered from the
         pages, plus the portion itself), decoded rows through the paged kernel; operands that those do not take (fp32,
-        unusual head sizes) go through the paged row kernel.  `rule`: ops.ScoreRule; `gate`: output times sigmoid(gate)."""
+        unusual head sizes) go through the paged row kernel.  `rule`: ops.ScoreRule; `gate` (one number per value
+        column) or `head_gate` (fp32, one per head): output times sigmoid(gate)."""
         kc, vc = self.cache.k[l], self.cache.v[l]
         nb, bs, G, dk = kc.shape
         dv = vc.shape[3]
@@ -115,22 +121,24 @@ class ModelRunner:
         paged = paged_ops.decode_supported(q, dk, dv, rule, gate)
         if (sb.spans and not flash) or (sb.rd < T and not paged):
             bt, seq = sb.row_tables()
-            return paged_ops.paged_attention_rows(q, kc, vc, bt, seq, sb.pos, scale, rule, gate)
+            return paged_ops.paged_attention_rows(q, kc, vc, bt, seq, sb.pos, scale, rule, gate, head_gate=head_gate)
         a = torch.empty((T, H * dv), dtype=q.dtype, device=self.device)
         for i, (r0, r1, start) in enumerate(sb.spans):
             L = r1 - r0
-            first = rule.first_key(start) if rule is not None else 0
-            if first == start:
+            kept, first = rule.key_ranges(start) if rule is not None else (0, 0)
+            if first == start and kept == 0:
                 kk, vv = k2[r0:r1].view(1, L, G, dk), v2[r0:r1].view(1, L, G, dv)
             else:
-                cs = sb.key_slots(i, first)
+                cs = sb.key_slots(i, first, kept)
                 kk = ops.gather_rows(kc.view(nb * bs, G * dk), cs).view(1, -1, G, dk)
                 vv = ops.gather_rows(vc.view(nb * bs, G * dv), cs).view(1, -1, G, dv)
             attn_ops.prompt_attention(q[r0:r1].view(1, L, H, dk), kk, vv, scale, out=a[r0:r1].view(1, L, H, dv), rule=rule,
-                                      gate=None if gate is None else gate[r0:r1])
+                                      gate=None if gate is None else gate[r0:r1],
+                                      head_gate=None if head_gate is None else head_gate[r0:r1])
         if sb.rd < T:
             paged_ops.paged_attention_decode(q[sb.rd:], kc, vc, sb.bt, sb.ctx, scale, out=a[sb.rd:], rule=rule,
-                                             gate=None if gate is None else gate[sb.rd:])
+                                             gate=None if gate is None else gate[sb.rd:],
+                                             head_gate=None if head_gate is None else head_gate[sb.rd:])
         return a
 
     # ---- one model pass ----------------------------------------------------------------------------------------------
@@ -184,7 +192,12 @@ class ModelRunner:
             width = max(len(self.cache.block_table(s_)) for s_ in dec_ids)
             bt = self._fill_tables(dec_ids, width).to(dev)
             ctx = torch.tensor(dec_len, dtype=torch.int32, device=dev)
-        sb = StepBatch(host[0], host[1], host[2], spans, rd, tables, bt, ctx, bs)
+        segments = None
+        if self.recurrent:
+            table = [(r0, r1 - r0, self.cache.state_slot(c[0]), start) for (r0, r1, start), c in zip(spans, chunks)]
+            table += [(rd + i, 1, self.cache.state_slot(s_), n - 1) for i, (s_, n) in enumerate(zip(dec_ids, dec_len))]
+            segments = Segments.of(table, dev)
+        sb = StepBatch(host[0], host[1], host[2], spans, rd, tables, bt, ctx, bs, segments)
         # logits only where they are asked for: by default the last row of every chunk that completes its prompt, and the
         # decode rows
         want = []
@@ -210,12 +223,15 @@ class ModelRunner:
         return [], (self.decode(dec_ids, dec_tok, dec_len) if dec_ids else None)
 
     # ---- decode ------------------------------------------------------------------------------------------------------
-    def _decode_body(self, ids, ctx, bt):
+    def _decode_segments(self, seq_ids, context_lens) -> list:
+        return [(i, 1, self.cache.state_slot(s), n - 1) for i, (s, n) in enumerate(zip(seq_ids, context_lens))]
+
+    def _decode_body(self, ids, ctx, bt, segments=None):
         """The device-side part of a decode step on static tensors (captured into a CUDA graph per batch size)."""
         B, bs = ids.shape[0], self.block_size
         pos = (ctx - 1).to(torch.int64)
         slots = bt.gather(1, (pos // bs).view(B, 1)).view(B).to(torch.int64) * bs + pos % bs
-        return self._run(StepBatch(ids, pos, slots, [], 0, [], bt, ctx, bs), None)
+        return self._run(StepBatch(ids, pos, slots, [], 0, [], bt, ctx, bs, segments), None)
 
     def _fill_tables(self, seq_ids, width: int) -> torch.Tensor:
         tables = [self.cache.block_table(s) for s in seq_ids]
@@ -235,7 +251,8 @@ class ModelRunner:
         ctx = torch.tensor(context_lens, dtype=torch.int32, device=dev)
         max_blocks = max(len(self.cache.block_table(s)) for s in seq_ids)
         bt = self._fill_tables(seq_ids, max_blocks).to(dev)
-        return self._decode_body(ids, ctx, bt)
+        seg = Segments.of(self._decode_segments(seq_ids, context_lens), dev) if self.recurrent else None
+        return self._decode_body(ids, ctx, bt, seg)
 
     def _table_width(self, context_lens) -> int:
         """Block-table columns of a graphed decode step: the model's whole context when that is at most 1024 blocks, else
@@ -249,7 +266,7 @@ class ModelRunner:
     def _decode_graphed(self, seq_ids, last_tokens, context_lens) -> torch.Tensor:
         """Replays one captured CUDA graph per batch size: the 10 to 20 launches per layer of a decode step are
         launch-bound from Python, the graph submits them in one call.  Inputs live in static device tensors that
-        are refreshed (three small copies) before each replay."""
+        are refreshed (a few small copies) before each replay."""
         B = len(seq_ids)
         dev = self.device
         width = self._table_width(context_lens)
@@ -258,18 +275,22 @@ class ModelRunner:
             ids = torch.zeros(B, dtype=torch.int64, device=dev)
             ctx = torch.ones(B, dtype=torch.int32, device=dev)
             bt = torch.zeros((B, width), dtype=torch.int32, device=dev)
-            g = {"ids": ids, "ctx": ctx, "bt": bt, "graph": None, "out": None}
+            g = {"ids": ids, "ctx": ctx, "bt": bt, "seg": None, "graph": None, "out": None}
+            if self.recurrent:
+                g["seg"] = Segments(torch.zeros((B, 4), dtype=torch.int32, device=dev), None)
             self._graphs[(B, width)] = g
         g["ids"].copy_(torch.tensor(last_tokens, dtype=torch.int64), non_blocking=True)
         g["ctx"].copy_(torch.tensor(context_lens, dtype=torch.int32), non_blocking=True)
         g["bt"].copy_(self._fill_tables(seq_ids, width), non_blocking=True)
+        if g["seg"] is not None:
+            g["seg"].table.copy_(torch.tensor(self._decode_segments(seq_ids, context_lens), dtype=torch.int32), non_blocking=True)
         if g["graph"] is None:
             # first use of this batch size: one eager run (lazy kernel configuration, tensor-map cache), then capture
-            out = self._decode_body(g["ids"], g["ctx"], g["bt"])
+            out = self._decode_body(g["ids"], g["ctx"], g["bt"], g["seg"])
             torch.cuda.current_stream().synchronize()
             graph = torch.cuda.CUDAGraph()
             with torch.cuda.graph(graph):
-                g["out"] = self._decode_body(g["ids"], g["ctx"], g["bt"])
+                g["out"] = self._decode_body(g["ids"], g["ctx"], g["bt"], g["seg"])
             g["graph"] = graph
             return out
         g["graph"].replay()
@@ -277,7 +298,7 @@ class ModelRunner:
 
 
 def load_runner(model: str, device=None, dtype=None, num_blocks: int = 1024, block_size: int = 16, weights: str | None = None,
-                seed: int = 0, **overrides) -> ModelRunner:
+                seed: int = 0, num_slots: int = 64, **overrides) -> ModelRunner:
     """Runner of a preset name or of a model folder (config.json + model.safetensors, the model class chosen by the
     configuration); `weights` names another safetensors file.  Without weights: random initialisation."""
     from ..models.registry import load_tensors, resolve_config
@@ -285,4 +306,5 @@ def load_runner(model: str, device=None, dtype=None, num_blocks: int = 1024, blo
     if device is None:
         device = "cuda" if torch.cuda.is_available() else "cpu"
     params = build_weights(cfg, device, dtype, load_tensors(model, weights), seed)
-    return ModelRunner(cfg, params=params, device=device, num_blocks=num_blocks, block_size=block_size, seed=seed)
+    return ModelRunner(cfg, params=params, device=device, num_blocks=num_blocks, block_size=block_size, seed=seed,
+                       num_slots=num_slots)

@@ -4,7 +4,7 @@
 
 Every input line is one step, a JSON object: {"step": 0, "entries": [{"id": "a", "tokens": [5, 17, 3], "want": [0, 2]}],
 "end": []}.  `tokens` are a request's next tokens, `want` the places among them whose logits are written, `end` the
-requests whose pages are given back after the step.  All entries of a step are one batch of `ModelRunner.step`, the call
+requests whose pages and state slot are given back after the step; at most four are live at any time.  All entries of a step are one batch of `ModelRunner.step`, the call
 the serving engine makes: portions of prompts beside single decoded tokens, steps of decoded tokens alone from a CUDA
 graph.  A step with wanted places writes OUT/<step>.f32 (little-endian 32-bit floats [wanted, vocab], in the order of the
 entries and of `want`); after every step a line "done <step>" is printed.  Nothing is sampled.
@@ -17,6 +17,7 @@ import os
 import sys
 
 PAGE = 16
+LIVE_REQUESTS = 4                     # state slots of models with recurrent layers
 
 
 def parse_args(argv=None):
@@ -92,7 +93,7 @@ def main(argv=None) -> int:
             raise RuntimeError("trace_run needs a CUDA device")
         torch.cuda.set_device(torch.device(a.device))
     runner = load_runner(a.model, device=a.device, dtype=getattr(torch, a.dtype), num_blocks=max(1, -(-a.max_tokens // PAGE)),
-                         block_size=PAGE)
+                         block_size=PAGE, num_slots=LIVE_REQUESTS)
     replay = TraceReplay(runner)
     for line in sys.stdin:
         if not line.strip():

@@ -1,5 +1,5 @@
-"""Inference weights (bf16; layered decoders also fp32), optionally sharded for tensor parallelism, under the parameter names the model
-runner uses.  Column-parallel matrices (QKV, gate/up, LM head) keep `1 / world` of their rows, row-parallel ones
+"""Inference weights (bf16; layered decoders also fp32), optionally sharded for tensor parallelism, under the parameter names the
+model runner uses.  Column-parallel matrices (QKV, gate/up, LM head) keep `1 / world` of their rows, row-parallel ones
 (attention output, down projection) `1 / world` of their columns; norms and the embedding are replicated."""
 from __future__ import annotations
 
@@ -9,6 +9,7 @@ import zlib
 import torch
 
 from ..models.config import GPTConfig
+from ..models.layered import ParallelSpec, up8
 
 
 class InferenceWeights:
@@ -107,9 +108,10 @@ class InferenceWeights:
     @classmethod
     def layered(cls, cfg, device, dtype=None, tensors: dict | None = None, seed: int = 0) -> "InferenceWeights":
         """Weights of a layered decoder (models.layered.LayeredConfig) in the layout of the serving kernels: one packed
-        attention projection [q | k | v | gate], experts stacked as [E, 2 ff, d] (gate over up) and [E, d, ff], the head
-        padded to whole GEMM tiles.  `tensors`: an unsharded checkpoint under `cfg.tensor_shapes()` names, loaded
-        strictly; None: random initialisation on the device.  `dtype`: bf16 or fp32 (default: bf16 on a GPU)."""
+        projection for everything that reads the same input (`packed_columns`), experts stacked as [E, 2 ff, d] (gate over up)
+        and [E, d, ff], the head padded to whole GEMM tiles; per-channel and per-head constants of recurrent layers in fp32.
+        `tensors`: an unsharded checkpoint under `cfg.tensor_shapes()` names, loaded strictly; None: random initialisation on
+        the device.  `dtype`: bf16 or fp32 (default: bf16 on a GPU).  Layers that share another's tensors have none here."""
         from ..core.errors import SerializationError, ShapeMismatch
         dev = torch.device(device)
         dt = dtype or (torch.bfloat16 if dev.type == "cuda" else torch.float32)
@@ -125,36 +127,54 @@ class InferenceWeights:
                 if tuple(tensors[k].shape) != tuple(want) and tensors[k].numel() != math.prod(want):
                     raise ShapeMismatch(want, tensors[k].shape, k)
 
-        def get(name):
+        def get(name, dt=dt):
             shape = shapes[name]
             if tensors is not None:
                 return tensors[name].reshape(shape).to(dev, dt)
-            if name.endswith("norm") or name.endswith("norm1") or name.endswith("norm2"):
+            last = name.rsplit(".", 1)[-1]
+            if last in ("norm", "norm1", "norm2", "out", "D"):
                 return torch.ones(shape, dtype=dt, device=dev)
-            if name.endswith(".b"):
+            if last == "b" and len(shape) == 1:
                 return torch.zeros(shape, dtype=dt, device=dev)
-            if name.endswith("vmix"):
+            if last in ("vmix", "alpha"):
                 return torch.full(shape, 0.5, dtype=dt, device=dev)
             g = torch.Generator(device=dev).manual_seed(zlib.crc32(f"{seed}/{name}".encode()))
-            return torch.empty(shape, dtype=torch.float32, device=dev).normal_(0.0, cfg.init_std, generator=g).to(dt)
+            if last == "A_log":
+                return torch.empty(shape, dtype=torch.float32, device=dev).uniform_(1.0, 16.0, generator=g).log().to(dt)
+            if last == "dt_bias":
+                return torch.empty(shape, dtype=torch.float32, device=dev).uniform_(-6.0, -2.0, generator=g).to(dt)
+            std = shape[-1] ** -0.5 if last == "conv" else cfg.init_std
+            return torch.empty(shape, dtype=torch.float32, device=dev).normal_(0.0, std, generator=g).to(dt)
+
+        def f32(name):
+            return get(name, torch.float32).contiguous()
 
         def gate_up(p, ff, out):
-            """gate rows over up rows; a hidden size that is not a multiple of 8 gets zero rows (silu(0) * 0 = 0)."""
+            """gate rows over up rows; a hidden size that is not a multiple of 8 gets zero rows (act(0) * 0 = 0)."""
             f8 = out.shape[0] // 2
             out[:ff] = get(p + "gate")
             out[f8:f8 + ff] = get(p + "up")
 
-        def up8(n):
-            return (n + 7) // 8 * 8
-
         d = cfg.d_model
         t = {"embed": get("embed"), "head": torch.zeros((cfg.vocab_padded, d), dtype=dt, device=dev)}
         t["head"][:cfg.vocab_size] = get("head")
-        t["final.norm"], t["final.norm.b"] = get("final.norm"), get("final.norm.b")
+
+        def norm(name):
+            if cfg.design.norm == "dyt":
+                t[name], t[name + ".b"], t[name + ".alpha"] = f32(name), f32(name + ".b"), f32(name + ".alpha").reshape(1)
+            else:
+                t[name], t[name + ".b"] = get(name), get(name + ".b")
+
+        norm("final.norm")
         for i, s in enumerate(cfg.layers):
+            if cfg.owner(i) != i:
+                continue
+            if cfg.design.block == "parallel":
+                norm(f"l{i}.norm1")
+                cls._parallel_block(t, f"l{i}.", s, d, get, f32, dt, dev)
+                continue
             p, m = f"l{i}.", s.mlp
-            for nm in ("norm1", "norm1.b"):
-                t[p + nm] = get(p + nm)
+            norm(p + "norm1")
             t[p + "attn.in"] = torch.cat([get(p + "mix." + c) for c in "qkvg"], 0)
             t[p + "attn.out"] = get(p + "mix.o")
             t[p + "attn.q_norm"], t[p + "attn.k_norm"] = get(p + "mix.q.norm"), get(p + "mix.k.norm")
@@ -162,8 +182,7 @@ class InferenceWeights:
                 t[p + "attn.mix"] = get(p + "mix.vmix").float().reshape(1).contiguous()
             if m is None:
                 continue
-            for nm in ("norm2", "norm2.b"):
-                t[p + nm] = get(p + nm)
+            norm(p + "norm2")
             t[p + "moe.router"] = get(p + "mlp.router")
             f8 = up8(m.ff)
             w1 = torch.zeros((m.experts, 2 * f8, d), dtype=dt, device=dev)
@@ -180,3 +199,74 @@ class InferenceWeights:
                 w2[:, :m.shared_ff] = get(p + "mlp.shared.down")
                 t[p + "shared.in"], t[p + "shared.out"] = w1, w2
         return cls(t, dt)
+
+    @staticmethod
+    def _parallel_block(t, p, s, d, get, f32, dt, dev) -> None:
+        """One layer whose mixer and feed-forward read the same input (`packed_columns` gives the columns)."""
+        cols, gates = packed_columns(s)
+        x = p + "mix."
+        par = isinstance(s.mixer, ParallelSpec)
+        parts = {"gate": p + "mlp.gate", "up": p + "mlp.up"}
+        if par:
+            w_in = get(x + "right.in")
+            inner, ch = s.mixer.right.inner, s.mixer.right.channels
+            parts.update({"q": x + "left.q", "k": x + "left.k", "v": x + "left.v", "z": w_in[:inner], "conv": w_in[inner:inner + ch]})
+            small = {"g": x + "left.g", "dt": w_in[inner + ch:]}
+        else:
+            parts.update({"q": x + "q", "k": x + "k", "v": x + "v", "z": x + "g"})
+            small = {"b": x + "b", "a": x + "a"}
+        for name, table, src in (("in", cols, parts), ("gates", gates, small)):
+            w = torch.zeros((table["end"][0], d), dtype=dt, device=dev)
+            for nm, (lo, n) in table.items():
+                if nm != "end":
+                    part = src[nm]
+                    w[lo:lo + n] = get(part) if isinstance(part, str) else part
+            t[p + name] = w
+        if par:
+            r = x + "right."
+            t[p + "left.o"], t[p + "right.o"] = get(x + "left.o"), get(r + "o")
+            t[p + "left.out"], t[p + "right.out"] = f32(x + "left.out"), f32(x + "right.out")
+            t[p + "conv"], t[p + "conv.b"] = f32(r + "conv"), f32(r + "conv.b")
+            for nm in ("dt_bias", "A_log", "D", "norm"):
+                t[p + nm] = f32(r + nm)
+            if s.mlp is not None:
+                t[p + "down"] = torch.zeros((d, up8(s.mlp.ff)), dtype=dt, device=dev)
+                t[p + "down"][:, :s.mlp.ff] = get(p + "mlp.down")
+            return
+        t[p + "conv"] = torch.cat([f32(x + c + ".conv") for c in "qkv"], 0)
+        for nm in ("dt_bias", "A_log", "norm"):
+            t[p + nm] = f32(x + nm)
+        # mixer and feed-forward outputs are added anyway: one product over the joined columns
+        n = s.mixer.heads * s.mixer.vdim
+        t[p + "out"] = torch.zeros((d, up8(n) + (up8(s.mlp.ff) if s.mlp is not None else 0)), dtype=dt, device=dev)
+        t[p + "out"][:, :n] = get(x + "o")
+        if s.mlp is not None:
+            t[p + "out"][:, up8(n):up8(n) + s.mlp.ff] = get(p + "mlp.down")
+
+
+def packed_columns(s) -> tuple:
+    """Columns of the two products over a parallel block's input: ({name: (first, count)} of the one in the activation dtype,
+    the same for the one whose results stay fp32: step sizes, decays and per-head gates).  "end": (total, 0).  Sections start at
+    multiples of 8; what the convolution reads is contiguous ("conv"; for a delta mixer that is q, k and v)."""
+    m = s.mixer
+    if isinstance(m, ParallelSpec):
+        a, r = m.left, m.right
+        groups = [[("q", a.heads * a.dim), ("k", a.kv_heads * a.dim), ("v", a.kv_heads * a.vdim)], [("z", r.inner)], [("conv", r.channels)]]
+        small = [[("g", a.heads)], [("dt", r.heads)]]
+    else:
+        groups = [[("q", m.kv_heads * m.dim), ("k", m.kv_heads * m.dim), ("v", m.heads * m.vdim)], [("z", m.heads * m.vdim)]]
+        small = [[("b", m.heads)], [("a", m.heads)]]
+    if s.mlp is not None:
+        groups.append([("gate", s.mlp.ff)])
+        groups.append([("up", s.mlp.ff)])
+
+    def place(groups):
+        out, at = {}, 0
+        for g in groups:
+            for nm, n in g:
+                out[nm] = (at, n)
+                at += n
+            at = up8(at)
+        out["end"] = (at, 0)
+        return out
+    return place(groups), place(small)
