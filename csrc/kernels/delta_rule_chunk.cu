@@ -1,0 +1,517 @@
+// Gated delta rule over prompts, chunked: 64 tokens at a time become matrix products on the tensor cores.
+//
+// With c_t the running sum of the logarithms of the decays inside a chunk, k and q unit vectors (q scaled) and S0 the state in
+// front of it, the corrections u_t = beta_t (v_t - decay_t S_{t-1}^T k_t) of a chunk solve a unit lower triangular system
+//   (I + L) U = R,  L_ts = beta_t exp(c_t - c_s) (k_t . k_s) for s < t,  R_t = beta_t (v_t - exp(c_t) S0^T k_t)
+// and then
+//   o_t = exp(c_t) S0^T q_t + sum_{s <= t} exp(c_t - c_s) (q_t . k_s) u_s,   S = exp(c_end) S0 + sum_s exp(c_end - c_s) k_s u_s^T
+// (the WY form of products of Householder-like matrices; Yang et al., "Gated Delta Networks: Improving Mamba2 with Delta Rule").
+//
+// Two kernels.  The first works on all chunks of all sequences at once: T = (I + L)^-1, the masked products q . k and the
+// per-token factors.  The second walks a sequence's chunks in order, one CTA (8 warps) per head and value columns, with the state
+// in fp32 accumulator registers.  Queries and keys enter the products as the bf16 numbers the convolution left; their norms, the
+// decays and beta are fp32 factors outside.  T, R, the state and what is added to it are split into two bf16 numbers (about 16 bits).
+#include "recurrent.h"
+
+#include "recurrent.cuh"
+#include "warp_mma.cuh"
+
+namespace rb {
+
+constexpr int kDcChunk = 64;
+constexpr float kDcUnitEps = 1e-6f;
+constexpr float kDcLog2e = 1.4426950408889634f;
+
+// scratch of one (chunk, head): T high half, T low half, A = masked q . k (bf16 [64, 64] each), then fp32 factors
+constexpr int kDcMat = kDcChunk * kDcChunk * 2;
+constexpr int kDcFactors = 5;              // [64] each: beta, key read-out, query read-out, key write, and one with exp(c_end) in [0]
+constexpr int kDcScratch = 3 * kDcMat + kDcFactors * kDcChunk * 4;
+
+// ---- first kernel: one CTA (4 warps) per chunk and head
+template <int DK>
+struct DcPrepSmem {
+  static constexpr int kPitch = DK + 8, kLPitch = kDcChunk + 4;
+  static constexpr int kQ = 0;
+  static constexpr int kK = kQ + kDcChunk * kPitch * 2;
+  static constexpr int kL = kK + kDcChunk * kPitch * 2;              // fp32 [64][68]: L, then (blocks solved so far) T
+  static constexpr int kT = kL + kDcChunk * kLPitch * 4;
+  static constexpr int kW = kT + kDcChunk * kLPitch * 4;             // fp32 [48][20] products of blocks
+  static constexpr int kF = kW + 48 * 20 * 4;                        // fp32 [4][64]: c, beta, 1 / |k|, scale / |q|
+  static constexpr int kTotal = kF + 4 * kDcChunk * 4;
+};
+
+template <int DK>
+__global__ void __launch_bounds__(128)
+delta_rule_prepare_kernel(const RbDeltaRuleArgs a) {
+  using L = DcPrepSmem<DK>;
+  constexpr int P = L::kPitch, LP = L::kLPitch;
+  extern __shared__ __align__(16) uint8_t dp_smem[];
+  const uint32_t sQ = smem_u32(dp_smem) + L::kQ, sK = smem_u32(dp_smem) + L::kK;
+  float* Lm = reinterpret_cast<float*>(dp_smem + L::kL);
+  float* T = reinterpret_cast<float*>(dp_smem + L::kT);
+  float* W = reinterpret_cast<float*>(dp_smem + L::kW);
+  float* cum = reinterpret_cast<float*>(dp_smem + L::kF);
+  float *beta = cum + kDcChunk, *rk = beta + kDcChunk, *rq = rk + kDcChunk;
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int gq = lane >> 2, tq = lane & 3;
+  const int h = blockIdx.x, tile = blockIdx.y;
+  const RcSegment seg = rc_segment(a.segments, a.tiles[2 * tile], a.num_slots);
+  const int off = a.tiles[2 * tile + 1];
+  if (off >= seg.len) return;
+  const int m_rows = min(kDcChunk, seg.len - off);
+  const int g = h / (a.heads / a.kv_heads);
+  const __nv_bfloat16* rows = reinterpret_cast<const __nv_bfloat16*>(a.qkv) + static_cast<long long>(seg.first + off) * a.ld_qkv;
+  const long long offQ = static_cast<long long>(g) * a.dk, offK = static_cast<long long>(a.kv_heads + g) * a.dk;
+  for (int i = tid; i < kDcChunk * (DK / 8); i += 128) {
+    const int r = i / (DK / 8), c = (i - r * (DK / 8)) * 8;
+    const bool ok = r < m_rows && c < a.dk;
+    const __nv_bfloat16* src = rows + (ok ? r * a.ld_qkv + c : 0);
+    wm_cp16(sQ + (r * P + c) * 2, ok ? src + offQ : rows, ok);
+    wm_cp16(sK + (r * P + c) * 2, ok ? src + offK : rows, ok);
+  }
+  wm_cp_commit();
+  if (warp == 0) {                                 // beta and running log2 decays, two tokens per lane
+    const float rate2 = expf(a.a_log[h]) * kDcLog2e, dt_bias = a.dt_bias[h];
+    float s[2];
+#pragma unroll
+    for (int i = 0; i < 2; ++i) {
+      const int t = 2 * lane + i;
+      const long long at = static_cast<long long>(seg.first + off + t) * a.ld_ab + h;
+      beta[t] = t < m_rows ? rc_sigmoid(a.b_raw[at]) : 0.f;
+      s[i] = t < m_rows ? -rate2 * rc_softplus(a.a_raw[at] + dt_bias) : 0.f;
+    }
+    float run = s[0] + s[1];
+#pragma unroll
+    for (int o = 1; o < 32; o <<= 1) {
+      const float u = __shfl_up_sync(0xffffffffu, run, o);
+      if (lane >= o) run += u;
+    }
+    cum[2 * lane] = run - s[1];
+    cum[2 * lane + 1] = run;
+  }
+  for (int i = tid; i < kDcChunk * LP; i += 128) T[i] = 0.f;
+  wm_cp_wait<0>();
+  __syncthreads();
+  {                                                // norms: two threads per row, one for the query and one for the key
+    const int r = tid & 63;
+    const __nv_bfloat16* row = reinterpret_cast<const __nv_bfloat16*>(dp_smem + (tid < 64 ? L::kQ : L::kK)) + r * P;
+    float s = 0.f;
+#pragma unroll 4
+    for (int c = 0; c < DK; c += 8) {
+      float v[8];
+      RcVec<__nv_bfloat16, 8>::load(row + c, v);
+#pragma unroll
+      for (int i = 0; i < 8; ++i) s = fmaf(v[i], v[i], s);
+    }
+    const float inv = 1.f / sqrtf(s + kDcUnitEps);
+    if (tid < 64) rq[r] = inv * rsqrtf(static_cast<float>(a.dk));
+    else rk[r] = inv;
+  }
+  __syncthreads();
+  uint8_t* scratch = reinterpret_cast<uint8_t*>(a.scratch) + (static_cast<long long>(tile) * a.heads + h) * kDcScratch;
+  __nv_bfloat16* outA = reinterpret_cast<__nv_bfloat16*>(scratch + 2 * kDcMat);
+  // ---- L and A: rows warp 16 .. + 16
+  {
+    uint32_t kf[DK / 16][4], qf[DK / 16][4];
+#pragma unroll
+    for (int k = 0; k < DK / 16; ++k) {
+      wm_ldsm_x4(wm_a(sK, P, warp * 16, k * 16, lane), kf[k]);
+      wm_ldsm_x4(wm_a(sQ, P, warp * 16, k * 16, lane), qf[k]);
+    }
+#pragma unroll
+    for (int sb = 0; sb < 4; ++sb) {
+      float kk[2][4], qk[2][4];
+#pragma unroll
+      for (int i = 0; i < 2; ++i)
+#pragma unroll
+        for (int j = 0; j < 4; ++j) kk[i][j] = qk[i][j] = 0.f;
+      if (sb <= warp) {
+#pragma unroll
+        for (int k = 0; k < DK / 16; ++k) {
+          uint32_t b[4];
+          wm_ldsm_x4(wm_b(sK, P, sb * 16, k * 16, lane), b);
+          wm_mma(kk[0], kf[k], b[0], b[1]);
+          wm_mma(kk[1], kf[k], b[2], b[3]);
+          wm_mma(qk[0], qf[k], b[0], b[1]);
+          wm_mma(qk[1], qf[k], b[2], b[3]);
+        }
+      }
+#pragma unroll
+      for (int i = 0; i < 2; ++i)
+#pragma unroll
+        for (int r = 0; r < 2; ++r) {
+          const int t = warp * 16 + gq + 8 * r, s = sb * 16 + i * 8 + 2 * tq;
+          float v[2];
+#pragma unroll
+          for (int j = 0; j < 2; ++j) {
+            const float d = s + j <= t ? wm_ex2(cum[t] - cum[s + j]) * rk[s + j] : 0.f;
+            Lm[t * LP + s + j] = s + j < t ? beta[t] * rk[t] * d * kk[i][2 * r + j] : 0.f;
+            v[j] = rq[t] * d * qk[i][2 * r + j];
+          }
+          *reinterpret_cast<uint32_t*>(outA + t * kDcChunk + s) = pack_bf16x2(v[0], v[1]);
+        }
+    }
+  }
+  __syncthreads();
+  // ---- T = (I + L)^-1: the four diagonal blocks of 16 by forward substitution, one thread per column ...
+  if (tid < 64) {
+    const int b0 = tid & ~15, j = tid & 15;
+    float x[16];
+#pragma unroll
+    for (int t = 0; t < 16; ++t) {
+      float v = t == j ? 1.f : 0.f;
+#pragma unroll
+      for (int s = 0; s < t; ++s) v = fmaf(-Lm[(b0 + t) * LP + b0 + s], x[s], v);
+      x[t] = v;                                    // zero above the diagonal
+      T[(b0 + t) * LP + b0 + j] = v;
+    }
+  }
+  __syncthreads();
+  // ---- ... then the blocks below: T_ij = -T_ii sum_{j <= k < i} L_ik T_kj, one distance i - j after the other
+#pragma unroll
+  for (int d = 1; d < 4; ++d) {
+    const int items = (4 - d) * 256;
+    for (int e = tid; e < items; e += 128) {
+      const int blk = e >> 8, r = (e >> 4) & 15, c = e & 15, i = blk + d;      // block row i, block column blk
+      float v = 0.f;
+      for (int k = blk * 16; k < i * 16; ++k) v = fmaf(Lm[(i * 16 + r) * LP + k], T[k * LP + blk * 16 + c], v);
+      W[(blk * 16 + r) * 20 + c] = v;
+    }
+    __syncthreads();
+    for (int e = tid; e < items; e += 128) {
+      const int blk = e >> 8, r = (e >> 4) & 15, c = e & 15, i = blk + d;
+      float v = 0.f;
+#pragma unroll
+      for (int k = 0; k < 16; ++k) v = fmaf(T[(i * 16 + r) * LP + i * 16 + k], W[(blk * 16 + k) * 20 + c], v);
+      T[(i * 16 + r) * LP + blk * 16 + c] = -v;
+    }
+    __syncthreads();
+  }
+  for (int e = tid; e < kDcChunk * kDcChunk / 8; e += 128) {
+    const int r = e >> 3, c = (e & 7) * 8;
+    uint32_t hi[4], lo[4];
+#pragma unroll
+    for (int k = 0; k < 4; ++k) wm_split(T[r * LP + c + 2 * k], T[r * LP + c + 2 * k + 1], hi[k], lo[k]);
+    *reinterpret_cast<uint4*>(scratch + (r * kDcChunk + c) * 2) = make_uint4(hi[0], hi[1], hi[2], hi[3]);
+    *reinterpret_cast<uint4*>(scratch + kDcMat + (r * kDcChunk + c) * 2) = make_uint4(lo[0], lo[1], lo[2], lo[3]);
+  }
+  if (tid < kDcChunk) {
+    float* f = reinterpret_cast<float*>(scratch + 3 * kDcMat);
+    const float c = cum[tid], c_end = cum[kDcChunk - 1], e = wm_ex2(c);
+    f[tid] = beta[tid];
+    f[kDcChunk + tid] = rk[tid] * e;
+    f[2 * kDcChunk + tid] = rq[tid] * e;
+    f[3 * kDcChunk + tid] = rk[tid] * wm_ex2(c_end - c);
+    f[4 * kDcChunk + tid] = wm_ex2(c_end);
+  }
+}
+
+// ---- second kernel
+template <int DK, int COLS>
+struct DcSmem {
+  static constexpr int kPitch = DK + 8, kVPitch = COLS + 8, kMPitch = kDcChunk + 8;
+  // one stage: what a chunk reads
+  static constexpr int kQ = 0;
+  static constexpr int kK = kQ + kDcChunk * kPitch * 2;
+  static constexpr int kV = kK + kDcChunk * kPitch * 2;
+  static constexpr int kM = kV + kDcChunk * kVPitch * 2;             // T high, T low, A
+  static constexpr int kF = kM + 3 * kDcChunk * kMPitch * 2;
+  static constexpr int kStage = kF + kDcFactors * kDcChunk * 4;
+  static constexpr int kS = 2 * kStage;                              // state, high and low half
+  static constexpr int kR = kS + 2 * DK * kVPitch * 2;               // R, high and low half
+  static constexpr int kU = kR + 2 * kDcChunk * kVPitch * 2;         // U (rounded)
+  static constexpr int kUs = kU + kDcChunk * kVPitch * 2;            // U scaled by what it adds to the state, high and low half
+  static constexpr int kTotal = kUs + 2 * kDcChunk * kVPitch * 2;
+};
+
+template <int DK, int COLS>
+__global__ void __launch_bounds__(256, 1)
+delta_rule_chunk_kernel(const RbDeltaRuleArgs a) {
+  using L = DcSmem<DK, COLS>;
+  constexpr int P = L::kPitch, VP = L::kVPitch, MP = L::kMPitch;
+  constexpr int MT = DK / 64, NJ = COLS / 32;      // state: MT row tiles; columns of a warp: NJ pairs of n-tiles
+  extern __shared__ __align__(16) uint8_t dc_smem[];
+  const uint32_t base = smem_u32(dc_smem);
+  const uint32_t sS = base + L::kS, sR = base + L::kR, sU = base + L::kU, sUs = base + L::kUs;
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int gq = lane >> 2, tq = lane & 3;
+  const int wc = warp >> 2, wr = wc ? 3 - (warp & 3) : (warp & 3);
+  const int ctiles = (a.dv + COLS - 1) / COLS;
+  const int h = blockIdx.x / ctiles, c0 = (blockIdx.x - h * ctiles) * COLS;
+  const RcSegment seg = rc_segment(a.segments, blockIdx.y, a.num_slots);
+  if (seg.len <= 0) return;
+  int tile0 = 0;                                   // first chunk of this segment in the scratch
+  for (int i = 0; i < static_cast<int>(blockIdx.y); ++i) tile0 += (max(0, a.segments[4 * i + 1]) + kDcChunk - 1) / kDcChunk;
+  const int g = h / (a.heads / a.kv_heads);
+  const __nv_bfloat16* qkv = reinterpret_cast<const __nv_bfloat16*>(a.qkv) + static_cast<long long>(seg.first) * a.ld_qkv;
+  const long long offQ = static_cast<long long>(g) * a.dk, offK = static_cast<long long>(a.kv_heads + g) * a.dk;
+  const long long offV = 2ll * a.kv_heads * a.dk + static_cast<long long>(h) * a.dv + c0;
+  const int chunks = (seg.len + kDcChunk - 1) / kDcChunk;
+
+  auto request = [&](int ci) {                     // everything chunk ci reads, into stage ci & 1
+    const uint32_t st = base + (ci & 1) * L::kStage;
+    const int t0 = ci * kDcChunk, m_rows = min(kDcChunk, seg.len - t0);
+    const __nv_bfloat16* rows = qkv + static_cast<long long>(t0) * a.ld_qkv;
+    for (int i = tid; i < kDcChunk * (DK / 8); i += 256) {
+      const int r = i / (DK / 8), c = (i - r * (DK / 8)) * 8;
+      const bool ok = r < m_rows && c < a.dk;
+      const __nv_bfloat16* src = rows + (ok ? r * a.ld_qkv + c : 0);
+      wm_cp16(st + L::kQ + (r * P + c) * 2, ok ? src + offQ : rows, ok);
+      wm_cp16(st + L::kK + (r * P + c) * 2, ok ? src + offK : rows, ok);
+    }
+    for (int i = tid; i < kDcChunk * (COLS / 8); i += 256) {
+      const int r = i / (COLS / 8), c = (i - r * (COLS / 8)) * 8;
+      const bool ok = r < m_rows && c0 + c < a.dv;
+      wm_cp16(st + L::kV + (r * VP + c) * 2, ok ? rows + r * a.ld_qkv + offV + c : rows, ok);
+    }
+    const uint8_t* scratch = reinterpret_cast<const uint8_t*>(a.scratch) + (static_cast<long long>(tile0 + ci) * a.heads + h) * kDcScratch;
+    for (int i = tid; i < 3 * kDcChunk * 8; i += 256) {
+      const int r = i >> 3, c = (i & 7) * 8;       // r: matrix * 64 + row
+      wm_cp16(st + L::kM + (r * MP + c) * 2, scratch + (r * kDcChunk + c) * 2, true);
+    }
+    if (tid < kDcFactors * kDcChunk / 4) wm_cp16(st + L::kF + tid * 16, scratch + 3 * kDcMat + tid * 16, true);
+    wm_cp_commit();
+  };
+  request(0);
+
+  // this thread's part of the state: rows n = wr DK/4 + 16 m + gq (+ 8), columns wc COLS/2 + 8 j + 2 tq (+ 1)
+  const int n_base = wr * (DK / 4) + gq, v_base = wc * (COLS / 2) + 2 * tq;
+  float S[MT][2 * NJ][4];
+  float* slot = a.state + (static_cast<long long>(seg.slot) * a.heads + h) * a.dk * a.dv;
+#pragma unroll
+  for (int m = 0; m < MT; ++m)
+#pragma unroll
+    for (int j = 0; j < 2 * NJ; ++j)
+#pragma unroll
+      for (int r = 0; r < 2; ++r) {
+        const int n = n_base + 16 * m + 8 * r, v = c0 + v_base + 8 * j;
+        float2 s = make_float2(0.f, 0.f);
+        if (seg.start > 0 && n < a.dk && v < a.dv) s = *reinterpret_cast<const float2*>(slot + static_cast<long long>(n) * a.dv + v);
+        S[m][j][2 * r] = s.x;
+        S[m][j][2 * r + 1] = s.y;
+      }
+  auto publish = [&]() {                           // the state as two bf16 numbers
+#pragma unroll
+    for (int m = 0; m < MT; ++m)
+#pragma unroll
+      for (int j = 0; j < 2 * NJ; ++j)
+#pragma unroll
+        for (int r = 0; r < 2; ++r) {
+          uint32_t hi, lo;
+          wm_split(S[m][j][2 * r], S[m][j][2 * r + 1], hi, lo);
+          const int at = ((n_base + 16 * m + 8 * r) * VP + v_base + 8 * j) * 2;
+          *reinterpret_cast<uint32_t*>(dc_smem + L::kS + at) = hi;
+          *reinterpret_cast<uint32_t*>(dc_smem + L::kS + DK * VP * 2 + at) = lo;
+        }
+  };
+  publish();
+
+  for (int ci = 0; ci < chunks; ++ci) {
+    wm_cp_wait<0>();
+    __syncthreads();                               // this chunk's tiles and the state have arrived
+    if (ci + 1 < chunks) request(ci + 1);
+    const uint32_t st = base + (ci & 1) * L::kStage;
+    const uint8_t* stp = dc_smem + (ci & 1) * L::kStage;
+    const float* f = reinterpret_cast<const float*>(stp + L::kF);
+    const int r0 = wr * 16 + gq, r1 = r0 + 8;
+    // ---- S0^T k and S0^T q for rows wr 16 .. + 16
+    float pm[2 * NJ][4], y[2 * NJ][4];
+#pragma unroll
+    for (int j = 0; j < 2 * NJ; ++j)
+#pragma unroll
+      for (int i = 0; i < 4; ++i) pm[j][i] = y[j][i] = 0.f;
+#pragma unroll
+    for (int k = 0; k < DK / 16; ++k) {
+      uint32_t kf[4], qf[4];
+      wm_ldsm_x4(wm_a(st + L::kK, P, wr * 16, k * 16, lane), kf);
+      wm_ldsm_x4(wm_a(st + L::kQ, P, wr * 16, k * 16, lane), qf);
+#pragma unroll
+      for (int j = 0; j < NJ; ++j) {
+        uint32_t b[4], bl[4];
+        wm_ldsm_x4_t(wm_b_t(sS, VP, wc * (COLS / 2) + j * 16, k * 16, lane), b);
+        wm_ldsm_x4_t(wm_b_t(sS + DK * VP * 2, VP, wc * (COLS / 2) + j * 16, k * 16, lane), bl);
+        wm_mma(pm[2 * j], kf, b[0], b[1]);
+        wm_mma(pm[2 * j + 1], kf, b[2], b[3]);
+        wm_mma(y[2 * j], qf, b[0], b[1]);
+        wm_mma(y[2 * j + 1], qf, b[2], b[3]);
+        wm_mma(pm[2 * j], kf, bl[0], bl[1]);
+        wm_mma(pm[2 * j + 1], kf, bl[2], bl[3]);
+      }
+    }
+    // ---- R
+    const __nv_bfloat16* V = reinterpret_cast<const __nv_bfloat16*>(stp + L::kV);
+#pragma unroll
+    for (int r = 0; r < 2; ++r) {
+      const int t = r ? r1 : r0;
+      const float be = f[t], kd = f[kDcChunk + t];
+#pragma unroll
+      for (int j = 0; j < 2 * NJ; ++j) {
+        const float2 v = unpack_bf16x2(*reinterpret_cast<const uint32_t*>(V + t * VP + v_base + 8 * j));
+        uint32_t hi, lo;
+        wm_split(be * (v.x - kd * pm[j][2 * r]), be * (v.y - kd * pm[j][2 * r + 1]), hi, lo);
+        const int at = (t * VP + v_base + 8 * j) * 2;
+        *reinterpret_cast<uint32_t*>(dc_smem + L::kR + at) = hi;
+        *reinterpret_cast<uint32_t*>(dc_smem + L::kR + kDcChunk * VP * 2 + at) = lo;
+      }
+    }
+    __syncthreads();
+    // ---- U = T R
+    float u[2 * NJ][4];
+#pragma unroll
+    for (int j = 0; j < 2 * NJ; ++j) u[j][0] = u[j][1] = u[j][2] = u[j][3] = 0.f;
+#pragma unroll
+    for (int k = 0; k < 4; ++k) {
+      if (k > wr) break;
+      uint32_t th[4], tl[4];
+      wm_ldsm_x4(wm_a(st + L::kM, MP, wr * 16, k * 16, lane), th);
+      wm_ldsm_x4(wm_a(st + L::kM + kDcChunk * MP * 2, MP, wr * 16, k * 16, lane), tl);
+#pragma unroll
+      for (int j = 0; j < NJ; ++j) {
+        uint32_t b[4], bl[4];
+        wm_ldsm_x4_t(wm_b_t(sR, VP, wc * (COLS / 2) + j * 16, k * 16, lane), b);
+        wm_ldsm_x4_t(wm_b_t(sR + kDcChunk * VP * 2, VP, wc * (COLS / 2) + j * 16, k * 16, lane), bl);
+        wm_mma(u[2 * j], th, b[0], b[1]);
+        wm_mma(u[2 * j + 1], th, b[2], b[3]);
+        wm_mma(u[2 * j], tl, b[0], b[1]);
+        wm_mma(u[2 * j + 1], tl, b[2], b[3]);
+        wm_mma(u[2 * j], th, bl[0], bl[1]);
+        wm_mma(u[2 * j + 1], th, bl[2], bl[3]);
+      }
+    }
+#pragma unroll
+    for (int r = 0; r < 2; ++r) {
+      const int t = r ? r1 : r0;
+      const float ks = f[3 * kDcChunk + t];
+#pragma unroll
+      for (int j = 0; j < 2 * NJ; ++j) {
+        const int at = (t * VP + v_base + 8 * j) * 2;
+        uint32_t hi, lo;
+        wm_split(ks * u[j][2 * r], ks * u[j][2 * r + 1], hi, lo);
+        *reinterpret_cast<uint32_t*>(dc_smem + L::kU + at) = pack_bf16x2(u[j][2 * r], u[j][2 * r + 1]);
+        *reinterpret_cast<uint32_t*>(dc_smem + L::kUs + at) = hi;
+        *reinterpret_cast<uint32_t*>(dc_smem + L::kUs + kDcChunk * VP * 2 + at) = lo;
+      }
+    }
+    __syncthreads();
+    // ---- state behind the chunk
+    const float e_end = f[4 * kDcChunk];
+#pragma unroll
+    for (int m = 0; m < MT; ++m)
+#pragma unroll
+      for (int j = 0; j < 2 * NJ; ++j)
+#pragma unroll
+        for (int i = 0; i < 4; ++i) S[m][j][i] *= e_end;
+#pragma unroll
+    for (int k = 0; k < 4; ++k) {
+      uint32_t af[MT][4];
+#pragma unroll
+      for (int m = 0; m < MT; ++m) wm_ldsm_x4_t(wm_a_t(st + L::kK, P, wr * (DK / 4) + m * 16, k * 16, lane), af[m]);
+#pragma unroll
+      for (int j = 0; j < NJ; ++j) {
+        uint32_t b[4], bl[4];
+        wm_ldsm_x4_t(wm_b_t(sUs, VP, wc * (COLS / 2) + j * 16, k * 16, lane), b);
+        wm_ldsm_x4_t(wm_b_t(sUs + kDcChunk * VP * 2, VP, wc * (COLS / 2) + j * 16, k * 16, lane), bl);
+#pragma unroll
+        for (int m = 0; m < MT; ++m) {
+          wm_mma(S[m][2 * j], af[m], b[0], b[1]);
+          wm_mma(S[m][2 * j + 1], af[m], b[2], b[3]);
+          wm_mma(S[m][2 * j], af[m], bl[0], bl[1]);
+          wm_mma(S[m][2 * j + 1], af[m], bl[2], bl[3]);
+        }
+      }
+    }
+    publish();                                     // every warp has read the old one
+    // ---- o = exp(c) S0^T q + A U
+    const float q0 = f[2 * kDcChunk + r0], q1 = f[2 * kDcChunk + r1];
+#pragma unroll
+    for (int j = 0; j < 2 * NJ; ++j) { y[j][0] *= q0; y[j][1] *= q0; y[j][2] *= q1; y[j][3] *= q1; }
+#pragma unroll
+    for (int k = 0; k < 4; ++k) {
+      if (k > wr) break;
+      uint32_t af[4];
+      wm_ldsm_x4(wm_a(st + L::kM + 2 * kDcChunk * MP * 2, MP, wr * 16, k * 16, lane), af);
+#pragma unroll
+      for (int j = 0; j < NJ; ++j) {
+        uint32_t b[4];
+        wm_ldsm_x4_t(wm_b_t(sU, VP, wc * (COLS / 2) + j * 16, k * 16, lane), b);
+        wm_mma(y[2 * j], af, b[0], b[1]);
+        wm_mma(y[2 * j + 1], af, b[2], b[3]);
+      }
+    }
+    const int t0 = ci * kDcChunk;
+    __nv_bfloat16* out = reinterpret_cast<__nv_bfloat16*>(a.o) + static_cast<long long>(seg.first + t0) * a.ld_o + static_cast<long long>(h) * a.dv + c0;
+#pragma unroll
+    for (int j = 0; j < 2 * NJ; ++j) {
+      const int v = v_base + 8 * j;
+      if (c0 + v >= a.dv) continue;
+      if (t0 + r0 < seg.len) *reinterpret_cast<uint32_t*>(out + r0 * a.ld_o + v) = pack_bf16x2(y[j][0], y[j][1]);
+      if (t0 + r1 < seg.len) *reinterpret_cast<uint32_t*>(out + r1 * a.ld_o + v) = pack_bf16x2(y[j][2], y[j][3]);
+    }
+  }
+#pragma unroll
+  for (int m = 0; m < MT; ++m)
+#pragma unroll
+    for (int j = 0; j < 2 * NJ; ++j)
+#pragma unroll
+      for (int r = 0; r < 2; ++r) {
+        const int n = n_base + 16 * m + 8 * r, v = c0 + v_base + 8 * j;
+        if (n < a.dk && v < a.dv)
+          *reinterpret_cast<float2*>(slot + static_cast<long long>(n) * a.dv + v) = make_float2(S[m][j][2 * r], S[m][j][2 * r + 1]);
+      }
+}
+
+template <int DK, int COLS>
+int dc_main_launch(const RbDeltaRuleArgs& a, cudaStream_t s) {
+  static_assert(DcSmem<DK, COLS>::kTotal <= 227 * 1024, "shared memory of a CTA");
+  auto kern = delta_rule_chunk_kernel<DK, COLS>;
+  const int smem = DcSmem<DK, COLS>::kTotal;
+  static bool cfg_dev[64] = {false};
+  bool& cfg = cfg_dev[rbhost::device_slot()];
+  if (!cfg) {
+    const cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+    if (e != cudaSuccess) return static_cast<int>(e);
+    cfg = true;
+  }
+  kern<<<dim3(a.heads * ((a.dv + COLS - 1) / COLS), a.num_segments), 256, smem, s>>>(a);
+  return static_cast<int>(cudaGetLastError());
+}
+
+template <int DK>
+int dc_launch(const RbDeltaRuleArgs& a, cudaStream_t s) {
+  auto prep = delta_rule_prepare_kernel<DK>;
+  const int smem = DcPrepSmem<DK>::kTotal;
+  static bool cfg_dev[64] = {false};
+  bool& cfg = cfg_dev[rbhost::device_slot()];
+  if (!cfg) {
+    const cudaError_t e = cudaFuncSetAttribute(prep, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+    if (e != cudaSuccess) return static_cast<int>(e);
+    cfg = true;
+  }
+  prep<<<dim3(a.heads, a.num_tiles), 128, smem, s>>>(a);
+  const int rc = static_cast<int>(cudaGetLastError());
+  if (rc) return rc;
+  // narrow column tiles (twice the CTAs) while wide ones would leave half of the SMs idle
+  const long long wide = static_cast<long long>(a.heads) * ((a.dv + 63) / 64) * a.num_segments;
+  return wide * 2 <= rbhost::device_sm_count() || a.dv <= 32 ? dc_main_launch<DK, 32>(a, s) : dc_main_launch<DK, 64>(a, s);
+}
+
+}  // namespace rb
+
+RB_API long long rb_delta_rule_scratch_bytes(int num_tiles, int heads) {
+  return static_cast<long long>(num_tiles) * heads * rb::kDcScratch;
+}
+
+RB_API int rb_delta_rule_chunked(const RbDeltaRuleArgs* args, void* stream_v) {
+  const RbDeltaRuleArgs& a = *args;
+  if (a.num_segments <= 0) return 0;
+  if (!a.qkv || !a.a_raw || !a.b_raw || !a.dt_bias || !a.a_log || !a.state || !a.o || !a.segments || !a.tiles || !a.scratch || a.f32 ||
+      a.heads <= 0 || a.kv_heads <= 0 || a.heads % a.kv_heads || a.dk <= 0 || a.dv <= 0 || a.num_slots <= 0 || a.num_tiles <= 0 ||
+      a.num_segments > 65535 || a.num_tiles > 65535)
+    return -1;
+  if (a.dk > 128 || ((a.dk | a.dv) & 7) || (a.ld_qkv & 7) || (a.ld_o & 1)) return -9;
+  if (((reinterpret_cast<uintptr_t>(a.qkv) | reinterpret_cast<uintptr_t>(a.state) | reinterpret_cast<uintptr_t>(a.scratch)) & 15) ||
+      (reinterpret_cast<uintptr_t>(a.o) & 3))
+    return -9;
+  cudaStream_t s = reinterpret_cast<cudaStream_t>(stream_v);
+  return a.dk <= 64 ? rb::dc_launch<64>(a, s) : rb::dc_launch<128>(a, s);
+}

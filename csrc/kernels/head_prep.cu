@@ -42,9 +42,11 @@ __device__ __forceinline__ void hp_put(float* p, float v) { *p = v; }
 struct HpItem {
   int kind, head;                                  // 0 query, 1 key, 2 value
 };
+// query heads without a norm need no work at all
+__host__ __device__ __forceinline__ int hp_queries(const RbHeadPrepArgs& a) { return a.q_gamma ? a.heads : 0; }
 __device__ __forceinline__ HpItem hp_item(int i, const RbHeadPrepArgs& a) {
-  if (i < a.heads) return {0, i};
-  i -= a.heads;
+  if (i < hp_queries(a)) return {0, i};
+  i -= hp_queries(a);
   if (i < a.kv_heads) return {1, i};
   return {2, i - a.kv_heads};
 }
@@ -54,7 +56,7 @@ __global__ void __launch_bounds__(128)
 head_prep_kernel(const RbHeadPrepArgs a RB_BOUNDS_PARAM) {
   using V = HpVec<T>;
   const int sub = threadIdx.x & (LANES - 1);
-  const int items = a.heads + 2 * a.kv_heads;
+  const int items = hp_queries(a) + 2 * a.kv_heads;
   const long long total = a.tokens * items;
   const long long per_grid = static_cast<long long>(gridDim.x) * (blockDim.x / LANES);
   const long long rounds = (total + per_grid - 1) / per_grid;
@@ -119,7 +121,7 @@ template <typename T>
 __global__ void __launch_bounds__(128)
 head_prep_scalar_kernel(const RbHeadPrepArgs a RB_BOUNDS_PARAM) {
   const int lane = threadIdx.x & 31;
-  const int items = a.heads + 2 * a.kv_heads;
+  const int items = hp_queries(a) + 2 * a.kv_heads;
   const long long total = a.tokens * items;
   const long long stride = static_cast<long long>(gridDim.x) * (blockDim.x >> 5);
   for (long long g = static_cast<long long>(blockIdx.x) * (blockDim.x >> 5) + (threadIdx.x >> 5); g < total; g += stride) {
@@ -163,7 +165,7 @@ int hp_launch(const RbHeadPrepArgs& a, cudaStream_t s) {
                          reinterpret_cast<uintptr_t>(a.k_cache) | reinterpret_cast<uintptr_t>(a.v_cache);
   const bool vec = !(bits & 15) && !((a.ld | a.off_q | a.off_k | a.off_v | a.dk | a.dv | (a.v_first ? a.ld_vf : 0)) % N) &&
                    a.dk <= 16 * N * kHpMaxVec && a.dv <= 16 * N * kHpMaxVec;
-  const long long total = a.tokens * (a.heads + 2 * a.kv_heads);
+  const long long total = a.tokens * (hp_queries(a) + 2 * a.kv_heads);
   const bool narrow = a.dk <= 8 * N && a.dv <= 8 * N;        // one vector per lane of a group of 8
   const int per_block = vec ? (narrow ? 16 : 8) : 4;
   long long blocks = (total + per_block - 1) / per_block;

@@ -42,6 +42,10 @@ typedef struct RbStateSpaceArgs {
   int num_segments, num_tiles, heads, groups, p, n, f32, num_slots;
 } RbStateSpaceArgs;
 int rb_state_space_scan(const RbStateSpaceArgs* args, void* stream);
+// The same for prompts on the tensor cores: bf16, n <= 128, n and p multiples of 8 (-9 otherwise).  `tiles` lists spans of `span`
+// rows (a multiple of 64, in order, every one listed), which run side by side.  span_state fp32 [num_tiles, heads, n, p] and
+// span_decay fp32 [num_tiles, heads] are scratch; both may be NULL when no segment has more than one span.
+int rb_state_space_chunked(const RbStateSpaceArgs* args, float* span_state, float* span_decay, int span, void* stream);
 
 // Gated delta rule.  Per value head h of query / key head g = h / (heads / kv_heads), with beta = sigmoid(b_raw),
 // decay = exp(-exp(a_log[h]) softplus(a_raw + dt_bias[h])), k' = k / sqrt(|k|^2 + 1e-6), q' = dk^(-1/2) q / sqrt(|q|^2 + 1e-6):
@@ -63,6 +67,10 @@ typedef struct RbDeltaRuleArgs {
   int num_segments, num_tiles, heads, kv_heads, dk, dv, f32, num_slots;
 } RbDeltaRuleArgs;
 int rb_delta_rule_scan(const RbDeltaRuleArgs* args, void* stream);
+// The same for prompts on the tensor cores: bf16, dk <= 128, dk and dv multiples of 8 (-9 otherwise).  `tiles` lists pieces of 64
+// rows, in order, every one listed; scratch: rb_delta_rule_scratch_bytes(num_tiles, heads) bytes.
+long long rb_delta_rule_scratch_bytes(int num_tiles, int heads);
+int rb_delta_rule_chunked(const RbDeltaRuleArgs* args, void* stream);
 
 // Every row of y consists of `parts` equal parts.  gate_first: u = y silu(z), out = u / rms(u) * weight; else:
 // out = y / rms(y) * weight * silu(z); rms over a part, with eps inside the root.  weight fp32 [weight_n]: the whole row or one

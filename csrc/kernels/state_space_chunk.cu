@@ -1,0 +1,308 @@
+// Mamba-2 state-space recurrence over prompts, chunked: 64 tokens at a time become matrix products on the tensor cores.
+//
+// With c_t the running sum of the logarithms of the decays inside a chunk and S0 the state in front of it,
+//   y_t = exp(c_t) C_t S0 + sum_{s <= t} exp(c_t - c_s) dt_s (C_t . B_s) x_s + D x_t
+//   S   = exp(c_end) S0 + sum_s B_s (exp(c_end - c_s) dt_s x_s)^T
+// One CTA (8 warps) owns 64 value columns of one head over a span of chunks.  The state stays in fp32 accumulator registers; its
+// bf16 copy in shared memory is the operand of the read-out only.  What enters the state is split into two bf16 numbers (about 16
+// bits), decays and step sizes are fp32, so the state itself is good to fp32-like accuracy.
+//
+// A long segment is cut into spans that run side by side: a first pass computes what every span but the last adds to the state
+// (from zero) and its total decay, and each span of the second pass starts from the combination of those before it.
+#include "recurrent.h"
+
+#include "recurrent.cuh"
+#include "warp_mma.cuh"
+
+namespace rb {
+
+constexpr int kScChunk = 64;
+constexpr int kScCols = 64;
+constexpr int kScThreads = 256;
+constexpr float kScLog2e = 1.4426950408889634f;
+
+template <int N>
+struct ScSmem {
+  static constexpr int kPitch = N + 8, kXPitch = kScCols + 8;
+  static constexpr int kC = 0;
+  static constexpr int kB = kC + kScChunk * kPitch * 2;
+  static constexpr int kX = kB + kScChunk * kPitch * 2;
+  static constexpr int kXs = kX + kScChunk * kXPitch * 2;           // scaled x: high half, low half
+  static constexpr int kS = kXs + 2 * kScChunk * kXPitch * 2;
+  static constexpr int kCum = kS + N * kXPitch * 2;                  // fp32 [64] cumulative log2 decay, then [64] step sizes
+  static constexpr int kTotal = kCum + 2 * kScChunk * 4;
+};
+
+template <int N, bool STATE_ONLY>
+__global__ void __launch_bounds__(kScThreads, 2)
+state_space_chunk_kernel(const RbStateSpaceArgs a, float* __restrict__ span_state, float* __restrict__ span_decay, int span) {
+  using L = ScSmem<N>;
+  constexpr int MT = N / 64;                       // 16-row tiles of the state per warp
+  constexpr int NP = L::kPitch, XP = L::kXPitch;
+  extern __shared__ __align__(16) uint8_t sc_smem[];
+  const uint32_t base = smem_u32(sc_smem);
+  const uint32_t sC = base + L::kC, sB = base + L::kB, sX = base + L::kX, sXs = base + L::kXs, sS = base + L::kS;
+  float* cum = reinterpret_cast<float*>(sc_smem + L::kCum);
+  float* dts = cum + kScChunk;
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int gq = lane >> 2, tq = lane & 3;
+  const int wc = warp >> 2, wr = wc ? 3 - (warp & 3) : (warp & 3);   // the causal work of a scheduler's two warps adds up evenly
+  const int ptiles = (a.p + kScCols - 1) / kScCols;
+  const int h = blockIdx.x / ptiles, c0 = (blockIdx.x - h * ptiles) * kScCols;
+  const int tile = blockIdx.y;
+  const RcSegment seg = rc_segment(a.segments, a.tiles[2 * tile], a.num_slots);
+  const int off = a.tiles[2 * tile + 1];
+  const int end = min(seg.len, off + span);
+  if (off >= seg.len) return;
+  if (STATE_ONLY && end == seg.len) return;        // nobody starts from what the last span adds
+  const int g = h / (a.heads / a.groups);
+  const __nv_bfloat16* xbc = reinterpret_cast<const __nv_bfloat16*>(a.xbc);
+  const long long offX = static_cast<long long>(h) * a.p + c0;
+  const long long offB = static_cast<long long>(a.heads) * a.p + static_cast<long long>(g) * a.n;
+  const long long offC = offB + static_cast<long long>(a.groups) * a.n;
+  const float rate2 = expf(a.a_log[h]) * kScLog2e, dt_bias = a.dt_bias[h], dskip = a.D[h];
+
+  // this thread's part of the state: rows n = wr N/4 + 16 m + gq (+ 8), columns wc 32 + 8 j + 2 tq (+ 1)
+  const int n_base = wr * (N / 4) + gq, p_base = wc * 32 + 2 * tq;
+  float S[MT][4][4];
+#pragma unroll
+  for (int m = 0; m < MT; ++m)
+#pragma unroll
+    for (int j = 0; j < 4; ++j) S[m][j][0] = S[m][j][1] = S[m][j][2] = S[m][j][3] = 0.f;
+  auto each = [&](auto f) {                        // f(two neighbouring entries, row, column)
+#pragma unroll
+    for (int m = 0; m < MT; ++m)
+#pragma unroll
+      for (int j = 0; j < 4; ++j)
+#pragma unroll
+        for (int r = 0; r < 2; ++r) {
+          const int n = n_base + 16 * m + 8 * r, p = c0 + p_base + 8 * j;
+          if (n < a.n && p < a.p) f(S[m][j][2 * r], S[m][j][2 * r + 1], static_cast<long long>(n) * a.p + p);
+        }
+  };
+  const long long state_n = static_cast<long long>(a.n) * a.p;
+  float* slot = a.state + (static_cast<long long>(seg.slot) * a.heads + h) * state_n;
+  if (!STATE_ONLY) {
+    if (seg.start > 0)
+      each([&](float& u, float& v, long long i) { const float2 s = *reinterpret_cast<const float2*>(slot + i); u = s.x; v = s.y; });
+    for (int t = tile - off / span; t < tile; ++t) {               // spans of this segment in front of this one
+      const float d = wm_ex2(span_decay[static_cast<long long>(t) * a.heads + h]);
+      const float* add = span_state + (static_cast<long long>(t) * a.heads + h) * state_n;
+      each([&](float& u, float& v, long long i) {
+        const float2 s = *reinterpret_cast<const float2*>(add + i);
+        u = fmaf(u, d, s.x);
+        v = fmaf(v, d, s.y);
+      });
+    }
+  }
+  float total = 0.f;
+
+  for (int t0 = off; t0 < end; t0 += kScChunk) {
+    const int m_rows = min(kScChunk, end - t0);
+    const __nv_bfloat16* rows = xbc + static_cast<long long>(seg.first + t0) * a.ld_xbc;
+    // ---- tiles of this chunk (rows past the end and columns past the real sizes are zero)
+    for (int i = tid; i < kScChunk * (N / 8); i += kScThreads) {
+      const int r = i / (N / 8), c = (i - r * (N / 8)) * 8;
+      const bool ok = r < m_rows && c < a.n;
+      const __nv_bfloat16* src = rows + (ok ? r * a.ld_xbc + c : 0);
+      wm_cp16(sB + (r * NP + c) * 2, ok ? src + offB : rows, ok);
+      if (!STATE_ONLY) wm_cp16(sC + (r * NP + c) * 2, ok ? src + offC : rows, ok);
+    }
+    for (int i = tid; i < kScChunk * (kScCols / 8); i += kScThreads) {
+      const int r = i / (kScCols / 8), c = (i - r * (kScCols / 8)) * 8;
+      const bool ok = r < m_rows && c0 + c < a.p;
+      wm_cp16(sX + (r * XP + c) * 2, ok ? rows + r * a.ld_xbc + offX + c : rows, ok);
+    }
+    wm_cp_commit();
+    if (warp == 0) {                               // step sizes and running log2 decays, two tokens per lane
+      float d[2], s[2];
+#pragma unroll
+      for (int i = 0; i < 2; ++i) {
+        const int t = 2 * lane + i;
+        d[i] = t < m_rows ? rc_softplus(a.dt_raw[static_cast<long long>(seg.first + t0 + t) * a.ld_dt + h] + dt_bias) : 0.f;
+        s[i] = -rate2 * d[i];
+      }
+      float run = s[0] + s[1];
+#pragma unroll
+      for (int o = 1; o < 32; o <<= 1) {
+        const float u = __shfl_up_sync(0xffffffffu, run, o);
+        if (lane >= o) run += u;
+      }
+      cum[2 * lane] = run - s[1];
+      cum[2 * lane + 1] = run;
+      dts[2 * lane] = d[0];
+      dts[2 * lane + 1] = d[1];
+    }
+    // ---- bf16 copy of the state in front of the chunk
+    if (!STATE_ONLY) {
+#pragma unroll
+      for (int m = 0; m < MT; ++m)
+#pragma unroll
+        for (int j = 0; j < 4; ++j)
+#pragma unroll
+          for (int r = 0; r < 2; ++r)
+            *reinterpret_cast<uint32_t*>(sc_smem + L::kS + ((n_base + 16 * m + 8 * r) * XP + p_base + 8 * j) * 2) =
+                pack_bf16x2(S[m][j][2 * r], S[m][j][2 * r + 1]);
+    }
+    wm_cp_wait<0>();
+    __syncthreads();
+    const float c_end = cum[kScChunk - 1];
+    // ---- x scaled by what it adds to the state
+    for (int i = tid; i < kScChunk * (kScCols / 8); i += kScThreads) {
+      const int r = i / (kScCols / 8), c = (i - r * (kScCols / 8)) * 8;
+      const float w = dts[r] * wm_ex2(c_end - cum[r]);
+      float v[8];
+      RcVec<__nv_bfloat16, 8>::load(reinterpret_cast<const __nv_bfloat16*>(sc_smem + L::kX) + r * XP + c, v);
+      uint32_t hi[4], lo[4];
+#pragma unroll
+      for (int k = 0; k < 4; ++k) wm_split(w * v[2 * k], w * v[2 * k + 1], hi[k], lo[k]);
+      *reinterpret_cast<uint4*>(sc_smem + L::kXs + (r * XP + c) * 2) = make_uint4(hi[0], hi[1], hi[2], hi[3]);
+      *reinterpret_cast<uint4*>(sc_smem + L::kXs + ((kScChunk + r) * XP + c) * 2) = make_uint4(lo[0], lo[1], lo[2], lo[3]);
+    }
+    if (!STATE_ONLY) {
+      // ---- y of rows wr 16 .. + 16, columns wc 32 .. + 32
+      float y[4][4];
+#pragma unroll
+      for (int j = 0; j < 4; ++j) y[j][0] = y[j][1] = y[j][2] = y[j][3] = 0.f;
+      uint32_t cf[N / 16][4];
+#pragma unroll
+      for (int k = 0; k < N / 16; ++k) {
+        wm_ldsm_x4(wm_a(sC, NP, wr * 16, k * 16, lane), cf[k]);
+#pragma unroll
+        for (int j = 0; j < 2; ++j) {
+          uint32_t b[4];
+          wm_ldsm_x4_t(wm_b_t(sS, XP, wc * 32 + j * 16, k * 16, lane), b);
+          wm_mma(y[2 * j], cf[k], b[0], b[1]);
+          wm_mma(y[2 * j + 1], cf[k], b[2], b[3]);
+        }
+      }
+      const int r0 = wr * 16 + gq, r1 = r0 + 8;
+      const float ct0 = cum[r0], ct1 = cum[r1];
+      const float e0 = wm_ex2(ct0), e1 = wm_ex2(ct1);
+#pragma unroll
+      for (int j = 0; j < 4; ++j) { y[j][0] *= e0; y[j][1] *= e0; y[j][2] *= e1; y[j][3] *= e1; }
+#pragma unroll
+      for (int sb = 0; sb < 4; ++sb) {             // 16 earlier tokens at a time
+        if (sb > wr) break;
+        float gacc[2][4];
+#pragma unroll
+        for (int i = 0; i < 2; ++i) gacc[i][0] = gacc[i][1] = gacc[i][2] = gacc[i][3] = 0.f;
+#pragma unroll
+        for (int k = 0; k < N / 16; ++k) {
+          uint32_t b[4];
+          wm_ldsm_x4(wm_b(sB, NP, sb * 16, k * 16, lane), b);
+          wm_mma(gacc[0], cf[k], b[0], b[1]);
+          wm_mma(gacc[1], cf[k], b[2], b[3]);
+        }
+        uint32_t af[4];
+#pragma unroll
+        for (int i = 0; i < 2; ++i) {
+          const int s0 = sb * 16 + i * 8 + 2 * tq;
+          const float2 cs = *reinterpret_cast<const float2*>(cum + s0), ds = *reinterpret_cast<const float2*>(dts + s0);
+          const float m00 = s0 <= r0 ? gacc[i][0] * ds.x * wm_ex2(ct0 - cs.x) : 0.f;
+          const float m01 = s0 + 1 <= r0 ? gacc[i][1] * ds.y * wm_ex2(ct0 - cs.y) : 0.f;
+          const float m10 = s0 <= r1 ? gacc[i][2] * ds.x * wm_ex2(ct1 - cs.x) : 0.f;
+          const float m11 = s0 + 1 <= r1 ? gacc[i][3] * ds.y * wm_ex2(ct1 - cs.y) : 0.f;
+          af[2 * i] = pack_bf16x2(m00, m01);
+          af[2 * i + 1] = pack_bf16x2(m10, m11);
+        }
+#pragma unroll
+        for (int j = 0; j < 2; ++j) {
+          uint32_t b[4];
+          wm_ldsm_x4_t(wm_b_t(sX, XP, wc * 32 + j * 16, sb * 16, lane), b);
+          wm_mma(y[2 * j], af, b[0], b[1]);
+          wm_mma(y[2 * j + 1], af, b[2], b[3]);
+        }
+      }
+      // ---- + D x, out
+      __nv_bfloat16* out = reinterpret_cast<__nv_bfloat16*>(a.y) + static_cast<long long>(seg.first + t0) * a.ld_y + offX;
+      const __nv_bfloat16* xs = reinterpret_cast<const __nv_bfloat16*>(sc_smem + L::kX);
+#pragma unroll
+      for (int j = 0; j < 4; ++j) {
+        const int p = p_base + 8 * j;
+        if (c0 + p >= a.p) continue;
+#pragma unroll
+        for (int r = 0; r < 2; ++r) {
+          const int t = r ? r1 : r0;
+          if (t >= m_rows) continue;
+          const float2 x = unpack_bf16x2(*reinterpret_cast<const uint32_t*>(xs + t * XP + p));
+          *reinterpret_cast<uint32_t*>(out + static_cast<long long>(t) * a.ld_y + p) =
+              pack_bf16x2(fmaf(dskip, x.x, y[j][2 * r]), fmaf(dskip, x.y, y[j][2 * r + 1]));
+        }
+      }
+    }
+    __syncthreads();                               // the scaled x is complete
+    // ---- state behind the chunk
+    const float e_end = wm_ex2(c_end);
+    total += c_end;
+#pragma unroll
+    for (int m = 0; m < MT; ++m)
+#pragma unroll
+      for (int j = 0; j < 4; ++j)
+#pragma unroll
+        for (int i = 0; i < 4; ++i) S[m][j][i] *= e_end;
+#pragma unroll
+    for (int k = 0; k < kScChunk / 16; ++k) {
+      uint32_t af[MT][4];
+#pragma unroll
+      for (int m = 0; m < MT; ++m) wm_ldsm_x4_t(wm_a_t(sB, NP, wr * (N / 4) + m * 16, k * 16, lane), af[m]);
+#pragma unroll
+      for (int half = 0; half < 2; ++half)
+#pragma unroll
+        for (int j = 0; j < 2; ++j) {
+          uint32_t b[4];
+          wm_ldsm_x4_t(wm_b_t(sXs + half * kScChunk * XP * 2, XP, wc * 32 + j * 16, k * 16, lane), b);
+#pragma unroll
+          for (int m = 0; m < MT; ++m) {
+            wm_mma(S[m][2 * j], af[m], b[0], b[1]);
+            wm_mma(S[m][2 * j + 1], af[m], b[2], b[3]);
+          }
+        }
+    }
+    __syncthreads();                               // every warp is done with the tiles
+  }
+  if (STATE_ONLY) {
+    float* dst = span_state + (static_cast<long long>(tile) * a.heads + h) * state_n;
+    each([&](float& u, float& v, long long i) { *reinterpret_cast<float2*>(dst + i) = make_float2(u, v); });
+    if (tid == 0 && c0 == 0) span_decay[static_cast<long long>(tile) * a.heads + h] = total;
+  } else if (end == seg.len) {
+    each([&](float& u, float& v, long long i) { *reinterpret_cast<float2*>(slot + i) = make_float2(u, v); });
+  }
+}
+
+template <int N>
+int sc_chunk_launch(const RbStateSpaceArgs& a, float* span_state, float* span_decay, int span, cudaStream_t s) {
+  const int smem = ScSmem<N>::kTotal;
+  auto first = state_space_chunk_kernel<N, true>;
+  auto second = state_space_chunk_kernel<N, false>;
+  static bool cfg_dev[64] = {false};
+  bool& cfg = cfg_dev[rbhost::device_slot()];
+  if (!cfg) {
+    cudaError_t e = cudaFuncSetAttribute(first, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+    if (e == cudaSuccess) e = cudaFuncSetAttribute(second, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+    if (e != cudaSuccess) return static_cast<int>(e);
+    cfg = true;
+  }
+  const dim3 grid(a.heads * ((a.p + kScCols - 1) / kScCols), a.num_tiles);
+  if (span_state) first<<<grid, kScThreads, smem, s>>>(a, span_state, span_decay, span);
+  second<<<grid, kScThreads, smem, s>>>(a, span_state, span_decay, span);
+  return static_cast<int>(cudaGetLastError());
+}
+
+}  // namespace rb
+
+RB_API int rb_state_space_chunked(const RbStateSpaceArgs* args, float* span_state, float* span_decay, int span, void* stream_v) {
+  const RbStateSpaceArgs& a = *args;
+  if (a.num_tiles <= 0) return 0;
+  if (!a.xbc || !a.dt_raw || !a.dt_bias || !a.a_log || !a.D || !a.state || !a.y || !a.segments || !a.tiles || a.f32 || a.heads <= 0 ||
+      a.groups <= 0 || a.heads % a.groups || a.p <= 0 || a.n <= 0 || a.num_slots <= 0 || a.num_tiles > 65535 || span <= 0 ||
+      span % rb::kScChunk || (span_state != nullptr) != (span_decay != nullptr))
+    return -1;
+  if (a.n > 128 || ((a.n | a.p) & 7) || ((a.ld_xbc | a.ld_y) & 7)) return -9;
+  if ((reinterpret_cast<uintptr_t>(a.xbc) | reinterpret_cast<uintptr_t>(a.y) | reinterpret_cast<uintptr_t>(a.state) |
+       reinterpret_cast<uintptr_t>(span_state)) & 15)
+    return -9;
+  cudaStream_t s = reinterpret_cast<cudaStream_t>(stream_v);
+  return a.n <= 64 ? rb::sc_chunk_launch<64>(a, span_state, span_decay, span, s)
+                   : rb::sc_chunk_launch<128>(a, span_state, span_decay, span, s);
+}

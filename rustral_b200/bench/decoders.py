@@ -81,7 +81,8 @@ def _time(fn, iters: int, warmup: int = 3, flush=None) -> float:
 
 
 def throughput(cfg, prompts=((4, 2048), (1, 8192)), decodes=((1, 2048), (32, 2048), (64, 4000)), iters: int = 8) -> dict:
-    runner = ModelRunner(cfg, params=build_weights(cfg, "cuda"), device="cuda", num_blocks=64 * 4096 // 16 + 64, block_size=16)
+    runner = ModelRunner(cfg, params=build_weights(cfg, "cuda"), device="cuda", num_blocks=64 * 4096 // 16 + 64, block_size=16,
+                         num_slots=max(B for B, _ in decodes))
     g = torch.Generator().manual_seed(0)
     out = {}
     for n, L in prompts:

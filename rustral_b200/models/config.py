@@ -3,7 +3,7 @@ from __future__ import annotations
 
 from dataclasses import dataclass, asdict
 
-from .layered import LayeredConfig, uniform_layers
+from .layered import LayeredConfig, hybrid_layers, uniform_layers
 
 
 @dataclass
@@ -95,12 +95,29 @@ PRESETS = {
                         mixer=dict(heads=32, kv_heads=8, dim=128, vdim=128, scale=0.08838834764831845, softcap=30.0, chunk=8192,
                                    v_mix=True),
                         mlp=dict(ff=1792, experts=32, top=7, groups=4, keep=2, shared_ff=1792)),
+    # layered decoders whose mixers carry state (order: p = attention beside a state-space mixer, d = delta rule)
+    "vafodra-test": dict(arch="Vafodra", vocab_size=1000, d_model=128, seq_len=512, embed_scale=6.0, residual_mult=0.4, order="pdpd",
+                         weights_of={2: 0},
+                         left=dict(heads=6, kv_heads=2, dim=48, vdim=32, scale=0.15, window=40, keep_first=3),
+                         right=dict(heads=4, vdim=40, state=24, groups=2, norm_groups=4, conv=3),
+                         delta=dict(heads=6, kv_heads=3, dim=24, vdim=40, conv=4), ff=dict(p=192, d=256)),
+    # about the size of a Llama-8B layer: same width, heads and head size, the feed-forward takes what the mixers leave of the
+    # parameters
+    "vafodra-8b": dict(arch="Vafodra", vocab_size=128256, d_model=4096, embed_scale=1.0, residual_mult=0.5, order="ppdp" * 8,
+                       left=dict(heads=32, kv_heads=8, dim=128, vdim=128, scale=0.08838834764831845, window=2048, keep_first=4),
+                       right=dict(heads=128, vdim=64, state=128, groups=8, norm_groups=8, conv=4),
+                       delta=dict(heads=32, kv_heads=16, dim=128, vdim=128, conv=4), ff=dict(p=5376, d=12288)),
 }
 
 
 def preset(name: str, **overrides):
     cfg = dict(PRESETS[name])
     cfg.update(overrides)
+    if "order" in cfg:
+        if "n_layer" in cfg:
+            cfg["order"] = (cfg["order"] * cfg["n_layer"])[:cfg.pop("n_layer")]
+        cfg["layers"] = hybrid_layers(*(cfg.pop(k) for k in ("order", "left", "right", "delta", "ff")), cfg.pop("weights_of", None))
+        return LayeredConfig(**cfg)
     if "mixer" in cfg:
         cfg["layers"] = uniform_layers(cfg.pop("n_layer"), cfg.pop("mixer"), cfg.pop("mlp"))
         return LayeredConfig(**cfg)

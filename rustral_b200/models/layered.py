@@ -408,8 +408,10 @@ def uniform_layers(n: int, mixer: dict, mlp: dict | None) -> tuple:
     return tuple(LayerSpec(AttentionSpec(**mixer), MoESpec(**mlp) if mlp else None) for _ in range(n))
 
 
-def hybrid_layers(order: str, left: dict, right: dict, delta: dict, ff: int | None, weights_of: dict | None = None) -> tuple:
-    """Layers of a Vafodra model: 'p' a parallel mixer (`left`, `right`), 'd' a delta mixer; `weights_of`: layer -> owner."""
+def hybrid_layers(order: str, left: dict, right: dict, delta: dict, ff: dict, weights_of: dict | None = None) -> tuple:
+    """Layers of a Vafodra model: 'p' a parallel mixer (`left`, `right`), 'd' a delta mixer; `ff`: hidden size of the
+    feed-forward behind either ({'p': .., 'd': ..}, 0: none); `weights_of`: layer -> owner."""
     fixed = {k: v for k, v in DESIGNS["Vafodra"].attention.items() if k != "sliding"}
+    act = DESIGNS["Vafodra"].act
     mixers = {"p": ParallelSpec(AttentionSpec(**left, **fixed), StateSpaceSpec(**right)), "d": DeltaSpec(**delta)}
-    return tuple(LayerSpec(mixers[c], DenseSpec(ff) if ff else None, (weights_of or {}).get(i)) for i, c in enumerate(order))
+    return tuple(LayerSpec(mixers[c], DenseSpec(ff[c], act) if ff[c] else None, (weights_of or {}).get(i)) for i, c in enumerate(order))

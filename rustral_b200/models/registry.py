@@ -57,7 +57,8 @@ _GPT_KERNELS = ("gemm_tcgen05", "embedding", "elementwise", "norm", "rope", "att
 _LAYERED_KERNELS = ("gemm_tcgen05", "gemm_f32", "embedding", "elementwise", "residual_norm", "head_prep", "moe",
                     "attention_fwd2", "paged_attention")
 _HYBRID_KERNELS = ("gemm_tcgen05", "gemm_f32", "embedding", "elementwise", "residual_norm", "head_prep", "moe", "attention_fwd2",
-                   "paged_attention", "short_conv", "state_space", "delta_rule", "gated_norm")
+                   "paged_attention", "short_conv", "state_space", "state_space_chunk", "delta_rule",
+                   "delta_rule_chunk", "gated_norm")
 
 ARCHITECTURES = {a.name: a for a in (
     Architecture("gpt2", _gpt_config, "GPTBody", False, _gpt_weights, _GPT_KERNELS),

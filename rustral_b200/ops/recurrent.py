@@ -18,6 +18,12 @@ N.optional_sig("rb_short_conv", [N.C.POINTER(N.RbShortConvArgs), N.c_void_p])
 N.optional_sig("rb_state_space_scan", [N.C.POINTER(N.RbStateSpaceArgs), N.c_void_p])
 N.optional_sig("rb_delta_rule_scan", [N.C.POINTER(N.RbDeltaRuleArgs), N.c_void_p])
 N.optional_sig("rb_gated_norm", [N.C.POINTER(N.RbGatedNormArgs), N.c_void_p])
+N.optional_sig("rb_state_space_chunked", [N.C.POINTER(N.RbStateSpaceArgs), N.c_void_p, N.c_void_p, N.c_int, N.c_void_p])
+N.optional_sig("rb_delta_rule_chunked", [N.C.POINTER(N.RbDeltaRuleArgs), N.c_void_p])
+N.optional_sig("rb_delta_rule_scratch_bytes", [N.c_int, N.c_int], N.c_ll)
+N._LAUNCHES["rb_delta_rule_chunked"] = 2
+
+CHUNK = 64                                            # tokens per step of the chunked kernels
 
 
 class Segments:
@@ -31,6 +37,7 @@ class Segments:
         self.table, self.rows = table, rows
         self.n = table.shape[0]
         self._tiles: dict = {}
+        self._split = None
 
     @classmethod
     def of(cls, rows: list, device) -> "Segments":
@@ -40,6 +47,18 @@ class Segments:
     def single(self) -> bool:
         """Every segment is one row (a decode step)."""
         return self.rows is None or all(r[1] == 1 for r in self.rows)
+
+    def split(self) -> tuple:
+        """(segments of several rows, segments of one row), either None when there are none."""
+        if self._split is None:
+            if self.single:
+                self._split = (None, self)
+            else:
+                many = [i for i, r in enumerate(self.rows) if r[1] > 1]
+                one = [i for i, r in enumerate(self.rows) if r[1] <= 1]
+                part = lambda idx: Segments(self.table[torch.tensor(idx, device=self.table.device)], [self.rows[i] for i in idx])
+                self._split = (self if not one else part(many), part(one) if one else None)
+        return self._split
 
     def tiles(self, size: int) -> torch.Tensor:
         """int32 [tiles, 2]: (segment, first row inside it) of pieces of at most `size` rows."""
@@ -100,6 +119,30 @@ def _softplus(z):
     return torch.clamp(z, min=0) + torch.log1p(torch.exp(-z.abs()))
 
 
+def _chunked(x, rows: int, a: int, b: int) -> bool:
+    """Whether the tensor-core kernels take prompts of these operands: `rows` state rows, head sizes a and b."""
+    return x.dtype == torch.bfloat16 and rows <= 128 and a % 8 == 0 and b % 8 == 0 and x.stride(0) % 8 == 0 and x.data_ptr() % 16 == 0
+
+
+def _span(seg: Segments, ctas_per_span: int, slots: int = 2 * 148) -> int:
+    """Rows per span of the chunked state-space kernel: the power of two for which the spans that run side by side cost least
+    (rounds of `slots` CTAs, and about half of that again for the first pass where segments have several spans)."""
+    lens = [r[1] for r in seg.rows]
+    best, span = None, CHUNK
+    size = 256
+    while True:
+        spans = sum(-(-n // size) for n in lens)
+        rows = min(size, max(lens))
+        cost = -(-spans * ctas_per_span // slots) * (rows + 64.0)
+        if spans > len(lens):
+            cost += 0.5 * -(-(spans - len(lens)) * ctas_per_span // slots) * (rows + 64.0)
+        if best is None or cost < best:
+            best, span = cost, size
+        if size >= max(lens):
+            return span
+        size *= 2
+
+
 def state_space(xbc, dt_raw, *, dt_bias, a_log, D, state, heads: int, groups: int, vdim: int, n: int, seg: Segments, out=None):
     """Mamba-2 recurrence.  xbc [rows, heads * vdim + 2 * groups * n] = x | B | C behind the convolution; dt_raw fp32
     [rows, heads]; dt_bias, a_log, D fp32 [heads]; state fp32 [slots, heads, n, up4(vdim)].  Returns y [rows, heads * vdim]."""
@@ -123,12 +166,23 @@ def state_space(xbc, dt_raw, *, dt_bias, a_log, D, state, heads: int, groups: in
     if n > MAX_STATE_ROWS:
         raise ValueError(f"state_space: at most {MAX_STATE_ROWS} state rows per head")
     _check(dt_raw, torch.float32, "state_space")
+    many, one = seg.split() if _chunked(xbc, n, n, vdim) and out.stride(0) % 8 == 0 and out.data_ptr() % 16 == 0 else (None, seg)
     a = N.RbStateSpaceArgs()
     a.xbc, a.ld_xbc, a.dt_raw, a.ld_dt, a.y, a.ld_y = xbc.data_ptr(), xbc.stride(0), dt_raw.data_ptr(), dt_raw.stride(0), out.data_ptr(), out.stride(0)
     a.dt_bias, a.a_log, a.D, a.state, a.num_slots = dt_bias.data_ptr(), a_log.data_ptr(), D.data_ptr(), state.data_ptr(), state.shape[0]
-    a.segments, a.num_segments = seg.table.data_ptr(), seg.n
     a.heads, a.groups, a.p, a.n, a.f32 = heads, groups, vdim, n, int(xbc.dtype == torch.float32)
-    N.check(N.kernels().rb_state_space_scan(a, N.stream_ptr()), "rb_state_space_scan")
+    if one is not None:
+        a.segments, a.num_segments = one.table.data_ptr(), one.n
+        N.check(N.kernels().rb_state_space_scan(a, N.stream_ptr()), "rb_state_space_scan")
+    if many is not None:
+        span = _span(many, heads * ((vdim + 63) // 64))
+        tiles = many.tiles(span)
+        a.segments, a.num_segments, a.tiles, a.num_tiles = many.table.data_ptr(), many.n, tiles.data_ptr(), tiles.shape[0]
+        states = decays = None
+        if tiles.shape[0] > many.n:
+            states = torch.empty((tiles.shape[0], heads, n, vdim), dtype=torch.float32, device=xbc.device)
+            decays = torch.empty((tiles.shape[0], heads), dtype=torch.float32, device=xbc.device)
+        N.check(N.kernels().rb_state_space_chunked(a, N.ptr(states), N.ptr(decays), span, N.stream_ptr()), "rb_state_space_chunked")
     return out
 
 
@@ -161,13 +215,22 @@ def delta_rule(qkv, a_raw, b_raw, *, dt_bias, a_log, state, heads: int, kv_heads
     _check(b_raw, torch.float32, "delta_rule")
     if a_raw.stride(0) != b_raw.stride(0):
         raise ValueError("delta_rule: a_raw and b_raw must have the same pitch")
+    many, one = seg.split() if _chunked(qkv, dk, dk, dv) and out.stride(0) % 2 == 0 and out.data_ptr() % 4 == 0 else (None, seg)
     a = N.RbDeltaRuleArgs()
     a.qkv, a.ld_qkv, a.o, a.ld_o = qkv.data_ptr(), qkv.stride(0), out.data_ptr(), out.stride(0)
     a.a_raw, a.b_raw, a.ld_ab = a_raw.data_ptr(), b_raw.data_ptr(), a_raw.stride(0)
     a.dt_bias, a.a_log, a.state, a.num_slots = dt_bias.data_ptr(), a_log.data_ptr(), state.data_ptr(), state.shape[0]
-    a.segments, a.num_segments = seg.table.data_ptr(), seg.n
     a.heads, a.kv_heads, a.dk, a.dv, a.f32 = heads, kv_heads, dk, dv, int(qkv.dtype == torch.float32)
-    N.check(N.kernels().rb_delta_rule_scan(a, N.stream_ptr()), "rb_delta_rule_scan")
+    lib = N.kernels()
+    if one is not None:
+        a.segments, a.num_segments = one.table.data_ptr(), one.n
+        N.check(lib.rb_delta_rule_scan(a, N.stream_ptr()), "rb_delta_rule_scan")
+    if many is not None:
+        tiles = many.tiles(CHUNK)
+        scratch = torch.empty(lib.rb_delta_rule_scratch_bytes(tiles.shape[0], heads), dtype=torch.uint8, device=qkv.device)
+        a.segments, a.num_segments, a.tiles, a.num_tiles = many.table.data_ptr(), many.n, tiles.data_ptr(), tiles.shape[0]
+        a.scratch = scratch.data_ptr()
+        N.check(lib.rb_delta_rule_chunked(a, N.stream_ptr()), "rb_delta_rule_chunked")
     return out
 
 
