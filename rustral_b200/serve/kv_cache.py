@@ -197,8 +197,9 @@ class PagedCache:
             raise InvalidArgument("PagedCache: num_blocks and block_size must be positive")
         self.k = self.v = None
         self.state = [{} for _ in range(num_layers)]
-        self.num_slots = num_slots if layers is not None and any(c.state for c in layers) else 0
-        if self.num_slots and self._lib.rb_ba_set_state_slots(self._h, num_slots) != 0:
+        recurrent = layers is not None and any(c.state for c in layers)
+        self.num_slots = num_slots if recurrent else 0
+        if recurrent and self._lib.rb_ba_set_state_slots(self._h, num_slots) != 0:
             raise InvalidArgument("PagedCache: num_slots must be positive")
         if allocate_storage and layers is not None:
             def pages(c, d):
