@@ -7,10 +7,14 @@
 //   o_t = exp(c_t) S0^T q_t + sum_{s <= t} exp(c_t - c_s) (q_t . k_s) u_s,   S = exp(c_end) S0 + sum_s exp(c_end - c_s) k_s u_s^T
 // (the WY form of products of Householder-like matrices; Yang et al., "Gated Delta Networks: Improving Mamba2 with Delta Rule").
 //
-// Two kernels.  The first works on all chunks of all sequences at once: T = (I + L)^-1, the masked products q . k and the
-// per-token factors.  The second walks a sequence's chunks in order, one CTA (8 warps) per head and value columns, with the state
-// in fp32 accumulator registers.  Queries and keys enter the products as the bf16 numbers the convolution left; their norms, the
-// decays and beta are fp32 factors outside.  T, R, the state and what is added to it are split into two bf16 numbers (about 16 bits).
+// With T = (I + L)^-1, A the masked products exp(c_t - c_s) (q_t . k_s) and U = T R, nothing but R is needed of a chunk once S0 is
+// known: o = exp(c) S0^T q + (A T) R and S = exp(c_end) S0 + W^T R with W = T^T diag(exp(c_end - c)) K.  (A T also has none of the
+// cancellation between A and U when keys are much alike.)
+//
+// Two kernels.  The first works on all chunks of all sequences at once: A T, W and the per-token factors.  The second walks a
+// sequence's chunks in order, one CTA (8 warps) per head and value columns, with the state in fp32 accumulator registers.  Queries
+// and keys enter the products as the bf16 numbers the convolution left; their norms, the decays and beta are fp32 factors outside.
+// R, W, the state and what is added to it are split into two bf16 numbers (about 16 bits).
 #include "recurrent.h"
 
 #include "recurrent.cuh"
@@ -22,10 +26,10 @@ constexpr int kDcChunk = 64;
 constexpr float kDcUnitEps = 1e-6f;
 constexpr float kDcLog2e = 1.4426950408889634f;
 
-// scratch of one (chunk, head): T high half, T low half, A = masked q . k (bf16 [64, 64] each), then fp32 factors
+// scratch of one (chunk, head): A T (bf16 [64, 64]), W (bf16 [64, DK], high and low half), then fp32 factors
 constexpr int kDcMat = kDcChunk * kDcChunk * 2;
-constexpr int kDcFactors = 5;              // [64] each: beta, key read-out, query read-out, key write, and one with exp(c_end) in [0]
-constexpr int kDcScratch = 3 * kDcMat + kDcFactors * kDcChunk * 4;
+constexpr int kDcFactors = 4;              // [64] each: beta, key read-out, query read-out, and one with exp(c_end) in [0]
+__host__ __device__ constexpr int dc_scratch(int DK) { return kDcMat + 2 * kDcChunk * DK * 2 + kDcFactors * kDcChunk * 4; }
 
 // ---- first kernel: one CTA (4 warps) per chunk and head
 template <int DK>
@@ -33,8 +37,9 @@ struct DcPrepSmem {
   static constexpr int kPitch = DK + 8, kLPitch = kDcChunk + 4;
   static constexpr int kQ = 0;
   static constexpr int kK = kQ + kDcChunk * kPitch * 2;
-  static constexpr int kL = kK + kDcChunk * kPitch * 2;              // fp32 [64][68]: L, then (blocks solved so far) T
-  static constexpr int kT = kL + kDcChunk * kLPitch * 4;
+  static constexpr int kTPitch = kDcChunk + 8;
+  static constexpr int kL = kK + kDcChunk * kPitch * 2;              // fp32 [64][68]: L; later T as bf16 [2][64][72]
+  static constexpr int kT = kL + 2 * kDcChunk * kTPitch * 2;         // fp32 [64][68]
   static constexpr int kW = kT + kDcChunk * kLPitch * 4;             // fp32 [48][20] products of blocks
   static constexpr int kF = kW + 48 * 20 * 4;                        // fp32 [4][64]: c, beta, 1 / |k|, scale / |q|
   static constexpr int kTotal = kF + 4 * kDcChunk * 4;
@@ -108,9 +113,9 @@ delta_rule_prepare_kernel(const RbDeltaRuleArgs a) {
     else rk[r] = inv;
   }
   __syncthreads();
-  uint8_t* scratch = reinterpret_cast<uint8_t*>(a.scratch) + (static_cast<long long>(tile) * a.heads + h) * kDcScratch;
-  __nv_bfloat16* outA = reinterpret_cast<__nv_bfloat16*>(scratch + 2 * kDcMat);
-  // ---- L and A: rows warp 16 .. + 16
+  uint8_t* scratch = reinterpret_cast<uint8_t*>(a.scratch) + (static_cast<long long>(tile) * a.heads + h) * dc_scratch(DK);
+  // ---- L and A: rows warp 16 .. + 16; A stays in registers as the A operand of A T, high and low half
+  uint32_t ah[4][4], al[4][4];
   {
     uint32_t kf[DK / 16][4], qf[DK / 16][4];
 #pragma unroll
@@ -148,7 +153,7 @@ delta_rule_prepare_kernel(const RbDeltaRuleArgs a) {
             Lm[t * LP + s + j] = s + j < t ? beta[t] * rk[t] * d * kk[i][2 * r + j] : 0.f;
             v[j] = rq[t] * d * qk[i][2 * r + j];
           }
-          *reinterpret_cast<uint32_t*>(outA + t * kDcChunk + s) = pack_bf16x2(v[0], v[1]);
+          wm_split(v[0], v[1], ah[sb][2 * i + r], al[sb][2 * i + r]);
         }
     }
   }
@@ -187,22 +192,99 @@ delta_rule_prepare_kernel(const RbDeltaRuleArgs a) {
     }
     __syncthreads();
   }
+  const uint32_t sT = smem_u32(dp_smem) + L::kL;
+  constexpr int TP = L::kTPitch;
   for (int e = tid; e < kDcChunk * kDcChunk / 8; e += 128) {
     const int r = e >> 3, c = (e & 7) * 8;
     uint32_t hi[4], lo[4];
 #pragma unroll
     for (int k = 0; k < 4; ++k) wm_split(T[r * LP + c + 2 * k], T[r * LP + c + 2 * k + 1], hi[k], lo[k]);
-    *reinterpret_cast<uint4*>(scratch + (r * kDcChunk + c) * 2) = make_uint4(hi[0], hi[1], hi[2], hi[3]);
-    *reinterpret_cast<uint4*>(scratch + kDcMat + (r * kDcChunk + c) * 2) = make_uint4(lo[0], lo[1], lo[2], lo[3]);
+    *reinterpret_cast<uint4*>(dp_smem + L::kL + (r * TP + c) * 2) = make_uint4(hi[0], hi[1], hi[2], hi[3]);
+    *reinterpret_cast<uint4*>(dp_smem + L::kL + ((kDcChunk + r) * TP + c) * 2) = make_uint4(lo[0], lo[1], lo[2], lo[3]);
+  }
+  __syncthreads();
+  // ---- A T: rows warp 16 .. + 16
+  {
+    __nv_bfloat16* out = reinterpret_cast<__nv_bfloat16*>(scratch);
+#pragma unroll
+    for (int nb = 0; nb < 4; ++nb) {
+      float acc[2][4];
+#pragma unroll
+      for (int i = 0; i < 2; ++i) acc[i][0] = acc[i][1] = acc[i][2] = acc[i][3] = 0.f;
+#pragma unroll
+      for (int k = 0; k < 4; ++k) {
+        if (k < nb || k > warp) continue;          // both are lower triangular
+        uint32_t b[4], bl[4];
+        wm_ldsm_x4_t(wm_b_t(sT, TP, nb * 16, k * 16, lane), b);
+        wm_ldsm_x4_t(wm_b_t(sT + kDcChunk * TP * 2, TP, nb * 16, k * 16, lane), bl);
+        wm_mma(acc[0], ah[k], b[0], b[1]);
+        wm_mma(acc[1], ah[k], b[2], b[3]);
+        wm_mma(acc[0], al[k], b[0], b[1]);
+        wm_mma(acc[1], al[k], b[2], b[3]);
+        wm_mma(acc[0], ah[k], bl[0], bl[1]);
+        wm_mma(acc[1], ah[k], bl[2], bl[3]);
+      }
+#pragma unroll
+      for (int i = 0; i < 2; ++i)
+#pragma unroll
+        for (int r = 0; r < 2; ++r)
+          *reinterpret_cast<uint32_t*>(out + (warp * 16 + gq + 8 * r) * kDcChunk + nb * 16 + i * 8 + 2 * tq) =
+              pack_bf16x2(acc[i][2 * r], acc[i][2 * r + 1]);
+    }
+  }
+  // ---- W = T^T diag(1 / |k| exp(c_end - c)) K: rows (columns of T) warp 16 .. + 16
+  {
+    const float c_end = cum[kDcChunk - 1];
+    uint32_t th[4][4], tl[4][4];                   // scaled T^T as the A operand
+#pragma unroll
+    for (int k = 0; k < 4; ++k) {
+      if (k < warp) continue;                      // T is lower triangular
+#pragma unroll
+      for (int half = 0; half < 2; ++half) {       // columns k 16 + 8 half + 2 tq (+ 1)
+        const int t = k * 16 + half * 8 + 2 * tq;
+        const float w0 = rk[t] * wm_ex2(c_end - cum[t]), w1 = rk[t + 1] * wm_ex2(c_end - cum[t + 1]);
+#pragma unroll
+        for (int r = 0; r < 2; ++r) {
+          const int s = warp * 16 + gq + 8 * r;
+          wm_split(w0 * T[t * LP + s], w1 * T[(t + 1) * LP + s], th[k][2 * half + r], tl[k][2 * half + r]);
+        }
+      }
+    }
+    __nv_bfloat16* out = reinterpret_cast<__nv_bfloat16*>(scratch + kDcMat);
+#pragma unroll
+    for (int nb = 0; nb < DK / 16; ++nb) {
+      float acc[2][4];
+#pragma unroll
+      for (int i = 0; i < 2; ++i) acc[i][0] = acc[i][1] = acc[i][2] = acc[i][3] = 0.f;
+#pragma unroll
+      for (int k = 0; k < 4; ++k) {
+        if (k < warp) continue;
+        uint32_t b[4];
+        wm_ldsm_x4_t(wm_b_t(sK, P, nb * 16, k * 16, lane), b);
+        wm_mma(acc[0], th[k], b[0], b[1]);
+        wm_mma(acc[1], th[k], b[2], b[3]);
+        wm_mma(acc[0], tl[k], b[0], b[1]);
+        wm_mma(acc[1], tl[k], b[2], b[3]);
+      }
+#pragma unroll
+      for (int i = 0; i < 2; ++i)
+#pragma unroll
+        for (int r = 0; r < 2; ++r) {
+          uint32_t hi, lo;
+          wm_split(acc[i][2 * r], acc[i][2 * r + 1], hi, lo);
+          const int at = (warp * 16 + gq + 8 * r) * DK + nb * 16 + i * 8 + 2 * tq;
+          *reinterpret_cast<uint32_t*>(out + at) = hi;
+          *reinterpret_cast<uint32_t*>(out + kDcChunk * DK + at) = lo;
+        }
+    }
   }
   if (tid < kDcChunk) {
-    float* f = reinterpret_cast<float*>(scratch + 3 * kDcMat);
-    const float c = cum[tid], c_end = cum[kDcChunk - 1], e = wm_ex2(c);
+    float* f = reinterpret_cast<float*>(scratch + kDcMat + 2 * kDcChunk * DK * 2);
+    const float e = wm_ex2(cum[tid]);
     f[tid] = beta[tid];
     f[kDcChunk + tid] = rk[tid] * e;
     f[2 * kDcChunk + tid] = rq[tid] * e;
-    f[3 * kDcChunk + tid] = rk[tid] * wm_ex2(c_end - c);
-    f[4 * kDcChunk + tid] = wm_ex2(c_end);
+    f[3 * kDcChunk + tid] = wm_ex2(cum[kDcChunk - 1]);
   }
 }
 
@@ -210,18 +292,17 @@ delta_rule_prepare_kernel(const RbDeltaRuleArgs a) {
 template <int DK, int COLS>
 struct DcSmem {
   static constexpr int kPitch = DK + 8, kVPitch = COLS + 8, kMPitch = kDcChunk + 8;
-  // one stage: what a chunk reads
+  // one stage: what a chunk reads; the high half of R replaces V element by element
   static constexpr int kQ = 0;
   static constexpr int kK = kQ + kDcChunk * kPitch * 2;
   static constexpr int kV = kK + kDcChunk * kPitch * 2;
-  static constexpr int kM = kV + kDcChunk * kVPitch * 2;             // T high, T low, A
-  static constexpr int kF = kM + 3 * kDcChunk * kMPitch * 2;
+  static constexpr int kM = kV + kDcChunk * kVPitch * 2;             // A T
+  static constexpr int kW = kM + kDcChunk * kMPitch * 2;             // W, high and low half
+  static constexpr int kF = kW + 2 * kDcChunk * kPitch * 2;
   static constexpr int kStage = kF + kDcFactors * kDcChunk * 4;
   static constexpr int kS = 2 * kStage;                              // state, high and low half
-  static constexpr int kR = kS + 2 * DK * kVPitch * 2;               // R, high and low half
-  static constexpr int kU = kR + 2 * kDcChunk * kVPitch * 2;         // U (rounded)
-  static constexpr int kUs = kU + kDcChunk * kVPitch * 2;            // U scaled by what it adds to the state, high and low half
-  static constexpr int kTotal = kUs + 2 * kDcChunk * kVPitch * 2;
+  static constexpr int kR = kS + 2 * DK * kVPitch * 2;               // low half of R
+  static constexpr int kTotal = kR + kDcChunk * kVPitch * 2;
 };
 
 template <int DK, int COLS>
@@ -232,7 +313,7 @@ delta_rule_chunk_kernel(const RbDeltaRuleArgs a) {
   constexpr int MT = DK / 64, NJ = COLS / 32;      // state: MT row tiles; columns of a warp: NJ pairs of n-tiles
   extern __shared__ __align__(16) uint8_t dc_smem[];
   const uint32_t base = smem_u32(dc_smem);
-  const uint32_t sS = base + L::kS, sR = base + L::kR, sU = base + L::kU, sUs = base + L::kUs;
+  const uint32_t sS = base + L::kS, sRl = base + L::kR;
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int gq = lane >> 2, tq = lane & 3;
   const int wc = warp >> 2, wr = wc ? 3 - (warp & 3) : (warp & 3);
@@ -264,12 +345,16 @@ delta_rule_chunk_kernel(const RbDeltaRuleArgs a) {
       const bool ok = r < m_rows && c0 + c < a.dv;
       wm_cp16(st + L::kV + (r * VP + c) * 2, ok ? rows + r * a.ld_qkv + offV + c : rows, ok);
     }
-    const uint8_t* scratch = reinterpret_cast<const uint8_t*>(a.scratch) + (static_cast<long long>(tile0 + ci) * a.heads + h) * kDcScratch;
-    for (int i = tid; i < 3 * kDcChunk * 8; i += 256) {
-      const int r = i >> 3, c = (i & 7) * 8;       // r: matrix * 64 + row
+    const uint8_t* scratch = reinterpret_cast<const uint8_t*>(a.scratch) + (static_cast<long long>(tile0 + ci) * a.heads + h) * dc_scratch(DK);
+    for (int i = tid; i < kDcChunk * 8; i += 256) {
+      const int r = i >> 3, c = (i & 7) * 8;
       wm_cp16(st + L::kM + (r * MP + c) * 2, scratch + (r * kDcChunk + c) * 2, true);
     }
-    if (tid < kDcFactors * kDcChunk / 4) wm_cp16(st + L::kF + tid * 16, scratch + 3 * kDcMat + tid * 16, true);
+    for (int i = tid; i < 2 * kDcChunk * (DK / 8); i += 256) {
+      const int r = i / (DK / 8), c = (i - r * (DK / 8)) * 8;         // r: half * 64 + row
+      wm_cp16(st + L::kW + (r * P + c) * 2, scratch + kDcMat + (r * DK + c) * 2, true);
+    }
+    if (tid < kDcFactors * kDcChunk / 4) wm_cp16(st + L::kF + tid * 16, scratch + kDcMat + 2 * kDcChunk * DK * 2 + tid * 16, true);
     wm_cp_commit();
   };
   request(0);
@@ -339,105 +424,66 @@ delta_rule_chunk_kernel(const RbDeltaRuleArgs a) {
       }
     }
     // ---- R
-    const __nv_bfloat16* V = reinterpret_cast<const __nv_bfloat16*>(stp + L::kV);
+    uint8_t* V = dc_smem + (ci & 1) * L::kStage + L::kV;
 #pragma unroll
     for (int r = 0; r < 2; ++r) {
       const int t = r ? r1 : r0;
       const float be = f[t], kd = f[kDcChunk + t];
 #pragma unroll
       for (int j = 0; j < 2 * NJ; ++j) {
-        const float2 v = unpack_bf16x2(*reinterpret_cast<const uint32_t*>(V + t * VP + v_base + 8 * j));
+        const int at = (t * VP + v_base + 8 * j) * 2;
+        const float2 v = unpack_bf16x2(*reinterpret_cast<const uint32_t*>(V + at));
         uint32_t hi, lo;
         wm_split(be * (v.x - kd * pm[j][2 * r]), be * (v.y - kd * pm[j][2 * r + 1]), hi, lo);
-        const int at = (t * VP + v_base + 8 * j) * 2;
-        *reinterpret_cast<uint32_t*>(dc_smem + L::kR + at) = hi;
-        *reinterpret_cast<uint32_t*>(dc_smem + L::kR + kDcChunk * VP * 2 + at) = lo;
+        *reinterpret_cast<uint32_t*>(V + at) = hi;
+        *reinterpret_cast<uint32_t*>(dc_smem + L::kR + at) = lo;
       }
     }
     __syncthreads();
-    // ---- U = T R
-    float u[2 * NJ][4];
-#pragma unroll
-    for (int j = 0; j < 2 * NJ; ++j) u[j][0] = u[j][1] = u[j][2] = u[j][3] = 0.f;
-#pragma unroll
-    for (int k = 0; k < 4; ++k) {
-      if (k > wr) break;
-      uint32_t th[4], tl[4];
-      wm_ldsm_x4(wm_a(st + L::kM, MP, wr * 16, k * 16, lane), th);
-      wm_ldsm_x4(wm_a(st + L::kM + kDcChunk * MP * 2, MP, wr * 16, k * 16, lane), tl);
-#pragma unroll
-      for (int j = 0; j < NJ; ++j) {
-        uint32_t b[4], bl[4];
-        wm_ldsm_x4_t(wm_b_t(sR, VP, wc * (COLS / 2) + j * 16, k * 16, lane), b);
-        wm_ldsm_x4_t(wm_b_t(sR + kDcChunk * VP * 2, VP, wc * (COLS / 2) + j * 16, k * 16, lane), bl);
-        wm_mma(u[2 * j], th, b[0], b[1]);
-        wm_mma(u[2 * j + 1], th, b[2], b[3]);
-        wm_mma(u[2 * j], tl, b[0], b[1]);
-        wm_mma(u[2 * j + 1], tl, b[2], b[3]);
-        wm_mma(u[2 * j], th, bl[0], bl[1]);
-        wm_mma(u[2 * j + 1], th, bl[2], bl[3]);
-      }
-    }
-#pragma unroll
-    for (int r = 0; r < 2; ++r) {
-      const int t = r ? r1 : r0;
-      const float ks = f[3 * kDcChunk + t];
-#pragma unroll
-      for (int j = 0; j < 2 * NJ; ++j) {
-        const int at = (t * VP + v_base + 8 * j) * 2;
-        uint32_t hi, lo;
-        wm_split(ks * u[j][2 * r], ks * u[j][2 * r + 1], hi, lo);
-        *reinterpret_cast<uint32_t*>(dc_smem + L::kU + at) = pack_bf16x2(u[j][2 * r], u[j][2 * r + 1]);
-        *reinterpret_cast<uint32_t*>(dc_smem + L::kUs + at) = hi;
-        *reinterpret_cast<uint32_t*>(dc_smem + L::kUs + kDcChunk * VP * 2 + at) = lo;
-      }
-    }
-    __syncthreads();
+    const uint32_t sRh = st + L::kV;
     // ---- state behind the chunk
-    const float e_end = f[4 * kDcChunk];
+    const float e_end = f[3 * kDcChunk];
 #pragma unroll
     for (int m = 0; m < MT; ++m)
 #pragma unroll
       for (int j = 0; j < 2 * NJ; ++j)
 #pragma unroll
         for (int i = 0; i < 4; ++i) S[m][j][i] *= e_end;
-#pragma unroll
-    for (int k = 0; k < 4; ++k) {
-      uint32_t af[MT][4];
-#pragma unroll
-      for (int m = 0; m < MT; ++m) wm_ldsm_x4_t(wm_a_t(st + L::kK, P, wr * (DK / 4) + m * 16, k * 16, lane), af[m]);
-#pragma unroll
-      for (int j = 0; j < NJ; ++j) {
-        uint32_t b[4], bl[4];
-        wm_ldsm_x4_t(wm_b_t(sUs, VP, wc * (COLS / 2) + j * 16, k * 16, lane), b);
-        wm_ldsm_x4_t(wm_b_t(sUs + kDcChunk * VP * 2, VP, wc * (COLS / 2) + j * 16, k * 16, lane), bl);
-#pragma unroll
-        for (int m = 0; m < MT; ++m) {
-          wm_mma(S[m][2 * j], af[m], b[0], b[1]);
-          wm_mma(S[m][2 * j + 1], af[m], b[2], b[3]);
-          wm_mma(S[m][2 * j], af[m], bl[0], bl[1]);
-          wm_mma(S[m][2 * j + 1], af[m], bl[2], bl[3]);
-        }
-      }
-    }
-    publish();                                     // every warp has read the old one
-    // ---- o = exp(c) S0^T q + A U
     const float q0 = f[2 * kDcChunk + r0], q1 = f[2 * kDcChunk + r1];
 #pragma unroll
     for (int j = 0; j < 2 * NJ; ++j) { y[j][0] *= q0; y[j][1] *= q0; y[j][2] *= q1; y[j][3] *= q1; }
 #pragma unroll
     for (int k = 0; k < 4; ++k) {
-      if (k > wr) break;
-      uint32_t af[4];
-      wm_ldsm_x4(wm_a(st + L::kM + 2 * kDcChunk * MP * 2, MP, wr * 16, k * 16, lane), af);
+      uint32_t wh[MT][4], wl[MT][4], af[4];
+#pragma unroll
+      for (int m = 0; m < MT; ++m) {
+        wm_ldsm_x4_t(wm_a_t(st + L::kW, P, wr * (DK / 4) + m * 16, k * 16, lane), wh[m]);
+        wm_ldsm_x4_t(wm_a_t(st + L::kW + kDcChunk * P * 2, P, wr * (DK / 4) + m * 16, k * 16, lane), wl[m]);
+      }
+      if (k <= wr) wm_ldsm_x4(wm_a(st + L::kM, MP, wr * 16, k * 16, lane), af);
 #pragma unroll
       for (int j = 0; j < NJ; ++j) {
-        uint32_t b[4];
-        wm_ldsm_x4_t(wm_b_t(sU, VP, wc * (COLS / 2) + j * 16, k * 16, lane), b);
-        wm_mma(y[2 * j], af, b[0], b[1]);
-        wm_mma(y[2 * j + 1], af, b[2], b[3]);
+        uint32_t b[4], bl[4];
+        wm_ldsm_x4_t(wm_b_t(sRh, VP, wc * (COLS / 2) + j * 16, k * 16, lane), b);
+        wm_ldsm_x4_t(wm_b_t(sRl, VP, wc * (COLS / 2) + j * 16, k * 16, lane), bl);
+#pragma unroll
+        for (int m = 0; m < MT; ++m) {
+          wm_mma(S[m][2 * j], wh[m], b[0], b[1]);
+          wm_mma(S[m][2 * j + 1], wh[m], b[2], b[3]);
+          wm_mma(S[m][2 * j], wl[m], b[0], b[1]);
+          wm_mma(S[m][2 * j + 1], wl[m], b[2], b[3]);
+          wm_mma(S[m][2 * j], wh[m], bl[0], bl[1]);
+          wm_mma(S[m][2 * j + 1], wh[m], bl[2], bl[3]);
+        }
+        if (k <= wr) {                             // o = exp(c) S0^T q + (A T) R
+          wm_mma(y[2 * j], af, b[0], b[1]);
+          wm_mma(y[2 * j + 1], af, b[2], b[3]);
+          wm_mma(y[2 * j], af, bl[0], bl[1]);
+          wm_mma(y[2 * j + 1], af, bl[2], bl[3]);
+        }
       }
     }
+    publish();                                     // every warp has read the old one
     const int t0 = ci * kDcChunk;
     __nv_bfloat16* out = reinterpret_cast<__nv_bfloat16*>(a.o) + static_cast<long long>(seg.first + t0) * a.ld_o + static_cast<long long>(h) * a.dv + c0;
 #pragma unroll
@@ -497,8 +543,8 @@ int dc_launch(const RbDeltaRuleArgs& a, cudaStream_t s) {
 
 }  // namespace rb
 
-RB_API long long rb_delta_rule_scratch_bytes(int num_tiles, int heads) {
-  return static_cast<long long>(num_tiles) * heads * rb::kDcScratch;
+RB_API long long rb_delta_rule_scratch_bytes(int num_tiles, int heads, int dk) {
+  return static_cast<long long>(num_tiles) * heads * rb::dc_scratch(dk <= 64 ? 64 : 128);
 }
 
 RB_API int rb_delta_rule_chunked(const RbDeltaRuleArgs* args, void* stream_v) {

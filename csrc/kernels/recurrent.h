@@ -68,8 +68,8 @@ typedef struct RbDeltaRuleArgs {
 } RbDeltaRuleArgs;
 int rb_delta_rule_scan(const RbDeltaRuleArgs* args, void* stream);
 // The same for prompts on the tensor cores: bf16, dk <= 128, dk and dv multiples of 8 (-9 otherwise).  `tiles` lists pieces of 64
-// rows, in order, every one listed; scratch: rb_delta_rule_scratch_bytes(num_tiles, heads) bytes.
-long long rb_delta_rule_scratch_bytes(int num_tiles, int heads);
+// rows, in order, every one listed; scratch: rb_delta_rule_scratch_bytes(num_tiles, heads, dk) bytes.
+long long rb_delta_rule_scratch_bytes(int num_tiles, int heads, int dk);
 int rb_delta_rule_chunked(const RbDeltaRuleArgs* args, void* stream);
 
 // Every row of y consists of `parts` equal parts.  gate_first: u = y silu(z), out = u / rms(u) * weight; else:

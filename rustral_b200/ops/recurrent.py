@@ -20,7 +20,7 @@ N.optional_sig("rb_delta_rule_scan", [N.C.POINTER(N.RbDeltaRuleArgs), N.c_void_p
 N.optional_sig("rb_gated_norm", [N.C.POINTER(N.RbGatedNormArgs), N.c_void_p])
 N.optional_sig("rb_state_space_chunked", [N.C.POINTER(N.RbStateSpaceArgs), N.c_void_p, N.c_void_p, N.c_int, N.c_void_p])
 N.optional_sig("rb_delta_rule_chunked", [N.C.POINTER(N.RbDeltaRuleArgs), N.c_void_p])
-N.optional_sig("rb_delta_rule_scratch_bytes", [N.c_int, N.c_int], N.c_ll)
+N.optional_sig("rb_delta_rule_scratch_bytes", [N.c_int, N.c_int, N.c_int], N.c_ll)
 N._LAUNCHES["rb_delta_rule_chunked"] = 2
 
 CHUNK = 64                                            # tokens per step of the chunked kernels
@@ -227,7 +227,7 @@ def delta_rule(qkv, a_raw, b_raw, *, dt_bias, a_log, state, heads: int, kv_heads
         N.check(lib.rb_delta_rule_scan(a, N.stream_ptr()), "rb_delta_rule_scan")
     if many is not None:
         tiles = many.tiles(CHUNK)
-        scratch = torch.empty(lib.rb_delta_rule_scratch_bytes(tiles.shape[0], heads), dtype=torch.uint8, device=qkv.device)
+        scratch = torch.empty(lib.rb_delta_rule_scratch_bytes(tiles.shape[0], heads, dk), dtype=torch.uint8, device=qkv.device)
         a.segments, a.num_segments, a.tiles, a.num_tiles = many.table.data_ptr(), many.n, tiles.data_ptr(), tiles.shape[0]
         a.scratch = scratch.data_ptr()
         N.check(lib.rb_delta_rule_chunked(a, N.stream_ptr()), "rb_delta_rule_chunked")
