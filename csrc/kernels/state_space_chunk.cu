@@ -25,12 +25,12 @@ template <int N>
 struct ScSmem {
   static constexpr int kPitch = N + 8, kXPitch = kScCols + 8;
   static constexpr int kC = 0;
-  static constexpr int kB = kC + kScChunk * kPitch * 2;
-  static constexpr int kX = kB + kScChunk * kPitch * 2;
+  static constexpr int kB = kC + kScChunk * kPitch * 2;             // two buffers
+  static constexpr int kX = kB + 2 * kScChunk * kPitch * 2;
   static constexpr int kXs = kX + kScChunk * kXPitch * 2;           // scaled x: high half, low half
   static constexpr int kS = kXs + 2 * kScChunk * kXPitch * 2;
-  static constexpr int kCum = kS + N * kXPitch * 2;                  // fp32 [64] cumulative log2 decay, then [64] step sizes
-  static constexpr int kTotal = kCum + 2 * kScChunk * 4;
+  static constexpr int kCum = kS + N * kXPitch * 2;                  // two buffers: fp32 [64] running log2 decays, [64] step sizes
+  static constexpr int kTotal = kCum + 4 * kScChunk * 4;
 };
 
 template <int N, bool STATE_ONLY>
@@ -41,9 +41,7 @@ state_space_chunk_kernel(const RbStateSpaceArgs a, float* __restrict__ span_stat
   constexpr int NP = L::kPitch, XP = L::kXPitch;
   extern __shared__ __align__(16) uint8_t sc_smem[];
   const uint32_t base = smem_u32(sc_smem);
-  const uint32_t sC = base + L::kC, sB = base + L::kB, sX = base + L::kX, sXs = base + L::kXs, sS = base + L::kS;
-  float* cum = reinterpret_cast<float*>(sc_smem + L::kCum);
-  float* dts = cum + kScChunk;
+  const uint32_t sC = base + L::kC, sX = base + L::kX, sXs = base + L::kXs, sS = base + L::kS;
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int gq = lane >> 2, tq = lane & 3;
   const int wc = warp >> 2, wr = wc ? 3 - (warp & 3) : (warp & 3);   // the causal work of a scheduler's two warps adds up evenly
@@ -97,55 +95,96 @@ state_space_chunk_kernel(const RbStateSpaceArgs a, float* __restrict__ span_stat
   }
   float total = 0.f;
 
-  for (int t0 = off; t0 < end; t0 += kScChunk) {
+  // Tiles of a chunk (rows past the end and columns past the real sizes are zero).  B has two buffers; C and x are free again
+  // behind the second barrier of a chunk, so the next chunk's are requested there and arrive under the state's products.
+  auto request_b = [&](int t0) {
     const int m_rows = min(kScChunk, end - t0);
     const __nv_bfloat16* rows = xbc + static_cast<long long>(seg.first + t0) * a.ld_xbc;
-    // ---- tiles of this chunk (rows past the end and columns past the real sizes are zero)
+    const uint32_t dst = base + L::kB + ((t0 - off) / kScChunk & 1) * kScChunk * NP * 2;
     for (int i = tid; i < kScChunk * (N / 8); i += kScThreads) {
       const int r = i / (N / 8), c = (i - r * (N / 8)) * 8;
       const bool ok = r < m_rows && c < a.n;
-      const __nv_bfloat16* src = rows + (ok ? r * a.ld_xbc + c : 0);
-      wm_cp16(sB + (r * NP + c) * 2, ok ? src + offB : rows, ok);
-      if (!STATE_ONLY) wm_cp16(sC + (r * NP + c) * 2, ok ? src + offC : rows, ok);
+      wm_cp16(dst + (r * NP + c) * 2, ok ? rows + r * a.ld_xbc + offB + c : rows, ok);
+    }
+  };
+  auto request_cx = [&](int t0) {
+    const int m_rows = min(kScChunk, end - t0);
+    const __nv_bfloat16* rows = xbc + static_cast<long long>(seg.first + t0) * a.ld_xbc;
+    if (!STATE_ONLY) {
+      for (int i = tid; i < kScChunk * (N / 8); i += kScThreads) {
+        const int r = i / (N / 8), c = (i - r * (N / 8)) * 8;
+        const bool ok = r < m_rows && c < a.n;
+        wm_cp16(sC + (r * NP + c) * 2, ok ? rows + r * a.ld_xbc + offC + c : rows, ok);
+      }
     }
     for (int i = tid; i < kScChunk * (kScCols / 8); i += kScThreads) {
       const int r = i / (kScCols / 8), c = (i - r * (kScCols / 8)) * 8;
       const bool ok = r < m_rows && c0 + c < a.p;
       wm_cp16(sX + (r * XP + c) * 2, ok ? rows + r * a.ld_xbc + offX + c : rows, ok);
     }
-    wm_cp_commit();
-    if (warp == 0) {                               // step sizes and running log2 decays, two tokens per lane
-      float d[2], s[2];
+  };
+  // Step sizes and running log2 decays by warp 0, two tokens per lane; the raw values are fetched one chunk earlier still.
+  float raw[2] = {0.f, 0.f};
+  auto fetch_dt = [&](int t0) {
 #pragma unroll
-      for (int i = 0; i < 2; ++i) {
-        const int t = 2 * lane + i;
-        d[i] = t < m_rows ? rc_softplus(a.dt_raw[static_cast<long long>(seg.first + t0 + t) * a.ld_dt + h] + dt_bias) : 0.f;
-        s[i] = -rate2 * d[i];
-      }
-      float run = s[0] + s[1];
-#pragma unroll
-      for (int o = 1; o < 32; o <<= 1) {
-        const float u = __shfl_up_sync(0xffffffffu, run, o);
-        if (lane >= o) run += u;
-      }
-      cum[2 * lane] = run - s[1];
-      cum[2 * lane + 1] = run;
-      dts[2 * lane] = d[0];
-      dts[2 * lane + 1] = d[1];
+    for (int i = 0; i < 2; ++i) {
+      const int t = t0 + 2 * lane + i;
+      if (t < end) raw[i] = a.dt_raw[static_cast<long long>(seg.first + t) * a.ld_dt + h];
     }
-    // ---- bf16 copy of the state in front of the chunk
-    if (!STATE_ONLY) {
+  };
+  auto scan_dt = [&](int t0) {
+    float* cum = reinterpret_cast<float*>(sc_smem + L::kCum) + ((t0 - off) / kScChunk & 1) * 2 * kScChunk;
+    float d[2], s[2];
 #pragma unroll
-      for (int m = 0; m < MT; ++m)
-#pragma unroll
-        for (int j = 0; j < 4; ++j)
-#pragma unroll
-          for (int r = 0; r < 2; ++r)
-            *reinterpret_cast<uint32_t*>(sc_smem + L::kS + ((n_base + 16 * m + 8 * r) * XP + p_base + 8 * j) * 2) =
-                pack_bf16x2(S[m][j][2 * r], S[m][j][2 * r + 1]);
+    for (int i = 0; i < 2; ++i) {
+      d[i] = t0 + 2 * lane + i < end ? rc_softplus(raw[i] + dt_bias) : 0.f;
+      s[i] = -rate2 * d[i];
     }
+    float run = s[0] + s[1];
+#pragma unroll
+    for (int o = 1; o < 32; o <<= 1) {
+      const float u = __shfl_up_sync(0xffffffffu, run, o);
+      if (lane >= o) run += u;
+    }
+    cum[2 * lane] = run - s[1];
+    cum[2 * lane + 1] = run;
+    cum[kScChunk + 2 * lane] = d[0];
+    cum[kScChunk + 2 * lane + 1] = d[1];
+  };
+  auto publish = [&]() {                           // bf16 copy of the state for the read-out
+#pragma unroll
+    for (int m = 0; m < MT; ++m)
+#pragma unroll
+      for (int j = 0; j < 4; ++j)
+#pragma unroll
+        for (int r = 0; r < 2; ++r)
+          *reinterpret_cast<uint32_t*>(sc_smem + L::kS + ((n_base + 16 * m + 8 * r) * XP + p_base + 8 * j) * 2) =
+              pack_bf16x2(S[m][j][2 * r], S[m][j][2 * r + 1]);
+  };
+  request_b(off);
+  request_cx(off);
+  wm_cp_commit();
+  if (warp == 0) {
+    fetch_dt(off);
+    scan_dt(off);
+    fetch_dt(off + kScChunk);
+  }
+  if (!STATE_ONLY) publish();
+
+  for (int t0 = off; t0 < end; t0 += kScChunk) {
+    const int m_rows = min(kScChunk, end - t0);
+    const int par = (t0 - off) / kScChunk & 1;
+    const uint32_t sB = base + L::kB + par * kScChunk * NP * 2;
+    const float* cum = reinterpret_cast<const float*>(sc_smem + L::kCum) + par * 2 * kScChunk;
+    const float* dts = cum + kScChunk;
+    const bool more = t0 + kScChunk < end;
     wm_cp_wait<0>();
-    __syncthreads();
+    __syncthreads();                               // tiles, step sizes and the state in front of the chunk have arrived
+    if (more) request_b(t0 + kScChunk);
+    if (warp == 0 && more) {
+      scan_dt(t0 + kScChunk);
+      fetch_dt(t0 + 2 * kScChunk);
+    }
     const float c_end = cum[kScChunk - 1];
     // ---- x scaled by what it adds to the state
     for (int i = tid; i < kScChunk * (kScCols / 8); i += kScThreads) {
@@ -231,7 +270,9 @@ state_space_chunk_kernel(const RbStateSpaceArgs a, float* __restrict__ span_stat
         }
       }
     }
-    __syncthreads();                               // the scaled x is complete
+    __syncthreads();                               // the scaled x is complete; C, x and the copy of the state are free
+    if (more) request_cx(t0 + kScChunk);
+    wm_cp_commit();
     // ---- state behind the chunk
     const float e_end = wm_ex2(c_end);
     total += c_end;
@@ -259,7 +300,7 @@ state_space_chunk_kernel(const RbStateSpaceArgs a, float* __restrict__ span_stat
           }
         }
     }
-    __syncthreads();                               // every warp is done with the tiles
+    if (!STATE_ONLY) publish();
   }
   if (STATE_ONLY) {
     float* dst = span_state + (static_cast<long long>(tile) * a.heads + h) * state_n;
