@@ -42,7 +42,8 @@ struct DcPrepSmem {
   static constexpr int kT = kL + 2 * kDcChunk * kTPitch * 2;         // fp32 [64][68]
   static constexpr int kW = kT + kDcChunk * kLPitch * 4;             // fp32 [48][20] products of blocks
   static constexpr int kF = kW + 48 * 20 * 4;                        // fp32 [4][64]: c, beta, 1 / |k|, scale / |q|
-  static constexpr int kTotal = kF + 4 * kDcChunk * 4;
+  static constexpr int kW2 = kF + 4 * kDcChunk * 4;                  // staging of W's low half
+  static constexpr int kTotal = kW2 + kDcChunk * kPitch * 2;
 };
 
 template <int DK>
@@ -164,31 +165,49 @@ delta_rule_prepare_kernel(const RbDeltaRuleArgs a) {
     float x[16];
 #pragma unroll
     for (int t = 0; t < 16; ++t) {
-      float v = t == j ? 1.f : 0.f;
+      const float4* row = reinterpret_cast<const float4*>(Lm + (b0 + t) * LP + b0);
+      float v0 = t == j ? 1.f : 0.f, v1 = 0.f;
 #pragma unroll
-      for (int s = 0; s < t; ++s) v = fmaf(-Lm[(b0 + t) * LP + b0 + s], x[s], v);
-      x[t] = v;                                    // zero above the diagonal
-      T[(b0 + t) * LP + b0 + j] = v;
+      for (int s = 0; s < t; s += 4) {
+        const float4 l = row[s / 4];
+        v0 = fmaf(-l.x, x[s], v0);
+        if (s + 1 < t) v1 = fmaf(-l.y, x[s + 1], v1);
+        if (s + 2 < t) v0 = fmaf(-l.z, x[s + 2], v0);
+        if (s + 3 < t) v1 = fmaf(-l.w, x[s + 3], v1);
+      }
+      x[t] = v0 + v1;                              // zero above the diagonal
+      T[(b0 + t) * LP + b0 + j] = x[t];
     }
   }
   __syncthreads();
   // ---- ... then the blocks below: T_ij = -T_ii sum_{j <= k < i} L_ik T_kj, one distance i - j after the other
+  auto dot16 = [&](const float* row, const float* colm, int pitch) {
+    float v0 = 0.f, v1 = 0.f;
+#pragma unroll
+    for (int k = 0; k < 16; k += 4) {
+      const float4 l = *reinterpret_cast<const float4*>(row + k);
+      v0 = fmaf(l.x, colm[k * pitch], v0);
+      v1 = fmaf(l.y, colm[(k + 1) * pitch], v1);
+      v0 = fmaf(l.z, colm[(k + 2) * pitch], v0);
+      v1 = fmaf(l.w, colm[(k + 3) * pitch], v1);
+    }
+    return v0 + v1;
+  };
 #pragma unroll
   for (int d = 1; d < 4; ++d) {
-    const int items = (4 - d) * 256;
-    for (int e = tid; e < items; e += 128) {
-      const int blk = e >> 8, r = (e >> 4) & 15, c = e & 15, i = blk + d;      // block row i, block column blk
+#pragma unroll
+    for (int e = 0; e < (4 - d) * 2; ++e) {        // 128 entries at a time
+      const int blk = e >> 1, r = (e & 1) * 8 + (tid >> 4), c = tid & 15, i = blk + d;      // block row i, block column blk
       float v = 0.f;
-      for (int k = blk * 16; k < i * 16; ++k) v = fmaf(Lm[(i * 16 + r) * LP + k], T[k * LP + blk * 16 + c], v);
+#pragma unroll
+      for (int k = 0; k < d; ++k) v += dot16(Lm + (i * 16 + r) * LP + (blk + k) * 16, T + (blk + k) * 16 * LP + blk * 16 + c, LP);
       W[(blk * 16 + r) * 20 + c] = v;
     }
     __syncthreads();
-    for (int e = tid; e < items; e += 128) {
-      const int blk = e >> 8, r = (e >> 4) & 15, c = e & 15, i = blk + d;
-      float v = 0.f;
 #pragma unroll
-      for (int k = 0; k < 16; ++k) v = fmaf(T[(i * 16 + r) * LP + i * 16 + k], W[(blk * 16 + k) * 20 + c], v);
-      T[(i * 16 + r) * LP + blk * 16 + c] = -v;
+    for (int e = 0; e < (4 - d) * 2; ++e) {
+      const int blk = e >> 1, r = (e & 1) * 8 + (tid >> 4), c = tid & 15, i = blk + d;
+      T[(i * 16 + r) * LP + blk * 16 + c] = -dot16(T + (i * 16 + r) * LP + i * 16, W + blk * 16 * 20 + c, 20);
     }
     __syncthreads();
   }
@@ -272,10 +291,16 @@ delta_rule_prepare_kernel(const RbDeltaRuleArgs a) {
         for (int r = 0; r < 2; ++r) {
           uint32_t hi, lo;
           wm_split(acc[i][2 * r], acc[i][2 * r + 1], hi, lo);
-          const int at = (warp * 16 + gq + 8 * r) * DK + nb * 16 + i * 8 + 2 * tq;
-          *reinterpret_cast<uint32_t*>(out + at) = hi;
-          *reinterpret_cast<uint32_t*>(out + kDcChunk * DK + at) = lo;
+          const int at = ((warp * 16 + gq + 8 * r) * P + nb * 16 + i * 8 + 2 * tq) * 2;
+          *reinterpret_cast<uint32_t*>(dp_smem + L::kQ + at) = hi;             // the queries' tile is free
+          *reinterpret_cast<uint32_t*>(dp_smem + L::kW2 + at) = lo;
         }
+    }
+    __syncwarp();                                  // every warp copies its own rows
+    for (int e = lane; e < 2 * 16 * (DK / 8); e += 32) {
+      const int half = e / (16 * (DK / 8)), q = e - half * 16 * (DK / 8), r = warp * 16 + q / (DK / 8), c = (q % (DK / 8)) * 8;
+      *reinterpret_cast<uint4*>(out + (half * kDcChunk + r) * DK + c) =
+          *reinterpret_cast<const uint4*>(dp_smem + (half ? L::kW2 : L::kQ) + (r * P + c) * 2);
     }
   }
   if (tid < kDcChunk) {

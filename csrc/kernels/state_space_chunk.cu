@@ -21,27 +21,28 @@ constexpr int kScCols = 64;
 constexpr int kScThreads = 256;
 constexpr float kScLog2e = 1.4426950408889634f;
 
-template <int N>
+template <int N, bool STATE_ONLY>
 struct ScSmem {
   static constexpr int kPitch = N + 8, kXPitch = kScCols + 8;
-  static constexpr int kC = 0;
-  static constexpr int kB = kC + kScChunk * kPitch * 2;             // two buffers
-  static constexpr int kX = kB + 2 * kScChunk * kPitch * 2;
-  static constexpr int kXs = kX + kScChunk * kXPitch * 2;           // scaled x: high half, low half
-  static constexpr int kS = kXs + 2 * kScChunk * kXPitch * 2;
-  static constexpr int kCum = kS + N * kXPitch * 2;                  // two buffers: fp32 [64] running log2 decays, [64] step sizes
-  static constexpr int kTotal = kCum + 4 * kScChunk * 4;
+  static constexpr int kB = 0;                                       // two buffers
+  static constexpr int kX = kB + 2 * kScChunk * kPitch * 2;          // two buffers
+  static constexpr int kXs = kX + 2 * kScChunk * kXPitch * 2;        // scaled x, permuted rows: high half, low half
+  static constexpr int kCum = kXs + 2 * kScChunk * kScCols * 2;      // two buffers: fp32 [64] running log2 decays, [64] step sizes
+  static constexpr int kC = kCum + 4 * kScChunk * 4;
+  static constexpr int kM = kC + (STATE_ONLY ? 0 : kScChunk * kPitch * 2);       // masked products C . B, permuted rows
+  static constexpr int kS = kM + (STATE_ONLY ? 0 : kScChunk * kScChunk * 2);     // bf16 copy of the state
+  static constexpr int kTotal = kS + (STATE_ONLY ? 0 : N * kXPitch * 2);
 };
 
 template <int N, bool STATE_ONLY>
-__global__ void __launch_bounds__(kScThreads, 2)
+__global__ void __launch_bounds__(kScThreads, STATE_ONLY ? 3 : 2)
 state_space_chunk_kernel(const RbStateSpaceArgs a, float* __restrict__ span_state, float* __restrict__ span_decay, int span) {
-  using L = ScSmem<N>;
+  using L = ScSmem<N, STATE_ONLY>;
   constexpr int MT = N / 64;                       // 16-row tiles of the state per warp
   constexpr int NP = L::kPitch, XP = L::kXPitch;
   extern __shared__ __align__(16) uint8_t sc_smem[];
   const uint32_t base = smem_u32(sc_smem);
-  const uint32_t sC = base + L::kC, sX = base + L::kX, sXs = base + L::kXs, sS = base + L::kS;
+  const uint32_t sC = base + L::kC, sXs = base + L::kXs, sM = base + L::kM, sS = base + L::kS;
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int gq = lane >> 2, tq = lane & 3;
   const int wc = warp >> 2, wr = wc ? 3 - (warp & 3) : (warp & 3);   // the causal work of a scheduler's two warps adds up evenly
@@ -95,9 +96,9 @@ state_space_chunk_kernel(const RbStateSpaceArgs a, float* __restrict__ span_stat
   }
   float total = 0.f;
 
-  // Tiles of a chunk (rows past the end and columns past the real sizes are zero).  B has two buffers; C and x are free again
-  // behind the second barrier of a chunk, so the next chunk's are requested there and arrive under the state's products.
-  auto request_b = [&](int t0) {
+  // Tiles of a chunk (rows past the end and columns past the real sizes are zero).  B and x have two buffers; C is free again
+  // behind the second barrier of a chunk, so the next chunk's is requested there and arrives under the state's products.
+  auto request_bx = [&](int t0) {
     const int m_rows = min(kScChunk, end - t0);
     const __nv_bfloat16* rows = xbc + static_cast<long long>(seg.first + t0) * a.ld_xbc;
     const uint32_t dst = base + L::kB + ((t0 - off) / kScChunk & 1) * kScChunk * NP * 2;
@@ -106,21 +107,21 @@ state_space_chunk_kernel(const RbStateSpaceArgs a, float* __restrict__ span_stat
       const bool ok = r < m_rows && c < a.n;
       wm_cp16(dst + (r * NP + c) * 2, ok ? rows + r * a.ld_xbc + offB + c : rows, ok);
     }
-  };
-  auto request_cx = [&](int t0) {
-    const int m_rows = min(kScChunk, end - t0);
-    const __nv_bfloat16* rows = xbc + static_cast<long long>(seg.first + t0) * a.ld_xbc;
-    if (!STATE_ONLY) {
-      for (int i = tid; i < kScChunk * (N / 8); i += kScThreads) {
-        const int r = i / (N / 8), c = (i - r * (N / 8)) * 8;
-        const bool ok = r < m_rows && c < a.n;
-        wm_cp16(sC + (r * NP + c) * 2, ok ? rows + r * a.ld_xbc + offC + c : rows, ok);
-      }
-    }
+    const uint32_t dst_x = base + L::kX + ((t0 - off) / kScChunk & 1) * kScChunk * XP * 2;
     for (int i = tid; i < kScChunk * (kScCols / 8); i += kScThreads) {
       const int r = i / (kScCols / 8), c = (i - r * (kScCols / 8)) * 8;
       const bool ok = r < m_rows && c0 + c < a.p;
-      wm_cp16(sX + (r * XP + c) * 2, ok ? rows + r * a.ld_xbc + offX + c : rows, ok);
+      wm_cp16(dst_x + (r * XP + c) * 2, ok ? rows + r * a.ld_xbc + offX + c : rows, ok);
+    }
+  };
+  auto request_c = [&](int t0) {
+    if (STATE_ONLY) return;
+    const int m_rows = min(kScChunk, end - t0);
+    const __nv_bfloat16* rows = xbc + static_cast<long long>(seg.first + t0) * a.ld_xbc;
+    for (int i = tid; i < kScChunk * (N / 8); i += kScThreads) {
+      const int r = i / (N / 8), c = (i - r * (N / 8)) * 8;
+      const bool ok = r < m_rows && c < a.n;
+      wm_cp16(sC + (r * NP + c) * 2, ok ? rows + r * a.ld_xbc + offC + c : rows, ok);
     }
   };
   // Step sizes and running log2 decays by warp 0, two tokens per lane; the raw values are fetched one chunk earlier still.
@@ -161,8 +162,8 @@ state_space_chunk_kernel(const RbStateSpaceArgs a, float* __restrict__ span_stat
           *reinterpret_cast<uint32_t*>(sc_smem + L::kS + ((n_base + 16 * m + 8 * r) * XP + p_base + 8 * j) * 2) =
               pack_bf16x2(S[m][j][2 * r], S[m][j][2 * r + 1]);
   };
-  request_b(off);
-  request_cx(off);
+  request_bx(off);
+  request_c(off);
   wm_cp_commit();
   if (warp == 0) {
     fetch_dt(off);
@@ -174,13 +175,14 @@ state_space_chunk_kernel(const RbStateSpaceArgs a, float* __restrict__ span_stat
   for (int t0 = off; t0 < end; t0 += kScChunk) {
     const int m_rows = min(kScChunk, end - t0);
     const int par = (t0 - off) / kScChunk & 1;
-    const uint32_t sB = base + L::kB + par * kScChunk * NP * 2;
+    const uint32_t sB = base + L::kB + par * kScChunk * NP * 2, sX = base + L::kX + par * kScChunk * XP * 2;
+    const __nv_bfloat16* xs = reinterpret_cast<const __nv_bfloat16*>(sc_smem + L::kX) + par * kScChunk * XP;
     const float* cum = reinterpret_cast<const float*>(sc_smem + L::kCum) + par * 2 * kScChunk;
     const float* dts = cum + kScChunk;
     const bool more = t0 + kScChunk < end;
     wm_cp_wait<0>();
     __syncthreads();                               // tiles, step sizes and the state in front of the chunk have arrived
-    if (more) request_b(t0 + kScChunk);
+    if (more) request_bx(t0 + kScChunk);
     if (warp == 0 && more) {
       scan_dt(t0 + kScChunk);
       fetch_dt(t0 + 2 * kScChunk);
@@ -191,60 +193,89 @@ state_space_chunk_kernel(const RbStateSpaceArgs a, float* __restrict__ span_stat
       const int r = i / (kScCols / 8), c = (i - r * (kScCols / 8)) * 8;
       const float w = dts[r] * wm_ex2(c_end - cum[r]);
       float v[8];
-      RcVec<__nv_bfloat16, 8>::load(reinterpret_cast<const __nv_bfloat16*>(sc_smem + L::kX) + r * XP + c, v);
+      RcVec<__nv_bfloat16, 8>::load(xs + r * XP + c, v);
       uint32_t hi[4], lo[4];
 #pragma unroll
       for (int k = 0; k < 4; ++k) wm_split(w * v[2 * k], w * v[2 * k + 1], hi[k], lo[k]);
-      *reinterpret_cast<uint4*>(sc_smem + L::kXs + (r * XP + c) * 2) = make_uint4(hi[0], hi[1], hi[2], hi[3]);
-      *reinterpret_cast<uint4*>(sc_smem + L::kXs + ((kScChunk + r) * XP + c) * 2) = make_uint4(lo[0], lo[1], lo[2], lo[3]);
+      *reinterpret_cast<uint4*>(sc_smem + L::kXs + wm_swz(r, c >> 3)) = make_uint4(hi[0], hi[1], hi[2], hi[3]);
+      *reinterpret_cast<uint4*>(sc_smem + L::kXs + kScChunk * 128 + wm_swz(r, c >> 3)) = make_uint4(lo[0], lo[1], lo[2], lo[3]);
     }
+    float y[4][4];                                 // y of rows wr 16 .. + 16, columns wc 32 .. + 32
+    const int r0 = wr * 16 + gq, r1 = r0 + 8;
     if (!STATE_ONLY) {
-      // ---- y of rows wr 16 .. + 16, columns wc 32 .. + 32
-      float y[4][4];
+      // ---- C S0, and one or two of the ten blocks (16 x 16) of C B^T on and below the diagonal: those of the warp's own rows in
+      // the same loop, the three that are left by the warps of the first rows, which have the least to do behind the barrier
+      const int own = wr > 0 ? wr - wc : (wc == 0 ? 0 : -1);
 #pragma unroll
       for (int j = 0; j < 4; ++j) y[j][0] = y[j][1] = y[j][2] = y[j][3] = 0.f;
-      uint32_t cf[N / 16][4];
-#pragma unroll
-      for (int k = 0; k < N / 16; ++k) {
-        wm_ldsm_x4(wm_a(sC, NP, wr * 16, k * 16, lane), cf[k]);
-#pragma unroll
-        for (int j = 0; j < 2; ++j) {
-          uint32_t b[4];
-          wm_ldsm_x4_t(wm_b_t(sS, XP, wc * 32 + j * 16, k * 16, lane), b);
-          wm_mma(y[2 * j], cf[k], b[0], b[1]);
-          wm_mma(y[2 * j + 1], cf[k], b[2], b[3]);
-        }
-      }
-      const int r0 = wr * 16 + gq, r1 = r0 + 8;
-      const float ct0 = cum[r0], ct1 = cum[r1];
-      const float e0 = wm_ex2(ct0), e1 = wm_ex2(ct1);
-#pragma unroll
-      for (int j = 0; j < 4; ++j) { y[j][0] *= e0; y[j][1] *= e0; y[j][2] *= e1; y[j][3] *= e1; }
-#pragma unroll
-      for (int sb = 0; sb < 4; ++sb) {             // 16 earlier tokens at a time
-        if (sb > wr) break;
-        float gacc[2][4];
+      float gacc[2][4];
+      auto clear = [&]() {
 #pragma unroll
         for (int i = 0; i < 2; ++i) gacc[i][0] = gacc[i][1] = gacc[i][2] = gacc[i][3] = 0.f;
-#pragma unroll
-        for (int k = 0; k < N / 16; ++k) {
-          uint32_t b[4];
-          wm_ldsm_x4(wm_b(sB, NP, sb * 16, k * 16, lane), b);
-          wm_mma(gacc[0], cf[k], b[0], b[1]);
-          wm_mma(gacc[1], cf[k], b[2], b[3]);
-        }
-        uint32_t af[4];
+      };
+      auto store_block = [&](int tb, int sb) {     // decays, step sizes and the mask; bf16
+        const int ta = tb * 16 + gq, tb8 = ta + 8;
+        const float ca = cum[ta], cb = cum[tb8];
 #pragma unroll
         for (int i = 0; i < 2; ++i) {
           const int s0 = sb * 16 + i * 8 + 2 * tq;
           const float2 cs = *reinterpret_cast<const float2*>(cum + s0), ds = *reinterpret_cast<const float2*>(dts + s0);
-          const float m00 = s0 <= r0 ? gacc[i][0] * ds.x * wm_ex2(ct0 - cs.x) : 0.f;
-          const float m01 = s0 + 1 <= r0 ? gacc[i][1] * ds.y * wm_ex2(ct0 - cs.y) : 0.f;
-          const float m10 = s0 <= r1 ? gacc[i][2] * ds.x * wm_ex2(ct1 - cs.x) : 0.f;
-          const float m11 = s0 + 1 <= r1 ? gacc[i][3] * ds.y * wm_ex2(ct1 - cs.y) : 0.f;
-          af[2 * i] = pack_bf16x2(m00, m01);
-          af[2 * i + 1] = pack_bf16x2(m10, m11);
+          const float m00 = s0 <= ta ? gacc[i][0] * ds.x * wm_ex2(ca - cs.x) : 0.f;
+          const float m01 = s0 + 1 <= ta ? gacc[i][1] * ds.y * wm_ex2(ca - cs.y) : 0.f;
+          const float m10 = s0 <= tb8 ? gacc[i][2] * ds.x * wm_ex2(cb - cs.x) : 0.f;
+          const float m11 = s0 + 1 <= tb8 ? gacc[i][3] * ds.y * wm_ex2(cb - cs.y) : 0.f;
+          *reinterpret_cast<uint32_t*>(sc_smem + L::kM + wm_swz(ta, s0 >> 3) + (s0 & 7) * 2) = pack_bf16x2(m00, m01);
+          *reinterpret_cast<uint32_t*>(sc_smem + L::kM + wm_swz(tb8, s0 >> 3) + (s0 & 7) * 2) = pack_bf16x2(m10, m11);
         }
+      };
+      clear();
+#pragma unroll
+      for (int k = 0; k < N / 16; ++k) {
+        uint32_t cf[4];
+        wm_ldsm_x4(wm_a(sC, NP, wr * 16, k * 16, lane), cf);
+#pragma unroll
+        for (int j = 0; j < 2; ++j) {
+          uint32_t b[4];
+          wm_ldsm_x4_t(wm_b_t(sS, XP, wc * 32 + j * 16, k * 16, lane), b);
+          wm_mma(y[2 * j], cf, b[0], b[1]);
+          wm_mma(y[2 * j + 1], cf, b[2], b[3]);
+        }
+        if (own >= 0) {
+          uint32_t b[4];
+          wm_ldsm_x4(wm_b(sB, NP, own * 16, k * 16, lane), b);
+          wm_mma(gacc[0], cf, b[0], b[1]);
+          wm_mma(gacc[1], cf, b[2], b[3]);
+        }
+      }
+      if (own >= 0) store_block(wr, own);
+      if (wr == 0) {
+        for (int e = 0; e <= wc; ++e) {            // (2, 0); (3, 0), (3, 1)
+          clear();
+#pragma unroll
+          for (int k = 0; k < N / 16; ++k) {
+            uint32_t cf[4], b[4];
+            wm_ldsm_x4(wm_a(sC, NP, (2 + wc) * 16, k * 16, lane), cf);
+            wm_ldsm_x4(wm_b(sB, NP, e * 16, k * 16, lane), b);
+            wm_mma(gacc[0], cf, b[0], b[1]);
+            wm_mma(gacc[1], cf, b[2], b[3]);
+          }
+          store_block(2 + wc, e);
+        }
+      }
+      const float e0 = wm_ex2(cum[r0]), e1 = wm_ex2(cum[r1]);
+#pragma unroll
+      for (int j = 0; j < 4; ++j) { y[j][0] *= e0; y[j][1] *= e0; y[j][2] *= e1; y[j][3] *= e1; }
+    }
+    __syncthreads();                               // the scaled x and the masked products are complete; C and the state's copy are free
+    if (more) request_c(t0 + kScChunk);
+    wm_cp_commit();
+    if (!STATE_ONLY) {
+      // ---- + (masked C B^T) x + D x, out
+#pragma unroll
+      for (int sb = 0; sb < 4; ++sb) {
+        if (sb > wr) break;
+        uint32_t af[4];
+        wm_ldsm_x4(wm_a_swz(sM, wr * 16, sb * 16, lane), af);
 #pragma unroll
         for (int j = 0; j < 2; ++j) {
           uint32_t b[4];
@@ -253,9 +284,7 @@ state_space_chunk_kernel(const RbStateSpaceArgs a, float* __restrict__ span_stat
           wm_mma(y[2 * j + 1], af, b[2], b[3]);
         }
       }
-      // ---- + D x, out
       __nv_bfloat16* out = reinterpret_cast<__nv_bfloat16*>(a.y) + static_cast<long long>(seg.first + t0) * a.ld_y + offX;
-      const __nv_bfloat16* xs = reinterpret_cast<const __nv_bfloat16*>(sc_smem + L::kX);
 #pragma unroll
       for (int j = 0; j < 4; ++j) {
         const int p = p_base + 8 * j;
@@ -270,9 +299,6 @@ state_space_chunk_kernel(const RbStateSpaceArgs a, float* __restrict__ span_stat
         }
       }
     }
-    __syncthreads();                               // the scaled x is complete; C, x and the copy of the state are free
-    if (more) request_cx(t0 + kScChunk);
-    wm_cp_commit();
     // ---- state behind the chunk
     const float e_end = wm_ex2(c_end);
     total += c_end;
@@ -292,7 +318,7 @@ state_space_chunk_kernel(const RbStateSpaceArgs a, float* __restrict__ span_stat
 #pragma unroll
         for (int j = 0; j < 2; ++j) {
           uint32_t b[4];
-          wm_ldsm_x4_t(wm_b_t(sXs + half * kScChunk * XP * 2, XP, wc * 32 + j * 16, k * 16, lane), b);
+          wm_ldsm_x4_t(wm_b_t_swz(sXs + half * kScChunk * 128, wc * 32 + j * 16, k * 16, lane), b);
 #pragma unroll
           for (int m = 0; m < MT; ++m) {
             wm_mma(S[m][2 * j], af[m], b[0], b[1]);
@@ -313,20 +339,21 @@ state_space_chunk_kernel(const RbStateSpaceArgs a, float* __restrict__ span_stat
 
 template <int N>
 int sc_chunk_launch(const RbStateSpaceArgs& a, float* span_state, float* span_decay, int span, cudaStream_t s) {
-  const int smem = ScSmem<N>::kTotal;
+  const int smem1 = ScSmem<N, true>::kTotal, smem2 = ScSmem<N, false>::kTotal;
+  static_assert(2 * (ScSmem<N, false>::kTotal + 1024) <= 228 * 1024, "two CTAs share an SM");
   auto first = state_space_chunk_kernel<N, true>;
   auto second = state_space_chunk_kernel<N, false>;
   static bool cfg_dev[64] = {false};
   bool& cfg = cfg_dev[rbhost::device_slot()];
   if (!cfg) {
-    cudaError_t e = cudaFuncSetAttribute(first, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
-    if (e == cudaSuccess) e = cudaFuncSetAttribute(second, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+    cudaError_t e = cudaFuncSetAttribute(first, cudaFuncAttributeMaxDynamicSharedMemorySize, smem1);
+    if (e == cudaSuccess) e = cudaFuncSetAttribute(second, cudaFuncAttributeMaxDynamicSharedMemorySize, smem2);
     if (e != cudaSuccess) return static_cast<int>(e);
     cfg = true;
   }
   const dim3 grid(a.heads * ((a.p + kScCols - 1) / kScCols), a.num_tiles);
-  if (span_state) first<<<grid, kScThreads, smem, s>>>(a, span_state, span_decay, span);
-  second<<<grid, kScThreads, smem, s>>>(a, span_state, span_decay, span);
+  if (span_state) first<<<grid, kScThreads, smem1, s>>>(a, span_state, span_decay, span);
+  second<<<grid, kScThreads, smem2, s>>>(a, span_state, span_decay, span);
   return static_cast<int>(cudaGetLastError());
 }
 
