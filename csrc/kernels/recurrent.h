@@ -39,11 +39,12 @@ typedef struct RbStateSpaceArgs {
   const int* segments;
   const int* tiles;          // chunked form: [num_tiles, 2]: segment, first row inside it
   long long ld_xbc, ld_dt, ld_y;
+  long long rows;            // chunked form: rows of xbc
   int num_segments, num_tiles, heads, groups, p, n, f32, num_slots;
 } RbStateSpaceArgs;
 int rb_state_space_scan(const RbStateSpaceArgs* args, void* stream);
 // The same for prompts on the tensor cores: bf16, n <= 128, n and p multiples of 8 (-9 otherwise).  `tiles` lists spans of `span`
-// rows (a multiple of 64, in order, every one listed), which run side by side.  span_state fp32 [num_tiles, heads, n, p] and
+// rows (a multiple of 128, in order, every one listed), which run side by side.  span_state fp32 [num_tiles, heads, n, p] and
 // span_decay fp32 [num_tiles, heads] are scratch; both may be NULL when no segment has more than one span.
 int rb_state_space_chunked(const RbStateSpaceArgs* args, float* span_state, float* span_decay, int span, void* stream);
 

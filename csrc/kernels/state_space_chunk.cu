@@ -1,51 +1,84 @@
-// Mamba-2 state-space recurrence over prompts, chunked: 64 tokens at a time become matrix products on the tensor cores.
+// Mamba-2 state-space recurrence over prompts, chunked: 128 tokens at a time become matrix products on the 5th-generation tensor
+// cores.
 //
 // With c_t the running sum of the logarithms of the decays inside a chunk and S0 the state in front of it,
 //   y_t = exp(c_t) C_t S0 + sum_{s <= t} exp(c_t - c_s) dt_s (C_t . B_s) x_s + D x_t
 //   S   = exp(c_end) S0 + sum_s B_s (exp(c_end - c_s) dt_s x_s)^T
-// One CTA (8 warps) owns 64 value columns of one head over a span of chunks.  The state stays in fp32 accumulator registers; its
-// bf16 copy in shared memory is the operand of the read-out only.  What enters the state is split into two bf16 numbers (about 16
-// bits), decays and step sizes are fp32, so the state itself is good to fp32-like accuracy.
+// One CTA owns 64 value columns of one head over a span of chunks.  Its roles:
+//   warp 0   TMA: C, B and x of a chunk, two stages
+//   warp 1   issues the MMAs:  G = C B^T,  Y2 = C S0,  dS = B^T xs,  Y1 = M x   (accumulators in TMEM, all 512 columns)
+//   warp 2   step sizes, running log decays and the factors made of them, one chunk ahead
+//   group 1  (warps 4-7)    M = G times decays and step sizes below the diagonal, bf16 in TMEM: the A operand of Y1
+//   group 2  (warps 8-11)   xs = x scaled by what it adds to the state, then S = exp(c_end) S + dS; one state row per thread
+//   group 3  (warps 12-15)  y = exp(c_t) Y2 + Y1 + D x
+// The state stays in fp32 registers; its bf16 copy in shared memory is the operand of the read-out only.  xs is split into two bf16
+// numbers (about 16 bits), decays and step sizes are fp32, so the state itself is good to fp32-like accuracy.
 //
-// A long segment is cut into spans that run side by side: a first pass computes what every span but the last adds to the state
-// (from zero) and its total decay, and each span of the second pass starts from the combination of those before it.
+// Decays inside M: for 32 x 32 blocks below the diagonal exp(c_t - c_s) = exp(c_t - c_e) exp(c_e - c_s) with e the block's last
+// token; both factors are at most 1, and only diagonal blocks need an exponential per element.
+//
+// A long segment is cut into spans that run side by side: a first pass (STATE_ONLY) computes what every span but the last adds to
+// the state (from zero) and its total decay, and each span of the second pass starts from the combination of those before it.
+// Rows behind the segment's end are other sequences' rows: their step size counts as zero, and nothing of them is stored.
 #include "recurrent.h"
 
 #include "recurrent.cuh"
-#include "warp_mma.cuh"
 
 namespace rb {
 
-constexpr int kScChunk = 64;
+constexpr int kScChunk = 128;
 constexpr int kScCols = 64;
-constexpr int kScThreads = 256;
+constexpr int kScThreads = 512;
 constexpr float kScLog2e = 1.4426950408889634f;
 
-template <int N, bool STATE_ONLY>
 struct ScSmem {
-  static constexpr int kPitch = N + 8, kXPitch = kScCols + 8;
-  static constexpr int kB = 0;                                       // two buffers
-  static constexpr int kX = kB + 2 * kScChunk * kPitch * 2;          // two buffers
-  static constexpr int kXs = kX + 2 * kScChunk * kXPitch * 2;        // scaled x, permuted rows: high half, low half
-  static constexpr int kCum = kXs + 2 * kScChunk * kScCols * 2;      // two buffers: fp32 [64] running log2 decays, [64] step sizes
-  static constexpr int kC = kCum + 4 * kScChunk * 4;
-  static constexpr int kM = kC + (STATE_ONLY ? 0 : kScChunk * kPitch * 2);       // masked products C . B, permuted rows
-  static constexpr int kS = kM + (STATE_ONLY ? 0 : kScChunk * kScChunk * 2);     // bf16 copy of the state
-  static constexpr int kTotal = kS + (STATE_ONLY ? 0 : N * kXPitch * 2);
+  static constexpr int kAtom = kScChunk * 128;                       // 128 rows of 64 bf16, 128-byte swizzle
+  static constexpr int kC = 0;
+  static constexpr int kB = kC + 2 * kAtom;
+  static constexpr int kX = kB + 2 * kAtom;
+  static constexpr int kStage = kX + kAtom;
+  static constexpr int kXs = 2 * kStage;                             // scaled x: high half, low half
+  static constexpr int kS = kXs + 2 * kAtom;                         // bf16 copy of the state [128 rows][64]
+  static constexpr int kTab = kS + kAtom;                            // two buffers of fp32 [4][128]
+  static constexpr int kBar = kTab + 2 * 4 * kScChunk * 4;
+  static constexpr int kNumBars = 2 + 2 + 2 + 2 + 6;
+  static constexpr int kTotal = kBar + kNumBars * 8 + 16;
 };
+static_assert(ScSmem::kTotal + 1024 <= 227 * 1024, "shared memory of a CTA");
 
-template <int N, bool STATE_ONLY>
-__global__ void __launch_bounds__(kScThreads, STATE_ONLY ? 3 : 2)
-state_space_chunk_kernel(const RbStateSpaceArgs a, float* __restrict__ span_state, float* __restrict__ span_decay, int span) {
-  using L = ScSmem<N, STATE_ONLY>;
-  constexpr int MT = N / 64;                       // 16-row tiles of the state per warp
-  constexpr int NP = L::kPitch, XP = L::kXPitch;
-  extern __shared__ __align__(16) uint8_t sc_smem[];
-  const uint32_t base = smem_u32(sc_smem);
-  const uint32_t sC = base + L::kC, sXs = base + L::kXs, sM = base + L::kM, sS = base + L::kS;
+// columns of TMEM
+constexpr int kTmG = 0, kTmM = 256, kTmY1 = 320, kTmY2 = 384, kTmS = 448;
+
+__device__ __forceinline__ float sc_ex2(float x) {
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+// v = hi + lo with both halves bf16
+__device__ __forceinline__ void sc_split(float a, float b, uint32_t& hi, uint32_t& lo) {
+  hi = pack_bf16x2(a, b);
+  const float2 h = unpack_bf16x2(hi);
+  lo = pack_bf16x2(a - h.x, b - h.y);
+}
+// 16-byte piece `piece` of row `row` of a 128-byte swizzled tile
+__device__ __forceinline__ int sc_piece(int row, int piece) { return row * 128 + ((piece ^ (row & 7)) << 4); }
+
+template <bool STATE_ONLY>
+__global__ void __launch_bounds__(kScThreads, 1)
+state_space_chunk_kernel(const __grid_constant__ CUtensorMap tmC, const __grid_constant__ CUtensorMap tmB,
+                         const __grid_constant__ CUtensorMap tmX, const RbStateSpaceArgs a, float* __restrict__ span_state,
+                         float* __restrict__ span_decay, int span, unsigned int* status) {
+  using L = ScSmem;
+  extern __shared__ __align__(1024) uint8_t sc_raw[];
+  uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(sc_raw) + 1023) & ~uintptr_t(1023));
+  const uint32_t base = smem_u32(smem);
+  const uint32_t b0 = base + L::kBar;
+  const uint32_t bar_full = b0, bar_empty = b0 + 16, bar_g = b0 + 32, bar_tab = b0 + 48;      // [2] each
+  const uint32_t bar_m = b0 + 64, bar_y = b0 + 72, bar_yfree = b0 + 80, bar_xs = b0 + 88, bar_ds = b0 + 96, bar_s0 = b0 + 104;
+  uint32_t* tmem_ptr_smem = reinterpret_cast<uint32_t*>(smem + L::kBar + L::kNumBars * 8);
+  volatile int* abort_flag = reinterpret_cast<volatile int*>(tmem_ptr_smem + 1);
+
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
-  const int gq = lane >> 2, tq = lane & 3;
-  const int wc = warp >> 2, wr = wc ? 3 - (warp & 3) : (warp & 3);   // the causal work of a scheduler's two warps adds up evenly
   const int ptiles = (a.p + kScCols - 1) / kScCols;
   const int h = blockIdx.x / ptiles, c0 = (blockIdx.x - h * ptiles) * kScCols;
   const int tile = blockIdx.y;
@@ -54,323 +87,403 @@ state_space_chunk_kernel(const RbStateSpaceArgs a, float* __restrict__ span_stat
   const int end = min(seg.len, off + span);
   if (off >= seg.len) return;
   if (STATE_ONLY && end == seg.len) return;        // nobody starts from what the last span adds
+  const int chunks = (end - off + kScChunk - 1) / kScChunk;
   const int g = h / (a.heads / a.groups);
-  const __nv_bfloat16* xbc = reinterpret_cast<const __nv_bfloat16*>(a.xbc);
-  const long long offX = static_cast<long long>(h) * a.p + c0;
-  const long long offB = static_cast<long long>(a.heads) * a.p + static_cast<long long>(g) * a.n;
-  const long long offC = offB + static_cast<long long>(a.groups) * a.n;
-  const float rate2 = expf(a.a_log[h]) * kScLog2e, dt_bias = a.dt_bias[h], dskip = a.D[h];
+  const int ksteps_n = (a.n + 15) / 16;            // products over the state rows
+  const int atoms = a.n > 64 ? 2 : 1;
 
-  // this thread's part of the state: rows n = wr N/4 + 16 m + gq (+ 8), columns wc 32 + 8 j + 2 tq (+ 1)
-  const int n_base = wr * (N / 4) + gq, p_base = wc * 32 + 2 * tq;
-  float S[MT][4][4];
-#pragma unroll
-  for (int m = 0; m < MT; ++m)
-#pragma unroll
-    for (int j = 0; j < 4; ++j) S[m][j][0] = S[m][j][1] = S[m][j][2] = S[m][j][3] = 0.f;
-  auto each = [&](auto f) {                        // f(two neighbouring entries, row, column)
-#pragma unroll
-    for (int m = 0; m < MT; ++m)
-#pragma unroll
-      for (int j = 0; j < 4; ++j)
-#pragma unroll
-        for (int r = 0; r < 2; ++r) {
-          const int n = n_base + 16 * m + 8 * r, p = c0 + p_base + 8 * j;
-          if (n < a.n && p < a.p) f(S[m][j][2 * r], S[m][j][2 * r + 1], static_cast<long long>(n) * a.p + p);
-        }
-  };
-  const long long state_n = static_cast<long long>(a.n) * a.p;
-  float* slot = a.state + (static_cast<long long>(seg.slot) * a.heads + h) * state_n;
-  if (!STATE_ONLY) {
-    if (seg.start > 0)
-      each([&](float& u, float& v, long long i) { const float2 s = *reinterpret_cast<const float2*>(slot + i); u = s.x; v = s.y; });
-    for (int t = tile - off / span; t < tile; ++t) {               // spans of this segment in front of this one
-      const float d = wm_ex2(span_decay[static_cast<long long>(t) * a.heads + h]);
-      const float* add = span_state + (static_cast<long long>(t) * a.heads + h) * state_n;
-      each([&](float& u, float& v, long long i) {
-        const float2 s = *reinterpret_cast<const float2*>(add + i);
-        u = fmaf(u, d, s.x);
-        v = fmaf(v, d, s.y);
-      });
+  if (tid == 0) {
+    for (int s = 0; s < 2; ++s) {
+      mbar_init(bar_full + 8 * s, 1);
+      mbar_init(bar_empty + 8 * s, STATE_ONLY ? 1 : 5);
+      mbar_init(bar_g + 8 * s, 1);
+      mbar_init(bar_tab + 8 * s, 1);
     }
+    mbar_init(bar_m, 4);
+    mbar_init(bar_y, 1);
+    mbar_init(bar_yfree, 4);
+    mbar_init(bar_xs, 4);
+    mbar_init(bar_ds, 1);
+    mbar_init(bar_s0, 4);
+    *abort_flag = 0;
+    fence_mbar_init();
+    tma_prefetch_desc(&tmC);
+    tma_prefetch_desc(&tmB);
+    tma_prefetch_desc(&tmX);
   }
-  float total = 0.f;
+  if (atoms == 1) {                                // the state has 128 rows in TMEM: columns 64 .. 127 of B are zero
+    for (int i = tid; i < 2 * L::kAtom / 16; i += kScThreads) {
+      const int s = i / (L::kAtom / 16);
+      *reinterpret_cast<uint4*>(smem + s * L::kStage + L::kB + L::kAtom + (i - s * (L::kAtom / 16)) * 16) = make_uint4(0u, 0u, 0u, 0u);
+    }
+    fence_proxy_async_smem();
+  }
+  if (warp == 1) {
+    tmem_alloc(smem_u32(tmem_ptr_smem), 512);
+    tmem_relinquish();
+  }
+  tc_fence_before();
+  __syncthreads();
+  tc_fence_after();
+  const uint32_t tmem = *tmem_ptr_smem;
 
-  // Tiles of a chunk (rows past the end and columns past the real sizes are zero).  B and x have two buffers; C is free again
-  // behind the second barrier of a chunk, so the next chunk's is requested there and arrives under the state's products.
-  auto request_bx = [&](int t0) {
-    const int m_rows = min(kScChunk, end - t0);
-    const __nv_bfloat16* rows = xbc + static_cast<long long>(seg.first + t0) * a.ld_xbc;
-    const uint32_t dst = base + L::kB + ((t0 - off) / kScChunk & 1) * kScChunk * NP * 2;
-    for (int i = tid; i < kScChunk * (N / 8); i += kScThreads) {
-      const int r = i / (N / 8), c = (i - r * (N / 8)) * 8;
-      const bool ok = r < m_rows && c < a.n;
-      wm_cp16(dst + (r * NP + c) * 2, ok ? rows + r * a.ld_xbc + offB + c : rows, ok);
-    }
-    const uint32_t dst_x = base + L::kX + ((t0 - off) / kScChunk & 1) * kScChunk * XP * 2;
-    for (int i = tid; i < kScChunk * (kScCols / 8); i += kScThreads) {
-      const int r = i / (kScCols / 8), c = (i - r * (kScCols / 8)) * 8;
-      const bool ok = r < m_rows && c0 + c < a.p;
-      wm_cp16(dst_x + (r * XP + c) * 2, ok ? rows + r * a.ld_xbc + offX + c : rows, ok);
-    }
-  };
-  auto request_c = [&](int t0) {
-    if (STATE_ONLY) return;
-    const int m_rows = min(kScChunk, end - t0);
-    const __nv_bfloat16* rows = xbc + static_cast<long long>(seg.first + t0) * a.ld_xbc;
-    for (int i = tid; i < kScChunk * (N / 8); i += kScThreads) {
-      const int r = i / (N / 8), c = (i - r * (N / 8)) * 8;
-      const bool ok = r < m_rows && c < a.n;
-      wm_cp16(sC + (r * NP + c) * 2, ok ? rows + r * a.ld_xbc + offC + c : rows, ok);
-    }
-  };
-  // Step sizes and running log2 decays by warp 0, two tokens per lane; the raw values are fetched one chunk earlier still.
-  float raw[2] = {0.f, 0.f};
-  auto fetch_dt = [&](int t0) {
-#pragma unroll
-    for (int i = 0; i < 2; ++i) {
-      const int t = t0 + 2 * lane + i;
-      if (t < end) raw[i] = a.dt_raw[static_cast<long long>(seg.first + t) * a.ld_dt + h];
-    }
-  };
-  auto scan_dt = [&](int t0) {
-    float* cum = reinterpret_cast<float*>(sc_smem + L::kCum) + ((t0 - off) / kScChunk & 1) * 2 * kScChunk;
-    float d[2], s[2];
-#pragma unroll
-    for (int i = 0; i < 2; ++i) {
-      d[i] = t0 + 2 * lane + i < end ? rc_softplus(raw[i] + dt_bias) : 0.f;
-      s[i] = -rate2 * d[i];
-    }
-    float run = s[0] + s[1];
-#pragma unroll
-    for (int o = 1; o < 32; o <<= 1) {
-      const float u = __shfl_up_sync(0xffffffffu, run, o);
-      if (lane >= o) run += u;
-    }
-    cum[2 * lane] = run - s[1];
-    cum[2 * lane + 1] = run;
-    cum[kScChunk + 2 * lane] = d[0];
-    cum[kScChunk + 2 * lane + 1] = d[1];
-  };
-  auto publish = [&]() {                           // bf16 copy of the state for the read-out
-#pragma unroll
-    for (int m = 0; m < MT; ++m)
-#pragma unroll
-      for (int j = 0; j < 4; ++j)
-#pragma unroll
-        for (int r = 0; r < 2; ++r)
-          *reinterpret_cast<uint32_t*>(sc_smem + L::kS + ((n_base + 16 * m + 8 * r) * XP + p_base + 8 * j) * 2) =
-              pack_bf16x2(S[m][j][2 * r], S[m][j][2 * r + 1]);
-  };
-  request_bx(off);
-  request_c(off);
-  wm_cp_commit();
   if (warp == 0) {
-    fetch_dt(off);
-    scan_dt(off);
-    fetch_dt(off + kScChunk);
-  }
-  if (!STATE_ONLY) publish();
-
-  for (int t0 = off; t0 < end; t0 += kScChunk) {
-    const int m_rows = min(kScChunk, end - t0);
-    const int par = (t0 - off) / kScChunk & 1;
-    const uint32_t sB = base + L::kB + par * kScChunk * NP * 2, sX = base + L::kX + par * kScChunk * XP * 2;
-    const __nv_bfloat16* xs = reinterpret_cast<const __nv_bfloat16*>(sc_smem + L::kX) + par * kScChunk * XP;
-    const float* cum = reinterpret_cast<const float*>(sc_smem + L::kCum) + par * 2 * kScChunk;
-    const float* dts = cum + kScChunk;
-    const bool more = t0 + kScChunk < end;
-    wm_cp_wait<0>();
-    __syncthreads();                               // tiles, step sizes and the state in front of the chunk have arrived
-    if (more) request_bx(t0 + kScChunk);
-    if (warp == 0 && more) {
-      scan_dt(t0 + kScChunk);
-      fetch_dt(t0 + 2 * kScChunk);
+    if (lane == 0) {
+      // ------------------------------------------------------------------ TMA
+      for (int i = 0; i < chunks; ++i) {
+        const int s = i & 1, row = seg.first + off + i * kScChunk;
+        if (!mbar_wait(bar_empty + 8 * s, ((i >> 1) & 1) ^ 1, abort_flag, status, 61)) break;
+        const uint32_t st = base + s * L::kStage, bar = bar_full + 8 * s;
+        mbar_arrive_expect_tx(bar, L::kAtom * (1 + (STATE_ONLY ? 1 : 2) * atoms));
+        for (int k = 0; k < atoms; ++k) {
+          tma_load_4d(st + L::kB + k * L::kAtom, &tmB, k * 64, g, row, 0, bar);
+          if (!STATE_ONLY) tma_load_4d(st + L::kC + k * L::kAtom, &tmC, k * 64, g, row, 0, bar);
+        }
+        tma_load_4d(st + L::kX, &tmX, c0, h, row, 0, bar);
+      }
     }
-    const float c_end = cum[kScChunk - 1];
-    // ---- x scaled by what it adds to the state
-    for (int i = tid; i < kScChunk * (kScCols / 8); i += kScThreads) {
-      const int r = i / (kScCols / 8), c = (i - r * (kScCols / 8)) * 8;
-      const float w = dts[r] * wm_ex2(c_end - cum[r]);
-      float v[8];
-      RcVec<__nv_bfloat16, 8>::load(xs + r * XP + c, v);
-      uint32_t hi[4], lo[4];
-#pragma unroll
-      for (int k = 0; k < 4; ++k) wm_split(w * v[2 * k], w * v[2 * k + 1], hi[k], lo[k]);
-      *reinterpret_cast<uint4*>(sc_smem + L::kXs + wm_swz(r, c >> 3)) = make_uint4(hi[0], hi[1], hi[2], hi[3]);
-      *reinterpret_cast<uint4*>(sc_smem + L::kXs + kScChunk * 128 + wm_swz(r, c >> 3)) = make_uint4(lo[0], lo[1], lo[2], lo[3]);
-    }
-    float y[4][4];                                 // y of rows wr 16 .. + 16, columns wc 32 .. + 32
-    const int r0 = wr * 16 + gq, r1 = r0 + 8;
-    if (!STATE_ONLY) {
-      // ---- C S0, and one or two of the ten blocks (16 x 16) of C B^T on and below the diagonal: those of the warp's own rows in
-      // the same loop, the three that are left by the warps of the first rows, which have the least to do behind the barrier
-      const int own = wr > 0 ? wr - wc : (wc == 0 ? 0 : -1);
-#pragma unroll
-      for (int j = 0; j < 4; ++j) y[j][0] = y[j][1] = y[j][2] = y[j][3] = 0.f;
-      float gacc[2][4];
-      auto clear = [&]() {
-#pragma unroll
-        for (int i = 0; i < 2; ++i) gacc[i][0] = gacc[i][1] = gacc[i][2] = gacc[i][3] = 0.f;
+  } else if (warp == 1) {
+    if (lane == 0) {
+      // ------------------------------------------------------------------ MMA
+      constexpr uint32_t idesc_g = umma_idesc_bf16(128, 128, 0, 0);
+      constexpr uint32_t idesc_y = umma_idesc_bf16(128, kScCols, 0, 1);       // A K-major (C) or in TMEM (M), B MN-major
+      constexpr uint32_t idesc_s = umma_idesc_bf16(128, kScCols, 1, 1);       // A = B^T: MN-major
+      auto issue_g = [&](int i) -> bool {
+        if (!mbar_wait(bar_full + 8 * (i & 1), (i >> 1) & 1, abort_flag, status, 62)) return false;
+        if (STATE_ONLY) return true;
+        tc_fence_after();
+        const uint32_t st = base + (i & 1) * L::kStage;
+        for (int k = 0; k < ksteps_n; ++k) {
+          const uint32_t o = (k >> 2) * L::kAtom + (k & 3) * 32;
+          umma_bf16_ss(tmem + kTmG + (i & 1) * 128, umma_smem_desc_sw128(st + L::kC + o, 16, 1024),
+                       umma_smem_desc_sw128(st + L::kB + o, 16, 1024), idesc_g, k != 0 ? 1u : 0u);
+        }
+        umma_commit(bar_g + 8 * (i & 1));
+        return true;
       };
-      auto store_block = [&](int tb, int sb) {     // decays, step sizes and the mask; bf16
-        const int ta = tb * 16 + gq, tb8 = ta + 8;
-        const float ca = cum[ta], cb = cum[tb8];
-#pragma unroll
-        for (int i = 0; i < 2; ++i) {
-          const int s0 = sb * 16 + i * 8 + 2 * tq;
-          const float2 cs = *reinterpret_cast<const float2*>(cum + s0), ds = *reinterpret_cast<const float2*>(dts + s0);
-          const float m00 = s0 <= ta ? gacc[i][0] * ds.x * wm_ex2(ca - cs.x) : 0.f;
-          const float m01 = s0 + 1 <= ta ? gacc[i][1] * ds.y * wm_ex2(ca - cs.y) : 0.f;
-          const float m10 = s0 <= tb8 ? gacc[i][2] * ds.x * wm_ex2(cb - cs.x) : 0.f;
-          const float m11 = s0 + 1 <= tb8 ? gacc[i][3] * ds.y * wm_ex2(cb - cs.y) : 0.f;
-          *reinterpret_cast<uint32_t*>(sc_smem + L::kM + wm_swz(ta, s0 >> 3) + (s0 & 7) * 2) = pack_bf16x2(m00, m01);
-          *reinterpret_cast<uint32_t*>(sc_smem + L::kM + wm_swz(tb8, s0 >> 3) + (s0 & 7) * 2) = pack_bf16x2(m10, m11);
+      bool ok = issue_g(0);
+      for (int i = 0; i < chunks && ok; ++i) {
+        const uint32_t st = base + (i & 1) * L::kStage;
+        if (i + 1 < chunks && !issue_g(i + 1)) break;       // its buffer's last reader has arrived on bar_m
+        if (!STATE_ONLY) {
+          if (!mbar_wait(bar_s0, i & 1, abort_flag, status, 63)) break;
+          if (!mbar_wait(bar_yfree, (i & 1) ^ 1, abort_flag, status, 64)) break;
+          tc_fence_after();
+          for (int k = 0; k < ksteps_n; ++k)
+            umma_bf16_ss(tmem + kTmY2, umma_smem_desc_sw128(st + L::kC + (k >> 2) * L::kAtom + (k & 3) * 32, 16, 1024),
+                         umma_smem_desc_sw128(base + L::kS + k * 2048, L::kAtom, 1024), idesc_y, k != 0 ? 1u : 0u);
         }
-      };
-      clear();
+        if (!mbar_wait(bar_xs, i & 1, abort_flag, status, 65)) break;
+        tc_fence_after();
 #pragma unroll
-      for (int k = 0; k < N / 16; ++k) {
-        uint32_t cf[4];
-        wm_ldsm_x4(wm_a(sC, NP, wr * 16, k * 16, lane), cf);
+        for (int half = 0; half < 2; ++half)
 #pragma unroll
-        for (int j = 0; j < 2; ++j) {
-          uint32_t b[4];
-          wm_ldsm_x4_t(wm_b_t(sS, XP, wc * 32 + j * 16, k * 16, lane), b);
-          wm_mma(y[2 * j], cf, b[0], b[1]);
-          wm_mma(y[2 * j + 1], cf, b[2], b[3]);
+          for (int k = 0; k < kScChunk / 16; ++k)
+            umma_bf16_ss(tmem + kTmS, umma_smem_desc_sw128(st + L::kB + k * 2048, L::kAtom, 1024),
+                         umma_smem_desc_sw128(base + L::kXs + half * L::kAtom + k * 2048, L::kAtom, 1024), idesc_s,
+                         (half | k) != 0 ? 1u : 0u);
+        umma_commit(bar_ds);
+        if (!STATE_ONLY) {
+          if (!mbar_wait(bar_m, i & 1, abort_flag, status, 66)) break;
+          tc_fence_after();
+#pragma unroll
+          for (int k = 0; k < kScChunk / 16; ++k)
+            umma_bf16_ts(tmem + kTmY1, tmem + kTmM + k * 8, umma_smem_desc_sw128(st + L::kX + k * 2048, L::kAtom, 1024), idesc_y,
+                         k != 0 ? 1u : 0u);
+          umma_commit(bar_y);
         }
-        if (own >= 0) {
-          uint32_t b[4];
-          wm_ldsm_x4(wm_b(sB, NP, own * 16, k * 16, lane), b);
-          wm_mma(gacc[0], cf, b[0], b[1]);
-          wm_mma(gacc[1], cf, b[2], b[3]);
-        }
+        umma_commit(bar_empty + 8 * (i & 1));
       }
-      if (own >= 0) store_block(wr, own);
-      if (wr == 0) {
-        for (int e = 0; e <= wc; ++e) {            // (2, 0); (3, 0), (3, 1)
-          clear();
-#pragma unroll
-          for (int k = 0; k < N / 16; ++k) {
-            uint32_t cf[4], b[4];
-            wm_ldsm_x4(wm_a(sC, NP, (2 + wc) * 16, k * 16, lane), cf);
-            wm_ldsm_x4(wm_b(sB, NP, e * 16, k * 16, lane), b);
-            wm_mma(gacc[0], cf, b[0], b[1]);
-            wm_mma(gacc[1], cf, b[2], b[3]);
-          }
-          store_block(2 + wc, e);
-        }
-      }
-      const float e0 = wm_ex2(cum[r0]), e1 = wm_ex2(cum[r1]);
-#pragma unroll
-      for (int j = 0; j < 4; ++j) { y[j][0] *= e0; y[j][1] *= e0; y[j][2] *= e1; y[j][3] *= e1; }
     }
-    __syncthreads();                               // the scaled x and the masked products are complete; C and the state's copy are free
-    if (more) request_c(t0 + kScChunk);
-    wm_cp_commit();
+  } else if (warp == 2) {
+    // -------------------------------------------------------------------- factors of a chunk, four tokens per lane
+    const float rate2 = expf(a.a_log[h]) * kScLog2e, dt_bias = a.dt_bias[h];
+    float raw[4] = {0.f, 0.f, 0.f, 0.f}, total = 0.f;
+    auto fetch = [&](int i) {
+#pragma unroll
+      for (int k = 0; k < 4; ++k) {
+        const int t = off + i * kScChunk + 4 * lane + k;
+        if (t < end) raw[k] = a.dt_raw[static_cast<long long>(seg.first + t) * a.ld_dt + h];
+      }
+    };
+    fetch(0);
+    for (int i = 0; i < chunks; ++i) {
+      float d[4], c[4];
+#pragma unroll
+      for (int k = 0; k < 4; ++k) {
+        d[k] = off + i * kScChunk + 4 * lane + k < end ? rc_softplus(raw[k] + dt_bias) : 0.f;
+        c[k] = (k ? c[k ? k - 1 : 0] : 0.f) - rate2 * d[k];
+      }
+      if (i + 1 < chunks) fetch(i + 1);
+      float run = c[3];
+#pragma unroll
+      for (int o = 1; o < 32; o <<= 1) {
+        const float u = __shfl_up_sync(0xffffffffu, run, o);
+        if (lane >= o) run += u;
+      }
+      const float before = run - c[3];
+      const float c_end = __shfl_sync(0xffffffffu, run, 31), c_blk = __shfl_sync(0xffffffffu, run, lane | 7);
+      total += c_end;
+      if (!mbar_wait(bar_empty + 8 * (i & 1), ((i >> 1) & 1) ^ 1, abort_flag, status, 67)) break;
+      float4* tab = reinterpret_cast<float4*>(smem + L::kTab + (i & 1) * 4 * kScChunk * 4) + lane;
+      float v[4][4];
+#pragma unroll
+      for (int k = 0; k < 4; ++k) {
+        v[0][k] = before + c[k];
+        v[1][k] = d[k];
+        v[2][k] = d[k] * sc_ex2(c_blk - v[0][k]);  // towards the end of the token's block of 32
+        v[3][k] = d[k] * sc_ex2(c_end - v[0][k]);  // towards the end of the chunk
+      }
+#pragma unroll
+      for (int q = 0; q < 4; ++q) tab[q * 32] = make_float4(v[q][0], v[q][1], v[q][2], v[q][3]);
+      __syncwarp();
+      if (lane == 0) mbar_arrive(bar_tab + 8 * (i & 1));
+    }
+    if (STATE_ONLY && lane == 0 && c0 == 0) span_decay[static_cast<long long>(tile) * a.heads + h] = total;
+  } else if (warp >= 4 && warp < 8) {
     if (!STATE_ONLY) {
-      // ---- + (masked C B^T) x + D x, out
-#pragma unroll
-      for (int sb = 0; sb < 4; ++sb) {
-        if (sb > wr) break;
-        uint32_t af[4];
-        wm_ldsm_x4(wm_a_swz(sM, wr * 16, sb * 16, lane), af);
-#pragma unroll
-        for (int j = 0; j < 2; ++j) {
-          uint32_t b[4];
-          wm_ldsm_x4_t(wm_b_t(sX, XP, wc * 32 + j * 16, sb * 16, lane), b);
-          wm_mma(y[2 * j], af, b[0], b[1]);
-          wm_mma(y[2 * j + 1], af, b[2], b[3]);
-        }
+      // ------------------------------------------------------------------ M, one row per thread
+      const int wq = warp & 3, row = wq * 32 + lane;
+      const uint32_t lane_off = static_cast<uint32_t>(wq * 32) << 16;
+      const uint32_t tm = tmem + kTmM + lane_off;
+      {
+        const uint32_t zero[16] = {0u, 0u, 0u, 0u, 0u, 0u, 0u, 0u, 0u, 0u, 0u, 0u, 0u, 0u, 0u, 0u};
+        for (int b = wq + 1; b < 4; ++b) tmem_st_32x16(tm + b * 16, zero);     // above the diagonal, for good
       }
-      __nv_bfloat16* out = reinterpret_cast<__nv_bfloat16*>(a.y) + static_cast<long long>(seg.first + t0) * a.ld_y + offX;
+      for (int i = 0; i < chunks; ++i) {
+        const float* tab = reinterpret_cast<const float*>(smem + L::kTab + (i & 1) * 4 * kScChunk * 4);
+        if (!mbar_wait(bar_tab + 8 * (i & 1), (i >> 1) & 1, abort_flag, status, 68)) break;
+        if (!mbar_wait(bar_g + 8 * (i & 1), (i >> 1) & 1, abort_flag, status, 69)) break;
+        if (!mbar_wait(bar_y, (i & 1) ^ 1, abort_flag, status, 70)) break;     // Y1 of the chunk before has read M
+        tc_fence_after();
+        const float ct = tab[row];
+        for (int b = 0; b <= wq; ++b) {
+          uint32_t r[32];
+          tmem_ld_32x32(tmem + kTmG + (i & 1) * 128 + lane_off + b * 32, r);
+          tmem_ld_wait();
+          uint32_t packed[16];
+          if (b < wq) {
+            const float e = sc_ex2(ct - tab[b * 32 + 31]);
+            const float4* f = reinterpret_cast<const float4*>(tab + 2 * kScChunk + b * 32);
 #pragma unroll
-      for (int j = 0; j < 4; ++j) {
-        const int p = p_base + 8 * j;
-        if (c0 + p >= a.p) continue;
+            for (int q = 0; q < 8; ++q) {
+              const float4 u = f[q];
+              packed[2 * q] = pack_bf16x2(__uint_as_float(r[4 * q]) * e * u.x, __uint_as_float(r[4 * q + 1]) * e * u.y);
+              packed[2 * q + 1] = pack_bf16x2(__uint_as_float(r[4 * q + 2]) * e * u.z, __uint_as_float(r[4 * q + 3]) * e * u.w);
+            }
+          } else {
+            const float4* cs = reinterpret_cast<const float4*>(tab + b * 32);
+            const float4* ds = reinterpret_cast<const float4*>(tab + kScChunk + b * 32);
 #pragma unroll
-        for (int r = 0; r < 2; ++r) {
-          const int t = r ? r1 : r0;
-          if (t >= m_rows) continue;
-          const float2 x = unpack_bf16x2(*reinterpret_cast<const uint32_t*>(xs + t * XP + p));
-          *reinterpret_cast<uint32_t*>(out + static_cast<long long>(t) * a.ld_y + p) =
-              pack_bf16x2(fmaf(dskip, x.x, y[j][2 * r]), fmaf(dskip, x.y, y[j][2 * r + 1]));
-        }
-      }
-    }
-    // ---- state behind the chunk
-    const float e_end = wm_ex2(c_end);
-    total += c_end;
-#pragma unroll
-    for (int m = 0; m < MT; ++m)
-#pragma unroll
-      for (int j = 0; j < 4; ++j)
-#pragma unroll
-        for (int i = 0; i < 4; ++i) S[m][j][i] *= e_end;
-#pragma unroll
-    for (int k = 0; k < kScChunk / 16; ++k) {
-      uint32_t af[MT][4];
-#pragma unroll
-      for (int m = 0; m < MT; ++m) wm_ldsm_x4_t(wm_a_t(sB, NP, wr * (N / 4) + m * 16, k * 16, lane), af[m]);
-#pragma unroll
-      for (int half = 0; half < 2; ++half)
-#pragma unroll
-        for (int j = 0; j < 2; ++j) {
-          uint32_t b[4];
-          wm_ldsm_x4_t(wm_b_t_swz(sXs + half * kScChunk * 128, wc * 32 + j * 16, k * 16, lane), b);
-#pragma unroll
-          for (int m = 0; m < MT; ++m) {
-            wm_mma(S[m][2 * j], af[m], b[0], b[1]);
-            wm_mma(S[m][2 * j + 1], af[m], b[2], b[3]);
+            for (int q = 0; q < 8; ++q) {
+              const float4 c = cs[q], d = ds[q];
+              const float m0 = 4 * q <= lane ? __uint_as_float(r[4 * q]) * d.x * sc_ex2(ct - c.x) : 0.f;
+              const float m1 = 4 * q + 1 <= lane ? __uint_as_float(r[4 * q + 1]) * d.y * sc_ex2(ct - c.y) : 0.f;
+              const float m2 = 4 * q + 2 <= lane ? __uint_as_float(r[4 * q + 2]) * d.z * sc_ex2(ct - c.z) : 0.f;
+              const float m3 = 4 * q + 3 <= lane ? __uint_as_float(r[4 * q + 3]) * d.w * sc_ex2(ct - c.w) : 0.f;
+              packed[2 * q] = pack_bf16x2(m0, m1);
+              packed[2 * q + 1] = pack_bf16x2(m2, m3);
+            }
           }
+          tmem_st_32x16(tm + b * 16, packed);
         }
+        tmem_st_wait();
+        tc_fence_before();
+        __syncwarp();
+        if (lane == 0) mbar_arrive(bar_m);
+      }
     }
+  } else if (warp >= 8 && warp < 12) {
+    // -------------------------------------------------------------------- xs and the state: token row, then state row per thread
+    const int row = (warp & 3) * 32 + lane;
+    const uint32_t ts = tmem + kTmS + (static_cast<uint32_t>((warp & 3) * 32) << 16);
+    const long long state_n = static_cast<long long>(a.n) * a.p;
+    const long long at = static_cast<long long>(row) * a.p + c0;
+    float* slot = a.state + (static_cast<long long>(seg.slot) * a.heads + h) * state_n;
+    const bool live = row < a.n;
+    const int cols = min(kScCols, a.p - c0);       // multiple of 8
+    float S[kScCols];
+#pragma unroll
+    for (int j = 0; j < kScCols; j += 4) {
+      float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+      if (!STATE_ONLY && seg.start > 0 && live && j < cols) v = *reinterpret_cast<const float4*>(slot + at + j);
+      S[j] = v.x; S[j + 1] = v.y; S[j + 2] = v.z; S[j + 3] = v.w;
+    }
+    if (!STATE_ONLY) {
+      for (int t = tile - off / span; t < tile; ++t) {               // spans of this segment in front of this one
+        const float d = sc_ex2(span_decay[static_cast<long long>(t) * a.heads + h]);
+        const float* add = span_state + (static_cast<long long>(t) * a.heads + h) * state_n + at;
+#pragma unroll
+        for (int j = 0; j < kScCols; j += 4) {
+          if (!live || j >= cols) continue;
+          const float4 v = *reinterpret_cast<const float4*>(add + j);
+          S[j] = fmaf(S[j], d, v.x); S[j + 1] = fmaf(S[j + 1], d, v.y);
+          S[j + 2] = fmaf(S[j + 2], d, v.z); S[j + 3] = fmaf(S[j + 3], d, v.w);
+        }
+      }
+    }
+    auto publish = [&]() {                         // bf16 copy of the state for the read-out
+#pragma unroll
+      for (int q = 0; q < kScCols / 8; ++q)
+        *reinterpret_cast<uint4*>(smem + L::kS + sc_piece(row, q)) =
+            make_uint4(pack_bf16x2(S[8 * q], S[8 * q + 1]), pack_bf16x2(S[8 * q + 2], S[8 * q + 3]),
+                       pack_bf16x2(S[8 * q + 4], S[8 * q + 5]), pack_bf16x2(S[8 * q + 6], S[8 * q + 7]));
+      fence_proxy_async_smem();
+      __syncwarp();
+      if (lane == 0) mbar_arrive(bar_s0);
+    };
     if (!STATE_ONLY) publish();
+    bool ok = true;
+    for (int i = 0; i < chunks; ++i) {
+      const float* tab = reinterpret_cast<const float*>(smem + L::kTab + (i & 1) * 4 * kScChunk * 4);
+      const uint8_t* x = smem + (i & 1) * L::kStage + L::kX;
+      ok = mbar_wait(bar_tab + 8 * (i & 1), (i >> 1) & 1, abort_flag, status, 71) &&
+           mbar_wait(bar_full + 8 * (i & 1), (i >> 1) & 1, abort_flag, status, 72);
+      if (!ok) break;
+      const float w = tab[3 * kScChunk + row], e_end = sc_ex2(tab[kScChunk - 1]);
+#pragma unroll
+      for (int q = 0; q < kScCols / 8; ++q) {
+        float v[8];
+        RcVec<__nv_bfloat16, 8>::load(reinterpret_cast<const __nv_bfloat16*>(x + sc_piece(row, q)), v);
+        uint32_t hi[4], lo[4];
+#pragma unroll
+        for (int k = 0; k < 4; ++k) sc_split(w * v[2 * k], w * v[2 * k + 1], hi[k], lo[k]);
+        *reinterpret_cast<uint4*>(smem + L::kXs + sc_piece(row, q)) = make_uint4(hi[0], hi[1], hi[2], hi[3]);
+        *reinterpret_cast<uint4*>(smem + L::kXs + L::kAtom + sc_piece(row, q)) = make_uint4(lo[0], lo[1], lo[2], lo[3]);
+      }
+      fence_proxy_async_smem();
+      __syncwarp();
+      if (lane == 0) mbar_arrive(bar_xs);
+      ok = mbar_wait(bar_ds, i & 1, abort_flag, status, 73);
+      if (!ok) break;
+      tc_fence_after();
+#pragma unroll
+      for (int q = 0; q < kScCols / 32; ++q) {
+        uint32_t r[32];
+        tmem_ld_32x32(ts + q * 32, r);
+        tmem_ld_wait();
+#pragma unroll
+        for (int j = 0; j < 32; ++j) S[q * 32 + j] = fmaf(S[q * 32 + j], e_end, __uint_as_float(r[j]));
+      }
+      tc_fence_before();
+      if (!STATE_ONLY && i + 1 < chunks) publish();
+    }
+    if (ok && live && (STATE_ONLY || end == seg.len)) {
+      float* dst = STATE_ONLY ? span_state + (static_cast<long long>(tile) * a.heads + h) * state_n : slot;
+#pragma unroll
+      for (int j = 0; j < kScCols; j += 4)
+        if (j < cols) *reinterpret_cast<float4*>(dst + at + j) = make_float4(S[j], S[j + 1], S[j + 2], S[j + 3]);
+    }
+  } else if (warp >= 12) {
+    if (!STATE_ONLY) {
+      // ------------------------------------------------------------------ y, one row per thread
+      const int row = (warp & 3) * 32 + lane;
+      const uint32_t ty = tmem + (static_cast<uint32_t>((warp & 3) * 32) << 16);
+      const float dskip = a.D[h];
+      const int cols = min(kScCols, a.p - c0);
+      for (int i = 0; i < chunks; ++i) {
+        const float* tab = reinterpret_cast<const float*>(smem + L::kTab + (i & 1) * 4 * kScChunk * 4);
+        const uint8_t* x = smem + (i & 1) * L::kStage + L::kX;
+        if (!mbar_wait(bar_tab + 8 * (i & 1), (i >> 1) & 1, abort_flag, status, 74)) break;
+        if (!mbar_wait(bar_full + 8 * (i & 1), (i >> 1) & 1, abort_flag, status, 75)) break;
+        const float e = sc_ex2(tab[row]);
+        if (!mbar_wait(bar_y, i & 1, abort_flag, status, 76)) break;
+        tc_fence_after();
+        uint32_t packed[kScCols / 2];
+#pragma unroll
+        for (int q = 0; q < kScCols / 32; ++q) {
+          uint32_t y1[32], y2[32];
+          tmem_ld_32x32(ty + kTmY1 + q * 32, y1);
+          tmem_ld_32x32(ty + kTmY2 + q * 32, y2);
+          tmem_ld_wait();
+#pragma unroll
+          for (int k = 0; k < 4; ++k) {
+            float v[8];
+            RcVec<__nv_bfloat16, 8>::load(reinterpret_cast<const __nv_bfloat16*>(x + sc_piece(row, q * 4 + k)), v);
+#pragma unroll
+            for (int j = 0; j < 8; ++j)
+              v[j] = fmaf(dskip, v[j], fmaf(e, __uint_as_float(y2[8 * k + j]), __uint_as_float(y1[8 * k + j])));
+#pragma unroll
+            for (int j = 0; j < 4; ++j) packed[q * 16 + k * 4 + j] = pack_bf16x2(v[2 * j], v[2 * j + 1]);
+          }
+        }
+        tc_fence_before();
+        __syncwarp();
+        if (lane == 0) {
+          mbar_arrive(bar_yfree);
+          mbar_arrive(bar_empty + 8 * (i & 1));
+        }
+        const int t = off + i * kScChunk + row;
+        if (t < end) {
+          __nv_bfloat16* out = reinterpret_cast<__nv_bfloat16*>(a.y) + static_cast<long long>(seg.first + t) * a.ld_y +
+                               static_cast<long long>(h) * a.p + c0;
+#pragma unroll
+          for (int q = 0; q < kScCols / 8; ++q)
+            if (q * 8 < cols)
+              *reinterpret_cast<uint4*>(out + q * 8) = make_uint4(packed[4 * q], packed[4 * q + 1], packed[4 * q + 2], packed[4 * q + 3]);
+        }
+      }
+    }
   }
-  if (STATE_ONLY) {
-    float* dst = span_state + (static_cast<long long>(tile) * a.heads + h) * state_n;
-    each([&](float& u, float& v, long long i) { *reinterpret_cast<float2*>(dst + i) = make_float2(u, v); });
-    if (tid == 0 && c0 == 0) span_decay[static_cast<long long>(tile) * a.heads + h] = total;
-  } else if (end == seg.len) {
-    each([&](float& u, float& v, long long i) { *reinterpret_cast<float2*>(slot + i) = make_float2(u, v); });
-  }
-}
 
-template <int N>
-int sc_chunk_launch(const RbStateSpaceArgs& a, float* span_state, float* span_decay, int span, cudaStream_t s) {
-  const int smem1 = ScSmem<N, true>::kTotal, smem2 = ScSmem<N, false>::kTotal;
-  static_assert(2 * (ScSmem<N, false>::kTotal + 1024) <= 228 * 1024, "two CTAs share an SM");
-  auto first = state_space_chunk_kernel<N, true>;
-  auto second = state_space_chunk_kernel<N, false>;
-  static bool cfg_dev[64] = {false};
-  bool& cfg = cfg_dev[rbhost::device_slot()];
-  if (!cfg) {
-    cudaError_t e = cudaFuncSetAttribute(first, cudaFuncAttributeMaxDynamicSharedMemorySize, smem1);
-    if (e == cudaSuccess) e = cudaFuncSetAttribute(second, cudaFuncAttributeMaxDynamicSharedMemorySize, smem2);
-    if (e != cudaSuccess) return static_cast<int>(e);
-    cfg = true;
+  tc_fence_before();
+  __syncthreads();
+  if (warp == 1) {
+    if (*abort_flag) {
+      // a wait gave up: let copies and MMAs in flight land before the accumulators are released
+      const unsigned long long t0 = globaltimer_ns();
+      while (globaltimer_ns() - t0 < 200000ull) __nanosleep(1000);
+    }
+    tc_fence_after();
+    tmem_dealloc(tmem, 512);
   }
-  const dim3 grid(a.heads * ((a.p + kScCols - 1) / kScCols), a.num_tiles);
-  if (span_state) first<<<grid, kScThreads, smem1, s>>>(a, span_state, span_decay, span);
-  second<<<grid, kScThreads, smem2, s>>>(a, span_state, span_decay, span);
-  return static_cast<int>(cudaGetLastError());
 }
 
 }  // namespace rb
+
+namespace {
+// [rows, heads, size] part of a packed row-major matrix, 64 columns of 128 rows of one head at a time
+const CUtensorMap* sc_map(const void* base, int size, int heads, long long rows, long long ld, int* err) {
+  const uint64_t dims[4] = {(uint64_t)size, (uint64_t)heads, (uint64_t)rows, 1};
+  const uint64_t str[3] = {(uint64_t)size * 2, (uint64_t)ld * 2, (uint64_t)(rows * ld) * 2};
+  const uint32_t box[4] = {64, 1, (uint32_t)rb::kScChunk, 1};
+  return rbhost::get_tmap_4d(base, 2, dims, str, box, 1, err);
+}
+}  // namespace
 
 RB_API int rb_state_space_chunked(const RbStateSpaceArgs* args, float* span_state, float* span_decay, int span, void* stream_v) {
   const RbStateSpaceArgs& a = *args;
   if (a.num_tiles <= 0) return 0;
   if (!a.xbc || !a.dt_raw || !a.dt_bias || !a.a_log || !a.D || !a.state || !a.y || !a.segments || !a.tiles || a.f32 || a.heads <= 0 ||
-      a.groups <= 0 || a.heads % a.groups || a.p <= 0 || a.n <= 0 || a.num_slots <= 0 || a.num_tiles > 65535 || span <= 0 ||
-      span % rb::kScChunk || (span_state != nullptr) != (span_decay != nullptr))
+      a.groups <= 0 || a.heads % a.groups || a.p <= 0 || a.n <= 0 || a.num_slots <= 0 || a.num_tiles > 65535 || a.rows <= 0 ||
+      span <= 0 || span % rb::kScChunk || (span_state != nullptr) != (span_decay != nullptr))
     return -1;
   if (a.n > 128 || ((a.n | a.p) & 7) || ((a.ld_xbc | a.ld_y) & 7)) return -9;
   if ((reinterpret_cast<uintptr_t>(a.xbc) | reinterpret_cast<uintptr_t>(a.y) | reinterpret_cast<uintptr_t>(a.state) |
        reinterpret_cast<uintptr_t>(span_state)) & 15)
     return -9;
+  const __nv_bfloat16* x = reinterpret_cast<const __nv_bfloat16*>(a.xbc);
+  const __nv_bfloat16* b = x + static_cast<long long>(a.heads) * a.p;
+  const __nv_bfloat16* c = b + static_cast<long long>(a.groups) * a.n;
+  int err = 0;
+  const CUtensorMap* tx = sc_map(x, a.p, a.heads, a.rows, a.ld_xbc, &err);
+  const CUtensorMap* tb = sc_map(b, a.n, a.groups, a.rows, a.ld_xbc, &err);
+  const CUtensorMap* tc = sc_map(c, a.n, a.groups, a.rows, a.ld_xbc, &err);
+  if (!tx || !tb || !tc) return err ? err : -5;
+  auto first = rb::state_space_chunk_kernel<true>;
+  auto second = rb::state_space_chunk_kernel<false>;
+  const int smem = rb::ScSmem::kTotal + 1024;
+  static bool cfg_dev[64] = {false};
+  bool& cfg = cfg_dev[rbhost::device_slot()];
+  if (!cfg) {
+    cudaError_t e = cudaFuncSetAttribute(first, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+    if (e == cudaSuccess) e = cudaFuncSetAttribute(second, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+    if (e != cudaSuccess) return static_cast<int>(e);
+    cfg = true;
+  }
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream_v);
-  return a.n <= 64 ? rb::sc_chunk_launch<64>(a, span_state, span_decay, span, s)
-                   : rb::sc_chunk_launch<128>(a, span_state, span_decay, span, s);
+  const dim3 grid(a.heads * ((a.p + rb::kScCols - 1) / rb::kScCols), a.num_tiles);
+  if (span_state) first<<<grid, rb::kScThreads, smem, s>>>(*tc, *tb, *tx, a, span_state, span_decay, span, rbhost::status_ptr());
+  second<<<grid, rb::kScThreads, smem, s>>>(*tc, *tb, *tx, a, span_state, span_decay, span, rbhost::status_ptr());
+  return static_cast<int>(cudaGetLastError());
 }

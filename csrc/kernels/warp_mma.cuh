@@ -38,14 +38,6 @@ __device__ __forceinline__ uint32_t wm_b(uint32_t base, int pitch, int n0, int k
 __device__ __forceinline__ uint32_t wm_b_t(uint32_t base, int pitch, int n0, int k0, int lane) {
   return base + ((k0 + (lane & 7) + ((lane >> 3) & 1) * 8) * pitch + n0 + (lane >> 4) * 8) * 2;
 }
-// The same for tiles of 64 columns without padding: the 16-byte pieces of row r are permuted by r & 7.
-__device__ __forceinline__ uint32_t wm_swz(int row, int piece) { return row * 128 + ((piece ^ (row & 7)) << 4); }
-__device__ __forceinline__ uint32_t wm_a_swz(uint32_t base, int r0, int k0, int lane) {
-  return base + wm_swz(r0 + (lane & 15), (k0 >> 3) + (lane >> 4));
-}
-__device__ __forceinline__ uint32_t wm_b_t_swz(uint32_t base, int n0, int k0, int lane) {
-  return base + wm_swz(k0 + (lane & 7) + ((lane >> 3) & 1) * 8, (n0 >> 3) + (lane >> 4));
-}
 // 16-byte asynchronous global -> shared copy; !ok writes zeros and reads nothing
 __device__ __forceinline__ void wm_cp16(uint32_t dst, const void* src, bool ok) {
   asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst), "l"(src), "r"(ok ? 16 : 0) : "memory");

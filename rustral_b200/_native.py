@@ -122,6 +122,7 @@ class RbStateSpaceArgs(C.Structure):
     _fields_ = [
         ("xbc", c_void_p), ("dt_raw", c_void_p), ("dt_bias", c_void_p), ("a_log", c_void_p), ("D", c_void_p), ("state", c_void_p),
         ("y", c_void_p), ("segments", c_void_p), ("tiles", c_void_p), ("ld_xbc", c_ll), ("ld_dt", c_ll), ("ld_y", c_ll),
+        ("rows", c_ll),
         ("num_segments", c_int), ("num_tiles", c_int), ("heads", c_int), ("groups", c_int), ("p", c_int), ("n", c_int),
         ("f32", c_int), ("num_slots", c_int),
     ]

@@ -124,18 +124,18 @@ def _chunked(x, rows: int, a: int, b: int) -> bool:
     return x.dtype == torch.bfloat16 and rows <= 128 and a % 8 == 0 and b % 8 == 0 and x.stride(0) % 8 == 0 and x.data_ptr() % 16 == 0
 
 
-def _span(seg: Segments, ctas_per_span: int, slots: int = 2 * 148) -> int:
+def _span(seg: Segments, ctas_per_span: int, slots: int = 148) -> int:
     """Rows per span of the chunked state-space kernel: the power of two for which the spans that run side by side cost least
     (rounds of `slots` CTAs, and about half of that again for the first pass where segments have several spans)."""
     lens = [r[1] for r in seg.rows]
-    best, span = None, CHUNK
+    best, span = None, 0
     size = 256
     while True:
         spans = sum(-(-n // size) for n in lens)
         rows = min(size, max(lens))
-        cost = -(-spans * ctas_per_span // slots) * (rows + 64.0)
+        cost = -(-spans * ctas_per_span // slots) * (rows + 256.0)
         if spans > len(lens):
-            cost += 0.5 * -(-(spans - len(lens)) * ctas_per_span // slots) * (rows + 64.0)
+            cost += 0.5 * -(-(spans - len(lens)) * ctas_per_span // slots) * (rows + 256.0)
         if best is None or cost < best:
             best, span = cost, size
         if size >= max(lens):
@@ -178,6 +178,7 @@ def state_space(xbc, dt_raw, *, dt_bias, a_log, D, state, heads: int, groups: in
         span = _span(many, heads * ((vdim + 63) // 64))
         tiles = many.tiles(span)
         a.segments, a.num_segments, a.tiles, a.num_tiles = many.table.data_ptr(), many.n, tiles.data_ptr(), tiles.shape[0]
+        a.rows = rows
         states = decays = None
         if tiles.shape[0] > many.n:
             states = torch.empty((tiles.shape[0], heads, n, vdim), dtype=torch.float32, device=xbc.device)
