@@ -5,12 +5,16 @@
 //   y_t = exp(c_t) C_t S0 + sum_{s <= t} exp(c_t - c_s) dt_s (C_t . B_s) x_s + D x_t
 //   S   = exp(c_end) S0 + sum_s B_s (exp(c_end - c_s) dt_s x_s)^T
 // One CTA owns 64 value columns of one head over a span of chunks.  Its roles:
-//   warp 0   TMA: C, B and x of a chunk, two stages
-//   warp 1   issues the MMAs:  G = C B^T,  Y2 = C S0,  dS = B^T xs,  Y1 = M x   (accumulators in TMEM, all 512 columns)
+//   warp 0   TMA: B, C and x of a chunk, two buffers each, refilled as soon as their own last reader is done
+//   warp 1   issues the MMAs:  dS = B^T xs,  Y2 = C S0,  G = C B^T (of the next chunk),  Y1 = M x   (accumulators in TMEM, all
+//            512 columns)
 //   warp 2   step sizes, running log decays and the factors made of them, one chunk ahead
-//   group 1  (warps 4-7)    M = G times decays and step sizes below the diagonal, bf16 in TMEM: the A operand of Y1
-//   group 2  (warps 8-11)   xs = x scaled by what it adds to the state, then S = exp(c_end) S + dS; one state row per thread
-//   group 3  (warps 12-15)  y = exp(c_t) Y2 + Y1 + D x
+//   group 1  (warps 4-7)    M = G times decays and step sizes below the diagonal, plus D on it, bf16 in TMEM over G itself: the A
+//            operand of Y1
+//   groups 2, 3 (warps 8-15) xs = x scaled by what it adds to the state, as soon as the chunk before has read its own; then
+//   group 2  S = exp(c_end) S + dS, one state row per thread
+//   group 3  y = exp(c_t) Y2 + Y1
+// The chain from chunk to chunk is xs -> dS; the state's update, its copy, M and y run beside the next chunk's products.
 // The state stays in fp32 registers; its bf16 copy in shared memory is the operand of the read-out only.  xs is split into two bf16
 // numbers (about 16 bits), decays and step sizes are fp32, so the state itself is good to fp32-like accuracy.
 //
@@ -41,13 +45,13 @@ struct ScSmem {
   static constexpr int kS = kXs + 2 * kAtom;                         // bf16 copy of the state [128 rows][64]
   static constexpr int kTab = kS + kAtom;                            // two buffers of fp32 [4][128]
   static constexpr int kBar = kTab + 2 * 4 * kScChunk * 4;
-  static constexpr int kNumBars = 2 + 2 + 2 + 2 + 6;
+  static constexpr int kNumBars = 6 + 6 + 2 + 2 + 7;
   static constexpr int kTotal = kBar + kNumBars * 8 + 16;
 };
 static_assert(ScSmem::kTotal + 1024 <= 227 * 1024, "shared memory of a CTA");
 
 // columns of TMEM
-constexpr int kTmG = 0, kTmM = 256, kTmY1 = 320, kTmY2 = 384, kTmS = 448;
+constexpr int kTmG = 0, kTmY1 = 256, kTmY2 = 320, kTmS = 384;       // two buffers of G (M over it) and of dS
 
 __device__ __forceinline__ float sc_ex2(float x) {
   float y;
@@ -73,8 +77,10 @@ state_space_chunk_kernel(const __grid_constant__ CUtensorMap tmC, const __grid_c
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(sc_raw) + 1023) & ~uintptr_t(1023));
   const uint32_t base = smem_u32(smem);
   const uint32_t b0 = base + L::kBar;
-  const uint32_t bar_full = b0, bar_empty = b0 + 16, bar_g = b0 + 32, bar_tab = b0 + 48;      // [2] each
-  const uint32_t bar_m = b0 + 64, bar_y = b0 + 72, bar_yfree = b0 + 80, bar_xs = b0 + 88, bar_ds = b0 + 96, bar_s0 = b0 + 104;
+  const uint32_t bar_bfull = b0, bar_cfull = b0 + 16, bar_xfull = b0 + 32, bar_bempty = b0 + 48, bar_cempty = b0 + 64,
+                 bar_xempty = b0 + 80, bar_g = b0 + 96, bar_tab = b0 + 112;                    // [2] each
+  const uint32_t bar_m = b0 + 128, bar_y = b0 + 136, bar_yfree = b0 + 144, bar_xs = b0 + 152, bar_ds = b0 + 160, bar_s0 = b0 + 168,
+                 bar_y2 = b0 + 176;
   uint32_t* tmem_ptr_smem = reinterpret_cast<uint32_t*>(smem + L::kBar + L::kNumBars * 8);
   volatile int* abort_flag = reinterpret_cast<volatile int*>(tmem_ptr_smem + 1);
 
@@ -89,20 +95,24 @@ state_space_chunk_kernel(const __grid_constant__ CUtensorMap tmC, const __grid_c
   if (STATE_ONLY && end == seg.len) return;        // nobody starts from what the last span adds
   const int chunks = (end - off + kScChunk - 1) / kScChunk;
   const int g = h / (a.heads / a.groups);
-  const int ksteps_n = (a.n + 15) / 16;            // products over the state rows
   const int atoms = a.n > 64 ? 2 : 1;
 
   if (tid == 0) {
     for (int s = 0; s < 2; ++s) {
-      mbar_init(bar_full + 8 * s, 1);
-      mbar_init(bar_empty + 8 * s, STATE_ONLY ? 1 : 5);
+      mbar_init(bar_bfull + 8 * s, 1);
+      mbar_init(bar_cfull + 8 * s, 1);
+      mbar_init(bar_xfull + 8 * s, 1);
+      mbar_init(bar_bempty + 8 * s, 1);
+      mbar_init(bar_cempty + 8 * s, 1);
+      mbar_init(bar_xempty + 8 * s, 1);
       mbar_init(bar_g + 8 * s, 1);
       mbar_init(bar_tab + 8 * s, 1);
     }
     mbar_init(bar_m, 4);
     mbar_init(bar_y, 1);
     mbar_init(bar_yfree, 4);
-    mbar_init(bar_xs, 4);
+    mbar_init(bar_xs, 8);
+    mbar_init(bar_y2, 1);
     mbar_init(bar_ds, 1);
     mbar_init(bar_s0, 4);
     *abort_flag = 0;
@@ -127,73 +137,128 @@ state_space_chunk_kernel(const __grid_constant__ CUtensorMap tmC, const __grid_c
   tc_fence_after();
   const uint32_t tmem = *tmem_ptr_smem;
 
+  // xs of chunk i: half of a token's columns per thread of groups 2 and 3.  Gives exp(c_end) to group 2 and the row's exp(c_t) to
+  // group 3 (the tables are free once Y1 is done); false: a wait gave up.
+  auto scale_x = [&](int i, float& e) -> bool {
+    const float* tab = reinterpret_cast<const float*>(smem + L::kTab + (i & 1) * 4 * kScChunk * 4);
+    const uint8_t* x = smem + (i & 1) * L::kStage + L::kX;
+    if (!mbar_wait(bar_tab + 8 * (i & 1), (i >> 1) & 1, abort_flag, status, 71)) return false;
+    if (!mbar_wait(bar_xfull + 8 * (i & 1), (i >> 1) & 1, abort_flag, status, 72)) return false;
+    const int row = (warp & 3) * 32 + lane, q0 = warp < 12 ? 0 : kScCols / 16;
+    const float w = tab[3 * kScChunk + row];
+    e = sc_ex2(tab[warp < 12 ? kScChunk - 1 : row]);
+#pragma unroll
+    for (int q = 0; q < kScCols / 16; ++q) {
+      float v[8];
+      RcVec<__nv_bfloat16, 8>::load(reinterpret_cast<const __nv_bfloat16*>(x + sc_piece(row, q0 + q)), v);
+      uint32_t hi[4], lo[4];
+#pragma unroll
+      for (int k = 0; k < 4; ++k) sc_split(w * v[2 * k], w * v[2 * k + 1], hi[k], lo[k]);
+      *reinterpret_cast<uint4*>(smem + L::kXs + sc_piece(row, q0 + q)) = make_uint4(hi[0], hi[1], hi[2], hi[3]);
+      *reinterpret_cast<uint4*>(smem + L::kXs + L::kAtom + sc_piece(row, q0 + q)) = make_uint4(lo[0], lo[1], lo[2], lo[3]);
+    }
+    fence_proxy_async_smem();
+    __syncwarp();
+    if (lane == 0) mbar_arrive(bar_xs);
+    return true;
+  };
+
   if (warp == 0) {
     if (lane == 0) {
       // ------------------------------------------------------------------ TMA
       for (int i = 0; i < chunks; ++i) {
         const int s = i & 1, row = seg.first + off + i * kScChunk;
-        if (!mbar_wait(bar_empty + 8 * s, ((i >> 1) & 1) ^ 1, abort_flag, status, 61)) break;
-        const uint32_t st = base + s * L::kStage, bar = bar_full + 8 * s;
-        mbar_arrive_expect_tx(bar, L::kAtom * (1 + (STATE_ONLY ? 1 : 2) * atoms));
-        for (int k = 0; k < atoms; ++k) {
-          tma_load_4d(st + L::kB + k * L::kAtom, &tmB, k * 64, g, row, 0, bar);
-          if (!STATE_ONLY) tma_load_4d(st + L::kC + k * L::kAtom, &tmC, k * 64, g, row, 0, bar);
+        const uint32_t st = base + s * L::kStage, par = ((i >> 1) & 1) ^ 1;
+        if (!mbar_wait(bar_bempty + 8 * s, par, abort_flag, status, 61)) break;
+        mbar_arrive_expect_tx(bar_bfull + 8 * s, L::kAtom * atoms);
+        for (int k = 0; k < atoms; ++k) tma_load_4d(st + L::kB + k * L::kAtom, &tmB, k * 64, g, row, 0, bar_bfull + 8 * s);
+        if (!STATE_ONLY) {
+          if (!mbar_wait(bar_cempty + 8 * s, par, abort_flag, status, 78)) break;
+          mbar_arrive_expect_tx(bar_cfull + 8 * s, L::kAtom * atoms);
+          for (int k = 0; k < atoms; ++k) tma_load_4d(st + L::kC + k * L::kAtom, &tmC, k * 64, g, row, 0, bar_cfull + 8 * s);
         }
-        tma_load_4d(st + L::kX, &tmX, c0, h, row, 0, bar);
+        if (!mbar_wait(bar_xempty + 8 * s, par, abort_flag, status, 79)) break;
+        mbar_arrive_expect_tx(bar_xfull + 8 * s, L::kAtom);
+        tma_load_4d(st + L::kX, &tmX, c0, h, row, 0, bar_xfull + 8 * s);
       }
     }
   } else if (warp == 1) {
-    if (lane == 0) {
-      // ------------------------------------------------------------------ MMA
-      constexpr uint32_t idesc_g = umma_idesc_bf16(128, 128, 0, 0);
-      constexpr uint32_t idesc_y = umma_idesc_bf16(128, kScCols, 0, 1);       // A K-major (C) or in TMEM (M), B MN-major
-      constexpr uint32_t idesc_s = umma_idesc_bf16(128, kScCols, 1, 1);       // A = B^T: MN-major
-      auto issue_g = [&](int i) -> bool {
-        if (!mbar_wait(bar_full + 8 * (i & 1), (i >> 1) & 1, abort_flag, status, 62)) return false;
-        if (STATE_ONLY) return true;
-        tc_fence_after();
-        const uint32_t st = base + (i & 1) * L::kStage;
-        for (int k = 0; k < ksteps_n; ++k) {
-          const uint32_t o = (k >> 2) * L::kAtom + (k & 3) * 32;
-          umma_bf16_ss(tmem + kTmG + (i & 1) * 128, umma_smem_desc_sw128(st + L::kC + o, 16, 1024),
-                       umma_smem_desc_sw128(st + L::kB + o, 16, 1024), idesc_g, k != 0 ? 1u : 0u);
+    // -------------------------------------------------------------------- MMA: the whole warp walks, one elected lane issues
+    constexpr uint32_t idesc_g = umma_idesc_bf16(128, 128, 0, 0);
+    constexpr uint32_t idesc_y = umma_idesc_bf16(128, kScCols, 0, 1);         // A K-major (C) or in TMEM (M), B MN-major
+    constexpr uint32_t idesc_s = umma_idesc_bf16(128, kScCols, 1, 1);         // A = B^T: MN-major
+    // descriptors of the first stage and the first 16 of the contraction; an offset of o bytes is o / 16 in the address field
+    constexpr uint64_t kStage = L::kStage / 16, kAtom = L::kAtom / 16, kRows = 2048 / 16;
+    const uint64_t dC = umma_smem_desc_sw128(base + L::kC, 16, 1024), dB = umma_smem_desc_sw128(base + L::kB, 16, 1024);
+    const uint64_t dBt = umma_smem_desc_sw128(base + L::kB, L::kAtom, 1024), dX = umma_smem_desc_sw128(base + L::kX, L::kAtom, 1024);
+    const uint64_t dXs = umma_smem_desc_sw128(base + L::kXs, L::kAtom, 1024), dS0 = umma_smem_desc_sw128(base + L::kS, L::kAtom, 1024);
+    const int n = a.n;
+    auto issue_g = [&](int i) -> bool {
+      if (!mbar_wait(bar_bfull + 8 * (i & 1), (i >> 1) & 1, abort_flag, status, 62)) return false;
+      if (STATE_ONLY) return true;
+      if (!mbar_wait(bar_cfull + 8 * (i & 1), (i >> 1) & 1, abort_flag, status, 80)) return false;
+      tc_fence_after();
+      if (elect_one()) {
+        const uint64_t st = (i & 1) * kStage;
+        const uint32_t d = tmem + kTmG + (i & 1) * 128;
+#pragma unroll
+        for (int k = 0; k < 8; ++k) {
+          if (k * 16 >= n) break;                  // the rest of the columns is zero
+          const uint64_t o = st + (k >> 2) * kAtom + (k & 3) * 2;
+          umma_bf16_ss(d, dC + o, dB + o, idesc_g, k != 0 ? 1u : 0u);
         }
         umma_commit(bar_g + 8 * (i & 1));
-        return true;
-      };
-      bool ok = issue_g(0);
-      for (int i = 0; i < chunks && ok; ++i) {
-        const uint32_t st = base + (i & 1) * L::kStage;
-        if (i + 1 < chunks && !issue_g(i + 1)) break;       // its buffer's last reader has arrived on bar_m
-        if (!STATE_ONLY) {
-          if (!mbar_wait(bar_s0, i & 1, abort_flag, status, 63)) break;
-          if (!mbar_wait(bar_yfree, (i & 1) ^ 1, abort_flag, status, 64)) break;
-          tc_fence_after();
-          for (int k = 0; k < ksteps_n; ++k)
-            umma_bf16_ss(tmem + kTmY2, umma_smem_desc_sw128(st + L::kC + (k >> 2) * L::kAtom + (k & 3) * 32, 16, 1024),
-                         umma_smem_desc_sw128(base + L::kS + k * 2048, L::kAtom, 1024), idesc_y, k != 0 ? 1u : 0u);
-        }
-        if (!mbar_wait(bar_xs, i & 1, abort_flag, status, 65)) break;
-        tc_fence_after();
+      }
+      __syncwarp();
+      return true;
+    };
+    bool ok = issue_g(0);
+    for (int i = 0; i < chunks && ok; ++i) {
+      const uint64_t st = (i & 1) * kStage;
+      if (!mbar_wait(bar_xs, i & 1, abort_flag, status, 63)) break;
+      tc_fence_after();
+      if (elect_one()) {
+        const uint32_t d = tmem + kTmS + (i & 1) * 64;
 #pragma unroll
         for (int half = 0; half < 2; ++half)
 #pragma unroll
           for (int k = 0; k < kScChunk / 16; ++k)
-            umma_bf16_ss(tmem + kTmS, umma_smem_desc_sw128(st + L::kB + k * 2048, L::kAtom, 1024),
-                         umma_smem_desc_sw128(base + L::kXs + half * L::kAtom + k * 2048, L::kAtom, 1024), idesc_s,
-                         (half | k) != 0 ? 1u : 0u);
+            umma_bf16_ss(d, dBt + st + k * kRows, dXs + half * kAtom + k * kRows, idesc_s, (half | k) != 0 ? 1u : 0u);
         umma_commit(bar_ds);
+        umma_commit(bar_bempty + 8 * (i & 1));
+      }
+      __syncwarp();
+      if (!STATE_ONLY) {
+        if (!mbar_wait(bar_s0, i & 1, abort_flag, status, 64)) break;
+        if (!mbar_wait(bar_yfree, (i & 1) ^ 1, abort_flag, status, 65)) break;
+        tc_fence_after();
+        if (elect_one()) {
+#pragma unroll
+          for (int k = 0; k < 8; ++k) {
+            if (k * 16 >= n) break;
+            umma_bf16_ss(tmem + kTmY2, dC + st + (k >> 2) * kAtom + (k & 3) * 2, dS0 + k * kRows, idesc_y, k != 0 ? 1u : 0u);
+          }
+          umma_commit(bar_y2);
+          umma_commit(bar_cempty + 8 * (i & 1));
+        }
+        __syncwarp();
+      }
+      if (i + 1 < chunks && !issue_g(i + 1)) break;         // behind Y1 of the chunk before, which read its buffer
+      if (!STATE_ONLY) {
+        if (!mbar_wait(bar_m, i & 1, abort_flag, status, 66)) break;
+        tc_fence_after();
+      }
+      if (elect_one()) {
         if (!STATE_ONLY) {
-          if (!mbar_wait(bar_m, i & 1, abort_flag, status, 66)) break;
-          tc_fence_after();
+          const uint32_t m = tmem + kTmG + (i & 1) * 128;
 #pragma unroll
           for (int k = 0; k < kScChunk / 16; ++k)
-            umma_bf16_ts(tmem + kTmY1, tmem + kTmM + k * 8, umma_smem_desc_sw128(st + L::kX + k * 2048, L::kAtom, 1024), idesc_y,
-                         k != 0 ? 1u : 0u);
+            umma_bf16_ts(tmem + kTmY1, m + k * 8, dX + st + k * kRows, idesc_y, k != 0 ? 1u : 0u);
           umma_commit(bar_y);
         }
-        umma_commit(bar_empty + 8 * (i & 1));
+        umma_commit(bar_xempty + 8 * (i & 1));
       }
+      __syncwarp();
     }
   } else if (warp == 2) {
     // -------------------------------------------------------------------- factors of a chunk, four tokens per lane
@@ -224,7 +289,7 @@ state_space_chunk_kernel(const __grid_constant__ CUtensorMap tmC, const __grid_c
       const float before = run - c[3];
       const float c_end = __shfl_sync(0xffffffffu, run, 31), c_blk = __shfl_sync(0xffffffffu, run, lane | 7);
       total += c_end;
-      if (!mbar_wait(bar_empty + 8 * (i & 1), ((i >> 1) & 1) ^ 1, abort_flag, status, 67)) break;
+      if (!mbar_wait(bar_xempty + 8 * (i & 1), ((i >> 1) & 1) ^ 1, abort_flag, status, 67)) break;
       float4* tab = reinterpret_cast<float4*>(smem + L::kTab + (i & 1) * 4 * kScChunk * 4) + lane;
       float v[4][4];
 #pragma unroll
@@ -245,21 +310,18 @@ state_space_chunk_kernel(const __grid_constant__ CUtensorMap tmC, const __grid_c
       // ------------------------------------------------------------------ M, one row per thread
       const int wq = warp & 3, row = wq * 32 + lane;
       const uint32_t lane_off = static_cast<uint32_t>(wq * 32) << 16;
-      const uint32_t tm = tmem + kTmM + lane_off;
-      {
-        const uint32_t zero[16] = {0u, 0u, 0u, 0u, 0u, 0u, 0u, 0u, 0u, 0u, 0u, 0u, 0u, 0u, 0u, 0u};
-        for (int b = wq + 1; b < 4; ++b) tmem_st_32x16(tm + b * 16, zero);     // above the diagonal, for good
-      }
+      const float dskip = a.D[h];
+      const uint32_t zero[16] = {0u, 0u, 0u, 0u, 0u, 0u, 0u, 0u, 0u, 0u, 0u, 0u, 0u, 0u, 0u, 0u};
       for (int i = 0; i < chunks; ++i) {
         const float* tab = reinterpret_cast<const float*>(smem + L::kTab + (i & 1) * 4 * kScChunk * 4);
         if (!mbar_wait(bar_tab + 8 * (i & 1), (i >> 1) & 1, abort_flag, status, 68)) break;
         if (!mbar_wait(bar_g + 8 * (i & 1), (i >> 1) & 1, abort_flag, status, 69)) break;
-        if (!mbar_wait(bar_y, (i & 1) ^ 1, abort_flag, status, 70)) break;     // Y1 of the chunk before has read M
         tc_fence_after();
+        const uint32_t tm = tmem + kTmG + (i & 1) * 128 + lane_off;            // block b's M (16 columns) never reaches past block b
         const float ct = tab[row];
         for (int b = 0; b <= wq; ++b) {
           uint32_t r[32];
-          tmem_ld_32x32(tmem + kTmG + (i & 1) * 128 + lane_off + b * 32, r);
+          tmem_ld_32x32(tm + b * 32, r);
           tmem_ld_wait();
           uint32_t packed[16];
           if (b < wq) {
@@ -277,16 +339,17 @@ state_space_chunk_kernel(const __grid_constant__ CUtensorMap tmC, const __grid_c
 #pragma unroll
             for (int q = 0; q < 8; ++q) {
               const float4 c = cs[q], d = ds[q];
-              const float m0 = 4 * q <= lane ? __uint_as_float(r[4 * q]) * d.x * sc_ex2(ct - c.x) : 0.f;
-              const float m1 = 4 * q + 1 <= lane ? __uint_as_float(r[4 * q + 1]) * d.y * sc_ex2(ct - c.y) : 0.f;
-              const float m2 = 4 * q + 2 <= lane ? __uint_as_float(r[4 * q + 2]) * d.z * sc_ex2(ct - c.z) : 0.f;
-              const float m3 = 4 * q + 3 <= lane ? __uint_as_float(r[4 * q + 3]) * d.w * sc_ex2(ct - c.w) : 0.f;
+              const float m0 = 4 * q <= lane ? fmaf(__uint_as_float(r[4 * q]) * d.x, sc_ex2(ct - c.x), 4 * q == lane ? dskip : 0.f) : 0.f;
+              const float m1 = 4 * q + 1 <= lane ? fmaf(__uint_as_float(r[4 * q + 1]) * d.y, sc_ex2(ct - c.y), 4 * q + 1 == lane ? dskip : 0.f) : 0.f;
+              const float m2 = 4 * q + 2 <= lane ? fmaf(__uint_as_float(r[4 * q + 2]) * d.z, sc_ex2(ct - c.z), 4 * q + 2 == lane ? dskip : 0.f) : 0.f;
+              const float m3 = 4 * q + 3 <= lane ? fmaf(__uint_as_float(r[4 * q + 3]) * d.w, sc_ex2(ct - c.w), 4 * q + 3 == lane ? dskip : 0.f) : 0.f;
               packed[2 * q] = pack_bf16x2(m0, m1);
               packed[2 * q + 1] = pack_bf16x2(m2, m3);
             }
           }
           tmem_st_32x16(tm + b * 16, packed);
         }
+        for (int b = wq + 1; b < 4; ++b) tmem_st_32x16(tm + b * 16, zero);     // above the diagonal
         tmem_st_wait();
         tc_fence_before();
         __syncwarp();
@@ -294,7 +357,7 @@ state_space_chunk_kernel(const __grid_constant__ CUtensorMap tmC, const __grid_c
       }
     }
   } else if (warp >= 8 && warp < 12) {
-    // -------------------------------------------------------------------- xs and the state: token row, then state row per thread
+    // -------------------------------------------------------------------- xs and the state
     const int row = (warp & 3) * 32 + lane;
     const uint32_t ts = tmem + kTmS + (static_cast<uint32_t>((warp & 3) * 32) << 16);
     const long long state_n = static_cast<long long>(a.n) * a.p;
@@ -332,41 +395,29 @@ state_space_chunk_kernel(const __grid_constant__ CUtensorMap tmC, const __grid_c
       __syncwarp();
       if (lane == 0) mbar_arrive(bar_s0);
     };
+    float e_end = 1.f, e_next = 1.f;
+    bool ok = scale_x(0, e_end);
     if (!STATE_ONLY) publish();
-    bool ok = true;
-    for (int i = 0; i < chunks; ++i) {
-      const float* tab = reinterpret_cast<const float*>(smem + L::kTab + (i & 1) * 4 * kScChunk * 4);
-      const uint8_t* x = smem + (i & 1) * L::kStage + L::kX;
-      ok = mbar_wait(bar_tab + 8 * (i & 1), (i >> 1) & 1, abort_flag, status, 71) &&
-           mbar_wait(bar_full + 8 * (i & 1), (i >> 1) & 1, abort_flag, status, 72);
-      if (!ok) break;
-      const float w = tab[3 * kScChunk + row], e_end = sc_ex2(tab[kScChunk - 1]);
-#pragma unroll
-      for (int q = 0; q < kScCols / 8; ++q) {
-        float v[8];
-        RcVec<__nv_bfloat16, 8>::load(reinterpret_cast<const __nv_bfloat16*>(x + sc_piece(row, q)), v);
-        uint32_t hi[4], lo[4];
-#pragma unroll
-        for (int k = 0; k < 4; ++k) sc_split(w * v[2 * k], w * v[2 * k + 1], hi[k], lo[k]);
-        *reinterpret_cast<uint4*>(smem + L::kXs + sc_piece(row, q)) = make_uint4(hi[0], hi[1], hi[2], hi[3]);
-        *reinterpret_cast<uint4*>(smem + L::kXs + L::kAtom + sc_piece(row, q)) = make_uint4(lo[0], lo[1], lo[2], lo[3]);
-      }
-      fence_proxy_async_smem();
-      __syncwarp();
-      if (lane == 0) mbar_arrive(bar_xs);
+    for (int i = 0; i < chunks && ok; ++i) {
       ok = mbar_wait(bar_ds, i & 1, abort_flag, status, 73);
       if (!ok) break;
+      if (i + 1 < chunks && !(ok = scale_x(i + 1, e_next))) break;
       tc_fence_after();
 #pragma unroll
       for (int q = 0; q < kScCols / 32; ++q) {
         uint32_t r[32];
-        tmem_ld_32x32(ts + q * 32, r);
+        tmem_ld_32x32(ts + (i & 1) * 64 + q * 32, r);
         tmem_ld_wait();
 #pragma unroll
         for (int j = 0; j < 32; ++j) S[q * 32 + j] = fmaf(S[q * 32 + j], e_end, __uint_as_float(r[j]));
       }
       tc_fence_before();
-      if (!STATE_ONLY && i + 1 < chunks) publish();
+      e_end = e_next;
+      if (!STATE_ONLY && i + 1 < chunks) {
+        ok = mbar_wait(bar_y2, i & 1, abort_flag, status, 77);       // the copy has been read
+        if (!ok) break;
+        publish();
+      }
     }
     if (ok && live && (STATE_ONLY || end == seg.len)) {
       float* dst = STATE_ONLY ? span_state + (static_cast<long long>(tile) * a.heads + h) * state_n : slot;
@@ -375,18 +426,18 @@ state_space_chunk_kernel(const __grid_constant__ CUtensorMap tmC, const __grid_c
         if (j < cols) *reinterpret_cast<float4*>(dst + at + j) = make_float4(S[j], S[j + 1], S[j + 2], S[j + 3]);
     }
   } else if (warp >= 12) {
-    if (!STATE_ONLY) {
-      // ------------------------------------------------------------------ y, one row per thread
-      const int row = (warp & 3) * 32 + lane;
-      const uint32_t ty = tmem + (static_cast<uint32_t>((warp & 3) * 32) << 16);
-      const float dskip = a.D[h];
-      const int cols = min(kScCols, a.p - c0);
-      for (int i = 0; i < chunks; ++i) {
-        const float* tab = reinterpret_cast<const float*>(smem + L::kTab + (i & 1) * 4 * kScChunk * 4);
-        const uint8_t* x = smem + (i & 1) * L::kStage + L::kX;
-        if (!mbar_wait(bar_tab + 8 * (i & 1), (i >> 1) & 1, abort_flag, status, 74)) break;
-        if (!mbar_wait(bar_full + 8 * (i & 1), (i >> 1) & 1, abort_flag, status, 75)) break;
-        const float e = sc_ex2(tab[row]);
+    // -------------------------------------------------------------------- xs and y, one row per thread
+    const int row = (warp & 3) * 32 + lane;
+    const uint32_t ty = tmem + (static_cast<uint32_t>((warp & 3) * 32) << 16);
+    const int cols = min(kScCols, a.p - c0);
+    float e = 1.f, e_next = 1.f;
+    bool ok = scale_x(0, e);
+    for (int i = 0; i < chunks && ok; ++i) {
+      if (i + 1 < chunks) {
+        ok = mbar_wait(bar_ds, i & 1, abort_flag, status, 74) && scale_x(i + 1, e_next);
+        if (!ok) break;
+      }
+      if (!STATE_ONLY) {
         if (!mbar_wait(bar_y, i & 1, abort_flag, status, 76)) break;
         tc_fence_after();
         uint32_t packed[kScCols / 2];
@@ -397,22 +448,14 @@ state_space_chunk_kernel(const __grid_constant__ CUtensorMap tmC, const __grid_c
           tmem_ld_32x32(ty + kTmY2 + q * 32, y2);
           tmem_ld_wait();
 #pragma unroll
-          for (int k = 0; k < 4; ++k) {
-            float v[8];
-            RcVec<__nv_bfloat16, 8>::load(reinterpret_cast<const __nv_bfloat16*>(x + sc_piece(row, q * 4 + k)), v);
-#pragma unroll
-            for (int j = 0; j < 8; ++j)
-              v[j] = fmaf(dskip, v[j], fmaf(e, __uint_as_float(y2[8 * k + j]), __uint_as_float(y1[8 * k + j])));
-#pragma unroll
-            for (int j = 0; j < 4; ++j) packed[q * 16 + k * 4 + j] = pack_bf16x2(v[2 * j], v[2 * j + 1]);
-          }
+          for (int j = 0; j < 16; ++j)
+            packed[q * 16 + j] = pack_bf16x2(fmaf(e, __uint_as_float(y2[2 * j]), __uint_as_float(y1[2 * j])),
+                                             fmaf(e, __uint_as_float(y2[2 * j + 1]), __uint_as_float(y1[2 * j + 1])));
         }
         tc_fence_before();
         __syncwarp();
-        if (lane == 0) {
-          mbar_arrive(bar_yfree);
-          mbar_arrive(bar_empty + 8 * (i & 1));
-        }
+        if (lane == 0) mbar_arrive(bar_yfree);
+        e = e_next;
         const int t = off + i * kScChunk + row;
         if (t < end) {
           __nv_bfloat16* out = reinterpret_cast<__nv_bfloat16*>(a.y) + static_cast<long long>(seg.first + t) * a.ld_y +
