@@ -26,12 +26,16 @@ constexpr int kDcChunk = 64;
 constexpr float kDcUnitEps = 1e-6f;
 constexpr float kDcLog2e = 1.4426950408889634f;
 
-// scratch of one (chunk, head): A T (bf16 [64, 64]), W (bf16 [64, DK], high and low half), then fp32 factors
-constexpr int kDcMat = kDcChunk * kDcChunk * 2;
+// scratch of one (chunk, head), rows padded as the second kernel wants them in shared memory (it fetches the block as a whole):
+// A T (bf16 [64][72]), W (bf16 [64][DK + 8], high and low half), then fp32 factors
+constexpr int kDcMPitch = kDcChunk + 8;
+constexpr int kDcMat = kDcChunk * kDcMPitch * 2;
 constexpr int kDcFactors = 4;              // [64] each: beta, key read-out, query read-out, and one with exp(c_end) in [0]
-__host__ __device__ constexpr int dc_scratch(int DK) { return kDcMat + 2 * kDcChunk * DK * 2 + kDcFactors * kDcChunk * 4; }
+__host__ __device__ constexpr int dc_half(int DK) { return kDcChunk * (DK + 8) * 2; }
+__host__ __device__ constexpr int dc_scratch(int DK) { return kDcMat + 2 * dc_half(DK) + kDcFactors * kDcChunk * 4; }
 
-// ---- first kernel: one CTA (4 warps) per chunk and head
+// ---- first kernel: one CTA (8 warps) per chunk and head
+constexpr int kDpThreads = 256;
 template <int DK>
 struct DcPrepSmem {
   static constexpr int kPitch = DK + 8, kLPitch = kDcChunk + 4;
@@ -42,12 +46,13 @@ struct DcPrepSmem {
   static constexpr int kT = kL + 2 * kDcChunk * kTPitch * 2;         // fp32 [64][68]
   static constexpr int kW = kT + kDcChunk * kLPitch * 4;             // fp32 [48][20] products of blocks
   static constexpr int kF = kW + 48 * 20 * 4;                        // fp32 [4][64]: c, beta, 1 / |k|, scale / |q|
-  static constexpr int kW2 = kF + 4 * kDcChunk * 4;                  // staging of W's low half
-  static constexpr int kTotal = kW2 + kDcChunk * kPitch * 2;
+  static constexpr int kTotal = kF + 4 * kDcChunk * 4;
+  // W is staged before it leaves: the high half over the queries, the low half over T
+  static_assert(kDcChunk * kPitch * 2 <= kW - kT, "staging of the low half");
 };
 
 template <int DK>
-__global__ void __launch_bounds__(128)
+__global__ void __launch_bounds__(kDpThreads, 2)
 delta_rule_prepare_kernel(const RbDeltaRuleArgs a) {
   using L = DcPrepSmem<DK>;
   constexpr int P = L::kPitch, LP = L::kLPitch;
@@ -60,6 +65,7 @@ delta_rule_prepare_kernel(const RbDeltaRuleArgs a) {
   float *beta = cum + kDcChunk, *rk = beta + kDcChunk, *rq = rk + kDcChunk;
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int gq = lane >> 2, tq = lane & 3;
+  const int wr = warp & 3, side = warp >> 2;       // rows wr 16 .. + 16 of the products k . k (side 0) or q . k (side 1)
   const int h = blockIdx.x, tile = blockIdx.y;
   const RcSegment seg = rc_segment(a.segments, a.tiles[2 * tile], a.num_slots);
   const int off = a.tiles[2 * tile + 1];
@@ -68,7 +74,7 @@ delta_rule_prepare_kernel(const RbDeltaRuleArgs a) {
   const int g = h / (a.heads / a.kv_heads);
   const __nv_bfloat16* rows = reinterpret_cast<const __nv_bfloat16*>(a.qkv) + static_cast<long long>(seg.first + off) * a.ld_qkv;
   const long long offQ = static_cast<long long>(g) * a.dk, offK = static_cast<long long>(a.kv_heads + g) * a.dk;
-  for (int i = tid; i < kDcChunk * (DK / 8); i += 128) {
+  for (int i = tid; i < kDcChunk * (DK / 8); i += kDpThreads) {
     const int r = i / (DK / 8), c = (i - r * (DK / 8)) * 8;
     const bool ok = r < m_rows && c < a.dk;
     const __nv_bfloat16* src = rows + (ok ? r * a.ld_qkv + c : 0);
@@ -95,66 +101,62 @@ delta_rule_prepare_kernel(const RbDeltaRuleArgs a) {
     cum[2 * lane] = run - s[1];
     cum[2 * lane + 1] = run;
   }
-  for (int i = tid; i < kDcChunk * LP; i += 128) T[i] = 0.f;
+  for (int i = tid; i < kDcChunk * LP; i += kDpThreads) T[i] = 0.f;
   wm_cp_wait<0>();
   __syncthreads();
-  {                                                // norms: two threads per row, one for the query and one for the key
-    const int r = tid & 63;
-    const __nv_bfloat16* row = reinterpret_cast<const __nv_bfloat16*>(dp_smem + (tid < 64 ? L::kQ : L::kK)) + r * P;
+  {                                                // norms: two threads per row of either
+    const int r = (tid & 127) >> 1, half = tid & 1;
+    const __nv_bfloat16* row = reinterpret_cast<const __nv_bfloat16*>(dp_smem + (tid < 128 ? L::kQ : L::kK)) + r * P + half * (DK / 2);
     float s = 0.f;
 #pragma unroll 4
-    for (int c = 0; c < DK; c += 8) {
+    for (int c = 0; c < DK / 2; c += 8) {
       float v[8];
       RcVec<__nv_bfloat16, 8>::load(row + c, v);
 #pragma unroll
       for (int i = 0; i < 8; ++i) s = fmaf(v[i], v[i], s);
     }
+    s += __shfl_xor_sync(0xffffffffu, s, 1);
     const float inv = 1.f / sqrtf(s + kDcUnitEps);
-    if (tid < 64) rq[r] = inv * rsqrtf(static_cast<float>(a.dk));
-    else rk[r] = inv;
+    if (half == 0) {
+      if (tid < 128) rq[r] = inv * rsqrtf(static_cast<float>(a.dk));
+      else rk[r] = inv;
+    }
   }
   __syncthreads();
   uint8_t* scratch = reinterpret_cast<uint8_t*>(a.scratch) + (static_cast<long long>(tile) * a.heads + h) * dc_scratch(DK);
-  // ---- L and A: rows warp 16 .. + 16; A stays in registers as the A operand of A T, high and low half
+  // ---- L (side 0) and A (side 1); A stays in registers as the A operand of A T, high and low half
   uint32_t ah[4][4], al[4][4];
   {
-    uint32_t kf[DK / 16][4], qf[DK / 16][4];
+    uint32_t xf[DK / 16][4];
 #pragma unroll
-    for (int k = 0; k < DK / 16; ++k) {
-      wm_ldsm_x4(wm_a(sK, P, warp * 16, k * 16, lane), kf[k]);
-      wm_ldsm_x4(wm_a(sQ, P, warp * 16, k * 16, lane), qf[k]);
-    }
+    for (int k = 0; k < DK / 16; ++k) wm_ldsm_x4(wm_a(side ? sQ : sK, P, wr * 16, k * 16, lane), xf[k]);
 #pragma unroll
     for (int sb = 0; sb < 4; ++sb) {
-      float kk[2][4], qk[2][4];
+      if (sb > wr) break;                          // what lies above the diagonal is never read
+      float acc[2][4];
 #pragma unroll
-      for (int i = 0; i < 2; ++i)
+      for (int i = 0; i < 2; ++i) acc[i][0] = acc[i][1] = acc[i][2] = acc[i][3] = 0.f;
 #pragma unroll
-        for (int j = 0; j < 4; ++j) kk[i][j] = qk[i][j] = 0.f;
-      if (sb <= warp) {
-#pragma unroll
-        for (int k = 0; k < DK / 16; ++k) {
-          uint32_t b[4];
-          wm_ldsm_x4(wm_b(sK, P, sb * 16, k * 16, lane), b);
-          wm_mma(kk[0], kf[k], b[0], b[1]);
-          wm_mma(kk[1], kf[k], b[2], b[3]);
-          wm_mma(qk[0], qf[k], b[0], b[1]);
-          wm_mma(qk[1], qf[k], b[2], b[3]);
-        }
+      for (int k = 0; k < DK / 16; ++k) {
+        uint32_t b[4];
+        wm_ldsm_x4(wm_b(sK, P, sb * 16, k * 16, lane), b);
+        wm_mma(acc[0], xf[k], b[0], b[1]);
+        wm_mma(acc[1], xf[k], b[2], b[3]);
       }
 #pragma unroll
       for (int i = 0; i < 2; ++i)
 #pragma unroll
         for (int r = 0; r < 2; ++r) {
-          const int t = warp * 16 + gq + 8 * r, s = sb * 16 + i * 8 + 2 * tq;
+          const int t = wr * 16 + gq + 8 * r, s = sb * 16 + i * 8 + 2 * tq;
           float v[2];
 #pragma unroll
-          for (int j = 0; j < 2; ++j) {
-            const float d = s + j <= t ? wm_ex2(cum[t] - cum[s + j]) * rk[s + j] : 0.f;
-            Lm[t * LP + s + j] = s + j < t ? beta[t] * rk[t] * d * kk[i][2 * r + j] : 0.f;
-            v[j] = rq[t] * d * qk[i][2 * r + j];
+          for (int j = 0; j < 2; ++j) v[j] = s + j <= t ? wm_ex2(cum[t] - cum[s + j]) * rk[s + j] * acc[i][2 * r + j] : 0.f;
+          if (side == 0) {
+            const float f = beta[t] * rk[t];
+            *reinterpret_cast<float2*>(Lm + t * LP + s) = make_float2(s < t ? f * v[0] : 0.f, s + 1 < t ? f * v[1] : 0.f);
+          } else {
+            wm_split(rq[t] * v[0], rq[t] * v[1], ah[sb][2 * i + r], al[sb][2 * i + r]);
           }
-          wm_split(v[0], v[1], ah[sb][2 * i + r], al[sb][2 * i + r]);
         }
     }
   }
@@ -195,25 +197,23 @@ delta_rule_prepare_kernel(const RbDeltaRuleArgs a) {
   };
 #pragma unroll
   for (int d = 1; d < 4; ++d) {
+    const int r = tid >> 4, c = tid & 15;          // one entry of every block per thread
 #pragma unroll
-    for (int e = 0; e < (4 - d) * 2; ++e) {        // 128 entries at a time
-      const int blk = e >> 1, r = (e & 1) * 8 + (tid >> 4), c = tid & 15, i = blk + d;      // block row i, block column blk
+    for (int blk = 0; blk < 4 - d; ++blk) {        // block row blk + d, block column blk
       float v = 0.f;
 #pragma unroll
-      for (int k = 0; k < d; ++k) v += dot16(Lm + (i * 16 + r) * LP + (blk + k) * 16, T + (blk + k) * 16 * LP + blk * 16 + c, LP);
+      for (int k = 0; k < d; ++k) v += dot16(Lm + ((blk + d) * 16 + r) * LP + (blk + k) * 16, T + (blk + k) * 16 * LP + blk * 16 + c, LP);
       W[(blk * 16 + r) * 20 + c] = v;
     }
     __syncthreads();
 #pragma unroll
-    for (int e = 0; e < (4 - d) * 2; ++e) {
-      const int blk = e >> 1, r = (e & 1) * 8 + (tid >> 4), c = tid & 15, i = blk + d;
-      T[(i * 16 + r) * LP + blk * 16 + c] = -dot16(T + (i * 16 + r) * LP + i * 16, W + blk * 16 * 20 + c, 20);
-    }
+    for (int blk = 0; blk < 4 - d; ++blk)
+      T[((blk + d) * 16 + r) * LP + blk * 16 + c] = -dot16(T + ((blk + d) * 16 + r) * LP + (blk + d) * 16, W + blk * 16 * 20 + c, 20);
     __syncthreads();
   }
   const uint32_t sT = smem_u32(dp_smem) + L::kL;
   constexpr int TP = L::kTPitch;
-  for (int e = tid; e < kDcChunk * kDcChunk / 8; e += 128) {
+  for (int e = tid; e < kDcChunk * kDcChunk / 8; e += kDpThreads) {
     const int r = e >> 3, c = (e & 7) * 8;
     uint32_t hi[4], lo[4];
 #pragma unroll
@@ -221,9 +221,28 @@ delta_rule_prepare_kernel(const RbDeltaRuleArgs a) {
     *reinterpret_cast<uint4*>(dp_smem + L::kL + (r * TP + c) * 2) = make_uint4(hi[0], hi[1], hi[2], hi[3]);
     *reinterpret_cast<uint4*>(dp_smem + L::kL + ((kDcChunk + r) * TP + c) * 2) = make_uint4(lo[0], lo[1], lo[2], lo[3]);
   }
-  __syncthreads();
-  // ---- A T: rows warp 16 .. + 16
+  // ---- W = T^T diag(1 / |k| exp(c_end - c)) K: rows (columns of T) wr 16 .. + 16; T^T, scaled, is the A operand
+  uint32_t th[4][4], tl[4][4];
   {
+    const float c_end = cum[kDcChunk - 1];
+#pragma unroll
+    for (int k = 0; k < 4; ++k) {
+      if (k < wr) continue;                        // T is lower triangular
+#pragma unroll
+      for (int half = 0; half < 2; ++half) {       // columns k 16 + 8 half + 2 tq (+ 1)
+        const int t = k * 16 + half * 8 + 2 * tq;
+        const float w0 = rk[t] * wm_ex2(c_end - cum[t]), w1 = rk[t + 1] * wm_ex2(c_end - cum[t + 1]);
+#pragma unroll
+        for (int r = 0; r < 2; ++r) {
+          const int s = wr * 16 + gq + 8 * r;
+          wm_split(w0 * T[t * LP + s], w1 * T[(t + 1) * LP + s], th[k][2 * half + r], tl[k][2 * half + r]);
+        }
+      }
+    }
+  }
+  __syncthreads();                                 // T is free: staging of W's low half
+  // ---- A T: rows wr 16 .. + 16
+  if (side == 1) {
     __nv_bfloat16* out = reinterpret_cast<__nv_bfloat16*>(scratch);
 #pragma unroll
     for (int nb = 0; nb < 4; ++nb) {
@@ -232,7 +251,7 @@ delta_rule_prepare_kernel(const RbDeltaRuleArgs a) {
       for (int i = 0; i < 2; ++i) acc[i][0] = acc[i][1] = acc[i][2] = acc[i][3] = 0.f;
 #pragma unroll
       for (int k = 0; k < 4; ++k) {
-        if (k < nb || k > warp) continue;          // both are lower triangular
+        if (k < nb || k > wr) continue;            // both are lower triangular
         uint32_t b[4], bl[4];
         wm_ldsm_x4_t(wm_b_t(sT, TP, nb * 16, k * 16, lane), b);
         wm_ldsm_x4_t(wm_b_t(sT + kDcChunk * TP * 2, TP, nb * 16, k * 16, lane), bl);
@@ -247,37 +266,22 @@ delta_rule_prepare_kernel(const RbDeltaRuleArgs a) {
       for (int i = 0; i < 2; ++i)
 #pragma unroll
         for (int r = 0; r < 2; ++r)
-          *reinterpret_cast<uint32_t*>(out + (warp * 16 + gq + 8 * r) * kDcChunk + nb * 16 + i * 8 + 2 * tq) =
+          *reinterpret_cast<uint32_t*>(out + (wr * 16 + gq + 8 * r) * kDcMPitch + nb * 16 + i * 8 + 2 * tq) =
               pack_bf16x2(acc[i][2 * r], acc[i][2 * r + 1]);
     }
   }
-  // ---- W = T^T diag(1 / |k| exp(c_end - c)) K: rows (columns of T) warp 16 .. + 16
   {
-    const float c_end = cum[kDcChunk - 1];
-    uint32_t th[4][4], tl[4][4];                   // scaled T^T as the A operand
-#pragma unroll
-    for (int k = 0; k < 4; ++k) {
-      if (k < warp) continue;                      // T is lower triangular
-#pragma unroll
-      for (int half = 0; half < 2; ++half) {       // columns k 16 + 8 half + 2 tq (+ 1)
-        const int t = k * 16 + half * 8 + 2 * tq;
-        const float w0 = rk[t] * wm_ex2(c_end - cum[t]), w1 = rk[t + 1] * wm_ex2(c_end - cum[t + 1]);
-#pragma unroll
-        for (int r = 0; r < 2; ++r) {
-          const int s = warp * 16 + gq + 8 * r;
-          wm_split(w0 * T[t * LP + s], w1 * T[(t + 1) * LP + s], th[k][2 * half + r], tl[k][2 * half + r]);
-        }
-      }
-    }
-    __nv_bfloat16* out = reinterpret_cast<__nv_bfloat16*>(scratch + kDcMat);
-#pragma unroll
-    for (int nb = 0; nb < DK / 16; ++nb) {
+    // columns: the first five eighths by side 0, the rest by side 1
+    constexpr int kCut = DK / 16 * 5 / 8;
+    const int nb0 = side ? kCut : 0, nb1 = side ? DK / 16 : kCut;
+#pragma unroll 1
+    for (int nb = nb0; nb < nb1; ++nb) {
       float acc[2][4];
 #pragma unroll
       for (int i = 0; i < 2; ++i) acc[i][0] = acc[i][1] = acc[i][2] = acc[i][3] = 0.f;
 #pragma unroll
       for (int k = 0; k < 4; ++k) {
-        if (k < warp) continue;
+        if (k < wr) continue;
         uint32_t b[4];
         wm_ldsm_x4_t(wm_b_t(sK, P, nb * 16, k * 16, lane), b);
         wm_mma(acc[0], th[k], b[0], b[1]);
@@ -291,20 +295,22 @@ delta_rule_prepare_kernel(const RbDeltaRuleArgs a) {
         for (int r = 0; r < 2; ++r) {
           uint32_t hi, lo;
           wm_split(acc[i][2 * r], acc[i][2 * r + 1], hi, lo);
-          const int at = ((warp * 16 + gq + 8 * r) * P + nb * 16 + i * 8 + 2 * tq) * 2;
-          *reinterpret_cast<uint32_t*>(dp_smem + L::kQ + at) = hi;             // the queries' tile is free
-          *reinterpret_cast<uint32_t*>(dp_smem + L::kW2 + at) = lo;
+          const int at = ((wr * 16 + gq + 8 * r) * P + nb * 16 + i * 8 + 2 * tq) * 2;
+          *reinterpret_cast<uint32_t*>(dp_smem + L::kQ + at) = hi;
+          *reinterpret_cast<uint32_t*>(dp_smem + L::kT + at) = lo;
         }
     }
-    __syncwarp();                                  // every warp copies its own rows
-    for (int e = lane; e < 2 * 16 * (DK / 8); e += 32) {
-      const int half = e / (16 * (DK / 8)), q = e - half * 16 * (DK / 8), r = warp * 16 + q / (DK / 8), c = (q % (DK / 8)) * 8;
-      *reinterpret_cast<uint4*>(out + (half * kDcChunk + r) * DK + c) =
-          *reinterpret_cast<const uint4*>(dp_smem + (half ? L::kW2 : L::kQ) + (r * P + c) * 2);
+    __syncwarp();                                  // every warp copies its own rows and columns
+    uint8_t* out = scratch + kDcMat;
+    const int pieces = (nb1 - nb0) * 2;
+    for (int e = lane; e < 2 * 16 * pieces; e += 32) {
+      const int half = e / (16 * pieces), q = e - half * 16 * pieces, r = wr * 16 + q / pieces, c = (nb0 * 2 + q % pieces) * 8;
+      *reinterpret_cast<uint4*>(out + half * dc_half(DK) + (r * P + c) * 2) =
+          *reinterpret_cast<const uint4*>(dp_smem + (half ? L::kT : L::kQ) + (r * P + c) * 2);
     }
   }
   if (tid < kDcChunk) {
-    float* f = reinterpret_cast<float*>(scratch + kDcMat + 2 * kDcChunk * DK * 2);
+    float* f = reinterpret_cast<float*>(scratch + kDcMat + 2 * dc_half(DK));
     const float e = wm_ex2(cum[tid]);
     f[tid] = beta[tid];
     f[kDcChunk + tid] = rk[tid] * e;
@@ -316,29 +322,47 @@ delta_rule_prepare_kernel(const RbDeltaRuleArgs a) {
 // ---- second kernel
 template <int DK, int COLS>
 struct DcSmem {
-  static constexpr int kPitch = DK + 8, kVPitch = COLS + 8, kMPitch = kDcChunk + 8;
+  static constexpr int kPitch = DK + 8, kVPitch = COLS + 8, kMPitch = kDcMPitch;
+  static constexpr int kAtom = kDcChunk * 128;                       // 64 rows of 64 bf16, 128-byte swizzle
   // one stage: what a chunk reads; the high half of R replaces V element by element
   static constexpr int kQ = 0;
-  static constexpr int kK = kQ + kDcChunk * kPitch * 2;
-  static constexpr int kV = kK + kDcChunk * kPitch * 2;
-  static constexpr int kM = kV + kDcChunk * kVPitch * 2;             // A T
-  static constexpr int kW = kM + kDcChunk * kMPitch * 2;             // W, high and low half
-  static constexpr int kF = kW + 2 * kDcChunk * kPitch * 2;
-  static constexpr int kStage = kF + kDcFactors * kDcChunk * 4;
+  static constexpr int kK = kQ + (DK / 64) * kAtom;
+  static constexpr int kM = kK + (DK / 64) * kAtom;                  // A T, W (high and low half) and the factors, as in the scratch
+  static constexpr int kW = kM + kDcMat;
+  static constexpr int kF = kW + 2 * dc_half(DK);
+  static constexpr int kV = kF + kDcFactors * kDcChunk * 4;
+  static constexpr int kStage = kV + kDcChunk * kVPitch * 2;
   static constexpr int kS = 2 * kStage;                              // state, high and low half
   static constexpr int kR = kS + 2 * DK * kVPitch * 2;               // low half of R
-  static constexpr int kTotal = kR + kDcChunk * kVPitch * 2;
+  static constexpr int kBar = kR + kDcChunk * kVPitch * 2;
+  static constexpr int kTotal = kBar + 2 * 8 + 16;
+  static_assert(kStage % 1024 == 0, "swizzled tiles start at multiples of 1024 bytes");
 };
+
+// A fragment, rows [r0, r0 + 16), columns [k0, k0 + 16), of a tile in 128-byte swizzled atoms of 64 columns
+__device__ __forceinline__ uint32_t dc_a(uint32_t base, int atom, int r0, int k0, int lane) {
+  const int row = r0 + (lane & 15), piece = (k0 >> 3) + (lane >> 4);
+  return base + (piece >> 3) * atom + row * 128 + (((piece & 7) ^ (row & 7)) << 4);
+}
+
+// untiled copy of a contiguous block, completion counted on an mbarrier
+__device__ __forceinline__ void dc_bulk_load(uint32_t dst, const void* src, uint32_t bytes, uint32_t bar) {
+  asm volatile("cp.async.bulk.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1], %2, [%3];"
+               ::"r"(dst), "l"(src), "r"(bytes), "r"(bar) : "memory");
+}
 
 template <int DK, int COLS>
 __global__ void __launch_bounds__(256, 1)
-delta_rule_chunk_kernel(const RbDeltaRuleArgs a) {
+delta_rule_chunk_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK, const RbDeltaRuleArgs a,
+                        unsigned int* status) {
   using L = DcSmem<DK, COLS>;
   constexpr int P = L::kPitch, VP = L::kVPitch, MP = L::kMPitch;
   constexpr int MT = DK / 64, NJ = COLS / 32;      // state: MT row tiles; columns of a warp: NJ pairs of n-tiles
-  extern __shared__ __align__(16) uint8_t dc_smem[];
+  extern __shared__ __align__(1024) uint8_t dc_raw[];
+  uint8_t* dc_smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(dc_raw) + 1023) & ~uintptr_t(1023));
   const uint32_t base = smem_u32(dc_smem);
-  const uint32_t sS = base + L::kS, sRl = base + L::kR;
+  const uint32_t sS = base + L::kS, sRl = base + L::kR, bar = base + L::kBar;      // bar[2]
+  volatile int* abort_flag = reinterpret_cast<volatile int*>(dc_smem + L::kBar + 16);
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int gq = lane >> 2, tq = lane & 3;
   const int wc = warp >> 2, wr = wc ? 3 - (warp & 3) : (warp & 3);
@@ -350,36 +374,41 @@ delta_rule_chunk_kernel(const RbDeltaRuleArgs a) {
   for (int i = 0; i < static_cast<int>(blockIdx.y); ++i) tile0 += (max(0, a.segments[4 * i + 1]) + kDcChunk - 1) / kDcChunk;
   const int g = h / (a.heads / a.kv_heads);
   const __nv_bfloat16* qkv = reinterpret_cast<const __nv_bfloat16*>(a.qkv) + static_cast<long long>(seg.first) * a.ld_qkv;
-  const long long offQ = static_cast<long long>(g) * a.dk, offK = static_cast<long long>(a.kv_heads + g) * a.dk;
   const long long offV = 2ll * a.kv_heads * a.dk + static_cast<long long>(h) * a.dv + c0;
   const int chunks = (seg.len + kDcChunk - 1) / kDcChunk;
+  if (tid == 0) {
+    mbar_init(bar, 1);
+    mbar_init(bar + 8, 1);
+    *abort_flag = 0;
+    fence_mbar_init();
+    tma_prefetch_desc(&tmQ);
+    tma_prefetch_desc(&tmK);
+  }
+  __syncthreads();
 
-  auto request = [&](int ci) {                     // everything chunk ci reads, into stage ci & 1
+  // Everything chunk ci reads, into stage ci & 1.  Rows behind the segment's end are other sequences' queries and keys: beta is
+  // zero there and nothing of them is stored.
+  auto request = [&](int ci) {
     const uint32_t st = base + (ci & 1) * L::kStage;
     const int t0 = ci * kDcChunk, m_rows = min(kDcChunk, seg.len - t0);
-    const __nv_bfloat16* rows = qkv + static_cast<long long>(t0) * a.ld_qkv;
-    for (int i = tid; i < kDcChunk * (DK / 8); i += 256) {
-      const int r = i / (DK / 8), c = (i - r * (DK / 8)) * 8;
-      const bool ok = r < m_rows && c < a.dk;
-      const __nv_bfloat16* src = rows + (ok ? r * a.ld_qkv + c : 0);
-      wm_cp16(st + L::kQ + (r * P + c) * 2, ok ? src + offQ : rows, ok);
-      wm_cp16(st + L::kK + (r * P + c) * 2, ok ? src + offK : rows, ok);
+    if (tid == 0) {
+      const uint32_t b = bar + 8 * (ci & 1);
+      fence_proxy_async_smem();                    // the stage was read (and V written) by ordinary accesses
+      mbar_arrive_expect_tx(b, 2 * (DK / 64) * L::kAtom + dc_scratch(DK));
+#pragma unroll
+      for (int k = 0; k < DK / 64; ++k) {
+        tma_load_4d(st + L::kK + k * L::kAtom, &tmK, k * 64, g, seg.first + t0, 0, b);
+        tma_load_4d(st + L::kQ + k * L::kAtom, &tmQ, k * 64, g, seg.first + t0, 0, b);
+      }
+      dc_bulk_load(st + L::kM, reinterpret_cast<const uint8_t*>(a.scratch) + (static_cast<long long>(tile0 + ci) * a.heads + h) * dc_scratch(DK),
+                   dc_scratch(DK), b);
     }
+    const __nv_bfloat16* rows = qkv + static_cast<long long>(t0) * a.ld_qkv + offV;
     for (int i = tid; i < kDcChunk * (COLS / 8); i += 256) {
       const int r = i / (COLS / 8), c = (i - r * (COLS / 8)) * 8;
       const bool ok = r < m_rows && c0 + c < a.dv;
-      wm_cp16(st + L::kV + (r * VP + c) * 2, ok ? rows + r * a.ld_qkv + offV + c : rows, ok);
+      wm_cp16(st + L::kV + (r * VP + c) * 2, ok ? rows + r * a.ld_qkv + c : qkv, ok);
     }
-    const uint8_t* scratch = reinterpret_cast<const uint8_t*>(a.scratch) + (static_cast<long long>(tile0 + ci) * a.heads + h) * dc_scratch(DK);
-    for (int i = tid; i < kDcChunk * 8; i += 256) {
-      const int r = i >> 3, c = (i & 7) * 8;
-      wm_cp16(st + L::kM + (r * MP + c) * 2, scratch + (r * kDcChunk + c) * 2, true);
-    }
-    for (int i = tid; i < 2 * kDcChunk * (DK / 8); i += 256) {
-      const int r = i / (DK / 8), c = (i - r * (DK / 8)) * 8;         // r: half * 64 + row
-      wm_cp16(st + L::kW + (r * P + c) * 2, scratch + kDcMat + (r * DK + c) * 2, true);
-    }
-    if (tid < kDcFactors * kDcChunk / 4) wm_cp16(st + L::kF + tid * 16, scratch + kDcMat + 2 * kDcChunk * DK * 2 + tid * 16, true);
     wm_cp_commit();
   };
   request(0);
@@ -416,9 +445,11 @@ delta_rule_chunk_kernel(const RbDeltaRuleArgs a) {
   };
   publish();
 
+  bool ok = true;
   for (int ci = 0; ci < chunks; ++ci) {
     wm_cp_wait<0>();
-    __syncthreads();                               // this chunk's tiles and the state have arrived
+    ok = mbar_wait(bar + 8 * (ci & 1), (ci >> 1) & 1, abort_flag, status, 91) && ok;
+    __syncthreads();                               // this chunk's tiles and the state have arrived, for every warp
     if (ci + 1 < chunks) request(ci + 1);
     const uint32_t st = base + (ci & 1) * L::kStage;
     const uint8_t* stp = dc_smem + (ci & 1) * L::kStage;
@@ -433,8 +464,8 @@ delta_rule_chunk_kernel(const RbDeltaRuleArgs a) {
 #pragma unroll
     for (int k = 0; k < DK / 16; ++k) {
       uint32_t kf[4], qf[4];
-      wm_ldsm_x4(wm_a(st + L::kK, P, wr * 16, k * 16, lane), kf);
-      wm_ldsm_x4(wm_a(st + L::kQ, P, wr * 16, k * 16, lane), qf);
+      wm_ldsm_x4(dc_a(st + L::kK, L::kAtom, wr * 16, k * 16, lane), kf);
+      wm_ldsm_x4(dc_a(st + L::kQ, L::kAtom, wr * 16, k * 16, lane), qf);
 #pragma unroll
       for (int j = 0; j < NJ; ++j) {
         uint32_t b[4], bl[4];
@@ -526,16 +557,24 @@ delta_rule_chunk_kernel(const RbDeltaRuleArgs a) {
 #pragma unroll
       for (int r = 0; r < 2; ++r) {
         const int n = n_base + 16 * m + 8 * r, v = c0 + v_base + 8 * j;
-        if (n < a.dk && v < a.dv)
+        if (ok && n < a.dk && v < a.dv)
           *reinterpret_cast<float2*>(slot + static_cast<long long>(n) * a.dv + v) = make_float2(S[m][j][2 * r], S[m][j][2 * r + 1]);
       }
 }
 
+// [rows, heads, dk] part of a packed row-major matrix, 64 columns of 64 rows of one head at a time
+const CUtensorMap* dc_map(const void* base, int dk, int heads, long long rows, long long ld, int* err) {
+  const uint64_t dims[4] = {(uint64_t)dk, (uint64_t)heads, (uint64_t)rows, 1};
+  const uint64_t str[3] = {(uint64_t)dk * 2, (uint64_t)ld * 2, (uint64_t)(rows * ld) * 2};
+  const uint32_t box[4] = {64, 1, (uint32_t)kDcChunk, 1};
+  return rbhost::get_tmap_4d(base, 2, dims, str, box, 1, err);
+}
+
 template <int DK, int COLS>
-int dc_main_launch(const RbDeltaRuleArgs& a, cudaStream_t s) {
-  static_assert(DcSmem<DK, COLS>::kTotal <= 227 * 1024, "shared memory of a CTA");
+int dc_main_launch(const RbDeltaRuleArgs& a, const CUtensorMap* tq, const CUtensorMap* tk, cudaStream_t s) {
+  const int smem = DcSmem<DK, COLS>::kTotal + 1024;
+  static_assert(DcSmem<DK, COLS>::kTotal + 1024 <= 227 * 1024, "shared memory of a CTA");
   auto kern = delta_rule_chunk_kernel<DK, COLS>;
-  const int smem = DcSmem<DK, COLS>::kTotal;
   static bool cfg_dev[64] = {false};
   bool& cfg = cfg_dev[rbhost::device_slot()];
   if (!cfg) {
@@ -543,7 +582,7 @@ int dc_main_launch(const RbDeltaRuleArgs& a, cudaStream_t s) {
     if (e != cudaSuccess) return static_cast<int>(e);
     cfg = true;
   }
-  kern<<<dim3(a.heads * ((a.dv + COLS - 1) / COLS), a.num_segments), 256, smem, s>>>(a);
+  kern<<<dim3(a.heads * ((a.dv + COLS - 1) / COLS), a.num_segments), 256, smem, s>>>(*tq, *tk, a, rbhost::status_ptr());
   return static_cast<int>(cudaGetLastError());
 }
 
@@ -558,12 +597,18 @@ int dc_launch(const RbDeltaRuleArgs& a, cudaStream_t s) {
     if (e != cudaSuccess) return static_cast<int>(e);
     cfg = true;
   }
-  prep<<<dim3(a.heads, a.num_tiles), 128, smem, s>>>(a);
+  const __nv_bfloat16* q = reinterpret_cast<const __nv_bfloat16*>(a.qkv);
+  int err = 0;
+  const CUtensorMap* tq = dc_map(q, a.dk, a.kv_heads, a.rows, a.ld_qkv, &err);
+  const CUtensorMap* tk = dc_map(q + static_cast<long long>(a.kv_heads) * a.dk, a.dk, a.kv_heads, a.rows, a.ld_qkv, &err);
+  if (!tq || !tk) return err ? err : -5;
+  prep<<<dim3(a.heads, a.num_tiles), kDpThreads, smem, s>>>(a);
   const int rc = static_cast<int>(cudaGetLastError());
   if (rc) return rc;
   // narrow column tiles (twice the CTAs) while wide ones would leave half of the SMs idle
   const long long wide = static_cast<long long>(a.heads) * ((a.dv + 63) / 64) * a.num_segments;
-  return wide * 2 <= rbhost::device_sm_count() || a.dv <= 32 ? dc_main_launch<DK, 32>(a, s) : dc_main_launch<DK, 64>(a, s);
+  return wide * 2 <= rbhost::device_sm_count() || a.dv <= 32 ? dc_main_launch<DK, 32>(a, tq, tk, s)
+                                                             : dc_main_launch<DK, 64>(a, tq, tk, s);
 }
 
 }  // namespace rb
@@ -576,7 +621,7 @@ RB_API int rb_delta_rule_chunked(const RbDeltaRuleArgs* args, void* stream_v) {
   const RbDeltaRuleArgs& a = *args;
   if (a.num_segments <= 0) return 0;
   if (!a.qkv || !a.a_raw || !a.b_raw || !a.dt_bias || !a.a_log || !a.state || !a.o || !a.segments || !a.tiles || !a.scratch || a.f32 ||
-      a.heads <= 0 || a.kv_heads <= 0 || a.heads % a.kv_heads || a.dk <= 0 || a.dv <= 0 || a.num_slots <= 0 || a.num_tiles <= 0 ||
+      a.heads <= 0 || a.kv_heads <= 0 || a.heads % a.kv_heads || a.dk <= 0 || a.dv <= 0 || a.num_slots <= 0 || a.num_tiles <= 0 || a.rows <= 0 ||
       a.num_segments > 65535 || a.num_tiles > 65535)
     return -1;
   if (a.dk > 128 || ((a.dk | a.dv) & 7) || (a.ld_qkv & 7) || (a.ld_o & 1)) return -9;

@@ -65,6 +65,7 @@ typedef struct RbDeltaRuleArgs {
   const int* tiles;
   void* scratch;             // chunked form
   long long ld_qkv, ld_ab, ld_o;
+  long long rows;            // chunked form: rows of qkv
   int num_segments, num_tiles, heads, kv_heads, dk, dv, f32, num_slots;
 } RbDeltaRuleArgs;
 int rb_delta_rule_scan(const RbDeltaRuleArgs* args, void* stream);

@@ -133,6 +133,7 @@ class RbDeltaRuleArgs(C.Structure):
         ("qkv", c_void_p), ("a_raw", c_void_p), ("b_raw", c_void_p), ("dt_bias", c_void_p), ("a_log", c_void_p),
         ("state", c_void_p), ("o", c_void_p), ("segments", c_void_p), ("tiles", c_void_p), ("scratch", c_void_p),
         ("ld_qkv", c_ll), ("ld_ab", c_ll), ("ld_o", c_ll),
+        ("rows", c_ll),
         ("num_segments", c_int), ("num_tiles", c_int), ("heads", c_int), ("kv_heads", c_int), ("dk", c_int), ("dv", c_int),
         ("f32", c_int), ("num_slots", c_int),
     ]

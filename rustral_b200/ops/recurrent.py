@@ -230,7 +230,7 @@ def delta_rule(qkv, a_raw, b_raw, *, dt_bias, a_log, state, heads: int, kv_heads
         tiles = many.tiles(CHUNK)
         scratch = torch.empty(lib.rb_delta_rule_scratch_bytes(tiles.shape[0], heads, dk), dtype=torch.uint8, device=qkv.device)
         a.segments, a.num_segments, a.tiles, a.num_tiles = many.table.data_ptr(), many.n, tiles.data_ptr(), tiles.shape[0]
-        a.scratch = scratch.data_ptr()
+        a.scratch, a.rows = scratch.data_ptr(), rows
         N.check(lib.rb_delta_rule_chunked(a, N.stream_ptr()), "rb_delta_rule_chunked")
     return out
 
