@@ -127,6 +127,13 @@ delta_rule_prepare_kernel(const RbDeltaRuleArgs a) {
   // ---- L (side 0) and A (side 1); A stays in registers as the A operand of A T, high and low half
   uint32_t ah[4][4], al[4][4];
   {
+    float ct[2], ft[2];                            // of the rows gq and gq + 8
+#pragma unroll
+    for (int r = 0; r < 2; ++r) {
+      const int t = wr * 16 + gq + 8 * r;
+      ct[r] = cum[t];
+      ft[r] = side ? rq[t] : beta[t] * rk[t];
+    }
     uint32_t xf[DK / 16][4];
 #pragma unroll
     for (int k = 0; k < DK / 16; ++k) wm_ldsm_x4(wm_a(side ? sQ : sK, P, wr * 16, k * 16, lane), xf[k]);
@@ -144,20 +151,18 @@ delta_rule_prepare_kernel(const RbDeltaRuleArgs a) {
         wm_mma(acc[1], xf[k], b[2], b[3]);
       }
 #pragma unroll
-      for (int i = 0; i < 2; ++i)
+      for (int i = 0; i < 2; ++i) {
+        const int s = sb * 16 + i * 8 + 2 * tq;
+        const float2 cs = *reinterpret_cast<const float2*>(cum + s), ks = *reinterpret_cast<const float2*>(rk + s);
 #pragma unroll
         for (int r = 0; r < 2; ++r) {
-          const int t = wr * 16 + gq + 8 * r, s = sb * 16 + i * 8 + 2 * tq;
-          float v[2];
-#pragma unroll
-          for (int j = 0; j < 2; ++j) v[j] = s + j <= t ? wm_ex2(cum[t] - cum[s + j]) * rk[s + j] * acc[i][2 * r + j] : 0.f;
-          if (side == 0) {
-            const float f = beta[t] * rk[t];
-            *reinterpret_cast<float2*>(Lm + t * LP + s) = make_float2(s < t ? f * v[0] : 0.f, s + 1 < t ? f * v[1] : 0.f);
-          } else {
-            wm_split(rq[t] * v[0], rq[t] * v[1], ah[sb][2 * i + r], al[sb][2 * i + r]);
-          }
+          const int t = wr * 16 + gq + 8 * r;
+          const float v0 = s <= t ? wm_ex2(ct[r] - cs.x) * ks.x * ft[r] * acc[i][2 * r] : 0.f;
+          const float v1 = s + 1 <= t ? wm_ex2(ct[r] - cs.y) * ks.y * ft[r] * acc[i][2 * r + 1] : 0.f;
+          if (side == 0) *reinterpret_cast<float2*>(Lm + t * LP + s) = make_float2(s < t ? v0 : 0.f, s + 1 < t ? v1 : 0.f);
+          else wm_split(v0, v1, ah[sb][2 * i + r], al[sb][2 * i + r]);
         }
+      }
     }
   }
   __syncthreads();
@@ -183,32 +188,36 @@ delta_rule_prepare_kernel(const RbDeltaRuleArgs a) {
   }
   __syncthreads();
   // ---- ... then the blocks below: T_ij = -T_ii sum_{j <= k < i} L_ik T_kj, one distance i - j after the other
-  auto dot16 = [&](const float* row, const float* colm, int pitch) {
-    float v0 = 0.f, v1 = 0.f;
+  // 64 threads per block, four neighbouring entries of a row each
+  const int gb = tid >> 6, er = (tid >> 2) & 15, ec = (tid & 3) * 4;
+  auto dot16 = [&](const float* row, const float* m, int pitch, float4& out) {
 #pragma unroll
     for (int k = 0; k < 16; k += 4) {
       const float4 l = *reinterpret_cast<const float4*>(row + k);
-      v0 = fmaf(l.x, colm[k * pitch], v0);
-      v1 = fmaf(l.y, colm[(k + 1) * pitch], v1);
-      v0 = fmaf(l.z, colm[(k + 2) * pitch], v0);
-      v1 = fmaf(l.w, colm[(k + 3) * pitch], v1);
+      const float lv[4] = {l.x, l.y, l.z, l.w};
+#pragma unroll
+      for (int q = 0; q < 4; ++q) {
+        const float4 u = *reinterpret_cast<const float4*>(m + (k + q) * pitch);
+        out.x = fmaf(lv[q], u.x, out.x); out.y = fmaf(lv[q], u.y, out.y);
+        out.z = fmaf(lv[q], u.z, out.z); out.w = fmaf(lv[q], u.w, out.w);
+      }
     }
-    return v0 + v1;
   };
 #pragma unroll
   for (int d = 1; d < 4; ++d) {
-    const int r = tid >> 4, c = tid & 15;          // one entry of every block per thread
+    const bool mine = gb < 4 - d;                  // block row gb + d, block column gb
+    if (mine) {
+      float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
 #pragma unroll
-    for (int blk = 0; blk < 4 - d; ++blk) {        // block row blk + d, block column blk
-      float v = 0.f;
-#pragma unroll
-      for (int k = 0; k < d; ++k) v += dot16(Lm + ((blk + d) * 16 + r) * LP + (blk + k) * 16, T + (blk + k) * 16 * LP + blk * 16 + c, LP);
-      W[(blk * 16 + r) * 20 + c] = v;
+      for (int k = 0; k < d; ++k) dot16(Lm + ((gb + d) * 16 + er) * LP + (gb + k) * 16, T + (gb + k) * 16 * LP + gb * 16 + ec, LP, v);
+      *reinterpret_cast<float4*>(W + (gb * 16 + er) * 20 + ec) = v;
     }
     __syncthreads();
-#pragma unroll
-    for (int blk = 0; blk < 4 - d; ++blk)
-      T[((blk + d) * 16 + r) * LP + blk * 16 + c] = -dot16(T + ((blk + d) * 16 + r) * LP + (blk + d) * 16, W + blk * 16 * 20 + c, 20);
+    if (mine) {
+      float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+      dot16(T + ((gb + d) * 16 + er) * LP + (gb + d) * 16, W + gb * 16 * 20 + ec, 20, v);
+      *reinterpret_cast<float4*>(T + ((gb + d) * 16 + er) * LP + gb * 16 + ec) = make_float4(-v.x, -v.y, -v.z, -v.w);
+    }
     __syncthreads();
   }
   const uint32_t sT = smem_u32(dp_smem) + L::kL;
@@ -231,7 +240,8 @@ delta_rule_prepare_kernel(const RbDeltaRuleArgs a) {
 #pragma unroll
       for (int half = 0; half < 2; ++half) {       // columns k 16 + 8 half + 2 tq (+ 1)
         const int t = k * 16 + half * 8 + 2 * tq;
-        const float w0 = rk[t] * wm_ex2(c_end - cum[t]), w1 = rk[t + 1] * wm_ex2(c_end - cum[t + 1]);
+        const float2 ck = *reinterpret_cast<const float2*>(cum + t), kk = *reinterpret_cast<const float2*>(rk + t);
+        const float w0 = kk.x * wm_ex2(c_end - ck.x), w1 = kk.y * wm_ex2(c_end - ck.y);
 #pragma unroll
         for (int r = 0; r < 2; ++r) {
           const int s = wr * 16 + gq + 8 * r;
