@@ -1,16 +1,17 @@
-// RMS norm over equal parts of a row with a silu gate before or behind it: the output stage of the recurrent mixers.  A warp
-// (parts up to 1024) or a CTA owns one part and keeps it in registers; sums are fp32.
+// RMS norm over equal parts of a row with a silu gate before or behind it: the output stage of the recurrent mixers.  Between
+// 8 lanes and a CTA own one part, by its size, and keep it in registers; sums are fp32.
 #include "recurrent.h"
 
 #include "recurrent.cuh"
 
 namespace rb {
 
-// sum over the lanes that own a part: a warp, or the whole CTA
+// sum over the lanes that own a part: up to a warp, or the whole CTA
 template <int L>
 __device__ __forceinline__ float gn_sum(float v, float* red) {
-  v = warp_sum(v);
-  if (L == 32) return v;
+#pragma unroll
+  for (int o = (L < 32 ? L : 32) / 2; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
+  if (L <= 32) return v;
   if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = v;
   __syncthreads();
   float s = 0.f;
@@ -23,9 +24,11 @@ template <typename T, int VEC, int CH, int L>
 __global__ void __launch_bounds__(256)
 gated_norm_kernel(const RbGatedNormArgs a) {
   __shared__ float red[8];
-  const int sub = L == 32 ? threadIdx.x & 31 : threadIdx.x;
-  const long long item = static_cast<long long>(blockIdx.x) * (256 / L) + (L == 32 ? threadIdx.x >> 5 : 0);
-  if (item >= static_cast<long long>(a.rows) * a.parts) return;      // whole warps (CTAs) leave together
+  const int sub = L <= 32 ? threadIdx.x & (L - 1) : threadIdx.x;
+  const long long total = static_cast<long long>(a.rows) * a.parts;
+  long long item = L <= 32 ? static_cast<long long>(blockIdx.x) * (256 / (L < 32 ? L : 32)) + threadIdx.x / L : blockIdx.x;
+  const bool idle = item >= total;                 // the last CTA's: they stay for the shuffles and compute a part once more
+  if (idle) item = total - 1;
   const long long t = item / a.parts;
   const int part = static_cast<int>(item - t * a.parts);
   const long long base = static_cast<long long>(part) * a.part_n;
@@ -49,6 +52,7 @@ gated_norm_kernel(const RbGatedNormArgs a) {
     }
   }
   const float r = 1.f / sqrtf(gn_sum<L>(sq, red) / static_cast<float>(a.part_n) + a.eps);
+  if (idle) return;
 #pragma unroll
   for (int c = 0; c < CH; ++c) {
     const int col = (c * L + sub) * VEC;
@@ -84,11 +88,12 @@ gated_norm_any_kernel(const RbGatedNormArgs a) {
 template <typename T, int VEC, int L>
 int gn_launch(const RbGatedNormArgs& a, cudaStream_t s) {
   const long long items = static_cast<long long>(a.rows) * a.parts;
-  const int grid = static_cast<int>((items + 256 / L - 1) / (256 / L));
+  const int per = L <= 32 ? 256 / L : 1, threads = L <= 32 ? 256 : L;
+  const int grid = static_cast<int>((items + per - 1) / per);
   const int ch = (a.part_n / VEC + L - 1) / L;
-  if (ch <= 1) gated_norm_kernel<T, VEC, 1, L><<<grid, 256, 0, s>>>(a);
-  else if (ch <= 2) gated_norm_kernel<T, VEC, 2, L><<<grid, 256, 0, s>>>(a);
-  else gated_norm_kernel<T, VEC, 4, L><<<grid, 256, 0, s>>>(a);
+  if (ch <= 1) gated_norm_kernel<T, VEC, 1, L><<<grid, threads, 0, s>>>(a);
+  else if (ch <= 2) gated_norm_kernel<T, VEC, 2, L><<<grid, threads, 0, s>>>(a);
+  else gated_norm_kernel<T, VEC, 4, L><<<grid, threads, 0, s>>>(a);
   return static_cast<int>(cudaGetLastError());
 }
 
@@ -96,7 +101,10 @@ template <typename T, int VEC>
 int gn_pick(const RbGatedNormArgs& a, cudaStream_t s) {
   const uintptr_t bits = reinterpret_cast<uintptr_t>(a.y) | reinterpret_cast<uintptr_t>(a.z) | reinterpret_cast<uintptr_t>(a.out);
   const bool vec = !(bits & 15) && !((a.ld_y | a.ld_z | a.ld_o | a.part_n) % VEC);
-  if (vec && a.part_n <= 32 * VEC * 4) return gn_launch<T, VEC, 32>(a, s);
+  if (vec && a.part_n <= 8 * VEC) return gn_launch<T, VEC, 8>(a, s);
+  if (vec && a.part_n <= 16 * VEC) return gn_launch<T, VEC, 16>(a, s);
+  if (vec && a.part_n <= 32 * VEC * 2) return gn_launch<T, VEC, 32>(a, s);
+  if (vec && a.part_n <= 128 * VEC * 2) return gn_launch<T, VEC, 128>(a, s);
   if (vec && a.part_n <= 256 * VEC * 4) return gn_launch<T, VEC, 256>(a, s);
   gated_norm_any_kernel<T><<<a.rows * a.parts, 256, 0, s>>>(a);
   return static_cast<int>(cudaGetLastError());

@@ -132,10 +132,22 @@ int rn_launch(const RbResidualNormArgs& a, cudaStream_t s) {
   return static_cast<int>(cudaGetLastError());
 }
 
+// two sums over the CTA at once; `red` holds two floats per warp
+__device__ __forceinline__ float2 rn_block_sum2(float v, float w, float2* red) {
+  v = warp_sum(v);
+  w = warp_sum(w);
+  const int warps = blockDim.x >> 5;
+  if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = make_float2(v, w);
+  __syncthreads();
+  float2 s = make_float2(0.f, 0.f);
+  for (int i = 0; i < warps; ++i) { s.x += red[i].x; s.y += red[i].y; }
+  return s;
+}
+
 template <int VEC, int CH>
 __global__ void __launch_bounds__(256)
 stream_update_kernel(const RbStreamUpdateArgs a) {
-  __shared__ float red[8];
+  __shared__ float2 red[8];
   const int t = blockIdx.x, n = a.n;
   float x[CH][VEC], va[CH][VEC], vb[CH][VEC], v[CH][VEC];
   float sa = 0.f, sb = 0.f;
@@ -153,8 +165,12 @@ stream_update_kernel(const RbStreamUpdateArgs a) {
     for (int i = 0; i < VEC; ++i) { sa = fmaf(va[c][i], va[c][i], sa); sb = fmaf(vb[c][i], vb[c][i], sb); }
   }
   const float inv_n = 1.f / static_cast<float>(n);
-  const float ra = a.a ? a.normed / sqrtf(rn_block_sum(sa, red) * inv_n + a.eps) : 0.f;
-  const float rb_ = a.b ? a.normed / sqrtf(rn_block_sum(sb, red) * inv_n + a.eps) : 0.f;
+  float ra = 0.f, rb_ = 0.f;
+  if (a.a || a.b) {
+    const float2 sums = rn_block_sum2(sa, sb, red);
+    ra = a.normed / sqrtf(sums.x * inv_n + a.eps);
+    rb_ = a.normed / sqrtf(sums.y * inv_n + a.eps);
+  }
   const bool add = a.a || a.b || a.c;
   const float alpha = a.h ? a.alpha[0] : 0.f;
 #pragma unroll

@@ -263,10 +263,12 @@ class LayeredConfig:
     arch: str = "Dolurax"
 
     def __post_init__(self):
-        if not self.layers or self.vocab_size < 1 or self.d_model < 8 or self.d_model % 8:
-            raise ValueError("layered decoder: at least one layer, and a width that is a multiple of 8")
         if self.arch not in DESIGNS:
             raise ValueError(f"layered decoder: unknown design {self.arch!r}")
+        if not self.layers or self.vocab_size < 1 or self.d_model < 1:
+            raise ValueError("layered decoder: at least one layer, and a positive width and vocabulary")
+        if self.d_model % 8 and any(isinstance(s.mlp, MoESpec) for s in self.layers):
+            raise ValueError("layered decoder: the width of a model with routed experts is a multiple of 8")
         mixing = [s.mixer for s in self.layers if getattr(s.mixer, "v_mix", False)]
         if len({a.kv_heads * a.vdim for a in mixing}) > 1:
             raise ValueError("layers that mix values must have the same number of value columns")

@@ -245,10 +245,10 @@ class ParallelBody:
         y = rc_ops.state_space(xbc, gate("dt"), dt_bias=P.w(p + "dt_bias"), a_log=P.w(p + "A_log"), D=P.w(p + "D"), state=state["state"],
                                heads=m.heads, groups=m.groups, vdim=m.vdim, n=m.state, seg=sb.segments)
         y = rc_ops.gated_norm(y, col("z"), P.w(p + "norm"), m.norm_groups, cfg.norm_eps, gate_first=True, out=y)
-        out = dict(a=gemm(o, P.w(p + "left.o"), out_dtype=torch.float32), wa=P.w(p + "left.out"),
-                   b=gemm(y, P.w(p + "right.o"), out_dtype=torch.float32), wb=P.w(p + "right.out"), normed=0.5)
+        out = dict(a=gemm(o, P.w(p + "left.o")), wa=P.w(p + "left.out"),
+                   b=gemm(y, P.w(p + "right.o")), wb=P.w(p + "right.out"), normed=0.5)
         if s.mlp is not None:
-            out["c"] = gemm(self._feed_forward(l, s, z), P.w(p + "down"), out_dtype=torch.float32)
+            out["c"] = gemm(self._feed_forward(l, s, z), P.w(p + "down"))
         return self._update(st, l, **out)
 
     def _delta(self, l, st, sb, s, p, col, gate, z):
@@ -264,7 +264,7 @@ class ParallelBody:
         rc_ops.gated_norm(o, col("z"), P.w(p + "norm"), m.heads, self.cfg.norm_eps, gate_first=False, out=o)
         if s.mlp is not None:
             self._feed_forward(l, s, z, out=joined[:, up8(n):])
-        return self._update(st, l, c=gemm(joined, w_out, out_dtype=torch.float32))
+        return self._update(st, l, c=gemm(joined, w_out))
 
     def head(self, st, rows):
         P = self.r.params

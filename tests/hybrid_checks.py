@@ -50,7 +50,7 @@ CONFIGS = {
     "wide": model([par(left(8, 2, 128, 72, 150, 5), right(4, 72, 128, 2, 2, 4), 96), delta(4, 2, 128, 136, 4, 104),
                    par(left(4, 4, 64, 128, 33, 130), right(2, 128, 64, 1, 4, 4), 96)], width=128, vocab=260),
     # sizes that are no multiple of 8, long filters, kept tokens beyond the window
-    "odd": model([par(left(6, 3, 20, 12, 24, 30), right(3, 20, 12, 3, 2, 6), 36), delta(4, 2, 20, 12, 5, 44)], width=72),
+    "odd": model([par(left(6, 3, 20, 12, 24, 30), right(3, 20, 12, 3, 2, 6), 36), delta(4, 2, 20, 12, 5, 44)], width=70),
 }
 
 

@@ -252,7 +252,7 @@ def test_portions_of_a_prompt_give_the_same_state():
 
 
 @BOTH
-@pytest.mark.parametrize("n,parts", [(24, 3), (96, 1), (90, 5), (1024, 8), (4096, 1), (4096, 32), (8200, 1), (520, 4)])
+@pytest.mark.parametrize("n,parts", [(24, 3), (96, 1), (90, 5), (1024, 8), (4096, 1), (4096, 32), (8200, 1), (520, 4), (2048, 32), (1536, 2), (3000, 1), (448, 2)])
 def test_gated_norm(n, parts, dtype):
     g = torch.Generator().manual_seed(n)
     y, z, w = torch.randn(19, n, generator=g).to(dtype), torch.randn(19, n + 8, generator=g).to(dtype), torch.randn(n, generator=g)
