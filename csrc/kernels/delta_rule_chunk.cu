@@ -52,7 +52,7 @@ struct DcPrepSmem {
 };
 
 template <int DK>
-__global__ void __launch_bounds__(kDpThreads, 2)
+__global__ void __launch_bounds__(kDpThreads, 3)
 delta_rule_prepare_kernel(const RbDeltaRuleArgs a) {
   using L = DcPrepSmem<DK>;
   constexpr int P = L::kPitch, LP = L::kLPitch;
@@ -312,11 +312,15 @@ delta_rule_prepare_kernel(const RbDeltaRuleArgs a) {
     }
     __syncwarp();                                  // every warp copies its own rows and columns
     uint8_t* out = scratch + kDcMat;
-    const int pieces = (nb1 - nb0) * 2;
-    for (int e = lane; e < 2 * 16 * pieces; e += 32) {
-      const int half = e / (16 * pieces), q = e - half * 16 * pieces, r = wr * 16 + q / pieces, c = (nb0 * 2 + q % pieces) * 8;
-      *reinterpret_cast<uint4*>(out + half * dc_half(DK) + (r * P + c) * 2) =
-          *reinterpret_cast<const uint4*>(dp_smem + (half ? L::kT : L::kQ) + (r * P + c) * 2);
+    // lanes: two rows of 16 at a time, the 16-byte pieces of a row side by side
+    const int r0 = wr * 16 + (lane >> 4), c = (nb0 * 2 + (lane & 15)) * 8;
+    if (c < nb1 * 16) {
+#pragma unroll
+      for (int r = r0; r < wr * 16 + 16; r += 2) {
+        const int at = (r * P + c) * 2;
+        *reinterpret_cast<uint4*>(out + at) = *reinterpret_cast<const uint4*>(dp_smem + L::kQ + at);
+        *reinterpret_cast<uint4*>(out + dc_half(DK) + at) = *reinterpret_cast<const uint4*>(dp_smem + L::kT + at);
+      }
     }
   }
   if (tid < kDcChunk) {
