@@ -67,7 +67,8 @@ def main(argv=None):
         dev = "cuda" if torch.cuda.is_available() else "cpu"
     # bf16 inference weights where the architecture has them: the trainer's flat buffers would not fit
     params = build_weights(cfg, dev, None, load_tensors(a.model), a.seed) if tp is None else None
-    runner = ModelRunner(cfg, params=params, device=dev, num_blocks=a.blocks, block_size=a.page, seed=a.seed, tp=tp)
+    runner = ModelRunner(cfg, params=params, device=dev, num_blocks=a.blocks, block_size=a.page, seed=a.seed, tp=tp,
+                         num_slots=a.max_batch)
     eng = ServingEngine(runner, max_batch_size=a.max_batch, prefill_chunk=a.prefill_chunk)
     # warm-up: one short request end to end
     eng.generate(list(range(1, 33)), 4)

@@ -306,14 +306,15 @@ def parse_args(argv=None):
     g.add_argument("--out-features", type=int, default=0)
     g.add_argument("--bias", action="store_true")
     e = ap.add_argument_group("decoder engine (/v1/generate)")
-    e.add_argument("--model", help="model preset (llama-8b, gpt2-small, dolurax-test, ...) or a folder with config.json and "
+    e.add_argument("--model", help="model preset (llama-8b, gpt2-small, dolurax-test, vafodra-test, ...) or a folder with config.json and "
                                    "model.safetensors")
     e.add_argument("--dtype", default=None, choices=["bfloat16", "float32"], help="for architectures that run in both")
     e.add_argument("--layers", type=int, default=0, help="override the preset's depth")
     e.add_argument("--weights", help="safetensors state dict of the model; random-init when absent")
     e.add_argument("--blocks", type=int, default=4096, help="KV-cache pages")
     e.add_argument("--page", type=int, default=16, help="tokens per KV-cache page")
-    e.add_argument("--max-batch", type=int, default=64)
+    e.add_argument("--max-batch", type=int, default=64, help="requests in one step; also the state slots of models with "
+                   "recurrent layers")
     e.add_argument("--eos-id", type=int, default=None)
     e.add_argument("--seed", type=int, default=0)
     return ap.parse_args(argv)

@@ -155,7 +155,7 @@ def test_short_conv(channels, taps, name, dtype):
 
 
 SSM = [  # heads, groups, vdim, state, shift of the logarithm of the decay rate
-    (2, 1, 64, 128, 0.0), (4, 2, 48, 32, -2.0), (2, 2, 128, 64, 1.5), (3, 1, 40, 24, -4.0), (2, 1, 72, 104, 0.0), (2, 1, 20, 12, 0.0), (1, 1, 8, 200, 0.0),
+    (2, 1, 64, 128, 0.0), (4, 2, 56, 40, -2.0), (2, 2, 128, 64, 1.5), (3, 1, 40, 24, -4.0), (2, 1, 72, 104, 0.0), (2, 1, 20, 12, 0.0), (1, 1, 8, 200, 0.0),
 ]
 
 
@@ -202,7 +202,7 @@ def test_state_space_spans_of_a_long_prompt():
 
 
 DELTA = [  # heads, kv heads, dk, dv, shift of the logarithm of the decay rate
-    (2, 1, 128, 64, 0.0), (4, 2, 32, 64, -2.0), (2, 2, 64, 128, 1.5), (3, 3, 24, 40, -4.0), (2, 1, 104, 136, -6.0), (2, 1, 20, 12, 0.0), (1, 1, 200, 8, 0.0),
+    (2, 1, 128, 64, 0.0), (4, 2, 40, 72, -2.0), (2, 2, 64, 128, 1.5), (3, 3, 24, 40, -4.0), (2, 1, 104, 136, -6.0), (2, 1, 20, 12, 0.0), (1, 1, 200, 8, 0.0),
 ]
 
 
