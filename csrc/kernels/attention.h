@@ -34,6 +34,11 @@ typedef struct RbAttnRule {
   const float* head_gate;
   long long ld_gate;
   int window, keep_first, sink;
+  // rot_dim > 0: queries and keys have a second part of rot_dim numbers.  A head's follows the head_dim numbers of its query (heads of q
+  // are head_dim + rot_dim or more apart); the keys share k_rot [seq_k, rot_dim], pitch ld_k_rot (batch 1).  The score is the sum of both.
+  int rot_dim;
+  const void* k_rot;
+  long long ld_k_rot;
 } RbAttnRule;
 int rb_attention_fwd_rule(const RbAttnArgs* args, const RbAttnRule* rule, void* stream);
 int rb_attention_fwd(const RbAttnArgs* args, void* stream);

@@ -17,6 +17,8 @@
 // real sizes are zero-filled by TMA), capped scores, a linear distance bias, chunked or windowed visibility (key blocks before a
 // tile's first visible key are skipped, so the two tiles may start at different blocks), first keys that a window keeps (their
 // blocks are walked before the window's), a sink in the softmax and a sigmoid output gate per value column or per head.
+// With DR > 0 queries and keys have a second part whose keys all heads share (rotary positions of latent attention): it is one more
+// 64-column piece of the Q and K tiles, loaded from its own array.
 //
 // Same semantics as the other forward kernels (causal alignment to the end of the keys, GQA, log-sum-exp output).
 // Replaces the reference's materialised-score attention (crates/nn/src/attention.rs:640-836).
@@ -47,6 +49,7 @@ struct F2Params {
   const float* head_gate;      // [seq_q, heads] or NULL
   long long ld_gate;
   int window, keep, sink;
+  int dr;                   // DR > 0: real size of the second part
 };
 
 __device__ __forceinline__ float f2_ex2(float x) {
@@ -175,26 +178,29 @@ __device__ __forceinline__ void tmem_ld_32x32_ptr(uint32_t taddr, uint32_t* r) {
       : "memory");
 }
 
+// D: columns of Q and K tiles, both parts
 template <int D, int DV>
 struct F2Smem {
-  static constexpr int kStages = D == 64 && DV == 64 ? 4 : D == 128 && DV == 128 ? 2 : 3;
+  static constexpr int kStages = D == 64 && DV == 64 ? 4 : D >= 128 && DV == 128 ? 2 : D == 192 ? 2 : 3;     // of K
+  static constexpr int kVStages = D == 192 && DV == 128 ? 1 : kStages;
   static constexpr int kHalf = kF2Tile * 128;                 // one 64-column swizzle atom: 128 rows x 128 B
   static constexpr int kTileBytes = (D / 64) * kHalf;         // a 128-row tile of Q or K
   static constexpr int kVTileBytes = (DV / 64) * kHalf;       // a 128-row tile of V
   static constexpr int kQ = 0;                                // two tiles
   static constexpr int kK = kQ + 2 * kTileBytes;
   static constexpr int kV = kK + kStages * kTileBytes;
-  static constexpr int kBar = kV + kStages * kVTileBytes;
-  static constexpr int kNumBars = 2 + 3 * kStages + 6;        // q[2], k_full/v_full/kv_empty[stages], s_full[2], p_full[2], o_ready[2]
+  static constexpr int kBar = kV + kVStages * kVTileBytes;
+  static constexpr int kNumBars = 2 + 2 * (kStages + kVStages) + 6;   // q[2], full and empty per K and V stage, s_full[2], p_full[2], o_ready[2]
   static constexpr int kTotal = kBar + kNumBars * 8 + 16;
 };
 
-template <int D, int DV, int kPolyEvery, bool RULE>
+template <int D, int DV, int kPolyEvery, bool RULE, int DR = 0>
 __global__ void __launch_bounds__(kF2Threads, 1)
 attn_fwd2_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK,
-                 const __grid_constant__ CUtensorMap tmV, F2Params p, unsigned int* status) {
-  using L = F2Smem<D, DV>;
-  constexpr int kStages = L::kStages;
+                 const __grid_constant__ CUtensorMap tmV, const __grid_constant__ CUtensorMap tmQr,
+                 const __grid_constant__ CUtensorMap tmKr, F2Params p, unsigned int* status) {
+  using L = F2Smem<D + DR, DV>;
+  constexpr int kStages = L::kStages, kVStages = L::kVStages;
   extern __shared__ __align__(1024) uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
   const uint32_t sbase = smem_u32(smem);
@@ -203,9 +209,10 @@ attn_fwd2_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
   const uint32_t b0 = smem_u32(bars);
   const uint32_t bar_q = b0;                                   // [2]
   const uint32_t bar_kfull = b0 + 16;                          // [kStages]
-  const uint32_t bar_vfull = bar_kfull + 8 * kStages;
-  const uint32_t bar_kvempty = bar_vfull + 8 * kStages;
-  const uint32_t bar_sfull = bar_kvempty + 8 * kStages;        // [2]
+  const uint32_t bar_kempty = bar_kfull + 8 * kStages;
+  const uint32_t bar_vfull = bar_kempty + 8 * kStages;         // [kVStages]
+  const uint32_t bar_vempty = bar_vfull + 8 * kVStages;
+  const uint32_t bar_sfull = bar_vempty + 8 * kVStages;        // [2]
   const uint32_t bar_pfull = bar_sfull + 16;                   // [2]
   const uint32_t bar_oready = bar_pfull + 16;                  // [2]
   uint32_t* tmem_ptr_smem = reinterpret_cast<uint32_t*>(bars + L::kNumBars);
@@ -265,8 +272,11 @@ attn_fwd2_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
     }
     for (int s = 0; s < kStages; ++s) {
       mbar_init(bar_kfull + 8 * s, 1);
+      mbar_init(bar_kempty + 8 * s, 1);
+    }
+    for (int s = 0; s < kVStages; ++s) {
       mbar_init(bar_vfull + 8 * s, 1);
-      mbar_init(bar_kvempty + 8 * s, 1);
+      mbar_init(bar_vempty + 8 * s, 1);
     }
     *abort_flag = 0;
     fence_mbar_init();
@@ -295,18 +305,24 @@ attn_fwd2_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
 #pragma unroll
         for (int hf = 0; hf < D / 64; ++hf)
           tma_load_4d(sQ + t * L::kTileBytes + hf * L::kHalf, &tmQ, hf * 64, h, q0 + t * kF2Tile, b, bar_q + 8 * t);
+        if (DR > 0)
+          tma_load_4d(sQ + t * L::kTileBytes + (D / 64) * L::kHalf, &tmQr, 0, h, q0 + t * kF2Tile, b, bar_q + 8 * t);
       }
       for (int j = f_min; j < n_max; ++j) {
         const int s = (j - f_min) % kStages, use = (j - f_min) / kStages;
-        if (!mbar_wait(bar_kvempty + 8 * s, (use & 1) ^ 1, abort_flag, status, 41)) break;
+        if (!mbar_wait(bar_kempty + 8 * s, (use & 1) ^ 1, abort_flag, status, 41)) break;
         mbar_arrive_expect_tx(bar_kfull + 8 * s, L::kTileBytes);
 #pragma unroll
         for (int hf = 0; hf < D / 64; ++hf)
           tma_load_4d(sK + s * L::kTileBytes + hf * L::kHalf, &tmK, hf * 64, hk, block_at(j) * kF2Tile, b, bar_kfull + 8 * s);
-        mbar_arrive_expect_tx(bar_vfull + 8 * s, L::kVTileBytes);
+        if (DR > 0)
+          tma_load_4d(sK + s * L::kTileBytes + (D / 64) * L::kHalf, &tmKr, 0, 0, block_at(j) * kF2Tile, b, bar_kfull + 8 * s);
+        const int v = (j - f_min) % kVStages, vuse = (j - f_min) / kVStages;
+        if (!mbar_wait(bar_vempty + 8 * v, (vuse & 1) ^ 1, abort_flag, status, 49)) break;
+        mbar_arrive_expect_tx(bar_vfull + 8 * v, L::kVTileBytes);
 #pragma unroll
         for (int hf = 0; hf < DV / 64; ++hf)
-          tma_load_4d(sV + s * L::kVTileBytes + hf * L::kHalf, &tmV, hf * 64, hk, block_at(j) * kF2Tile, b, bar_vfull + 8 * s);
+          tma_load_4d(sV + v * L::kVTileBytes + hf * L::kHalf, &tmV, hf * 64, hk, block_at(j) * kF2Tile, b, bar_vfull + 8 * v);
       }
     }
   } else if (warp == 9) {
@@ -319,8 +335,9 @@ attn_fwd2_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
         if (!mbar_wait(bar_kfull + 8 * s, ((j - f_min) / kStages) & 1, abort_flag, status, 42)) return false;
         tc_fence_after();
 #pragma unroll
-        for (int ks = 0; ks < D / 16; ++ks) {
-          if (RULE && ks * 16 >= p.dk) break;               // the rest of the columns is zero
+        for (int ks = 0; ks < (D + DR) / 16; ++ks) {
+          if (RULE && ks < D / 16 && ks * 16 >= p.dk) continue;            // the rest of the columns is zero
+          if (DR > 0 && ks >= D / 16 && (ks - D / 16) * 16 >= p.dr) continue;
           const uint32_t off = (ks >> 2) * L::kHalf + (ks & 3) * 32;
           umma_bf16_ss(tmem_base + t * 128, umma_smem_desc_sw128(sQ + t * L::kTileBytes + off, 16, 1024),
                        umma_smem_desc_sw128(sK + s * L::kTileBytes + off, 16, 1024), idesc_qk, ks != 0 ? 1u : 0u);
@@ -335,9 +352,10 @@ attn_fwd2_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
         ok = mbar_wait(bar_q + 8 * t, 0, abort_flag, status, 43);
         if (ok && f_of(t) == f_min) ok = issue_qk(f_min, t);  // a tile that starts later gets its first product below
       }
+      if (ok && f_min < n_max) umma_commit(bar_kempty);                          // the first key block: every product that reads it has been issued
       for (int j = f_min; j < n_max && ok; ++j) {
-        const int s = (j - f_min) % kStages;
-        if (!mbar_wait(bar_vfull + 8 * s, ((j - f_min) / kStages) & 1, abort_flag, status, 44)) break;
+        const int v = (j - f_min) % kVStages;
+        if (!mbar_wait(bar_vfull + 8 * v, ((j - f_min) / kVStages) & 1, abort_flag, status, 44)) break;
 #pragma unroll
         for (int t = 0; t < 2; ++t) {
           if (j >= n_of(t) || !ok) continue;
@@ -352,13 +370,15 @@ attn_fwd2_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
 #pragma unroll
           for (int ks = 0; ks < kF2Tile / 16; ++ks) {
             // V: 16 key rows of 128 B per step; 64-wide head-dim atoms L::kHalf apart
-            const uint64_t db = umma_smem_desc_sw128(sV + s * L::kVTileBytes + ks * 2048, L::kHalf, 1024);
+            const uint64_t db = umma_smem_desc_sw128(sV + v * L::kVTileBytes + ks * 2048, L::kHalf, 1024);
             umma_bf16_ts(tmem_o, tmem_p + ks * 8, db, idesc_pv, (j > f_of(t) || ks != 0) ? 1u : 0u);
           }
           umma_commit(bar_oready + 8 * t);
           if (j + 1 < n_of(t)) ok = issue_qk(j + 1, t);          // overwrites S_t / P_t: ordered behind PV(j, t)
         }
-        if (ok) umma_commit(bar_kvempty + 8 * s);               // every MMA that read stage s has been issued
+        if (!ok) break;
+        umma_commit(bar_vempty + 8 * v);                        // every MMA that reads this V stage, and the next K stage, is issued
+        if (j + 1 < n_max) umma_commit(bar_kempty + 8 * ((j + 1 - f_min) % kStages));
       }
     }
   }
@@ -372,8 +392,9 @@ attn_fwd2_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
     const uint32_t lane_off = static_cast<uint32_t>(wq * 32) << 16;
     const uint32_t tmem_s = tmem_base + t * 128 + lane_off;
     const uint32_t tmem_o = tmem_base + 256 + t * 128 + lane_off;
-    // RULE: scores are turned into log2 units when they are read (cap, bias), so the softmax runs with scale 1
-    const float sl2 = RULE ? 1.f : p.scale * kF2Log2e;
+    // RULE: scores with a cap or a bias are turned into log2 units when they are read, so the softmax runs with scale 1
+    const bool shaped = RULE && (p.softcap > 0.f || p.slopes != nullptr);
+    const float sl2 = shaped ? 1.f : p.scale * kF2Log2e;
     const float rule_c1 = RULE && p.softcap > 0.f ? p.scale / p.softcap : 0.f;
     const float rule_c2 = RULE ? (p.softcap > 0.f ? p.softcap : p.scale) * kF2Log2e : 0.f;
     const float slope2 = RULE && p.slopes ? p.slopes[h] * kF2Log2e : 0.f;
@@ -420,7 +441,7 @@ attn_fwd2_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
             tmem_ld_wait();
             f2_cap_scores_wide(r, rule_c1, rule_c2, slope2, bias0);
           }
-        } else {
+        } else if (shaped) {
 #pragma unroll
           for (int i = 0; i < 128; ++i)
             r[i] = __float_as_uint(fmaf(__uint_as_float(r[i]), rule_c2, fmaf(slope2, static_cast<float>(i), bias0)));
@@ -582,11 +603,11 @@ const CUtensorMap* f2_make_map(const void* base, const long long* strides, int s
   return rbhost::get_tmap_4d(base, 2, dims, str, box, 1, err);
 }
 
-template <int D, int DV, int P, bool RULE>
+template <int D, int DV, int P, bool RULE, int DR = 0>
 int f2_launch(const CUtensorMap* tq, const CUtensorMap* tk, const CUtensorMap* tv, const rb::F2Params& p, dim3 grid,
-              cudaStream_t stream) {
-  auto kern = rb::attn_fwd2_kernel<D, DV, P, RULE>;
-  const int smem = rb::F2Smem<D, DV>::kTotal + 1024;
+              cudaStream_t stream, const CUtensorMap* tqr = nullptr, const CUtensorMap* tkr = nullptr) {
+  auto kern = rb::attn_fwd2_kernel<D, DV, P, RULE, DR>;
+  const int smem = rb::F2Smem<D + DR, DV>::kTotal + 1024;
   static bool cfg_dev[64] = {false};
   bool& cfg = cfg_dev[rbhost::device_slot()];
   if (!cfg) {
@@ -594,7 +615,7 @@ int f2_launch(const CUtensorMap* tq, const CUtensorMap* tk, const CUtensorMap* t
     if (e != cudaSuccess) return static_cast<int>(e);
     cfg = true;
   }
-  kern<<<grid, rb::kF2Threads, smem, stream>>>(*tq, *tk, *tv, p, rbhost::status_ptr());
+  kern<<<grid, rb::kF2Threads, smem, stream>>>(*tq, *tk, *tv, tqr ? *tqr : *tq, tkr ? *tkr : *tk, p, rbhost::status_ptr());
   return static_cast<int>(cudaGetLastError());
 }
 }  // namespace
@@ -663,6 +684,11 @@ RB_API int rb_attention_fwd_rule(const RbAttnArgs* a, const RbAttnRule* r, void*
     for (int j = 0; j < 3; ++j)
       if (strs[i][j] % 8 || strs[i][j] <= 0) return -9;            // TMA strides are multiples of 16 bytes
   if (r->gate && r->ld_gate % 8) return -9;
+  const int dr = r->rot_dim;
+  if (dr) {
+    if (dr < 0 || a->batch != 1 || !r->k_rot || r->softcap > 0.f || r->slopes || r->window || r->chunk) return -1;
+    if (dr > 64 || (dr & 7) || r->ld_k_rot % 8 || r->ld_k_rot < dr || (reinterpret_cast<uintptr_t>(r->k_rot) & 15)) return -9;
+  }
   int err = 0;
   const CUtensorMap* tq = f2_make_map(a->q, a->q_strides, a->seq_q, a->heads, a->batch, dk, &err);
   const CUtensorMap* tk = f2_make_map(a->k, a->k_strides, a->seq_k, a->kv_heads, a->batch, dk, &err);
@@ -675,9 +701,21 @@ RB_API int rb_attention_fwd_rule(const RbAttnArgs* a, const RbAttnRule* r, void*
   p.scale = a->scale;
   p.dk = dk; p.dv = dv; p.softcap = r->softcap; p.slopes = r->slopes; p.chunk = r->chunk;
   p.gate = reinterpret_cast<const __nv_bfloat16*>(r->gate); p.ld_gate = r->ld_gate;
-  p.head_gate = r->head_gate; p.window = r->window; p.keep = r->window > 0 ? r->keep_first : 0; p.sink = r->sink;
+  p.dr = dr; p.head_gate = r->head_gate; p.window = r->window; p.keep = r->window > 0 ? r->keep_first : 0; p.sink = r->sink;
   cudaStream_t stream = reinterpret_cast<cudaStream_t>(stream_v);
   const dim3 grid((a->seq_q + 2 * rb::kF2Tile - 1) / (2 * rb::kF2Tile), a->heads, a->batch);
+  if (dr) {
+    const long long qr_s[3] = {a->q_strides[0], a->q_strides[1], a->q_strides[2]};
+    const long long kr_s[3] = {r->ld_k_rot * a->seq_k, r->ld_k_rot, r->ld_k_rot};
+    const CUtensorMap* tqr = f2_make_map(reinterpret_cast<const __nv_bfloat16*>(a->q) + dk, qr_s, a->seq_q, a->heads, 1, dr, &err);
+    const CUtensorMap* tkr = f2_make_map(r->k_rot, kr_s, a->seq_k, 1, 1, dr, &err);
+    if (!tqr || !tkr) return err ? err : -5;
+    if (dk <= 64)
+      return dv <= 64 ? f2_launch<64, 64, 0, true, 64>(tq, tk, tv, p, grid, stream, tqr, tkr)
+                      : f2_launch<64, 128, 0, true, 64>(tq, tk, tv, p, grid, stream, tqr, tkr);
+    return dv <= 64 ? f2_launch<128, 64, 0, true, 64>(tq, tk, tv, p, grid, stream, tqr, tkr)
+                    : f2_launch<128, 128, 0, true, 64>(tq, tk, tv, p, grid, stream, tqr, tkr);
+  }
   if (dk <= 64)
     return dv <= 64 ? f2_launch<64, 64, 0, true>(tq, tk, tv, p, grid, stream) : f2_launch<64, 128, 0, true>(tq, tk, tv, p, grid, stream);
   return dv <= 64 ? f2_launch<128, 64, 0, true>(tq, tk, tv, p, grid, stream) : f2_launch<128, 128, 0, true>(tq, tk, tv, p, grid, stream);

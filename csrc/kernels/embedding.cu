@@ -153,7 +153,7 @@ namespace rb {
 template <typename T>
 __global__ void __launch_bounds__(128)
 embedding_residual_kernel(const long long* __restrict__ ids, const T* __restrict__ table, float* __restrict__ x,
-                          T* __restrict__ h, long long tokens, int dim, long long vocab, float scale RB_BOUNDS_PARAM) {
+                          T* __restrict__ h, long long ld_h, long long tokens, int dim, long long vocab, float scale RB_BOUNDS_PARAM) {
   const long long total = tokens * dim;
   const long long stride = static_cast<long long>(gridDim.x) * blockDim.x;
   for (long long i = static_cast<long long>(blockIdx.x) * blockDim.x + threadIdx.x; i < total; i += stride) {
@@ -166,12 +166,12 @@ embedding_residual_kernel(const long long* __restrict__ ids, const T* __restrict
     }
     const T v = table[id * dim + c];
     x[i] = scale * static_cast<float>(v);
-    if (h) h[i] = static_cast<T>(x[i]);
+    if (h) h[t * ld_h + c] = static_cast<T>(x[i]);
   }
 }
 }  // namespace rb
 
-RB_API int rb_embedding_residual(const long long* ids, const void* table, int table_f32, float* x, void* h, long long tokens,
+RB_API int rb_embedding_residual(const long long* ids, const void* table, int table_f32, float* x, void* h, long long ld_h, long long tokens,
                                  int dim, long long vocab, float scale, void* stream_v) {
   if (tokens <= 0 || dim <= 0 || vocab <= 0) return -1;
   cudaStream_t stream = reinterpret_cast<cudaStream_t>(stream_v);
@@ -179,10 +179,10 @@ RB_API int rb_embedding_residual(const long long* ids, const void* table, int ta
   if (blocks > 148LL * 32) blocks = 148LL * 32;
   if (table_f32)
     rb::embedding_residual_kernel<float><<<static_cast<int>(blocks), 128, 0, stream>>>(
-        ids, reinterpret_cast<const float*>(table), x, reinterpret_cast<float*>(h), tokens, dim, vocab, scale RB_BOUNDS_ARG);
+        ids, reinterpret_cast<const float*>(table), x, reinterpret_cast<float*>(h), ld_h, tokens, dim, vocab, scale RB_BOUNDS_ARG);
   else
     rb::embedding_residual_kernel<__nv_bfloat16><<<static_cast<int>(blocks), 128, 0, stream>>>(
-        ids, reinterpret_cast<const __nv_bfloat16*>(table), x, reinterpret_cast<__nv_bfloat16*>(h), tokens, dim, vocab, scale
+        ids, reinterpret_cast<const __nv_bfloat16*>(table), x, reinterpret_cast<__nv_bfloat16*>(h), ld_h, tokens, dim, vocab, scale
         RB_BOUNDS_ARG);
   return static_cast<int>(cudaGetLastError());
 }

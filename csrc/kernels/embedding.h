@@ -7,9 +7,9 @@ extern "C" {
 int rb_embedding_fwd(const long long* ids, const void* wte, const void* wpe, void* out, long long tokens, int dim,
                      int seq_len, long long vocab, void* stream);
 // Start of a 32-bit residual stream: x[t, :] = scale * table[ids[t], :], and h[t, :] = the same row in the table's type
-// when h != NULL (operand of the first matrix products).  table bf16 or fp32.
-int rb_embedding_residual(const long long* ids, const void* table, int table_f32, float* x, void* h, long long tokens, int dim,
-                          long long vocab, float scale, void* stream);
+// (pitch ld_h) when h != NULL (operand of the first matrix products).  table bf16 or fp32.
+int rb_embedding_residual(const long long* ids, const void* table, int table_f32, float* x, void* h, long long ld_h,
+                          long long tokens, int dim, long long vocab, float scale, void* stream);
 // Ints of scratch rb_embedding_bwd needs for `tokens` ids over a table of `vocab` rows.
 long long rb_embedding_bwd_scratch_ints(long long tokens, long long vocab);
 // dwte[ids[t], :] += dy[t, :] (fp32 accumulate, rows visited in ascending t: bit-reproducible);

@@ -13,7 +13,7 @@ constexpr int kSgTile = 64, kSgK = 16;
 
 __global__ void __launch_bounds__(256)
 gemm_f32_kernel(const float* __restrict__ a, long long lda, const float* __restrict__ b, long long ldb, float* __restrict__ d,
-                long long ldd, int M, int N, int K, float alpha, const int* __restrict__ tile_expert,
+                long long ldd, int M, int N, int K, float alpha, const float* __restrict__ bias, int relu2, const int* __restrict__ tile_expert,
                 const int* __restrict__ num_m_tiles, long long b_expert_stride) {
   __shared__ float as[kSgK][kSgTile + 4], bs[kSgK][kSgTile + 4];
   const int n0 = blockIdx.x * kSgTile;
@@ -59,7 +59,10 @@ gemm_f32_kernel(const float* __restrict__ a, long long lda, const float* __restr
 #pragma unroll
     for (int j = 0; j < 4; ++j) {
       const int n = n0 + tx * 4 + j;
-      if (n < N) d[static_cast<long long>(m) * ldd + n] = alpha * acc[i][j];
+      if (n >= N) continue;
+      float v = alpha * acc[i][j] + (bias ? bias[n] : 0.f);
+      if (relu2) { v = fmaxf(v, 0.f); v *= v; }
+      d[static_cast<long long>(m) * ldd + n] = v;
     }
   }
 }
@@ -67,13 +70,13 @@ gemm_f32_kernel(const float* __restrict__ a, long long lda, const float* __restr
 }  // namespace rb
 
 RB_API int rb_gemm_f32(const float* a, long long lda, const float* b, long long ldb, float* d, long long ldd, int M, int N,
-                       int K, float alpha, const int* tile_expert, const int* num_m_tiles, long long b_expert_stride,
+                       int K, float alpha, const float* bias, int relu2, const int* tile_expert, const int* num_m_tiles, long long b_expert_stride,
                        void* stream_v) {
   if (M <= 0 || N <= 0 || K <= 0 || !a || !b || !d) return -1;
   if (tile_expert && (!num_m_tiles || b_expert_stride <= 0)) return -8;
   const dim3 grid((N + rb::kSgTile - 1) / rb::kSgTile, (M + rb::kSgTile - 1) / rb::kSgTile);
   if (grid.y > 65535) return -1;
-  rb::gemm_f32_kernel<<<grid, 256, 0, reinterpret_cast<cudaStream_t>(stream_v)>>>(a, lda, b, ldb, d, ldd, M, N, K, alpha,
+  rb::gemm_f32_kernel<<<grid, 256, 0, reinterpret_cast<cudaStream_t>(stream_v)>>>(a, lda, b, ldb, d, ldd, M, N, K, alpha, bias, relu2,
                                                                                  tile_expert, num_m_tiles, b_expert_stride);
   return static_cast<int>(cudaGetLastError());
 }

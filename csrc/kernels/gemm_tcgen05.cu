@@ -181,7 +181,7 @@ __device__ __forceinline__ void epilogue_math(const EpiParams& ep, uint32_t (&r)
 
   if (PRE_ONLY) return;
 
-  if (ep.act == RB_ACT_GELU || ep.act == RB_ACT_RELU || ep.act == RB_ACT_SILU) {
+  if (ep.act == RB_ACT_GELU || ep.act == RB_ACT_RELU || ep.act == RB_ACT_SILU || ep.act == RB_ACT_RELU2) {
     if (ep.aux_out != nullptr) {   // keep the pre-activation for the backward pass
       __nv_bfloat16* ap = ep.aux_out + row * ep.ld_aux_out + col0;
       if (!STORE_AUX) {
@@ -208,6 +208,9 @@ __device__ __forceinline__ void epilogue_math(const EpiParams& ep, uint32_t (&r)
     } else if (ep.act == RB_ACT_RELU) {
 #pragma unroll
       for (int j = 0; j < 32; ++j) v[j] = fmaxf(v[j], 0.f);
+    } else if (ep.act == RB_ACT_RELU2) {
+#pragma unroll
+      for (int j = 0; j < 32; ++j) { const float r = fmaxf(v[j], 0.f); v[j] = r * r; }
     } else {
 #pragma unroll
       for (int j = 0; j < 32; ++j) v[j] = silu(v[j]);
@@ -1500,6 +1503,7 @@ RB_API int rb_gemm_bf16(const RbGemmArgs* args, void* stream_v) {
   if (g.a_scale && (reinterpret_cast<uintptr_t>(g.a_scale) & 3)) return -3;
   if (g.b_scale && (reinterpret_cast<uintptr_t>(g.b_scale) & 15)) return -3;
   if ((g.act >= RB_ACT_DGELU && g.act <= RB_ACT_MUL) && !g.aux_in) return -4;
+  if (g.act == RB_ACT_RELU2 && g.aux_out) return -4;
 
   if (g.group_mode < 0 || g.group_mode > 2) return -8;
   if (g.group_mode == 1 && (!g.tile_expert || !g.num_m_tiles || g.b_expert_rows <= 0)) return -8;

@@ -13,7 +13,8 @@ enum RbAct {
   RB_ACT_DGELU = 4,   // multiply the result by gelu'(aux_in)
   RB_ACT_DRELU = 5,   // zero the result where aux_in <= 0
   RB_ACT_DSILU = 6,   // multiply the result by silu'(aux_in)
-  RB_ACT_MUL = 7      // multiply the result by aux_in
+  RB_ACT_MUL = 7,     // multiply the result by aux_in
+  RB_ACT_RELU2 = 8    // the square of relu (inference: no pre-activation is kept)
 };
 
 typedef struct RbGemmArgs {

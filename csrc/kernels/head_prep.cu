@@ -1,6 +1,6 @@
 // Per-head work between the packed attention projection and the attention kernels, in one pass: RMS norm of every query
-// and key head, mixing of the values with an earlier layer's values of the same token, and the append of keys and values
-// to their cache slots.  Norms and mixing are fp32.  A group of 8 or 16 lanes owns one head of one token with 16-byte accesses;
+// and key head, rotary positions on them (neighbours paired, cosines and sines from a table that all layers share), mixing of the
+// values with an earlier layer's values of the same token, and the append of keys and values to their cache slots.  All of it is fp32.  A group of 8 or 16 lanes owns one head of one token with 16-byte accesses;
 // head sizes that are not whole vectors take the scalar form (one warp per head).
 #include "head_prep.h"
 
@@ -42,8 +42,15 @@ __device__ __forceinline__ void hp_put(float* p, float v) { *p = v; }
 struct HpItem {
   int kind, head;                                  // 0 query, 1 key, 2 value
 };
-// query heads without a norm need no work at all
-__host__ __device__ __forceinline__ int hp_queries(const RbHeadPrepArgs& a) { return a.q_gamma ? a.heads : 0; }
+// query heads without a norm and positions need no work at all
+__host__ __device__ __forceinline__ int hp_queries(const RbHeadPrepArgs& a) { return a.q_gamma || a.rot ? a.heads : 0; }
+// (u, v) at columns c, c + 1 of token t
+__device__ __forceinline__ void hp_rotate(const RbHeadPrepArgs& a, long long t, int c, float& u, float& v) {
+  const float2 cs = __ldg(reinterpret_cast<const float2*>(a.rot + t * a.rot_dims + c));
+  const float x = u;
+  u = x * cs.x - v * cs.y;
+  v = v * cs.x + x * cs.y;
+}
 __device__ __forceinline__ HpItem hp_item(int i, const RbHeadPrepArgs& a) {
   if (i < hp_queries(a)) return {0, i};
   i -= hp_queries(a);
@@ -68,12 +75,15 @@ head_prep_kernel(const RbHeadPrepArgs a RB_BOUNDS_PARAM) {
     const int dim = it.kind == 2 ? a.dv : a.dk;
     const long long off = it.kind == 0 ? a.off_q : it.kind == 1 ? a.off_k : a.off_v;
     T* row = reinterpret_cast<T*>(a.p) + t * a.ld + off + static_cast<long long>(it.head) * dim;
+    const T* gamma = reinterpret_cast<const T*>(it.kind == 0 ? a.q_gamma : it.kind == 1 ? a.k_gamma : nullptr);
+    const int rotated = it.kind != 2 && a.rot ? a.rot_dims : 0;
+    const int used = it.kind == 0 && !gamma ? rotated : dim;   // the rest of a query without a norm stays as it is
     float v[kHpMaxVec][V::N];
     float sq = 0.f;
 #pragma unroll
     for (int c = 0; c < kHpMaxVec; ++c) {
       const int col = (c * LANES + sub) * V::N;
-      if (live && col < dim) {
+      if (live && col < used) {
         V::load(row + col, v[c]);
 #pragma unroll
         for (int i = 0; i < V::N; ++i) sq += v[c][i] * v[c][i];
@@ -82,7 +92,6 @@ head_prep_kernel(const RbHeadPrepArgs a RB_BOUNDS_PARAM) {
 #pragma unroll
     for (int o = LANES / 2; o > 0; o >>= 1) sq += __shfl_xor_sync(0xffffffffu, sq, o);
     if (!live) continue;
-    const T* gamma = reinterpret_cast<const T*>(it.kind == 0 ? a.q_gamma : it.kind == 1 ? a.k_gamma : nullptr);
     const bool mixed = it.kind == 2 && a.v_first != nullptr;
     const float rstd = gamma ? rsqrtf(sq / static_cast<float>(dim) + a.eps) : 1.f;
     const float lam = mixed ? a.mix[0] : 0.f;
@@ -97,7 +106,7 @@ head_prep_kernel(const RbHeadPrepArgs a RB_BOUNDS_PARAM) {
 #pragma unroll
     for (int c = 0; c < kHpMaxVec; ++c) {
       const int col = (c * LANES + sub) * V::N;
-      if (col >= dim) continue;
+      if (col >= used) continue;
       if (gamma) {
         float w[V::N];
         V::load(gamma + col, w);
@@ -110,13 +119,18 @@ head_prep_kernel(const RbHeadPrepArgs a RB_BOUNDS_PARAM) {
 #pragma unroll
         for (int i = 0; i < V::N; ++i) v[c][i] = (1.f - lam) * v[c][i] + lam * w[i];
       }
-      if (gamma || mixed) V::store(row + col, v[c]);
+      if (col < rotated) {
+#pragma unroll
+        for (int i = 0; i < V::N; i += 2)
+          if (col + i < rotated) hp_rotate(a, t, col + i, v[c][i], v[c][i + 1]);
+      }
+      if (gamma || mixed || col < rotated) V::store(row + col, v[c]);
       if (cache) V::store(cache + col, v[c]);
     }
   }
 }
 
-// any head size and alignment: one warp per head, element by element
+// any head size and alignment: one warp per head, pair by pair
 template <typename T>
 __global__ void __launch_bounds__(128)
 head_prep_scalar_kernel(const RbHeadPrepArgs a RB_BOUNDS_PARAM) {
@@ -146,13 +160,21 @@ head_prep_scalar_kernel(const RbHeadPrepArgs a RB_BOUNDS_PARAM) {
       if (slot >= 0 && slot < a.num_slots)
         cache = reinterpret_cast<T*>(it.kind == 1 ? a.k_cache : a.v_cache) + (slot * a.kv_heads + it.head) * dim;
     }
-    for (int c = lane; c < dim; c += 32) {
-      float x = hp_get(row + c);
-      if (gamma) x = x * rstd * hp_get(gamma + c);
-      if (mixed) x = (1.f - lam) * x + lam * hp_get(reinterpret_cast<const T*>(a.v_first) + t * a.ld_vf +
-                                                    static_cast<long long>(it.head) * dim + c);
-      hp_put(row + c, x);
-      if (cache) hp_put(cache + c, x);
+    const int rotated = it.kind != 2 && a.rot ? a.rot_dims : 0;
+    for (int c = 2 * lane; c < dim; c += 64) {
+      float x[2] = {0.f, 0.f};
+      const int n = min(2, dim - c);
+      for (int i = 0; i < n; ++i) {
+        x[i] = hp_get(row + c + i);
+        if (gamma) x[i] = x[i] * rstd * hp_get(gamma + c + i);
+        if (mixed) x[i] = (1.f - lam) * x[i] + lam * hp_get(reinterpret_cast<const T*>(a.v_first) + t * a.ld_vf +
+                                                            static_cast<long long>(it.head) * dim + c + i);
+      }
+      if (c < rotated) hp_rotate(a, t, c, x[0], x[1]);
+      for (int i = 0; i < n; ++i) {
+        hp_put(row + c + i, x[i]);
+        if (cache) hp_put(cache + c + i, x[i]);
+      }
     }
   }
 }
@@ -185,6 +207,7 @@ RB_API int rb_head_prep(const RbHeadPrepArgs* args, void* stream_v) {
   const RbHeadPrepArgs& a = *args;
   if (a.tokens <= 0) return 0;
   if (!a.p || a.heads <= 0 || a.kv_heads <= 0 || a.dk <= 0 || a.dv <= 0) return -1;
+  if (a.rot && (a.rot_dims <= 0 || (a.rot_dims & 1) || a.rot_dims > a.dk || (reinterpret_cast<uintptr_t>(a.rot) & 7))) return -1;
   if ((a.k_cache == nullptr) != (a.v_cache == nullptr) || (a.k_cache && !a.slots) || (a.v_first && !a.mix)) return -1;
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream_v);
   return a.f32 ? rb::hp_launch<float>(a, s) : rb::hp_launch<__nv_bfloat16>(a, s);

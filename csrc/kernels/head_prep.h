@@ -12,11 +12,13 @@ typedef struct RbHeadPrepArgs {
   void* k_cache;              // [num_slots, kv_heads, dk] / [num_slots, kv_heads, dv], type of p, or both NULL
   void* v_cache;
   const long long* slots;     // cache slot of every token (negative: not stored)
+  const float* rot;           // [tokens, rot_dims / 2] pairs (cos, sin) (rb_rotary_table), or NULL: queries and keys are not rotated
   long long ld, off_q, off_k, off_v, ld_vf, tokens, num_slots;
-  int f32, heads, kv_heads, dk, dv;
+  int f32, heads, kv_heads, dk, dv, rot_dims;
   float eps;
 } RbHeadPrepArgs;
-// In place: q <- rms(q) * q_gamma, k <- rms(k) * k_gamma, v <- (1 - mix) v + mix v_first; k and v also go to their slots.
+// In place: q <- rms(q) * q_gamma, k <- rms(k) * k_gamma, then neighbouring pairs of their first rot_dims numbers are rotated;
+// v <- (1 - mix) v + mix v_first; k and v also go to their slots.
 int rb_head_prep(const RbHeadPrepArgs* args, void* stream);
 #ifdef __cplusplus
 }

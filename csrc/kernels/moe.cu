@@ -185,11 +185,114 @@ moe_route_groups_kernel(const float* __restrict__ logits, int T, int E, int k, i
   }
 }
 
-// act(gate) * up over the rows that hold a token; act: silu, or relu
-template <typename T, int N, bool RELU>
+// Router with sigmoid scores: one warp per token, R experts per lane.  Choice scores can have either sign, so their keys are the
+// float's bits mapped to unsigned order (0 = not available).
+__device__ __forceinline__ unsigned int route_key(float v) {
+  const unsigned int b = __float_as_uint(v);
+  return b & 0x80000000u ? ~b : b | 0x80000000u;
+}
+__device__ __forceinline__ float route_unkey(unsigned int k) { return __uint_as_float(k & 0x80000000u ? k & 0x7fffffffu : ~k); }
+template <int R>
+__global__ void __launch_bounds__(128)
+moe_route_sigmoid_kernel(const float* __restrict__ logits, const float* __restrict__ correction, int T, int E, int k, int groups, int keep,
+                         int group_best, int renorm, float eps, int* __restrict__ idx, float* __restrict__ w) {
+  extern __shared__ unsigned int route_sm[];
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+  const int t = blockIdx.x * (blockDim.x >> 5) + warp;
+  if (t >= T) return;
+  const float* x = logits + static_cast<long long>(t) * E;
+  float s[R];
+  unsigned int key[R];
+#pragma unroll
+  for (int r = 0; r < R; ++r) {
+    const int e = lane + 32 * r;
+    s[r] = e < E ? 1.f / (1.f + expf(-x[e])) : 0.f;
+    key[r] = e < E ? route_key(s[r] + (correction ? correction[e] : 0.f)) : 0u;
+  }
+  if (groups > 1 && keep < groups) {
+    unsigned int* all = route_sm + warp * (E + groups);
+    unsigned int* gkey = all + E;
+    const int per = E / groups;
+#pragma unroll
+    for (int r = 0; r < R; ++r)
+      if (lane + 32 * r < E) all[lane + 32 * r] = key[r];
+    __syncwarp();
+    for (int g = lane; g < groups; g += 32) {
+      unsigned int m0 = 0u, m1 = 0u;
+      for (int e = g * per; e < (g + 1) * per; ++e) {
+        const unsigned int v = all[e];
+        m1 = max(m1, min(m0, v));
+        m0 = max(m0, v);
+      }
+      float sum = route_unkey(m0);
+      if (group_best > 1 && m1 != 0u) sum += route_unkey(m1);
+      gkey[g] = route_key(sum);
+    }
+    __syncwarp();
+    for (int j = 0; j < keep; ++j) {                   // the best groups, ties to the lower one, end up as 0
+      unsigned int bv = 0u;
+      int bi = groups;
+      for (int g = lane; g < groups; g += 32)
+        if (gkey[g] > bv) { bv = gkey[g]; bi = g; }
+      const unsigned int best = __reduce_max_sync(0xffffffffu, bv);
+      const int at = __reduce_min_sync(0xffffffffu, bv == best ? bi : groups);
+      if (at < groups && (at & 31) == lane) gkey[at] = 0u;
+      __syncwarp();
+    }
+#pragma unroll
+    for (int r = 0; r < R; ++r)
+      if (lane + 32 * r < E && gkey[(lane + 32 * r) / per] != 0u) key[r] = 0u;
+  }
+  float tot = 0.f, mine = 0.f;                         // lane j keeps the j-th weight (written in rounds of 32)
+  int mine_e = 0;
+  for (int j = 0; j < k; ++j) {
+    unsigned int bv = 0u;
+    int bi = E;
+    float bs = 0.f;
+#pragma unroll
+    for (int r = 0; r < R; ++r)
+      if (key[r] > bv) { bv = key[r]; bi = lane + 32 * r; bs = s[r]; }
+    const unsigned int best = __reduce_max_sync(0xffffffffu, bv);
+    int at = __reduce_min_sync(0xffffffffu, bv == best ? bi : E);
+    if (at >= E) at = 0;                               // nothing available (scores that are not numbers)
+    const float p = __shfl_sync(0xffffffffu, bs, at & 31);
+#pragma unroll
+    for (int r = 0; r < R; ++r)
+      if (at == lane + 32 * r) key[r] = 0u;
+    tot += p;
+    if ((j & 31) == lane) { mine = p; mine_e = at; }
+    if (((j & 31) == 31 || j == k - 1) && (j & ~31) + lane < k) {
+      idx[static_cast<long long>(t) * k + (j & ~31) + lane] = mine_e;
+      w[static_cast<long long>(t) * k + (j & ~31) + lane] = renorm && k <= 32 ? mine / (tot + eps) : mine;
+    }
+  }
+  if (renorm && k > 32) {
+    __syncwarp();
+    for (int j = lane; j < k; j += 32) w[static_cast<long long>(t) * k + j] /= tot + eps;
+  }
+}
+
+// act(gate) * up over the rows that hold a token; ACT 0: silu, 1: relu, 2: clamped (both bounded by `limit`, up shifted by one)
+template <int ACT>
+__device__ __forceinline__ float glu(float g, float u, float limit) {
+  if (ACT == 1) return fmaxf(g, 0.f) * u;
+  if (ACT == 0) return silu(g) * u;
+  g = fminf(g, limit);
+  u = fminf(fmaxf(u, -limit), limit);
+  return __fdividef(g, 1.f + __expf(-1.702f * g)) * (u + 1.f);
+}
+template <int ACT>
+__device__ __forceinline__ float glu_exact(float g, float u, float limit) {
+  if (ACT == 1) return fmaxf(g, 0.f) * u;
+  if (ACT == 0) return g / (1.f + expf(-g)) * u;
+  g = fminf(g, limit);
+  u = fminf(fmaxf(u, -limit), limit);
+  return g / (1.f + expf(-1.702f * g)) * (u + 1.f);
+}
+template <typename T, int N, int ACT>
 __global__ void __launch_bounds__(256)
 swiglu_slots_kernel(const T* __restrict__ gu, long long ld_gu, T* __restrict__ h, long long ld_h, int n, int F,
-                    const int* __restrict__ slot_pos) {
+                    const int* __restrict__ slot_pos, float limit) {
   const int chunks = F / N;
   const long long total = static_cast<long long>(n) * chunks;
   const long long stride = static_cast<long long>(gridDim.x) * blockDim.x;
@@ -204,14 +307,14 @@ swiglu_slots_kernel(const T* __restrict__ gu, long long ld_gu, T* __restrict__ h
 #pragma unroll
       for (int j = 0; j < 4; ++j) {
         const float2 a = unpack_bf16x2(gw[j]), b = unpack_bf16x2(uw[j]);
-        o[j] = RELU ? pack_bf16x2(fmaxf(a.x, 0.f) * b.x, fmaxf(a.y, 0.f) * b.y) : pack_bf16x2(silu(a.x) * b.x, silu(a.y) * b.y);
+        o[j] = pack_bf16x2(glu<ACT>(a.x, b.x, limit), glu<ACT>(a.y, b.y, limit));
       }
       *reinterpret_cast<uint4*>(h + r * ld_h + c) = make_uint4(o[0], o[1], o[2], o[3]);
     } else {
 #pragma unroll
       for (int j = 0; j < N; ++j) {
         const float g = static_cast<float>(gu[r * ld_gu + c + j]), u = static_cast<float>(gu[r * ld_gu + F + c + j]);
-        h[r * ld_h + c + j] = static_cast<T>((RELU ? fmaxf(g, 0.f) : g / (1.f + expf(-g))) * u);
+        h[r * ld_h + c + j] = static_cast<T>(glu_exact<ACT>(g, u, limit));
       }
     }
   }
@@ -417,29 +520,48 @@ RB_API int rb_moe_route_groups(const float* logits, int T, int E, int k, int gro
   else return -1;
   return static_cast<int>(cudaGetLastError());
 }
+RB_API int rb_moe_route_sigmoid(const float* logits, const float* correction, int T, int E, int k, int groups, int keep,
+                                int group_best, int renorm, float eps, int* idx, float* w, void* stream_v) {
+  if (groups < 1) groups = 1;
+  if (keep < 1 || keep > groups) keep = groups;
+  if (T <= 0 || E <= 0 || k <= 0 || k > E || E % groups || k > keep * (E / groups) || group_best < 1 || group_best > 2) return -1;
+  const size_t smem = groups > 1 && keep < groups ? sizeof(float) * 4 * static_cast<size_t>(E + groups) : 0;
+  auto run = [&](auto kern) {
+    kern<<<(T + 3) / 4, 128, smem, RB_ST>>>(logits, correction, T, E, k, groups, keep, group_best, renorm, eps, idx, w);
+    return static_cast<int>(cudaGetLastError());
+  };
+  if (E <= 32) return run(rb::moe_route_sigmoid_kernel<1>);
+  if (E <= 64) return run(rb::moe_route_sigmoid_kernel<2>);
+  if (E <= 128) return run(rb::moe_route_sigmoid_kernel<4>);
+  if (E <= 256) return run(rb::moe_route_sigmoid_kernel<8>);
+  if (E <= 1024) return run(rb::moe_route_sigmoid_kernel<32>);
+  return -1;
+}
 namespace {
-template <bool RELU>
-int glu_launch(const void* gu, long long ld_gu, void* h, long long ld_h, int n, int F, int f32, const int* slot_pos, cudaStream_t s) {
+template <int ACT>
+int glu_launch(const void* gu, long long ld_gu, void* h, long long ld_h, int n, int F, int f32, const int* slot_pos, float limit,
+               cudaStream_t s) {
   const bool vec = !f32 && !((F | ld_gu | ld_h) & 7) && !((reinterpret_cast<uintptr_t>(gu) | reinterpret_cast<uintptr_t>(h)) & 15);
   const int grid = rb::grid1d(static_cast<long long>(n) * (vec ? F / 8 : F), 256);
   if (f32)
-    rb::swiglu_slots_kernel<float, 1, RELU><<<grid, 256, 0, s>>>(reinterpret_cast<const float*>(gu), ld_gu,
-                                                                reinterpret_cast<float*>(h), ld_h, n, F, slot_pos);
+    rb::swiglu_slots_kernel<float, 1, ACT><<<grid, 256, 0, s>>>(reinterpret_cast<const float*>(gu), ld_gu,
+                                                               reinterpret_cast<float*>(h), ld_h, n, F, slot_pos, limit);
   else if (vec)
-    rb::swiglu_slots_kernel<__nv_bfloat16, 8, RELU><<<grid, 256, 0, s>>>(reinterpret_cast<const __nv_bfloat16*>(gu), ld_gu,
-                                                                        reinterpret_cast<__nv_bfloat16*>(h), ld_h, n, F, slot_pos);
+    rb::swiglu_slots_kernel<__nv_bfloat16, 8, ACT><<<grid, 256, 0, s>>>(reinterpret_cast<const __nv_bfloat16*>(gu), ld_gu,
+                                                                       reinterpret_cast<__nv_bfloat16*>(h), ld_h, n, F, slot_pos, limit);
   else
-    rb::swiglu_slots_kernel<__nv_bfloat16, 1, RELU><<<grid, 256, 0, s>>>(reinterpret_cast<const __nv_bfloat16*>(gu), ld_gu,
-                                                                        reinterpret_cast<__nv_bfloat16*>(h), ld_h, n, F, slot_pos);
+    rb::swiglu_slots_kernel<__nv_bfloat16, 1, ACT><<<grid, 256, 0, s>>>(reinterpret_cast<const __nv_bfloat16*>(gu), ld_gu,
+                                                                       reinterpret_cast<__nv_bfloat16*>(h), ld_h, n, F, slot_pos, limit);
   return static_cast<int>(cudaGetLastError());
 }
 }  // namespace
 
 RB_API int rb_swiglu_slots(const void* gu, long long ld_gu, void* h, long long ld_h, int n, int F, int f32,
-                           const int* slot_pos, int relu, void* stream_v) {
-  if (n <= 0 || F <= 0) return -1;
-  return relu ? glu_launch<true>(gu, ld_gu, h, ld_h, n, F, f32, slot_pos, RB_ST)
-              : glu_launch<false>(gu, ld_gu, h, ld_h, n, F, f32, slot_pos, RB_ST);
+                           const int* slot_pos, int act, float limit, void* stream_v) {
+  if (n <= 0 || F <= 0 || act < 0 || act > 2) return -1;
+  if (act == 2) return glu_launch<2>(gu, ld_gu, h, ld_h, n, F, f32, slot_pos, limit, RB_ST);
+  return act == 1 ? glu_launch<1>(gu, ld_gu, h, ld_h, n, F, f32, slot_pos, limit, RB_ST)
+                  : glu_launch<0>(gu, ld_gu, h, ld_h, n, F, f32, slot_pos, limit, RB_ST);
 }
 RB_API int rb_moe_scatter(const void* x, const int* slot_pos, void* xp, int slots, int k, int dim, void* stream_v) {
   if (slots <= 0 || k <= 0 || dim <= 0 || (dim % 8)) return -1;

@@ -385,7 +385,7 @@ __device__ __forceinline__ float pr_get(const float* p) { return *p; }
 __device__ __forceinline__ void pr_put(__nv_bfloat16* p, float v) { *p = __float2bfloat16(v); }
 __device__ __forceinline__ void pr_put(float* p, float v) { *p = v; }
 
-constexpr int kPrMaxV = 16;                // value columns per lane: dv <= 512
+constexpr int kPrMaxV = 16;                // value columns per lane; heads with more than 512 take several CTAs
 
 // One warp per (row, query head): lanes are keys for the scores, value columns for the weighted sum.
 template <typename T>
@@ -401,6 +401,9 @@ paged_rows_kernel(const RbPagedRowsArgs a RB_BOUNDS_PARAM) {
   const T* qg = reinterpret_cast<const T*>(a.q) + r * a.ld_q + static_cast<long long>(h) * a.dk;
   for (int c = lane; c < a.dk; c += 32) q[c] = pr_get(qg + c);
   __syncwarp();
+  const long long ld_kc = a.ld_kc ? a.ld_kc : static_cast<long long>(a.kv_heads) * a.dk;
+  const long long ld_vc = a.ld_vc ? a.ld_vc : static_cast<long long>(a.kv_heads) * a.dv;
+  const int v0 = blockIdx.y * 32 * kPrMaxV;                            // first value column of this CTA
   const long long pos = a.row_pos[r];
   const int* table = a.block_tables + static_cast<long long>(a.row_seq[r]) * a.max_blocks;
   // visible keys are numbered without gaps: number v is key v below `kept`, else key v + gap
@@ -428,7 +431,7 @@ paged_rows_kernel(const RbPagedRowsArgs a RB_BOUNDS_PARAM) {
         blk = 0;
       }
       slot = static_cast<long long>(blk) * a.block_size + (j - bi * a.block_size);
-      const T* k = K + (slot * a.kv_heads + hk) * a.dk;
+      const T* k = K + slot * ld_kc + static_cast<long long>(hk) * a.dk;
       float d = 0.f;
       for (int c = 0; c < a.dk; ++c) d = fmaf(q[c], pr_get(k + c), d);
       s = d * a.scale;
@@ -446,11 +449,11 @@ paged_rows_kernel(const RbPagedRowsArgs a RB_BOUNDS_PARAM) {
     for (int jj = 0; jj < n; ++jj) {
       const float pj = __shfl_sync(0xffffffffu, p, jj);
       const long long sj = __shfl_sync(0xffffffffu, slot, jj);
-      const T* vals = V + (sj * a.kv_heads + hk) * a.dv;
+      const T* vals = V + sj * ld_vc + static_cast<long long>(hk) * a.dv + v0;
 #pragma unroll
       for (int i = 0; i < kPrMaxV; ++i) {
         const int c = i * 32 + lane;
-        if (c < a.dv) acc[i] = fmaf(pj, pr_get(vals + c), acc[i]);
+        if (v0 + c < a.dv) acc[i] = fmaf(pj, pr_get(vals + c), acc[i]);
       }
     }
   }
@@ -459,7 +462,7 @@ paged_rows_kernel(const RbPagedRowsArgs a RB_BOUNDS_PARAM) {
   const float inv = a.head_gate ? 1.f / (l * (1.f + expf(-a.head_gate[r * a.ld_g + h]))) : 1.f / l;
 #pragma unroll
   for (int i = 0; i < kPrMaxV; ++i) {
-    const int c = i * 32 + lane;
+    const int c = v0 + i * 32 + lane;
     if (c < a.dv) pr_put(o + c, acc[i] * inv * (g ? 1.f / (1.f + expf(-pr_get(g + c))) : 1.f));
   }
 }
@@ -470,12 +473,12 @@ RB_API int rb_paged_attention_rows(const RbPagedRowsArgs* args, void* stream_v) 
   const RbPagedRowsArgs& a = *args;
   if (a.rows <= 0) return 0;
   if (!a.q || !a.out || !a.k_cache || !a.v_cache || !a.block_tables || !a.row_seq || !a.row_pos || a.heads <= 0 ||
-      a.kv_heads <= 0 || a.heads % a.kv_heads || a.dk <= 0 || a.dv <= 0 || a.dv > 32 * rb::kPrMaxV || a.dk > 2048 ||
+      a.kv_heads <= 0 || a.heads % a.kv_heads || a.dk <= 0 || a.dv <= 0 || a.dk > 2048 ||
       a.block_size <= 0 || a.max_blocks <= 0)
     return -1;
   cudaStream_t stream = reinterpret_cast<cudaStream_t>(stream_v);
   const long long items = static_cast<long long>(a.rows) * a.heads;
-  const int grid = static_cast<int>((items + 3) / 4);
+  const dim3 grid(static_cast<unsigned int>((items + 3) / 4), (a.dv + 32 * rb::kPrMaxV - 1) / (32 * rb::kPrMaxV));
   const size_t smem = sizeof(float) * 4 * a.dk;
   if (a.f32) rb::paged_rows_kernel<float><<<grid, 128, smem, stream>>>(a RB_BOUNDS_ARG);
   else rb::paged_rows_kernel<__nv_bfloat16><<<grid, 128, smem, stream>>>(a RB_BOUNDS_ARG);

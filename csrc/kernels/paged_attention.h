@@ -51,15 +51,15 @@ int rb_paged_attention_decode_rule(const RbPagedDecodeArgs* args, void* stream);
 typedef struct RbPagedRowsArgs {
   const void* q;
   void* out;
-  const void* k_cache;       // [num_blocks, block_size, kv_heads, dk]
-  const void* v_cache;       // [num_blocks, block_size, kv_heads, dv]
+  const void* k_cache;       // [num_blocks, block_size, kv_heads, dk], consecutive slots ld_kc apart (0: kv_heads * dk)
+  const void* v_cache;       // [num_blocks, block_size, kv_heads, dv], ld_vc apart; both may be columns of one array
   const int* block_tables;   // [sequences, max_blocks]
   const int* row_seq;
   const long long* row_pos;
   const float* slopes;
   const void* gate;
   const float* head_gate;
-  long long ld_q, ld_o, ld_g, num_blocks;
+  long long ld_q, ld_o, ld_g, num_blocks, ld_kc, ld_vc;
   int f32, rows, max_blocks, heads, kv_heads, dk, dv, block_size, chunk, window, keep_first, sink;
   float scale, softcap;
 } RbPagedRowsArgs;

@@ -1,6 +1,7 @@
 // Norm on a sublayer's output, added to a 32-bit residual stream, in one pass: x += norm(source), h = copy of x for the
 // next matrix product.  The source is a plain row (attention output projection) or the weighted sum of a token's expert
 // rows plus the shared expert's row, so a routed feed-forward's combine, norm and residual add are one launch.
+// Where a norm stands in front of the next sublayer too, h is that norm of the new residual.
 // Statistics, sums and the residual are fp32; one CTA owns a row and keeps it in registers.
 //
 // The second kernel serves blocks whose sublayers are computed side by side: up to two RMS-normed outputs and a plain one are
@@ -102,6 +103,7 @@ residual_norm_kernel(const RbResidualNormArgs a) {
       for (int i = 0; i < VEC; ++i) { const float d = v[c][i] - mean; sq += d * d; }
     }
   const float rstd = rsqrtf(rn_block_sum(sq, red) * inv_n + a.eps);
+  float next = 0.f;
 #pragma unroll
   for (int c = 0; c < CH; ++c) {
     const int col = (c * blockDim.x + threadIdx.x) * VEC;
@@ -114,7 +116,24 @@ residual_norm_kernel(const RbResidualNormArgs a) {
 #pragma unroll
     for (int i = 0; i < VEC; ++i) o[i] = xr[c][i] + ((v[c][i] - mean) * rstd * g[i] + b[i]);
     if (a.x) rn_store<VEC>(a.x, t * a.ldx + col, 1, o);
-    if (a.h) rn_store<VEC>(a.h, t * a.ldh + col, a.h_f32, o);
+    if (a.next_gamma) {
+#pragma unroll
+      for (int i = 0; i < VEC; ++i) { xr[c][i] = o[i]; next = fmaf(o[i], o[i], next); }
+    } else if (a.h) {
+      rn_store<VEC>(a.h, t * a.ldh + col, a.h_f32, o);
+    }
+  }
+  if (!a.next_gamma) return;
+  const float scale = 1.f / sqrtf(rn_block_sum(next, red) * inv_n + a.eps);
+#pragma unroll
+  for (int c = 0; c < CH; ++c) {
+    const int col = (c * blockDim.x + threadIdx.x) * VEC;
+    if (col >= n) continue;
+    float g[VEC];
+    rn_load<VEC>(a.next_gamma, col, a.param_f32, g);
+#pragma unroll
+    for (int i = 0; i < VEC; ++i) g[i] *= xr[c][i] * scale;
+    rn_store<VEC>(a.h, t * a.ldh + col, a.h_f32, g);
   }
 }
 
@@ -236,9 +255,10 @@ RB_API int rb_residual_norm(const RbResidualNormArgs* args, void* stream_v) {
   const RbResidualNormArgs& a = *args;
   if (a.rows <= 0 || a.n <= 0 || !a.y || !a.gamma || (!a.x && !a.h)) return -1;
   if (a.slot_pos && (!a.slot_w || a.k <= 0)) return -1;
+  if (a.next_gamma && (!a.x || !a.h)) return -1;
   const uintptr_t bits = reinterpret_cast<uintptr_t>(a.y) | reinterpret_cast<uintptr_t>(a.add) |
                          reinterpret_cast<uintptr_t>(a.gamma) | reinterpret_cast<uintptr_t>(a.beta) |
-                         reinterpret_cast<uintptr_t>(a.x) | reinterpret_cast<uintptr_t>(a.h);
+                         reinterpret_cast<uintptr_t>(a.next_gamma) | reinterpret_cast<uintptr_t>(a.x) | reinterpret_cast<uintptr_t>(a.h);
   const bool vec = !(bits & 15) && !((a.n | a.ldy | a.ld_add | a.ldx | a.ldh) & 3);
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream_v);
   return vec ? rb::rn_launch<4>(a, s) : rb::rn_launch<1>(a, s);

@@ -11,6 +11,7 @@ typedef struct RbResidualNormArgs {
   const void* add;
   const void* gamma;        // bf16 or fp32 [n] (param_f32)
   const void* beta;         // same type, or NULL
+  const void* next_gamma;   // with x: h receives rms(new x) * next_gamma, the next sublayer's input; or NULL
   float* x;                 // fp32 residual [rows, n], updated in place: x += norm(source); NULL: no residual
   void* h;                  // copy of the new residual (without x: the normalised row), bf16 or fp32, or NULL
   long long ldy, ld_add, ldx, ldh;

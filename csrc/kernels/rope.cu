@@ -50,6 +50,55 @@ rope_kernel(__nv_bfloat16* __restrict__ x, long long ld, const long long* __rest
   }
 }
 
+// Cosines and sines of position * frequency for all pairs, once per step for every layer that shares them.  The angle is formed and
+// reduced in double precision, so it is as good at position 10^6 as at 10.
+__global__ void __launch_bounds__(256)
+rotary_table_kernel(const long long* __restrict__ positions, const double* __restrict__ freqs, float magnitude, float2* __restrict__ out,
+                    long long rows, int pairs) {
+  const long long total = rows * pairs;
+  const long long stride = static_cast<long long>(gridDim.x) * blockDim.x;
+  const double two_pi = 6.283185307179586476925;
+  for (long long i = static_cast<long long>(blockIdx.x) * blockDim.x + threadIdx.x; i < total; i += stride) {
+    const long long t = i / pairs;
+    const double a = static_cast<double>(positions[t]) * freqs[i - t * pairs];
+    float s, c;
+    sincosf(static_cast<float>(a - two_pi * rint(a / two_pi)), &s, &c);
+    out[i] = make_float2(c * magnitude, s * magnitude);
+  }
+}
+
+// One thread per PAIRS neighbouring pairs of a head; x points at the first rotated column of head 0.
+template <typename T, int PAIRS>
+__global__ void __launch_bounds__(256)
+rotate_pairs_kernel(T* __restrict__ x, long long ld, const float2* __restrict__ table, long long rows, int heads, long long pitch, int pairs) {
+  const int units = pairs / PAIRS;
+  const long long total = rows * heads * units;
+  const long long stride = static_cast<long long>(gridDim.x) * blockDim.x;
+  for (long long i = static_cast<long long>(blockIdx.x) * blockDim.x + threadIdx.x; i < total; i += stride) {
+    const int u = static_cast<int>(i % units) * PAIRS;
+    const long long th = i / units;
+    const int h = static_cast<int>(th % heads);
+    const long long t = th / heads;
+    T* p = x + t * ld + h * pitch + 2 * u;
+    const float2* cs = table + t * pairs + u;
+    if (PAIRS == 4) {                                          // bf16, 16 bytes
+      uint4 raw = *reinterpret_cast<const uint4*>(p);
+      uint32_t* w = reinterpret_cast<uint32_t*>(&raw);
+#pragma unroll
+      for (int j = 0; j < 4; ++j) {
+        const float2 a = unpack_bf16x2(w[j]), f = __ldg(cs + j);
+        w[j] = pack_bf16x2(a.x * f.x - a.y * f.y, a.y * f.x + a.x * f.y);
+      }
+      *reinterpret_cast<uint4*>(p) = raw;
+    } else {
+      const float a = static_cast<float>(p[0]), b = static_cast<float>(p[1]);
+      const float2 f = __ldg(cs);
+      p[0] = static_cast<T>(a * f.x - b * f.y);
+      p[1] = static_cast<T>(b * f.x + a * f.y);
+    }
+  }
+}
+
 __global__ void __launch_bounds__(256)
 swiglu_fwd_kernel(const __nv_bfloat16* __restrict__ gu, long long ld_gu, __nv_bfloat16* __restrict__ h, long long ld_h,
                   long long tokens, int F) {
@@ -119,6 +168,27 @@ RB_API int rb_rope(void* x, long long ld, const long long* positions, long long 
   rb::rope_kernel<<<rb::grid1d(total), 256, 0, reinterpret_cast<cudaStream_t>(stream_v)>>>(
       reinterpret_cast<__nv_bfloat16*>(x), ld, positions, tokens, heads, head_dim, seq_len < 1 ? 1 : seq_len, pos_offset,
       log2f(theta), inverse);
+  return static_cast<int>(cudaGetLastError());
+}
+
+RB_API int rb_rotary_table(const long long* positions, const double* freqs, float magnitude, float* out, long long rows, int pairs,
+                           void* stream_v) {
+  if (rows <= 0 || pairs <= 0 || (reinterpret_cast<uintptr_t>(out) & 7)) return -1;
+  rb::rotary_table_kernel<<<rb::grid1d(rows * pairs), 256, 0, reinterpret_cast<cudaStream_t>(stream_v)>>>(
+      positions, freqs, magnitude, reinterpret_cast<float2*>(out), rows, pairs);
+  return static_cast<int>(cudaGetLastError());
+}
+
+RB_API int rb_rotate_pairs(void* x, long long ld, const float* table, long long rows, int heads, long long pitch, int pairs, int f32,
+                           void* stream_v) {
+  if (rows <= 0 || heads <= 0 || pairs <= 0 || pitch < 2 * pairs || (reinterpret_cast<uintptr_t>(table) & 7)) return -1;
+  cudaStream_t s = reinterpret_cast<cudaStream_t>(stream_v);
+  const float2* cs = reinterpret_cast<const float2*>(table);
+  const bool vec = !f32 && !(pairs & 3) && !((ld | pitch) & 7) && !(reinterpret_cast<uintptr_t>(x) & 15);
+  const int grid = rb::grid1d(rows * heads * (vec ? pairs / 4 : pairs));
+  if (f32) rb::rotate_pairs_kernel<float, 1><<<grid, 256, 0, s>>>(reinterpret_cast<float*>(x), ld, cs, rows, heads, pitch, pairs);
+  else if (vec) rb::rotate_pairs_kernel<__nv_bfloat16, 4><<<grid, 256, 0, s>>>(reinterpret_cast<__nv_bfloat16*>(x), ld, cs, rows, heads, pitch, pairs);
+  else rb::rotate_pairs_kernel<__nv_bfloat16, 1><<<grid, 256, 0, s>>>(reinterpret_cast<__nv_bfloat16*>(x), ld, cs, rows, heads, pitch, pairs);
   return static_cast<int>(cudaGetLastError());
 }
 

@@ -55,13 +55,14 @@ class RbAttnArgs(C.Structure):
 
 class RbAttnRule(C.Structure):
     _fields_ = [("v_dim", c_int), ("softcap", c_float), ("slopes", c_void_p), ("chunk", c_int), ("gate", c_void_p),
-                ("head_gate", c_void_p), ("ld_gate", c_ll), ("window", c_int), ("keep_first", c_int), ("sink", c_int)]
+                ("head_gate", c_void_p), ("ld_gate", c_ll), ("window", c_int), ("keep_first", c_int), ("sink", c_int),
+                ("rot_dim", c_int), ("k_rot", c_void_p), ("ld_k_rot", c_ll)]
 
 
 class RbResidualNormArgs(C.Structure):
     _fields_ = [
         ("y", c_void_p), ("slot_pos", c_void_p), ("slot_w", c_void_p), ("add", c_void_p), ("gamma", c_void_p), ("beta", c_void_p),
-        ("x", c_void_p), ("h", c_void_p),
+        ("next_gamma", c_void_p), ("x", c_void_p), ("h", c_void_p),
         ("ldy", c_ll), ("ld_add", c_ll), ("ldx", c_ll), ("ldh", c_ll),
         ("y_f32", c_int), ("param_f32", c_int), ("h_f32", c_int),
         ("k", c_int), ("rows", c_int), ("n", c_int), ("rms", c_int), ("eps", c_float),
@@ -71,9 +72,9 @@ class RbResidualNormArgs(C.Structure):
 class RbHeadPrepArgs(C.Structure):
     _fields_ = [
         ("p", c_void_p), ("q_gamma", c_void_p), ("k_gamma", c_void_p), ("v_first", c_void_p), ("mix", c_void_p),
-        ("k_cache", c_void_p), ("v_cache", c_void_p), ("slots", c_void_p),
+        ("k_cache", c_void_p), ("v_cache", c_void_p), ("slots", c_void_p), ("rot", c_void_p),
         ("ld", c_ll), ("off_q", c_ll), ("off_k", c_ll), ("off_v", c_ll), ("ld_vf", c_ll), ("tokens", c_ll), ("num_slots", c_ll),
-        ("f32", c_int), ("heads", c_int), ("kv_heads", c_int), ("dk", c_int), ("dv", c_int), ("eps", c_float),
+        ("f32", c_int), ("heads", c_int), ("kv_heads", c_int), ("dk", c_int), ("dv", c_int), ("rot_dims", c_int), ("eps", c_float),
     ]
 
 
@@ -81,7 +82,7 @@ class RbPagedRowsArgs(C.Structure):
     _fields_ = [
         ("q", c_void_p), ("out", c_void_p), ("k_cache", c_void_p), ("v_cache", c_void_p), ("block_tables", c_void_p),
         ("row_seq", c_void_p), ("row_pos", c_void_p), ("slopes", c_void_p), ("gate", c_void_p), ("head_gate", c_void_p),
-        ("ld_q", c_ll), ("ld_o", c_ll), ("ld_g", c_ll), ("num_blocks", c_ll),
+        ("ld_q", c_ll), ("ld_o", c_ll), ("ld_g", c_ll), ("num_blocks", c_ll), ("ld_kc", c_ll), ("ld_vc", c_ll),
         ("f32", c_int), ("rows", c_int), ("max_blocks", c_int), ("heads", c_int), ("kv_heads", c_int), ("dk", c_int),
         ("dv", c_int), ("block_size", c_int), ("chunk", c_int), ("window", c_int), ("keep_first", c_int), ("sink", c_int),
         ("scale", c_float), ("softcap", c_float),
@@ -97,6 +98,32 @@ class RbPagedDecodeArgs(C.Structure):
         ("batch", c_int), ("max_blocks", c_int), ("heads", c_int), ("kv_heads", c_int), ("dk", c_int), ("dv", c_int),
         ("block_size", c_int), ("chunk", c_int), ("window", c_int), ("keep_first", c_int), ("sink", c_int),
         ("scale", c_float), ("softcap", c_float),
+    ]
+
+
+class RbLatentPrepArgs(C.Structure):
+    _fields_ = [
+        ("p", c_void_p), ("q_gamma", c_void_p), ("kv_gamma", c_void_p), ("table", c_void_p), ("cache", c_void_p), ("slots", c_void_p),
+        ("ld", c_ll), ("off_q", c_ll), ("off_kv", c_ll), ("tokens", c_ll), ("num_slots", c_ll),
+        ("f32", c_int), ("q_rank", c_int), ("rank", c_int), ("rot", c_int), ("pairs", c_int), ("eps", c_float),
+    ]
+
+
+class RbHeadProductArgs(C.Structure):
+    _fields_ = [
+        ("x", c_void_p), ("w", c_void_p), ("y", c_void_p), ("gate", c_void_p), ("table", c_void_p),
+        ("ld_x", c_ll), ("x_head", c_ll), ("ld_w", c_ll), ("w_head", c_ll), ("ld_y", c_ll), ("y_head", c_ll), ("ld_g", c_ll),
+        ("f32", c_int), ("rows", c_int), ("heads", c_int), ("n", c_int), ("k", c_int), ("transposed", c_int), ("tail", c_int),
+        ("tail_off", c_int), ("pairs", c_int),
+    ]
+
+
+class RbLatentDecodeArgs(C.Structure):
+    _fields_ = [
+        ("q", c_void_p), ("out", c_void_p), ("cache", c_void_p), ("block_tables", c_void_p), ("context_lens", c_void_p),
+        ("scratch", c_void_p), ("ld_q", c_ll), ("ld_o", c_ll), ("num_blocks", c_ll),
+        ("batch", c_int), ("max_blocks", c_int), ("heads", c_int), ("rank", c_int), ("rot", c_int), ("block_size", c_int),
+        ("scale", c_float),
     ]
 
 
@@ -155,7 +182,7 @@ class RbAdamArgs(C.Structure):
     ]
 
 
-ACT = {"none": 0, "gelu": 1, "relu": 2, "silu": 3, "dgelu": 4, "drelu": 5, "dsilu": 6, "mul": 7}
+ACT = {"none": 0, "gelu": 1, "relu": 2, "silu": 3, "dgelu": 4, "drelu": 5, "dsilu": 6, "mul": 7, "relu2": 8}
 
 
 class NativeError(RuntimeError):

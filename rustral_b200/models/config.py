@@ -3,7 +3,7 @@ from __future__ import annotations
 
 from dataclasses import dataclass, asdict
 
-from .layered import LayeredConfig, hybrid_layers, uniform_layers
+from .layered import LayeredConfig, LoopSpec, hybrid_layers, sandwich_layers, uniform_layers
 
 
 @dataclass
@@ -107,6 +107,22 @@ PRESETS = {
                        left=dict(heads=32, kv_heads=8, dim=128, vdim=128, scale=0.08838834764831845, window=2048, keep_first=4),
                        right=dict(heads=128, vdim=64, state=128, groups=8, norm_groups=8, conv=4),
                        delta=dict(heads=32, kv_heads=16, dim=128, vdim=128, conv=4), ff=dict(p=5376, d=12288)),
+    # layered decoders with norms around every sublayer (order: w = windowed attention, l = latent attention); layers
+    # loop.start .. loop.stop - 1 run several times
+    "bikilix-test": dict(arch="Bikilix", vocab_size=1000, d_model=128, seq_len=512, embed_scale=2.0, order="wlwl", dense=(0,), ff=192,
+                         loop=dict(start=1, stop=3, times=2),
+                         attention=dict(heads=6, kv_heads=2, dim=48, vdim=32, scale=0.15, window=40, rot=dict(dims=16, base=10000.0)),
+                         latent=dict(heads=3, dim=24, rot_dim=16, vdim=40, kv_rank=48, q_rank=56, scale=0.2,
+                                     rot=dict(dims=16, base=20000.0, factor=4.0, original=128, fast=16.0, slow=1.0, scaled=True)),
+                         moe=dict(ff=64, experts=12, top=3, groups=3, keep=2, limit=2.0)),
+    # about the size of Llama-8B layers: same width and heads; a third of the layers run twice
+    "bikilix-moe": dict(arch="Bikilix", vocab_size=128256, d_model=4096, order="wwl" * 8, dense=(0,), ff=14336,
+                        loop=dict(start=6, stop=14, times=2),
+                        attention=dict(heads=32, kv_heads=8, dim=128, vdim=128, scale=0.08838834764831845, window=2048,
+                                       rot=dict(dims=64, base=500000.0)),
+                        latent=dict(heads=32, dim=128, rot_dim=64, vdim=128, kv_rank=512, q_rank=1536, scale=0.07216878364870322,
+                                    rot=dict(dims=64, base=500000.0, factor=8.0, original=4096, fast=32.0, slow=1.0, scaled=True)),
+                        moe=dict(ff=2048, experts=32, top=7, groups=4, keep=2, limit=7.0)),
 }
 
 
@@ -116,6 +132,12 @@ def preset(name: str, **overrides):
     if "order" in cfg:
         if "n_layer" in cfg:
             cfg["order"] = (cfg["order"] * cfg["n_layer"])[:cfg.pop("n_layer")]
+        if cfg["arch"] == "Bikilix":
+            n, loop = len(cfg["order"]), cfg.pop("loop", None)
+            cfg["layers"] = sandwich_layers(*(cfg.pop(k) for k in ("order", "attention", "latent", "ff", "moe")), cfg.pop("dense", ()))
+            if loop and loop["start"] < n:
+                cfg["loop"] = LoopSpec(loop["start"], min(loop["stop"], n), loop["times"])
+            return LayeredConfig(**cfg)
         cfg["layers"] = hybrid_layers(*(cfg.pop(k) for k in ("order", "left", "right", "delta", "ff")), cfg.pop("weights_of", None))
         return LayeredConfig(**cfg)
     if "mixer" in cfg:

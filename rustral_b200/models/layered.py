@@ -10,14 +10,70 @@ every sublayer's output, added to a 32-bit residual; scaled and capped logits.
 Vafodra: one element-wise "norm" (dynamic tanh) in front of a layer whose mixer and dense feed-forward both read its output and
 are added to the residual together; mixers are sliding-window attention (first tokens kept, a sink in the softmax, one output
 gate per head) side by side with a Mamba-2 state-space mixer, or a gated delta rule; layers can share another one's tensors.
+
+Bikilix: an RMS norm in front of every sublayer and another on its output; sliding-window attention with projection biases and
+partial rotary positions, or latent attention (keys and values come from one small cached vector per token) with rotated and
+unrotated key parts and an element-wise output gate; dense squared-ReLU feed-forwards or routed experts with clamped gates, chosen by
+corrected sigmoid scores; a run of layers can be passed through several times, each pass starting from a product of the stream
+and the embedding; the embedding table is the output head.
 """
 from __future__ import annotations
 
-from dataclasses import asdict, dataclass
+import math
+from dataclasses import asdict, dataclass, field
 
 
 def up8(n: int) -> int:
     return (n + 7) // 8 * 8
+
+
+@dataclass(frozen=True)
+class RotarySpec:
+    """Rotary positions on the first `dims` numbers of a head, neighbours paired.  `factor` > 1: YaRN scaling, which leaves pairs
+    that turn at least `fast` times within `original` positions alone and slows those that turn at most `slow` times."""
+    dims: int
+    base: float
+    factor: float = 1.0
+    original: int = 0
+    fast: float = 32.0
+    slow: float = 1.0
+    scaled: bool = False
+
+    def __post_init__(self):
+        if self.dims < 0 or self.dims % 2 or self.base <= 1.0 or (self.scaled and (self.factor <= 0.0 or self.original <= 0 or self.fast <= 0.0
+                                                                                   or self.slow <= 0.0)):
+            raise ValueError(f"invalid rotary positions: {self}")
+
+    def frequencies(self) -> list:
+        """Angle per position of every pair."""
+        f = [self.base ** (-2.0 * i / self.dims) for i in range(self.dims // 2)]
+        if not self.scaled:
+            return f
+
+        def place(turns):                 # where (a fractional index) the pairs turn this often within `original` positions
+            return self.dims * math.log(self.original / (2.0 * math.pi * turns)) / (2.0 * math.log(self.base))
+        lo, hi = max(math.floor(place(self.fast)), 0), min(math.ceil(place(self.slow)), self.dims - 1)
+        ramp = [min(max((i - lo) / max(hi - lo, 0.001), 0.0), 1.0) for i in range(len(f))]
+        return [fi / self.factor * r + fi * (1.0 - r) for fi, r in zip(f, ramp)]
+
+    @property
+    def magnitude(self) -> float:
+        """Factor on cosines and sines."""
+        return 0.1 * math.log(self.factor) + 1.0 if self.scaled else 1.0
+
+    @classmethod
+    def from_json(cls, r: dict | None) -> "RotarySpec | None":
+        if not r:
+            return None
+        s = r.get("scaling")
+        kw = dict(factor=float(s["factor"]), original=int(s["original"]), fast=float(s["fast"]), slow=float(s["slow"]), scaled=True) if s else {}
+        return cls(dims=int(r["dims"]), base=float(r["base"]), **kw)
+
+    def to_json(self) -> dict:
+        r = {"dims": self.dims, "base": self.base}
+        if self.scaled:
+            r["scaling"] = {"factor": self.factor, "original": self.original, "fast": self.fast, "slow": self.slow}
+        return r
 
 
 @dataclass(frozen=True)
@@ -35,13 +91,17 @@ class AttentionSpec:
     qk_norm: bool = True         # RMS norm of every query and key head
     distance_bias: bool = True   # a linear distance bias with one slope per head
     sink: bool = False           # a further score 0 without a value in the softmax
-    gate: str = "element"        # sigmoid output gate: one number per value column ("element") or per head ("head")
+    gate: str = "element"        # sigmoid output gate: one number per value column ("element"), per head ("head"), or "none"
+    rot: RotarySpec | None = None        # rotary positions on queries and keys
+    bias: bool = False           # the query, key and value projections have biases
 
     def __post_init__(self):
         if min(self.heads, self.kv_heads, self.dim, self.vdim) < 1 or self.heads % self.kv_heads or self.chunk < 0:
             raise ValueError(f"invalid attention layer: {self}")
-        if self.window < 0 or self.keep_first < 0 or (self.window and self.chunk) or self.gate not in ("element", "head"):
+        if self.window < 0 or self.keep_first < 0 or (self.window and self.chunk) or self.gate not in ("element", "head", "none"):
             raise ValueError(f"invalid attention layer: {self}")
+        if self.rot is not None and self.rot.dims > self.dim:
+            raise ValueError(f"more rotated dimensions than a head has: {self}")
 
     @property
     def packed(self) -> int:
@@ -49,9 +109,12 @@ class AttentionSpec:
         return self.heads * self.dim + self.kv_heads * (self.dim + self.vdim) + (self.heads * self.vdim if self.gate == "element" else 0)
 
     def tensor_shapes(self, p: str, d: int) -> dict:
-        gate = self.heads * self.vdim if self.gate == "element" else self.heads
         t = {p + "q": (self.heads * self.dim, d), p + "k": (self.kv_heads * self.dim, d), p + "v": (self.kv_heads * self.vdim, d),
-             p + "g": (gate, d), p + "o": (d, self.heads * self.vdim)}
+             p + "o": (d, self.heads * self.vdim)}
+        if self.gate != "none":
+            t[p + "g"] = (self.heads * self.vdim if self.gate == "element" else self.heads, d)
+        if self.bias:
+            t.update({p + c + ".b": t[p + c][:1] for c in "qkv"})
         if self.qk_norm:
             t[p + "q.norm"] = t[p + "k.norm"] = (self.dim,)
         if self.v_mix:
@@ -65,7 +128,8 @@ class AttentionSpec:
         sliding = fixed.pop("sliding", False)
         return cls(heads=int(m["heads"]), kv_heads=int(m["kv_heads"]), dim=int(m["dim"]), vdim=int(m["vdim"]), scale=float(m["scale"]),
                    softcap=float(m.get("softcap") or 0.0), v_mix=bool(m.get("v_mix", False)), chunk=0 if sliding else size,
-                   window=size if sliding else 0, keep_first=int(mask.get("keep_first") or 0) if sliding else 0, **fixed)
+                   window=size if sliding else 0, keep_first=int(mask.get("keep_first") or 0) if sliding else 0,
+                   rot=RotarySpec.from_json(m.get("rot")), **fixed)
 
     def to_json(self) -> dict:
         m = {"heads": self.heads, "kv_heads": self.kv_heads, "dim": self.dim, "vdim": self.vdim, "scale": self.scale}
@@ -77,7 +141,56 @@ class AttentionSpec:
             m["mask"] = {"size": self.chunk}
         elif self.window:
             m["mask"] = {"size": self.window, "keep_first": self.keep_first}
+        if self.rot is not None:
+            m["rot"] = self.rot.to_json()
         return m
+
+
+@dataclass(frozen=True)
+class LatentSpec:
+    """Latent attention: keys (their unrotated part) and values of all heads are products of one normed vector per token, which is
+    what the cache holds beside a rotated key part that the heads share.  Queries come through a normed vector of their own."""
+    heads: int
+    dim: int                     # unrotated query / key size of a head
+    rot_dim: int                 # rotated query / key size
+    vdim: int
+    kv_rank: int                 # size of the cached vector
+    q_rank: int
+    scale: float
+    rot: RotarySpec
+    gate: str = "element"        # sigmoid output gate, one number per value column ("none": no gate)
+
+    def __post_init__(self):
+        if min(self.heads, self.dim, self.rot_dim, self.vdim, self.kv_rank, self.q_rank) < 1 or self.rot.dims > self.rot_dim or \
+                self.gate not in ("element", "none"):
+            raise ValueError(f"invalid latent attention layer: {self}")
+
+    @property
+    def qk_dim(self) -> int:
+        return self.dim + self.rot_dim
+
+    @property
+    def cached(self) -> int:
+        """Numbers per token in the cache."""
+        return self.kv_rank + self.rot_dim
+
+    def tensor_shapes(self, p: str, d: int) -> dict:
+        H = self.heads
+        t = {p + "dq": (self.q_rank, d), p + "dq.norm": (self.q_rank,), p + "uq": (H * self.qk_dim, self.q_rank),
+             p + "dkv": (self.cached, d), p + "dkv.norm": (self.kv_rank,), p + "uk": (H * self.dim, self.kv_rank),
+             p + "uv": (H * self.vdim, self.kv_rank), p + "o": (d, H * self.vdim)}
+        if self.gate == "element":
+            t[p + "g"] = (H * self.vdim, d)
+        return t
+
+    @classmethod
+    def from_json(cls, m: dict) -> "LatentSpec":
+        return cls(heads=int(m["heads"]), dim=int(m["dim"]), rot_dim=int(m["rot_dim"]), vdim=int(m["vdim"]), kv_rank=int(m["kv_rank"]),
+                   q_rank=int(m["q_rank"]), scale=float(m["scale"]), rot=RotarySpec.from_json(m["rot"]))
+
+    def to_json(self) -> dict:
+        m = {k: getattr(self, k) for k in ("heads", "dim", "rot_dim", "vdim", "kv_rank", "q_rank", "scale")}
+        return {**m, "rot": self.rot.to_json()}
 
 
 @dataclass(frozen=True)
@@ -172,14 +285,25 @@ class MoESpec:
     groups: int = 1              # equal groups of neighbouring experts ...
     keep: int = 1                # ... of which the best `keep` can be chosen from
     shared_ff: int = 0           # hidden size of the expert that every token uses (0: none)
+    score: str = "softmax"       # router scores: "softmax" over the experts, or "sigmoid" of every logit by itself
+    correction: bool = False     # a vector is added to the scores for the choice, not for the weights
+    group_best: int = 1          # a group counts as the sum of its this many largest choice scores
+    renorm: bool = True          # weights are divided by their sum
+    act: str = "silu"            # act(gate) * up; "clamped": see ops.moe.swiglu_rows
+    limit: float = 0.0           # of the clamped activation
 
     def __post_init__(self):
+        if self.score not in ("softmax", "sigmoid") or self.act not in ("silu", "clamped") or self.group_best not in (1, 2) or \
+                (self.score == "softmax" and (self.correction or self.group_best != 1)) or (self.act == "clamped") != (self.limit > 0.0):
+            raise ValueError(f"invalid routed feed-forward: {self}")
         if self.experts % self.groups or not 1 <= self.keep <= self.groups or \
                 not 1 <= self.top <= self.keep * (self.experts // self.groups):
             raise ValueError(f"invalid routed feed-forward: {self}")
 
     def tensor_shapes(self, p: str, d: int) -> dict:
         t = {p + "router": (self.experts, d)}
+        if self.correction:
+            t[p + "correction"] = (self.experts,)
         for e in range(self.experts):
             t.update(_ffn_shapes(f"{p}e{e}.", self.ff, d))
         if self.shared_ff:
@@ -187,16 +311,19 @@ class MoESpec:
         return t
 
     @classmethod
-    def from_json(cls, f: dict) -> "MoESpec":
+    def from_json(cls, f: dict, **fixed) -> "MoESpec":
         r, g = f["router"], f["router"].get("groups") or {}
         return cls(ff=int(f["expert"]["ff"]), experts=int(r["experts"]), top=int(r["top"]), groups=int(g.get("count", 1)),
-                   keep=int(g.get("keep", 1)), shared_ff=int((f.get("shared") or {}).get("ff") or 0))
+                   keep=int(g.get("keep", 1)), shared_ff=int((f.get("shared") or {}).get("ff") or 0),
+                   limit=float(f["expert"].get("limit") or 0.0), **fixed)
 
     def to_json(self) -> dict:
         router = {"experts": self.experts, "top": self.top}
         if self.groups > 1:
             router["groups"] = {"count": self.groups, "keep": self.keep}
         mlp = {"kind": "moe", "expert": {"ff": self.ff}, "router": router}
+        if self.limit:
+            mlp["expert"]["limit"] = self.limit
         if self.shared_ff:
             mlp["shared"] = {"ff": self.shared_ff}
         return mlp
@@ -205,14 +332,16 @@ class MoESpec:
 @dataclass(frozen=True)
 class DenseSpec:
     ff: int
-    act: str = "relu"            # of the gate: act(gate) * up
+    act: str = "relu"            # of the gate: act(gate) * up; not gated: act(up)
+    gated: bool = True
 
     def __post_init__(self):
-        if self.ff < 1 or self.act not in ("relu", "silu"):
+        if self.ff < 1 or self.act not in (("relu", "silu") if self.gated else ("relu2",)):
             raise ValueError(f"invalid dense feed-forward: {self}")
 
     def tensor_shapes(self, p: str, d: int) -> dict:
-        return _ffn_shapes(p, self.ff, d)
+        t = _ffn_shapes(p, self.ff, d)
+        return t if self.gated else {k: v for k, v in t.items() if k != p + "gate"}
 
     def to_json(self) -> dict:
         return {"kind": "dense", "ff": self.ff}
@@ -224,9 +353,21 @@ def _ffn_shapes(p: str, ff: int, d: int) -> dict:
 
 @dataclass(frozen=True)
 class LayerSpec:
-    mixer: AttentionSpec | ParallelSpec | DeltaSpec
+    mixer: AttentionSpec | ParallelSpec | DeltaSpec | LatentSpec
     mlp: MoESpec | DenseSpec | None = None
     weights_of: int | None = None        # the layer whose tensors this one uses (with a cache or state of its own)
+
+
+@dataclass(frozen=True)
+class LoopSpec:
+    """Layers start .. stop - 1 run `times` times in a row with the same weights and a cache of their own in each pass."""
+    start: int
+    stop: int
+    times: int
+
+    def __post_init__(self):
+        if not 0 <= self.start < self.stop or self.times < 1:
+            raise ValueError(f"invalid loop: {self}")
 
 
 @dataclass(frozen=True)
@@ -234,16 +375,23 @@ class Design:
     """What a layered design fixes for all its models."""
     mixers: tuple                        # mixer types a layer can have
     mlps: tuple                          # kinds of feed-forward
-    block: str                           # "output_norm": norm on every sublayer's output; "parallel": one norm in front of both
-    norm: str                            # "layer" or "dyt"
+    block: str                           # "output_norm": norm on every sublayer's output; "parallel": one norm in front of both;
+                                         # "sandwich": a norm in front of every sublayer and one on its output
+    norm: str                            # "layer", "dyt" or "rms" (weights stored as the difference from one)
     attention: dict                      # fixed fields of AttentionSpec ("sliding": the mask is a window)
     act: str = "silu"
+    experts: dict = field(default_factory=dict)      # fixed fields of MoESpec
+    gated: bool = True                   # dense feed-forwards have a gate
+    tied: bool = False                   # the embedding table is the output head
 
 
 DESIGNS = {
     "Dolurax": Design(("attention",), ("moe",), "output_norm", "layer", {}),
     "Vafodra": Design(("parallel", "delta"), ("dense",), "parallel", "dyt",
                       dict(sliding=True, qk_norm=False, distance_bias=False, sink=True, gate="head"), act="relu"),
+    "Bikilix": Design(("attention", "latent_attention"), ("dense", "moe"), "sandwich", "rms",
+                      dict(sliding=True, qk_norm=False, distance_bias=False, gate="none", bias=True), act="relu2",
+                      experts=dict(score="sigmoid", correction=True, group_best=2, renorm=False, act="clamped"), gated=False, tied=True),
 }
 
 
@@ -261,6 +409,7 @@ class LayeredConfig:
     init_std: float = 0.02
     vocab_multiple: int = 128    # rows of the output head are padded to this multiple for aligned GEMM tiles
     arch: str = "Dolurax"
+    loop: LoopSpec | None = None         # layers that run several times
 
     def __post_init__(self):
         if self.arch not in DESIGNS:
@@ -272,6 +421,8 @@ class LayeredConfig:
         mixing = [s.mixer for s in self.layers if getattr(s.mixer, "v_mix", False)]
         if len({a.kv_heads * a.vdim for a in mixing}) > 1:
             raise ValueError("layers that mix values must have the same number of value columns")
+        if self.loop is not None and (self.loop.stop > len(self.layers) or self.design.block != "sandwich"):
+            raise ValueError(f"{self.arch} with {len(self.layers)} layers cannot have {self.loop}")
         for i, s in enumerate(self.layers):
             o = self.layers[self.owner(i)]
             if (o.mixer, o.mlp) != (s.mixer, s.mlp):
@@ -284,6 +435,15 @@ class LayeredConfig:
     @property
     def n_layer(self) -> int:
         return len(self.layers)
+
+    @property
+    def runs(self) -> tuple:
+        """(layer, number of the pass it opens or None) in the order the layers run."""
+        n, lp = self.n_layer, self.loop
+        if lp is None:
+            return tuple((i, None) for i in range(n))
+        body = [(i, t if i == lp.start else None) for t in range(lp.times) for i in range(lp.start, lp.stop)]
+        return (*((i, None) for i in range(lp.start)), *body, *((i, None) for i in range(lp.stop, n)))
 
     @property
     def vocab_padded(self) -> int:
@@ -332,7 +492,9 @@ class LayeredConfig:
             kind, m, f = e.get("type", design.mixers[0]), e["mixer"], e.get("mlp")
             if kind not in design.mixers:
                 raise ValueError(f"layer {i}: unknown mixer {kind!r}")
-            if kind == "parallel":
+            if kind == "latent_attention":
+                mixer = LatentSpec.from_json(m)
+            elif kind == "parallel":
                 mixer = ParallelSpec(AttentionSpec.from_json(m["left"], **design.attention), StateSpaceSpec.from_json(m["right"]))
             elif kind == "delta":
                 mixer = DeltaSpec.from_json(m)
@@ -340,27 +502,31 @@ class LayeredConfig:
                 mixer = AttentionSpec.from_json(m, **design.attention)
             mlp = None
             if f is not None:
-                if f.get("kind", design.mlps[0]) not in design.mlps:
-                    raise ValueError(f"layer {i}: unknown feed-forward {f['kind']!r}")
-                mlp = MoESpec.from_json(f) if design.mlps == ("moe",) else DenseSpec(int(f["ff"]), design.act)
+                fkind = f.get("kind", design.mlps[0])
+                if fkind not in design.mlps:
+                    raise ValueError(f"layer {i}: unknown feed-forward {fkind!r}")
+                mlp = MoESpec.from_json(f, **design.experts) if fkind == "moe" else DenseSpec(int(f["ff"]), design.act, design.gated)
             layers.append(LayerSpec(mixer, mlp, e.get("weights_of")))
         kw = dict(vocab_size=int(d["vocab"]), d_model=int(d["width"]), layers=tuple(layers), norm_eps=float(d["norm"]["eps"]),
                   logit_scale=float(d.get("logit_scale", 1.0)), logit_softcap=float(d.get("logit_softcap") or 0.0),
                   embed_scale=float((d.get("embedding") or {}).get("scale", 1.0)),
                   residual_mult=float(d.get("residual_mult", 1.0)), arch=arch)
+        if d.get("loop"):
+            kw["loop"] = LoopSpec(**{k: int(d["loop"][k]) for k in ("start", "stop", "times")})
         kw.update(overrides)
         return cls(**kw)
 
     def to_json(self) -> dict:
         """The `config.json` form (inverse of `from_json`)."""
-        types = {AttentionSpec: "attention", ParallelSpec: "parallel", DeltaSpec: "delta"}
+        types = {AttentionSpec: "attention", ParallelSpec: "parallel", DeltaSpec: "delta", LatentSpec: "latent_attention"}
 
         def layer(s):
             e = {"type": types[type(s.mixer)], "mixer": s.mixer.to_json(), "mlp": None if s.mlp is None else s.mlp.to_json()}
             if s.weights_of is not None:
                 e["weights_of"] = s.weights_of
             return e
-        return {"architecture": self.arch, "vocab": self.vocab_size, "width": self.d_model, "norm": {"eps": self.norm_eps},
+        loop = {} if self.loop is None else {"loop": asdict(self.loop)}
+        return {"architecture": self.arch, **loop, "vocab": self.vocab_size, "width": self.d_model, "norm": {"eps": self.norm_eps},
                 "embedding": {"scale": self.embed_scale}, "residual_mult": self.residual_mult,
                 "logit_scale": self.logit_scale, "logit_softcap": self.logit_softcap or None,
                 "layers": [layer(s) for s in self.layers]}
@@ -371,9 +537,13 @@ class LayeredConfig:
         d = self.d_model
         t = {"embed": (self.vocab_size, d)}
 
+        if self.loop is not None:
+            t["loop.in"], t["loop.step"] = (d, 2 * d), (self.loop.times, d)
+
         def norm(name):
             t[name] = (d,)
-            t[name + ".b"] = (d,)
+            if self.design.norm != "rms":
+                t[name + ".b"] = (d,)
             if self.design.norm == "dyt":
                 t[name + ".alpha"] = ()
 
@@ -381,20 +551,28 @@ class LayeredConfig:
             if self.owner(i) != i:
                 continue
             p = f"l{i}."
+            sandwich = self.design.block == "sandwich"
             norm(p + "norm1")
+            if sandwich:
+                norm(p + "norm1b")
             t.update(s.mixer.tensor_shapes(p + "mix.", d))
             if s.mlp is not None:
-                if self.design.block == "output_norm":
+                if sandwich or self.design.block == "output_norm":
                     norm(p + "norm2")
+                if sandwich:
+                    norm(p + "norm2b")
                 t.update(s.mlp.tensor_shapes(p + "mlp.", d))
         norm("final.norm")
-        t["head"] = (self.vocab_size, d)
+        if not self.design.tied:
+            t["head"] = (self.vocab_size, d)
         return t
 
     def unused_tensors(self) -> set:
         """Names a checkpoint may hold although no layer reads them: the mixing share of a layer that does not mix, the
         second norm of a layer without a feed-forward."""
         out = set()
+        if self.design.block == "sandwich":
+            return {f"l{i}.{n}" for i, s in enumerate(self.layers) if s.mlp is None for n in ("norm2", "norm2b")}
         if self.design.block != "output_norm":
             return out
         for i, s in enumerate(self.layers):
@@ -417,3 +595,15 @@ def hybrid_layers(order: str, left: dict, right: dict, delta: dict, ff: dict, we
     act = DESIGNS["Vafodra"].act
     mixers = {"p": ParallelSpec(AttentionSpec(**left, **fixed), StateSpaceSpec(**right)), "d": DeltaSpec(**delta)}
     return tuple(LayerSpec(mixers[c], DenseSpec(ff[c], act) if ff[c] else None, (weights_of or {}).get(i)) for i, c in enumerate(order))
+
+
+def sandwich_layers(order: str, attention: dict, latent: dict, ff: int, moe: dict, dense: tuple = ()) -> tuple:
+    """Layers of a Bikilix model: 'w' a windowed attention layer (`attention`), 'l' a latent one (`latent`); the layers whose index is in
+    `dense` have a dense feed-forward of hidden size `ff`, the others routed experts (`moe`)."""
+    design = DESIGNS["Bikilix"]
+
+    def rot(m):
+        return {**m, "rot": RotarySpec(**m["rot"])}
+    mixers = {"w": AttentionSpec(**rot(attention), **{k: v for k, v in design.attention.items() if k != "sliding"}), "l": LatentSpec(**rot(latent))}
+    return tuple(LayerSpec(mixers[c], DenseSpec(ff, design.act, design.gated) if i in dense else MoESpec(**moe, **design.experts))
+                 for i, c in enumerate(order))

@@ -60,11 +60,14 @@ _HYBRID_KERNELS = ("gemm_tcgen05", "gemm_f32", "embedding", "elementwise", "resi
                    "paged_attention", "short_conv", "state_space", "state_space_chunk", "delta_rule",
                    "delta_rule_chunk", "gated_norm")
 
+_SANDWICH_KERNELS = (*_LAYERED_KERNELS, "rope", "latent_attention")
+
 ARCHITECTURES = {a.name: a for a in (
     Architecture("gpt2", _gpt_config, "GPTBody", False, _gpt_weights, _GPT_KERNELS),
     Architecture("llama", _gpt_config, "GPTBody", False, _gpt_weights, _GPT_KERNELS),
     Architecture("Dolurax", LayeredConfig.from_json, "LayeredBody", True, _layered_weights, _LAYERED_KERNELS),
     Architecture("Vafodra", LayeredConfig.from_json, "ParallelBody", True, _layered_weights, _HYBRID_KERNELS),
+    Architecture("Bikilix", LayeredConfig.from_json, "SandwichBody", True, _layered_weights, _SANDWICH_KERNELS),
 )}
 
 

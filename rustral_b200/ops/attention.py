@@ -207,6 +207,35 @@ def prompt_attention(q, k, v, scale: float, out, rule: ScoreRule | None = None, 
     return out
 
 
+def split_supported(dn: int, dr: int, dv: int, *views) -> bool:
+    """Whether `prompt_attention_split` takes these head sizes and operands (2-D row-strided views; None: absent)."""
+    views = [t for t in views if t is not None]
+    if not views[0].is_cuda:
+        return True
+    if any(t.dtype != torch.bfloat16 or t.stride(0) % 8 or t.data_ptr() % 16 for t in views):
+        return False
+    return (dn | dr | dv) % 8 == 0 and max(dn, dv) <= 128 and dr <= 64
+
+
+def prompt_attention_split(q, k, v, k_rot, scale: float, out, gate=None):
+    """Causal attention of a prompt portion whose keys have a second part that all heads share: q [1, L, H, dn + dr], k [1, S, H, dn],
+    k_rot [S, dr], v [1, S, H, dv], out [1, L, H, dv]; score = (q[:dn] . k + q[dn:] . k_rot) * scale.  `gate` [L, H * dv]: out <- out *
+    sigmoid(gate).  On a GPU dr is at most 64 (bf16, sizes in multiples of 8, at most 128)."""
+    dn, dv, dr = k.shape[3], v.shape[3], k_rot.shape[1]
+    if not q.is_cuda:
+        kk = torch.cat([k.float(), k_rot.float()[None, :, None, :].expand(1, k.shape[1], k.shape[2], dr)], -1)
+        o = attention_reference(q.float(), kk, v, True, scale)
+        out.copy_(o if gate is None else o * torch.sigmoid(gate.float().reshape(o.shape)))
+        return out
+    a, r = N.RbAttnArgs(), N.RbAttnRule()
+    _fill(a, q[..., :dn], k, v, out, True, scale)
+    r.v_dim, r.rot_dim, r.k_rot, r.ld_k_rot = dv, dr, k_rot.data_ptr(), k_rot.stride(0)
+    if gate is not None:
+        r.gate, r.ld_gate = gate.data_ptr(), gate.stride(0)
+    N.check(N.kernels().rb_attention_fwd_rule(a, r, N.stream_ptr()), "rb_attention_fwd_rule")
+    return out
+
+
 def attention_backward(do, q, k, v, o, lse, causal: bool, scale: float, dq=None, dk=None, dv=None, impl: str | None = None,
                        kv_lens=None):
     B, Sq, H, D = q.shape

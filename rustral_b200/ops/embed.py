@@ -42,24 +42,27 @@ def embedding_forward(ids: torch.Tensor, wte: torch.Tensor, wpe=None, seq_len: i
     return y
 
 
-N.optional_sig("rb_embedding_residual", [N.c_void_p, N.c_void_p, N.c_int, N.c_void_p, N.c_void_p, N.c_ll, N.c_int, N.c_ll,
+N.optional_sig("rb_embedding_residual", [N.c_void_p, N.c_void_p, N.c_int, N.c_void_p, N.c_void_p, N.c_ll, N.c_ll, N.c_int, N.c_ll,
                                         N.c_float, N.c_void_p])
 
 
-def embedding_residual(ids: torch.Tensor, table: torch.Tensor, scale: float = 1.0, want_h: bool = True):
+def embedding_residual(ids: torch.Tensor, table: torch.Tensor, scale: float = 1.0, want_h: bool = True, h=None):
     """Start of a 32-bit residual stream: (x fp32 [tokens, dim] = scale * rows of the table, h = the same rows in the table's
-    dtype; x itself for an fp32 table; None without `want_h`)."""
+    dtype; x itself for an fp32 table; None without `want_h`).  `h`: a row-strided tensor of the table's dtype that receives the
+    copy."""
     f32 = table.dtype == torch.float32
     if not table.is_cuda:
         x = table[ids].float() * scale
+        if h is not None:
+            return x, h.copy_(x)
         return x, (None if not want_h else x if f32 else x.to(table.dtype))
     tokens, dim = ids.numel(), table.shape[1]
     x = torch.empty((tokens, dim), dtype=torch.float32, device=table.device)
-    h = None
-    if want_h:
+    own = h is not None
+    if want_h and not own:
         h = x if f32 else torch.empty((tokens, dim), dtype=table.dtype, device=table.device)
     N.check(N.kernels().rb_embedding_residual(ids.data_ptr(), table.data_ptr(), int(f32), x.data_ptr(),
-                                              None if f32 else N.ptr(h), tokens, dim, table.shape[0], scale, N.stream_ptr()),
+                                              N.ptr(h) if own or not f32 else None, h.stride(0) if own else dim, tokens, dim, table.shape[0], scale, N.stream_ptr()),
             "rb_embedding_residual")
     return x, h
 

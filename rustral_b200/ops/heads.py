@@ -1,17 +1,20 @@
-"""Per-head work between a packed attention projection and the attention kernels: query / key norm, value mixing, cache append."""
+"""Per-head work between a packed attention projection and the attention kernels: query / key norm, rotary positions, value mixing,
+cache append."""
 from __future__ import annotations
 
 import torch
 
 from .. import _native as N
+from .rotary import rotate_pairs
 
 N.optional_sig("rb_head_prep", [N.C.POINTER(N.RbHeadPrepArgs), N.c_void_p])
 
 
 def head_prep_(p, heads: int, kv_heads: int, dk: int, dv: int, *, q_gamma=None, k_gamma=None, eps: float = 1e-5, v_first=None,
-               mix=None, k_cache=None, v_cache=None, slots=None):
+               mix=None, k_cache=None, v_cache=None, slots=None, rot=None):
     """In place on `p` = [q | k | v | ...] ([tokens, >= heads * dk + kv_heads * (dk + dv)]): every query and key head gets an
-    RMS norm (weights `q_gamma` / `k_gamma` [dk], None: no norm), the values become (1 - mix) v + mix v_first (`v_first`:
+    RMS norm (weights `q_gamma` / `k_gamma` [dk], None: no norm) and rotary positions (`rot`: fp32 [tokens, pairs, 2] of
+    `rotary_table`, on the first 2 * pairs numbers), the values become (1 - mix) v + mix v_first (`v_first`:
     [tokens, kv_heads * dv], `mix` fp32 [1]; None: unchanged), and keys and values are stored in their cache slots."""
     T = p.shape[0]
     ok, ov = heads * dk, (heads + kv_heads) * dk
@@ -22,6 +25,9 @@ def head_prep_(p, heads: int, kv_heads: int, dk: int, dv: int, *, q_gamma=None, 
                 x = p[:, lo:lo + n * dk].float().view(T, n, dk)
                 x = x * torch.rsqrt((x * x).mean(-1, keepdim=True) + eps) * g.float()
                 p[:, lo:lo + n * dk] = x.reshape(T, n * dk).to(p.dtype)
+            if rot is not None:
+                x = p[:, lo:lo + n * dk].reshape(T, n, dk)
+                p[:, lo:lo + n * dk] = rotate_pairs(x, rot).reshape(T, n * dk)
         if v_first is not None:
             lam = mix.float()
             p[:, ov:end] = ((1 - lam) * p[:, ov:end].float() + lam * v_first.float()).to(p.dtype)
@@ -39,6 +45,8 @@ def head_prep_(p, heads: int, kv_heads: int, dk: int, dv: int, *, q_gamma=None, 
     if k_cache is not None:
         a.k_cache, a.v_cache, a.slots = k_cache.data_ptr(), v_cache.data_ptr(), slots.data_ptr()
         a.num_slots = k_cache.shape[0] * k_cache.shape[1]
+    if rot is not None:
+        a.rot, a.rot_dims = rot.data_ptr(), 2 * rot.shape[1]
     a.off_q, a.off_k, a.off_v, a.tokens = 0, ok, ov, T
     a.heads, a.kv_heads, a.dk, a.dv, a.eps = heads, kv_heads, dk, dv, eps
     N.check(N.kernels().rb_head_prep(a, N.stream_ptr()), "rb_head_prep")

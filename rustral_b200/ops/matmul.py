@@ -16,7 +16,7 @@ import torch
 
 from .. import _native as N
 
-_ACT_FWD = {"gelu", "relu", "silu"}
+_ACT_FWD = {"gelu", "relu", "silu", "relu2"}
 _ACT_BWD = {"dgelu", "drelu", "dsilu", "mul"}
 
 
@@ -38,6 +38,8 @@ def act_reference(name: str, x: torch.Tensor) -> torch.Tensor:
         return torch.relu(x)
     if name == "silu":
         return x * torch.sigmoid(x)
+    if name == "relu2":
+        return torch.relu(x) ** 2
     return x
 
 
@@ -183,11 +185,12 @@ def set_plan_hook(fn) -> None:
 
 
 N.optional_sig("rb_gemm_f32", [N.c_void_p, N.c_ll, N.c_void_p, N.c_ll, N.c_void_p, N.c_ll, N.c_int, N.c_int, N.c_int, N.c_float,
-                               N.c_void_p, N.c_void_p, N.c_ll, N.c_void_p])
+                               N.c_void_p, N.c_int, N.c_void_p, N.c_void_p, N.c_ll, N.c_void_p])
 
 
-def _gemm_f32(a, b, out, alpha, tile_expert=None, num_tiles=None, expert_stride=0) -> torch.Tensor:
-    """True fp32 product (the 32-bit serving mode); `tile_expert` / `num_tiles`: the grouped form over stacked experts."""
+def _gemm_f32(a, b, out, alpha, tile_expert=None, num_tiles=None, expert_stride=0, bias=None, act="none") -> torch.Tensor:
+    """True fp32 product (the 32-bit serving mode) with a bias and relu2; `tile_expert` / `num_tiles`: the grouped form over
+    stacked experts."""
     M, K = a.shape
     Nn = b.shape[0]
     if a.stride(1) != 1 or b.stride(1) != 1:
@@ -196,7 +199,7 @@ def _gemm_f32(a, b, out, alpha, tile_expert=None, num_tiles=None, expert_stride=
     if M == 0 or Nn == 0:
         return out
     N.check(N.kernels().rb_gemm_f32(a.data_ptr(), a.stride(0), b.data_ptr(), b.stride(0), out.data_ptr(), out.stride(0), M, Nn, K,
-                                    alpha, N.ptr(tile_expert), N.ptr(num_tiles), expert_stride, N.stream_ptr()), "rb_gemm_f32")
+                                    alpha, N.ptr(bias), int(act == "relu2"), N.ptr(tile_expert), N.ptr(num_tiles), expert_stride, N.stream_ptr()), "rb_gemm_f32")
     return out
 
 
@@ -232,10 +235,12 @@ def gemm(a: torch.Tensor, b: torch.Tensor, *, a_mn: bool = False, b_mn: bool = F
         return _gemm_cpu(a, b, a_mn, b_mn, bias, act, residual, aux_in, aux_out, out, out_dtype, accumulate, alpha)
 
     if a.dtype == torch.float32 and b.dtype == torch.float32:
-        if (a_mn or b_mn or act != "none" or accumulate or peer is not None or out_dtype != torch.float32
-                or any(t is not None for t in (bias, residual, aux_in, aux_out, row_scale, col_scale))):
-            raise TypeError("gemm: fp32 CUDA operands take the plain product only (no epilogue, no transposed operand)")
-        return _gemm_f32(a, b, out, alpha)
+        if (a_mn or b_mn or act not in ("none", "relu2") or accumulate or peer is not None or out_dtype != torch.float32
+                or any(t is not None for t in (residual, aux_in, aux_out, row_scale, col_scale))):
+            raise TypeError("gemm: fp32 CUDA operands take the plain product, a bias and relu2 only (no transposed operand)")
+        if bias is not None and (bias.dtype != torch.float32 or bias.numel() != Nn or not bias.is_contiguous()):
+            raise TypeError("gemm: the bias of fp32 operands is a contiguous fp32 vector")
+        return _gemm_f32(a, b, out, alpha, bias=bias, act=act)
     if a.dtype != torch.bfloat16 or b.dtype != torch.bfloat16:
         raise TypeError("gemm: CUDA operands must be both bf16 (accumulation is fp32) or both fp32")
     if M == 0 or Nn == 0:
@@ -386,6 +391,8 @@ class _LinearFn(torch.autograd.Function):
 
     @staticmethod
     def forward(ctx, x, w, bias, act, residual):
+        if act == "relu2":
+            raise ValueError("linear: relu2 has no backward pass (inference only)")
         x2 = x.reshape(-1, x.shape[-1])
         need_pre = act in _ACT_FWD and (x.requires_grad or w.requires_grad)
         pre = torch.empty((x2.shape[0], w.shape[0]), dtype=x.dtype, device=x.device) if need_pre else None

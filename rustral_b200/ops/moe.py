@@ -19,7 +19,8 @@ P, I, F, LL = N.c_void_p, N.c_int, N.c_float, N.c_ll
 N.optional_sig("rb_moe_route", [P, I, I, I, I, P, P, P, P])
 N.optional_sig("rb_moe_route_bwd", [P, P, P, P, P, I, I, I, I, F, P, P])
 N.optional_sig("rb_moe_route_groups", [P, I, I, I, I, I, I, F, P, P, P])
-N.optional_sig("rb_swiglu_slots", [P, LL, P, LL, I, I, I, P, I, P])
+N.optional_sig("rb_moe_route_sigmoid", [P, P, I, I, I, I, I, I, I, F, P, P, P])
+N.optional_sig("rb_swiglu_slots", [P, LL, P, LL, I, I, I, P, I, F, P])
 N.optional_sig("rb_moe_scatter", [P, P, P, I, I, I, P])
 N._LAUNCHES["rb_moe_plan"] = 2
 N.optional_sig("rb_moe_plan", [P, I, I, I, P, P, P, P, P, P, I, P])
@@ -76,21 +77,55 @@ def route_groups(logits: torch.Tensor, k: int, groups: int = 1, keep: int = 1, r
     return idx, w
 
 
-def swiglu_rows(gu: torch.Tensor, pl: MoEPlan | None = None, act: str = "silu", out=None) -> torch.Tensor:
-    """act(gate) * up for gu = [gate | up] rows (row-strided views allowed, `out` too), bf16 or fp32; act "silu" or "relu".  With
-    a plan only the rows that hold a token are computed; padding rows of the expert buffer are left unwritten."""
+def route_sigmoid(logits: torch.Tensor, k: int, groups: int = 1, keep: int = 1, correction=None, group_best: int = 1,
+                  renorm: bool = False, eps: float = 1e-20):
+    """Group-limited top-k routing by sigmoid scores: choice scores are sigmoid(logit) + correction (fp32 [E], of either sign); a
+    group counts as the sum of its `group_best` (1 or 2) largest choice scores and only experts of the best `keep` groups can be
+    chosen; the weights are the chosen sigmoids without the correction, divided by (their sum + eps) with `renorm`.  logits fp32
+    [T, E] -> (idx int32 [T, k], w fp32 [T, k])."""
+    T, E = logits.shape
+    if not logits.is_cuda:
+        s = torch.sigmoid(logits.float())
+        c = s if correction is None else s + correction.float()
+        if groups > 1 and keep < groups:
+            per = E // groups
+            best = c.view(T, groups, per).topk(min(group_best, per), -1).values.sum(-1)
+            kept = torch.sort(-best, dim=-1, stable=True).indices[:, :keep]
+            ok = torch.zeros((T, groups), dtype=torch.bool).scatter_(1, kept, True)
+            c = c.masked_fill(~ok.repeat_interleave(per, 1), float("-inf"))
+        order = torch.sort(-c, dim=-1, stable=True).indices[:, :k]
+        w = s.gather(1, order)
+        return order.to(torch.int32), w / (w.sum(-1, keepdim=True) + eps) if renorm else w
+    idx = torch.empty((T, k), dtype=torch.int32, device=logits.device)
+    w = torch.empty((T, k), dtype=torch.float32, device=logits.device)
+    N.check(N.kernels().rb_moe_route_sigmoid(logits.data_ptr(), N.ptr(correction), T, E, k, groups, keep, group_best, int(renorm),
+                                             float(eps), idx.data_ptr(), w.data_ptr(), N.stream_ptr()), "rb_moe_route_sigmoid")
+    return idx, w
+
+
+_GLU = {"silu": 0, "relu": 1, "clamped": 2}
+
+
+def swiglu_rows(gu: torch.Tensor, pl: MoEPlan | None = None, act: str = "silu", out=None, limit: float = 0.0) -> torch.Tensor:
+    """act(gate) * up for gu = [gate | up] rows (row-strided views allowed, `out` too), bf16 or fp32; act "silu", "relu", or
+    "clamped": g sigmoid(1.702 g) (u + 1) with g = min(gate, limit) and u = clamp(up, -limit, limit).  With a plan only the rows that hold a token are computed; padding rows of the expert buffer are left unwritten."""
     rows, F2 = gu.shape
-    if act not in ("silu", "relu"):
+    if act not in _GLU:
         raise ValueError(f"swiglu_rows: unknown activation {act!r}")
     if not gu.is_cuda:
         g, u = gu.float()[:, :F2 // 2], gu.float()[:, F2 // 2:]
-        h = ((torch.relu(g) if act == "relu" else g * torch.sigmoid(g)) * u).to(gu.dtype)
+        if act == "clamped":
+            g, u = g.clamp(max=limit), u.clamp(-limit, limit) + 1.0
+            h = g * torch.sigmoid(1.702 * g) * u
+        else:
+            h = (torch.relu(g) if act == "relu" else g * torch.sigmoid(g)) * u
+        h = h.to(gu.dtype)
         return h if out is None else out.copy_(h)
     h = out if out is not None else torch.empty((rows, F2 // 2), dtype=gu.dtype, device=gu.device)
     n = rows if pl is None else pl.slot_pos.numel()
     N.check(N.kernels().rb_swiglu_slots(gu.data_ptr(), gu.stride(0), h.data_ptr(), h.stride(0), n, F2 // 2,
                                         int(gu.dtype == torch.float32), None if pl is None else pl.slot_pos.data_ptr(),
-                                        int(act == "relu"), N.stream_ptr()), "rb_swiglu_slots")
+                                        _GLU[act], float(limit), N.stream_ptr()), "rb_swiglu_slots")
     return h
 
 

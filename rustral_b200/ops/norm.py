@@ -148,12 +148,13 @@ def rms_norm(x, gamma, eps: float = 1e-5):
 N.optional_sig("rb_residual_norm", [N.C.POINTER(N.RbResidualNormArgs), N.c_void_p])
 
 
-def residual_norm(y, gamma, beta, eps: float, rms: bool = False, *, x=None, h=None, routed=None, add=None):
+def residual_norm(y, gamma, beta, eps: float, rms: bool = False, *, x=None, h=None, routed=None, add=None, next_gamma=None):
     """Norm of a sublayer's output added to a 32-bit residual stream.
 
     source row t = y[t], or with `routed` = (slot_pos int32 [T * k], weights fp32 [T, k]) the weighted sum of token t's
     expert rows of `y`; `add` (same dtype as y) is added to it.  With `x` (fp32 [T, n]): x += norm(source) in place and
-    `h` receives a copy in its own dtype.  Without `x`: `h` receives norm(source).  Returns h (x when h is None)."""
+    `h` receives a copy in its own dtype, or with `next_gamma` (dtype of gamma) rms(x) * next_gamma.  Without `x`: `h` receives
+    norm(source).  Returns h (x when h is None)."""
     rows = x.shape[0] if x is not None else h.shape[0]
     n = y.shape[1]
     if not y.is_cuda:
@@ -166,7 +167,7 @@ def residual_norm(y, gamma, beta, eps: float, rms: bool = False, *, x=None, h=No
         o = norm_forward(src, gamma, beta, eps, rms)[0].float()
         if x is not None:
             x += o
-            o = x
+            o = x if next_gamma is None else norm_forward(x, next_gamma, None, eps, True)[0]
         if h is not None:
             h.copy_(o)
         return h if h is not None else x
@@ -179,6 +180,7 @@ def residual_norm(y, gamma, beta, eps: float, rms: bool = False, *, x=None, h=No
     if routed is not None:
         slot_pos, w = routed
         a.slot_pos, a.slot_w, a.k = slot_pos.data_ptr(), w.data_ptr(), w.shape[1]
+    a.next_gamma = N.ptr(next_gamma)
     a.gamma, a.beta, a.param_f32 = gamma.data_ptr(), N.ptr(beta), int(gamma.dtype == torch.float32)
     if x is not None:
         if x.dtype != torch.float32:

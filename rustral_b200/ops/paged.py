@@ -110,7 +110,7 @@ def paged_attention_rows(q, k_cache, v_cache, block_tables, row_seq, row_pos, sc
                          gate=None, out=None, head_gate=None):
     """Attention over the pages for any rows of a batch.  q: [rows, heads * dk] (row-strided views allowed); row r is the
     token at position row_pos[r] (int64) of the sequence with pages block_tables[row_seq[r]] (int32); its own key is
-    already in the cache.  Takes bf16 and fp32 and any head sizes.  `gate` [rows, heads * dv] or `head_gate` fp32 [rows, heads]:
+    already in the cache.  Takes bf16 and fp32 and any head sizes; `v_cache` may be the first columns of `k_cache`.  `gate` [rows, heads * dv] or `head_gate` fp32 [rows, heads]:
     output times sigmoid(gate)."""
     nb, bs, hk, dk = k_cache.shape
     dv = v_cache.shape[3]
@@ -118,7 +118,7 @@ def paged_attention_rows(q, k_cache, v_cache, block_tables, row_seq, row_pos, sc
     rule = rule or ScoreRule()
     out = out if out is not None else torch.empty((rows, heads * dv), dtype=q.dtype, device=q.device)
     if not q.is_cuda:
-        kc, vc = k_cache.view(nb * bs, hk, dk), v_cache.view(nb * bs, hk, dv)
+        kc, vc = k_cache.view(nb * bs, hk, dk), v_cache.reshape(nb * bs, hk, dv)
         for r in range(rows):
             n, table = int(row_pos[r]) + 1, block_tables[int(row_seq[r])].long()
             kept, lo = rule.key_ranges(n - 1)
@@ -133,6 +133,7 @@ def paged_attention_rows(q, k_cache, v_cache, block_tables, row_seq, row_pos, sc
     a = N.RbPagedRowsArgs()
     a.q, a.ld_q, a.out, a.ld_o = q.data_ptr(), q.stride(0), out.data_ptr(), out.stride(0)
     a.k_cache, a.v_cache, a.num_blocks, a.block_size = k_cache.data_ptr(), v_cache.data_ptr(), nb, bs
+    a.ld_kc, a.ld_vc = k_cache.stride(1), v_cache.stride(1)
     a.block_tables, a.max_blocks = block_tables.data_ptr(), block_tables.shape[1]
     a.row_seq, a.row_pos = row_seq.data_ptr(), row_pos.data_ptr()
     if gate is not None:

@@ -43,6 +43,48 @@ def rope_(x2: torch.Tensor, heads: int, head_dim: int, seq_len: int = 0, positio
     return x2
 
 
+N.optional_sig("rb_rotary_table", [N.c_void_p, N.c_void_p, N.c_float, N.c_void_p, N.c_ll, N.c_int, N.c_void_p])
+N.optional_sig("rb_rotate_pairs", [N.c_void_p, N.c_ll, N.c_void_p, N.c_ll, N.c_int, N.c_ll, N.c_int, N.c_int, N.c_void_p])
+
+
+def rotary_table(positions: torch.Tensor, freqs: torch.Tensor, magnitude: float = 1.0) -> torch.Tensor:
+    """fp32 [rows, pairs, 2]: cosine and sine of position * freqs[pair] (fp64, on the positions' device), times `magnitude`."""
+    rows, pairs = positions.numel(), freqs.numel()
+    if not positions.is_cuda:
+        a = positions.double()[:, None] * freqs[None, :]
+        return (torch.stack([torch.cos(a), torch.sin(a)], -1) * magnitude).float()
+    out = torch.empty((rows, pairs, 2), dtype=torch.float32, device=positions.device)
+    if rows and pairs:
+        N.check(N.kernels().rb_rotary_table(positions.data_ptr(), freqs.data_ptr(), magnitude, out.data_ptr(), rows, pairs,
+                                            N.stream_ptr()), "rb_rotary_table")
+    return out
+
+
+def rotate_pairs(x3: torch.Tensor, table: torch.Tensor) -> torch.Tensor:
+    """Reference form: a copy of x3 [rows, heads, size] with neighbouring pairs (2i, 2i + 1) of its first 2 * pairs numbers rotated."""
+    y, n = x3.clone(), 2 * table.shape[1]
+    c, s = table[:, None, :, 0], table[:, None, :, 1]
+    u, v = x3[..., 0:n:2].float(), x3[..., 1:n:2].float()
+    y[..., 0:n:2], y[..., 1:n:2] = (u * c - v * s).to(x3.dtype), (v * c + u * s).to(x3.dtype)
+    return y
+
+
+def rotate_pairs_(x2: torch.Tensor, heads: int, pitch: int, first: int, table: torch.Tensor) -> torch.Tensor:
+    """In place on every head of x2 [rows, >= heads * pitch] (bf16 or fp32): the neighbouring pairs that start at column `first` of
+    the head turn by `table` (see rotary_table)."""
+    rows, n = x2.shape[0], 2 * table.shape[1]
+    if rows == 0 or n == 0:
+        return x2
+    if not x2.is_cuda:
+        v = x2[:, :heads * pitch].reshape(rows, heads, pitch)
+        v[..., first:] = rotate_pairs(v[..., first:], table)
+        x2[:, :heads * pitch] = v.reshape(rows, heads * pitch)
+        return x2
+    N.check(N.kernels().rb_rotate_pairs(x2[:, first:].data_ptr(), x2.stride(0), table.data_ptr(), rows, heads, pitch, table.shape[1],
+                                        int(x2.dtype == torch.float32), N.stream_ptr()), "rb_rotate_pairs")
+    return x2
+
+
 class _RopeFn(torch.autograd.Function):
     @staticmethod
     def forward(ctx, x, seq_len, positions, pos_offset, theta):

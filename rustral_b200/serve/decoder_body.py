@@ -4,7 +4,8 @@ A body knows a model's mathematics only: embedding, one layer, output head, and 
 rows a step holds, where their keys and values go, which kernels attend for which rows, and graph capture belong to the
 runner (serve.model_runner), so every body gets prefill, chunked prefill, mixed batches and graphed decoding from it.
 
-`embed` returns the stream that `layer` takes and returns; `head` turns selected rows of it into logits.
+`embed` returns the stream that `layer` takes and returns; `head` turns selected rows of it into logits.  `depth` is the number of
+layers that run (and have a cache each): a layer that is passed through several times counts as often.
 """
 from __future__ import annotations
 
@@ -13,7 +14,8 @@ import math
 import torch
 
 from .. import ops
-from ..models.layered import ParallelSpec, up8
+from ..models.layered import DenseSpec, LatentSpec, ParallelSpec, up8
+from ..ops import latent as latent_ops
 from ..ops import moe as moe_ops
 from ..ops import norm as norm_ops
 from ..ops import paged as paged_ops
@@ -23,7 +25,7 @@ from ..ops.attention import ScoreRule, distance_slopes
 from ..ops.heads import head_prep_
 from ..ops.matmul import gemm
 from .kv_cache import CacheLayer
-from .weights import packed_columns
+from .weights import latent_columns, packed_columns
 
 
 class GPTBody:
@@ -33,6 +35,7 @@ class GPTBody:
         self.r, self.cfg = runner, runner.cfg
         self.rms = self.cfg.arch == "llama"
         self.scale = 1.0 / math.sqrt(self.cfg.head_dim)
+        self.depth = self.cfg.n_layer
 
     def cache_layers(self) -> list:
         return None                                   # uniform: the cache's num_layers / num_kv_heads / head_dim form
@@ -91,11 +94,12 @@ class GPTBody:
 
 class Stream:
     """Residual stream of a layered decoder: `x` fp32, `h` its copy in the activation dtype (the operand of the next
-    products; `x` itself in 32-bit), `v_first` the value columns of the first layer that mixes values."""
-    __slots__ = ("x", "h", "v_first")
+    products; `x` itself in 32-bit), `v_first` the value columns of the first layer that mixes values, `pair` the copies of the
+    stream and of the embedding side by side that a pass through repeated layers starts from."""
+    __slots__ = ("x", "h", "v_first", "pair")
 
     def __init__(self, x, h):
-        self.x, self.h, self.v_first = x, h, None
+        self.x, self.h, self.v_first, self.pair = x, h, None, None
 
 
 class LayeredBody:
@@ -109,6 +113,7 @@ class LayeredBody:
         self.r, self.cfg = runner, runner.cfg
         if runner.tp is not None:
             raise ValueError("tensor-parallel serving covers the llama family")
+        self.depth = self.cfg.n_layer
         slopes = {}
         self.rules = []
         for s in self.cfg.layers:
@@ -179,6 +184,7 @@ class ParallelBody:
         self.r, self.cfg = runner, runner.cfg
         if runner.tp is not None:
             raise ValueError("tensor-parallel serving covers the llama family")
+        self.depth = self.cfg.n_layer
         self.columns = [packed_columns(s) for s in self.cfg.layers]
         self.prefix = [f"l{self.cfg.owner(i)}." for i in range(self.cfg.n_layer)]
         slopes = {}
@@ -273,4 +279,129 @@ class ParallelBody:
         logits = gemm(h, P.w("head"), out_dtype=torch.float32)
         if self.cfg.logit_scale != 1.0 or self.cfg.logit_softcap:
             ops.scale_softcap_(logits, self.cfg.logit_scale, self.cfg.logit_softcap)
+        return logits
+
+
+class SandwichBody:
+    """Layered decoders with a norm in front of every sublayer and one on its output (Bikilix); some layers can run several times.
+
+    Per layer: one packed projection of everything that reads the first norm; attention (head rotation + cache append in one kernel) or
+    latent attention; output projection; then its norm, residual add and the norm in front of the feed-forward in one kernel; dense or
+    routed feed-forward; its norm (with the experts' combine), residual add and the next layer's norm in one kernel.  In front of a
+    pass the stream becomes a product of itself and the embedding: both are kept side by side as the product's operand."""
+
+    def __init__(self, runner):
+        self.r, self.cfg = runner, runner.cfg
+        if runner.tp is not None:
+            raise ValueError("tensor-parallel serving covers the llama family")
+        self.runs = self.cfg.runs
+        self.depth = len(self.runs)
+        freqs = {s.mixer.rot: torch.tensor(s.mixer.rot.frequencies(), dtype=torch.float64) for s in self.cfg.layers if s.mixer.rot is not None}
+        self.freqs = {rot: f.to(runner.device) for rot, f in freqs.items()}
+        self.columns = [latent_columns(s.mixer) if isinstance(s.mixer, LatentSpec) else None for s in self.cfg.layers]
+        self.rules = [self._rule(s.mixer) for s in self.cfg.layers]
+
+    @staticmethod
+    def _rule(m):
+        if isinstance(m, LatentSpec):
+            return None
+        rule = ScoreRule(softcap=m.softcap, chunk=m.chunk, window=m.window, keep_first=m.keep_first, sink=m.sink)
+        return None if rule.plain and m.dim == m.vdim and m.dim in (64, 128) else rule      # plain attention of those sizes needs no rule
+
+    def cache_layers(self) -> list:
+        out = []
+        for i, _ in self.runs:
+            m = self.cfg.layers[i].mixer
+            out.append(CacheLayer(1, m.cached, m.kv_rank, joint=True) if isinstance(m, LatentSpec) else CacheLayer(m.kv_heads, m.dim, m.vdim))
+        return out
+
+    def _rotation(self, rot, sb):
+        return None if rot is None or rot.dims == 0 else sb.rotation(rot, self.freqs[rot])
+
+    def _start(self, st, run, y=None, name=None, **kw):
+        """What stands between sublayers: x += norm(y) (none without `y`), then the operand that run number `run` starts from: its
+        norm of the stream, or the stream's copy beside the embedding in front of a pass (the stream itself behind the last layer)."""
+        P, eps = self.r.params, self.cfg.norm_eps
+        i, opens = self.runs[run] if run < self.depth else (None, None)
+        gamma = P.w(f"l{i}.norm1") if i is not None else None
+        if opens is not None:
+            left = st.pair[:, :self.cfg.d_model]
+            if y is not None:
+                norm_ops.residual_norm(y, P.w(name), None, eps, True, x=st.x, h=left, **kw)
+            st.x = gemm(st.pair, P.w("loop.in"), bias=P.w("loop.step")[opens], out_dtype=torch.float32)
+            y = None
+        if i is None:
+            norm_ops.residual_norm(y, P.w(name), None, eps, True, x=st.x, **kw)
+        elif y is None:
+            st.h = norm_ops.residual_norm(st.x, gamma, None, eps, True, h=torch.empty_like(st.x, dtype=self.r.dtype))
+        else:
+            norm_ops.residual_norm(y, P.w(name), None, eps, True, x=st.x, h=st.h, next_gamma=gamma, **kw)
+        return st
+
+    def embed(self, sb):
+        P, d, scale = self.r.params, self.cfg.d_model, self.cfg.embed_scale
+        if self.cfg.loop is None:
+            st = Stream(ops.embedding_residual(sb.ids, P.w("embed"), scale, want_h=False)[0], None)
+        else:
+            pair = torch.empty((sb.rows, 2 * d), dtype=self.r.dtype, device=self.r.device)
+            x, _ = ops.embedding_residual(sb.ids, P.w("embed"), scale, h=pair[:, d:])
+            st = Stream(x, None)
+            st.pair = pair
+            if self.runs[0][1] is not None:                       # the first pass starts from the embedding twice
+                pair[:, :d] = pair[:, d:]
+        return self._start(st, 0)
+
+    def layer(self, run, st, sb):
+        r, P = self.r, self.r.params
+        i, _ = self.runs[run]
+        s, p = self.cfg.layers[i], f"l{i}."
+        o = (self._latent if isinstance(s.mixer, LatentSpec) else self._attention)(run, i, s.mixer, p, st.h, sb)
+        y = gemm(o, P.w(p + "attn.out"), out_dtype=torch.float32)
+        if s.mlp is None:
+            return self._start(st, run + 1, y, p + "norm1b")
+        norm_ops.residual_norm(y, P.w(p + "norm1b"), None, self.cfg.norm_eps, True, x=st.x, h=st.h, next_gamma=P.w(p + "norm2"))
+        if isinstance(s.mlp, DenseSpec):
+            y = gemm(gemm(st.h, P.w(p + "up"), act=s.mlp.act), P.w(p + "down"), out_dtype=torch.float32)
+            return self._start(st, run + 1, y, p + "norm2b")
+        y, routed = self._experts(st.h, s.mlp, p)
+        return self._start(st, run + 1, y, p + "norm2b", routed=routed)
+
+    def _attention(self, run, i, a, p, h, sb):
+        r, P = self.r, self.r.params
+        H, G, dk, dv = a.heads, a.kv_heads, a.dim, a.vdim
+        z = gemm(h, P.w(p + "attn.in"), bias=P.w(p + "attn.in.b") if a.bias else None)
+        ov = (H + G) * dk
+        head_prep_(z, H, G, dk, dv, k_cache=r.cache.k[run], v_cache=r.cache.v[run], slots=sb.slots, rot=self._rotation(a.rot, sb))
+        return r.attend(run, z[:, :H * dk], z[:, H * dk:ov], z[:, ov:], sb, a.scale, self.rules[i])
+
+    def _latent(self, run, i, m, p, h, sb):
+        r, P, cols = self.r, self.r.params, self.columns[i]
+        z = gemm(h, P.w(p + "attn.in"))
+        part = lambda c: z[:, cols[c][0]:cols[c][0] + cols[c][1]]
+        table = sb.rotation(m.rot, self.freqs[m.rot])
+        latent_ops.latent_prep_(z, cols["q"][0], m.q_rank, cols["kv"][0], m.kv_rank, m.rot_dim, q_gamma=P.w(p + "attn.q_norm"),
+                                kv_gamma=P.w(p + "attn.kv_norm"), eps=self.cfg.norm_eps, table=table, cache=r.cache.k[run], slots=sb.slots)
+        q = gemm(part("q"), P.w(p + "attn.uq"))
+        return r.attend_latent(run, q, part("kv"), sb, m, P.w(p + "attn.ukv"), table, part("g") if "g" in cols else None)
+
+    def _experts(self, h, m, p):
+        P = self.r.params
+        logits = gemm(h, P.w(p + "moe.router"), out_dtype=torch.float32)
+        if m.score == "sigmoid":
+            idx, w = moe_ops.route_sigmoid(logits, m.top, m.groups, m.keep, P.w(p + "moe.correction") if m.correction else None,
+                                           m.group_best, m.renorm)
+        else:
+            idx, w = moe_ops.route_groups(logits, m.top, m.groups, m.keep, m.renorm)
+        pl = moe_ops.plan(idx, m.experts)
+        gu = moe_ops.grouped_gemm(moe_ops.scatter_tokens(h, pl), P.w(p + "moe.w1"), pl)
+        y = moe_ops.grouped_gemm(moe_ops.swiglu_rows(gu, pl, m.act, limit=m.limit), P.w(p + "moe.w2"), pl)
+        return y, (pl.slot_pos, w)
+
+    def head(self, st, rows):
+        P, cfg = self.r.params, self.cfg
+        x = st.x if rows is None else ops.gather_rows(st.x, rows)
+        h = norm_ops.residual_norm(x, P.w("final.norm"), None, cfg.norm_eps, True, h=torch.empty_like(x, dtype=self.r.dtype))
+        logits = gemm(h, P.w("head"), out_dtype=torch.float32)
+        if cfg.logit_scale != 1.0 or cfg.logit_softcap:
+            ops.scale_softcap_(logits, cfg.logit_scale, cfg.logit_softcap)
         return logits

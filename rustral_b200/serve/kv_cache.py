@@ -169,11 +169,13 @@ class SlidingWindowCache(KVCache):
 @dataclass(frozen=True)
 class CacheLayer:
     """What one layer stores: per token `kv_heads` keys of size `k_dim` and values of size `v_dim` (kv_heads 0: none), and
-    per sequence the tensors of `state`, each (name, shape, dtype or None for the cache's)."""
+    per sequence the tensors of `state`, each (name, shape, dtype or None for the cache's).  `joint`: the values are the first
+    `v_dim` numbers of the keys and take no room of their own."""
     kv_heads: int = 0
     k_dim: int = 0
     v_dim: int = 0
     state: tuple = ()
+    joint: bool = False
 
 
 class PagedCache:
@@ -205,7 +207,8 @@ class PagedCache:
             def pages(c, d):
                 return torch.zeros((num_blocks, block_size, c.kv_heads, d), dtype=dtype, device=device) if c.kv_heads else None
             self.k = [pages(c, c.k_dim) for c in layers]
-            self.v = [pages(c, c.v_dim) for c in layers]
+            self.v = [k[..., :c.v_dim] if c.joint else pages(c, c.v_dim) for c, k in zip(layers, self.k)]
+            self._joint = [c.joint for c in layers]
             self.state = [{n: torch.zeros((num_slots, *shape), dtype=dt or dtype, device=device) for n, shape, dt in c.state}
                           for c in layers]
         elif allocate_storage:
@@ -260,7 +263,9 @@ class PagedCache:
     def memory_bytes(self) -> int:
         if self.k is None:
             return 0
-        held = [t for c in (self.k, self.v) for t in c if t is not None] + [t for d in self.state for t in d.values()]
+        joint = getattr(self, "_joint", [False] * len(self.v))
+        held = [*self.k, *(v for v, j in zip(self.v, joint) if not j)]
+        held = [t for t in held if t is not None] + [t for d in self.state for t in d.values()]
         return sum(t.numel() * t.element_size() for t in held)
 
 

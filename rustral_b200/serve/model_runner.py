@@ -15,7 +15,10 @@ import torch
 from .. import ops
 from ..models.registry import architecture, build_weights
 from ..ops import attention as attn_ops
+from ..ops import latent as latent_ops
 from ..ops import paged as paged_ops
+from ..ops import rotary as rope_ops
+from ..ops.matmul import gemm
 from ..ops.recurrent import Segments
 from ..runtime.fused_gpt import FlatParams
 from . import decoder_body
@@ -34,7 +37,26 @@ class StepBatch:
         self.bt, self.ctx = bt, ctx                               # decode rows: block tables, context lengths (int32)
         self.block_size = block_size
         self.segments = segments
-        self._keys, self._row_tables = {}, None
+        self._keys, self._row_tables, self._rotations, self._all_keys = {}, None, {}, None
+
+    def rotation(self, rot, freqs: torch.Tensor) -> torch.Tensor:
+        """Cosines and sines of the rows' positions for the rotary positions `rot` (models.layered.RotarySpec), one table for all
+        layers that share them."""
+        if rot not in self._rotations:
+            self._rotations[rot] = rope_ops.rotary_table(self.pos, freqs, rot.magnitude)
+        return self._rotations[rot]
+
+    def all_keys(self):
+        """(cache slots of every position up to the end of each portion, one portion after the other; first entry of each portion and
+        the end).  Slots are None where the portions are whole prompts: the keys are the step's own rows."""
+        if self._all_keys is None:
+            ends = [0]
+            for r0, r1, start in self.spans:
+                ends.append(ends[-1] + start + r1 - r0)
+            whole = all(start == 0 for _, _, start in self.spans)
+            slots = None if whole else torch.cat([self.key_slots(i, 0) for i in range(len(self.spans))])
+            self._all_keys = (slots, ends)
+        return self._all_keys
 
     def key_slots(self, i: int, first: int, kept: int = 0) -> torch.Tensor:
         """Cache slots of positions 0 .. `kept` and `first` .. end of portion i (earlier portions and this one)."""
@@ -141,11 +163,43 @@ class ModelRunner:
                                              head_gate=None if head_gate is None else head_gate[sb.rd:])
         return a
 
+    def attend_latent(self, l: int, q, kv, sb: StepBatch, m, w_ukv, table, gate=None) -> torch.Tensor:
+        """Latent attention of layer `l` (`m`: models.layered.LatentSpec) for every row of `sb`.  q [rows, heads * qk_dim] (not rotated
+        yet), kv [rows, cached]: the vectors and rotated key parts, already in the cache; w_ukv: the heads' key products, then their
+        value products.  Prompt portions form keys and values of all positions they see and go through the flash kernel; decoded rows
+        (and portions that it does not take) work on the cached vectors."""
+        H, dn, dr, dv, R = m.heads, m.dim, m.rot_dim, m.vdim, m.kv_rank
+        cache, T, rd = self.cache.k[l], sb.rows, sb.rd
+        a = torch.empty((T, H * dv), dtype=q.dtype, device=self.device)
+        flash = False
+        if sb.spans:
+            slots, ends = sb.all_keys()
+            keys = kv[:rd] if slots is None else ops.gather_rows(cache.view(-1, m.cached), slots)
+            flash = attn_ops.split_supported(dn, dr, dv, q, keys, keys[:, R:], gate)
+        if flash:
+            both = gemm(keys[:, :R], w_ukv)                       # keys of all heads, then values of all heads
+            rope_ops.rotate_pairs_(q[:rd], H, m.qk_dim, dn, table[:rd])
+            for i, (r0, r1, _) in enumerate(sb.spans):
+                L, k0, k1 = r1 - r0, ends[i], ends[i + 1]
+                attn_ops.prompt_attention_split(q[r0:r1].view(1, L, H, dn + dr), both[k0:k1, :H * dn].view(1, -1, H, dn),
+                                                both[k0:k1, H * dn:].view(1, -1, H, dv), keys[k0:k1, R:], m.scale,
+                                                out=a[r0:r1].view(1, L, H, dv), gate=None if gate is None else gate[r0:r1])
+        lo = rd if flash else 0                                   # rows that work on the cached vectors
+        if lo < T:
+            qa = latent_ops.head_product(q[lo:], m.qk_dim, w_ukv[:H * dn], H, R, dn, transposed=True, tail=dr, table=table[lo:])
+            if lo == rd and latent_ops.latent_decode_supported(qa, R, dr):
+                c = latent_ops.latent_decode(qa, cache, R, sb.bt, sb.ctx, m.scale)
+            else:
+                bt, seq = sb.row_tables()
+                c = paged_ops.paged_attention_rows(qa, cache, self.cache.v[l], bt, seq[lo:], sb.pos[lo:], m.scale)
+            latent_ops.head_product(c, R, w_ukv[H * dn:], H, dv, R, transposed=False, gate=None if gate is None else gate[lo:], out=a[lo:])
+        return a
+
     # ---- one model pass ----------------------------------------------------------------------------------------------
     def _run(self, sb: StepBatch, rows) -> torch.Tensor | None:
         """All layers over the rows of `sb`; logits of the rows `rows` (int64 tensor, None: every row, [] : none)."""
         x = self.body.embed(sb)
-        for l in range(self.cfg.n_layer):
+        for l in range(self.body.depth):
             x = self.body.layer(l, x, sb)
         logits = None if isinstance(rows, list) else self.body.head(x, rows)
         if self.tp is not None:

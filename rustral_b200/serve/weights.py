@@ -9,7 +9,7 @@ import zlib
 import torch
 
 from ..models.config import GPTConfig
-from ..models.layered import ParallelSpec, up8
+from ..models.layered import DenseSpec, LatentSpec, ParallelSpec, up8
 
 
 class InferenceWeights:
@@ -132,6 +132,8 @@ class InferenceWeights:
             if tensors is not None:
                 return tensors[name].reshape(shape).to(dev, dt)
             last = name.rsplit(".", 1)[-1]
+            if last == "correction" or (cfg.design.norm == "rms" and (last in ("norm1", "norm1b", "norm2", "norm2b") or name == "final.norm")):
+                return torch.zeros(shape, dtype=dt, device=dev)
             if last in ("norm", "norm1", "norm2", "out", "D"):
                 return torch.ones(shape, dtype=dt, device=dev)
             if last == "b" and len(shape) == 1:
@@ -156,16 +158,38 @@ class InferenceWeights:
             out[f8:f8 + ff] = get(p + "up")
 
         d = cfg.d_model
-        t = {"embed": get("embed"), "head": torch.zeros((cfg.vocab_padded, d), dtype=dt, device=dev)}
-        t["head"][:cfg.vocab_size] = get("head")
+        t = {"head": torch.zeros((cfg.vocab_padded, d), dtype=dt, device=dev)}
+        if cfg.design.tied:
+            t["head"][:cfg.vocab_size] = get("embed")
+            t["embed"] = t["head"][:cfg.vocab_size]
+        else:
+            t["embed"] = get("embed")
+            t["head"][:cfg.vocab_size] = get("head")
 
         def norm(name):
-            if cfg.design.norm == "dyt":
+            if cfg.design.norm == "rms":
+                t[name] = 1.0 + f32(name)                  # stored as the difference from one
+            elif cfg.design.norm == "dyt":
                 t[name], t[name + ".b"], t[name + ".alpha"] = f32(name), f32(name + ".b"), f32(name + ".alpha").reshape(1)
             else:
                 t[name], t[name + ".b"] = get(name), get(name + ".b")
 
+        def experts(p, m):
+            """Router and stacked experts of one layer."""
+            t[p + "moe.router"] = get(p + "mlp.router")
+            if m.correction:
+                t[p + "moe.correction"] = f32(p + "mlp.correction")
+            f8 = up8(m.ff)
+            w1 = torch.zeros((m.experts, 2 * f8, d), dtype=dt, device=dev)
+            w2 = torch.zeros((m.experts, d, f8), dtype=dt, device=dev)
+            for e in range(m.experts):
+                gate_up(f"{p}mlp.e{e}.", m.ff, w1[e])
+                w2[e, :, :m.ff] = get(f"{p}mlp.e{e}.down")
+            t[p + "moe.w1"], t[p + "moe.w2"] = w1, w2
+
         norm("final.norm")
+        if cfg.loop is not None:
+            t["loop.in"], t["loop.step"] = get("loop.in"), get("loop.step")
         for i, s in enumerate(cfg.layers):
             if cfg.owner(i) != i:
                 continue
@@ -175,6 +199,17 @@ class InferenceWeights:
                 continue
             p, m = f"l{i}.", s.mlp
             norm(p + "norm1")
+            if cfg.design.block == "sandwich":
+                norm(p + "norm1b")
+                cls._mixer_in_front(t, p, s.mixer, d, get, f32, dt, dev)
+                if m is not None:
+                    norm(p + "norm2")
+                    norm(p + "norm2b")
+                    if isinstance(m, DenseSpec):
+                        t[p + "up"], t[p + "down"] = _pitched(get(p + "mlp.up")), _pitched(get(p + "mlp.down"))
+                    else:
+                        experts(p, m)
+                continue
             t[p + "attn.in"] = torch.cat([get(p + "mix." + c) for c in "qkvg"], 0)
             t[p + "attn.out"] = get(p + "mix.o")
             t[p + "attn.q_norm"], t[p + "attn.k_norm"] = get(p + "mix.q.norm"), get(p + "mix.k.norm")
@@ -183,14 +218,7 @@ class InferenceWeights:
             if m is None:
                 continue
             norm(p + "norm2")
-            t[p + "moe.router"] = get(p + "mlp.router")
-            f8 = up8(m.ff)
-            w1 = torch.zeros((m.experts, 2 * f8, d), dtype=dt, device=dev)
-            w2 = torch.zeros((m.experts, d, f8), dtype=dt, device=dev)
-            for e in range(m.experts):
-                gate_up(f"{p}mlp.e{e}.", m.ff, w1[e])
-                w2[e, :, :m.ff] = get(f"{p}mlp.e{e}.down")
-            t[p + "moe.w1"], t[p + "moe.w2"] = w1, w2
+            experts(p, m)
             if m.shared_ff:
                 f8 = up8(m.shared_ff)
                 w1 = torch.zeros((2 * f8, d), dtype=dt, device=dev)
@@ -199,6 +227,27 @@ class InferenceWeights:
                 w2[:, :m.shared_ff] = get(p + "mlp.shared.down")
                 t[p + "shared.in"], t[p + "shared.out"] = w1, w2
         return cls(t, dt)
+
+    @staticmethod
+    def _mixer_in_front(t, p, m, d, get, f32, dt, dev) -> None:
+        """The mixer of a layer with a norm in front: one packed projection of everything that reads it (`latent_columns` for
+        latent attention, whose key and value products of all heads are stacked)."""
+        x = p + "mix."
+        t[p + "attn.out"] = _pitched(get(x + "o"))
+        if not isinstance(m, LatentSpec):
+            t[p + "attn.in"] = torch.cat([get(x + c) for c in "qkv"], 0)
+            if m.bias:
+                t[p + "attn.in.b"] = torch.cat([get(x + c + ".b") for c in "qkv"], 0)
+            return
+        cols = latent_columns(m)
+        w = torch.zeros((cols["end"][0], d), dtype=dt, device=dev)
+        for nm, src in (("q", "dq"), ("kv", "dkv"), ("g", "g")):
+            if nm in cols:
+                w[cols[nm][0]:cols[nm][0] + cols[nm][1]] = get(x + src)
+        t[p + "attn.in"] = w
+        t[p + "attn.q_norm"], t[p + "attn.kv_norm"] = f32(x + "dq.norm"), f32(x + "dkv.norm")
+        t[p + "attn.uq"] = _pitched(get(x + "uq"))
+        t[p + "attn.ukv"] = _pitched(torch.cat([get(x + "uk"), get(x + "uv")], 0))
 
     @staticmethod
     def _parallel_block(t, p, s, d, get, f32, dt, dev) -> None:
@@ -270,3 +319,24 @@ def packed_columns(s) -> tuple:
         out["end"] = (at, 0)
         return out
     return place(groups), place(small)
+
+
+def latent_columns(m) -> dict:
+    """Columns of the packed projection of a latent attention layer: query latent, cached vector with the shared key part, gate; every
+    section starts at a multiple of 8."""
+    out, at = {}, 0
+    for nm, n in (("q", m.q_rank), ("kv", m.cached), ("g", m.heads * m.vdim if m.gate == "element" else 0)):
+        if n:
+            out[nm] = (at, n)
+            at = up8(at + n)
+    out["end"] = (at, 0)
+    return out
+
+
+def _pitched(w: torch.Tensor) -> torch.Tensor:
+    """The same matrix with rows that start at multiples of 8 elements (a view of a wider buffer where its own are not)."""
+    if w.shape[1] % 8 == 0:
+        return w
+    out = torch.zeros((w.shape[0], up8(w.shape[1])), dtype=w.dtype, device=w.device)
+    out[:, :w.shape[1]] = w
+    return out[:, :w.shape[1]]
