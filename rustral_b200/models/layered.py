@@ -109,10 +109,10 @@ class AttentionSpec:
         return self.heads * self.dim + self.kv_heads * (self.dim + self.vdim) + (self.heads * self.vdim if self.gate == "element" else 0)
 
     def tensor_shapes(self, p: str, d: int) -> dict:
-        t = {p + "q": (self.heads * self.dim, d), p + "k": (self.kv_heads * self.dim, d), p + "v": (self.kv_heads * self.vdim, d),
-             p + "o": (d, self.heads * self.vdim)}
+        t = {p + "q": (self.heads * self.dim, d), p + "k": (self.kv_heads * self.dim, d), p + "v": (self.kv_heads * self.vdim, d)}
         if self.gate != "none":
             t[p + "g"] = (self.heads * self.vdim if self.gate == "element" else self.heads, d)
+        t[p + "o"] = (d, self.heads * self.vdim)
         if self.bias:
             t.update({p + c + ".b": t[p + c][:1] for c in "qkv"})
         if self.qk_norm:

@@ -10,6 +10,8 @@ and the cached decode its TransformerDecoder::generate_token does not have (full
 """
 from __future__ import annotations
 
+import gc
+
 import torch
 
 from .. import ops
@@ -343,8 +345,15 @@ class ModelRunner:
             out = self._decode_body(g["ids"], g["ctx"], g["bt"], g["seg"])
             torch.cuda.current_stream().synchronize()
             graph = torch.cuda.CUDAGraph()
-            with torch.cuda.graph(graph):
-                g["out"] = self._decode_body(g["ids"], g["ctx"], g["bt"], g["seg"])
+            # A collection in the middle of a capture could destroy an earlier runner's graphs, which ends the capture with an error
+            collecting = gc.isenabled()
+            gc.disable()
+            try:
+                with torch.cuda.graph(graph):
+                    g["out"] = self._decode_body(g["ids"], g["ctx"], g["bt"], g["seg"])
+            finally:
+                if collecting:
+                    gc.enable()
             g["graph"] = graph
             return out
         g["graph"].replay()

@@ -178,3 +178,10 @@ def forward(cfg, w, tokens, layers_out=None):
         if layers_out is not None:
             layers_out.append(x)
     return centred_norm(x, w["final.norm"], eps) @ w["embed"].T
+
+
+def greedy(cfg, w, prompt, n):
+    toks = list(prompt)
+    for _ in range(n):
+        toks.append(int(forward(cfg, w, toks)[-1].argmax()))
+    return toks[len(prompt):]
