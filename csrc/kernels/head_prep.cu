@@ -179,6 +179,56 @@ head_prep_scalar_kernel(const RbHeadPrepArgs a RB_BOUNDS_PARAM) {
   }
 }
 
+// Without norms and mixing: positions and append only.  One CTA per token, a thread per vector: the rotated vectors of the queries, then
+// those of the keys and the values.
+template <typename T>
+__global__ void __launch_bounds__(256)
+head_rotate_append_kernel(const RbHeadPrepArgs a RB_BOUNDS_PARAM) {
+  using V = HpVec<T>;
+  const long long t = blockIdx.x;
+  T* row = reinterpret_cast<T*>(a.p) + t * a.ld;
+  const int rotated = a.rot ? a.rot_dims : 0;
+  const int uq = (rotated + V::N - 1) / V::N, uk = a.dk / V::N, uv = a.dv / V::N;
+  const int nq = a.heads * uq, nk = a.kv_heads * uk, total = nq + nk + a.kv_heads * uv;
+  bool stored = false;
+  long long slot = 0;
+  if (a.k_cache) {
+    slot = a.slots[t];
+    if (slot >= a.num_slots && threadIdx.x == 0) RB_BOUNDS_HIT(103);       // a negative slot means "skip this token"
+    stored = slot >= 0 && slot < a.num_slots;
+  }
+  for (int u = threadIdx.x; u < total; u += blockDim.x) {
+    int head, col;
+    T* src;
+    T* dst = nullptr;
+    if (u < nq) {
+      head = u / uq;
+      col = (u - head * uq) * V::N;
+      src = row + a.off_q + head * a.dk + col;
+    } else if (u < nq + nk) {
+      head = (u - nq) / uk;
+      col = (u - nq - head * uk) * V::N;
+      src = row + a.off_k + head * a.dk + col;
+      if (stored) dst = reinterpret_cast<T*>(a.k_cache) + (slot * a.kv_heads + head) * a.dk + col;
+    } else {
+      col = (u - nq - nk) * V::N;                                          // the value heads are contiguous on both sides
+      src = row + a.off_v + col;
+      if (stored) dst = reinterpret_cast<T*>(a.v_cache) + slot * a.kv_heads * a.dv + col;
+    }
+    const bool turn = u < nq + nk && col < rotated;
+    if (!turn && !dst) continue;
+    float v[V::N];
+    V::load(src, v);
+    if (turn) {
+#pragma unroll
+      for (int i = 0; i < V::N; i += 2)
+        if (col + i < rotated) hp_rotate(a, t, col + i, v[i], v[i + 1]);
+      V::store(src, v);
+    }
+    if (dst) V::store(dst, v);
+  }
+}
+
 template <typename T>
 int hp_launch(const RbHeadPrepArgs& a, cudaStream_t s) {
   constexpr int N = HpVec<T>::N;
@@ -192,7 +242,10 @@ int hp_launch(const RbHeadPrepArgs& a, cudaStream_t s) {
   const int per_block = vec ? (narrow ? 16 : 8) : 4;
   long long blocks = (total + per_block - 1) / per_block;
   if (blocks > 148LL * 16) blocks = 148LL * 16;
-  if (vec && narrow)
+  const int units = (a.rot ? a.heads * ((a.rot_dims + N - 1) / N) : 0) + a.kv_heads * (a.dk + a.dv) / N;
+  if (vec && !a.q_gamma && !a.k_gamma && !a.v_first && a.tokens <= 0x7fffffffLL)
+    head_rotate_append_kernel<T><<<static_cast<int>(a.tokens), units <= 64 ? 64 : units <= 128 ? 128 : 256, 0, s>>>(a RB_BOUNDS_ARG);
+  else if (vec && narrow)
     head_prep_kernel<T, 8><<<static_cast<int>(blocks), 128, 0, s>>>(a RB_BOUNDS_ARG);
   else if (vec)
     head_prep_kernel<T, 16><<<static_cast<int>(blocks), 128, 0, s>>>(a RB_BOUNDS_ARG);

@@ -6,6 +6,7 @@
 // form keys and values (attention_fwd2.cu takes the shared rotated part as it is).
 #include "latent_attention.h"
 
+#include "latent_common.cuh"
 #include "rb_common.cuh"
 #include "warp_mma.cuh"
 
@@ -121,13 +122,14 @@ int lp_launch(const RbLatentPrepArgs& a, cudaStream_t s) {
 // ---- one small product per head ------------------------------------------------------------------------------------------------
 // 64 tokens x BN columns of one head per CTA, 64-deep slices through a ring of shared-memory stages, a warp owns 16 tokens.  Batches of
 // decoded tokens are far smaller than a tcgen05 tile's 128 rows per head; the kernel is bound by reading the weights.
-constexpr int kHpStages = 3, kHpRows = 64, kHpK = 64, kHpPitch = 72;
+constexpr int kHpRows = 64, kHpK = 64, kHpPitch = 72;
 
 template <int BN, bool TR>
 struct HpSmem {
+  static constexpr int kStages = BN == 32 ? 8 : 4;       // narrow tiles serve few heads: depth instead of CTAs
   static constexpr int kWRows = TR ? kHpK : BN, kWPitch = TR ? BN + 8 : kHpPitch;
   static constexpr int kX = kHpRows * kHpPitch, kStage = kX + kWRows * kWPitch;
-  static constexpr int kBytes = kHpStages * kStage * 2;
+  static constexpr int kBytes = kStages * kStage * 2;
 };
 
 template <int BN, bool TR>
@@ -142,7 +144,7 @@ head_product_kernel(const RbHeadProductArgs a) {
   const int steps = (a.k + kHpK - 1) / kHpK;
   auto request = [&](int st) {
     if (st < steps) {
-      __nv_bfloat16* xs = hp_sm + (st % kHpStages) * S::kStage;
+      __nv_bfloat16* xs = hp_sm + (st % S::kStages) * S::kStage;
       const uint32_t xb = smem_u32(xs), wb = smem_u32(xs + S::kX);
       const int k0 = st * kHpK;
 #pragma unroll
@@ -165,15 +167,15 @@ head_product_kernel(const RbHeadProductArgs a) {
   float acc[BN / 8][4];
 #pragma unroll
   for (int i = 0; i < BN / 8; ++i) acc[i][0] = acc[i][1] = acc[i][2] = acc[i][3] = 0.f;
-  request(0);
-  request(1);
+#pragma unroll
+  for (int i = 0; i < S::kStages - 1; ++i) request(i);
   const bool active = r0 + warp * 16 < a.rows;
   for (int st = 0; st < steps; ++st) {
-    wm_cp_wait<1>();
+    wm_cp_wait<S::kStages - 2>();
     __syncthreads();                                     // slice st has landed for everyone, slice st - 1 is no longer read
-    request(st + 2);
+    request(st + S::kStages - 1);
     if (!active) continue;
-    const uint32_t xb = smem_u32(hp_sm + (st % kHpStages) * S::kStage), wb = xb + S::kX * 2;
+    const uint32_t xb = smem_u32(hp_sm + (st % S::kStages) * S::kStage), wb = xb + S::kX * 2;
 #pragma unroll
     for (int k0 = 0; k0 < kHpK; k0 += 16) {
       uint32_t af[4];
@@ -208,16 +210,20 @@ head_product_kernel(const RbHeadProductArgs a) {
       *reinterpret_cast<uint32_t*>(Y + r * a.ld_y + n) = pack_bf16x2(u, v);
     }
   }
-  if (a.tail && blockIdx.x == 0) {
-    const int rows = min(kHpRows, a.rows - r0), pairs = a.tail / 2;
-    for (int i = threadIdx.x; i < rows * pairs; i += 128) {
-      const int r = r0 + i / pairs, c = i % pairs;
-      float2 z = unpack_bf16x2(*reinterpret_cast<const uint32_t*>(X + r * a.ld_x + a.tail_off + 2 * c));
-      if (c < a.pairs) {
-        const float2 cs = __ldg(reinterpret_cast<const float2*>(a.table) + static_cast<long long>(r) * a.pairs + c);
-        z = make_float2(z.x * cs.x - z.y * cs.y, z.y * cs.x + z.x * cs.y);
+  if (a.tail) {                                          // 8 columns of one row per thread, spread over the head's CTAs
+    const int units = a.tail / 8, total = min(kHpRows, a.rows - r0) * units;
+    for (int i = blockIdx.x * 128 + threadIdx.x; i < total; i += gridDim.x * 128) {
+      const int r = r0 + i / units, c = i % units * 8;
+      uint4 u = *reinterpret_cast<const uint4*>(X + r * a.ld_x + a.tail_off + c);
+      uint32_t* w = reinterpret_cast<uint32_t*>(&u);
+#pragma unroll
+      for (int q = 0; q < 4; ++q) {
+        if (c / 2 + q >= a.pairs) break;
+        const float2 cs = __ldg(reinterpret_cast<const float2*>(a.table) + static_cast<long long>(r) * a.pairs + c / 2 + q);
+        const float2 z = unpack_bf16x2(w[q]);
+        w[q] = pack_bf16x2(z.x * cs.x - z.y * cs.y, z.y * cs.x + z.x * cs.y);
       }
-      *reinterpret_cast<uint32_t*>(Y + r * a.ld_y + a.n + 2 * c) = pack_bf16x2(z.x, z.y);
+      *reinterpret_cast<uint4*>(Y + r * a.ld_y + a.n + c) = u;
     }
   }
 }
@@ -266,7 +272,7 @@ head_product_plain_kernel(const RbHeadProductArgs a) {
   }
 }
 
-// ---- decode -------------------------------------------------------------------------------------------------------------------------
+// ---- decode: page sizes and rotated parts that latent_decode_tc.cu does not take --------------------------------------------------------
 // One CTA = (slice of the context, sequence, 16 MT heads).  64 tokens at a time are copied into one of two shared-memory tiles (the next
 // tile flies while this one is used) and serve all heads, for the scores and for the weighted sum.
 //   scores: the warps form 4 groups over the columns times 2 over the tokens; a warp's share of the queries stays in registers, the
@@ -287,7 +293,7 @@ struct LdSmem {
 
 template <int MT, int VW, int KMAX>
 __global__ void __launch_bounds__(kLdWarps * 32, 1)
-latent_decode_kernel(const RbLatentDecodeArgs a, int slice, int nsplit RB_BOUNDS_PARAM) {
+latent_decode_kernel(const RbLatentDecodeArgs a, int nsplit RB_BOUNDS_PARAM) {
   using S = LdSmem<MT>;
   extern __shared__ __align__(16) uint8_t ld_sm[];
   const int width = a.rank + a.rot, width16 = (width + 15) / 16 * 16, pitch = width16 + 8;
@@ -300,6 +306,7 @@ latent_decode_kernel(const RbLatentDecodeArgs a, int slice, int nsplit RB_BOUNDS
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int gq = lane >> 2, tq = lane & 3;
   const int ctx = a.context_lens[b];
+  const int slice = latent_chunk(ctx, nsplit);
   const int t_begin = sp * slice;
   if (t_begin >= ctx) return;
   const int t_end = min(ctx, t_begin + slice);
@@ -505,10 +512,11 @@ latent_decode_kernel(const RbLatentDecodeArgs a, int slice, int nsplit RB_BOUNDS
 
 // out[b, h, :] = merge over the slices that hold tokens of sequence b; a thread owns two columns
 __global__ void __launch_bounds__(256)
-latent_merge_kernel(const float* __restrict__ partial, const int* __restrict__ context_lens, int heads, int rank, int slice, int nsplit,
+latent_merge_kernel(const float* __restrict__ partial, const int* __restrict__ context_lens, int heads, int rank, int nsplit,
                     __nv_bfloat16* __restrict__ out, long long ld_o) {
   const int h = blockIdx.x, b = blockIdx.y;
-  const int n = min(nsplit, (context_lens[b] + slice - 1) / slice);
+  const int ctx = context_lens[b], slice = latent_chunk(ctx, nsplit);
+  const int n = min(nsplit, (ctx + slice - 1) / slice);
   const float* base = partial + (static_cast<long long>(b) * heads + h) * nsplit * (rank + 2);
   float mx = -INFINITY;
   for (int s = 0; s < n; ++s) mx = fmaxf(mx, base[static_cast<long long>(s) * (rank + 2)]);
@@ -528,7 +536,7 @@ latent_merge_kernel(const float* __restrict__ partial, const int* __restrict__ c
 }
 
 template <int MT, int VW, int KMAX>
-int ld_launch(const RbLatentDecodeArgs& a, int slice, int nsplit, cudaStream_t s) {
+int ld_launch(const RbLatentDecodeArgs& a, int nsplit, cudaStream_t s) {
   auto kern = latent_decode_kernel<MT, VW, KMAX>;
   const int smem = LdSmem<MT>::bytes((a.rank + a.rot + 15) / 16 * 16);
   static bool cfg[64] = {};
@@ -539,17 +547,22 @@ int ld_launch(const RbLatentDecodeArgs& a, int slice, int nsplit, cudaStream_t s
     if (e != cudaSuccess) return static_cast<int>(e);
     done = true;
   }
-  kern<<<dim3((a.heads + 16 * MT - 1) / (16 * MT), nsplit, a.batch), kLdWarps * 32, smem, s>>>(a, slice, nsplit RB_BOUNDS_ARG);
-  if (nsplit > 1)
-    latent_merge_kernel<<<dim3(a.heads, a.batch), a.rank <= 128 ? 64 : 256, 0, s>>>(a.scratch, a.context_lens, a.heads, a.rank, slice, nsplit,
-                                                                                  reinterpret_cast<__nv_bfloat16*>(a.out), a.ld_o);
+  kern<<<dim3((a.heads + 16 * MT - 1) / (16 * MT), nsplit, a.batch), kLdWarps * 32, smem, s>>>(a, nsplit RB_BOUNDS_ARG);
   return static_cast<int>(cudaGetLastError());
 }
 
-// Tokens per slice: enough slices to fill the GPU where the batch alone does not
-inline int ld_slice(int batch, int heads) {
-  const int ctas = batch * ((heads + 31) / 32);
-  return ctas >= 64 ? 512 : ctas >= 16 ? 256 : 128;
+// Slices per sequence: as many as make a launch of one CTA per SM shortest, for contexts of 4096 tokens (or what the tables can hold).
+// It depends on the batch and the tables' width only, which a captured graph keeps.
+inline int ld_splits(int batch, int heads, long long capacity) {
+  const long long ctas = static_cast<long long>(batch) * ((heads + 31) / 32);
+  const long long ctx = capacity < 4096 ? capacity : 4096;
+  int best = 1;
+  long long best_cost = 0;
+  for (int s = 1; s <= 64 && (s == 1 || (s - 1) * 128 < capacity); ++s) {
+    const long long cost = (ctas * s + 147) / 148 * ((ctx + s - 1) / s + 256);
+    if (s == 1 || cost < best_cost) { best = s; best_cost = cost; }
+  }
+  return best;
 }
 
 }  // namespace rb
@@ -589,8 +602,7 @@ RB_API int rb_head_product(const RbHeadProductArgs* args, void* stream_v) {
 }
 
 RB_API long long rb_latent_decode_scratch_floats(int batch, int heads, int rank, int max_blocks, int block_size) {
-  const int slice = rb::ld_slice(batch, heads);
-  const long long nsplit = (static_cast<long long>(max_blocks) * block_size + slice - 1) / slice;
+  const int nsplit = rb::ld_splits(batch, heads, static_cast<long long>(max_blocks) * block_size);
   return nsplit > 1 ? static_cast<long long>(batch) * heads * nsplit * (rank + 2) : 1;
 }
 
@@ -605,14 +617,16 @@ RB_API int rb_latent_decode(const RbLatentDecodeArgs* args, void* stream_v) {
       (reinterpret_cast<uintptr_t>(a.scratch) & 7))
     return -2;
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream_v);
-  const int slice = rb::ld_slice(a.batch, a.heads);
-  const long long nsplit = (static_cast<long long>(a.max_blocks) * a.block_size + slice - 1) / slice;
-  if (nsplit > 65535) return -1;
-  const int width = a.rank + a.rot, n = static_cast<int>(nsplit);
-  const bool two = a.heads > 16;
-  if (a.rank <= 128 && width <= 256)
-    return two ? rb::ld_launch<2, 16, 4>(a, slice, n, s) : rb::ld_launch<1, 16, 4>(a, slice, n, s);
-  if (a.rank <= 256 && width <= 384)
-    return two ? rb::ld_launch<2, 32, 6>(a, slice, n, s) : rb::ld_launch<1, 32, 6>(a, slice, n, s);
-  return two ? rb::ld_launch<2, 64, 10>(a, slice, n, s) : rb::ld_launch<1, 64, 10>(a, slice, n, s);
+  const int n = rb::ld_splits(a.batch, a.heads, static_cast<long long>(a.max_blocks) * a.block_size), width = a.rank + a.rot;
+  int rc = rb::latent_decode_tc(a, n, s);
+  if (rc == -9) {
+    const bool two = a.heads > 16;
+    if (a.rank <= 128 && width <= 256) rc = two ? rb::ld_launch<2, 16, 4>(a, n, s) : rb::ld_launch<1, 16, 4>(a, n, s);
+    else if (a.rank <= 256 && width <= 384) rc = two ? rb::ld_launch<2, 32, 6>(a, n, s) : rb::ld_launch<1, 32, 6>(a, n, s);
+    else rc = two ? rb::ld_launch<2, 64, 10>(a, n, s) : rb::ld_launch<1, 64, 10>(a, n, s);
+  }
+  if (rc || n == 1) return rc;
+  rb::latent_merge_kernel<<<dim3(a.heads, a.batch), a.rank <= 128 ? 64 : 256, 0, s>>>(a.scratch, a.context_lens, a.heads, a.rank, n,
+                                                                                    reinterpret_cast<__nv_bfloat16*>(a.out), a.ld_o);
+  return static_cast<int>(cudaGetLastError());
 }

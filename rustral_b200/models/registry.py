@@ -60,7 +60,7 @@ _HYBRID_KERNELS = ("gemm_tcgen05", "gemm_f32", "embedding", "elementwise", "resi
                    "paged_attention", "short_conv", "state_space", "state_space_chunk", "delta_rule",
                    "delta_rule_chunk", "gated_norm")
 
-_SANDWICH_KERNELS = (*_LAYERED_KERNELS, "rope", "latent_attention")
+_SANDWICH_KERNELS = (*_LAYERED_KERNELS, "rope", "latent_attention", "latent_decode_tc")
 
 ARCHITECTURES = {a.name: a for a in (
     Architecture("gpt2", _gpt_config, "GPTBody", False, _gpt_weights, _GPT_KERNELS),
