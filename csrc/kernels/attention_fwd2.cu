@@ -296,7 +296,7 @@ attn_fwd2_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
   if (warp >= 8) {
   setmaxnreg_dec<56>();
   if (warp == 8) {
-    if (lane == 0) {
+    if (elect_one()) {
       // ---------------------------------------------------------------- TMA producer
 #pragma unroll
       for (int t = 0; t < 2; ++t) {
@@ -326,21 +326,25 @@ attn_fwd2_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
       }
     }
   } else if (warp == 9) {
-    if (lane == 0) {
+    // elect_one, not lane 0: the compiler then knows that one lane runs this and keeps the descriptors in uniform registers
+    if (elect_one()) {
       // ---------------------------------------------------------------- MMA issuer
+      // descriptors of the first tile and stage; an offset of o bytes is o / 16 in the address field
+      const uint64_t dQ = umma_smem_desc_sw128(sQ, 16, 1024), dK = umma_smem_desc_sw128(sK, 16, 1024), dV = umma_smem_desc_sw128(sV, L::kHalf, 1024);
       constexpr uint32_t idesc_qk = umma_idesc_bf16(128, 128, 0, 0);
       constexpr uint32_t idesc_pv = umma_idesc_bf16(128, DV, 0, 1);        // A = P (TMEM, K-major), B = V MN-major
       auto issue_qk = [&](int j, int t) -> bool {
         const int s = (j - f_min) % kStages;
         if (!mbar_wait(bar_kfull + 8 * s, ((j - f_min) / kStages) & 1, abort_flag, status, 42)) return false;
         tc_fence_after();
+        uint64_t q = dQ + t * (L::kTileBytes / 16), k = dK + s * (L::kTileBytes / 16);
+        asm volatile("" : "+l"(q), "+l"(k));                  // keeps the sums below from being formed ahead of the loop and spilled
 #pragma unroll
         for (int ks = 0; ks < (D + DR) / 16; ++ks) {
           if (RULE && ks < D / 16 && ks * 16 >= p.dk) continue;            // the rest of the columns is zero
           if (DR > 0 && ks >= D / 16 && (ks - D / 16) * 16 >= p.dr) continue;
-          const uint32_t off = (ks >> 2) * L::kHalf + (ks & 3) * 32;
-          umma_bf16_ss(tmem_base + t * 128, umma_smem_desc_sw128(sQ + t * L::kTileBytes + off, 16, 1024),
-                       umma_smem_desc_sw128(sK + s * L::kTileBytes + off, 16, 1024), idesc_qk, ks != 0 ? 1u : 0u);
+          const uint64_t off = (ks >> 2) * (L::kHalf / 16) + (ks & 3) * 2;
+          umma_bf16_ss(tmem_base + t * 128, q + off, k + off, idesc_qk, ks != 0 ? 1u : 0u);
         }
         umma_commit(bar_sfull + 8 * t);
         return true;
@@ -367,11 +371,12 @@ attn_fwd2_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
           tc_fence_after();
           const uint32_t tmem_p = tmem_base + t * 128;              // packed bf16 pairs: 8 columns per 16 keys
           const uint32_t tmem_o = tmem_base + 256 + t * 128;
+          uint64_t dv = dV + v * (L::kVTileBytes / 16);
+          asm volatile("" : "+l"(dv));
 #pragma unroll
           for (int ks = 0; ks < kF2Tile / 16; ++ks) {
             // V: 16 key rows of 128 B per step; 64-wide head-dim atoms L::kHalf apart
-            const uint64_t db = umma_smem_desc_sw128(sV + v * L::kVTileBytes + ks * 2048, L::kHalf, 1024);
-            umma_bf16_ts(tmem_o, tmem_p + ks * 8, db, idesc_pv, (j > f_of(t) || ks != 0) ? 1u : 0u);
+            umma_bf16_ts(tmem_o, tmem_p + ks * 8, dv + ks * (2048 / 16), idesc_pv, (j > f_of(t) || ks != 0) ? 1u : 0u);
           }
           umma_commit(bar_oready + 8 * t);
           if (j + 1 < n_of(t)) ok = issue_qk(j + 1, t);          // overwrites S_t / P_t: ordered behind PV(j, t)

@@ -170,6 +170,16 @@ head_product_kernel(const RbHeadProductArgs a) {
 #pragma unroll
   for (int i = 0; i < S::kStages - 1; ++i) request(i);
   const bool active = r0 + warp * 16 < a.rows;
+  const int g = lane >> 2, tq = lane & 3;
+  const __nv_bfloat16* G = a.gate ? reinterpret_cast<const __nv_bfloat16*>(a.gate) + static_cast<long long>(h) * a.n : nullptr;
+  uint32_t gates[BN / 8][2];                             // requested under the first slices
+#pragma unroll
+  for (int nt = 0; nt < BN / 8; ++nt)
+#pragma unroll
+    for (int half = 0; half < 2; ++half) {
+      const int n = n0 + nt * 8 + 2 * tq, r = r0 + warp * 16 + g + 8 * half;
+      gates[nt][half] = G && n < a.n && r < a.rows ? *reinterpret_cast<const uint32_t*>(G + r * a.ld_g + n) : 0u;
+    }
   for (int st = 0; st < steps; ++st) {
     wm_cp_wait<S::kStages - 2>();
     __syncthreads();                                     // slice st has landed for everyone, slice st - 1 is no longer read
@@ -190,9 +200,7 @@ head_product_kernel(const RbHeadProductArgs a) {
       }
     }
   }
-  const int g = lane >> 2, tq = lane & 3;
   __nv_bfloat16* Y = reinterpret_cast<__nv_bfloat16*>(a.y) + h * a.y_head;
-  const __nv_bfloat16* G = a.gate ? reinterpret_cast<const __nv_bfloat16*>(a.gate) + static_cast<long long>(h) * a.n : nullptr;
 #pragma unroll
   for (int nt = 0; nt < BN / 8; ++nt) {
     const int n = n0 + nt * 8 + 2 * tq;
@@ -203,7 +211,7 @@ head_product_kernel(const RbHeadProductArgs a) {
       if (r >= a.rows) continue;
       float u = acc[nt][2 * half], v = acc[nt][2 * half + 1];
       if (G) {
-        const float2 z = unpack_bf16x2(*reinterpret_cast<const uint32_t*>(G + r * a.ld_g + n));
+        const float2 z = unpack_bf16x2(gates[nt][half]);
         u = __fdividef(u, 1.f + __expf(-z.x));
         v = __fdividef(v, 1.f + __expf(-z.y));
       }
@@ -510,28 +518,37 @@ latent_decode_kernel(const RbLatentDecodeArgs a, int nsplit RB_BOUNDS_PARAM) {
     }
 }
 
-// out[b, h, :] = merge over the slices that hold tokens of sequence b; a thread owns two columns
+// out[b, h, :] = merge over the slices that hold tokens of sequence b (at most 64); a thread owns two columns
 __global__ void __launch_bounds__(256)
 latent_merge_kernel(const float* __restrict__ partial, const int* __restrict__ context_lens, int heads, int rank, int nsplit,
                     __nv_bfloat16* __restrict__ out, long long ld_o) {
-  const int h = blockIdx.x, b = blockIdx.y;
+  const int h = blockIdx.x, b = blockIdx.y, lane = threadIdx.x & 31;
   const int ctx = context_lens[b], slice = latent_chunk(ctx, nsplit);
   const int n = min(nsplit, (ctx + slice - 1) / slice);
-  const float* base = partial + (static_cast<long long>(b) * heads + h) * nsplit * (rank + 2);
-  float mx = -INFINITY;
-  for (int s = 0; s < n; ++s) mx = fmaxf(mx, base[static_cast<long long>(s) * (rank + 2)]);
-  for (int c = 2 * threadIdx.x; c < rank; c += 2 * blockDim.x) {
-    float u = 0.f, v = 0.f, den = 0.f;
+  const long long pitch = rank + 2;
+  const float* base = partial + (static_cast<long long>(b) * heads + h) * nsplit * pitch;
+  // every warp by itself: lane s has the factors of slices s and s + 32
+  const float m0 = lane < n ? base[lane * pitch] : -INFINITY, m1 = lane + 32 < n ? base[(lane + 32) * pitch] : -INFINITY;
+  const float l0 = lane < n ? base[lane * pitch + 1] : 0.f, l1 = lane + 32 < n ? base[(lane + 32) * pitch + 1] : 0.f;
+  const float mx = warp_max(fmaxf(m0, m1));
+  float s0 = wm_ex2(m0 - mx), s1 = wm_ex2(m1 - mx);
+  const float den = warp_sum(fmaf(l0, s0, l1 * s1));
+  const float inv = den > 0.f ? 1.f / den : 0.f;
+  s0 *= inv;
+  s1 *= inv;
+  for (int c0 = 0; c0 < rank; c0 += 2 * blockDim.x) {
+    const int c = c0 + 2 * threadIdx.x;
+    float u = 0.f, v = 0.f;
+#pragma unroll 4
     for (int s = 0; s < n; ++s) {
-      const float* p = base + static_cast<long long>(s) * (rank + 2);
-      const float sc = wm_ex2(p[0] - mx);
-      const float2 z = *reinterpret_cast<const float2*>(p + 2 + c);
-      den = fmaf(p[1], sc, den);
-      u = fmaf(z.x, sc, u);
-      v = fmaf(z.y, sc, v);
+      const float sc = __shfl_sync(0xffffffffu, s < 32 ? s0 : s1, s & 31);
+      if (c < rank) {
+        const float2 z = *reinterpret_cast<const float2*>(base + s * pitch + 2 + c);
+        u = fmaf(z.x, sc, u);
+        v = fmaf(z.y, sc, v);
+      }
     }
-    const float inv = den > 0.f ? 1.f / den : 0.f;
-    *reinterpret_cast<uint32_t*>(out + b * ld_o + static_cast<long long>(h) * rank + c) = pack_bf16x2(u * inv, v * inv);
+    if (c < rank) *reinterpret_cast<uint32_t*>(out + b * ld_o + static_cast<long long>(h) * rank + c) = pack_bf16x2(u, v);
   }
 }
 

@@ -1,15 +1,20 @@
 // Latent attention, decoding, on the 5th-generation tensor cores (rb_latent_decode for the sizes below; latent_attention.cu has the
 // interface and the form for all others).
 //
-// One CTA = (16 or 32 heads, slice of the context, sequence).  128 cached tokens at a time are the M of both products, the heads the N:
+// One CTA = (16 or 32 heads, slice of the context, sequence).  Tiles of 64 cached tokens; the M of the products are cached rows, then
+// columns of the cached vectors, the N are heads:
 //     S^T [tokens, heads]  = C [tokens, rank + rot] Q^T        A: cached rows as they lie, K-major
 //     O^T [rank, heads]   += C^T [rank, tokens] P^T            A: the same bytes, MN-major
 // so a tile's shared memory is filled once by TMA, page by page, and no thread ever touches it.  S^T and O^T live in TMEM.
-// The columns of the cached vectors come in pieces of 128 through a ring of five; a piece is released as soon as its product with P is
-// done, so the next tile streams in while this one is worked off.
-// Softmax (warps 0-3, one token per thread): a head's maximum over the tokens by a transposing butterfly in every warp and one exchange
-// between the warps; sums are kept per thread until the end.  O is rescaled only when a maximum has grown by more than 2^8.
-// Warp 4 issues the copies, warp 5 the products.
+// Products this narrow cost the same whatever their N and whether M is 64 or 128.  So a product of the scores takes two blocks of 64
+// columns at once: its A has the tokens' first block in rows 0 - 63 and their second block in rows 64 - 127 (the order in which they lie
+// in shared memory anyway), its B both blocks of the queries; the two diagonal quarters of the result, added, are the scores.
+// The columns come in pieces of 128 through a ring that holds 2.5 tiles of the widest vectors; a piece is released as soon as its product
+// with P is done, and whichever of the next scores and the next sum is ready first is issued first.
+// Softmax (warps 0-3): warps 2 and 3 hand their quarter of the scores over, a thread of warps 0 and 1 has a token.  A head's maximum over
+// the tokens comes by a transposing butterfly in either warp and one exchange between them; sums are kept per thread until the end.  O is
+// rescaled only when a maximum has grown by more than 2^8, by all four warps.
+// Warps 4-7 issue the copies (a page each), warp 8 the products.
 #include "latent_attention.h"
 
 #include "rb_common.cuh"
@@ -17,8 +22,8 @@
 
 namespace rb {
 
-constexpr int kLtThreads = 192, kLtTile = 128, kLtRing = 5;
-constexpr int kLtAtom = kLtTile * 128;               // 64 columns of 128 tokens
+constexpr int kLtThreads = 288, kLtTile = 64, kLtCopyWarps = 4;
+constexpr int kLtAtom = kLtTile * 128;               // 64 columns of a tile
 constexpr int kLtPiece = 2 * kLtAtom;
 
 struct LtParams {
@@ -36,7 +41,8 @@ __device__ __forceinline__ float lt_ex2(float x) {
   asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
   return y;
 }
-__device__ __forceinline__ void lt_sync_softmax() { asm volatile("bar.sync 1, 128;" ::: "memory"); }
+__device__ __forceinline__ void lt_sync_four() { asm volatile("bar.sync 1, 128;" ::: "memory"); }     // warps 0-3
+__device__ __forceinline__ void lt_sync_two() { asm volatile("bar.sync 2, 64;" ::: "memory"); }       // warps 0, 1
 
 template <int N>
 __device__ __forceinline__ void lt_ld(uint32_t taddr, uint32_t (&r)[N]) {
@@ -79,13 +85,15 @@ __device__ __forceinline__ float lt_reduce(const float (&v)[N]) {
 
 template <int N, int RP>
 struct LtSmem {
+  static constexpr int kSlots = N == 16 ? 11 : 10;
   static constexpr int kRing = 0;
-  static constexpr int kRot = kRing + kLtRing * kLtPiece;             // rotated parts of a tile
-  static constexpr int kQ = kRot + kLtAtom;                           // 2 RP + 1 pieces of 64 columns, N rows
-  static constexpr int kP = kQ + (2 * RP + 1) * N * 128;              // 2 pieces of 64 tokens, N rows
-  static constexpr int kRed = kP + 2 * N * 128;                       // [2][4][N] maxima, [4][2 N] maxima and factors of each warp
-  static constexpr int kBar = kRed + (8 + 8) * N * 4;
-  static constexpr int kNumBars = 2 * kLtRing + 7;                    // q, full / empty per slot, rot full / empty, s[2], p, o
+  static constexpr int kRot = kRing + kSlots * kLtPiece;              // rotated parts of two tiles
+  static constexpr int kQ = kRot + 2 * kLtAtom;                       // 2 RP + 1 pieces of 64 columns, N rows
+  static constexpr int kP = kQ + (2 * RP + 1) * N * 128;              // N rows of 64 tokens
+  static constexpr int kHand = kP + N * 128;                          // [N][64] scores that warps 2 and 3 hand over
+  static constexpr int kRed = kHand + N * 64 * 4;                     // [2][2][N] maxima of warps 0 and 1, [N] maxima, [N] factors, a flag
+  static constexpr int kBar = kRed + 6 * N * 4 + 16;
+  static constexpr int kNumBars = 2 * kSlots + 9;                     // q, full / empty per slot, rot full[2] / empty[2], s[2], p, o
   static constexpr int kTotal = kBar + kNumBars * 8 + 16;
 };
 
@@ -99,12 +107,16 @@ latent_decode_tc_kernel(const __grid_constant__ CUtensorMap tmC, const __grid_co
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(lt_raw) + 1023) & ~uintptr_t(1023));
   const uint32_t sbase = smem_u32(smem);
   const uint32_t sRing = sbase + L::kRing, sRot = sbase + L::kRot, sQ = sbase + L::kQ, sP = sbase + L::kP;
+  float* hand = reinterpret_cast<float*>(smem + L::kHand);
   float* red = reinterpret_cast<float*>(smem + L::kRed);
+  float* m_sh = red + 4 * N;
+  float* f_sh = red + 5 * N;
+  volatile int* any_sh = reinterpret_cast<volatile int*>(red + 6 * N);
   uint64_t* bars = reinterpret_cast<uint64_t*>(smem + L::kBar);
   const uint32_t bar_q = smem_u32(bars);
-  const uint32_t bar_full = bar_q + 8, bar_empty = bar_full + 8 * kLtRing;
-  const uint32_t bar_rfull = bar_empty + 8 * kLtRing, bar_rempty = bar_rfull + 8;
-  const uint32_t bar_s = bar_rempty + 8, bar_p = bar_s + 16, bar_o = bar_p + 8;
+  const uint32_t bar_full = bar_q + 8, bar_empty = bar_full + 8 * L::kSlots;
+  const uint32_t bar_rfull = bar_empty + 8 * L::kSlots, bar_rempty = bar_rfull + 16;
+  const uint32_t bar_s = bar_rempty + 16, bar_p = bar_s + 16, bar_o = bar_p + 8;
   uint32_t* tmem_ptr = reinterpret_cast<uint32_t*>(bars + L::kNumBars);
   volatile int* abort_flag = reinterpret_cast<volatile int*>(tmem_ptr + 1);
 
@@ -117,18 +129,36 @@ latent_decode_tc_kernel(const __grid_constant__ CUtensorMap tmC, const __grid_co
   const int t_end = min(ctx, t_begin + chunk);
   const int tiles = (t_end - t_begin + kLtTile - 1) / kLtTile;
   const int nheads = min(N, p.heads - h0);
-  constexpr uint32_t kTmemCols = (RP + 2) * N <= 64 ? 64 : (RP + 2) * N <= 128 ? 128 : 256;
+  constexpr int kO = 4 * N;                            // TMEM: both score accumulators (2 N columns each), then RP pieces of O^T
+  constexpr uint32_t kTmemCols = kO + RP * N <= 128 ? 128 : 256;
+
+  // copies: first cache row of page `k` of tile j (-1: past the end)
+  auto page_row = [&](int j, int k) {
+    const int tok = t_begin + j * kLtTile + k * p.block_size;
+    if (j >= tiles || k * p.block_size >= kLtTile || tok >= t_end) return -1;
+    const int bi = tok / p.block_size;
+    int blk = bi < p.max_blocks ? p.block_tables[static_cast<long long>(b) * p.max_blocks + bi] : -1;
+    if (blk < 0 || blk >= p.num_blocks) {              // corrupt tables read block 0 instead of faulting
+      RB_BOUNDS_HIT(104);
+      blk = 0;
+    }
+    return blk * p.block_size;
+  };
+  const int k0 = warp - 4, k1 = k0 + kLtCopyWarps;     // pages of a tile that a copying warp takes (eight with pages of 8 tokens)
+  int row0 = -1, row1 = -1;
+  if (warp >= 4 && warp < 8) { row0 = page_row(0, k0); row1 = page_row(0, k1); }
 
   if (threadIdx.x == 0) {
     mbar_init(bar_q, 1);
-    for (int s = 0; s < kLtRing; ++s) {
-      mbar_init(bar_full + 8 * s, 1);
+    for (int s = 0; s < L::kSlots; ++s) {
+      mbar_init(bar_full + 8 * s, kLtCopyWarps);
       mbar_init(bar_empty + 8 * s, 1);
     }
-    mbar_init(bar_rfull, 1);
-    mbar_init(bar_rempty, 1);
-    mbar_init(bar_s, 1);
-    mbar_init(bar_s + 8, 1);
+    for (int s = 0; s < 2; ++s) {
+      mbar_init(bar_rfull + 8 * s, kLtCopyWarps);
+      mbar_init(bar_rempty + 8 * s, 1);
+      mbar_init(bar_s + 8 * s, 1);
+    }
     mbar_init(bar_p, 4);
     mbar_init(bar_o, 1);
     *abort_flag = 0;
@@ -138,221 +168,254 @@ latent_decode_tc_kernel(const __grid_constant__ CUtensorMap tmC, const __grid_co
     tma_prefetch_desc(&tmQ);
     tma_prefetch_desc(&tmQr);
   }
-  if (warp == 5) {
+  if (warp == 8) {
     tmem_alloc(smem_u32(tmem_ptr), kTmemCols);
     tmem_relinquish();
   }
   tc_fence_before();
   __syncthreads();
   tc_fence_after();
-  const uint32_t tmem = *tmem_ptr;                     // S^T in columns [0, 2N), then RP pieces of O^T
+  const uint32_t tmem = *tmem_ptr;
 
-  if (warp == 4) {
-    // ---------------------------------------------------------------- copies: a lane per page of the tile
-    if (lane == 0) {
+  if (warp == 8) {
+    // ---------------------------------------------------------------- products: one elected lane
+    if (elect_one()) {
       mbar_arrive_expect_tx(bar_q, (2 * RP + 1) * N * 128);
 #pragma unroll
       for (int i = 0; i < 2 * RP; ++i) tma_load_4d(sQ + i * N * 128, &tmQ, i * 64, h0, b, 0, bar_q);
       tma_load_4d(sQ + 2 * RP * N * 128, &tmQr, 0, h0, b, 0, bar_q);
-    }
-    __syncwarp();
-    const int per = kLtTile / p.block_size;            // pages per tile
-    const int* table = p.block_tables + static_cast<long long>(b) * p.max_blocks;
-    auto page_row = [&](int j) {                       // first cache row of this lane's page of tile j (-1: past the end)
-      const int tok = t_begin + j * kLtTile + lane * p.block_size;
-      if (lane >= per || tok >= t_end) return -1;
-      const int bi = tok / p.block_size;
-      int blk = bi < p.max_blocks ? table[bi] : -1;
-      if (blk < 0 || blk >= p.num_blocks) {            // corrupt tables read block 0 instead of faulting
-        RB_BOUNDS_HIT(104);
-        blk = 0;
-      }
-      return blk * p.block_size;
-    };
-    int row = page_row(0);
-    bool ok = true;
-    for (int j = 0; j < tiles && ok; ++j) {
-      const int next = j + 1 < tiles ? page_row(j + 1) : -1;
-      const int pages = __popc(__ballot_sync(0xffffffffu, row >= 0));
-      const uint32_t bytes = pages * p.block_size * 128;
-      const uint32_t dst = lane * p.block_size * 128;
-      for (int i = 0; i < RP && ok; ++i) {
-        const int c = j * RP + i, s = c % kLtRing;
-        ok = mbar_wait(bar_empty + 8 * s, ((c / kLtRing) & 1) ^ 1, abort_flag, status, 61);
-        ok = __all_sync(0xffffffffu, ok);
-        if (!ok) break;
-        if (lane == 0) mbar_arrive_expect_tx(bar_full + 8 * s, 2 * bytes);
-        __syncwarp();
-        if (row >= 0) {
-          tma_load_4d(sRing + s * kLtPiece + dst, &tmC, i * 128, row, 0, 0, bar_full + 8 * s);
-          tma_load_4d(sRing + s * kLtPiece + kLtAtom + dst, &tmC, i * 128 + 64, row, 0, 0, bar_full + 8 * s);
-        }
-      }
-      if (!ok) break;
-      ok = mbar_wait(bar_rempty, (j & 1) ^ 1, abort_flag, status, 62);
-      ok = __all_sync(0xffffffffu, ok);
-      if (!ok) break;
-      if (lane == 0) mbar_arrive_expect_tx(bar_rfull, bytes);
-      __syncwarp();
-      if (row >= 0) tma_load_4d(sRot + dst, &tmCr, 0, row, 0, 0, bar_rfull);
-      row = next;
-    }
-  } else if (warp == 5) {
-    if (lane == 0) {
-      // ---------------------------------------------------------------- products
-      constexpr uint32_t idesc_s = umma_idesc_bf16(128, N, 0, 0);
+      constexpr uint32_t idesc_s = umma_idesc_bf16(128, 2 * N, 0, 0);
+      constexpr uint32_t idesc_r = umma_idesc_bf16(128, N, 0, 0);
       constexpr uint32_t idesc_o = umma_idesc_bf16(128, N, 1, 0);
-      auto scores = [&](int j) -> bool {               // S^T of tile j
-        const uint32_t d = tmem + (j & 1) * N;
-        for (int i = 0; i < RP; ++i) {
-          const int c = j * RP + i, s = c % kLtRing;
-          if (!mbar_wait(bar_full + 8 * s, (c / kLtRing) & 1, abort_flag, status, 63)) return false;
+      // descriptors of the first piece; an offset of o bytes is o / 16 in the address field
+      constexpr uint64_t kPiece = kLtPiece / 16, kAtom = kLtAtom / 16, kRows = 2048 / 16, kHeads = N * 128 / 16;
+      const uint64_t dC = umma_smem_desc_sw128(sRing, 16, 1024), dCt = umma_smem_desc_sw128(sRing, kLtAtom, 1024);
+      const uint64_t dR = umma_smem_desc_sw128(sRot, 16, 1024), dQ = umma_smem_desc_sw128(sQ, 16, 1024), dP = umma_smem_desc_sw128(sP, 16, 1024);
+      int sj = 0, ss = 0, sphase = 0;                  // next scores: tile, slot and phase of its next piece
+      int si = 0;                                      // that piece (RP: the rotated part)
+      int os = 0;                                      // slot of the first piece of the next sum
+      bool ok = mbar_wait(bar_q, 0, abort_flag, status, 63);
+      // Scores as far as their operands are there, `all`: until tile sj is through (a tile has to come).
+      auto scores = [&](bool all) {
+        const uint32_t d = tmem + (sj & 1) * 2 * N;
+        while (si < RP) {
+          if (all ? !mbar_wait(bar_full + 8 * ss, sphase, abort_flag, status, 64) : !mbar_test(bar_full + 8 * ss, sphase)) return !all;
           tc_fence_after();
+          const uint64_t da = dC + ss * kPiece, dq = dQ + 2 * si * kHeads;
 #pragma unroll
-          for (int ks = 0; ks < 8; ++ks) {
-            const uint32_t a = sRing + s * kLtPiece + (ks >> 2) * kLtAtom + (ks & 3) * 32;
-            const uint32_t q = sQ + (2 * i + (ks >> 2)) * N * 128 + (ks & 3) * 32;
-            umma_bf16_ss(d, umma_smem_desc_sw128(a, 16, 1024), umma_smem_desc_sw128(q, 16, 1024), idesc_s, (i | ks) != 0);
-          }
+          for (int ks = 0; ks < 4; ++ks) umma_bf16_ss(d, da + ks * 2, dq + ks * 2, idesc_s, (si | ks) != 0);
+          ++si;
+          if (++ss == L::kSlots) { ss = 0; sphase ^= 1; }
         }
-        if (!mbar_wait(bar_rfull, j & 1, abort_flag, status, 64)) return false;
+        if (all ? !mbar_wait(bar_rfull + 8 * (sj & 1), (sj >> 1) & 1, abort_flag, status, 68)
+                : !mbar_test(bar_rfull + 8 * (sj & 1), (sj >> 1) & 1))
+          return !all;
         tc_fence_after();
+        // rows 64 - 127 of this A are whatever lies behind: they end up where nobody looks
 #pragma unroll
-        for (int ks = 0; ks < 4; ++ks)
-          umma_bf16_ss(d, umma_smem_desc_sw128(sRot + ks * 32, 16, 1024), umma_smem_desc_sw128(sQ + 2 * RP * N * 128 + ks * 32, 16, 1024),
-                       idesc_s, 1u);
-        umma_commit(bar_rempty);
-        umma_commit(bar_s + 8 * (j & 1));
+        for (int ks = 0; ks < 4; ++ks) umma_bf16_ss(d, dR + (sj & 1) * kAtom + ks * 2, dQ + 2 * RP * kHeads + ks * 2, idesc_r, 1u);
+        umma_commit(bar_rempty + 8 * (sj & 1));
+        umma_commit(bar_s + 8 * (sj & 1));
+        ++sj;
+        si = 0;
         return true;
       };
-      constexpr bool kAhead = 2 * RP <= kLtRing;       // two tiles fit the ring: the next scores are issued before this tile's sum
-      bool ok = mbar_wait(bar_q, 0, abort_flag, status, 65);
-      if (ok && kAhead) ok = scores(0);
-      for (int j = 0; j < tiles && ok; ++j) {
-        if (kAhead ? j + 1 < tiles : true) ok = scores(kAhead ? j + 1 : j);
-        if (!ok || !mbar_wait(bar_p, j & 1, abort_flag, status, 66)) break;
+      for (int oj = 0; oj < tiles && ok; ++oj) {
+        if (sj <= oj) ok = scores(true);
+        // S^T of tile oj + 1 goes where that of oj - 1 was, read when P of oj - 1 came
+        while (ok && sj == oj + 1 && sj < tiles && !mbar_test(bar_p, oj & 1)) {
+          const int before = si;
+          ok = scores(false);
+          if (sj == oj + 1 && si == before) break;     // the operand is not there yet: P is more likely to come first
+        }
+        if (!ok || !mbar_wait(bar_p, oj & 1, abort_flag, status, 69)) break;
         tc_fence_after();
-        for (int i = 0; i < RP; ++i) {
-          const int s = (j * RP + i) % kLtRing;
 #pragma unroll
-          for (int ks = 0; ks < 8; ++ks)
-            umma_bf16_ss(tmem + (2 + i) * N, umma_smem_desc_sw128(sRing + s * kLtPiece + ks * 2048, kLtAtom, 1024),
-                         umma_smem_desc_sw128(sP + (ks >> 2) * N * 128 + (ks & 3) * 32, 16, 1024), idesc_o, (j | ks) != 0);
-          umma_commit(bar_empty + 8 * s);
+        for (int ks = 0; ks < kLtTile / 16; ++ks) {
+          int s = os;
+#pragma unroll
+          for (int i = 0; i < RP; ++i) {
+            umma_bf16_ss(tmem + kO + i * N, dCt + s * kPiece + ks * kRows, dP + ks * 2, idesc_o, (oj | ks) != 0);
+            s = s + 1 == L::kSlots ? 0 : s + 1;
+          }
+        }
+#pragma unroll
+        for (int i = 0; i < RP; ++i) {
+          umma_commit(bar_empty + 8 * os);
+          os = os + 1 == L::kSlots ? 0 : os + 1;
         }
         umma_commit(bar_o);
       }
     }
+    __syncwarp();
+  } else if (warp >= 4) {
+    // ---------------------------------------------------------------- copies
+    const uint32_t page = p.block_size * 128, to0 = k0 * page, to1 = k1 * page;
+    int s = 0, phase = 1;
+    bool ok = true;
+    for (int j = 0; j < tiles && ok; ++j) {
+      const int next0 = page_row(j + 1, k0), next1 = page_row(j + 1, k1);
+      const uint32_t bytes = ((row0 >= 0) + (row1 >= 0)) * page;
+      for (int i = 0; i < RP; ++i) {
+        ok = mbar_wait(bar_empty + 8 * s, phase, abort_flag, status, 61);
+        ok = __all_sync(0xffffffffu, ok);
+        if (!ok) break;
+        if (elect_one()) {
+          const uint32_t dst = sRing + s * kLtPiece, bar = bar_full + 8 * s;
+          mbar_arrive_expect_tx(bar, 2 * bytes);
+          if (row0 >= 0) {
+            tma_load_4d(dst + to0, &tmC, i * 128, row0, 0, 0, bar);
+            tma_load_4d(dst + kLtAtom + to0, &tmC, i * 128 + 64, row0, 0, 0, bar);
+          }
+          if (row1 >= 0) {
+            tma_load_4d(dst + to1, &tmC, i * 128, row1, 0, 0, bar);
+            tma_load_4d(dst + kLtAtom + to1, &tmC, i * 128 + 64, row1, 0, 0, bar);
+          }
+        }
+        __syncwarp();
+        if (++s == L::kSlots) { s = 0; phase ^= 1; }
+      }
+      if (!ok) break;
+      ok = mbar_wait(bar_rempty + 8 * (j & 1), ((j >> 1) & 1) ^ 1, abort_flag, status, 62);
+      ok = __all_sync(0xffffffffu, ok);
+      if (!ok) break;
+      if (elect_one()) {
+        const uint32_t dst = sRot + (j & 1) * kLtAtom, bar = bar_rfull + 8 * (j & 1);
+        mbar_arrive_expect_tx(bar, bytes);
+        if (row0 >= 0) tma_load_4d(dst + to0, &tmCr, 0, row0, 0, 0, bar);
+        if (row1 >= 0) tma_load_4d(dst + to1, &tmCr, 0, row1, 0, 0, bar);
+      }
+      __syncwarp();
+      row0 = next0;
+      row1 = next1;
+    }
   } else {
-    // ------------------------------------------------------------------ softmax, one token per thread.  After a wait that gave up the
-    // loop runs on without waiting, so that all four warps keep meeting at the named barrier.
+    // ------------------------------------------------------------------ softmax.  After a wait that gave up the loop runs on without
+    // waiting, so that the warps keep meeting at the named barriers.
     const uint32_t lane_off = static_cast<uint32_t>(warp * 32) << 16;
     const float sl2 = p.scale * 1.4426950408889634f;
-    float m_run = -INFINITY;                           // of head lane % N, the same in all warps
-    float l_part[N];                                   // of this thread's tokens
+    const bool owner = warp < 2;                       // has a token per thread
+    const int tok = (warp & 1) * 32 + lane;
+    float m_run = -INFINITY;                           // owners: of head lane % N, the same in both warps
+    float l_part[N];                                   // owners: of this thread's tokens
 #pragma unroll
     for (int h = 0; h < N; ++h) l_part[h] = 0.f;
-    float* mine = red + 8 * N + warp * 2 * N;          // maxima and factors for this warp's lanes to read
     bool ok = true;
     for (int j = 0; j < tiles; ++j) {
-      if (ok) ok = mbar_wait(bar_s + 8 * (j & 1), (j >> 1) & 1, abort_flag, status, 67);
+      if (ok) ok = mbar_wait(bar_s + 8 * (j & 1), (j >> 1) & 1, abort_flag, status, 65);
+      __syncwarp();
       tc_fence_after();
-      const int valid = t_end - t_begin - j * kLtTile;
-      const bool live = static_cast<int>(threadIdx.x) < valid;
       uint32_t raw[N];
-      lt_ld<N>(tmem + (j & 1) * N + lane_off, raw);
+      lt_ld<N>(tmem + (j & 1) * 2 * N + (owner ? 0 : N) + lane_off, raw);
       tmem_ld_wait();
-      float x[N];
+      if (!owner) {
 #pragma unroll
-      for (int h = 0; h < N; ++h) x[h] = live ? __uint_as_float(raw[h]) * sl2 : -INFINITY;
-      float mx = lt_reduce<N, true>(x);
-      float* r = red + (j & 1) * 4 * N;
-      if (lane < N) r[warp * N + lane] = mx;
-      lt_sync_softmax();
-      mx = fmaxf(fmaxf(r[lane % N], r[N + lane % N]), fmaxf(r[2 * N + lane % N], r[3 * N + lane % N]));
-      const bool grow = mx > m_run + 8.f;              // also when there is no maximum yet
-      const float m_new = grow ? mx : m_run;
-      const float factor = grow ? lt_ex2(m_run - m_new) : 1.f;
-      m_run = m_new;
-      __syncwarp();
-      if (lane < N) { mine[lane] = m_new; mine[N + lane] = factor; }
-      __syncwarp();
-      const bool any = __any_sync(0xffffffffu, grow);
+        for (int h = 0; h < N; ++h) hand[h * kLtTile + tok] = __uint_as_float(raw[h]);
+      }
+      lt_sync_four();                                  // both halves of the scores are there
+      float x[N];
+      const bool live = tok < t_end - t_begin - j * kLtTile;
+      if (owner) {
+#pragma unroll
+        for (int h = 0; h < N; ++h) x[h] = live ? (__uint_as_float(raw[h]) + hand[h * kLtTile + tok]) * sl2 : -INFINITY;
+        float mx = lt_reduce<N, true>(x);
+        float* r = red + (j & 1) * 2 * N;
+        if (lane < N) r[warp * N + lane] = mx;
+        lt_sync_two();
+        mx = fmaxf(r[lane % N], r[N + lane % N]);
+        const bool grow = mx > m_run + 8.f;            // also when there is no maximum yet
+        const float m_new = grow ? mx : m_run;
+        const float factor = grow ? lt_ex2(m_run - m_new) : 1.f;
+        m_run = m_new;
+        const bool any = __any_sync(0xffffffffu, grow);
+        if (warp == 0) {
+          if (lane < N) { m_sh[lane] = m_new; f_sh[lane] = factor; }
+          if (lane == 0) *any_sh = any;
+        }
+      }
+      lt_sync_four();                                  // maxima and factors are there
+      const bool any = *any_sh;
       if (j > 0) {                                     // O holds tiles 0 .. j - 1, and P is free again
-        if (ok) ok = mbar_wait(bar_o, (j - 1) & 1, abort_flag, status, 68);
+        if (ok) ok = mbar_wait(bar_o, (j - 1) & 1, abort_flag, status, 66);
+        __syncwarp();
         tc_fence_after();
         if (any) {
 #pragma unroll 1
           for (int i = 0; i < RP; ++i) {
             uint32_t o[N];
-            lt_ld<N>(tmem + (2 + i) * N + lane_off, o);
+            lt_ld<N>(tmem + kO + i * N + lane_off, o);
             tmem_ld_wait();
 #pragma unroll
             for (int h = 0; h < N; h += 4) {
-              const float4 f = *reinterpret_cast<const float4*>(mine + N + h);
+              const float4 f = *reinterpret_cast<const float4*>(f_sh + h);
               o[h] = __float_as_uint(__uint_as_float(o[h]) * f.x);
               o[h + 1] = __float_as_uint(__uint_as_float(o[h + 1]) * f.y);
               o[h + 2] = __float_as_uint(__uint_as_float(o[h + 2]) * f.z);
               o[h + 3] = __float_as_uint(__uint_as_float(o[h + 3]) * f.w);
             }
-            lt_st<N>(tmem + (2 + i) * N + lane_off, o);
+            lt_st<N>(tmem + kO + i * N + lane_off, o);
           }
           tmem_st_wait();
 #pragma unroll
-          for (int h = 0; h < N; ++h) l_part[h] *= mine[N + h];
+          for (int h = 0; h < N; ++h) l_part[h] *= f_sh[h];
         }
       }
-      // P^T as the B operand: rows are heads, 64 tokens per swizzled 128-byte row
-      const int tok = threadIdx.x;
-      uint8_t* prow = smem + L::kP + (tok >> 6) * N * 128 + (tok & 7) * 2;
-      const int piece = (tok & 63) >> 3;
+      if (owner) {
+        // P^T as the B operand: rows are heads, 64 tokens per swizzled 128-byte row
+        uint8_t* prow = smem + L::kP + (tok & 7) * 2;
+        const int piece = tok >> 3;
 #pragma unroll
-      for (int h = 0; h < N; h += 4) {
-        const float4 m4 = *reinterpret_cast<const float4*>(mine + h);
-        const float ms[4] = {m4.x, m4.y, m4.z, m4.w};
+        for (int h = 0; h < N; h += 4) {
+          const float4 m4 = *reinterpret_cast<const float4*>(m_sh + h);
+          const float ms[4] = {m4.x, m4.y, m4.z, m4.w};
 #pragma unroll
-        for (int i = 0; i < 4; ++i) {
-          const float e = lt_ex2(x[h + i] - ms[i]);
-          l_part[h + i] += e;
-          *reinterpret_cast<__nv_bfloat16*>(prow + (h + i) * 128 + ((piece ^ ((h + i) & 7)) << 4)) = __float2bfloat16(e);
-        }
-      }
-      if (!live) {                                     // rows without a token hold what was there before: 0 times that must be 0
-        for (int i = 0; i < RP; ++i) {
-          uint4* z = reinterpret_cast<uint4*>(smem + L::kRing + (j * RP + i) % kLtRing * kLtPiece + tok * 128);
-#pragma unroll
-          for (int c = 0; c < 8; ++c) {
-            z[c] = make_uint4(0u, 0u, 0u, 0u);
-            z[kLtAtom / 16 + c] = make_uint4(0u, 0u, 0u, 0u);
+          for (int i = 0; i < 4; ++i) {
+            const float e = lt_ex2(x[h + i] - ms[i]);
+            l_part[h + i] += e;
+            *reinterpret_cast<__nv_bfloat16*>(prow + (h + i) * 128 + ((piece ^ ((h + i) & 7)) << 4)) = __float2bfloat16(e);
           }
         }
+        if (!live) {                                   // rows without a token hold what was there before: 0 times that must be 0
+          for (int i = 0; i < RP; ++i) {
+            uint4* z = reinterpret_cast<uint4*>(smem + L::kRing + (j * RP + i) % L::kSlots * kLtPiece + tok * 128);
+#pragma unroll
+            for (int c = 0; c < 8; ++c) {
+              z[c] = make_uint4(0u, 0u, 0u, 0u);
+              z[kLtAtom / 16 + c] = make_uint4(0u, 0u, 0u, 0u);
+            }
+          }
+        }
+        fence_proxy_async_smem();
       }
-      fence_proxy_async_smem();
       tc_fence_before();
       __syncwarp();
       if (lane == 0) mbar_arrive(bar_p);
     }
     // ---- sums over the tokens, then this slice's (maximum, sum, O) per head, or the result when there is one slice only
-    const float part = lt_reduce<N, false>(l_part);
-    lt_sync_softmax();                                 // nobody reads the last maxima any more
-    if (lane < N) red[warp * N + lane] = part;
-    if (ok) ok = mbar_wait(bar_o, (tiles - 1) & 1, abort_flag, status, 69);
-    tc_fence_after();
-    lt_sync_softmax();
-    const int hl = lane % N;
-    const float sum = red[hl] + red[N + hl] + red[2 * N + hl] + red[3 * N + hl];
-    if (warp == 0 && p.splits > 1 && lane < nheads) {
-      float* pp = p.scratch + ((static_cast<long long>(b) * p.heads + h0 + lane) * p.splits + sp) * (p.rank + 2);
-      pp[0] = m_run;
-      pp[1] = sum;
-    }
-    if (lane < N) mine[lane] = 1.f / sum;
+    if (ok) ok = mbar_wait(bar_o, (tiles - 1) & 1, abort_flag, status, 67);     // also: nobody reads the last factors any more
     __syncwarp();
+    tc_fence_after();
+    if (owner) {
+      const float part = lt_reduce<N, false>(l_part);
+      lt_sync_two();                                   // nobody reads the last maxima any more
+      if (lane < N) red[warp * N + lane] = part;
+      lt_sync_two();
+      const float sum = red[lane % N] + red[N + lane % N];
+      if (warp == 0 && lane < N) {
+        f_sh[lane] = 1.f / sum;
+        if (p.splits > 1 && lane < nheads) {
+          float* pp = p.scratch + ((static_cast<long long>(b) * p.heads + h0 + lane) * p.splits + sp) * (p.rank + 2);
+          pp[0] = m_run;
+          pp[1] = sum;
+        }
+      }
+    }
+    lt_sync_four();
 #pragma unroll 1
     for (int i = 0; i < RP; ++i) {
       uint32_t o[N];
       __syncwarp();
-      lt_ld<N>(tmem + (2 + i) * N + lane_off, o);
+      lt_ld<N>(tmem + kO + i * N + lane_off, o);
       tmem_ld_wait();
       const int col = i * 128 + warp * 32 + lane;
       if (col < p.rank && p.splits > 1) {
@@ -364,14 +427,14 @@ latent_decode_tc_kernel(const __grid_constant__ CUtensorMap tmC, const __grid_co
         __nv_bfloat16* op = p.out + b * p.ld_o + static_cast<long long>(h0) * p.rank + col;
 #pragma unroll
         for (int h = 0; h < N; ++h)
-          if (h < nheads) op[static_cast<long long>(h) * p.rank] = __float2bfloat16(__uint_as_float(o[h]) * mine[h]);
+          if (h < nheads) op[static_cast<long long>(h) * p.rank] = __float2bfloat16(__uint_as_float(o[h]) * f_sh[h]);
       }
     }
   }
 
   tc_fence_before();
   __syncthreads();
-  if (warp == 5) {
+  if (warp == 8) {
     if (*abort_flag) {
       // a wait gave up: let copies and products in flight land before the accumulators are released
       const unsigned long long t0 = globaltimer_ns();
@@ -404,7 +467,7 @@ int lt_launch(const RbLatentDecodeArgs& a, int splits, const CUtensorMap* const 
 // -9: not a problem for this kernel
 int latent_decode_tc(const RbLatentDecodeArgs& a, int splits, cudaStream_t s) {
   const int bs = a.block_size, W = a.rank + a.rot;
-  if (a.rot < 8 || a.rot > 64 || a.rank > 512 || (bs != 8 && bs != 16 && bs != 32 && bs != 64 && bs != 128) || (a.ld_q & 7) ||
+  if (a.rot < 8 || a.rot > 64 || a.rank > 512 || (bs != 8 && bs != 16 && bs != 32 && bs != 64) || (a.ld_q & 7) ||
       ((reinterpret_cast<uintptr_t>(a.q) | reinterpret_cast<uintptr_t>(a.cache)) & 15) || a.num_blocks * bs >= (1ll << 24))
     return -9;
   const int n = a.heads > 16 ? 32 : 16, rp = (a.rank + 127) / 128;

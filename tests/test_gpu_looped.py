@@ -212,6 +212,22 @@ def test_latent_decode_finds_one_key_that_stands_out(ctx, far):
     close(got.view(H, R)[3], s[far, :R], 2e-2)
 
 
+@pytest.mark.parametrize("ctx", [1, 17, 63, 64, 65, 130, 1000])
+@pytest.mark.parametrize("R,dr,bs", [(64, 32, 16), (512, 64, 16), (256, 32, 64), (128, 64, 4)])
+def test_latent_decode_does_not_read_what_a_page_held_before(ctx, R, dr, bs):
+    """Rows of the last page behind the context can hold anything, also what is not a number."""
+    H = 18
+    s, q = rnd(ctx, R + dr, seed=1).bfloat16().float(), rnd(H, R + dr, seed=2).bfloat16().float()
+    cache, t = paged_slots(s, bs, BF16)
+    used = torch.zeros(cache.shape[:2], dtype=torch.bool)
+    for j in range(ctx):
+        used[t[j // bs], j % bs] = True
+    cache[~used] = float("nan")
+    bt = torch.cat([t, torch.zeros(9, dtype=torch.int32)])[None]
+    got = latent_decode(dev(q.view(1, -1), BF16), dev(cache), R, dev(bt), torch.tensor([ctx], dtype=torch.int32, device="cuda"), 0.1)
+    close(got.view(H, R), latent_want(q, s, R, 0.1), 1e-2)
+
+
 def test_row_kernel_with_more_value_columns_than_one_block():
     R, dr, H = 1100, 16, 2
     s, q = rnd(40, R + dr).bfloat16().float(), rnd(H, R + dr, seed=1).bfloat16().float()
