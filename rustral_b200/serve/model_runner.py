@@ -65,9 +65,9 @@ class StepBatch:
         key = (i, first, kept)
         if key not in self._keys:
             r0, r1, start = self.spans[i]
-            t, bs = self.tables[i], self.block_size
-            self._keys[key] = torch.tensor([t[p // bs] * bs + p % bs for r in (range(kept), range(first, start + r1 - r0)) for p in r],
-                                           dtype=torch.int64, device=self.ids.device)
+            bs = self.block_size
+            pos = torch.cat([torch.arange(kept), torch.arange(first, start + r1 - r0)])
+            self._keys[key] = (torch.tensor(self.tables[i], dtype=torch.int64)[pos // bs] * bs + pos % bs).to(self.ids.device)
         return self._keys[key]
 
     def row_tables(self):
