@@ -56,7 +56,7 @@ CONFIGS = {
     "odd": model([win(6, 3, 20, 12, 24, 6, mlp=moe(20, 10, 3, (5, 3))), lat(3, 12, 6, 10, 20, 28, mlp=dense(44)), lat(2, 13, 4, 11, 9, 7, mlp=dense(50))],
                  (1, 2, 1), width=72),
     # no loop
-    "straight": model([lat(4, 32, 16, 32, 64, 40, mlp=moe(32, 12, 2, (4, 3), 1.0)), win(4, 1, 96, 96, 30, 24, mlp=dense(64))], width=96),
+    "straight": model([lat(4, 40, 16, 32, 72, 40, mlp=moe(32, 10, 3, (5, 2), 0.8)), win(4, 1, 104, 96, 30, 20, mlp=dense(64))], width=96),
 }
 
 
