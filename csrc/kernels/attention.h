@@ -39,6 +39,10 @@ typedef struct RbAttnRule {
   int rot_dim;
   const void* k_rot;
   long long ld_k_rot;
+  // fp32 [heads] each, or both NULL: s <- s - log_amount[h] * ln(1 + log_rate[h] * (i - j)), log_rate not negative (without rot_dim)
+  const float* log_amount;
+  const float* log_rate;
+  float out_scale;         // of the output
 } RbAttnRule;
 int rb_attention_fwd_rule(const RbAttnArgs* args, const RbAttnRule* rule, void* stream);
 int rb_attention_fwd(const RbAttnArgs* args, void* stream);

@@ -14,7 +14,7 @@
 // polynomial on the FMA pipe (template parameter; off by default, see rb_attention_fwd_tc2).  Warp 8 is the TMA producer (Q once, K / V through a ring of stages), warp 9 issues MMAs.
 //
 // The RULE form serves inference of decoders with their own score rule: separate key / value head sizes (columns beyond the
-// real sizes are zero-filled by TMA), capped scores, a linear distance bias, chunked or windowed visibility (key blocks before a
+// real sizes are zero-filled by TMA), capped scores, a linear or (LOG) a logarithmic distance bias, chunked or windowed visibility (key blocks before a
 // tile's first visible key are skipped, so the two tiles may start at different blocks), first keys that a window keeps (their
 // blocks are walked before the window's), a sink in the softmax and a sigmoid output gate per value column or per head.
 // With DR > 0 queries and keys have a second part whose keys all heads share (rotary positions of latent attention): it is one more
@@ -50,6 +50,9 @@ struct F2Params {
   long long ld_gate;
   int window, keep, sink;
   int dr;                   // DR > 0: real size of the second part
+  const float* log_amount;  // LOG: [heads] each
+  const float* log_rate;
+  float out_scale;
 };
 
 __device__ __forceinline__ float f2_ex2(float x) {
@@ -134,6 +137,46 @@ __device__ __forceinline__ void f2_cap_scores_wide(uint32_t (&r)[128], float c, 
     r[i] = __float_as_uint(fmaf(-2.f * cap2, f2_rcp(1.f + e), cap2 + fmaf(slope2, static_cast<float>(i), bias0)));
   }
 }
+// r <- mul * r - amount * log2(1 + rate * (dist0 - i)) for the columns i of one thread's row (scores in log2 units; distances below 0 are
+// masked afterwards).  With u = i - 63.5 the logarithm is log2(a) + log2(e) ln(1 - x), a = 1 + rate (dist0 - 63.5), x = rate u / a: where
+// |x| <= 1/8 for all columns (`far`, which the warp's first row decides for all) five terms of ln's series (largest error 8e-7) on packed
+// pairs do, otherwise one logarithm per score.
+__device__ __forceinline__ float f2_lg2(float x) {
+  float y;
+  asm("lg2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+__device__ __forceinline__ void f2_log_bias(uint32_t (&r)[128], float mul, float amount, float rate, float dist0, bool far) {
+  if (!far) {
+#pragma unroll
+    for (int i = 0; i < 128; ++i) {
+      const float t = f2_lg2(fmaf(rate, fmaxf(dist0 - static_cast<float>(i), 0.f), 1.f));
+      r[i] = __float_as_uint(fmaf(-amount, t, mul * __uint_as_float(r[i])));
+    }
+    return;
+  }
+  const float a = fmaf(rate, dist0 - 63.5f, 1.f), rho = rate * f2_rcp(a), base = -amount * f2_lg2(a), top = amount * kF2Log2e;
+  const uint64_t m = f2_pack(mul, mul), b = f2_pack(base, base), step = f2_pack(2.f * rho, 2.f * rho);
+  const uint64_t k1 = f2_pack(top, top), k2 = f2_pack(top / 2.f, top / 2.f), k3 = f2_pack(top / 3.f, top / 3.f), k4 = f2_pack(top / 4.f, top / 4.f),
+                 k5 = f2_pack(top / 5.f, top / 5.f);
+#pragma unroll
+  for (int g = 0; g < 4; ++g) {
+    uint64_t x = f2_pack(rho * (g * 32 - 63.5f), rho * (g * 32 - 62.5f));
+#pragma unroll
+    for (int i = 0; i < 16; ++i) {
+      uint32_t& r0 = r[g * 32 + 2 * i];
+      uint32_t& r1 = r[g * 32 + 2 * i + 1];
+      uint64_t p = f2_fma2(x, k5, k4);
+      p = f2_fma2(p, x, k3);
+      p = f2_fma2(p, x, k2);
+      p = f2_fma2(p, x, k1);
+      p = f2_fma2(p, x, b);
+      p = f2_fma2(f2_pack(__uint_as_float(r0), __uint_as_float(r1)), m, p);
+      x = f2_add2(x, step);
+      f2_unpack(p, r0, r1);
+    }
+  }
+}
 // 2^x on the FMA / integer pipes: round-to-nearest split x = n + f, |f| <= 0.5, degree-4 polynomial for 2^f
 // (relative error about 4e-5, well below bf16 rounding), exponent added to the bit pattern.  x must be >= -126.
 __device__ __forceinline__ float f2_ex2_poly(float x) {
@@ -194,7 +237,7 @@ struct F2Smem {
   static constexpr int kTotal = kBar + kNumBars * 8 + 16;
 };
 
-template <int D, int DV, int kPolyEvery, bool RULE, int DR = 0>
+template <int D, int DV, int kPolyEvery, bool RULE, int DR = 0, bool LOG = false>
 __global__ void __launch_bounds__(kF2Threads, 1)
 attn_fwd2_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK,
                  const __grid_constant__ CUtensorMap tmV, const __grid_constant__ CUtensorMap tmQr,
@@ -398,11 +441,12 @@ attn_fwd2_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
     const uint32_t tmem_s = tmem_base + t * 128 + lane_off;
     const uint32_t tmem_o = tmem_base + 256 + t * 128 + lane_off;
     // RULE: scores with a cap or a bias are turned into log2 units when they are read, so the softmax runs with scale 1
-    const bool shaped = RULE && (p.softcap > 0.f || p.slopes != nullptr);
+    const bool shaped = RULE && (LOG || p.softcap > 0.f || p.slopes != nullptr);
     const float sl2 = shaped ? 1.f : p.scale * kF2Log2e;
     const float rule_c1 = RULE && p.softcap > 0.f ? p.scale / p.softcap : 0.f;
     const float rule_c2 = RULE ? (p.softcap > 0.f ? p.softcap : p.scale) * kF2Log2e : 0.f;
     const float slope2 = RULE && p.slopes ? p.slopes[h] * kF2Log2e : 0.f;
+    const float log_amount = LOG ? p.log_amount[h] : 0.f, log_rate = LOG ? p.log_rate[h] : 0.f;
     // first visible key of this row, apart from the kept ones below key_keep
     const int key_lo = !RULE ? 0 : p.chunk > 0 ? (q_idx + shift) / p.chunk * p.chunk : p.window > 0 ? q_idx + shift - p.window + 1 : 0;
     const int key_keep = RULE && p.window > 0 ? p.keep : 0;
@@ -446,10 +490,15 @@ attn_fwd2_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
             tmem_ld_wait();
             f2_cap_scores_wide(r, rule_c1, rule_c2, slope2, bias0);
           }
-        } else if (shaped) {
+        } else if (LOG ? p.slopes != nullptr : shaped) {
 #pragma unroll
           for (int i = 0; i < 128; ++i)
             r[i] = __float_as_uint(fmaf(__uint_as_float(r[i]), rule_c2, fmaf(slope2, static_cast<float>(i), bias0)));
+        }
+        if (LOG) {
+          const float nearest = static_cast<float>(q_idx - lane + shift - k0) - 63.5f;       // of the warp's first row, to the middle key
+          f2_log_bias(r, p.softcap > 0.f || p.slopes != nullptr ? 1.f : rule_c2, log_amount, log_rate, static_cast<float>(q_idx + shift - k0),
+                      log_rate * 63.5f <= 0.125f * fmaf(log_rate, nearest, 1.f));
         }
         if (k0 < key_lo) {
 #pragma unroll
@@ -547,6 +596,7 @@ attn_fwd2_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
     if (ok && nt > 0) {
       tc_fence_after();
       float inv = l_run > 0.f ? 1.f / l_run : 0.f;
+      if (RULE) inv *= p.out_scale;
       if (RULE && p.head_gate != nullptr && q_idx < p.seq_q)
         inv *= f2_rcp(1.f + f2_ex2(-p.head_gate[q_idx * p.ld_gate + h] * kF2Log2e));
       __nv_bfloat16* op = p.out + b * p.o_bs + h * p.o_hs + static_cast<long long>(q_idx) * p.o_rs;
@@ -608,10 +658,10 @@ const CUtensorMap* f2_make_map(const void* base, const long long* strides, int s
   return rbhost::get_tmap_4d(base, 2, dims, str, box, 1, err);
 }
 
-template <int D, int DV, int P, bool RULE, int DR = 0>
+template <int D, int DV, int P, bool RULE, int DR = 0, bool LOG = false>
 int f2_launch(const CUtensorMap* tq, const CUtensorMap* tk, const CUtensorMap* tv, const rb::F2Params& p, dim3 grid,
               cudaStream_t stream, const CUtensorMap* tqr = nullptr, const CUtensorMap* tkr = nullptr) {
-  auto kern = rb::attn_fwd2_kernel<D, DV, P, RULE, DR>;
+  auto kern = rb::attn_fwd2_kernel<D, DV, P, RULE, DR, LOG>;
   const int smem = rb::F2Smem<D + DR, DV>::kTotal + 1024;
   static bool cfg_dev[64] = {false};
   bool& cfg = cfg_dev[rbhost::device_slot()];
@@ -679,7 +729,7 @@ RB_API int rb_attention_fwd_rule(const RbAttnArgs* a, const RbAttnRule* r, void*
   if (a->batch <= 0 || a->heads <= 0 || a->kv_heads <= 0 || a->heads % a->kv_heads) return -1;
   if (dk <= 0 || dv <= 0 || dk > 128 || dv > 128 || ((dk | dv) & 7)) return -9;
   if (!a->causal || a->seq_q <= 0 || a->seq_k < a->seq_q || r->chunk < 0 || r->window < 0 || r->keep_first < 0 || (r->window && r->chunk) ||
-      ((r->gate || r->head_gate) && a->batch != 1) || (r->gate && r->head_gate))
+      !r->log_amount != !r->log_rate || ((r->gate || r->head_gate) && a->batch != 1) || (r->gate && r->head_gate))
     return -1;
   const void* ptrs[5] = {a->q, a->k, a->v, a->o, r->gate};
   for (int i = 0; i < 5; ++i)
@@ -691,7 +741,7 @@ RB_API int rb_attention_fwd_rule(const RbAttnArgs* a, const RbAttnRule* r, void*
   if (r->gate && r->ld_gate % 8) return -9;
   const int dr = r->rot_dim;
   if (dr) {
-    if (dr < 0 || a->batch != 1 || !r->k_rot || r->softcap > 0.f || r->slopes || r->window || r->chunk) return -1;
+    if (dr < 0 || a->batch != 1 || !r->k_rot || r->softcap > 0.f || r->slopes || r->log_rate || r->window || r->chunk) return -1;
     if (dr > 64 || (dr & 7) || r->ld_k_rot % 8 || r->ld_k_rot < dr || (reinterpret_cast<uintptr_t>(r->k_rot) & 15)) return -9;
   }
   int err = 0;
@@ -707,6 +757,7 @@ RB_API int rb_attention_fwd_rule(const RbAttnArgs* a, const RbAttnRule* r, void*
   p.dk = dk; p.dv = dv; p.softcap = r->softcap; p.slopes = r->slopes; p.chunk = r->chunk;
   p.gate = reinterpret_cast<const __nv_bfloat16*>(r->gate); p.ld_gate = r->ld_gate;
   p.dr = dr; p.head_gate = r->head_gate; p.window = r->window; p.keep = r->window > 0 ? r->keep_first : 0; p.sink = r->sink;
+  p.log_amount = r->log_amount; p.log_rate = r->log_rate; p.out_scale = r->out_scale;
   cudaStream_t stream = reinterpret_cast<cudaStream_t>(stream_v);
   const dim3 grid((a->seq_q + 2 * rb::kF2Tile - 1) / (2 * rb::kF2Tile), a->heads, a->batch);
   if (dr) {
@@ -720,6 +771,13 @@ RB_API int rb_attention_fwd_rule(const RbAttnArgs* a, const RbAttnRule* r, void*
                       : f2_launch<64, 128, 0, true, 64>(tq, tk, tv, p, grid, stream, tqr, tkr);
     return dv <= 64 ? f2_launch<128, 64, 0, true, 64>(tq, tk, tv, p, grid, stream, tqr, tkr)
                     : f2_launch<128, 128, 0, true, 64>(tq, tk, tv, p, grid, stream, tqr, tkr);
+  }
+  if (r->log_rate) {
+    if (dk <= 64)
+      return dv <= 64 ? f2_launch<64, 64, 0, true, 0, true>(tq, tk, tv, p, grid, stream)
+                      : f2_launch<64, 128, 0, true, 0, true>(tq, tk, tv, p, grid, stream);
+    return dv <= 64 ? f2_launch<128, 64, 0, true, 0, true>(tq, tk, tv, p, grid, stream)
+                    : f2_launch<128, 128, 0, true, 0, true>(tq, tk, tv, p, grid, stream);
   }
   if (dk <= 64)
     return dv <= 64 ? f2_launch<64, 64, 0, true>(tq, tk, tv, p, grid, stream) : f2_launch<64, 128, 0, true>(tq, tk, tv, p, grid, stream);

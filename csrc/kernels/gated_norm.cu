@@ -35,7 +35,7 @@ gated_norm_kernel(const RbGatedNormArgs a) {
   const T* y = reinterpret_cast<const T*>(a.y) + t * a.ld_y + base;
   const T* z = reinterpret_cast<const T*>(a.z) + t * a.ld_z + base;
   T* out = reinterpret_cast<T*>(a.out) + t * a.ld_o + base;
-  const float* w = a.weight + (a.weight_n == a.part_n ? 0 : base);
+  const float* w = a.weight ? a.weight + (a.weight_n == a.part_n ? 0 : base) : nullptr;
   float u[CH][VEC], gate[CH][VEC];
   float sq = 0.f;
 #pragma unroll
@@ -59,7 +59,7 @@ gated_norm_kernel(const RbGatedNormArgs a) {
     if (col >= a.part_n) continue;
     float o[VEC];
 #pragma unroll
-    for (int i = 0; i < VEC; ++i) o[i] = u[c][i] * r * w[col + i] * (a.gate_first ? 1.f : gate[c][i]);
+    for (int i = 0; i < VEC; ++i) o[i] = u[c][i] * r * (w ? w[col + i] : 1.f) * (a.gate_first ? 1.f : gate[c][i]);
     RcVec<T, VEC>::store(out + col, o);
   }
 }
@@ -74,7 +74,7 @@ gated_norm_any_kernel(const RbGatedNormArgs a) {
   const long long base = static_cast<long long>(part) * a.part_n;
   const T* y = reinterpret_cast<const T*>(a.y) + t * a.ld_y + base;
   const T* z = reinterpret_cast<const T*>(a.z) + t * a.ld_z + base;
-  const float* w = a.weight + (a.weight_n == a.part_n ? 0 : base);
+  const float* w = a.weight ? a.weight + (a.weight_n == a.part_n ? 0 : base) : nullptr;
   float sq = 0.f;
   for (int c = threadIdx.x; c < a.part_n; c += 256) {
     const float u = rc_get(y + c) * (a.gate_first ? rc_silu<T>(rc_get(z + c)) : 1.f);
@@ -82,7 +82,7 @@ gated_norm_any_kernel(const RbGatedNormArgs a) {
   }
   const float r = 1.f / sqrtf(gn_sum<256>(sq, red) / static_cast<float>(a.part_n) + a.eps);
   for (int c = threadIdx.x; c < a.part_n; c += 256)
-    rc_put(reinterpret_cast<T*>(a.out) + t * a.ld_o + base + c, rc_get(y + c) * rc_silu<T>(rc_get(z + c)) * r * w[c]);
+    rc_put(reinterpret_cast<T*>(a.out) + t * a.ld_o + base + c, rc_get(y + c) * rc_silu<T>(rc_get(z + c)) * r * (w ? w[c] : 1.f));
 }
 
 template <typename T, int VEC, int L>
@@ -115,7 +115,7 @@ int gn_pick(const RbGatedNormArgs& a, cudaStream_t s) {
 RB_API int rb_gated_norm(const RbGatedNormArgs* args, void* stream_v) {
   const RbGatedNormArgs& a = *args;
   if (a.rows <= 0) return 0;
-  if (!a.y || !a.z || !a.out || !a.weight || a.parts <= 0 || a.part_n <= 0 ||
+  if (!a.y || !a.z || !a.out || a.parts <= 0 || a.part_n <= 0 ||
       (a.weight_n != a.part_n && a.weight_n != a.parts * a.part_n))
     return -1;
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream_v);

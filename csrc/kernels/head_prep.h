@@ -1,4 +1,4 @@
-// C interface of the per-head preparation of a packed attention projection (head_prep.cu).
+// C interface of the preparation of a packed attention projection, per head or over whole rows (head_prep.cu).
 #pragma once
 #ifdef __cplusplus
 extern "C" {
@@ -16,10 +16,28 @@ typedef struct RbHeadPrepArgs {
   long long ld, off_q, off_k, off_v, ld_vf, tokens, num_slots;
   int f32, heads, kv_heads, dk, dv, rot_dims;
   float eps;
+  int half;                   // numbers i and i + rot_dims / 2 turn together instead of neighbours (no v_first then)
+  int values_are_keys;        // with half, dk == dv: the value columns and v_cache receive the keys as they were
+  float k_scale;              // with half: of the keys, behind the rotation
 } RbHeadPrepArgs;
 // In place: q <- rms(q) * q_gamma, k <- rms(k) * k_gamma, then neighbouring pairs of their first rot_dims numbers are rotated;
 // v <- (1 - mix) v + mix v_first; k and v also go to their slots.
 int rb_head_prep(const RbHeadPrepArgs* args, void* stream);
+// Rows q [nq] | k [nk] | v [nv] (nk = nv = 0: queries only), in place: q <- rms(q) * q_gamma * (1 + temp_coef ln(floor((pos + 1) /
+// temp_every) + 1)), k <- rms(k) * k_gamma, each norm over the whole part; k and v also go to their slots.
+typedef struct RbRowPrepArgs {
+  void* p;                    // [tokens, ld], bf16 or fp32 (f32)
+  const float* q_gamma;       // [nq]
+  const float* k_gamma;       // [nk]
+  void* k_cache;              // [num_slots, nk] / [num_slots, nv], type of p, or both NULL
+  void* v_cache;
+  const long long* slots;     // cache slot of every token (negative: not stored)
+  const long long* pos;       // position of every token (read with temp_every > 0)
+  long long ld, tokens, num_slots;
+  int f32, nq, nk, nv, temp_every;   // temp_every 0: no factor
+  float temp_coef, eps;
+} RbRowPrepArgs;
+int rb_row_prep(const RbRowPrepArgs* args, void* stream);
 #ifdef __cplusplus
 }
 #endif

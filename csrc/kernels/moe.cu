@@ -292,7 +292,7 @@ __device__ __forceinline__ float glu_exact(float g, float u, float limit) {
 template <typename T, int N, int ACT>
 __global__ void __launch_bounds__(256)
 swiglu_slots_kernel(const T* __restrict__ gu, long long ld_gu, T* __restrict__ h, long long ld_h, int n, int F,
-                    const int* __restrict__ slot_pos, float limit) {
+                    const int* __restrict__ slot_pos, const float* __restrict__ slot_w, float limit) {
   const int chunks = F / N;
   const long long total = static_cast<long long>(n) * chunks;
   const long long stride = static_cast<long long>(gridDim.x) * blockDim.x;
@@ -300,6 +300,7 @@ swiglu_slots_kernel(const T* __restrict__ gu, long long ld_gu, T* __restrict__ h
     const long long s = i / chunks;
     const int c = static_cast<int>(i - s * chunks) * N;
     const long long r = slot_pos ? slot_pos[s] : s;
+    const float w = slot_w ? slot_w[s] : 1.f;            // of the input of both products
     if (N == 8) {
       const uint4 g = *reinterpret_cast<const uint4*>(gu + r * ld_gu + c), u = *reinterpret_cast<const uint4*>(gu + r * ld_gu + F + c);
       const uint32_t gw[4] = {g.x, g.y, g.z, g.w}, uw[4] = {u.x, u.y, u.z, u.w};
@@ -307,14 +308,14 @@ swiglu_slots_kernel(const T* __restrict__ gu, long long ld_gu, T* __restrict__ h
 #pragma unroll
       for (int j = 0; j < 4; ++j) {
         const float2 a = unpack_bf16x2(gw[j]), b = unpack_bf16x2(uw[j]);
-        o[j] = pack_bf16x2(glu<ACT>(a.x, b.x, limit), glu<ACT>(a.y, b.y, limit));
+        o[j] = pack_bf16x2(glu<ACT>(w * a.x, w * b.x, limit), glu<ACT>(w * a.y, w * b.y, limit));
       }
       *reinterpret_cast<uint4*>(h + r * ld_h + c) = make_uint4(o[0], o[1], o[2], o[3]);
     } else {
 #pragma unroll
       for (int j = 0; j < N; ++j) {
         const float g = static_cast<float>(gu[r * ld_gu + c + j]), u = static_cast<float>(gu[r * ld_gu + F + c + j]);
-        h[r * ld_h + c + j] = static_cast<T>(glu_exact<ACT>(g, u, limit));
+        h[r * ld_h + c + j] = static_cast<T>(glu_exact<ACT>(w * g, w * u, limit));
       }
     }
   }
@@ -539,29 +540,29 @@ RB_API int rb_moe_route_sigmoid(const float* logits, const float* correction, in
 }
 namespace {
 template <int ACT>
-int glu_launch(const void* gu, long long ld_gu, void* h, long long ld_h, int n, int F, int f32, const int* slot_pos, float limit,
-               cudaStream_t s) {
+int glu_launch(const void* gu, long long ld_gu, void* h, long long ld_h, int n, int F, int f32, const int* slot_pos, const float* slot_w,
+               float limit, cudaStream_t s) {
   const bool vec = !f32 && !((F | ld_gu | ld_h) & 7) && !((reinterpret_cast<uintptr_t>(gu) | reinterpret_cast<uintptr_t>(h)) & 15);
   const int grid = rb::grid1d(static_cast<long long>(n) * (vec ? F / 8 : F), 256);
   if (f32)
     rb::swiglu_slots_kernel<float, 1, ACT><<<grid, 256, 0, s>>>(reinterpret_cast<const float*>(gu), ld_gu,
-                                                               reinterpret_cast<float*>(h), ld_h, n, F, slot_pos, limit);
+                                                               reinterpret_cast<float*>(h), ld_h, n, F, slot_pos, slot_w, limit);
   else if (vec)
     rb::swiglu_slots_kernel<__nv_bfloat16, 8, ACT><<<grid, 256, 0, s>>>(reinterpret_cast<const __nv_bfloat16*>(gu), ld_gu,
-                                                                       reinterpret_cast<__nv_bfloat16*>(h), ld_h, n, F, slot_pos, limit);
+                                                                       reinterpret_cast<__nv_bfloat16*>(h), ld_h, n, F, slot_pos, slot_w, limit);
   else
     rb::swiglu_slots_kernel<__nv_bfloat16, 1, ACT><<<grid, 256, 0, s>>>(reinterpret_cast<const __nv_bfloat16*>(gu), ld_gu,
-                                                                       reinterpret_cast<__nv_bfloat16*>(h), ld_h, n, F, slot_pos, limit);
+                                                                       reinterpret_cast<__nv_bfloat16*>(h), ld_h, n, F, slot_pos, slot_w, limit);
   return static_cast<int>(cudaGetLastError());
 }
 }  // namespace
 
 RB_API int rb_swiglu_slots(const void* gu, long long ld_gu, void* h, long long ld_h, int n, int F, int f32,
-                           const int* slot_pos, int act, float limit, void* stream_v) {
+                           const int* slot_pos, const float* slot_w, int act, float limit, void* stream_v) {
   if (n <= 0 || F <= 0 || act < 0 || act > 2) return -1;
-  if (act == 2) return glu_launch<2>(gu, ld_gu, h, ld_h, n, F, f32, slot_pos, limit, RB_ST);
-  return act == 1 ? glu_launch<1>(gu, ld_gu, h, ld_h, n, F, f32, slot_pos, limit, RB_ST)
-                  : glu_launch<0>(gu, ld_gu, h, ld_h, n, F, f32, slot_pos, limit, RB_ST);
+  if (act == 2) return glu_launch<2>(gu, ld_gu, h, ld_h, n, F, f32, slot_pos, slot_w, limit, RB_ST);
+  return act == 1 ? glu_launch<1>(gu, ld_gu, h, ld_h, n, F, f32, slot_pos, slot_w, limit, RB_ST)
+                  : glu_launch<0>(gu, ld_gu, h, ld_h, n, F, f32, slot_pos, slot_w, limit, RB_ST);
 }
 RB_API int rb_moe_scatter(const void* x, const int* slot_pos, void* xp, int slots, int k, int dim, void* stream_v) {
   if (slots <= 0 || k <= 0 || dim <= 0 || (dim % 8)) return -1;

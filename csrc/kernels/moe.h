@@ -24,11 +24,12 @@ int rb_moe_route_sigmoid(const float* logits, const float* correction, int T, in
                          int renorm, float eps, int* idx, float* w, void* stream);
 int rb_moe_route_groups(const float* logits, int T, int E, int k, int groups, int keep, int renorm, float eps, int* idx,
                         float* w, void* stream);
-// h[r, :] = act(gu[r, 0:F]) * gu[r, F:2F] for the rows r = slot_pos[0 .. n) (NULL: r = 0 .. n); act 0: silu, 1: relu, 2: clamped,
+// h[r, :] = act(gu[r, 0:F]) * gu[r, F:2F] for the rows r = slot_pos[0 .. n) (NULL: r = 0 .. n), gate and up of row slot_pos[s]
+// first multiplied by slot_w[s] (NULL: by 1); act 0: silu, 1: relu, 2: clamped,
 // g = min(gate, limit), u = clamp(up, -limit, limit), h = g sigmoid(1.702 g) (u + 1).  bf16 or fp32.  The permuted
 // expert buffers are sized for whole tiles per expert; going by slots touches only the rows that hold a token.
 int rb_swiglu_slots(const void* gu, long long ld_gu, void* h, long long ld_h, int n, int F, int f32, const int* slot_pos,
-                    int act, float limit, void* stream);
+                    const float* slot_w, int act, float limit, void* stream);
 // xp[slot_pos[s], :] = x[s / k, :] for the slots s < slots; padding rows of xp are not written (inference).  16-bit elements.
 int rb_moe_scatter(const void* x, const int* slot_pos, void* xp, int slots, int k, int dim, void* stream);
 // Plan of the permutation: slots s = t * k + j are grouped by expert, in ascending slot order inside an expert

@@ -79,7 +79,7 @@ __device__ __forceinline__ float pa_sigmoid(float x) { return __fdividef(1.f, 1.
 // of a tcgen05 tile, which is why this kernel is on the warp-level tensor path; it is bound by the K / V reads.
 //
 // DK / DV are the key / value head sizes rounded up to a compiled size; columns beyond the real sizes are zero-filled in
-// shared memory and never leave it.  RULE adds a score cap, a distance bias, chunked or windowed visibility, a
+// shared memory and never leave it.  RULE adds a score cap, a linear and a logarithmic distance bias, chunked or windowed visibility, a
 // sink and output gates (see RbPagedRowsArgs).  A window's slices cover the kept first tokens and then the window.
 struct PaRule {
   float softcap;
@@ -89,6 +89,9 @@ struct PaRule {
   const float* head_gate;
   long long ld_g;
   int window, keep, sink;
+  const float* log_amount;
+  const float* log_rate;
+  float out_scale;
 };
 // cap * tanh(s / cap) as cap * (1 - 2 / (1 + e^(2 s / cap))): two special-function instructions, absolute error about
 // 1e-7 * cap (tanh.approx would be off by 5e-4 of the score)
@@ -142,7 +145,12 @@ paged_decode_split_kernel(const __nv_bfloat16* __restrict__ q, long long ld_q, c
   const uint32_t vt_u32 = kt_u32 + kKTile * 2;
   const uint32_t q_u32 = smem_u32(q_sh);
   float slope0 = 0.f, slope1 = 0.f, two_over_cap = 0.f;
+  float amount0 = 0.f, amount1 = 0.f, rate0 = 0.f, rate1 = 0.f;
   if (RULE) {
+    if (rule.log_rate) {
+      if (gq < gcount) { amount0 = rule.log_amount[h_base + gq]; rate0 = rule.log_rate[h_base + gq]; }
+      if (gq + 8 < gcount) { amount1 = rule.log_amount[h_base + gq + 8]; rate1 = rule.log_rate[h_base + gq + 8]; }
+    }
     if (rule.slopes) {
       if (gq < gcount) slope0 = rule.slopes[h_base + gq];
       if (gq + 8 < gcount) slope1 = rule.slopes[h_base + gq + 8];
@@ -256,6 +264,10 @@ paged_decode_split_kernel(const __nv_bfloat16* __restrict__ q, long long ld_q, c
           const float dist = static_cast<float>(ctx - 1 - (num < vis.kept ? num : num + vis.gap));
           v0 = fmaf(-slope0, dist, v0);
           v1 = fmaf(-slope1, dist, v1);
+          if (rule.log_rate) {                       // distances behind the last token are masked below
+            v0 = fmaf(-amount0, __logf(fmaf(rate0, fmaxf(dist, 0.f), 1.f)), v0);
+            v1 = fmaf(-amount1, __logf(fmaf(rate1, fmaxf(dist, 0.f), 1.f)), v1);
+          }
         }
         s[n][j] = ok ? v0 : -INFINITY;
         s[n][2 + j] = ok ? v1 : -INFINITY;
@@ -344,7 +356,7 @@ paged_decode_split_kernel(const __nv_bfloat16* __restrict__ q, long long ld_q, c
         den = fmaf(den, sc, __expf(-top));
       }
       float o = num / den;
-      if (RULE) o *= pa_gate(rule, b, h_base + g, col);
+      if (RULE) o *= pa_gate(rule, b, h_base + g, col) * rule.out_scale;
       direct_out[b * ld_o + col] = __float2bfloat16(o);
       continue;
     }
@@ -375,7 +387,7 @@ paged_decode_merge_kernel(const float* __restrict__ partial, const int* __restri
   }
   const long long col = static_cast<long long>(h) * dv + d;
   float o = den > 0.f ? num / den : 0.f;
-  o *= pa_gate(rule, b, h, col);
+  o *= pa_gate(rule, b, h, col) * rule.out_scale;
   out[static_cast<long long>(b) * ld_o + col] = __float2bfloat16(o);
 }
 
@@ -412,6 +424,7 @@ paged_rows_kernel(const RbPagedRowsArgs a RB_BOUNDS_PARAM) {
   if (gap < 0) gap = 0;
   const long long count = pos + 1 - gap;
   const float slope = a.slopes ? a.slopes[h] : 0.f;
+  const float amount = a.log_rate ? a.log_amount[h] : 0.f, log_rate = a.log_rate ? a.log_rate[h] : 0.f;
   const T* K = reinterpret_cast<const T*>(a.k_cache);
   const T* V = reinterpret_cast<const T*>(a.v_cache);
   float acc[kPrMaxV];
@@ -437,6 +450,7 @@ paged_rows_kernel(const RbPagedRowsArgs a RB_BOUNDS_PARAM) {
       s = d * a.scale;
       if (a.softcap > 0.f) s = a.softcap * tanhf(s / a.softcap);
       s -= slope * static_cast<float>(pos - j);
+      if (a.log_rate) s -= amount * log1pf(log_rate * static_cast<float>(pos - j));
     }
     const float mn = fmaxf(m, warp_max(s));                          // finite: key j0 is always visible
     const float al = m == -INFINITY ? 0.f : expf(m - mn);
@@ -459,7 +473,7 @@ paged_rows_kernel(const RbPagedRowsArgs a RB_BOUNDS_PARAM) {
   }
   T* o = reinterpret_cast<T*>(a.out) + r * a.ld_o + static_cast<long long>(h) * a.dv;
   const T* g = a.gate ? reinterpret_cast<const T*>(a.gate) + r * a.ld_g + static_cast<long long>(h) * a.dv : nullptr;
-  const float inv = a.head_gate ? 1.f / (l * (1.f + expf(-a.head_gate[r * a.ld_g + h]))) : 1.f / l;
+  const float inv = a.out_scale * (a.head_gate ? 1.f / (l * (1.f + expf(-a.head_gate[r * a.ld_g + h]))) : 1.f / l);
 #pragma unroll
   for (int i = 0; i < kPrMaxV; ++i) {
     const int c = v0 + i * 32 + lane;
@@ -473,7 +487,7 @@ RB_API int rb_paged_attention_rows(const RbPagedRowsArgs* args, void* stream_v) 
   const RbPagedRowsArgs& a = *args;
   if (a.rows <= 0) return 0;
   if (!a.q || !a.out || !a.k_cache || !a.v_cache || !a.block_tables || !a.row_seq || !a.row_pos || a.heads <= 0 ||
-      a.kv_heads <= 0 || a.heads % a.kv_heads || a.dk <= 0 || a.dv <= 0 || a.dk > 2048 ||
+      a.kv_heads <= 0 || a.heads % a.kv_heads || a.dk <= 0 || a.dv <= 0 || a.dk > 2048 || !a.log_amount != !a.log_rate ||
       a.block_size <= 0 || a.max_blocks <= 0)
     return -1;
   cudaStream_t stream = reinterpret_cast<cudaStream_t>(stream_v);
@@ -530,7 +544,7 @@ int pd_launch(const RbPagedDecodeArgs& a, cudaStream_t stream) {
   }
   auto O = reinterpret_cast<__nv_bfloat16*>(a.out);
   const rb::PaRule rule = {a.softcap, a.slopes, a.chunk, reinterpret_cast<const __nv_bfloat16*>(a.gate), a.head_gate, a.ld_g,
-                           a.window, a.keep_first, a.sink};
+                           a.window, a.keep_first, a.sink, a.log_amount, a.log_rate, a.out_scale};
   const dim3 grid(a.batch, a.kv_heads, nsplit);
   for (int g0 = 0; g0 < group; g0 += rb::kMaxGroup)       // groups wider than 16 heads take several passes
     kern<<<grid, rb::kPaWarps * 32, smem, stream>>>(
@@ -556,7 +570,7 @@ RB_API int rb_paged_attention_decode_rule(const RbPagedDecodeArgs* args, void* s
   const RbPagedDecodeArgs& a = *args;
   if (a.batch <= 0) return 0;
   if (a.heads <= 0 || a.kv_heads <= 0 || a.heads % a.kv_heads || a.dk <= 0 || a.dv <= 0 || a.dk > 128 || a.dv > 128 ||
-      ((a.dk | a.dv) & 7) || a.block_size <= 0 || a.max_blocks <= 0 || !a.scratch || (a.ld_q & 1) ||
+      ((a.dk | a.dv) & 7) || a.block_size <= 0 || a.max_blocks <= 0 || !a.scratch || !a.log_amount != !a.log_rate || (a.ld_q & 1) ||
       a.num_blocks * a.block_size >= (1ll << 31))
     return -1;
   if ((reinterpret_cast<uintptr_t>(a.k_cache) | reinterpret_cast<uintptr_t>(a.v_cache)) & 15) return -2;
@@ -580,7 +594,7 @@ RB_API int rb_paged_attention_decode(const void* q, long long ld_q, void* out, l
   a.q = q; a.ld_q = ld_q; a.out = out; a.ld_o = ld_o; a.k_cache = k_cache; a.v_cache = v_cache;
   a.block_tables = block_tables; a.max_blocks = max_blocks; a.context_lens = context_lens; a.batch = batch;
   a.heads = heads; a.kv_heads = kv_heads; a.dk = a.dv = head_dim; a.block_size = block_size; a.num_blocks = num_blocks;
-  a.scale = scale; a.scratch = scratch;
+  a.scale = scale; a.scratch = scratch; a.out_scale = 1.f;
   cudaStream_t stream = reinterpret_cast<cudaStream_t>(stream_v);
   return head_dim == 128 ? pd_launch<128, 128, false>(a, stream) : pd_launch<64, 64, false>(a, stream);
 }

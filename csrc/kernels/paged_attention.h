@@ -20,7 +20,7 @@ int rb_paged_attention_decode(const void* q, long long ld_q, void* out, long lon
                               int batch, int heads, int kv_heads, int head_dim, int block_size, long long num_blocks,
                               float scale, float* scratch, void* stream);
 // The same decode attention with separate key / value head sizes (multiples of 8, at most 128), a score rule and an output
-// gate; softcap, slopes, chunk, window, sink and gates as in RbPagedRowsArgs below.  bf16 operands.  scratch: fp32
+// gate; softcap, slopes, log bias, chunk, window, sink, gates and out_scale as in RbPagedRowsArgs below.  bf16 operands.  scratch: fp32
 // [rb_paged_attention_scratch_floats(batch, heads, dv, max_blocks, block_size)].
 typedef struct RbPagedDecodeArgs {
   const void* q;             // [batch, heads * dk], pitch ld_q
@@ -36,6 +36,9 @@ typedef struct RbPagedDecodeArgs {
   long long ld_q, ld_o, ld_g, num_blocks;
   int batch, max_blocks, heads, kv_heads, dk, dv, block_size, chunk, window, keep_first, sink;
   float scale, softcap;
+  const float* log_amount;
+  const float* log_rate;
+  float out_scale;
 } RbPagedDecodeArgs;
 int rb_paged_attention_decode_rule(const RbPagedDecodeArgs* args, void* stream);
 // Attention over the pages for any rows of a batch (prompt portions and decoded tokens alike), any head sizes, bf16 or
@@ -45,7 +48,8 @@ int rb_paged_attention_decode_rule(const RbPagedDecodeArgs* args, void* stream);
 //   j < keep_first
 //   sink: a further score 0 without a value takes part in the softmax
 //   score = q . k * scale; softcap > 0: score <- softcap * tanh(score / softcap); slopes (fp32 [heads], or NULL):
-//   score <- score - slopes[h] * (pos - j)
+//   score <- score - slopes[h] * (pos - j); log_amount, log_rate (fp32 [heads] each, or both NULL):
+//   score <- score - log_amount[h] * ln(1 + log_rate[h] * (pos - j)), log_rate not negative; out_scale multiplies the output
 //   gate (type of q, pitch ld_g, [rows, heads * dv], or NULL) or head_gate (fp32 [rows, heads], pitch ld_g, or NULL): the output
 //   is multiplied by sigmoid(gate)
 typedef struct RbPagedRowsArgs {
@@ -62,6 +66,9 @@ typedef struct RbPagedRowsArgs {
   long long ld_q, ld_o, ld_g, num_blocks, ld_kc, ld_vc;
   int f32, rows, max_blocks, heads, kv_heads, dk, dv, block_size, chunk, window, keep_first, sink;
   float scale, softcap;
+  const float* log_amount;
+  const float* log_rate;
+  float out_scale;
 } RbPagedRowsArgs;
 int rb_paged_attention_rows(const RbPagedRowsArgs* args, void* stream);
 #ifdef __cplusplus

@@ -72,7 +72,7 @@ residual_norm_kernel(const RbResidualNormArgs a) {
     if (a.add) rn_load<VEC>(a.add, t * a.ld_add + col, a.y_f32, v[c]);
     if (a.slot_pos) {
       for (int j = 0; j < a.k; ++j) {                     // fixed order: reproducible
-        const float w = a.slot_w[static_cast<long long>(t) * a.k + j];
+        const float w = a.slot_w ? a.slot_w[static_cast<long long>(t) * a.k + j] : 1.f;
         float u[VEC];
         rn_load<VEC>(a.y, a.slot_pos[static_cast<long long>(t) * a.k + j] * a.ldy + col, a.y_f32, u);
 #pragma unroll
@@ -86,8 +86,9 @@ residual_norm_kernel(const RbResidualNormArgs a) {
     }
   }
   const float inv_n = 1.f / static_cast<float>(n);
+  const bool plain = a.gamma == nullptr;             // the source is added as it is
   float mean = 0.f;
-  if (!a.rms) {
+  if (!a.rms && !plain) {
     float s = 0.f;
 #pragma unroll
     for (int c = 0; c < CH; ++c)
@@ -95,23 +96,26 @@ residual_norm_kernel(const RbResidualNormArgs a) {
       for (int i = 0; i < VEC; ++i) s += v[c][i];
     mean = rn_block_sum(s, red) * inv_n;
   }
-  float sq = 0.f;
+  float rstd = 1.f;
+  if (!plain) {
+    float sq = 0.f;
 #pragma unroll
-  for (int c = 0; c < CH; ++c)
-    if ((c * blockDim.x + threadIdx.x) * VEC < n) {
+    for (int c = 0; c < CH; ++c)
+      if ((c * blockDim.x + threadIdx.x) * VEC < n) {
 #pragma unroll
-      for (int i = 0; i < VEC; ++i) { const float d = v[c][i] - mean; sq += d * d; }
-    }
-  const float rstd = rsqrtf(rn_block_sum(sq, red) * inv_n + a.eps);
+        for (int i = 0; i < VEC; ++i) { const float d = v[c][i] - mean; sq += d * d; }
+      }
+    rstd = rsqrtf(rn_block_sum(sq, red) * inv_n + a.eps);
+  }
   float next = 0.f;
 #pragma unroll
   for (int c = 0; c < CH; ++c) {
     const int col = (c * blockDim.x + threadIdx.x) * VEC;
     if (col >= n) continue;
     float g[VEC], b[VEC], o[VEC];
-    rn_load<VEC>(a.gamma, col, a.param_f32, g);
 #pragma unroll
-    for (int i = 0; i < VEC; ++i) b[i] = 0.f;
+    for (int i = 0; i < VEC; ++i) { g[i] = 1.f; b[i] = 0.f; }
+    if (!plain) rn_load<VEC>(a.gamma, col, a.param_f32, g);
     if (a.beta) rn_load<VEC>(a.beta, col, a.param_f32, b);
 #pragma unroll
     for (int i = 0; i < VEC; ++i) o[i] = xr[c][i] + ((v[c][i] - mean) * rstd * g[i] + b[i]);
@@ -253,8 +257,8 @@ RB_API int rb_stream_update(const RbStreamUpdateArgs* args, void* stream_v) {
 
 RB_API int rb_residual_norm(const RbResidualNormArgs* args, void* stream_v) {
   const RbResidualNormArgs& a = *args;
-  if (a.rows <= 0 || a.n <= 0 || !a.y || !a.gamma || (!a.x && !a.h)) return -1;
-  if (a.slot_pos && (!a.slot_w || a.k <= 0)) return -1;
+  if (a.rows <= 0 || a.n <= 0 || !a.y || (!a.gamma && (!a.x || a.beta)) || (!a.x && !a.h)) return -1;
+  if (a.slot_pos && a.k <= 0) return -1;
   if (a.next_gamma && (!a.x || !a.h)) return -1;
   const uintptr_t bits = reinterpret_cast<uintptr_t>(a.y) | reinterpret_cast<uintptr_t>(a.add) |
                          reinterpret_cast<uintptr_t>(a.gamma) | reinterpret_cast<uintptr_t>(a.beta) |

@@ -7,9 +7,9 @@ typedef struct RbResidualNormArgs {
   // source row t: y[t] (slot_pos NULL), or the routed sum  sum_j slot_w[t k + j] * y[slot_pos[t k + j]]; plus add[t] if given
   const void* y;
   const int* slot_pos;
-  const float* slot_w;
+  const float* slot_w;      // NULL: all are 1
   const void* add;
-  const void* gamma;        // bf16 or fp32 [n] (param_f32)
+  const void* gamma;        // bf16 or fp32 [n] (param_f32); NULL: x += source
   const void* beta;         // same type, or NULL
   const void* next_gamma;   // with x: h receives rms(new x) * next_gamma, the next sublayer's input; or NULL
   float* x;                 // fp32 residual [rows, n], updated in place: x += norm(source); NULL: no residual

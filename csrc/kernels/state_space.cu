@@ -1,4 +1,4 @@
-// Mamba-2 state-space recurrence.
+// Mamba-2 state-space recurrence, and the same with one fixed decay per head (retention).
 //
 // Scan form: one CTA owns 64 value columns of one head of one segment and keeps the state's columns in registers (fp32) while it
 // walks over the tokens; B, C, x and the step sizes of 8 tokens at a time are staged in shared memory.  With segments of one
@@ -38,7 +38,8 @@ state_space_scan_kernel(const RbStateSpaceArgs a) {
     S[i] = make_float4(0.f, 0.f, 0.f, 0.f);
     if (live && s.start > 0 && n < a.n) S[i] = st[n * row4];
   }
-  const float rate = expf(a.a_log[h]), dt_bias = a.dt_bias[h], dskip = a.D[h];
+  const bool fixed = a.decay != nullptr;
+  const float rate = fixed ? 0.f : expf(a.a_log[h]), dt_bias = fixed ? 0.f : a.dt_bias[h], dskip = a.D ? a.D[h] : 0.f;
   const T* xbc = reinterpret_cast<const T*>(a.xbc);
   const long long offB = static_cast<long long>(a.heads) * a.p + static_cast<long long>(g) * a.n;
   const long long offC = offB + static_cast<long long>(a.groups) * a.n;
@@ -55,9 +56,9 @@ state_space_scan_kernel(const RbStateSpaceArgs a) {
       sX[t][c] = c0 + c < a.p ? rc_get(xbc + (s.first + t0 + t) * a.ld_xbc + static_cast<long long>(h) * a.p + c0 + c) : 0.f;
     }
     if (tid < m) {
-      const float dt = rc_softplus(a.dt_raw[(s.first + t0 + tid) * a.ld_dt + h] + dt_bias);
+      const float dt = fixed ? 1.f : rc_softplus(a.dt_raw[(s.first + t0 + tid) * a.ld_dt + h] + dt_bias);
       sDt[tid] = dt;
-      sDecay[tid] = expf(-rate * dt);
+      sDecay[tid] = fixed ? a.decay[h] : expf(-rate * dt);
     }
     __syncthreads();
     for (int t = 0; t < m; ++t) {
@@ -106,7 +107,7 @@ int ss_launch(const RbStateSpaceArgs& a, cudaStream_t s) {
 RB_API int rb_state_space_scan(const RbStateSpaceArgs* args, void* stream_v) {
   const RbStateSpaceArgs& a = *args;
   if (a.num_segments <= 0) return 0;
-  if (!a.xbc || !a.dt_raw || !a.dt_bias || !a.a_log || !a.D || !a.state || !a.y || !a.segments || a.heads <= 0 || a.groups <= 0 ||
+  if (!a.xbc || (!a.decay && (!a.dt_raw || !a.dt_bias || !a.a_log)) || !a.state || !a.y || !a.segments || a.heads <= 0 || a.groups <= 0 ||
       a.heads % a.groups || a.p <= 0 || a.n <= 0 || a.n > 256 || a.num_slots <= 0 || a.num_segments > 65535 || a.heads > 65535)
     return -1;
   if (reinterpret_cast<uintptr_t>(a.state) & 15) return -2;

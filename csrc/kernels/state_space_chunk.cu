@@ -1,4 +1,4 @@
-// Mamba-2 state-space recurrence over prompts, chunked: 128 tokens at a time become matrix products on the 5th-generation tensor
+// Mamba-2 state-space recurrence over prompts (or the one with a fixed decay per head), chunked: 128 tokens at a time become matrix products on the 5th-generation tensor
 // cores.
 //
 // With c_t the running sum of the logarithms of the decays inside a chunk and S0 the state in front of it,
@@ -262,13 +262,14 @@ state_space_chunk_kernel(const __grid_constant__ CUtensorMap tmC, const __grid_c
     }
   } else if (warp == 2) {
     // -------------------------------------------------------------------- factors of a chunk, four tokens per lane
-    const float rate2 = expf(a.a_log[h]) * kScLog2e, dt_bias = a.dt_bias[h];
+    const bool fixed = a.decay != nullptr;         // steps of 1
+    const float rate2 = fixed ? -log2f(a.decay[h]) : expf(a.a_log[h]) * kScLog2e, dt_bias = fixed ? 0.f : a.dt_bias[h];
     float raw[4] = {0.f, 0.f, 0.f, 0.f}, total = 0.f;
     auto fetch = [&](int i) {
 #pragma unroll
       for (int k = 0; k < 4; ++k) {
         const int t = off + i * kScChunk + 4 * lane + k;
-        if (t < end) raw[k] = a.dt_raw[static_cast<long long>(seg.first + t) * a.ld_dt + h];
+        if (t < end && !fixed) raw[k] = a.dt_raw[static_cast<long long>(seg.first + t) * a.ld_dt + h];
       }
     };
     fetch(0);
@@ -276,7 +277,7 @@ state_space_chunk_kernel(const __grid_constant__ CUtensorMap tmC, const __grid_c
       float d[4], c[4];
 #pragma unroll
       for (int k = 0; k < 4; ++k) {
-        d[k] = off + i * kScChunk + 4 * lane + k < end ? rc_softplus(raw[k] + dt_bias) : 0.f;
+        d[k] = off + i * kScChunk + 4 * lane + k < end ? (fixed ? 1.f : rc_softplus(raw[k] + dt_bias)) : 0.f;
         c[k] = (k ? c[k ? k - 1 : 0] : 0.f) - rate2 * d[k];
       }
       if (i + 1 < chunks) fetch(i + 1);
@@ -310,7 +311,7 @@ state_space_chunk_kernel(const __grid_constant__ CUtensorMap tmC, const __grid_c
       // ------------------------------------------------------------------ M, one row per thread
       const int wq = warp & 3, row = wq * 32 + lane;
       const uint32_t lane_off = static_cast<uint32_t>(wq * 32) << 16;
-      const float dskip = a.D[h];
+      const float dskip = a.D ? a.D[h] : 0.f;
       const uint32_t zero[16] = {0u, 0u, 0u, 0u, 0u, 0u, 0u, 0u, 0u, 0u, 0u, 0u, 0u, 0u, 0u, 0u};
       for (int i = 0; i < chunks; ++i) {
         const float* tab = reinterpret_cast<const float*>(smem + L::kTab + (i & 1) * 4 * kScChunk * 4);
@@ -497,7 +498,7 @@ const CUtensorMap* sc_map(const void* base, int size, int heads, long long rows,
 RB_API int rb_state_space_chunked(const RbStateSpaceArgs* args, float* span_state, float* span_decay, int span, void* stream_v) {
   const RbStateSpaceArgs& a = *args;
   if (a.num_tiles <= 0) return 0;
-  if (!a.xbc || !a.dt_raw || !a.dt_bias || !a.a_log || !a.D || !a.state || !a.y || !a.segments || !a.tiles || a.f32 || a.heads <= 0 ||
+  if (!a.xbc || (!a.decay && (!a.dt_raw || !a.dt_bias || !a.a_log)) || !a.state || !a.y || !a.segments || !a.tiles || a.f32 || a.heads <= 0 ||
       a.groups <= 0 || a.heads % a.groups || a.p <= 0 || a.n <= 0 || a.num_slots <= 0 || a.num_tiles > 65535 || a.rows <= 0 ||
       span <= 0 || span % rb::kScChunk || (span_state != nullptr) != (span_decay != nullptr))
     return -1;

@@ -56,7 +56,8 @@ class RbAttnArgs(C.Structure):
 class RbAttnRule(C.Structure):
     _fields_ = [("v_dim", c_int), ("softcap", c_float), ("slopes", c_void_p), ("chunk", c_int), ("gate", c_void_p),
                 ("head_gate", c_void_p), ("ld_gate", c_ll), ("window", c_int), ("keep_first", c_int), ("sink", c_int),
-                ("rot_dim", c_int), ("k_rot", c_void_p), ("ld_k_rot", c_ll)]
+                ("rot_dim", c_int), ("k_rot", c_void_p), ("ld_k_rot", c_ll), ("log_amount", c_void_p), ("log_rate", c_void_p),
+                ("out_scale", c_float)]
 
 
 class RbResidualNormArgs(C.Structure):
@@ -75,6 +76,15 @@ class RbHeadPrepArgs(C.Structure):
         ("k_cache", c_void_p), ("v_cache", c_void_p), ("slots", c_void_p), ("rot", c_void_p),
         ("ld", c_ll), ("off_q", c_ll), ("off_k", c_ll), ("off_v", c_ll), ("ld_vf", c_ll), ("tokens", c_ll), ("num_slots", c_ll),
         ("f32", c_int), ("heads", c_int), ("kv_heads", c_int), ("dk", c_int), ("dv", c_int), ("rot_dims", c_int), ("eps", c_float),
+        ("half", c_int), ("values_are_keys", c_int), ("k_scale", c_float),
+    ]
+
+
+class RbRowPrepArgs(C.Structure):
+    _fields_ = [
+        ("p", c_void_p), ("q_gamma", c_void_p), ("k_gamma", c_void_p), ("k_cache", c_void_p), ("v_cache", c_void_p), ("slots", c_void_p),
+        ("pos", c_void_p), ("ld", c_ll), ("tokens", c_ll), ("num_slots", c_ll),
+        ("f32", c_int), ("nq", c_int), ("nk", c_int), ("nv", c_int), ("temp_every", c_int), ("temp_coef", c_float), ("eps", c_float),
     ]
 
 
@@ -85,7 +95,7 @@ class RbPagedRowsArgs(C.Structure):
         ("ld_q", c_ll), ("ld_o", c_ll), ("ld_g", c_ll), ("num_blocks", c_ll), ("ld_kc", c_ll), ("ld_vc", c_ll),
         ("f32", c_int), ("rows", c_int), ("max_blocks", c_int), ("heads", c_int), ("kv_heads", c_int), ("dk", c_int),
         ("dv", c_int), ("block_size", c_int), ("chunk", c_int), ("window", c_int), ("keep_first", c_int), ("sink", c_int),
-        ("scale", c_float), ("softcap", c_float),
+        ("scale", c_float), ("softcap", c_float), ("log_amount", c_void_p), ("log_rate", c_void_p), ("out_scale", c_float),
     ]
 
 
@@ -97,7 +107,7 @@ class RbPagedDecodeArgs(C.Structure):
         ("ld_q", c_ll), ("ld_o", c_ll), ("ld_g", c_ll), ("num_blocks", c_ll),
         ("batch", c_int), ("max_blocks", c_int), ("heads", c_int), ("kv_heads", c_int), ("dk", c_int), ("dv", c_int),
         ("block_size", c_int), ("chunk", c_int), ("window", c_int), ("keep_first", c_int), ("sink", c_int),
-        ("scale", c_float), ("softcap", c_float),
+        ("scale", c_float), ("softcap", c_float), ("log_amount", c_void_p), ("log_rate", c_void_p), ("out_scale", c_float),
     ]
 
 
@@ -151,7 +161,16 @@ class RbStateSpaceArgs(C.Structure):
         ("y", c_void_p), ("segments", c_void_p), ("tiles", c_void_p), ("ld_xbc", c_ll), ("ld_dt", c_ll), ("ld_y", c_ll),
         ("rows", c_ll),
         ("num_segments", c_int), ("num_tiles", c_int), ("heads", c_int), ("groups", c_int), ("p", c_int), ("n", c_int),
-        ("f32", c_int), ("num_slots", c_int),
+        ("f32", c_int), ("num_slots", c_int), ("decay", c_void_p),
+    ]
+
+
+class RbSelectiveScanArgs(C.Structure):
+    _fields_ = [
+        ("x", c_void_p), ("z", c_void_p), ("B", c_void_p), ("C", c_void_p), ("dt_raw", c_void_p), ("dt_bias", c_void_p), ("A", c_void_p),
+        ("D", c_void_p), ("state", c_void_p), ("y", c_void_p), ("segments", c_void_p),
+        ("ld_x", c_ll), ("ld_z", c_ll), ("ld_bc", c_ll), ("ld_dt", c_ll), ("ld_y", c_ll),
+        ("num_segments", c_int), ("num_slots", c_int), ("inner", c_int), ("n", c_int), ("f32", c_int), ("single", c_int), ("scale", c_float),
     ]
 
 

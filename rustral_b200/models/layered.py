@@ -16,6 +16,11 @@ partial rotary positions, or latent attention (keys and values come from one sma
 unrotated key parts and an element-wise output gate; dense squared-ReLU feed-forwards or routed experts with clamped gates, chosen by
 corrected sigmoid scores; a run of layers can be passed through several times, each pass starting from a product of the stream
 and the embedding; the embedding table is the output head.
+
+Seredra: an RMS norm with a single gain in front of every sublayer, outputs added as they are; attention with short convolutions over
+queries, keys and values, norms over whole projections, a query temperature and a logarithmic distance bias (keys and values can be
+another layer's), retention (linear attention with a fixed decay per head), or attention whose values are its keys beside a selective
+scan; dense squared-ReLU feed-forwards or routed experts whose sigmoid scores multiply the experts' inputs.
 """
 from __future__ import annotations
 
@@ -29,8 +34,9 @@ def up8(n: int) -> int:
 
 @dataclass(frozen=True)
 class RotarySpec:
-    """Rotary positions on the first `dims` numbers of a head, neighbours paired.  `factor` > 1: YaRN scaling, which leaves pairs
-    that turn at least `fast` times within `original` positions alone and slows those that turn at most `slow` times."""
+    """Rotary positions on the first `dims` numbers of a head: neighbours are paired, or with `half` numbers i and i + dims / 2.
+    `factor` > 1: YaRN scaling, which leaves pairs that turn at least `fast` times within `original` positions alone and slows those
+    that turn at most `slow` times."""
     dims: int
     base: float
     factor: float = 1.0
@@ -38,6 +44,7 @@ class RotarySpec:
     fast: float = 32.0
     slow: float = 1.0
     scaled: bool = False
+    half: bool = False
 
     def __post_init__(self):
         if self.dims < 0 or self.dims % 2 or self.base <= 1.0 or (self.scaled and (self.factor <= 0.0 or self.original <= 0 or self.fast <= 0.0
@@ -62,12 +69,12 @@ class RotarySpec:
         return 0.1 * math.log(self.factor) + 1.0 if self.scaled else 1.0
 
     @classmethod
-    def from_json(cls, r: dict | None) -> "RotarySpec | None":
+    def from_json(cls, r: dict | None, half: bool = False) -> "RotarySpec | None":
         if not r:
             return None
         s = r.get("scaling")
         kw = dict(factor=float(s["factor"]), original=int(s["original"]), fast=float(s["fast"]), slow=float(s["slow"]), scaled=True) if s else {}
-        return cls(dims=int(r["dims"]), base=float(r["base"]), **kw)
+        return cls(dims=int(r["dims"]), base=float(r["base"]), half=half, **kw)
 
     def to_json(self) -> dict:
         r = {"dims": self.dims, "base": self.base}
@@ -94,6 +101,14 @@ class AttentionSpec:
     gate: str = "element"        # sigmoid output gate: one number per value column ("element"), per head ("head"), or "none"
     rot: RotarySpec | None = None        # rotary positions on queries and keys
     bias: bool = False           # the query, key and value projections have biases
+    out_bias: bool = False       # the output projection has a bias
+    norm_over: str = "head"      # what a query / key norm spans: every "head" by itself, or "all" of the projection
+    conv: int = 0                # taps of a causal convolution on every channel of queries, keys and values (0: none)
+    temp_coef: float = 0.0       # queries at position p times 1 + temp_coef * ln(floor((p + 1) / temp_every) + 1)
+    temp_every: int = 0          # 0: no such factor
+    log_bias: bool = False       # r1 * ln(1 + r2 * distance) is taken off the scores, with two numbers per head
+    values_are_keys: bool = False        # values: the keys as projected, in front of norm and rotation
+    kv_from: int | None = None   # the layer whose cached keys and values are used instead of own ones
 
     def __post_init__(self):
         if min(self.heads, self.kv_heads, self.dim, self.vdim) < 1 or self.heads % self.kv_heads or self.chunk < 0:
@@ -102,6 +117,8 @@ class AttentionSpec:
             raise ValueError(f"invalid attention layer: {self}")
         if self.rot is not None and self.rot.dims > self.dim:
             raise ValueError(f"more rotated dimensions than a head has: {self}")
+        if self.norm_over not in ("head", "all") or self.conv < 0 or self.temp_every < 0 or (self.values_are_keys and self.vdim != self.dim):
+            raise ValueError(f"invalid attention layer: {self}")
 
     @property
     def packed(self) -> int:
@@ -110,13 +127,24 @@ class AttentionSpec:
 
     def tensor_shapes(self, p: str, d: int) -> dict:
         t = {p + "q": (self.heads * self.dim, d), p + "k": (self.kv_heads * self.dim, d), p + "v": (self.kv_heads * self.vdim, d)}
+        if self.values_are_keys:
+            del t[p + "v"]
+        if self.kv_from is not None:
+            t = {p + "q": t[p + "q"]}
+        own = [c for c in "qkv" if p + c in t]
         if self.gate != "none":
             t[p + "g"] = (self.heads * self.vdim if self.gate == "element" else self.heads, d)
         t[p + "o"] = (d, self.heads * self.vdim)
         if self.bias:
-            t.update({p + c + ".b": t[p + c][:1] for c in "qkv"})
+            t.update({p + c + ".b": t[p + c][:1] for c in own})
+        if self.out_bias:
+            t[p + "o.b"] = (d,)
+        if self.conv:
+            t.update({p + c + ".conv": (t[p + c][0], self.conv) for c in own})
         if self.qk_norm:
-            t[p + "q.norm"] = t[p + "k.norm"] = (self.dim,)
+            t.update({p + c + ".norm": (self.dim,) if self.norm_over == "head" else t[p + c][:1] for c in own if c != "v"})
+        if self.log_bias:
+            t[p + "r1"] = t[p + "r2"] = (self.heads,)
         if self.v_mix:
             t[p + "vmix"] = ()
         return t
@@ -125,11 +153,13 @@ class AttentionSpec:
     def from_json(cls, m: dict, **fixed) -> "AttentionSpec":
         mask = m.get("mask") or {}
         size = int(mask.get("size") or 0)
-        sliding = fixed.pop("sliding", False)
+        sliding, half = fixed.pop("sliding", False), fixed.pop("half", False)
+        temp = m.get("q_temp") or {}
         return cls(heads=int(m["heads"]), kv_heads=int(m["kv_heads"]), dim=int(m["dim"]), vdim=int(m["vdim"]), scale=float(m["scale"]),
                    softcap=float(m.get("softcap") or 0.0), v_mix=bool(m.get("v_mix", False)), chunk=0 if sliding else size,
                    window=size if sliding else 0, keep_first=int(mask.get("keep_first") or 0) if sliding else 0,
-                   rot=RotarySpec.from_json(m.get("rot")), **fixed)
+                   rot=RotarySpec.from_json(m.get("rot"), half), conv=int(m.get("conv") or 0), temp_coef=float(temp.get("coef", 0.0)),
+                   temp_every=int(temp.get("every", 0)), kv_from=None if m.get("kv_from") is None else int(m["kv_from"]), **fixed)
 
     def to_json(self) -> dict:
         m = {"heads": self.heads, "kv_heads": self.kv_heads, "dim": self.dim, "vdim": self.vdim, "scale": self.scale}
@@ -143,6 +173,12 @@ class AttentionSpec:
             m["mask"] = {"size": self.window, "keep_first": self.keep_first}
         if self.rot is not None:
             m["rot"] = self.rot.to_json()
+        if self.conv:
+            m["conv"] = self.conv
+        if self.temp_every:
+            m["q_temp"] = {"coef": self.temp_coef, "every": self.temp_every}
+        if self.kv_from is not None:
+            m["kv_from"] = self.kv_from
         return m
 
 
@@ -231,17 +267,75 @@ class StateSpaceSpec:
 
 
 @dataclass(frozen=True)
-class ParallelSpec:
-    """Attention and a state-space mixer side by side: half the sum of their outputs, each RMS-normed over the width."""
-    left: AttentionSpec
-    right: StateSpaceSpec
+class SelectiveSpec:
+    """Mamba: per channel a state of `state` numbers that decay and take up the input with a step size of the channel's own; step sizes
+    (through `dt_rank` numbers), B and C come from the channels behind the convolution."""
+    inner: int
+    state: int
+    dt_rank: int
+    conv: int = 4                # taps of the causal convolution over the channels
+
+    def __post_init__(self):
+        if min(self.inner, self.state, self.dt_rank, self.conv) < 1:
+            raise ValueError(f"invalid selective scan: {self}")
 
     def tensor_shapes(self, p: str, d: int) -> dict:
-        return {**self.left.tensor_shapes(p + "left.", d), **self.right.tensor_shapes(p + "right.", d),
-                p + "left.out": (d,), p + "right.out": (d,)}
+        return {p + "in": (2 * self.inner, d), p + "conv": (self.inner, self.conv), p + "conv.b": (self.inner,),
+                p + "x": (self.dt_rank + 2 * self.state, self.inner), p + "dt": (self.inner, self.dt_rank), p + "dt.b": (self.inner,),
+                p + "A_log": (self.inner, self.state), p + "D": (self.inner,), p + "o": (d, self.inner)}
+
+    @classmethod
+    def from_json(cls, m: dict) -> "SelectiveSpec":
+        return cls(inner=int(m["inner"]), state=int(m["state"]), dt_rank=int(m["dt_rank"]), conv=int(m["conv"]))
 
     def to_json(self) -> dict:
-        return {"left": self.left.to_json(), "right": self.right.to_json()}
+        return asdict(self)
+
+
+@dataclass(frozen=True)
+class ParallelSpec:
+    """Attention and a recurrent mixer side by side: half the sum of their outputs, each RMS-normed over the width, or with `scales` the
+    outputs as they are times one number each."""
+    left: AttentionSpec
+    right: StateSpaceSpec | SelectiveSpec
+    scales: tuple | None = None
+
+    def tensor_shapes(self, p: str, d: int) -> dict:
+        t = {**self.left.tensor_shapes(p + "left.", d), **self.right.tensor_shapes(p + "right.", d)}
+        return t if self.scales is not None else {**t, p + "left.out": (d,), p + "right.out": (d,)}
+
+    def to_json(self) -> dict:
+        m = {"left": self.left.to_json(), "right": self.right.to_json()}
+        return m if self.scales is None else {**m, "left_scale": self.scales[0], "right_scale": self.scales[1]}
+
+
+@dataclass(frozen=True)
+class RetentionSpec:
+    """Retention: linear attention with a fixed decay per head.  Per head a state [dim, vdim] that decays and takes up k v^T; the output,
+    normed per head, is gated."""
+    heads: int
+    dim: int
+    vdim: int
+    decay: tuple
+    rot: RotarySpec | None = None
+
+    def __post_init__(self):
+        if min(self.heads, self.dim, self.vdim) < 1 or len(self.decay) != self.heads or not all(0.0 < x <= 1.0 for x in self.decay) or \
+                (self.rot is not None and self.rot.dims > self.dim):
+            raise ValueError(f"invalid retention layer: {self}")
+
+    def tensor_shapes(self, p: str, d: int) -> dict:
+        n, nv = self.heads * self.dim, self.heads * self.vdim
+        return {p + "q": (n, d), p + "k": (n, d), p + "v": (nv, d), p + "g": (nv, d), p + "o": (d, nv)}
+
+    @classmethod
+    def from_json(cls, m: dict, half: bool = False) -> "RetentionSpec":
+        return cls(heads=int(m["heads"]), dim=int(m["dim"]), vdim=int(m["vdim"]), decay=tuple(float(x) for x in m["decay"]),
+                   rot=RotarySpec.from_json(m.get("rot"), half))
+
+    def to_json(self) -> dict:
+        m = {"heads": self.heads, "dim": self.dim, "vdim": self.vdim, "decay": list(self.decay)}
+        return m if self.rot is None else {**m, "rot": self.rot.to_json()}
 
 
 @dataclass(frozen=True)
@@ -291,9 +385,10 @@ class MoESpec:
     renorm: bool = True          # weights are divided by their sum
     act: str = "silu"            # act(gate) * up; "clamped": see ops.moe.swiglu_rows
     limit: float = 0.0           # of the clamped activation
+    weigh: str = "output"        # what an expert's weight multiplies: its "output" or its "input"
 
     def __post_init__(self):
-        if self.score not in ("softmax", "sigmoid") or self.act not in ("silu", "clamped") or self.group_best not in (1, 2) or \
+        if self.weigh not in ("output", "input") or self.score not in ("softmax", "sigmoid") or self.act not in ("silu", "clamped") or self.group_best not in (1, 2) or \
                 (self.score == "softmax" and (self.correction or self.group_best != 1)) or (self.act == "clamped") != (self.limit > 0.0):
             raise ValueError(f"invalid routed feed-forward: {self}")
         if self.experts % self.groups or not 1 <= self.keep <= self.groups or \
@@ -353,7 +448,7 @@ def _ffn_shapes(p: str, ff: int, d: int) -> dict:
 
 @dataclass(frozen=True)
 class LayerSpec:
-    mixer: AttentionSpec | ParallelSpec | DeltaSpec | LatentSpec
+    mixer: AttentionSpec | ParallelSpec | DeltaSpec | LatentSpec | RetentionSpec
     mlp: MoESpec | DenseSpec | None = None
     weights_of: int | None = None        # the layer whose tensors this one uses (with a cache or state of its own)
 
@@ -376,13 +471,17 @@ class Design:
     mixers: tuple                        # mixer types a layer can have
     mlps: tuple                          # kinds of feed-forward
     block: str                           # "output_norm": norm on every sublayer's output; "parallel": one norm in front of both;
-                                         # "sandwich": a norm in front of every sublayer and one on its output
-    norm: str                            # "layer", "dyt" or "rms" (weights stored as the difference from one)
-    attention: dict                      # fixed fields of AttentionSpec ("sliding": the mask is a window)
+                                         # "sandwich": a norm in front of every sublayer and one on its output;
+                                         # "pre": a norm in front of every sublayer, whose output is added as it is
+    norm: str                            # "layer", "dyt", "rms" (weights stored as the difference from one) or "gain" (RMS, one number)
+    attention: dict                      # fixed fields of AttentionSpec ("sliding": the mask is a window, "half": of its RotarySpec)
     act: str = "silu"
     experts: dict = field(default_factory=dict)      # fixed fields of MoESpec
     gated: bool = True                   # dense feed-forwards have a gate
     tied: bool = False                   # the embedding table is the output head
+    left: dict | None = None             # fixed fields of the attention in a parallel mixer, where they differ
+    selective: bool = False              # a parallel mixer's other side is a selective scan, and both sides have scales
+    half: bool = False                   # rotary positions of retention pair halves
 
 
 DESIGNS = {
@@ -392,6 +491,10 @@ DESIGNS = {
     "Bikilix": Design(("attention", "latent_attention"), ("dense", "moe"), "sandwich", "rms",
                       dict(sliding=True, qk_norm=False, distance_bias=False, gate="none", bias=True), act="relu2",
                       experts=dict(score="sigmoid", correction=True, group_best=2, renorm=False, act="clamped"), gated=False, tied=True),
+    "Seredra": Design(("attention", "parallel", "retention"), ("dense", "moe"), "pre", "gain",
+                      dict(distance_bias=False, gate="none", bias=True, out_bias=True, norm_over="all", log_bias=True),
+                      act="relu2", experts=dict(score="sigmoid", renorm=False, weigh="input"), gated=False,
+                      left=dict(distance_bias=False, gate="none", values_are_keys=True, half=True), selective=True, half=True),
 }
 
 
@@ -421,6 +524,13 @@ class LayeredConfig:
         mixing = [s.mixer for s in self.layers if getattr(s.mixer, "v_mix", False)]
         if len({a.kv_heads * a.vdim for a in mixing}) > 1:
             raise ValueError("layers that mix values must have the same number of value columns")
+        for i, s in enumerate(self.layers):
+            j = getattr(s.mixer, "kv_from", None)
+            if j is None:
+                continue
+            o = self.layers[j].mixer if 0 <= j < i else None
+            if not isinstance(o, AttentionSpec) or o.kv_from is not None or (o.kv_heads, o.dim, o.vdim) != (s.mixer.kv_heads, s.mixer.dim, s.mixer.vdim):
+                raise ValueError(f"layer {i} cannot use the keys and values of layer {j}")
         if self.loop is not None and (self.loop.stop > len(self.layers) or self.design.block != "sandwich"):
             raise ValueError(f"{self.arch} with {len(self.layers)} layers cannot have {self.loop}")
         for i, s in enumerate(self.layers):
@@ -495,7 +605,13 @@ class LayeredConfig:
             if kind == "latent_attention":
                 mixer = LatentSpec.from_json(m)
             elif kind == "parallel":
-                mixer = ParallelSpec(AttentionSpec.from_json(m["left"], **design.attention), StateSpaceSpec.from_json(m["right"]))
+                left = AttentionSpec.from_json(m["left"], **(design.attention if design.left is None else design.left))
+                if design.selective:
+                    mixer = ParallelSpec(left, SelectiveSpec.from_json(m["right"]), (float(m["left_scale"]), float(m["right_scale"])))
+                else:
+                    mixer = ParallelSpec(left, StateSpaceSpec.from_json(m["right"]))
+            elif kind == "retention":
+                mixer = RetentionSpec.from_json(m, design.half)
             elif kind == "delta":
                 mixer = DeltaSpec.from_json(m)
             else:
@@ -518,7 +634,7 @@ class LayeredConfig:
 
     def to_json(self) -> dict:
         """The `config.json` form (inverse of `from_json`)."""
-        types = {AttentionSpec: "attention", ParallelSpec: "parallel", DeltaSpec: "delta", LatentSpec: "latent_attention"}
+        types = {AttentionSpec: "attention", ParallelSpec: "parallel", DeltaSpec: "delta", LatentSpec: "latent_attention", RetentionSpec: "retention"}
 
         def layer(s):
             e = {"type": types[type(s.mixer)], "mixer": s.mixer.to_json(), "mlp": None if s.mlp is None else s.mlp.to_json()}
@@ -541,8 +657,8 @@ class LayeredConfig:
             t["loop.in"], t["loop.step"] = (d, 2 * d), (self.loop.times, d)
 
         def norm(name):
-            t[name] = (d,)
-            if self.design.norm != "rms":
+            t[name] = () if self.design.norm == "gain" else (d,)
+            if self.design.norm not in ("rms", "gain"):
                 t[name + ".b"] = (d,)
             if self.design.norm == "dyt":
                 t[name + ".alpha"] = ()
@@ -557,7 +673,7 @@ class LayeredConfig:
                 norm(p + "norm1b")
             t.update(s.mixer.tensor_shapes(p + "mix.", d))
             if s.mlp is not None:
-                if sandwich or self.design.block == "output_norm":
+                if self.design.block != "parallel":
                     norm(p + "norm2")
                 if sandwich:
                     norm(p + "norm2b")
@@ -571,7 +687,7 @@ class LayeredConfig:
         """Names a checkpoint may hold although no layer reads them: the mixing share of a layer that does not mix, the
         second norm of a layer without a feed-forward."""
         out = set()
-        if self.design.block == "sandwich":
+        if self.design.block in ("sandwich", "pre"):
             return {f"l{i}.{n}" for i, s in enumerate(self.layers) if s.mlp is None for n in ("norm2", "norm2b")}
         if self.design.block != "output_norm":
             return out
@@ -606,4 +722,24 @@ def sandwich_layers(order: str, attention: dict, latent: dict, ff: int, moe: dic
         return {**m, "rot": RotarySpec(**m["rot"])}
     mixers = {"w": AttentionSpec(**rot(attention), **{k: v for k, v in design.attention.items() if k != "sliding"}), "l": LatentSpec(**rot(latent))}
     return tuple(LayerSpec(mixers[c], DenseSpec(ff, design.act, design.gated) if i in dense else MoESpec(**moe, **design.experts))
+                 for i, c in enumerate(order))
+
+
+def prenorm_layers(order: str, attention: dict, left: dict, right: dict, scales: tuple, retention: dict, ff: int, moe: dict, dense: tuple = (),
+                   kv_from: dict | None = None) -> tuple:
+    """Layers of a Seredra model: 'a' an attention layer, 'p' a parallel one (`left`, `right`, `scales`), 'r' retention; the layers whose
+    index is in `dense` have a dense feed-forward of hidden size `ff`, the others routed experts (`moe`); `kv_from`: attention layer ->
+    the one whose keys and values it uses."""
+    design = DESIGNS["Seredra"]
+
+    def rot(m):
+        return {**m, "rot": RotarySpec(**m["rot"], half=True)}
+
+    def mixer(i, c):
+        if c == "a":
+            return AttentionSpec(**attention, **design.attention, kv_from=(kv_from or {}).get(i))
+        if c == "r":
+            return RetentionSpec(**rot(retention))
+        return ParallelSpec(AttentionSpec(**rot(left), **{k: v for k, v in design.left.items() if k != "half"}), SelectiveSpec(**right), scales)
+    return tuple(LayerSpec(mixer(i, c), DenseSpec(ff, design.act, design.gated) if i in dense else MoESpec(**moe, **design.experts))
                  for i, c in enumerate(order))

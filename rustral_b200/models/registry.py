@@ -61,6 +61,7 @@ _HYBRID_KERNELS = ("gemm_tcgen05", "gemm_f32", "embedding", "elementwise", "resi
                    "delta_rule_chunk", "gated_norm")
 
 _SANDWICH_KERNELS = (*_LAYERED_KERNELS, "rope", "latent_attention", "latent_decode_tc")
+_PRENORM_KERNELS = (*_LAYERED_KERNELS, "rope", "short_conv", "selective_scan", "state_space", "state_space_chunk", "gated_norm")
 
 ARCHITECTURES = {a.name: a for a in (
     Architecture("gpt2", _gpt_config, "GPTBody", False, _gpt_weights, _GPT_KERNELS),
@@ -68,6 +69,7 @@ ARCHITECTURES = {a.name: a for a in (
     Architecture("Dolurax", LayeredConfig.from_json, "LayeredBody", True, _layered_weights, _LAYERED_KERNELS),
     Architecture("Vafodra", LayeredConfig.from_json, "ParallelBody", True, _layered_weights, _HYBRID_KERNELS),
     Architecture("Bikilix", LayeredConfig.from_json, "SandwichBody", True, _layered_weights, _SANDWICH_KERNELS),
+    Architecture("Seredra", LayeredConfig.from_json, "PreNormBody", True, _layered_weights, _PRENORM_KERNELS),
 )}
 
 

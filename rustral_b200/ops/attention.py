@@ -17,13 +17,17 @@ class ScoreRule:
     the cap.  chunk > 0: position i sees j only when i // chunk == j // chunk (positions of the sequence; a kernel that is
     handed keys from a chunk's first one on may count from there).  window > 0: position i sees j only when i - j < window or
     j < keep_first (a kernel may be handed the kept keys and then those from the first query's window on).  sink: a further
-    score 0 without a value takes part in the softmax."""
+    score 0 without a value takes part in the softmax.  log_amount, log_rate (fp32 [heads] each): score <- score - log_amount[h] *
+    ln(1 + log_rate[h] * (i - j)), after the cap.  out_scale multiplies the output."""
     softcap: float = 0.0
     slopes: torch.Tensor | None = None
     chunk: int = 0
     window: int = 0
     keep_first: int = 0
     sink: bool = False
+    log_amount: torch.Tensor | None = None
+    log_rate: torch.Tensor | None = None
+    out_scale: float = 1.0
 
     def first_key(self, pos: int) -> int:
         """The first position that the token at `pos` can see, apart from the kept ones."""
@@ -35,13 +39,14 @@ class ScoreRule:
         """(kept, first): the token at `pos` and those behind it need the keys [0, kept) and [first, ...)."""
         first = self.first_key(pos)
         kept = self.keep_first if self.window else 0
-        if kept and self.slopes is not None:
+        if kept and (self.slopes is not None or self.log_rate is not None):
             first = 0                                         # a distance bias wants the keys without a gap
         return (0, 0) if first <= kept else (kept, first)
 
     @property
     def plain(self) -> bool:
-        return not self.softcap and self.slopes is None and not self.chunk and not self.window and not self.sink
+        return not self.softcap and self.slopes is None and not self.chunk and not self.window and not self.sink and \
+            self.log_rate is None and self.out_scale == 1.0
 
 
 def softmax_with_sink(s: torch.Tensor) -> torch.Tensor:
@@ -73,6 +78,9 @@ def attention_reference(q, k, v, causal: bool, scale: float | None = None, kv_le
             s = rule.softcap * torch.tanh(s / rule.softcap)
         if rule.slopes is not None:
             s = s - rule.slopes.to(q.device).float()[None, :, None, None] * (i - j).float()
+        if rule.log_rate is not None:
+            r1, r2 = (t.to(q.device).float()[None, :, None, None] for t in (rule.log_amount, rule.log_rate))
+            s = s - r1 * torch.log1p(r2 * (i - j).clamp(min=0).float())
         if rule.chunk:
             s = s.masked_fill(i // rule.chunk != j // rule.chunk, float("-inf"))
         if rule.window:
@@ -85,7 +93,8 @@ def attention_reference(q, k, v, causal: bool, scale: float | None = None, kv_le
     p = softmax_with_sink(s) if rule is not None and rule.sink else torch.softmax(s, -1)
     if kv_lens is not None:
         p = torch.nan_to_num(p, nan=0.0)                      # rows without a visible key
-    return (p @ vf).permute(0, 2, 1, 3).to(q.dtype)
+    o = (p @ vf).permute(0, 2, 1, 3)
+    return (o if rule is None or rule.out_scale == 1.0 else o * rule.out_scale).to(q.dtype)
 
 
 def _strides3(t):
@@ -199,6 +208,7 @@ def prompt_attention(q, k, v, scale: float, out, rule: ScoreRule | None = None, 
     _fill(a, q, k, v, out, True, scale)
     r.v_dim, r.softcap, r.slopes, r.chunk = dv, rule.softcap, N.ptr(rule.slopes), rule.chunk
     r.window, r.keep_first, r.sink = rule.window, rule.keep_first, int(rule.sink)
+    r.log_amount, r.log_rate, r.out_scale = N.ptr(rule.log_amount), N.ptr(rule.log_rate), rule.out_scale
     if gate is not None:
         r.gate, r.ld_gate = gate.data_ptr(), gate.stride(0)
     if head_gate is not None:
@@ -229,6 +239,7 @@ def prompt_attention_split(q, k, v, k_rot, scale: float, out, gate=None):
         return out
     a, r = N.RbAttnArgs(), N.RbAttnRule()
     _fill(a, q[..., :dn], k, v, out, True, scale)
+    r.out_scale = 1.0
     r.v_dim, r.rot_dim, r.k_rot, r.ld_k_rot = dv, dr, k_rot.data_ptr(), k_rot.stride(0)
     if gate is not None:
         r.gate, r.ld_gate = gate.data_ptr(), gate.stride(0)

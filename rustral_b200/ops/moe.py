@@ -20,7 +20,7 @@ N.optional_sig("rb_moe_route", [P, I, I, I, I, P, P, P, P])
 N.optional_sig("rb_moe_route_bwd", [P, P, P, P, P, I, I, I, I, F, P, P])
 N.optional_sig("rb_moe_route_groups", [P, I, I, I, I, I, I, F, P, P, P])
 N.optional_sig("rb_moe_route_sigmoid", [P, P, I, I, I, I, I, I, I, F, P, P, P])
-N.optional_sig("rb_swiglu_slots", [P, LL, P, LL, I, I, I, P, I, F, P])
+N.optional_sig("rb_swiglu_slots", [P, LL, P, LL, I, I, I, P, P, I, F, P])
 N.optional_sig("rb_moe_scatter", [P, P, P, I, I, I, P])
 N._LAUNCHES["rb_moe_plan"] = 2
 N.optional_sig("rb_moe_plan", [P, I, I, I, P, P, P, P, P, P, I, P])
@@ -106,14 +106,20 @@ def route_sigmoid(logits: torch.Tensor, k: int, groups: int = 1, keep: int = 1, 
 _GLU = {"silu": 0, "relu": 1, "clamped": 2}
 
 
-def swiglu_rows(gu: torch.Tensor, pl: MoEPlan | None = None, act: str = "silu", out=None, limit: float = 0.0) -> torch.Tensor:
+def swiglu_rows(gu: torch.Tensor, pl: MoEPlan | None = None, act: str = "silu", out=None, limit: float = 0.0,
+                weights=None) -> torch.Tensor:
     """act(gate) * up for gu = [gate | up] rows (row-strided views allowed, `out` too), bf16 or fp32; act "silu", "relu", or
-    "clamped": g sigmoid(1.702 g) (u + 1) with g = min(gate, limit) and u = clamp(up, -limit, limit).  With a plan only the rows that hold a token are computed; padding rows of the expert buffer are left unwritten."""
+    "clamped": g sigmoid(1.702 g) (u + 1) with g = min(gate, limit) and u = clamp(up, -limit, limit).  With a plan only the rows that hold a token are computed; padding rows of the expert buffer are left unwritten.
+    `weights` (with a plan, fp32 [T, k]): an expert's input was to be multiplied by its weight, so gate and up are, in front of act."""
     rows, F2 = gu.shape
     if act not in _GLU:
         raise ValueError(f"swiglu_rows: unknown activation {act!r}")
     if not gu.is_cuda:
         g, u = gu.float()[:, :F2 // 2], gu.float()[:, F2 // 2:]
+        if weights is not None:
+            ws = torch.ones(rows, 1)
+            ws[pl.slot_pos.long(), 0] = weights.float().reshape(-1)
+            g, u = g * ws, u * ws
         if act == "clamped":
             g, u = g.clamp(max=limit), u.clamp(-limit, limit) + 1.0
             h = g * torch.sigmoid(1.702 * g) * u
@@ -125,7 +131,7 @@ def swiglu_rows(gu: torch.Tensor, pl: MoEPlan | None = None, act: str = "silu", 
     n = rows if pl is None else pl.slot_pos.numel()
     N.check(N.kernels().rb_swiglu_slots(gu.data_ptr(), gu.stride(0), h.data_ptr(), h.stride(0), n, F2 // 2,
                                         int(gu.dtype == torch.float32), None if pl is None else pl.slot_pos.data_ptr(),
-                                        _GLU[act], float(limit), N.stream_ptr()), "rb_swiglu_slots")
+                                        N.ptr(weights), _GLU[act], float(limit), N.stream_ptr()), "rb_swiglu_slots")
     return h
 
 

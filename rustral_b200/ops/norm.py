@@ -154,17 +154,19 @@ def residual_norm(y, gamma, beta, eps: float, rms: bool = False, *, x=None, h=No
     source row t = y[t], or with `routed` = (slot_pos int32 [T * k], weights fp32 [T, k]) the weighted sum of token t's
     expert rows of `y`; `add` (same dtype as y) is added to it.  With `x` (fp32 [T, n]): x += norm(source) in place and
     `h` receives a copy in its own dtype, or with `next_gamma` (dtype of gamma) rms(x) * next_gamma.  Without `x`: `h` receives
-    norm(source).  Returns h (x when h is None)."""
+    norm(source).  `gamma` None: the source is added as it is (`next_gamma` is then fp32).  Expert weights None: all are 1.  Returns h
+    (x when h is None)."""
     rows = x.shape[0] if x is not None else h.shape[0]
     n = y.shape[1]
     if not y.is_cuda:
         src = y.float()
         if routed is not None:
             slot_pos, w = routed
-            src = (src[slot_pos.long()].view(rows, -1, n) * w.float()[:, :, None]).sum(1)
+            src = src[slot_pos.long()].view(rows, -1, n)
+            src = (src if w is None else src * w.float()[:, :, None]).sum(1)
         if add is not None:
             src = src + add.float()
-        o = norm_forward(src, gamma, beta, eps, rms)[0].float()
+        o = src if gamma is None else norm_forward(src, gamma, beta, eps, rms)[0].float()
         if x is not None:
             x += o
             o = x if next_gamma is None else norm_forward(x, next_gamma, None, eps, True)[0]
@@ -179,9 +181,9 @@ def residual_norm(y, gamma, beta, eps: float, rms: bool = False, *, x=None, h=No
         a.add, a.ld_add = add.data_ptr(), add.stride(0)
     if routed is not None:
         slot_pos, w = routed
-        a.slot_pos, a.slot_w, a.k = slot_pos.data_ptr(), w.data_ptr(), w.shape[1]
+        a.slot_pos, a.slot_w, a.k = slot_pos.data_ptr(), N.ptr(w), slot_pos.numel() // rows
     a.next_gamma = N.ptr(next_gamma)
-    a.gamma, a.beta, a.param_f32 = gamma.data_ptr(), N.ptr(beta), int(gamma.dtype == torch.float32)
+    a.gamma, a.beta, a.param_f32 = N.ptr(gamma), N.ptr(beta), int(gamma is None or gamma.dtype == torch.float32)
     if x is not None:
         if x.dtype != torch.float32:
             raise TypeError("residual_norm: the residual stream is fp32")

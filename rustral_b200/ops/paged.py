@@ -92,6 +92,7 @@ def paged_attention_decode(q, k_cache, v_cache, block_tables, context_lens, scal
         if head_gate is not None:
             a.head_gate, a.ld_g = head_gate.data_ptr(), head_gate.stride(0)
         a.window, a.keep_first, a.sink = rule.window, rule.keep_first, int(rule.sink)
+        a.log_amount, a.log_rate, a.out_scale = N.ptr(rule.log_amount), N.ptr(rule.log_rate), rule.out_scale
         a.scratch, a.batch, a.heads, a.kv_heads, a.dk, a.dv = scratch.data_ptr(), B, heads, hk, d, dv
         a.scale, a.softcap, a.slopes, a.chunk = scale, rule.softcap, N.ptr(rule.slopes), rule.chunk
         N.check(lib.rb_paged_attention_decode_rule(a, N.stream_ptr()), "rb_paged_attention_decode_rule")
@@ -141,6 +142,7 @@ def paged_attention_rows(q, k_cache, v_cache, block_tables, row_seq, row_pos, sc
     if head_gate is not None:
         a.head_gate, a.ld_g = head_gate.data_ptr(), head_gate.stride(0)
     a.window, a.keep_first, a.sink = rule.window, rule.keep_first, int(rule.sink)
+    a.log_amount, a.log_rate, a.out_scale = N.ptr(rule.log_amount), N.ptr(rule.log_rate), rule.out_scale
     a.f32, a.rows, a.heads, a.kv_heads, a.dk, a.dv = int(q.dtype == torch.float32), rows, heads, hk, dk, dv
     a.scale, a.softcap, a.slopes, a.chunk = scale, rule.softcap, N.ptr(rule.slopes), rule.chunk
     N.check(N.kernels().rb_paged_attention_rows(a, N.stream_ptr()), "rb_paged_attention_rows")

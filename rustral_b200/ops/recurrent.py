@@ -1,5 +1,5 @@
 """Mixers that carry state from token to token, over batches of unequal segments: short causal convolution, Mamba-2 state-space
-recurrence, gated delta rule, and the gated norm behind them.
+recurrence (with a fixed decay: retention), Mamba's selective scan, gated delta rule, and the gated norm behind them.
 
 Every op takes a `Segments` table (which rows belong to which sequence, where its state lives, whether it has just begun),
 reads and updates the state tensors in place, and treats a sequence's state as zero at position 0.
@@ -143,9 +143,11 @@ def _span(seg: Segments, ctas_per_span: int, slots: int = 148) -> int:
         size *= 2
 
 
-def state_space(xbc, dt_raw, *, dt_bias, a_log, D, state, heads: int, groups: int, vdim: int, n: int, seg: Segments, out=None):
-    """Mamba-2 recurrence.  xbc [rows, heads * vdim + 2 * groups * n] = x | B | C behind the convolution; dt_raw fp32
-    [rows, heads]; dt_bias, a_log, D fp32 [heads]; state fp32 [slots, heads, n, up4(vdim)].  Returns y [rows, heads * vdim]."""
+def state_space(xbc, dt_raw=None, *, dt_bias=None, a_log=None, D=None, state, heads: int, groups: int, vdim: int, n: int, seg: Segments,
+                decay=None, out=None):
+    """Mamba-2 recurrence, or with `decay` (fp32 [heads]; dt_raw, dt_bias and a_log None) one whose decays are fixed and whose step sizes
+    are 1.  xbc [rows, heads * vdim + 2 * groups * n] = x | B | C behind the convolution; dt_raw fp32
+    [rows, heads]; dt_bias, a_log, D fp32 [heads] (D None: 0); state fp32 [slots, heads, n, up4(vdim)].  Returns y [rows, heads * vdim]."""
     rows = xbc.shape[0]
     inner = heads * vdim
     out = out if out is not None else torch.empty((rows, inner), dtype=xbc.dtype, device=xbc.device)
@@ -154,22 +156,33 @@ def state_space(xbc, dt_raw, *, dt_bias, a_log, D, state, heads: int, groups: in
         x = xbc[:, :inner].float().view(rows, heads, vdim)
         B = xbc[:, inner:inner + groups * n].float().view(rows, groups, n).repeat_interleave(per, 1)
         C = xbc[:, inner + groups * n:inner + 2 * groups * n].float().view(rows, groups, n).repeat_interleave(per, 1)
-        dt = _softplus(dt_raw.float() + dt_bias)
-        decay = torch.exp(-torch.exp(a_log) * dt)
+        if decay is None:
+            dt = _softplus(dt_raw.float() + dt_bias)
+            decay = torch.exp(-torch.exp(a_log) * dt)
+        else:
+            dt, decay = torch.ones(rows, heads), decay.float().expand(rows, heads)
         for first, m, slot, start in seg.host():
             S = state[slot, :, :, :vdim].clone() if start > 0 else torch.zeros(heads, n, vdim)
             for t in range(first, first + m):
                 S = decay[t, :, None, None] * S + (dt[t, :, None] * B[t])[:, :, None] * x[t, :, None, :]
-                out[t] = (torch.einsum("hnp,hn->hp", S, C[t]) + D[:, None] * x[t]).reshape(-1).to(out.dtype)
+                y = torch.einsum("hnp,hn->hp", S, C[t])
+                out[t] = (y if D is None else y + D[:, None] * x[t]).reshape(-1).to(out.dtype)
             state[slot, :, :, :vdim] = S
         return out
     if n > MAX_STATE_ROWS:
         raise ValueError(f"state_space: at most {MAX_STATE_ROWS} state rows per head")
-    _check(dt_raw, torch.float32, "state_space")
+    if (decay is None) == (dt_raw is None):
+        raise ValueError("state_space: either step sizes or fixed decays")
     many, one = seg.split() if _chunked(xbc, n, n, vdim) and out.stride(0) % 8 == 0 and out.data_ptr() % 16 == 0 else (None, seg)
     a = N.RbStateSpaceArgs()
-    a.xbc, a.ld_xbc, a.dt_raw, a.ld_dt, a.y, a.ld_y = xbc.data_ptr(), xbc.stride(0), dt_raw.data_ptr(), dt_raw.stride(0), out.data_ptr(), out.stride(0)
-    a.dt_bias, a.a_log, a.D, a.state, a.num_slots = dt_bias.data_ptr(), a_log.data_ptr(), D.data_ptr(), state.data_ptr(), state.shape[0]
+    a.xbc, a.ld_xbc, a.y, a.ld_y = xbc.data_ptr(), xbc.stride(0), out.data_ptr(), out.stride(0)
+    if decay is None:
+        _check(dt_raw, torch.float32, "state_space")
+        a.dt_raw, a.ld_dt, a.dt_bias, a.a_log = dt_raw.data_ptr(), dt_raw.stride(0), dt_bias.data_ptr(), a_log.data_ptr()
+    else:
+        _check(decay, torch.float32, "state_space")
+        a.decay = decay.data_ptr()
+    a.D, a.state, a.num_slots = N.ptr(D), state.data_ptr(), state.shape[0]
     a.heads, a.groups, a.p, a.n, a.f32 = heads, groups, vdim, n, int(xbc.dtype == torch.float32)
     if one is not None:
         a.segments, a.num_segments = one.table.data_ptr(), one.n
@@ -184,6 +197,48 @@ def state_space(xbc, dt_raw, *, dt_bias, a_log, D, state, heads: int, groups: in
             states = torch.empty((tiles.shape[0], heads, n, vdim), dtype=torch.float32, device=xbc.device)
             decays = torch.empty((tiles.shape[0], heads), dtype=torch.float32, device=xbc.device)
         N.check(N.kernels().rb_state_space_chunked(a, N.ptr(states), N.ptr(decays), span, N.stream_ptr()), "rb_state_space_chunked")
+    return out
+
+
+N.optional_sig("rb_selective_scan", [N.C.POINTER(N.RbSelectiveScanArgs), N.c_void_p])
+MAX_CHANNEL_STATE = 256
+
+
+def selective_scan(x, dt_raw, B, C, z, *, A, D, dt_bias, state, seg: Segments, scale: float = 1.0, out=None):
+    """Mamba's recurrence.  Per channel c, with dt = softplus(dt_raw + dt_bias): S[c] <- exp(dt_c A[c]) S[c] + dt_c x_c B,
+    y_c = S[c] . C + D_c x_c; out = scale * y * silu(z).  x, z [rows, inner], B, C [rows, n] (one dtype, row-strided views allowed; B and
+    C with one pitch), dt_raw fp32 [rows, inner], A fp32 [inner, n] (negative), D, dt_bias fp32 [inner], state fp32 [slots, inner, up4(n)]."""
+    rows, inner = x.shape
+    n = A.shape[1]
+    out = out if out is not None else torch.empty((rows, inner), dtype=x.dtype, device=x.device)
+    if not x.is_cuda:
+        dt = _softplus(dt_raw.float() + dt_bias)
+        xf, zf = x.float(), z.float()
+        for first, m, slot, start in seg.host():
+            S = state[slot, :, :n].clone() if start > 0 else torch.zeros(inner, n)
+            for t in range(first, first + m):
+                S = torch.exp(dt[t, :, None] * A) * S + (dt[t] * xf[t])[:, None] * B[t].float()[None, :]
+                y = S @ C[t].float() + D * xf[t]
+                out[t] = (scale * y * (zf[t] * torch.sigmoid(zf[t]))).to(out.dtype)
+            state[slot, :, :n] = S
+        return out
+    if n > MAX_CHANNEL_STATE:
+        raise ValueError(f"selective_scan: at most {MAX_CHANNEL_STATE} numbers of state per channel")
+    for t in (dt_raw, A, D, dt_bias, state):
+        _check(t, torch.float32, "selective_scan")
+    for t in (z, B, C):
+        _check(t, x.dtype, "selective_scan")
+    if B.stride(0) != C.stride(0) or not A.is_contiguous():
+        raise ValueError("selective_scan: B and C have one pitch, and A is contiguous")
+    a = N.RbSelectiveScanArgs()
+    a.x, a.ld_x, a.z, a.ld_z, a.dt_raw, a.ld_dt = x.data_ptr(), x.stride(0), z.data_ptr(), z.stride(0), dt_raw.data_ptr(), dt_raw.stride(0)
+    a.B, a.C, a.ld_bc, a.y, a.ld_y = B.data_ptr(), C.data_ptr(), B.stride(0), out.data_ptr(), out.stride(0)
+    a.A, a.D, a.dt_bias, a.state, a.num_slots = A.data_ptr(), D.data_ptr(), dt_bias.data_ptr(), state.data_ptr(), state.shape[0]
+    a.inner, a.n, a.f32, a.scale = inner, n, int(x.dtype == torch.float32), scale
+    for part in seg.split():
+        if part is not None:
+            a.segments, a.num_segments, a.single = part.table.data_ptr(), part.n, int(part.single)
+            N.check(N.kernels().rb_selective_scan(a, N.stream_ptr()), "rb_selective_scan")
     return out
 
 
@@ -237,7 +292,7 @@ def delta_rule(qkv, a_raw, b_raw, *, dt_bias, a_log, state, heads: int, kv_heads
 
 def gated_norm(y, z, weight, parts: int, eps: float, gate_first: bool, out=None):
     """RMS norm of every one of `parts` equal parts of y's rows, gated with silu(z) before (gate_first) or behind the norm.
-    weight fp32: one per column, or one part's, shared by all parts."""
+    weight fp32: one per column, or one part's, shared by all parts (None: no weight)."""
     rows, n = y.shape
     m = n // parts
     out = out if out is not None else torch.empty((rows, n), dtype=y.dtype, device=y.device)
@@ -247,13 +302,15 @@ def gated_norm(y, z, weight, parts: int, eps: float, gate_first: bool, out=None)
         u = y.float().view(rows, parts, m)
         if gate_first:
             u = u * g
-        u = u * torch.rsqrt((u * u).mean(-1, keepdim=True) + eps) * weight.view(-1, m)
+        u = u * torch.rsqrt((u * u).mean(-1, keepdim=True) + eps)
+        if weight is not None:
+            u = u * weight.view(-1, m)
         if not gate_first:
             u = u * g
         return out.copy_(u.reshape(rows, n))
     a = N.RbGatedNormArgs()
     a.y, a.ld_y, a.z, a.ld_z, a.out, a.ld_o = y.data_ptr(), y.stride(0), z.data_ptr(), z.stride(0), out.data_ptr(), out.stride(0)
-    a.weight, a.weight_n = weight.data_ptr(), weight.numel()
+    a.weight, a.weight_n = N.ptr(weight), m if weight is None else weight.numel()
     a.rows, a.parts, a.part_n, a.f32, a.gate_first, a.eps = rows, parts, m, int(y.dtype == torch.float32), int(gate_first), eps
     N.check(N.kernels().rb_gated_norm(a, N.stream_ptr()), "rb_gated_norm")
     return out

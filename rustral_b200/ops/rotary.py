@@ -69,6 +69,15 @@ def rotate_pairs(x3: torch.Tensor, table: torch.Tensor) -> torch.Tensor:
     return y
 
 
+def rotate_halves(x3: torch.Tensor, table: torch.Tensor) -> torch.Tensor:
+    """Reference form: a copy of x3 [rows, heads, size] with numbers i and i + pairs of its first 2 * pairs numbers rotated together."""
+    y, n = x3.clone(), table.shape[1]
+    c, s = table[:, None, :, 0], table[:, None, :, 1]
+    u, v = x3[..., :n].float(), x3[..., n:2 * n].float()
+    y[..., :n], y[..., n:2 * n] = (u * c - v * s).to(x3.dtype), (v * c + u * s).to(x3.dtype)
+    return y
+
+
 def rotate_pairs_(x2: torch.Tensor, heads: int, pitch: int, first: int, table: torch.Tensor) -> torch.Tensor:
     """In place on every head of x2 [rows, >= heads * pitch] (bf16 or fp32): the neighbouring pairs that start at column `first` of
     the head turn by `table` (see rotary_table)."""

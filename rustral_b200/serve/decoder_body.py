@@ -14,7 +14,7 @@ import math
 import torch
 
 from .. import ops
-from ..models.layered import DenseSpec, LatentSpec, ParallelSpec, up8
+from ..models.layered import AttentionSpec, DenseSpec, LatentSpec, ParallelSpec, RetentionSpec, up8
 from ..ops import latent as latent_ops
 from ..ops import moe as moe_ops
 from ..ops import norm as norm_ops
@@ -22,10 +22,10 @@ from ..ops import paged as paged_ops
 from ..ops import recurrent as rc_ops
 from ..ops import rotary as rope_ops
 from ..ops.attention import ScoreRule, distance_slopes
-from ..ops.heads import head_prep_
+from ..ops.heads import head_prep_, row_prep_
 from ..ops.matmul import gemm
 from .kv_cache import CacheLayer
-from .weights import latent_columns, packed_columns
+from .weights import latent_columns, mixer_columns, packed_columns
 
 
 class GPTBody:
@@ -95,11 +95,12 @@ class GPTBody:
 class Stream:
     """Residual stream of a layered decoder: `x` fp32, `h` its copy in the activation dtype (the operand of the next
     products; `x` itself in 32-bit), `v_first` the value columns of the first layer that mixes values, `pair` the copies of the
-    stream and of the embedding side by side that a pass through repeated layers starts from."""
-    __slots__ = ("x", "h", "v_first", "pair")
+    stream and of the embedding side by side that a pass through repeated layers starts from, `kv` the step's keys and values of
+    layers whose cache others use."""
+    __slots__ = ("x", "h", "v_first", "pair", "kv")
 
     def __init__(self, x, h):
-        self.x, self.h, self.v_first, self.pair = x, h, None, None
+        self.x, self.h, self.v_first, self.pair, self.kv = x, h, None, None, {}
 
 
 class LayeredBody:
@@ -282,6 +283,32 @@ class ParallelBody:
         return logits
 
 
+def _rotation_frequencies(rots, device) -> dict:
+    """{rotary positions: angle per position of every pair (fp64)} of those that occur."""
+    return {rot: torch.tensor(rot.frequencies(), dtype=torch.float64).to(device) for rot in rots if rot is not None}
+
+
+def _rotation(sb, rot, freqs):
+    """The step's cosines and sines for `rot` (None: no rotation)."""
+    return None if rot is None or rot.dims == 0 else sb.rotation(rot, freqs[rot])
+
+
+def _experts(P, h, m, p):
+    """Routed feed-forward `m` (models.layered.MoESpec) over rows h: (expert rows, (their places, weights or None)) for the sum that
+    ops.norm.residual_norm takes."""
+    logits = gemm(h, P.w(p + "moe.router"), out_dtype=torch.float32)
+    if m.score == "sigmoid":
+        idx, w = moe_ops.route_sigmoid(logits, m.top, m.groups, m.keep, P.w(p + "moe.correction") if m.correction else None,
+                                       m.group_best, m.renorm)
+    else:
+        idx, w = moe_ops.route_groups(logits, m.top, m.groups, m.keep, m.renorm)
+    pl = moe_ops.plan(idx, m.experts)
+    gu = moe_ops.grouped_gemm(moe_ops.scatter_tokens(h, pl), P.w(p + "moe.w1"), pl)
+    at_input = m.weigh == "input"
+    y = moe_ops.grouped_gemm(moe_ops.swiglu_rows(gu, pl, m.act, limit=m.limit, weights=w if at_input else None), P.w(p + "moe.w2"), pl)
+    return y, (pl.slot_pos, None if at_input else w)
+
+
 class SandwichBody:
     """Layered decoders with a norm in front of every sublayer and one on its output (Bikilix); some layers can run several times.
 
@@ -296,8 +323,7 @@ class SandwichBody:
             raise ValueError("tensor-parallel serving covers the llama family")
         self.runs = self.cfg.runs
         self.depth = len(self.runs)
-        freqs = {s.mixer.rot: torch.tensor(s.mixer.rot.frequencies(), dtype=torch.float64) for s in self.cfg.layers if s.mixer.rot is not None}
-        self.freqs = {rot: f.to(runner.device) for rot, f in freqs.items()}
+        self.freqs = _rotation_frequencies([s.mixer.rot for s in self.cfg.layers], runner.device)
         self.columns = [latent_columns(s.mixer) if isinstance(s.mixer, LatentSpec) else None for s in self.cfg.layers]
         self.rules = [self._rule(s.mixer) for s in self.cfg.layers]
 
@@ -314,9 +340,6 @@ class SandwichBody:
             m = self.cfg.layers[i].mixer
             out.append(CacheLayer(1, m.cached, m.kv_rank, joint=True) if isinstance(m, LatentSpec) else CacheLayer(m.kv_heads, m.dim, m.vdim))
         return out
-
-    def _rotation(self, rot, sb):
-        return None if rot is None or rot.dims == 0 else sb.rotation(rot, self.freqs[rot])
 
     def _start(self, st, run, y=None, name=None, **kw):
         """What stands between sublayers: x += norm(y) (none without `y`), then the operand that run number `run` starts from: its
@@ -363,7 +386,7 @@ class SandwichBody:
         if isinstance(s.mlp, DenseSpec):
             y = gemm(gemm(st.h, P.w(p + "up"), act=s.mlp.act), P.w(p + "down"), out_dtype=torch.float32)
             return self._start(st, run + 1, y, p + "norm2b")
-        y, routed = self._experts(st.h, s.mlp, p)
+        y, routed = _experts(P, st.h, s.mlp, p)
         return self._start(st, run + 1, y, p + "norm2b", routed=routed)
 
     def _attention(self, run, i, a, p, h, sb):
@@ -371,31 +394,18 @@ class SandwichBody:
         H, G, dk, dv = a.heads, a.kv_heads, a.dim, a.vdim
         z = gemm(h, P.w(p + "attn.in"), bias=P.w(p + "attn.in.b") if a.bias else None)
         ov = (H + G) * dk
-        head_prep_(z, H, G, dk, dv, k_cache=r.cache.k[run], v_cache=r.cache.v[run], slots=sb.slots, rot=self._rotation(a.rot, sb))
+        head_prep_(z, H, G, dk, dv, k_cache=r.cache.k[run], v_cache=r.cache.v[run], slots=sb.slots, rot=_rotation(sb, a.rot, self.freqs))
         return r.attend(run, z[:, :H * dk], z[:, H * dk:ov], z[:, ov:], sb, a.scale, self.rules[i])
 
     def _latent(self, run, i, m, p, h, sb):
         r, P, cols = self.r, self.r.params, self.columns[i]
         z = gemm(h, P.w(p + "attn.in"))
         part = lambda c: z[:, cols[c][0]:cols[c][0] + cols[c][1]]
-        table = sb.rotation(m.rot, self.freqs[m.rot])
+        table = _rotation(sb, m.rot, self.freqs)
         latent_ops.latent_prep_(z, cols["q"][0], m.q_rank, cols["kv"][0], m.kv_rank, m.rot_dim, q_gamma=P.w(p + "attn.q_norm"),
                                 kv_gamma=P.w(p + "attn.kv_norm"), eps=self.cfg.norm_eps, table=table, cache=r.cache.k[run], slots=sb.slots)
         q = gemm(part("q"), P.w(p + "attn.uq"))
         return r.attend_latent(run, q, part("kv"), sb, m, P.w(p + "attn.ukv"), table, part("g") if "g" in cols else None)
-
-    def _experts(self, h, m, p):
-        P = self.r.params
-        logits = gemm(h, P.w(p + "moe.router"), out_dtype=torch.float32)
-        if m.score == "sigmoid":
-            idx, w = moe_ops.route_sigmoid(logits, m.top, m.groups, m.keep, P.w(p + "moe.correction") if m.correction else None,
-                                           m.group_best, m.renorm)
-        else:
-            idx, w = moe_ops.route_groups(logits, m.top, m.groups, m.keep, m.renorm)
-        pl = moe_ops.plan(idx, m.experts)
-        gu = moe_ops.grouped_gemm(moe_ops.scatter_tokens(h, pl), P.w(p + "moe.w1"), pl)
-        y = moe_ops.grouped_gemm(moe_ops.swiglu_rows(gu, pl, m.act, limit=m.limit), P.w(p + "moe.w2"), pl)
-        return y, (pl.slot_pos, w)
 
     def head(self, st, rows):
         P, cfg = self.r.params, self.cfg
@@ -404,4 +414,139 @@ class SandwichBody:
         logits = gemm(h, P.w("head"), out_dtype=torch.float32)
         if cfg.logit_scale != 1.0 or cfg.logit_softcap:
             ops.scale_softcap_(logits, cfg.logit_scale, cfg.logit_softcap)
+        return logits
+
+
+class PreNormBody:
+    """Layered decoders with a norm in front of every sublayer, whose output is added as it is (Seredra).
+
+    Per layer: one packed projection of everything that reads the first norm; the mixer; one output projection; residual add and the norm
+    in front of the feed-forward in one kernel; dense or routed feed-forward; residual add (with the experts' sum) and the next layer's
+    norm in one kernel.  Mixers: attention (short convolution; norm over the whole projection, temperature and cache append in one kernel;
+    an attention layer can use the cache of an earlier one), retention (the state-space recurrence with fixed decays), or attention whose
+    values are its keys beside a selective scan (both write one buffer, which one product reads)."""
+
+    def __init__(self, runner):
+        self.r, self.cfg = runner, runner.cfg
+        if runner.tp is not None:
+            raise ValueError("tensor-parallel serving covers the llama family")
+        self.depth = self.cfg.n_layer
+        mixers = [s.mixer for s in self.cfg.layers]
+        self.freqs = _rotation_frequencies([m.left.rot if isinstance(m, ParallelSpec) else m.rot for m in mixers], runner.device)
+        self.columns = [None if isinstance(m, AttentionSpec) else mixer_columns(m) for m in mixers]
+        self.rules = [self._rule(l, m) for l, m in enumerate(mixers)]
+        self.lent = {m.kv_from for m in mixers if isinstance(m, AttentionSpec) and m.kv_from is not None}
+
+    def _rule(self, l, m):
+        if isinstance(m, RetentionSpec):
+            return None
+        P, a, scale = self.r.params, m, 1.0
+        if isinstance(m, ParallelSpec):
+            a, scale = m.left, m.scales[0]
+        logs = dict(log_amount=P.w(f"l{l}.attn.r1"), log_rate=P.w(f"l{l}.attn.r2")) if a.log_bias else {}
+        return ScoreRule(a.softcap, None, a.chunk, a.window, a.keep_first, a.sink, out_scale=scale, **logs)
+
+    def cache_layers(self) -> list:
+        out = []
+        for s in self.cfg.layers:
+            m = s.mixer
+            if isinstance(m, RetentionSpec):
+                out.append(CacheLayer(state=(("state", (m.heads, m.dim, rc_ops.up4(m.vdim)), torch.float32),)))
+            elif isinstance(m, ParallelSpec):
+                a, r = m.left, m.right
+                out.append(CacheLayer(a.kv_heads, a.dim, a.vdim, (("conv", (r.conv - 1, r.inner), None),
+                                                                  ("state", (r.inner, rc_ops.up4(r.state)), torch.float32))))
+            else:
+                own = m.heads * m.dim + (m.kv_heads * (m.dim + m.vdim) if m.kv_from is None else 0)
+                out.append(CacheLayer(m.kv_heads, m.dim, m.vdim, (("conv", (m.conv - 1, own), None),) if m.conv else (), kv_of=m.kv_from))
+        return out
+
+    def _start(self, st, l, y=None, **kw):
+        """x += y (none without `y`; `kw`: see ops.norm.residual_norm), then the norm in front of layer l (the head takes its norm over
+        the wanted rows)."""
+        return self._add(st, self.r.params.w(f"l{l}.norm1") if l < self.depth else None, y, **kw)
+
+    def _add(self, st, gamma, y=None, **kw):
+        eps = self.cfg.norm_eps
+        if y is None:
+            st.h = norm_ops.residual_norm(st.x, gamma, None, eps, True, h=torch.empty_like(st.x, dtype=self.r.dtype))
+        else:
+            norm_ops.residual_norm(y, None, None, eps, True, x=st.x, h=None if gamma is None else st.h, next_gamma=gamma, **kw)
+        return st
+
+    def embed(self, sb):
+        x, _ = ops.embedding_residual(sb.ids, self.r.params.w("embed"), self.cfg.embed_scale, want_h=False)
+        return self._start(Stream(x, None), 0)
+
+    def layer(self, l, st, sb):
+        P, s, p = self.r.params, self.cfg.layers[l], f"l{l}."
+        m = s.mixer
+        mix = self._attention if isinstance(m, AttentionSpec) else self._retention if isinstance(m, RetentionSpec) else self._parallel
+        o = mix(l, m, p, st, sb)
+        y = gemm(o, P.w(p + "attn.out"), bias=P.w(p + "attn.out.b") if getattr(m, "out_bias", False) else None, out_dtype=torch.float32)
+        if s.mlp is None:
+            return self._start(st, l + 1, y)
+        self._add(st, P.w(p + "norm2"), y)
+        if isinstance(s.mlp, DenseSpec):
+            return self._start(st, l + 1, gemm(gemm(st.h, P.w(p + "up"), act=s.mlp.act), P.w(p + "down"), out_dtype=torch.float32))
+        y, routed = _experts(P, st.h, s.mlp, p)
+        return self._start(st, l + 1, y, routed=routed)
+
+    def _attention(self, l, a, p, st, sb):
+        r, P = self.r, self.r.params
+        H, dk, dv, own = a.heads, a.dim, a.vdim, a.kv_from is None
+        G = a.kv_heads if own else 0
+        z = gemm(st.h, P.w(p + "attn.in"), bias=P.w(p + "attn.in.b") if a.bias else None)
+        if a.conv:
+            z = rc_ops.short_conv(z, P.w(p + "attn.conv"), None, r.cache.state[l]["conv"], sb.segments, silu=False)
+        row_prep_(z, H, G, dk, dv, q_gamma=P.w(p + "attn.q_norm"), k_gamma=P.w(p + "attn.k_norm") if own else None, eps=self.cfg.norm_eps,
+                  pos=sb.pos, temp_coef=a.temp_coef, temp_every=a.temp_every, k_cache=r.cache.k[l], v_cache=r.cache.v[l], slots=sb.slots)
+        q, ov = z[:, :H * dk], (H + G) * dk
+        kv = (z[:, H * dk:ov], z[:, ov:]) if own else st.kv[a.kv_from]
+        if l in self.lent:
+            st.kv[l] = kv                                  # views: this layer's projection buffer stays alive
+        return r.attend(l, q, *kv, sb, a.scale, self.rules[l])
+
+    def _retention(self, l, m, p, st, sb):
+        P, cols, H = self.r.params, self.columns[l], m.heads
+        z = gemm(st.h, P.w(p + "attn.in"))
+        head_prep_(z, H, H, m.dim, m.dim, rot=_rotation(sb, m.rot, self.freqs), half=True, k_scale=m.dim ** -0.5, q_col=cols["q"][0],
+                   k_col=cols["k"][0])
+        o = rc_ops.state_space(z[:, :H * (m.vdim + 2 * m.dim)], decay=P.w(p + "attn.decay"), state=self.r.cache.state[l]["state"], heads=H,
+                               groups=H, vdim=m.vdim, n=m.dim, seg=sb.segments)
+        lo, n = cols["g"]
+        return rc_ops.gated_norm(o, z[:, lo:lo + n], None, H, self.cfg.norm_eps, gate_first=False, out=o)
+
+    def _parallel(self, l, m, p, st, sb):
+        r, P, cols = self.r, self.r.params, self.columns[l]
+        a, s = m.left, m.right
+        w_in, (lo, n) = P.w(p + "attn.in"), cols["v"]
+        z = torch.empty((sb.rows, up8(lo + n)), dtype=r.dtype, device=r.device)
+        gemm(st.h, w_in, out=z[:, :cols["end"][0]])
+        part = lambda c: z[:, cols[c][0]:cols[c][0] + cols[c][1]]
+        head_prep_(z, a.heads, a.kv_heads, a.dim, a.vdim, q_gamma=P.w(p + "attn.q_norm"), k_gamma=P.w(p + "attn.k_norm"), eps=self.cfg.norm_eps,
+                   rot=_rotation(sb, a.rot, self.freqs), half=True, k_cache=r.cache.k[l], v_cache=r.cache.v[l], slots=sb.slots, v_col=lo,
+                   values_are_keys=True)
+        n, state = a.heads * a.vdim, r.cache.state[l]
+        joined = torch.empty((sb.rows, P.w(p + "attn.out").shape[1]), dtype=r.dtype, device=r.device)       # attention | scan
+        for edge, room in ((n, up8(n)), (up8(n) + s.inner, joined.shape[1])):
+            if edge != room:
+                joined[:, edge:room] = 0
+        r.attend(l, part("q"), part("k"), part("v"), sb, a.scale, self.rules[l], out=joined[:, :n])
+        x = rc_ops.short_conv(part("conv"), P.w(p + "scan.conv"), P.w(p + "scan.conv.b"), state["conv"], sb.segments)
+        low = gemm(x, P.w(p + "scan.x"))
+        r8, ns = up8(s.dt_rank), s.state
+        dt = gemm(low[:, :r8], P.w(p + "scan.dt"), out_dtype=torch.float32)
+        rc_ops.selective_scan(x, dt, low[:, r8:r8 + ns], low[:, r8 + ns:], part("z"), A=P.w(p + "scan.A"), D=P.w(p + "scan.D"),
+                              dt_bias=P.w(p + "scan.dt.b"), state=state["state"], seg=sb.segments, scale=m.scales[1],
+                              out=joined[:, up8(n):up8(n) + s.inner])
+        return joined
+
+    def head(self, st, rows):
+        P = self.r.params
+        x = st.x if rows is None else ops.gather_rows(st.x, rows)
+        h = norm_ops.residual_norm(x, P.w("final.norm"), None, self.cfg.norm_eps, True, h=torch.empty_like(x, dtype=self.r.dtype))
+        logits = gemm(h, P.w("head"), out_dtype=torch.float32)
+        if self.cfg.logit_scale != 1.0 or self.cfg.logit_softcap:
+            ops.scale_softcap_(logits, self.cfg.logit_scale, self.cfg.logit_softcap)
         return logits

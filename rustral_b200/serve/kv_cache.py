@@ -170,12 +170,14 @@ class SlidingWindowCache(KVCache):
 class CacheLayer:
     """What one layer stores: per token `kv_heads` keys of size `k_dim` and values of size `v_dim` (kv_heads 0: none), and
     per sequence the tensors of `state`, each (name, shape, dtype or None for the cache's).  `joint`: the values are the first
-    `v_dim` numbers of the keys and take no room of their own."""
+    `v_dim` numbers of the keys and take no room of their own.  `kv_of`: an earlier layer whose keys and values this one uses (it stores
+    none of its own)."""
     kv_heads: int = 0
     k_dim: int = 0
     v_dim: int = 0
     state: tuple = ()
     joint: bool = False
+    kv_of: int | None = None
 
 
 class PagedCache:
@@ -206,9 +208,12 @@ class PagedCache:
         if allocate_storage and layers is not None:
             def pages(c, d):
                 return torch.zeros((num_blocks, block_size, c.kv_heads, d), dtype=dtype, device=device) if c.kv_heads else None
-            self.k = [pages(c, c.k_dim) for c in layers]
-            self.v = [k[..., :c.v_dim] if c.joint else pages(c, c.v_dim) for c, k in zip(layers, self.k)]
-            self._joint = [c.joint for c in layers]
+            self.k, self.v = [], []
+            for c in layers:
+                shared = c.kv_of is not None
+                self.k.append(self.k[c.kv_of] if shared else pages(c, c.k_dim))
+                self.v.append(self.v[c.kv_of] if shared else self.k[-1][..., :c.v_dim] if c.joint else pages(c, c.v_dim))
+            self._own = [(c.kv_of is None, c.kv_of is None and not c.joint) for c in layers]       # keys, values take room
             self.state = [{n: torch.zeros((num_slots, *shape), dtype=dt or dtype, device=device) for n, shape, dt in c.state}
                           for c in layers]
         elif allocate_storage:
@@ -263,8 +268,8 @@ class PagedCache:
     def memory_bytes(self) -> int:
         if self.k is None:
             return 0
-        joint = getattr(self, "_joint", [False] * len(self.v))
-        held = [*self.k, *(v for v, j in zip(self.v, joint) if not j)]
+        own = getattr(self, "_own", [(True, True)] * len(self.v))
+        held = [t for k, v, (ok, ov) in zip(self.k, self.v, own) for t, o in ((k, ok), (v, ov)) if o]
         held = [t for t in held if t is not None] + [t for d in self.state for t in d.values()]
         return sum(t.numel() * t.element_size() for t in held)
 

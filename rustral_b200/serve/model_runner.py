@@ -130,12 +130,12 @@ class ModelRunner:
         self._graphs: dict = {}
 
     # ---- attention over the rows of a step -------------------------------------------------------------------------
-    def attend(self, l: int, q, k2, v2, sb: StepBatch, scale: float, rule=None, gate=None, head_gate=None) -> torch.Tensor:
+    def attend(self, l: int, q, k2, v2, sb: StepBatch, scale: float, rule=None, gate=None, head_gate=None, out=None) -> torch.Tensor:
         """Attention of layer `l` for every row of `sb`; the rows' keys and values (`k2`, `v2`) are already in the cache.
         Prompt portions go through the flash kernel (keys: the cached positions the portion can still see, gathered from the
         pages, plus the portion itself), decoded rows through the paged kernel; operands that those do not take (fp32,
         unusual head sizes) go through the paged row kernel.  `rule`: ops.ScoreRule; `gate` (one number per value
-        column) or `head_gate` (fp32, one per head): output times sigmoid(gate)."""
+        column) or `head_gate` (fp32, one per head): output times sigmoid(gate); `out` (a row-strided view) receives it."""
         kc, vc = self.cache.k[l], self.cache.v[l]
         nb, bs, G, dk = kc.shape
         dv = vc.shape[3]
@@ -145,8 +145,8 @@ class ModelRunner:
         paged = paged_ops.decode_supported(q, dk, dv, rule, gate)
         if (sb.spans and not flash) or (sb.rd < T and not paged):
             bt, seq = sb.row_tables()
-            return paged_ops.paged_attention_rows(q, kc, vc, bt, seq, sb.pos, scale, rule, gate, head_gate=head_gate)
-        a = torch.empty((T, H * dv), dtype=q.dtype, device=self.device)
+            return paged_ops.paged_attention_rows(q, kc, vc, bt, seq, sb.pos, scale, rule, gate, out, head_gate)
+        a = out if out is not None else torch.empty((T, H * dv), dtype=q.dtype, device=self.device)
         for i, (r0, r1, start) in enumerate(sb.spans):
             L = r1 - r0
             kept, first = rule.key_ranges(start) if rule is not None else (0, 0)

@@ -9,7 +9,7 @@ import zlib
 import torch
 
 from ..models.config import GPTConfig
-from ..models.layered import DenseSpec, LatentSpec, ParallelSpec, up8
+from ..models.layered import AttentionSpec, DenseSpec, LatentSpec, ParallelSpec, RetentionSpec, up8
 
 
 class InferenceWeights:
@@ -136,14 +136,16 @@ class InferenceWeights:
                 return torch.zeros(shape, dtype=dt, device=dev)
             if last in ("norm", "norm1", "norm2", "out", "D"):
                 return torch.ones(shape, dtype=dt, device=dev)
-            if last == "b" and len(shape) == 1:
+            if last in ("r1", "r2"):
+                return torch.full(shape, 0.5, dtype=dt, device=dev)
+            if last == "b" and len(shape) == 1 and not name.endswith(".dt.b"):
                 return torch.zeros(shape, dtype=dt, device=dev)
             if last in ("vmix", "alpha"):
                 return torch.full(shape, 0.5, dtype=dt, device=dev)
             g = torch.Generator(device=dev).manual_seed(zlib.crc32(f"{seed}/{name}".encode()))
             if last == "A_log":
                 return torch.empty(shape, dtype=torch.float32, device=dev).uniform_(1.0, 16.0, generator=g).log().to(dt)
-            if last == "dt_bias":
+            if last == "dt_bias" or name.endswith(".dt.b"):
                 return torch.empty(shape, dtype=torch.float32, device=dev).uniform_(-6.0, -2.0, generator=g).to(dt)
             std = shape[-1] ** -0.5 if last == "conv" else cfg.init_std
             return torch.empty(shape, dtype=torch.float32, device=dev).normal_(0.0, std, generator=g).to(dt)
@@ -169,6 +171,8 @@ class InferenceWeights:
         def norm(name):
             if cfg.design.norm == "rms":
                 t[name] = 1.0 + f32(name)                  # stored as the difference from one
+            elif cfg.design.norm == "gain":
+                t[name] = f32(name).expand(d).contiguous()
             elif cfg.design.norm == "dyt":
                 t[name], t[name + ".b"], t[name + ".alpha"] = f32(name), f32(name + ".b"), f32(name + ".alpha").reshape(1)
             else:
@@ -199,12 +203,15 @@ class InferenceWeights:
                 continue
             p, m = f"l{i}.", s.mlp
             norm(p + "norm1")
-            if cfg.design.block == "sandwich":
-                norm(p + "norm1b")
-                cls._mixer_in_front(t, p, s.mixer, d, get, f32, dt, dev)
+            if cfg.design.block in ("sandwich", "pre"):
+                sandwich = cfg.design.block == "sandwich"
+                if sandwich:
+                    norm(p + "norm1b")
+                (cls._mixer_in_front if sandwich else cls._mixer_pre)(t, p, s.mixer, d, get, f32, dt, dev)
                 if m is not None:
                     norm(p + "norm2")
-                    norm(p + "norm2b")
+                    if sandwich:
+                        norm(p + "norm2b")
                     if isinstance(m, DenseSpec):
                         t[p + "up"], t[p + "down"] = _pitched(get(p + "mlp.up")), _pitched(get(p + "mlp.down"))
                     else:
@@ -248,6 +255,54 @@ class InferenceWeights:
         t[p + "attn.q_norm"], t[p + "attn.kv_norm"] = f32(x + "dq.norm"), f32(x + "dkv.norm")
         t[p + "attn.uq"] = _pitched(get(x + "uq"))
         t[p + "attn.ukv"] = _pitched(torch.cat([get(x + "uk"), get(x + "uv")], 0))
+
+    @staticmethod
+    def _mixer_pre(t, p, m, d, get, f32, dt, dev) -> None:
+        """The mixer of a layer whose output is added as it is: one packed projection of everything that reads the norm (`mixer_columns`),
+        and one output projection (both sides of a parallel mixer as one product over their joined outputs)."""
+        x = p + "mix."
+        if isinstance(m, AttentionSpec):
+            own = "qkv" if m.kv_from is None else "q"
+            t[p + "attn.in"] = torch.cat([get(x + c) for c in own], 0)
+            t[p + "attn.out"] = _pitched(get(x + "o"))
+            if m.bias:
+                t[p + "attn.in.b"] = torch.cat([get(x + c + ".b") for c in own], 0)
+            if m.out_bias:
+                t[p + "attn.out.b"] = get(x + "o.b")
+            if m.conv:
+                t[p + "attn.conv"] = torch.cat([f32(x + c + ".conv") for c in own], 0)
+            t.update({f"{p}attn.{c}_norm": f32(f"{x}{c}.norm") for c in own if c != "v"})
+            t[p + "attn.r1"], t[p + "attn.r2"] = f32(x + "r1"), f32(x + "r2")
+            return
+        cols = mixer_columns(m)
+        w = torch.zeros((cols["end"][0], d), dtype=dt, device=dev)
+        if isinstance(m, RetentionSpec):
+            parts = {c: get(x + c) for c in "qkvg"}
+            t[p + "attn.out"] = _pitched(get(x + "o"))
+            t[p + "attn.decay"] = torch.tensor(m.decay, dtype=torch.float32, device=dev)
+        else:
+            r, s = x + "right.", m.right
+            both = get(r + "in")
+            parts = {"q": get(x + "left.q"), "k": get(x + "left.k"), "conv": both[:s.inner], "z": both[s.inner:]}
+            t[p + "attn.q_norm"], t[p + "attn.k_norm"] = get(x + "left.q.norm"), get(x + "left.k.norm")
+            n = m.left.heads * m.left.vdim
+            out = torch.zeros((d, up8(n) + up8(s.inner)), dtype=dt, device=dev)
+            out[:, :n], out[:, up8(n):up8(n) + s.inner] = get(x + "left.o"), get(r + "o")
+            t[p + "attn.out"] = out
+            r8 = up8(s.dt_rank)                            # the rows behind the step sizes' are zero, and so is what they give
+            low = torch.zeros((r8 + 2 * s.state, s.inner), dtype=dt, device=dev)
+            src = get(r + "x")
+            low[:s.dt_rank], low[r8:] = src[:s.dt_rank], src[s.dt_rank:]
+            t[p + "scan.x"] = _pitched(low)
+            step = torch.zeros((s.inner, r8), dtype=dt, device=dev)
+            step[:, :s.dt_rank] = get(r + "dt")
+            t[p + "scan.dt"] = step
+            t[p + "scan.conv"], t[p + "scan.conv.b"] = f32(r + "conv"), f32(r + "conv.b")
+            t[p + "scan.dt.b"], t[p + "scan.D"] = f32(r + "dt.b"), f32(r + "D")
+            t[p + "scan.A"] = -torch.exp(f32(r + "A_log"))
+        for nm, part in parts.items():
+            w[cols[nm][0]:cols[nm][0] + cols[nm][1]] = part
+        t[p + "attn.in"] = w
 
     @staticmethod
     def _parallel_block(t, p, s, d, get, f32, dt, dev) -> None:
@@ -330,6 +385,26 @@ def latent_columns(m) -> dict:
             out[nm] = (at, n)
             at = up8(at + n)
     out["end"] = (at, 0)
+    return out
+
+
+def mixer_columns(m) -> dict:
+    """Columns of the packed projection of a retention or parallel mixer (sections start at multiples of 8).  Retention: what the state
+    takes up and reads is contiguous (v, k, q).  Parallel: "v", behind "end", is no product but the room for a copy of the keys."""
+    if isinstance(m, RetentionSpec):
+        groups = [[("v", m.heads * m.vdim), ("k", m.heads * m.dim), ("q", m.heads * m.dim)], [("g", m.heads * m.vdim)]]
+    else:
+        a, r = m.left, m.right
+        groups = [[("q", a.heads * a.dim), ("k", a.kv_heads * a.dim)], [("conv", r.inner)], [("z", r.inner)]]
+    out, at = {}, 0
+    for g in groups:
+        for nm, n in g:
+            out[nm] = (at, n)
+            at += n
+        at = up8(at)
+    out["end"] = (at, 0)
+    if not isinstance(m, RetentionSpec):
+        out["v"] = (at, m.left.kv_heads * m.left.vdim)
     return out
 
 
