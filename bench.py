@@ -41,7 +41,7 @@ def parse_args():
     ap.add_argument("--comm", default="auto", choices=["auto", "nccl", "fused"])
     ap.add_argument("--seq-len", type=int, default=0, help="override the preset's sequence length (tests only)")
     ap.add_argument("--layers", type=int, default=0, help="override the preset's depth (tests only)")
-    ap.add_argument("--decoders", nargs="?", const="dolurax", choices=["dolurax", "vafodra", "bikilix"], help="serving throughput of a layered "
+    ap.add_argument("--decoders", nargs="?", const="dolurax", choices=["dolurax", "vafodra", "bikilix", "seredra"], help="serving throughput of a layered "
                     "decoder (default: dolurax) beside the closest other one at equal size, and their kernels against the roofline "
                     "(one GPU), instead of the training benchmark")
     ap.add_argument("--decoder-size", default=None, help="with --decoders: only this size")
@@ -52,11 +52,11 @@ def decoder_arm(args):
     import torch
     sys.path.insert(0, os.path.dirname(os.path.abspath(__file__)))
     from rustral_b200 import _native
-    from rustral_b200.bench import decoders, hybrid, looped
+    from rustral_b200.bench import decoders, hybrid, looped, prenorm
     torch.cuda.set_device(0)
     sampler = ClockSampler(0)
     sampler.start()
-    out = {"dolurax": decoders, "vafodra": hybrid, "bikilix": looped}[args.decoders].run([args.decoder_size] if args.decoder_size else None)
+    out = {"dolurax": decoders, "vafodra": hybrid, "bikilix": looped, "seredra": prenorm}[args.decoders].run([args.decoder_size] if args.decoder_size else None)
     out["clocks"] = sampler.stop()
     out["device_status"] = _native.read_status()[0]
     print(json.dumps(out))

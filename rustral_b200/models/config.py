@@ -3,7 +3,7 @@ from __future__ import annotations
 
 from dataclasses import dataclass, asdict
 
-from .layered import LayeredConfig, LoopSpec, hybrid_layers, sandwich_layers, uniform_layers
+from .layered import LayeredConfig, LoopSpec, hybrid_layers, prenorm_layers, sandwich_layers, uniform_layers
 
 
 @dataclass
@@ -123,6 +123,25 @@ PRESETS = {
                         latent=dict(heads=32, dim=128, rot_dim=64, vdim=128, kv_rank=512, q_rank=1536, scale=0.07216878364870322,
                                     rot=dict(dims=64, base=500000.0, factor=8.0, original=4096, fast=32.0, slow=1.0, scaled=True)),
                         moe=dict(ff=2048, experts=32, top=7, groups=4, keep=2, limit=7.0)),
+    # layered decoders with a norm in front of every sublayer (order: p = attention beside a selective scan, r = retention, a = attention
+    # with short convolutions; kv_from: an attention layer -> the one whose keys and values it uses)
+    "seredra-test": dict(arch="Seredra", vocab_size=1000, d_model=128, seq_len=512, embed_scale=3.0, order="rapa", kv_from={3: 1}, dense=(1, 2),
+                         attention=dict(heads=6, kv_heads=2, dim=48, vdim=32, scale=0.15, conv=3, temp_coef=0.3, temp_every=40),
+                         left=dict(heads=3, kv_heads=1, dim=40, vdim=40, scale=0.16, softcap=15.0,
+                                   rot=dict(dims=32, base=10000.0, factor=4.0, original=128, fast=16.0, slow=1.0, scaled=True)),
+                         right=dict(inner=160, state=12, dt_rank=8, conv=4), scales=(0.8, 1.1),
+                         retention=dict(heads=3, dim=24, vdim=56, decay=(0.9, 0.97, 0.995), rot=dict(dims=24, base=100000.0)), ff=192,
+                         moe=dict(ff=64, experts=12, top=3)),
+    # about the size of Llama-8B layers: same width, heads and head size; every third layer an attention layer, every other of them
+    # without a cache of its own
+    "seredra-moe": dict(arch="Seredra", vocab_size=128256, d_model=4096, embed_scale=1.0, order="pra" * 10, kv_from={i: i - 3 for i in range(5, 30, 6)},
+                        dense=tuple(range(0, 30, 2)),
+                        attention=dict(heads=32, kv_heads=8, dim=128, vdim=128, scale=0.08838834764831845, conv=4, temp_coef=0.1, temp_every=8192),
+                        left=dict(heads=32, kv_heads=8, dim=128, vdim=128, scale=0.08838834764831845, softcap=50.0,
+                                  rot=dict(dims=128, base=500000.0, factor=8.0, original=8192, fast=32.0, slow=1.0, scaled=True)),
+                        right=dict(inner=8192, state=16, dt_rank=256, conv=4), scales=(1.0, 1.0),
+                        retention=dict(heads=32, dim=128, vdim=256, decay=tuple(1.0 - 2.0 ** (-5 - 7 * i / 31) for i in range(32)),
+                                       rot=dict(dims=128, base=10000.0)), ff=14336, moe=dict(ff=2048, experts=32, top=5)),
 }
 
 
@@ -137,6 +156,11 @@ def preset(name: str, **overrides):
             cfg["layers"] = sandwich_layers(*(cfg.pop(k) for k in ("order", "attention", "latent", "ff", "moe")), cfg.pop("dense", ()))
             if loop and loop["start"] < n:
                 cfg["loop"] = LoopSpec(loop["start"], min(loop["stop"], n), loop["times"])
+            return LayeredConfig(**cfg)
+        if cfg["arch"] == "Seredra":
+            keep = {i: j for i, j in cfg.pop("kv_from", {}).items() if i < len(cfg["order"]) and cfg["order"][i] == cfg["order"][j] == "a"}
+            cfg["layers"] = prenorm_layers(*(cfg.pop(k) for k in ("order", "attention", "left", "right", "scales", "retention", "ff", "moe")),
+                                           cfg.pop("dense", ()), keep)
             return LayeredConfig(**cfg)
         cfg["layers"] = hybrid_layers(*(cfg.pop(k) for k in ("order", "left", "right", "delta", "ff")), cfg.pop("weights_of", None))
         return LayeredConfig(**cfg)

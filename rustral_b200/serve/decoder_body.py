@@ -537,7 +537,7 @@ class PreNormBody:
         low = gemm(x, P.w(p + "scan.x"))
         r8, ns = up8(s.dt_rank), s.state
         dt = gemm(low[:, :r8], P.w(p + "scan.dt"), out_dtype=torch.float32)
-        rc_ops.selective_scan(x, dt, low[:, r8:r8 + ns], low[:, r8 + ns:], part("z"), A=P.w(p + "scan.A"), D=P.w(p + "scan.D"),
+        rc_ops.selective_scan(x, dt, low[:, r8:r8 + ns], low[:, r8 + ns:r8 + 2 * ns], part("z"), A=P.w(p + "scan.A"), D=P.w(p + "scan.D"),
                               dt_bias=P.w(p + "scan.dt.b"), state=state["state"], seg=sb.segments, scale=m.scales[1],
                               out=joined[:, up8(n):up8(n) + s.inner])
         return joined

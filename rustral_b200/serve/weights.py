@@ -290,9 +290,9 @@ class InferenceWeights:
             out[:, :n], out[:, up8(n):up8(n) + s.inner] = get(x + "left.o"), get(r + "o")
             t[p + "attn.out"] = out
             r8 = up8(s.dt_rank)                            # the rows behind the step sizes' are zero, and so is what they give
-            low = torch.zeros((r8 + 2 * s.state, s.inner), dtype=dt, device=dev)
+            low = torch.zeros((up8(r8 + 2 * s.state), s.inner), dtype=dt, device=dev)
             src = get(r + "x")
-            low[:s.dt_rank], low[r8:] = src[:s.dt_rank], src[s.dt_rank:]
+            low[:s.dt_rank], low[r8:r8 + 2 * s.state] = src[:s.dt_rank], src[s.dt_rank:]
             t[p + "scan.x"] = _pitched(low)
             step = torch.zeros((s.inner, r8), dtype=dt, device=dev)
             step[:, :s.dt_rank] = get(r + "dt")
