@@ -190,7 +190,7 @@ def kernels(s, T: int = 8192, L: int = 4096, B: int = 64, ctx: int = 4000, iters
             ob = 4 if kw.get("out_dtype") is f32 else 2
             time = lambda n_, k_, o_: max(2.0 * t * n_ * k_ / flops, (2.0 * (n_ * k_ + t * k_) + o_ * t * n_) / hbm)
             row(f"{name} {t}", lambda: gemm(a, b, **kw), time(n_, k_, ob), (f"product {lk} -> {ln}", lambda: gemm(la, lb), time(ln, lk, 2)))
-        product("packed projection with bias", (H + 2 * G) * dk, d, 4 * H * dk, d, bias=rnd((H + 2 * G) * dk))
+        product("packed projection with bias", (H + 2 * G) * dk, d, (H + 2 * G) * dk, d, bias=rnd((H + 2 * G) * dk))
         product("packed projection (parallel)", (H + G) * dk + 2 * inner, d, (H + 2 * G) * dk + inner + ch, d)
         product("packed projection (retention)", 2 * RH * (rn + rv), d, (H + 2 * G) * dk + inner + ch, d)
         product("step sizes, B and C", R + 2 * n, inner, hs, d)
