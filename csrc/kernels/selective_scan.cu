@@ -8,7 +8,8 @@
 // pairs.  Few segments take more lanes per channel and longer tiles: there a warp's latency counts.  Decoded
 // rows take a form without staging, whose traffic is the state, read and written once.
 //
-// fp32 operands take expf and plain arithmetic.
+// fp32 operands take correctly rounded decays (an error on one side, even of the last bit, adds up over a state's long memory) and plain
+// arithmetic.
 #include "recurrent.h"
 
 #include "recurrent.cuh"
@@ -52,7 +53,7 @@ template <int NI> struct SlState<float, NI> {
     float y = 0.f;
 #pragma unroll
     for (int i = 0; i < NI; ++i) {
-      s[i] = fmaf(expf(dt * rate[i]), s[i], u * B[i]);
+      s[i] = fmaf(__double2float_rn(exp(static_cast<double>(dt * rate[i]))), s[i], u * B[i]);
       y = fmaf(s[i], C[i], y);
     }
     return y;
