@@ -19,7 +19,7 @@ and the embedding; the embedding table is the output head.
 
 Seredra: an RMS norm with a single gain in front of every sublayer, outputs added as they are; attention with short convolutions over
 queries, keys and values, norms over whole projections, a query temperature and a logarithmic distance bias (keys and values can be
-another layer's), retention (linear attention with a fixed decay per head), or attention whose values are its keys beside a selective
+another layer's), retention (a matrix of state per head that decays at one rate), or attention whose values are its keys beside a selective
 scan; dense squared-ReLU feed-forwards or routed experts whose sigmoid scores multiply the experts' inputs.
 """
 from __future__ import annotations
@@ -107,7 +107,7 @@ class AttentionSpec:
     temp_coef: float = 0.0       # queries at position p times 1 + temp_coef * ln(floor((p + 1) / temp_every) + 1)
     temp_every: int = 0          # 0: no such factor
     log_bias: bool = False       # r1 * ln(1 + r2 * distance) is taken off the scores, with two numbers per head
-    values_are_keys: bool = False        # values: the keys as projected, in front of norm and rotation
+    values_are_keys: bool = False        # values: a copy of the unnormed, unrotated keys
     kv_from: int | None = None   # the layer whose cached keys and values are used instead of own ones
 
     def __post_init__(self):
@@ -311,8 +311,8 @@ class ParallelSpec:
 
 @dataclass(frozen=True)
 class RetentionSpec:
-    """Retention: linear attention with a fixed decay per head.  Per head a state [dim, vdim] that decays and takes up k v^T; the output,
-    normed per head, is gated."""
+    """Retention: every head multiplies its state [dim, vdim] by a constant of its own and takes up k v^T; what a query reads from it is
+    normed by itself and gated."""
     heads: int
     dim: int
     vdim: int
